@@ -24,6 +24,13 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
 ]
 
+# sources that keep the accurate forms of exp, division and square root
+ACCURATE = {"latent.cu"}
+
+
+def flags_for(src: str) -> list:
+    return [f for f in NVCC_FLAGS if f != "--use_fast_math" or os.path.basename(src) not in ACCURATE]
+
 
 def find_nvcc() -> str:
     for cand in (os.environ.get("NVCC"), shutil.which("nvcc"), "/usr/local/cuda/bin/nvcc"):
@@ -32,8 +39,8 @@ def find_nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def _digest(paths) -> str:
-    h = hashlib.sha256(" ".join(NVCC_FLAGS).encode())
+def _digest(paths, flags=NVCC_FLAGS) -> str:
+    h = hashlib.sha256(" ".join(flags).encode())
     for p in sorted(paths):
         with open(p, "rb") as f:
             h.update(f.read())
@@ -54,15 +61,12 @@ def build(verbose: bool = False, force: bool = False) -> str:
     hdrs = headers()
     jobs, objs = [], []
     for src in sources():
-        tag = _digest([src] + hdrs)
+        tag = _digest([src] + hdrs, flags_for(src))
         obj = os.path.join(OBJ_DIR, f"{os.path.basename(src)[:-3]}.{tag}.o")
         objs.append(obj)
         if force or not os.path.exists(obj):
             jobs.append((src, obj))
-    if verbose:
-        NVCC_FLAGS_V = NVCC_FLAGS + ["-Xptxas", "-v"]
-    else:
-        NVCC_FLAGS_V = NVCC_FLAGS
+    extra = ["-Xptxas", "-v"] if verbose else []
 
     def compile_one(job):
         src, obj = job
@@ -70,7 +74,7 @@ def build(verbose: bool = False, force: bool = False) -> str:
         for old in os.listdir(OBJ_DIR):
             if old.startswith(stem + ".") and old.endswith(".o"):
                 os.remove(os.path.join(OBJ_DIR, old))
-        r = subprocess.run([nvcc, *NVCC_FLAGS_V, "-c", src, "-o", obj], capture_output=True, text=True)
+        r = subprocess.run([nvcc, *flags_for(src), *extra, "-c", src, "-o", obj], capture_output=True, text=True)
         return src, r
 
     with cf.ThreadPoolExecutor(max_workers=min(8, max(1, len(jobs)))) as ex:

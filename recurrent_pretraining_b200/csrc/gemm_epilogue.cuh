@@ -18,6 +18,7 @@ enum OutMode : int {
   OUT_BF16_LSE = 10,     // head GEMM of the fused linear + cross-entropy: bf16 logits plus, per (row, column tile), the
                          // online-softmax partials (max, sum exp, sum exp * logit, sum logit^2) of the scaled logits
                          // and the target's logit; the [rows, vocab] logits never exist in fp32
+  OUT_BF16_BIAS_ACT = 11,  // bf16 store of act(acc + bias[col]), fp32 bias (may be null)
 };
 __host__ __device__ constexpr bool is_swiglu(int mode) { return mode == OUT_SWIGLU || mode == OUT_SWIGLU_SAVE; }
 
@@ -47,6 +48,9 @@ struct GemmParams {
   float* lse_tgt;
   const long long* lse_labels;
   float lse_scale;
+  // OUT_BF16_BIAS_ACT
+  const float* bias;   // [N] or null
+  int act;             // 0: none, 1: relu^2
 };
 
 // Linear tile index -> (m tile, n tile), grouped: GROUP consecutive m tiles are walked across all n tiles before the
@@ -123,6 +127,30 @@ __device__ __forceinline__ void rope_chunk(const GemmParams& p, int row, int col
           if (d >= p.rope_D) d -= p.rope_D;
         }
       }
+    }
+  }
+}
+
+// act(f + bias) on up to 32 accumulator columns starting at global column ``col`` (columns at or beyond p.N are left alone).
+__device__ __forceinline__ void bias_act_chunk(const GemmParams& p, int col, int width, float (&f)[32]) {
+  if (p.bias) {
+    if (col + width <= p.N && width == 32 && ((reinterpret_cast<uintptr_t>(p.bias + col) & 15) == 0)) {
+#pragma unroll
+      for (int q = 0; q < 8; ++q) {
+        const float4 b = __ldg(reinterpret_cast<const float4*>(p.bias + col) + q);
+        f[4 * q] += b.x; f[4 * q + 1] += b.y; f[4 * q + 2] += b.z; f[4 * q + 3] += b.w;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (i < width && col + i < p.N) f[i] += __ldg(p.bias + col + i);
+    }
+  }
+  if (p.act == 1) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float r = fmaxf(f[i], 0.f);
+      f[i] = r * r;
     }
   }
 }
@@ -268,7 +296,8 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tadd
             }
         }
       }
-    } else if constexpr (MODE == OUT_BF16 || MODE == OUT_BF16_RESID || MODE == OUT_BF16_ROPE || MODE == OUT_BF16_LSE) {
+    } else if constexpr (MODE == OUT_BF16 || MODE == OUT_BF16_RESID || MODE == OUT_BF16_ROPE || MODE == OUT_BF16_LSE ||
+                         MODE == OUT_BF16_BIAS_ACT) {
       uint32_t v[32];
       __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(row) * p.ldc + col;
       const bool vec = active && nvalid == width && ((reinterpret_cast<uintptr_t>(crow) & 15) == 0);
@@ -320,6 +349,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tadd
         }
       }
       if constexpr (MODE == OUT_BF16_ROPE) rope_chunk(p, row, col, width, f);
+      if constexpr (MODE == OUT_BF16_BIAS_ACT) bias_act_chunk(p, col, width, f);
       if constexpr (MODE == OUT_BF16_LSE) {
         float cm = -INFINITY;
 #pragma unroll
@@ -528,14 +558,18 @@ __device__ __forceinline__ void stage_row_bf16x64(uint8_t* tile, int lane, const
   }
 }
 
-// QKV projection: bias + rotation in registers, then the staged bf16 store (64 columns per box; the 48-column rest of a
-// 240-wide tile by per-thread stores).
-template <int BN>
-__device__ __forceinline__ void epilogue_tile_tma_rope(const GemmParams& p, const CUtensorMap* tmC, uint32_t taddr, int row0,
+// A column-wise epilogue in registers (MODE: bias + rotation of the QKV projection, or bias + activation), then the staged
+// bf16 store (64 columns per box; the 48-column rest of a 240-wide tile by per-thread stores).
+template <int BN, int MODE>
+__device__ __forceinline__ void epilogue_tile_tma_map(const GemmParams& p, const CUtensorMap* tmC, uint32_t taddr, int row0,
                                                        int n0, uint8_t* stage, int lane, int& buf) {
   constexpr int FULL = BN / 64 * 64;
   const int row = row0 + lane;
   const bool row_ok = row < p.M;
+  auto apply = [&](int col, int width, float (&f)[32]) {
+    if constexpr (MODE == OUT_BF16_ROPE) rope_chunk(p, row, col, width, f);
+    else bias_act_chunk(p, col, width, f);
+  };
 #pragma unroll 1
   for (int c0 = 0; c0 < FULL; c0 += 64) {
     uint32_t packed[2][16];
@@ -548,7 +582,7 @@ __device__ __forceinline__ void epilogue_tile_tma_rope(const GemmParams& p, cons
 #pragma unroll
       for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
       const int col = n0 + c0 + 32 * hh;
-      if (row_ok && col < p.N) rope_chunk(p, row, col, 32, f);
+      if (row_ok && col < p.N) apply(col, 32, f);
 #pragma unroll
       for (int i = 0; i < 16; ++i) packed[hh][i] = pack_bf16x2(f[2 * i], f[2 * i + 1]);
     }
@@ -579,7 +613,7 @@ __device__ __forceinline__ void epilogue_tile_tma_rope(const GemmParams& p, cons
       for (int i = 0; i < 16; ++i) f[i] = __uint_as_float(v[i]);
 #pragma unroll
       for (int i = 16; i < 32; ++i) f[i] = 0.f;
-      rope_chunk(p, row, col, 16, f);
+      apply(col, 16, f);
       __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(row) * p.ldc + col;
       const int nvalid = min(16, p.N - col);
       if (nvalid == 16 && ((reinterpret_cast<uintptr_t>(crow) & 15) == 0)) {

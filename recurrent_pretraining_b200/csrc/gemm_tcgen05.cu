@@ -382,6 +382,11 @@ B200_API void b200_gemm_set_lse(void* part, float* tgt, const long long* labels,
   g_lse = {part, tgt, labels, scale};
 }
 
+// Arguments of the next OUT_BF16_BIAS_ACT call (same convention).
+struct BiasArgs { const float* bias; int act; };
+static thread_local BiasArgs g_bias = {nullptr, 0};
+B200_API void b200_gemm_set_bias(const float* bias, int act) { g_bias = {bias, act}; }
+
 B200_API int b200_gemm(const void* A, const void* A2, const void* B, void* C, const void* resid, int M, int N,
                        int K1, int K2, int lda, int lda2, int ldb, int ldc, int ld_resid, int a_mn, int b_mn,
                        int out_mode, int bn, int max_ctas, void* stream, int* err) {
@@ -406,6 +411,7 @@ B200_API int b200_gemm(const void* A, const void* A2, const void* B, void* C, co
   p.rope_S = g_rope.S; p.rope_D = g_rope.D; p.rope_width = g_rope.width;
   p.lse_part = reinterpret_cast<float4*>(g_lse.part); p.lse_tgt = g_lse.tgt; p.lse_labels = g_lse.labels;
   p.lse_scale = g_lse.scale;
+  p.bias = g_bias.bias; p.act = g_bias.act;
   if (out_mode == OUT_BF16_LSE && (!p.lse_part || !p.lse_tgt || !p.lse_labels || a_mn || b_mn || bn != 256)) return -27;
   if (out_mode == OUT_BF16_ROPE && (!p.rope_cos || p.rope_D <= 0 || (p.rope_D & 1) || (p.rope_width & 1))) return -25;
   if (g_use_2cta && M >= 256 && (bn == 256 || bn == 240 || (is_swiglu(out_mode) && !a_mn && !b_mn))) {
@@ -457,6 +463,12 @@ B200_API int b200_gemm(const void* A, const void* A2, const void* B, void* C, co
     if (bn == 240) return launch<240, false, false, OUT_BF16_ROPE>(ta, ta2, tb, p, st, max_ctas);
     if (bn == 128) return launch<128, false, false, OUT_BF16_ROPE>(ta, ta2, tb, p, st, max_ctas);
     return launch<256, false, false, OUT_BF16_ROPE>(ta, ta2, tb, p, st, max_ctas);
+  }
+  if (out_mode == OUT_BF16_BIAS_ACT) {
+    if (a_mn || b_mn) return -24;
+    if (bn == 240) return launch<240, false, false, OUT_BF16_BIAS_ACT>(ta, ta2, tb, p, st, max_ctas);
+    if (bn == 128) return launch<128, false, false, OUT_BF16_BIAS_ACT>(ta, ta2, tb, p, st, max_ctas);
+    return launch<256, false, false, OUT_BF16_BIAS_ACT>(ta, ta2, tb, p, st, max_ctas);
   }
   if (!a_mn && !b_mn) {
     if (bn == 256) { DISPATCH_MODE(256, false, false) }

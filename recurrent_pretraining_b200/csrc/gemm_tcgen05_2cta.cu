@@ -348,8 +348,8 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
     uint32_t tcount = 0;
     constexpr bool F32_MODE = MODE == OUT_F32 || MODE == OUT_F32_ACC;
     // modes with a shared-memory staged epilogue
-    constexpr bool STAGED = (F32_MODE || MODE == OUT_BF16 || MODE == OUT_BF16_ROPE || MODE == OUT_SWIGLU ||
-                             MODE == OUT_SWIGLU_SAVE || MODE == OUT_DSWIGLU) && !AG;
+    constexpr bool STAGED = (F32_MODE || MODE == OUT_BF16 || MODE == OUT_BF16_ROPE ||
+                             MODE == OUT_BF16_BIAS_ACT || MODE == OUT_SWIGLU || MODE == OUT_SWIGLU_SAVE || MODE == OUT_DSWIGLU) && !AG;
     uint8_t* c_stage = smem + L::C_STAGE_OFFSET + quad * 8192;   // only backed by memory in the fp32 output modes
     int c_buf = 0;
     for (int tile = cluster_id; tile < num_tiles; tile += num_clusters, ++tcount) {
@@ -367,8 +367,8 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
         else epilogue_tile<BN_OUT, MODE>(p, taddr, m0 + quad * 32 + lane, n0);
       } else if constexpr (STAGED) {
         if (!p.tma_c) epilogue_tile<BN_OUT, MODE>(p, taddr, m0 + quad * 32 + lane, n0);
-        else if constexpr (MODE == OUT_BF16_ROPE)
-          epilogue_tile_tma_rope<BN_OUT>(p, &tmC, taddr, m0 + quad * 32, n0, c_stage, lane, c_buf);
+        else if constexpr (MODE == OUT_BF16_ROPE || MODE == OUT_BF16_BIAS_ACT)
+          epilogue_tile_tma_map<BN_OUT, MODE>(p, &tmC, taddr, m0 + quad * 32, n0, c_stage, lane, c_buf);
         else if constexpr (MODE == OUT_SWIGLU)
           epilogue_tile_tma_swiglu<BN_OUT>(p, &tmC, taddr, m0 + quad * 32, n0, c_stage, lane, c_buf);
         else if constexpr (MODE == OUT_SWIGLU_SAVE)
@@ -406,7 +406,7 @@ static int launch2(const CUtensorMap& ta, const CUtensorMap& ta2, const CUtensor
   using L = Smem2<BN>;
   auto kern = gemm2_kernel<BN, A_MN, B_MN, MODE, AG>;
   constexpr int SMEM = ((MODE == OUT_F32 || MODE == OUT_F32_ACC || MODE == OUT_BF16 || MODE == OUT_BF16_ROPE ||
-                         MODE == OUT_SWIGLU || MODE == OUT_SWIGLU_SAVE || MODE == OUT_DSWIGLU) && !AG)
+                         MODE == OUT_BF16_BIAS_ACT || MODE == OUT_SWIGLU || MODE == OUT_SWIGLU_SAVE || MODE == OUT_DSWIGLU) && !AG)
                             ? L::TOTAL_F32 : L::TOTAL;
   static int max_clusters = -1;
   if (max_clusters < 0) {
@@ -468,7 +468,8 @@ int gemm_2cta_dispatch(const void* A, const void* A2, const void* B, const GemmP
     pc.tma_c = 1;
   }
   static const bool tma_c16_on = [] { const char* e = getenv("B200_GEMM_TMA_C16"); return !(e && e[0] == '0'); }();
-  if ((out_mode == OUT_BF16 || out_mode == OUT_BF16_ROPE || out_mode == OUT_SWIGLU) && tma_c_on && tma_c16_on &&
+  if ((out_mode == OUT_BF16 || out_mode == OUT_BF16_ROPE || out_mode == OUT_BF16_BIAS_ACT ||
+       out_mode == OUT_SWIGLU) && tma_c_on && tma_c16_on &&
       make_tmap_2d_bf16(&tc, p.C, p.M, p.N, p.ldc, 32, 64) == 0) {
     tcp = &tc;
     pc.tma_c = 1;
@@ -517,6 +518,11 @@ int gemm_2cta_dispatch(const void* A, const void* A2, const void* B, const GemmP
     if (a_mn || b_mn) return -100;
     if (bn == 240) return launch2<240, false, false, OUT_BF16_ROPE>(ta, ta2, tb, pc, st, max_ctas, nullptr, tcp);
     return launch2<256, false, false, OUT_BF16_ROPE>(ta, ta2, tb, pc, st, max_ctas, nullptr, tcp);
+  }
+  if (out_mode == OUT_BF16_BIAS_ACT) {
+    if (a_mn || b_mn) return -100;
+    if (bn == 240) return launch2<240, false, false, OUT_BF16_BIAS_ACT>(ta, ta2, tb, pc, st, max_ctas, nullptr, tcp);
+    return launch2<256, false, false, OUT_BF16_BIAS_ACT>(ta, ta2, tb, pc, st, max_ctas, nullptr, tcp);
   }
   if (!a_mn && !b_mn) {
     if (bn == 256) { DISPATCH2(256, false, false) }

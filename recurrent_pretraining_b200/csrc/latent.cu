@@ -1,0 +1,716 @@
+// Kernels of the layered decoder models (latent attention over a per-token latent, fp32 residual stream) other than
+// the tensor-core attention tiles:
+//   * embed_resid      : token embedding into the fp32 residual stream and its operand-precision copy
+//   * latent_prep      : one packed projection row [q | gate | latent]: rotation of the q parts, latent norm, rotation of
+//                        the shared key part, append to the ring cache and to the step's key stream
+//   * latent_absorb    : the decode form of the same step; q is also carried through the key up-projection, so that the
+//                        scores are taken against the cached latents directly
+//   * window_attention : softmax over the keys of a sliding window, one query row per (token, head); generic in every
+//                        size, 32-bit throughout (step streams and ring caches)
+//   * latent_expand    : merge of the decode attention's key splits, value up-projection, output gate
+//   * rms_residual     : x += mult * rmsnorm(a + bias) * w on the fp32 residual stream
+//   * bias_act, rmsnorm_rows, gather_rows, sgemm_nt (true fp32 matrix product)
+// Storage types: bf16 (serving) or fp32; arithmetic is fp32.  This file is built without fast-math approximations.
+#include "common.cuh"
+
+namespace b200 {
+
+template <typename T> __device__ __forceinline__ float ldf(const T* p);
+template <> __device__ __forceinline__ float ldf<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ldf<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+template <typename T> __device__ __forceinline__ void stf(T* p, float v);
+template <> __device__ __forceinline__ void stf<float>(float* p, float v) { *p = v; }
+template <> __device__ __forceinline__ void stf<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// two neighbouring elements (address aligned to the pair)
+template <typename T> __device__ __forceinline__ float2 ld2(const T* p);
+template <> __device__ __forceinline__ float2 ld2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 ld2<__nv_bfloat16>(const __nv_bfloat16* p) {
+  return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+}
+// eight neighbouring elements (16-byte aligned rows)
+__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 q = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 f = unpack_bf16x2(w[j]);
+    v[2 * j] = f.x;
+    v[2 * j + 1] = f.y;
+  }
+}
+__device__ __forceinline__ void st8(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                            pack_bf16x2(v[6], v[7]));
+}
+__device__ __forceinline__ void clear8(float* p) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(0.f, 0.f, 0.f, 0.f);
+  reinterpret_cast<float4*>(p)[1] = make_float4(0.f, 0.f, 0.f, 0.f);
+}
+__device__ __forceinline__ void clear8(__nv_bfloat16*) {}
+
+template <int THREADS>
+__device__ __forceinline__ float block_total(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();   // the previous use of `red` is over
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < THREADS / 32; ++i) t += red[i];
+  return t;
+}
+__device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
+
+// ------------------------------------------------------------------------------------------------ embedding
+template <typename T>
+__global__ void __launch_bounds__(128)
+embed_resid_kernel(const long long* __restrict__ tok, const T* __restrict__ table, float* __restrict__ x,
+                   T* __restrict__ xb, int E, int ld_table, int ld_xb, long long vocab, int* err) {
+  const size_t t = blockIdx.x;
+  long long id = tok[t];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0) atomicCAS(err, 0, ERR_BAD_INDEX);
+  const T* src = table + static_cast<size_t>(ok ? id : 0) * ld_table;
+  for (int i = threadIdx.x; i < E; i += 128) {
+    const float v = ok ? ldf(src + i) : 0.f;
+    x[t * E + i] = v;
+    stf(xb + t * ld_xb + i, v);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ latent rows
+struct LatentRow {
+  // projection row: q at column 0 (head by head [dim | rot]), gate at off_g, latent [rank | rot] at off_d
+  int ld_in, off_g, off_d;
+  int H, dim, rot, rank, vdim;
+  int rank_pad, ld_lat;           // latent row: [c (rank) | 0 .. rank_pad | rotated key part (rot) | 0 .. ld_lat]
+  int cap;                        // ring slots of one sequence row
+  int own;                        // this layer has a latent projection of its own
+  float eps;
+  const float* norm_w;            // [rank]
+  const float* cosT;              // [positions, rot / 2], scaled
+  const float* sinT;
+  const int* pos;                 // [T]
+  const int* row;                 // [T] cache row
+};
+
+// latent part of one token -> cache row `dst_cache` (or null) and stream row `dst_stream` (or null)
+template <typename TI, typename T, int THREADS>
+__device__ __forceinline__ void latent_append(const LatentRow& L, const TI* in, int p, T* dst_cache, T* dst_stream, float* red) {
+  const TI* d = in + L.off_d;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < L.rank; i += THREADS) {
+    const float v = ldf(d + i);
+    ss += v * v;
+  }
+  const float rstd = 1.f / sqrtf(block_total<THREADS>(ss, red) / static_cast<float>(L.rank) + L.eps);
+  for (int i = threadIdx.x; i < L.ld_lat; i += THREADS) {
+    float v = 0.f;
+    if (i < L.rank) {
+      v = ldf(d + i) * rstd * L.norm_w[i];
+    } else if (i >= L.rank_pad && i < L.rank_pad + L.rot) {
+      const int j = i - L.rank_pad, pr = j >> 1;
+      const float u = ldf(d + L.rank + (j & ~1)), w = ldf(d + L.rank + (j | 1));
+      const float c = L.cosT[static_cast<size_t>(p) * (L.rot >> 1) + pr], s = L.sinT[static_cast<size_t>(p) * (L.rot >> 1) + pr];
+      v = (j & 1) ? w * c + u * s : u * c - w * s;
+    }
+    if (dst_cache) stf(dst_cache + i, v);
+    if (dst_stream) stf(dst_stream + i, v);
+  }
+}
+
+// One CTA per token of a packed step.  Rotates the q parts in place; appends the latent row to the stream at sidx[t] and,
+// for the last `cap` tokens of the sequence's portion (end[t] = position after its last token), to the ring (if there is one).
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_prep_kernel(T* __restrict__ in, LatentRow L, const int* __restrict__ sidx, const int* __restrict__ end,
+                   T* __restrict__ cache, T* __restrict__ stream) {
+  __shared__ float red[4];
+  const size_t t = blockIdx.x;
+  T* r = in + t * L.ld_in;
+  const int p = L.pos[t], half = L.rot >> 1, hd = L.dim + L.rot;
+  const float* ct = L.cosT + static_cast<size_t>(p) * half;
+  const float* st = L.sinT + static_cast<size_t>(p) * half;
+  for (int i = threadIdx.x; i < L.H * half; i += 128) {
+    const int h = i / half, j = i - h * half;
+    T* q = r + h * hd + L.dim + 2 * j;
+    const float u = ldf(q), v = ldf(q + 1), c = ct[j], s = st[j];
+    stf(q, u * c - v * s);
+    stf(q + 1, v * c + u * s);
+  }
+  if (L.own) {
+    T* dst = cache && p >= end[t] - L.cap ? cache + (static_cast<size_t>(L.row[t]) * L.cap + p % L.cap) * L.ld_lat : nullptr;
+    latent_append<T, T, 128>(L, r, p, dst, stream + static_cast<size_t>(sidx[t]) * L.ld_lat, red);
+  }
+}
+
+// Decode: in [B, ld_in] (fp32 accumulator or operand precision, not modified).  CTAs [0, B): row b's latent append and the
+// rotated / padding columns of qlat [B, H, ld_lat].  The others: (head, 128 latent columns, 8 rows) tiles of
+// qlat[b, h, r] = sum_d W_uk[h * dim + d, r] q[b, h, d].
+constexpr int ABS_ROWS = 8, ABS_COLS = 128;
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256)
+latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict__ w_uk, int ldw, T* __restrict__ cache,
+                     T* __restrict__ qlat, int B) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float sm[];
+  const int hd = L.dim + L.rot;
+  if (static_cast<int>(blockIdx.x) < B) {
+    const int b = blockIdx.x, p = L.pos[b], half = L.rot >> 1;
+    const TI* r = in + static_cast<size_t>(b) * L.ld_in;
+    const float* ct = L.cosT + static_cast<size_t>(p) * half;
+    const float* st = L.sinT + static_cast<size_t>(p) * half;
+    const int tail = L.ld_lat - L.rank;      // columns after the latent: padding and rotation
+    for (int i = threadIdx.x; i < L.H * tail; i += 256) {
+      const int h = i / tail, c = L.rank + (i - h * tail), j = c - L.rank_pad;
+      float v = 0.f;
+      if (j >= 0 && j < L.rot) {
+        const TI* q = r + h * hd + L.dim;
+        const float u = ldf(q + (j & ~1)), w = ldf(q + (j | 1)), cs = ct[j >> 1], sn = st[j >> 1];
+        v = (j & 1) ? w * cs + u * sn : u * cs - w * sn;
+      }
+      stf(qlat + (static_cast<size_t>(b) * L.H + h) * L.ld_lat + c, v);
+    }
+    if (L.own)
+      latent_append<TI, T, 256>(L, r, p, cache + (static_cast<size_t>(L.row[b]) * L.cap + p % L.cap) * L.ld_lat,
+                                static_cast<T*>(nullptr), sm);
+    return;
+  }
+  const int cols = (L.rank + ABS_COLS - 1) / ABS_COLS;
+  int id = blockIdx.x - B;
+  const int rc = id % cols;
+  id /= cols;
+  const int h = id % L.H, b0 = (id / L.H) * ABS_ROWS;
+  const int nb = min(ABS_ROWS, B - b0);
+  float* qs = sm;                                  // [ABS_ROWS][dim]
+  float* part = sm + ABS_ROWS * L.dim;             // [4][ABS_ROWS][ABS_COLS]
+  for (int i = threadIdx.x; i < ABS_ROWS * L.dim; i += 256) {
+    const int b = i / L.dim, d = i - b * L.dim;
+    qs[i] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
+  }
+  __syncthreads();
+  const int tx = threadIdx.x & 63, grp = threadIdx.x >> 6;
+  const int r = rc * ABS_COLS + 2 * tx;
+  float acc[ABS_ROWS][2];
+#pragma unroll
+  for (int b = 0; b < ABS_ROWS; ++b) acc[b][0] = acc[b][1] = 0.f;
+  if (r < L.rank) {                                // weight rows are padded: column r + 1 exists
+    const T* wp = w_uk + static_cast<size_t>(h) * L.dim * ldw + r;
+#pragma unroll 4
+    for (int d = grp; d < L.dim; d += 4) {
+      const float2 w = ld2(wp + static_cast<size_t>(d) * ldw);
+#pragma unroll
+      for (int b = 0; b < ABS_ROWS; ++b) {
+        const float q = qs[b * L.dim + d];
+        acc[b][0] += q * w.x;
+        acc[b][1] += q * w.y;
+      }
+    }
+  }
+#pragma unroll
+  for (int b = 0; b < ABS_ROWS; ++b) {
+    part[(grp * ABS_ROWS + b) * ABS_COLS + 2 * tx] = acc[b][0];
+    part[(grp * ABS_ROWS + b) * ABS_COLS + 2 * tx + 1] = acc[b][1];
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nb * ABS_COLS; i += 256) {
+    const int b = i / ABS_COLS, c = i - b * ABS_COLS;
+    if (rc * ABS_COLS + c >= L.rank) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int g = 0; g < 4; ++g) v += part[(g * ABS_ROWS + b) * ABS_COLS + c];
+    stf(qlat + (static_cast<size_t>(b0 + b) * L.H + h) * L.ld_lat + rc * ABS_COLS + c, v);
+  }
+}
+
+// dst[dst_idx[i], :] = src[src_idx[i], :], rows of `bytes` (a multiple of 16) bytes
+__global__ void __launch_bounds__(128)
+gather_rows_kernel(const uint4* __restrict__ src, const int* __restrict__ src_idx, uint4* __restrict__ dst,
+                   const int* __restrict__ dst_idx, int vec) {
+  const uint4* s = src + static_cast<size_t>(src_idx[blockIdx.x]) * vec;
+  uint4* d = dst + static_cast<size_t>(dst_idx[blockIdx.x]) * vec;
+  for (int i = threadIdx.x; i < vec; i += 128) d[i] = s[i];
+}
+
+// ------------------------------------------------------------------------------------------------ attention (generic)
+struct WindowAttn {
+  // score(t, h, key) = q[t, h, :d1] . k1[key, h, :] + q[t, h, d1:] . k2[key, :]
+  int H, d1, d2, vdim, window, splits;
+  float scale;
+  int q_stride, q_head;           // elements
+  int k1_stride, k1_head, k2_stride, v_stride, v_head;
+  const int* sidx;                // stream form: key index of the query itself ...
+  const int* kbase;               // ... and of the first key of its sequence
+  const int* pos;                 // ring form: position of the query ...
+  const int* row;                 // ... and its cache row (key of position p: row * cap + p % cap)
+  int cap;
+  // stream form: normalised, gated output; ring form (splits > 0 partials): unnormalised fp32 partials
+  int gate_ld, out_ld;
+  float* part_o;                  // [T, H, splits, vdim]
+  float* part_ml;                 // [T, H, splits, 2] (max in natural-log units, sum)
+};
+
+// CTA of four warps per (token, head, key split); a warp takes 32 keys at a time: one key per lane for the scores, one
+// value column per lane for the weighted sum.
+template <typename T>
+__global__ void __launch_bounds__(128)
+window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* __restrict__ k2, const T* __restrict__ v,
+                   const T* __restrict__ gate, T* __restrict__ out, const WindowAttn A) {
+  extern __shared__ float sm[];
+  const int dk = A.d1 + A.d2;
+  float* qs = sm;                                   // [dk]
+  float* ps = sm + dk;                              // [4][32]
+  float* os = ps + 128;                             // [4][vdim]
+  float* ml = os + 4 * A.vdim;                      // [4][2]
+  const int t = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* qp = q + static_cast<size_t>(t) * A.q_stride + static_cast<size_t>(h) * A.q_head;
+  for (int i = threadIdx.x; i < dk; i += 128) qs[i] = ldf(qp + i);
+  for (int i = threadIdx.x; i < 4 * A.vdim; i += 128) os[i] = 0.f;
+  __syncthreads();
+  const bool ring = A.pos != nullptr;
+  const int last = ring ? A.pos[t] : A.sidx[t];
+  const int first = max(ring ? 0 : A.kbase[t], last - A.window + 1);
+  const size_t ring0 = ring ? static_cast<size_t>(A.row[t]) * A.cap : 0;
+  const int nchunk = (last - first) / 32 + 1;
+  float m = -INFINITY, l = 0.f;
+  float* op = os + warp * A.vdim;
+  float* pp = ps + warp * 32;
+  for (int c = split * 4 + warp; c < nchunk; c += 4 * A.splits) {
+    const int j0 = first + c * 32, j = j0 + lane, n = min(32, last - j0 + 1);
+    float s = -INFINITY;
+    if (j <= last) {
+      const size_t key = ring ? ring0 + j % A.cap : static_cast<size_t>(j);
+      const T* a = k1 + key * A.k1_stride + static_cast<size_t>(h) * A.k1_head;
+      s = 0.f;
+      for (int i = 0; i < A.d1; ++i) s += qs[i] * ldf(a + i);
+      if (A.d2) {
+        const T* b = k2 + key * A.k2_stride;
+        for (int i = 0; i < A.d2; ++i) s += qs[A.d1 + i] * ldf(b + i);
+      }
+      s *= A.scale;
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float p = expf(s - mn), alpha = expf(m - mn);
+    l = l * alpha + warp_sum(p);
+    m = mn;
+    pp[lane] = p;
+    __syncwarp();
+    for (int d = lane; d < A.vdim; d += 32) {
+      float o = op[d] * alpha;
+      for (int k = 0; k < n; ++k) {
+        const size_t key = ring ? ring0 + (j0 + k) % A.cap : static_cast<size_t>(j0 + k);
+        o += pp[k] * ldf(v + key * A.v_stride + static_cast<size_t>(h) * A.v_head + d);
+      }
+      op[d] = o;
+    }
+    __syncwarp();
+  }
+  if (lane == 0) { ml[2 * warp] = m; ml[2 * warp + 1] = l; }
+  __syncthreads();
+  float mm = -INFINITY, ll = 0.f, wgt[4];
+#pragma unroll
+  for (int w = 0; w < 4; ++w) mm = fmaxf(mm, ml[2 * w]);
+#pragma unroll
+  for (int w = 0; w < 4; ++w) {
+    wgt[w] = ml[2 * w] == -INFINITY ? 0.f : expf(ml[2 * w] - mm);
+    ll += wgt[w] * ml[2 * w + 1];
+  }
+  const float inv = 1.f / ll;
+  for (int d = threadIdx.x; d < A.vdim; d += 128) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) o += wgt[w] * os[w * A.vdim + d];
+    if (A.part_o) {
+      const size_t pi = (static_cast<size_t>(t) * A.H + h) * A.splits + split;
+      A.part_o[pi * A.vdim + d] = o;
+      if (d == 0) { A.part_ml[2 * pi] = mm; A.part_ml[2 * pi + 1] = ll; }
+    } else {
+      const float g = sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + h * A.vdim + d));
+      stf(out + static_cast<size_t>(t) * A.out_ld + h * A.vdim + d, o * inv * g);
+    }
+  }
+}
+
+// out[b, h * vdim + v] = sigmoid(gate) * sum_r W_uv[h * vdim + v, r] o[b, h, r], o = merged key splits.
+// CTA: (head, 32 values, 8 rows).
+constexpr int EXP_ROWS = 8, EXP_COLS = 32;
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256)
+latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+                     const T* __restrict__ w_uv, int ldw, const TI* __restrict__ gate, int gate_ld, T* __restrict__ out,
+                     int out_ld, int B, int H, int rank, int vdim) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float os[];                    // [EXP_ROWS][rank_even]
+  __shared__ float wgt[EXP_ROWS][33];
+  const int h = blockIdx.x, v0 = blockIdx.y * EXP_COLS, b0 = blockIdx.z * EXP_ROWS;
+  const int nb = min(EXP_ROWS, B - b0), rs = (rank + 1) & ~1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp < nb) {                                 // warp b: weights of the splits of row b (splits <= 32)
+    const size_t base = (static_cast<size_t>(b0 + warp) * H + h) * splits;
+    const float2 e = lane < splits ? *reinterpret_cast<const float2*>(part_ml + (base + lane) * 2) : make_float2(-INFINITY, 0.f);
+    const float mm = warp_max(e.x);
+    const float a = e.x == -INFINITY ? 0.f : expf(e.x - mm);
+    const float ll = warp_sum(a * e.y);
+    wgt[warp][lane] = a / ll;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < EXP_ROWS * rs; i += 256) {
+    const int b = i / rs, r = i - b * rs;
+    float o = 0.f;
+    if (b < nb && r < rank) {
+      const float* p = part_o + (static_cast<size_t>(b0 + b) * H + h) * splits * rank + r;
+      for (int s = 0; s < splits; ++s) {
+        const float w = wgt[b][s];
+        if (w != 0.f) o += w * p[static_cast<size_t>(s) * rank];   // an empty split's partial is not initialised
+      }
+    }
+    os[i] = o;
+  }
+  __syncthreads();
+#pragma unroll 1
+  for (int k = 0; k < EXP_COLS / 8; ++k) {
+    const int v = v0 + warp * (EXP_COLS / 8) + k;
+    if (v >= vdim) break;
+    const T* wr = w_uv + (static_cast<size_t>(h) * vdim + v) * ldw;
+    float acc[EXP_ROWS];
+#pragma unroll
+    for (int b = 0; b < EXP_ROWS; ++b) acc[b] = 0.f;
+#pragma unroll 4
+    for (int r = 2 * lane; r < rank; r += 64) {    // weight rows are padded: column r + 1 exists (times a zero)
+      const float2 w = ld2(wr + r);
+#pragma unroll
+      for (int b = 0; b < EXP_ROWS; ++b) {
+        const float2 o = *reinterpret_cast<const float2*>(os + b * rs + r);
+        acc[b] += w.x * o.x + w.y * o.y;
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < EXP_ROWS; ++b) {
+      const float s = warp_sum(acc[b]);
+      if (lane == b && b < nb) {
+        const float g = sigmoid_f(ldf(gate + static_cast<size_t>(b0 + b) * gate_ld + h * vdim + v));
+        stf(out + static_cast<size_t>(b0 + b) * out_ld + h * vdim + v, s * g);
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ residual
+// x += mult * (s / rms(s)) * w with s = a + bias; xb = x in operand precision.  One CTA per row.  `clear`: a is the
+// accumulator of a stream-K GEMM and is handed back zeroed; zero[row, :nzero] is a second accumulator (consumed by earlier
+// kernels) that is re-armed here.
+template <typename TI, typename T, int NV>
+__global__ void __launch_bounds__(256)
+rms_residual_vec_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __restrict__ bias, const float* __restrict__ w,
+                        float* __restrict__ x, T* __restrict__ xb, int ld_xb, int E, float eps, float mult,
+                        float* __restrict__ zero, int nzero) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[8];
+  const size_t row = blockIdx.x;
+  const int nvec = E >> 3;
+  TI* ar = a + row * ld_a;
+  float s[NV][8], xv[NV][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nvec) {
+      ld8(ar + 8 * i, s[k]);
+      ld8(x + row * E + 8 * i, xv[k]);
+      if (bias) {
+        float b[8];
+        ld8(bias + 8 * i, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s[k][j] += b[j];
+      }
+      if (clear) clear8(ar + 8 * i);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += s[k][j] * s[k][j];
+    }
+  }
+  for (int i = threadIdx.x; i < nzero; i += 256) zero[row * nzero + i] = 0.f;
+  const float r = mult / sqrtf(block_total<256>(ss, red) / static_cast<float>(E) + eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nvec) {
+      float wv[8];
+      ld8(w + 8 * i, wv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) xv[k][j] += s[k][j] * r * wv[j];
+      st8(x + row * E + 8 * i, xv[k]);
+      st8(xb + row * ld_xb + 8 * i, xv[k]);
+    }
+  }
+}
+
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256)
+rms_residual_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __restrict__ bias, const float* __restrict__ w,
+                    float* __restrict__ x, T* __restrict__ xb, int ld_xb, int E, float eps, float mult,
+                    float* __restrict__ zero, int nzero) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[8];
+  const size_t row = blockIdx.x;
+  TI* ar = a + row * ld_a;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < E; i += 256) {
+    const float s = ldf(ar + i) + (bias ? bias[i] : 0.f);
+    ss += s * s;
+  }
+  for (int i = threadIdx.x; i < nzero; i += 256) zero[row * nzero + i] = 0.f;
+  const float r = mult / sqrtf(block_total<256>(ss, red) / static_cast<float>(E) + eps);
+  for (int i = threadIdx.x; i < E; i += 256) {
+    const float s = ldf(ar + i) + (bias ? bias[i] : 0.f);
+    if (clear) stf(ar + i, 0.f);
+    const float v = x[row * E + i] + s * r * w[i];
+    x[row * E + i] = v;
+    stf(xb + row * ld_xb + i, v);
+  }
+}
+
+// y[i] = rmsnorm(x[idx[i]]) * w in operand precision
+template <typename T>
+__global__ void __launch_bounds__(256)
+rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ idx, const float* __restrict__ w, T* __restrict__ y,
+                    int ld_y, int E, float eps) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[8];
+  const float* xr = x + static_cast<size_t>(idx ? idx[blockIdx.x] : static_cast<int>(blockIdx.x)) * E;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < E; i += 256) ss += xr[i] * xr[i];
+  const float r = 1.f / sqrtf(block_total<256>(ss, red) / static_cast<float>(E) + eps);
+  for (int i = threadIdx.x; i < E; i += 256) stf(y + static_cast<size_t>(blockIdx.x) * ld_y + i, xr[i] * r * w[i]);
+}
+
+// y = act(a + bias); act 0: none, 1: relu^2.  `clear` as above.
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256)
+bias_act_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __restrict__ bias, T* __restrict__ y, int ld_y, int N, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.y;
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i >= N) return;
+  float v = ldf(a + row * ld_a + i) + (bias ? bias[i] : 0.f);
+  if (clear) stf(a + row * ld_a + i, 0.f);
+  if (act == 1) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  stf(y + row * ld_y + i, v);
+}
+
+// ------------------------------------------------------------------------------------------------ fp32 matrix product
+// C[M, N] = act(A[M, K] B[N, K]^T + bias) in fp32 (FMA pipe): 64 x 64 tile per 256 threads, 4 x 4 per thread.
+constexpr int SG = 64, SGK = 16;
+__global__ void __launch_bounds__(256)
+sgemm_nt_kernel(const float* __restrict__ A, const float* __restrict__ B, const float* __restrict__ bias, float* __restrict__ C,
+                int M, int N, int K, int lda, int ldb, int ldc, int act) {
+  __shared__ float as[SGK][SG + 4], bs[SGK][SG + 4];
+  const int m0 = blockIdx.x * SG, n0 = blockIdx.y * SG;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += SGK) {
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = threadIdx.x + u * 256, r = i >> 4, c = i & 15;
+      as[c][r] = (m0 + r < M && k0 + c < K) ? A[static_cast<size_t>(m0 + r) * lda + k0 + c] : 0.f;
+      bs[c][r] = (n0 + r < N && k0 + c < K) ? B[static_cast<size_t>(n0 + r) * ldb + k0 + c] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < SGK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&as[k][4 * ty]), b = *reinterpret_cast<const float4*>(&bs[k][4 * tx]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += av[i] * bv[j];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + 4 * ty + i;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + 4 * tx + j;
+      if (m >= M || n >= N) continue;
+      float v = acc[i][j] + (bias ? bias[n] : 0.f);
+      if (act == 1) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
+      C[static_cast<size_t>(m) * ldc + n] = v;
+    }
+  }
+}
+
+}  // namespace b200
+
+using namespace b200;
+typedef __nv_bfloat16 bf16_t;
+#define STREAM reinterpret_cast<cudaStream_t>(stream)
+#define DONE (cudaGetLastError() == cudaSuccess ? 0 : -2)
+
+// Every `f32` argument: the operand storage type is fp32 instead of bf16; `in_f32`: the GEMM output is fp32.
+
+B200_API int b200_embed_resid(const long long* tok, const void* table, float* x, void* xb, int T, int E, int ld_table, int ld_xb,
+                              long long vocab, int f32, int* err, void* stream) {
+  if (T <= 0 || E <= 0 || vocab <= 0 || ld_table < E || ld_xb < E) return -1;
+  if (f32) embed_resid_kernel<float><<<T, 128, 0, STREAM>>>(tok, (const float*)table, x, (float*)xb, E, ld_table, ld_xb, vocab, err);
+  else embed_resid_kernel<bf16_t><<<T, 128, 0, STREAM>>>(tok, (const bf16_t*)table, x, (bf16_t*)xb, E, ld_table, ld_xb, vocab, err);
+  return DONE;
+}
+
+static bool latent_row_ok(const LatentRow& L) {
+  return L.H > 0 && L.dim > 0 && L.rot > 0 && !(L.rot & 1) && L.rank > 0 && L.rank_pad >= L.rank && !(L.rank_pad & 1) &&
+         L.ld_lat >= L.rank_pad + L.rot && L.cap > 0;
+}
+
+B200_API int b200_latent_prep(void* in, const LatentRow* Lp, const int* sidx, const int* end, void* cache, void* stream_buf, int T,
+                              int f32, void* stream) {
+  const LatentRow L = *Lp;
+  if (T <= 0 || !latent_row_ok(L) || (L.own && (!stream_buf || !sidx || !end))) return -1;
+  if (f32) latent_prep_kernel<float><<<T, 128, 0, STREAM>>>((float*)in, L, sidx, end, (float*)cache, (float*)stream_buf);
+  else latent_prep_kernel<bf16_t><<<T, 128, 0, STREAM>>>((bf16_t*)in, L, sidx, end, (bf16_t*)cache, (bf16_t*)stream_buf);
+  return DONE;
+}
+
+B200_API int b200_latent_absorb(const void* in, const LatentRow* Lp, const void* w_uk, int ldw, void* cache, void* qlat, int B,
+                                int in_f32, int f32, void* stream) {
+  const LatentRow L = *Lp;
+  if (B <= 0 || !latent_row_ok(L) || (ldw & 1) || ldw < ((L.rank + 1) & ~1) || (L.own && !cache) || (f32 && !in_f32)) return -1;
+  const int cols = (L.rank + ABS_COLS - 1) / ABS_COLS;
+  const dim3 grid(B + cols * L.H * ((B + ABS_ROWS - 1) / ABS_ROWS));
+  const size_t smem = (ABS_ROWS * L.dim + 4 * ABS_ROWS * ABS_COLS) * sizeof(float);
+  if (smem > 200 * 1024) return -1;
+#define GO(TI, T)                                                                                                      \
+  {                                                                                                                    \
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(latent_absorb_kernel<TI, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                 static_cast<int>(smem)) != cudaSuccess) return -3;                     \
+    launch_k(latent_absorb_kernel<TI, T>, grid, dim3(256), smem, STREAM, (const TI*)in, L, (const T*)w_uk, ldw, (T*)cache, (T*)qlat, B); \
+  }
+  if (f32) GO(float, float)
+  else if (in_f32) GO(float, bf16_t)
+  else GO(bf16_t, bf16_t)
+#undef GO
+  return DONE;
+}
+
+B200_API int b200_gather_rows(const void* src, const int* src_idx, void* dst, const int* dst_idx, int n, int row_bytes, void* stream) {
+  if (n <= 0) return 0;
+  if (row_bytes & 15) return -1;
+  gather_rows_kernel<<<n, 128, 0, STREAM>>>((const uint4*)src, src_idx, (uint4*)dst, dst_idx, row_bytes / 16);
+  return DONE;
+}
+
+B200_API int b200_window_attention(const void* q, const void* k1, const void* k2, const void* v, const void* gate, void* out,
+                                   const WindowAttn* Ap, int T, int f32, void* stream) {
+  const WindowAttn A = *Ap;
+  if (T <= 0 || A.H <= 0 || A.H > 65535 || A.d1 <= 0 || A.d2 < 0 || A.vdim <= 0 || A.window <= 0 || A.splits < 1 || A.splits > 32) return -1;
+  if (A.pos ? (!A.row || A.cap <= 0 || A.cap < A.window || !A.part_o || !A.part_ml) : (!A.sidx || !A.kbase || A.splits != 1 || A.part_o || !gate || !out))
+    return -1;
+  const size_t smem = (A.d1 + A.d2 + 128 + 4 * A.vdim + 8) * sizeof(float);
+  if (smem > 200 * 1024) return -1;
+  const dim3 grid(T, A.H, A.splits);
+#define GO(T_)                                                                                                         \
+  {                                                                                                                    \
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(window_attn_kernel<T_>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                                 static_cast<int>(smem)) != cudaSuccess) return -3;                     \
+    window_attn_kernel<T_><<<grid, 128, smem, STREAM>>>((const T_*)q, (const T_*)k1, (const T_*)k2, (const T_*)v,        \
+                                                        (const T_*)gate, (T_*)out, A);                                  \
+  }
+  if (f32) GO(float) else GO(bf16_t)
+#undef GO
+  return DONE;
+}
+
+B200_API int b200_latent_expand(const float* part_o, const float* part_ml, int splits, const void* w_uv, int ldw, const void* gate,
+                                int gate_ld, void* out, int out_ld, int B, int H, int rank, int vdim, int in_f32, int f32, void* stream) {
+  if (B <= 0 || splits < 1 || splits > 32 || (ldw & 1) || ldw < ((rank + 1) & ~1) || (f32 && !in_f32)) return -1;
+  const dim3 grid(H, (vdim + EXP_COLS - 1) / EXP_COLS, (B + EXP_ROWS - 1) / EXP_ROWS);
+  const size_t smem = EXP_ROWS * ((rank + 1) & ~1) * sizeof(float);
+  if (smem > 200 * 1024) return -1;
+#define GO(TI, T)                                                                                                      \
+  {                                                                                                                    \
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(latent_expand_kernel<TI, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                 static_cast<int>(smem)) != cudaSuccess) return -3;                     \
+    launch_k(latent_expand_kernel<TI, T>, grid, dim3(256), smem, STREAM, part_o, part_ml, splits, (const T*)w_uv, ldw,   \
+             (const TI*)gate, gate_ld, (T*)out, out_ld, B, H, rank, vdim);                                              \
+  }
+  if (f32) GO(float, float)
+  else if (in_f32) GO(float, bf16_t)
+  else GO(bf16_t, bf16_t)
+#undef GO
+  return DONE;
+}
+
+template <typename TI, typename T>
+static void launch_rms_residual(void* a, int ld_a, int clear, const float* bias, const float* w, float* x, void* xb, int ld_xb,
+                                int rows, int E, float eps, float mult, float* zero, int nzero, cudaStream_t st) {
+  const int nv = (E % 8 == 0 && ld_a % 8 == 0 && ld_xb % 8 == 0) ? (E / 8 + 255) / 256 : 0;
+  const bool aligned = !((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xb) |
+                          reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(bias)) & 15);
+#define GO(NV)                                                                                                        \
+  launch_k(rms_residual_vec_kernel<TI, T, NV>, dim3(rows), dim3(256), 0, st, (TI*)a, ld_a, clear, bias, w, x, (T*)xb, ld_xb, E, \
+           eps, mult, zero, nzero)
+  if (aligned && nv == 1) GO(1);
+  else if (aligned && nv == 2) GO(2);
+  else if (aligned && nv == 3) GO(3);
+  else if (aligned && nv == 4) GO(4);
+  else
+    launch_k(rms_residual_kernel<TI, T>, dim3(rows), dim3(256), 0, st, (TI*)a, ld_a, clear, bias, w, x, (T*)xb, ld_xb, E, eps, mult,
+             zero, nzero);
+#undef GO
+}
+
+B200_API int b200_rms_residual(void* a, int ld_a, int in_f32, int clear, const float* bias, const float* w, float* x, void* xb,
+                               int ld_xb, int rows, int E, float eps, float mult, float* zero, int nzero, int f32, void* stream) {
+  if (rows <= 0 || E <= 0 || (clear && !in_f32) || (f32 && !in_f32) || (nzero && !zero)) return -1;
+  if (f32) launch_rms_residual<float, float>(a, ld_a, clear, bias, w, x, xb, ld_xb, rows, E, eps, mult, zero, nzero, STREAM);
+  else if (in_f32) launch_rms_residual<float, bf16_t>(a, ld_a, clear, bias, w, x, xb, ld_xb, rows, E, eps, mult, zero, nzero, STREAM);
+  else launch_rms_residual<bf16_t, bf16_t>(a, ld_a, clear, bias, w, x, xb, ld_xb, rows, E, eps, mult, zero, nzero, STREAM);
+  return DONE;
+}
+
+B200_API int b200_rmsnorm_rows(const float* x, const int* idx, const float* w, void* y, int ld_y, int rows, int E, float eps, int f32,
+                               void* stream) {
+  if (rows <= 0) return 0;
+  if (f32) launch_k(rmsnorm_rows_kernel<float>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (float*)y, ld_y, E, eps);
+  else launch_k(rmsnorm_rows_kernel<bf16_t>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (bf16_t*)y, ld_y, E, eps);
+  return DONE;
+}
+
+B200_API int b200_bias_act(void* a, int ld_a, int in_f32, int clear, const float* bias, void* y, int ld_y, int rows, int N, int act,
+                           int f32, void* stream) {
+  if (rows <= 0 || rows > 65535 || N <= 0 || (clear && !in_f32) || (f32 && !in_f32)) return -1;
+  const dim3 grid((N + 255) / 256, rows);
+  if (f32) launch_k(bias_act_kernel<float, float>, grid, dim3(256), 0, STREAM, (float*)a, ld_a, clear, bias, (float*)y, ld_y, N, act);
+  else if (in_f32) launch_k(bias_act_kernel<float, bf16_t>, grid, dim3(256), 0, STREAM, (float*)a, ld_a, clear, bias, (bf16_t*)y, ld_y, N, act);
+  else launch_k(bias_act_kernel<bf16_t, bf16_t>, grid, dim3(256), 0, STREAM, (bf16_t*)a, ld_a, clear, bias, (bf16_t*)y, ld_y, N, act);
+  return DONE;
+}
+
+B200_API int b200_sgemm_nt(const float* A, const float* B, const float* bias, float* C, int M, int N, int K, int lda, int ldb, int ldc,
+                           int act, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || (N + SG - 1) / SG > 65535) return -1;
+  sgemm_nt_kernel<<<dim3((M + SG - 1) / SG, (N + SG - 1) / SG), 256, 0, STREAM>>>(A, B, bias, C, M, N, K, lda, ldb, ldc, act);
+  return DONE;
+}

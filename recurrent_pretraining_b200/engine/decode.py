@@ -20,18 +20,13 @@ exited; a sequence's token is frozen at its first exit (recpre/raven_modeling_mi
 from __future__ import annotations
 
 import ctypes as C
-import os
 
 import torch
 
 from ..ops import cuda as K
+from .base import BF16, PDL, SKINNY_ROWS, GraphRunner, skinny_linear
 
-BF16 = torch.bfloat16
 _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
-_set_pdl = K._sig("b200_set_pdl", [_i])
-PDL = os.environ.get("B200_DECODE_PDL", "0") == "1"  # measured within noise of off (23.1-23.5 vs 23.5 ms per token): off
-_skinny = K._sig("b200_gemm_skinny", [_vp] * 4 + [_i] * 7 + [_vp, _vp])
-_cast_zero = K._sig("b200_cast_zero", [_vp, _vp, C.c_longlong, _vp])
 _swiglu_acc = K._sig("b200_swiglu_acc", [_vp, _vp, C.c_longlong, _i, _vp])
 _norm_pair = K._sig("b200_add_rmsnorm_pair", [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _vp])
 _rope_append = K._sig("b200_rope_append", [_vp] * 8 + [_i] * 5 + [_vp, _i])
@@ -79,7 +74,7 @@ class StaticRecurrentKVCache:
         return 2 * self.k.numel() * 2 / 2**20
 
 
-class DecodeEngine:
+class DecodeEngine(GraphRunner):
     def __init__(self, model, max_batch: int, max_len: int, num_steps: int | None = None,
                  cache_lookup_strategy: str = "full", use_graphs: bool = True, attn_splits: int = 0,
                  max_steps: int | None = None):
@@ -87,7 +82,7 @@ class DecodeEngine:
         self.model, self.cfg = model, cfg
         self.dev = next(model.parameters()).device
         assert self.dev.type == "cuda" and next(model.parameters()).dtype == BF16, "engine runs bf16 weights on a GPU"
-        assert max_batch <= 64, "decode kernels cover batches up to 64 per replica"
+        assert max_batch <= SKINNY_ROWS, "decode kernels cover batches up to 64 per replica"
         self.B, self.Lmax = max_batch, max_len
         self.r = num_steps or cfg.mean_recurrence
         self.P, self.R, self.Cn = cfg.n_layers_in_prelude, cfg.n_layers_in_recurrent_block, cfg.n_layers_in_coda
@@ -139,23 +134,8 @@ class DecodeEngine:
 
     # -- kernels --------------------------------------------------------------------------------------
     def _linear(self, x, w, keep_f32: bool = False):
-        """x [B, K] bf16 -> [B, N] through the skinny weight-streaming GEMM.  Narrow outputs are accumulated over K
-        splits in the persistent fp32 ``work`` buffer (kept zero between uses by its consumers); ``keep_f32`` hands
-        that buffer to a fused consumer, otherwise it is converted (and cleared) here."""
-        Bt, Kd = x.shape
-        N = w.shape[0]
-        out = torch.empty(Bt, N, dtype=BF16, device=x.device)
-        work = self.work[: Bt * N].view(Bt, N) if Bt * N <= self.work.numel() else None
-        rc = _skinny(x.data_ptr(), w.data_ptr(), out.data_ptr(), K._ptr(work), Bt, N, Kd, x.stride(0), w.stride(0),
-                     N, 0, K._stream(), K.err_word(x.device).data_ptr())
-        K._launches += 1
-        if rc < 0:
-            raise RuntimeError(f"b200_gemm_skinny failed with code {rc}")
-        if rc == 1:
-            if keep_f32:
-                return work
-            K._check(_cast_zero(work.data_ptr(), out.data_ptr(), Bt * N, K._stream()), "cast_zero")
-        return out
+        """x [B, K] bf16 -> [B, N] through the skinny weight-streaming GEMM (``keep_f32``: see ``skinny_linear``)."""
+        return skinny_linear(x, w, self.work, keep_f32)
 
     def _all_blocks(self):
         t = self.model.transformer
@@ -243,33 +223,8 @@ class DecodeEngine:
         return self.logits[:B]
 
     # -- graph helpers ----------------------------------------------------------------------------------
-    def _run(self, key, fn):
-        """Replay ``fn`` as a CUDA graph.  ``fn`` must be idempotent (read inputs, write separate outputs): it is
-        executed once eagerly as a warm-up and once more during capture before the first replay."""
-        if not self.use_graphs:
-            return self._with_pdl(fn)
-        g = self._graphs.get(key)
-        if g is None:
-            self._with_pdl(fn)
-            torch.cuda.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                out = self._with_pdl(fn)
-            g = self._graphs[key] = (graph, out)
-        g[0].replay()
-        return g[1]
-
-    @staticmethod
-    def _with_pdl(fn):
-        """Run ``fn`` with programmatic dependent launch on for the decode kernels: each kernel's prologue overlaps the
-        tail of its predecessor (the attribute is recorded into a graph at capture time)."""
-        if not PDL:
-            return fn()
-        old = _set_pdl(1)
-        try:
-            return fn()
-        finally:
-            _set_pdl(old)
+    def _pdl_on(self) -> bool:
+        return PDL
 
     def _fresh_state(self, init_scale: float):
         self._seed += 1

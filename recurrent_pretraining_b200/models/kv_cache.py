@@ -219,3 +219,58 @@ class StaticRecurrentCache:
 
 
 HuginnStaticCache = StaticRecurrentCache
+
+
+class LatentRingCache:
+    """Cache of latent-attention layers: one row of ``ld_lat`` numbers per token (normed latent and rotated key part) in a ring
+    per sequence and source layer.  Position p lives in slot ``p % cap``; ``cap`` covers the widest window among the layers
+    that read the source layer's latents, so a sequence holds a bounded amount however long it grows.
+
+    Sequence rows are handed out by ``alloc`` and taken back by ``free``; a row that is used again needs no clearing, because
+    a reader only looks at positions its new owner has written.  Rows are added on demand (``generation`` counts those
+    reallocations: captured graphs that hold old addresses are then stale)."""
+
+    SLOTS = 128   # capacities are multiples of this many slots, so that a tile of keys stays inside one sequence's ring
+
+    def __init__(self, layouts: dict, windows: dict, max_rows: int, max_len: int, dtype: torch.dtype, device):
+        self.max_len, self.dtype, self.device = max_len, dtype, torch.device(device)
+        self.layouts, self.windows = layouts, windows
+        self.caps = {i: -(-min(w, max_len) // self.SLOTS) * self.SLOTS for i, w in windows.items()}
+        self.rows, self.generation = 0, 0
+        self.data: dict = {}
+        self.length: dict = {}            # row -> tokens held
+        self._free: list = []
+        self._grow(max_rows)
+
+    def _grow(self, rows: int) -> None:
+        for i, cap in self.caps.items():
+            new = torch.zeros(rows, cap, self.layouts[i].ld_lat, dtype=self.dtype, device=self.device)
+            if self.rows:
+                new[:self.rows] = self.data[i]
+            self.data[i] = new
+        self._free.extend(range(rows - 1, self.rows - 1, -1))
+        self._free.sort(reverse=True)
+        self.rows = rows
+        self.generation += 1
+
+    def alloc(self) -> int:
+        if not self._free:
+            self._grow(2 * self.rows)
+        row = self._free.pop()
+        self.length[row] = 0
+        return row
+
+    def free(self, row: int) -> None:
+        del self.length[row]              # KeyError: the row is not in use
+        self._free.append(row)
+
+    def advance(self, row: int, n: int) -> int:
+        """Book ``n`` more tokens for ``row``; returns the position of the first of them."""
+        start = self.length[row]
+        if start + n > self.max_len:
+            raise ValueError(f"sequence of {start + n} tokens in a cache for {self.max_len}")
+        self.length[row] = start + n
+        return start
+
+    def get_memory_usage(self) -> float:
+        return sum(t.numel() * t.element_size() for t in self.data.values()) / 2**20

@@ -64,6 +64,8 @@ OUT_BF16_ROPE = 7
 OUT_SWIGLU_SAVE = 8     # SwiGLU epilogue that also stores the pre-activation [gate | up] into ``resid``
 OUT_DSWIGLU = 9         # input-gradient GEMM whose epilogue applies the gate's derivative (``resid`` = pre-activation)
 OUT_BF16_LSE = 10       # head GEMM: bf16 logits + per-tile softmax partials + target logit (fused linear + CE)
+OUT_BF16_BIAS_ACT = 11  # bf16 act(acc + bias) with an fp32 column bias
+_set_bias = _sig("b200_gemm_set_bias", [_vp, _i])
 _set_lse = _sig("b200_gemm_set_lse", [_vp, _vp, _vp, _f])
 _ce_finish = _sig("b200_ce_finish", [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _f, _i, _f, _i, _vp])
 _set_rope = _sig("b200_gemm_set_rope", [_vp, _vp, _vp, _i, _i, _i])
@@ -145,9 +147,10 @@ def _mat(t: torch.Tensor):
 
 
 def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_mode=OUT_BF16, a2=None, resid=None, n_out=None, bn=0,
-         max_ctas=0, rope=None, lse=None):
+         max_ctas=0, rope=None, lse=None, bias=None, act=0):
     """C[M,N] (+)= A B^T.  ``a``: [M,K] (or [K,M] if a_mn), ``b``: [N,K] (or [K,N] if b_mn).
-    ``rope`` (OUT_BF16_ROPE): (cos [S, D/2] fp32, sin, bias flat fp32 or None, S, D, width of the q+k columns)."""
+    ``rope`` (OUT_BF16_ROPE): (cos [S, D/2] fp32, sin, bias flat fp32 or None, S, D, width of the q+k columns).
+    ``bias`` / ``act`` (OUT_BF16_BIAS_ACT): fp32 [N] or None, 0 = no activation, 1 = relu^2."""
     a, ar, ac, lda = _mat(a)
     b, br, bc, ldb = _mat(b)
     M, K1 = (ac, ar) if a_mn else (ar, ac)
@@ -164,7 +167,8 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_mode=OUT_BF16, a2=None, 
     if n_out is not None:
         N = n_out
     if out is None:
-        dt = BF16 if out_mode in (OUT_BF16, OUT_BF16_RESID, OUT_SWIGLU, OUT_BF16_ROPE, OUT_SWIGLU_SAVE, OUT_BF16_LSE) \
+        dt = BF16 if out_mode in (OUT_BF16, OUT_BF16_RESID, OUT_SWIGLU, OUT_BF16_ROPE, OUT_SWIGLU_SAVE, OUT_BF16_LSE,
+                                 OUT_BF16_BIAS_ACT) \
             else torch.float32
         if out_mode == OUT_DSWIGLU:      # [dgate | dup]: the tile epilogue writes both halves
             out = torch.empty((M, 2 * N), dtype=BF16, device=a.device)[:, :N]
@@ -191,6 +195,9 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_mode=OUT_BF16, a2=None, 
         assert tgt.numel() >= M and labels.dtype == torch.int64 and labels.is_contiguous()
         _set_lse(_ptr(part), _ptr(tgt), _ptr(labels), float(scale))
         bn = 256
+    if out_mode == OUT_BF16_BIAS_ACT:
+        assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= N)
+        _set_bias(_ptr(bias), int(act))
     rc = _gemm(_ptr(a), _ptr(a2), _ptr(b), _ptr(out), _ptr(resid), M, N, K1, K2, lda, lda2, ldb, out.stride(0),
                ld_resid, int(a_mn), int(b_mn), out_mode, bn, max_ctas, _stream(), _ptr(err_word(a.device)))
     _check(rc, "b200_gemm")

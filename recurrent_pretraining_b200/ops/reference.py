@@ -155,3 +155,49 @@ def adamw_step(p, g, m, v, lr, beta1, beta2, eps, wd, step, grad_scale=1.0):
     bc1, bc2 = 1 - beta1 ** step, 1 - beta2 ** step
     denom = (v.sqrt() / math.sqrt(bc2)).add_(eps)
     p.addcdiv_(m, denom, value=-lr / bc1)
+
+
+# ------------------------------------------------------------------------------------------
+# layered decoder models: latent attention, sliding window, fp32 residual stream
+# ------------------------------------------------------------------------------------------
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    return F.relu(x).square()
+
+
+def linear_act(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None) -> torch.Tensor:
+    """act(x w^T + bias) with an fp32 bias; result in x.dtype."""
+    y = F.linear(x, w).float()
+    if bias is not None:
+        y = y + bias
+    if act == "relu2":
+        y = relu2(y)
+    elif act is not None:
+        raise ValueError(f"unknown activation {act!r}")
+    return y.to(x.dtype)
+
+
+def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    x = x.float()
+    return x / torch.sqrt(x.square().mean(-1, keepdim=True) + eps)
+
+
+def rms_residual(x: torch.Tensor, a: torch.Tensor, bias: torch.Tensor | None, w: torch.Tensor, eps: float,
+                 mult: float) -> torch.Tensor:
+    """x + mult * rmsnorm(a + bias) * w on an fp32 residual stream."""
+    s = a.float() if bias is None else a.float() + bias
+    return x + mult * rms(s, eps) * w
+
+
+def rotate_pairs(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """Rotation of the interleaved pairs of the last dim; cos / sin broadcast against the pairs; fp32 result."""
+    u, v = x.float()[..., 0::2], x.float()[..., 1::2]
+    return torch.stack([u * cos - v * sin, v * cos + u * sin], dim=-1).flatten(-2)
+
+
+def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, visible: torch.Tensor, scale: float) -> torch.Tensor:
+    """q [T, H, D]; k, v [K, H, .] shared by all queries or [T, K, H, .] per query; visible [T, K] boolean.  fp32."""
+    q, k, v = q.float(), k.float(), v.float()
+    per_query = k.dim() == 4
+    s = torch.einsum("thd,tkhd->thk" if per_query else "thd,khd->thk", q, k) * scale
+    p = torch.softmax(s.masked_fill(~visible[:, None], float("-inf")), dim=-1)
+    return torch.einsum("thk,tkhd->thd" if per_query else "thk,khd->thd", p, v)

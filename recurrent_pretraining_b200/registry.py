@@ -185,6 +185,32 @@ configs: list[dict] = [
         mean_backprop_depth=2),
 ]
 
+
+
+# --------------------------------------------------------------------------------------
+# decoders described layer by layer (models/layered_config.py)
+# --------------------------------------------------------------------------------------
+def _gasovik(name, vocab, width, layers, heads, dim, rot_dim, vdim, kv_rank, window, ff, share_from=None, original=4096):
+    """``layers`` equal layers; from layer ``share_from`` on the latents of layer ``share_from - 1`` are shared."""
+    rot = {"base": 10000.0, "dims": rot_dim, "scaling": {"factor": 8.0, "original": original, "fast": 32.0, "slow": 1.0}}
+    out = []
+    for i in range(layers):
+        mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": window},
+                 "scale": (dim + rot_dim) ** -0.5, "rot": rot}
+        if share_from is not None and i >= share_from:
+            mixer["kv_from"] = share_from - 1
+        out.append({"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+    return {"name": name, "architecture": "Gasovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "layers": out}
+
+
+layered_configs: dict[str, dict] = {c["name"]: c for c in (
+    _gasovik("gasovik-tiny", 512, 128, 3, 4, 32, 16, 32, 64, 24, 256, share_from=2, original=64),
+    _gasovik("gasovik-1b", 65536, 2048, 16, 16, 128, 64, 128, 512, 1024, 8192, share_from=12),
+    # layers of the width and depth of the 3.5B recurrent flagship's core, for side-by-side timing
+    _gasovik("gasovik-core-5280", 65536, 5280, 4, 55, 96, 32, 96, 512, 4096, 17920),
+)}
+
 name_to_config: dict[str, dict] = {c["name"]: c for c in configs}
 
 
@@ -192,6 +218,8 @@ def lookup(name: str) -> dict:
     """Return a *copy* of the registry dict for ``name`` (also matches ``hf_config.name``)."""
     if name in name_to_config:
         return deepcopy(name_to_config[name])
+    if name in layered_configs:
+        return deepcopy(layered_configs[name])
     for c in configs:
         if c["hf_config"]["name"] == name:
             return deepcopy(c)
