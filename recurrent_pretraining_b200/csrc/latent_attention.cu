@@ -1,0 +1,434 @@
+// Sliding-window attention of a packed prompt step for latent-attention layers, on the 5th-generation tensor cores.
+//
+// Queries [T, H, dim + rot], unrotated keys [K, H, dim] and values [K, H, vdim] (one packed matrix), one rotated key part
+// [K, rot] shared by all heads.  Every size that is a multiple of eight is taken as it is: operand panels are 64 columns
+// wide and the copy engine zero-fills past dim, rot and vdim.
+//
+// One CTA per (256 queries of one sequence, head): two 128-query tiles share every key / value block and ping-pong on one
+// MMA issuer (the scheme of attn_fwd2_kernel in attention.cu):
+//   warps 0-3 / 4-7  softmax of tile A / B, one query row per thread: scores from tensor memory, window and causal mask on
+//                    the edge blocks, lazy rescale of the accumulator, bf16 weights written back over the scores
+//   warp 8           TMA: lane 0 queries and the key ring, lane 1 the value ring
+//   warp 9           MMA issuer: S = Q K^T over the unrotated and rotated panels, O += P V with P in tensor memory
+// Only key blocks that some query of a tile can see are visited.  The epilogue divides by the softmax sum and applies the
+// layer's output gate.
+#include <cuda.h>
+
+#include "common.cuh"
+
+namespace b200 {
+
+constexpr int LA_BM = 128;
+constexpr int LA_QPANEL = LA_BM * 128;   // 128 rows x 64 bf16
+constexpr int LA_MAX_STAGES = 3;
+
+struct LatentAttnParams {
+  int H, dim, rot, vdim, window;
+  int pn, pr, pv;               // 64-column panels of the unrotated, rotated and value parts
+  int kst, vst;                 // ring stages
+  float scale_log2;
+  const int4* tiles;            // {first query token, queries (1..256), stream index of the first query, first key of its sequence}
+  const __nv_bfloat16* gate;    // [T, ld_gate], head h at column h * vdim
+  __nv_bfloat16* out;           // [T, ld_out]
+  int ld_gate, ld_out;
+  int* err;
+};
+
+struct LatentAttnBars {
+  uint64_t q_full;
+  uint64_t k_full[LA_MAX_STAGES], k_empty[LA_MAX_STAGES], v_full[LA_MAX_STAGES], v_empty[LA_MAX_STAGES];
+  uint64_t s_full[2], p_ready[2], o_final[2];
+  uint32_t tmem_slot;
+  int abort_flag;
+};
+
+__device__ __forceinline__ float la_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int BN>
+__global__ void __launch_bounds__(384, 1)
+latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
+                   const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
+                   const __grid_constant__ CUtensorMap tmV, const LatentAttnParams p) {
+  constexpr int KPANEL = BN * 128;
+  constexpr uint32_t IDESC_S = make_idesc_bf16(LA_BM, BN, 0, 0);
+  constexpr int O_COL = 2 * BN, O_WIDTH = (512 - 2 * BN) / 2;
+  constexpr float RESCALE_THRESHOLD = 8.f;   // log2 units
+
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int kp = p.pn + p.pr;
+  const int q_bytes = kp * LA_QPANEL, k_bytes = kp * KPANEL, v_bytes = p.pv * KPANEL;
+  uint8_t* sQ = smem;                       // tile A, tile B
+  uint8_t* sK = sQ + 2 * q_bytes;
+  uint8_t* sV = sK + p.kst * k_bytes;
+  LatentAttnBars* bars = reinterpret_cast<LatentAttnBars*>(sV + p.vst * v_bytes);
+  volatile int* abort_flag = &bars->abort_flag;
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.x;
+  const int4 tile = p.tiles[blockIdx.y];
+  const int q0 = tile.x, nrows = tile.y, s0 = tile.z, kbase = tile.w;
+  const int kstart = max(kbase, s0 - p.window + 1);
+  // key blocks [jb, je) of both tiles, counted from kstart
+  const int last_a = min(LA_BM, nrows) - 1, last_b = nrows - 1;
+  const int je0 = (s0 + last_a - kstart) / BN + 1;
+  const int jb1 = nrows > LA_BM ? (max(kbase, s0 + LA_BM - p.window + 1) - kstart) / BN : 0;
+  const int je1 = nrows > LA_BM ? (s0 + last_b - kstart) / BN + 1 : 0;
+  const int nmax = max(je0, je1);
+
+  auto load_q = [&](int x) {
+    for (int c = 0; c < p.pn; ++c)
+      tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full, c * 64, h, q0 + x * LA_BM);
+    for (int c = 0; c < p.pr; ++c)
+      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full, c * 64, h, q0 + x * LA_BM);
+  };
+  auto load_k = [&](int j, int s) {
+    mbar_expect_tx(&bars->k_full[s], k_bytes);
+    for (int c = 0; c < p.pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, h, kstart + j * BN);
+    for (int c = 0; c < p.pr; ++c)
+      tma_load_2d(sK + s * k_bytes + (p.pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
+  };
+
+  // the TMA thread sets up the barriers and requests the queries and the first key block before the CTA-wide sync
+  if (threadIdx.x == 256) {
+    mbar_init(&bars->q_full, 1);
+    for (int i = 0; i < LA_MAX_STAGES; ++i) {
+      mbar_init(&bars->k_full[i], 1);
+      mbar_init(&bars->k_empty[i], 1);
+      mbar_init(&bars->v_full[i], 1);
+      mbar_init(&bars->v_empty[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&bars->s_full[i], 1);
+      mbar_init(&bars->p_ready[i], 4);
+      mbar_init(&bars->o_final[i], 1);
+    }
+    bars->abort_flag = 0;
+    fence_barrier_init();
+    fence_proxy_async_smem();
+    mbar_expect_tx(&bars->q_full, 2 * q_bytes);
+    load_q(0);
+    load_q(1);            // rows past the sequence are other tokens or zero; they are never stored
+    load_k(0, 0);
+  }
+  if (warp == 9) {
+    tmem_alloc(&bars->tmem_slot, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = bars->tmem_slot;
+
+  if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 72;");
+    if (warp == 8) {
+      if (lane == 0) {
+        int issued = 1;
+        for (int j = 1; j < nmax; ++j) {
+          const int s = j % p.kst;
+          if (!mbar_wait(&bars->k_empty[s], ((j / p.kst) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
+          load_k(j, s);
+          issued = j + 1;
+        }
+        // every issued load must land before the CTA exits
+        unsigned long long t0 = globaltimer_ns();
+        while (!mbar_try_wait(&bars->q_full, 0) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
+        for (int j = max(0, issued - p.kst); j < issued; ++j) {
+          t0 = globaltimer_ns();
+          while (!mbar_try_wait(&bars->k_full[j % p.kst], (j / p.kst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
+        }
+      } else if (lane == 1) {
+        int issued = 0;
+        for (int j = 0; j < nmax; ++j) {
+          const int s = j % p.vst;
+          if (!mbar_wait(&bars->v_empty[s], ((j / p.vst) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
+          mbar_expect_tx(&bars->v_full[s], v_bytes);
+          for (int c = 0; c < p.pv; ++c)
+            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, h, kstart + j * BN);
+          issued = j + 1;
+        }
+        for (int j = max(0, issued - p.vst); j < issued; ++j) {
+          const unsigned long long t0 = globaltimer_ns();
+          while (!mbar_try_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
+        }
+      }
+    } else if (warp == 9) {
+      if (lane == 0) {
+        const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV);
+        const uint32_t idesc_o = make_idesc_bf16(LA_BM, (p.vdim + 15) & ~15, 0, 1);
+        const int steps_n = (p.dim + 15) >> 4, steps_r = (p.rot + 15) >> 4;
+        auto issue_s = [&](int x, int j) {   // S_x = Q_x K_j^T
+          const uint32_t kb = aK + (j % p.kst) * k_bytes, qb = aQ + x * q_bytes;
+          const uint32_t d = tmem_base + x * BN;
+          for (int t = 0; t < steps_n; ++t)
+            umma_bf16(d, make_smem_desc(qb + (t >> 2) * LA_QPANEL + (t & 3) * 32, 16, 1024),
+                      make_smem_desc(kb + (t >> 2) * KPANEL + (t & 3) * 32, 16, 1024), IDESC_S, t ? 1u : 0u);
+          const uint32_t qr = qb + p.pn * LA_QPANEL, kr = kb + p.pn * KPANEL;
+          for (int t = 0; t < steps_r; ++t)
+            umma_bf16(d, make_smem_desc(qr + (t >> 2) * LA_QPANEL + (t & 3) * 32, 16, 1024),
+                      make_smem_desc(kr + (t >> 2) * KPANEL + (t & 3) * 32, 16, 1024), IDESC_S, 1u);
+          umma_commit(&bars->s_full[x]);
+        };
+        auto issue_pv = [&](int x, int j, bool first) {   // O_x += P_x V_j, P_x over the first BN / 2 columns of S_x
+          const uint32_t vb = aV + (j % p.vst) * v_bytes;
+#pragma unroll
+          for (int t = 0; t < BN / 16; ++t)
+            umma_bf16_ts(tmem_base + O_COL + x * O_WIDTH, tmem_base + x * BN + t * 8, make_smem_desc(vb + t * 2048, KPANEL, 1024),
+                         idesc_o, (first && t == 0) ? 0u : 1u);
+        };
+        bool ok = mbar_wait(&bars->q_full, 0, abort_flag, p.err, ERR_WAIT_ATTN) &&
+                  mbar_wait(&bars->k_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN);
+        if (ok) {
+          tc_fence_after();
+          issue_s(0, 0);
+          if (je1 > 0 && jb1 == 0) issue_s(1, 0);
+          umma_commit(&bars->k_empty[0]);
+        }
+        for (int j = 0; j < nmax && ok; ++j) {
+          if (!mbar_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
+          if (j + 1 < nmax && !mbar_wait(&bars->k_full[(j + 1) % p.kst], ((j + 1) / p.kst) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) {
+            ok = false;
+            break;
+          }
+          tc_fence_after();
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            const int jb = x ? jb1 : 0, je = x ? je1 : je0;
+            if (j >= jb && j < je) {
+              if (!mbar_wait(&bars->p_ready[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
+              tc_fence_after();
+              issue_pv(x, j, j == jb);
+              if (j + 1 == je) umma_commit(&bars->o_final[x]);
+            }
+            if (j + 1 >= jb && j + 1 < je) issue_s(x, j + 1);
+          }
+          if (!ok) break;
+          umma_commit(&bars->v_empty[j % p.vst]);
+          if (j + 1 < nmax) umma_commit(&bars->k_empty[(j + 1) % p.kst]);
+        }
+      }
+    }
+  } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");
+    const int x = warp >> 2;
+    const int quad = warp & 3;
+    const int r = x * LA_BM + quad * 32 + lane;              // query row of this thread inside the CTA's 256
+    const int jb = x ? jb1 : 0, je = x ? je1 : je0;
+    const int hi = s0 + r, lo = max(kbase, hi - p.window + 1);   // visible stream positions of the row
+    const int hi_first = s0 + x * LA_BM;                      // tile-wide: blocks inside [lo_last, hi_first] need no mask
+    const int lo_last = max(kbase, s0 + (x ? last_b : last_a) - p.window + 1);
+    const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
+    const uint32_t ts = tmem_base + x * BN + lane_addr;
+    const uint32_t to = tmem_base + O_COL + x * O_WIDTH + lane_addr;
+    const float scale_log2 = p.scale_log2;
+    float m = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (int j = jb; j < je && ok; ++j) {
+      if (!mbar_wait(&bars->s_full[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
+      tc_fence_after();
+      float sv[BN];
+#pragma unroll
+      for (int c = 0; c < BN; c += 32) {
+        uint32_t v[32];
+        tmem_ld_32x32(ts + c, v);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
+      }
+      tmem_ld_wait();
+      const int k0 = kstart + j * BN;
+      if (k0 < lo_last || k0 + BN - 1 > hi_first) {
+        const int cmin = lo - k0, cmax = hi - k0;
+#pragma unroll
+        for (int i = 0; i < BN; ++i)
+          if (i < cmin || i > cmax) sv[i] = -INFINITY;
+      }
+      float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
+#pragma unroll
+      for (int i = 4; i < BN; i += 4) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) mx4[k] = fmaxf(mx4[k], sv[i + k]);
+      }
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+      const float m_new = fmaxf(m, mx * scale_log2);
+      // raise the reference max only when it moved by more than the threshold (decided per warp)
+      const bool grow = (m_new - m > RESCALE_THRESHOLD) || (m == -INFINITY);
+      if (__any_sync(0xffffffffu, grow)) {
+        const float alpha = (m == -INFINITY) ? 0.f : la_ex2(m - m_new);
+        if (j > jb) {
+#pragma unroll 1
+          for (int c = 0; c < p.vdim; c += 32) {
+            uint32_t v[32];
+            tmem_ld_32x32(to + c, v);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
+            tmem_st_32x32(to + c, v);
+          }
+        }
+        l *= alpha;
+        m = m_new;
+      }
+      const float neg_m = (m == -INFINITY) ? 0.f : -m;        // a row may see nothing of the tile's first blocks
+      float rs[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int c = 0; c < BN; c += 32) {
+        uint32_t packed[16];
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          const float a = la_ex2(fmaf(sv[c + i], scale_log2, neg_m)), b = la_ex2(fmaf(sv[c + i + 1], scale_log2, neg_m));
+          rs[i & 2] += a;
+          rs[(i & 2) + 1] += b;
+          packed[i >> 1] = pack_bf16x2(a, b);
+        }
+        tmem_st_32x16(ts + (c >> 1), packed);
+      }
+      l += (rs[0] + rs[1]) + (rs[2] + rs[3]);
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->p_ready[x]);
+    }
+    if (ok && je > jb) {
+      if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
+        tc_fence_after();
+        const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
+        const size_t t = static_cast<size_t>(q0) + r;
+        const bool live = r < nrows;
+        const __nv_bfloat16* grow_ = p.gate + (live ? t : 0) * p.ld_gate + h * p.vdim;
+        __nv_bfloat16* orow = p.out + (live ? t : 0) * p.ld_out + h * p.vdim;
+#pragma unroll 1
+        for (int c = 0; c < p.vdim; c += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32(to + c, v);
+          tmem_ld_wait();
+          if (live) {
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+              if (c + 8 * q < p.vdim) {
+                const uint4 g4 = *reinterpret_cast<const uint4*>(grow_ + c + 8 * q);
+                const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+                uint32_t o[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const float2 g = unpack_bf16x2(gw[i]);
+                  o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * inv_l / (1.f + __expf(-g.x)),
+                                     __uint_as_float(v[8 * q + 2 * i + 1]) * inv_l / (1.f + __expf(-g.y)));
+                }
+                *reinterpret_cast<uint4*>(orow + c + 8 * q) = make_uint4(o[0], o[1], o[2], o[3]);
+              }
+            }
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 9) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+typedef CUresult (*EncodeTiledFnL)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// bf16 tensor [rows, (heads,) cols] with row pitch `ld` and head pitch `head` (elements); box: `box_rows` rows x 64 columns of
+// one head, 128-byte swizzle.  heads = 0: two-dimensional.
+static int make_tmap_rows(CUtensorMap* out, const void* base, uint64_t cols, uint64_t heads, uint64_t rows, uint64_t head, uint64_t ld,
+                          uint32_t box_rows) {
+  static EncodeTiledFnL enc = nullptr;
+  if (!enc) {
+    void* ptr = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) != cudaSuccess ||
+        q != cudaDriverEntryPointSuccess)
+      return -1;
+    enc = reinterpret_cast<EncodeTiledFnL>(ptr);
+  }
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (ld & 7) || (heads && (head & 7))) return -2;
+  const int rank = heads ? 3 : 2;
+  cuuint64_t dims[3] = {cols, heads ? heads : rows, rows};
+  cuuint64_t strides[2] = {(heads ? head : ld) * 2, ld * 2};
+  cuuint32_t box[3] = {64, heads ? 1u : box_rows, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), dims, strides, box, estr,
+             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? 0 : -3;
+}
+
+struct LatentAttnPlan { int bn, kst, vst, smem; };
+
+// Key-block width and ring depths for the given sizes; bn = 0: not covered.
+static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
+  LatentAttnPlan none = {0, 0, 0, 0};
+  if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot <= 0 || vdim <= 0) return none;
+  const int kp = (dim + 63) / 64 + (rot + 63) / 64, pv = (vdim + 63) / 64;
+  constexpr int LIMIT = 227 * 1024, FIXED = 1024 + 512;
+  for (int bn = 128; bn >= 64; bn -= 64) {
+    if (((vdim + 31) & ~31) > (512 - 2 * bn) / 2) continue;
+    for (int st = 5; st >= 4; --st) {        // three value stages before three key stages
+      const int kst = 2, vst = st - 2;
+      const int need = 2 * kp * LA_QPANEL + (kst * kp + vst * pv) * bn * 128 + FIXED;
+      if (need <= LIMIT) {
+        const int need3 = need + kp * bn * 128;
+        return need3 <= LIMIT ? LatentAttnPlan{bn, 3, vst, need3} : LatentAttnPlan{bn, kst, vst, need};
+      }
+    }
+  }
+  return none;
+}
+
+template <int BN>
+static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
+  auto kern = latent_attn_kernel<BN>;
+  static int configured = 0;
+  if (configured < plan.smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess) return -10;
+    configured = plan.smem;
+  }
+  kern<<<dim3(p.H, n_tiles), 384, plan.smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -11;
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+B200_API int b200_latent_attention_supported(int dim, int rot, int vdim) { return latent_attn_plan(dim, rot, vdim).bn > 0; }
+
+// q: [T, ld_q] (head h at column h (dim + rot)), kn / v: [K, ld_kv] (head h at column h dim / h vdim), kr: [K, ld_kr],
+// gate: [T, ld_gate], out: [T, ld_out]; tiles: int4 [n_tiles] as in LatentAttnParams.
+B200_API int b200_latent_attention(const void* q, const void* kn, const void* kr, const void* v, const void* gate, void* out,
+                                   const int* tiles, int n_tiles, int T, int K, int H, int dim, int rot, int vdim, int ld_q, int ld_kv,
+                                   int ld_kr, int ld_gate, int ld_out, int window, float scale, void* stream, int* err) {
+  const LatentAttnPlan plan = latent_attn_plan(dim, rot, vdim);
+  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || T <= 0 || K <= 0 || window <= 0) return -1;
+  if ((reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) || (ld_gate & 7) || (ld_out & 7)) return -2;
+  CUtensorMap tm[5];
+  const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(q);
+  int rc = make_tmap_rows(&tm[0], qb, dim, H, T, dim + rot, ld_q, LA_BM);
+  if (!rc) rc = make_tmap_rows(&tm[1], qb + dim, rot, H, T, dim + rot, ld_q, LA_BM);
+  if (!rc) rc = make_tmap_rows(&tm[2], kn, dim, H, K, dim, ld_kv, plan.bn);
+  if (!rc) rc = make_tmap_rows(&tm[3], kr, rot, 0, K, 0, ld_kr, plan.bn);
+  if (!rc) rc = make_tmap_rows(&tm[4], v, vdim, H, K, vdim, ld_kv, plan.bn);
+  if (rc) return rc;
+  LatentAttnParams p = {};
+  p.H = H; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
+  p.pn = (dim + 63) / 64; p.pr = (rot + 63) / 64; p.pv = (vdim + 63) / 64;
+  p.kst = plan.kst; p.vst = plan.vst;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.tiles = reinterpret_cast<const int4*>(tiles);
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
+  p.err = err;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return plan.bn == 128 ? launch_latent_attn<128>(tm, p, plan, n_tiles, st) : launch_latent_attn<64>(tm, p, plan, n_tiles, st);
+}
