@@ -28,6 +28,18 @@ template <> __device__ __forceinline__ float2 ld2<float>(const float* p) { retur
 template <> __device__ __forceinline__ float2 ld2<__nv_bfloat16>(const __nv_bfloat16* p) {
   return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
 }
+__device__ __forceinline__ void st2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void st2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); }
+// four neighbouring elements
+__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void ld4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
 // eight neighbouring elements (16-byte aligned rows)
 __device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
   const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
@@ -140,12 +152,23 @@ latent_prep_kernel(T* __restrict__ in, LatentRow L, const int* __restrict__ sidx
   const int p = L.pos[t], half = L.rot >> 1, hd = L.dim + L.rot;
   const float* ct = L.cosT + static_cast<size_t>(p) * half;
   const float* st = L.sinT + static_cast<size_t>(p) * half;
-  for (int i = threadIdx.x; i < L.H * half; i += 128) {
-    const int h = i / half, j = i - h * half;
-    T* q = r + h * hd + L.dim + 2 * j;
-    const float u = ldf(q), v = ldf(q + 1), c = ct[j], s = st[j];
-    stf(q, u * c - v * s);
-    stf(q + 1, v * c + u * s);
+  if ((L.dim & 1) == 0) {                           // pairs are aligned to two elements
+#pragma unroll 4
+    for (int i = threadIdx.x; i < L.H * half; i += 128) {
+      const int h = i / half, j = i - h * half;
+      T* q = r + h * hd + L.dim + 2 * j;
+      const float2 f = ld2(q);
+      const float c = ct[j], s = st[j];
+      st2(q, make_float2(f.x * c - f.y * s, f.y * c + f.x * s));
+    }
+  } else {
+    for (int i = threadIdx.x; i < L.H * half; i += 128) {
+      const int h = i / half, j = i - h * half;
+      T* q = r + h * hd + L.dim + 2 * j;
+      const float u = ldf(q), v = ldf(q + 1), c = ct[j], s = st[j];
+      stf(q, u * c - v * s);
+      stf(q + 1, v * c + u * s);
+    }
   }
   if (L.own) {
     T* dst = cache && p >= end[t] - L.cap ? cache + (static_cast<size_t>(L.row[t]) * L.cap + p % L.cap) * L.ld_lat : nullptr;
@@ -193,42 +216,49 @@ latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict
   const int h = id % L.H, b0 = (id / L.H) * ABS_ROWS;
   const int nb = min(ABS_ROWS, B - b0);
   float* qs = sm;                                  // [ABS_ROWS][dim]
-  float* part = sm + ABS_ROWS * L.dim;             // [4][ABS_ROWS][ABS_COLS]
+  float* part = sm + ABS_ROWS * ((L.dim + 3) & ~3);   // [8][ABS_ROWS][ABS_COLS]
   for (int i = threadIdx.x; i < ABS_ROWS * L.dim; i += 256) {
     const int b = i / L.dim, d = i - b * L.dim;
     qs[i] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
   }
   __syncthreads();
-  const int tx = threadIdx.x & 63, grp = threadIdx.x >> 6;
-  const int r = rc * ABS_COLS + 2 * tx;
-  float acc[ABS_ROWS][2];
+  const int tx = threadIdx.x & 31, grp = threadIdx.x >> 5;   // four columns per thread, eight groups over d
+  const int r = rc * ABS_COLS + 4 * tx;
+  float acc[ABS_ROWS][4];
 #pragma unroll
-  for (int b = 0; b < ABS_ROWS; ++b) acc[b][0] = acc[b][1] = 0.f;
-  if (r < L.rank) {                                // weight rows are padded: column r + 1 exists
+  for (int b = 0; b < ABS_ROWS; ++b)
+#pragma unroll
+    for (int k = 0; k < 4; ++k) acc[b][k] = 0.f;
+  if (r < L.rank) {                                // weight rows are padded to eight: columns up to r + 3 exist
     const T* wp = w_uk + static_cast<size_t>(h) * L.dim * ldw + r;
-#pragma unroll 4
-    for (int d = grp; d < L.dim; d += 4) {
-      const float2 w = ld2(wp + static_cast<size_t>(d) * ldw);
+    for (int d0 = grp; d0 < L.dim; d0 += 128) {
+      float w[16][4];
 #pragma unroll
-      for (int b = 0; b < ABS_ROWS; ++b) {
-        const float q = qs[b * L.dim + d];
-        acc[b][0] += q * w.x;
-        acc[b][1] += q * w.y;
+      for (int u = 0; u < 16; ++u)
+        if (d0 + 8 * u < L.dim) ld4(wp + static_cast<size_t>(d0 + 8 * u) * ldw, w[u]);
+#pragma unroll
+      for (int u = 0; u < 16; ++u) {
+        if (d0 + 8 * u < L.dim) {
+#pragma unroll
+          for (int b = 0; b < ABS_ROWS; ++b) {
+            const float q = qs[b * L.dim + d0 + 8 * u];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[b][k] += q * w[u][k];
+          }
+        }
       }
     }
   }
 #pragma unroll
-  for (int b = 0; b < ABS_ROWS; ++b) {
-    part[(grp * ABS_ROWS + b) * ABS_COLS + 2 * tx] = acc[b][0];
-    part[(grp * ABS_ROWS + b) * ABS_COLS + 2 * tx + 1] = acc[b][1];
-  }
+  for (int b = 0; b < ABS_ROWS; ++b)
+    *reinterpret_cast<float4*>(&part[(grp * ABS_ROWS + b) * ABS_COLS + 4 * tx]) = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
   __syncthreads();
   for (int i = threadIdx.x; i < nb * ABS_COLS; i += 256) {
     const int b = i / ABS_COLS, c = i - b * ABS_COLS;
     if (rc * ABS_COLS + c >= L.rank) continue;
     float v = 0.f;
 #pragma unroll
-    for (int g = 0; g < 4; ++g) v += part[(g * ABS_ROWS + b) * ABS_COLS + c];
+    for (int g = 0; g < 8; ++g) v += part[(g * ABS_ROWS + b) * ABS_COLS + c];
     stf(qlat + (static_cast<size_t>(b0 + b) * L.H + h) * L.ld_lat + rc * ABS_COLS + c, v);
   }
 }
@@ -342,20 +372,42 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   }
 }
 
+// Sum over the lanes of a warp of N values per lane (N a power of two <= 32) by halving exchanges: afterwards lane l holds the
+// total of value l % N.
+template <int N>
+__device__ __forceinline__ float warp_sum_many(float (&v)[N]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int off = 16; off >= N; off >>= 1) {
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[k] += __shfl_xor_sync(0xffffffffu, v[k], off);
+  }
+#pragma unroll
+  for (int off = N / 2; off > 0; off >>= 1) {
+#pragma unroll
+    for (int k = 0; k < off; ++k) {
+      const bool up = lane & off;
+      const float send = up ? v[k] : v[k + off], keep = up ? v[k + off] : v[k];
+      v[k] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+    }
+  }
+  return v[0];
+}
+
 // out[b, h * vdim + v] = sigmoid(gate) * sum_r W_uv[h * vdim + v, r] o[b, h, r], o = merged key splits.
-// CTA: (head, 32 values, 8 rows).
-constexpr int EXP_ROWS = 8, EXP_COLS = 32;
-template <typename TI, typename T>
+// CTA: (head, 32 values, ROWS rows); a warp forms four values of all its rows at once.
+constexpr int EXP_COLS = 32;
+template <typename TI, typename T, int ROWS>
 __global__ void __launch_bounds__(256)
 latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
                      const T* __restrict__ w_uv, int ldw, const TI* __restrict__ gate, int gate_ld, T* __restrict__ out,
                      int out_ld, int B, int H, int rank, int vdim) {
   pdl_trigger();
   pdl_wait();
-  extern __shared__ float os[];                    // [EXP_ROWS][rank_even]
-  __shared__ float wgt[EXP_ROWS][33];
-  const int h = blockIdx.x, v0 = blockIdx.y * EXP_COLS, b0 = blockIdx.z * EXP_ROWS;
-  const int nb = min(EXP_ROWS, B - b0), rs = (rank + 1) & ~1;
+  extern __shared__ float os[];                    // [ROWS][rank padded to eight]
+  __shared__ float wgt[ROWS][33];
+  const int h = blockIdx.x, v0 = blockIdx.y * EXP_COLS, b0 = blockIdx.z * ROWS;
+  const int nb = min(ROWS, B - b0), rs = (rank + 7) & ~7;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp < nb) {                                 // warp b: weights of the splits of row b (splits <= 32)
     const size_t base = (static_cast<size_t>(b0 + warp) * H + h) * splits;
@@ -366,44 +418,51 @@ latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__
     wgt[warp][lane] = a / ll;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < EXP_ROWS * rs; i += 256) {
+  for (int i = threadIdx.x; i < ROWS * rs; i += 256) {
     const int b = i / rs, r = i - b * rs;
     float o = 0.f;
     if (b < nb && r < rank) {
       const float* p = part_o + (static_cast<size_t>(b0 + b) * H + h) * splits * rank + r;
+#pragma unroll 8
       for (int s = 0; s < splits; ++s) {
-        const float w = wgt[b][s];
-        if (w != 0.f) o += w * p[static_cast<size_t>(s) * rank];   // an empty split's partial is not initialised
+        const float w = wgt[b][s], x = p[static_cast<size_t>(s) * rank];
+        o += w != 0.f ? w * x : 0.f;               // an empty split's partial is not initialised
       }
     }
     os[i] = o;
   }
   __syncthreads();
-#pragma unroll 1
-  for (int k = 0; k < EXP_COLS / 8; ++k) {
-    const int v = v0 + warp * (EXP_COLS / 8) + k;
-    if (v >= vdim) break;
-    const T* wr = w_uv + (static_cast<size_t>(h) * vdim + v) * ldw;
-    float acc[EXP_ROWS];
+  const int vw = v0 + warp * 4;
+  float acc[4 * ROWS];
 #pragma unroll
-    for (int b = 0; b < EXP_ROWS; ++b) acc[b] = 0.f;
-#pragma unroll 4
-    for (int r = 2 * lane; r < rank; r += 64) {    // weight rows are padded: column r + 1 exists (times a zero)
-      const float2 w = ld2(wr + r);
+  for (int i = 0; i < 4 * ROWS; ++i) acc[i] = 0.f;
+  const T* wr = w_uv + (static_cast<size_t>(h) * vdim + vw) * ldw;
+#pragma unroll 2
+  for (int r = 8 * lane; r < rs; r += 256) {       // weight rows are padded to eight with zeros
+    float w[4][8];
 #pragma unroll
-      for (int b = 0; b < EXP_ROWS; ++b) {
-        const float2 o = *reinterpret_cast<const float2*>(os + b * rs + r);
-        acc[b] += w.x * o.x + w.y * o.y;
+    for (int k = 0; k < 4; ++k) {
+      if (vw + k < vdim) ld8(wr + static_cast<size_t>(k) * ldw + r, w[k]);
+      else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) w[k][j] = 0.f;
       }
     }
 #pragma unroll
-    for (int b = 0; b < EXP_ROWS; ++b) {
-      const float s = warp_sum(acc[b]);
-      if (lane == b && b < nb) {
-        const float g = sigmoid_f(ldf(gate + static_cast<size_t>(b0 + b) * gate_ld + h * vdim + v));
-        stf(out + static_cast<size_t>(b0 + b) * out_ld + h * vdim + v, s * g);
-      }
+    for (int b = 0; b < ROWS; ++b) {
+      float o[8];
+      ld8(os + b * rs + r, o);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[b * 4 + k] += w[k][j] * o[j];
     }
+  }
+  const float s = warp_sum_many<4 * ROWS>(acc);
+  const int b = lane >> 2, v = vw + (lane & 3);
+  if (lane < 4 * ROWS && b < nb && v < vdim) {
+    const float g = sigmoid_f(ldf(gate + static_cast<size_t>(b0 + b) * gate_ld + h * vdim + v));
+    stf(out + static_cast<size_t>(b0 + b) * out_ld + h * vdim + v, s * g);
   }
 }
 
@@ -596,10 +655,10 @@ B200_API int b200_latent_prep(void* in, const LatentRow* Lp, const int* sidx, co
 B200_API int b200_latent_absorb(const void* in, const LatentRow* Lp, const void* w_uk, int ldw, void* cache, void* qlat, int B,
                                 int in_f32, int f32, void* stream) {
   const LatentRow L = *Lp;
-  if (B <= 0 || !latent_row_ok(L) || (ldw & 1) || ldw < ((L.rank + 1) & ~1) || (L.own && !cache) || (f32 && !in_f32)) return -1;
+  if (B <= 0 || !latent_row_ok(L) || (ldw & 7) || ldw < L.rank || (reinterpret_cast<uintptr_t>(w_uk) & 15) || (L.own && !cache) || (f32 && !in_f32)) return -1;
   const int cols = (L.rank + ABS_COLS - 1) / ABS_COLS;
   const dim3 grid(B + cols * L.H * ((B + ABS_ROWS - 1) / ABS_ROWS));
-  const size_t smem = (ABS_ROWS * L.dim + 4 * ABS_ROWS * ABS_COLS) * sizeof(float);
+  const size_t smem = (ABS_ROWS * ((L.dim + 3) & ~3) + 8 * ABS_ROWS * ABS_COLS) * sizeof(float);
   if (smem > 200 * 1024) return -1;
 #define GO(TI, T)                                                                                                      \
   {                                                                                                                    \
@@ -644,21 +703,29 @@ B200_API int b200_window_attention(const void* q, const void* k1, const void* k2
 
 B200_API int b200_latent_expand(const float* part_o, const float* part_ml, int splits, const void* w_uv, int ldw, const void* gate,
                                 int gate_ld, void* out, int out_ld, int B, int H, int rank, int vdim, int in_f32, int f32, void* stream) {
-  if (B <= 0 || splits < 1 || splits > 32 || (ldw & 1) || ldw < ((rank + 1) & ~1) || (f32 && !in_f32)) return -1;
-  const dim3 grid(H, (vdim + EXP_COLS - 1) / EXP_COLS, (B + EXP_ROWS - 1) / EXP_ROWS);
-  const size_t smem = EXP_ROWS * ((rank + 1) & ~1) * sizeof(float);
+  if (B <= 0 || splits < 1 || splits > 32 || (ldw & 7) || ldw < rank || (reinterpret_cast<uintptr_t>(w_uv) & 15) || (f32 && !in_f32)) return -1;
+  const int rows = B >= 8 ? 8 : (B > 1 ? 4 : 1);
+  const dim3 grid(H, (vdim + EXP_COLS - 1) / EXP_COLS, (B + rows - 1) / rows);
+  const size_t smem = rows * ((rank + 7) & ~7) * sizeof(float);
   if (smem > 200 * 1024) return -1;
-#define GO(TI, T)                                                                                                      \
+#define GO2(TI, T, R)                                                                                                  \
   {                                                                                                                    \
-    if (smem > 40 * 1024 && cudaFuncSetAttribute(latent_expand_kernel<TI, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(latent_expand_kernel<TI, T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                                  static_cast<int>(smem)) != cudaSuccess) return -3;                     \
-    launch_k(latent_expand_kernel<TI, T>, grid, dim3(256), smem, STREAM, part_o, part_ml, splits, (const T*)w_uv, ldw,   \
+    launch_k(latent_expand_kernel<TI, T, R>, grid, dim3(256), smem, STREAM, part_o, part_ml, splits, (const T*)w_uv, ldw, \
              (const TI*)gate, gate_ld, (T*)out, out_ld, B, H, rank, vdim);                                              \
+  }
+#define GO(TI, T)                        \
+  {                                      \
+    if (rows == 8) GO2(TI, T, 8)         \
+    else if (rows == 4) GO2(TI, T, 4)    \
+    else GO2(TI, T, 1)                   \
   }
   if (f32) GO(float, float)
   else if (in_f32) GO(float, bf16_t)
   else GO(bf16_t, bf16_t)
 #undef GO
+#undef GO2
   return DONE;
 }
 

@@ -162,24 +162,29 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV);
         const uint32_t idesc_o = make_idesc_bf16(LA_BM, (p.vdim + 15) & ~15, 0, 1);
         const int steps_n = (p.dim + 15) >> 4, steps_r = (p.rot + 15) >> 4;
+        // descriptors advance by their 16-byte-unit offsets: 2 per 16 K-major columns, 128 per 16 MN-major key rows
+        const uint64_t dq0 = make_smem_desc(aQ, 16, 1024), dk0 = make_smem_desc(aK, 16, 1024), dv0 = make_smem_desc(aV, KPANEL, 1024);
         auto issue_s = [&](int x, int j) {   // S_x = Q_x K_j^T
-          const uint32_t kb = aK + (j % p.kst) * k_bytes, qb = aQ + x * q_bytes;
+          uint64_t qd = dq0 + ((x * q_bytes) >> 4), kd = dk0 + (((j % p.kst) * k_bytes) >> 4);
           const uint32_t d = tmem_base + x * BN;
-          for (int t = 0; t < steps_n; ++t)
-            umma_bf16(d, make_smem_desc(qb + (t >> 2) * LA_QPANEL + (t & 3) * 32, 16, 1024),
-                      make_smem_desc(kb + (t >> 2) * KPANEL + (t & 3) * 32, 16, 1024), IDESC_S, t ? 1u : 0u);
-          const uint32_t qr = qb + p.pn * LA_QPANEL, kr = kb + p.pn * KPANEL;
-          for (int t = 0; t < steps_r; ++t)
-            umma_bf16(d, make_smem_desc(qr + (t >> 2) * LA_QPANEL + (t & 3) * 32, 16, 1024),
-                      make_smem_desc(kr + (t >> 2) * KPANEL + (t & 3) * 32, 16, 1024), IDESC_S, 1u);
+          uint32_t acc = 0u;
+          for (int c = 0; c < kp; ++c) {
+            const int left = c < p.pn ? steps_n - 4 * c : steps_r - 4 * (c - p.pn);
+            umma_bf16(d, qd, kd, IDESC_S, acc);
+            if (left > 1) umma_bf16(d, qd + 2, kd + 2, IDESC_S, 1u);
+            if (left > 2) umma_bf16(d, qd + 4, kd + 4, IDESC_S, 1u);
+            if (left > 3) umma_bf16(d, qd + 6, kd + 6, IDESC_S, 1u);
+            acc = 1u;
+            qd += LA_QPANEL >> 4;
+            kd += KPANEL >> 4;
+          }
           umma_commit(&bars->s_full[x]);
         };
         auto issue_pv = [&](int x, int j, bool first) {   // O_x += P_x V_j, P_x over the first BN / 2 columns of S_x
-          const uint32_t vb = aV + (j % p.vst) * v_bytes;
+          const uint64_t vd = dv0 + (((j % p.vst) * v_bytes) >> 4);
+          const uint32_t d = tmem_base + O_COL + x * O_WIDTH, a = tmem_base + x * BN;
 #pragma unroll
-          for (int t = 0; t < BN / 16; ++t)
-            umma_bf16_ts(tmem_base + O_COL + x * O_WIDTH, tmem_base + x * BN + t * 8, make_smem_desc(vb + t * 2048, KPANEL, 1024),
-                         idesc_o, (first && t == 0) ? 0u : 1u);
+          for (int t = 0; t < BN / 16; ++t) umma_bf16_ts(d, a + t * 8, vd + t * 128, idesc_o, (first && t == 0) ? 0u : 1u);
         };
         bool ok = mbar_wait(&bars->q_full, 0, abort_flag, p.err, ERR_WAIT_ATTN) &&
                   mbar_wait(&bars->k_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN);

@@ -99,11 +99,17 @@ class LayeredEngine(GraphRunner):
         y = skinny_linear(x, w, self._work[which], keep_f32=True, ld_out=(w.shape[0] + 7) // 8 * 8)
         return y, y.dtype == torch.float32
 
-    @staticmethod
-    def _splits(mix, B: int) -> int:
+    def _splits(self, mix, B: int) -> int:
         """Key splits of the decode attention: enough CTAs to fill the machine, at least 128 keys each."""
-        most = -(-mix.spec.window // 128)
-        return max(1, min(most, 16, (4 * 148) // max(1, B * mix.spec.heads)))
+        groups, fill = mix.spec.heads, 4 * 148          # generic kernel: a small CTA per head
+        if self.on_gpu and self.model.dtype == torch.bfloat16:
+            from ..ops import latent_attention as A
+
+            n = A.decode_group(mix.spec.heads, mix.spec.kv_rank, mix.layout.ld_lat)
+            if n:                                        # tensor-core kernel: one CTA per SM, n heads each
+                groups, fill = -(-mix.spec.heads // n), 148
+        tiles = min(mix.spec.window, self.max_len) // 128 + 1
+        return max(1, min(tiles, 32, fill // max(1, B * groups)))
 
     # -- generation --------------------------------------------------------------------------------------------------
     def prefill(self, rows: list, prompts: list) -> torch.Tensor:

@@ -8,8 +8,11 @@ CUDA-graphed recurrence, latent reuse and device-side KL exit, so the adaptive-d
 Pieces:
   * ``EngineBackend``  — a ``DecodeEngine`` on one GPU (bf16).
   * ``ModelBackend``   — the plain model ``generate`` path (any device; what the CPU tests use).
-  * ``BatchScheduler`` — thread-safe queue; a worker groups waiting requests that share prompt length and decoding
-                         options into one batch (up to ``max_batch``, waiting at most ``window_ms`` for company).
+  * ``LayeredBackend`` — a ``LayeredEngine`` (layered decoder models; prompts of any lengths in one batch, sampling).
+  * ``make_backend``   — the backend for a model.
+  * ``BatchScheduler`` — thread-safe queue; a worker groups waiting requests that share decoding options (and prompt
+                         length, unless the backend takes ragged batches) into one batch (up to ``max_batch``, waiting
+                         at most ``window_ms`` for company).
   * ``create_app``     — FastAPI app: ``/health``, ``/v1/models``, ``/v1/completions``.
 """
 from __future__ import annotations
@@ -33,10 +36,22 @@ class DecodeOptions:
     max_steps: Optional[int] = None
     continuous_compute: bool = False
     init_scale: float = 1.0                  # multiplies the sigma of the random start state (0 = deterministic)
+    do_sample: bool = False                  # sampling options: greedy decoding unless do_sample is set
+    temperature: Optional[float] = None
+    top_k: Optional[int] = None
+    top_p: Optional[float] = None
+    min_p: Optional[float] = None
+    repetition_penalty: Optional[float] = None
+
+    SAMPLING = ("do_sample", "temperature", "top_k", "top_p", "min_p", "repetition_penalty")
 
     def key(self):
         return (self.max_tokens, self.num_steps, self.criterion, self.exit_threshold, self.max_steps,
-                self.continuous_compute, self.init_scale)
+                self.continuous_compute, self.init_scale, *self.sampling().items())
+
+    def sampling(self) -> dict:
+        """The sampling options that are set."""
+        return {k: getattr(self, k) for k in self.SAMPLING if getattr(self, k) not in (None, False)}
 
 
 @dataclass
@@ -52,8 +67,13 @@ class Request:
     t_done: float = 0.0
 
 
+RAVEN_STOP_IDS = (65504, 65505, 65508)
+
+
 class ModelBackend:
     """Decoding through the model's own ``generate`` (greedy).  Works on CPU; batch rows are independent."""
+
+    ragged = False
 
     def __init__(self, model, max_batch: int = 8):
         self.model, self.max_batch = model.eval(), max_batch
@@ -64,7 +84,7 @@ class ModelBackend:
     def generate(self, prompts: list, opt: DecodeOptions):
         ids = torch.tensor(prompts, dtype=torch.long, device=self.device)
         kwargs = dict(max_new_tokens=opt.max_tokens, num_steps=opt.num_steps, continuous_compute=opt.continuous_compute,
-                      init_scale=opt.init_scale)
+                      init_scale=opt.init_scale, **opt.sampling())
         if opt.criterion:
             kwargs.update(criterion=opt.criterion, exit_threshold=opt.exit_threshold)
         kwargs = {k: v for k, v in kwargs.items() if v is not None}
@@ -77,6 +97,8 @@ class EngineBackend:
     """The native decode engine on one GPU.  The engine's buffers are sized for ``max_batch`` rows; smaller batches are
     padded by repeating the first prompt and the padding rows are dropped from the result."""
 
+    ragged = False
+
     def __init__(self, model, max_batch: int = 8, max_len: int = 4096, max_steps: int | None = None,
                  cache_lookup_strategy: str = "full"):
         from .decode import DecodeEngine
@@ -88,6 +110,8 @@ class EngineBackend:
 
     @torch.no_grad()
     def generate(self, prompts: list, opt: DecodeOptions):
+        if opt.sampling():
+            raise ValueError("the recurrent decode engine decodes greedily")
         rows = prompts + [prompts[0]] * (self.max_batch - len(prompts))
         ids = torch.tensor(rows, dtype=torch.long, device=self.device)
         tokens, stats = self.engine.generate(ids, opt.max_tokens, num_steps=opt.num_steps, criterion=opt.criterion,
@@ -102,8 +126,46 @@ class EngineBackend:
         return [tokens[i, P:].tolist() for i in range(len(prompts))], steps
 
 
+class LayeredBackend:
+    """The engine of the layered decoder models: prompts of a batch may differ in length; greedy or sampled."""
+
+    ragged = True
+
+    def __init__(self, model, max_batch: int = 8, max_len: int = 4096, stop_ids=()):
+        from .layered import LayeredEngine
+
+        self.engine = LayeredEngine(model, max_batch=max_batch, max_len=max_len)
+        self.max_batch, self.device, self.stop_ids = max_batch, self.engine.dev, tuple(stop_ids)
+        self.name = "layered-engine"
+
+    @torch.no_grad()
+    def generate(self, prompts: list, opt: DecodeOptions):
+        if opt.num_steps is not None or opt.criterion or opt.max_steps is not None or opt.continuous_compute:
+            raise ValueError("this model has no recurrence options")
+        outs = self.engine.generate(prompts, opt.max_tokens, stop_ids=self.stop_ids, **opt.sampling())
+        if self.device.type == "cuda":
+            from ..ops import cuda as K
+
+            status = K.check_device_status()
+            if status:
+                raise RuntimeError(f"decode kernels reported device status {status}")
+        return outs, None
+
+
+def make_backend(model, max_batch: int = 8, max_len: int = 4096, max_steps: int | None = None,
+                 cache_lookup_strategy: str = "full", stop_ids=None):
+    """The backend that serves ``model`` on the device it lies on."""
+    from ..models.layered import LayeredForCausalLM
+
+    if isinstance(model, LayeredForCausalLM):
+        return LayeredBackend(model, max_batch, max_len, stop_ids or ())
+    if next(model.parameters()).is_cuda:
+        return EngineBackend(model, max_batch, max_len, max_steps, cache_lookup_strategy)
+    return ModelBackend(model, max_batch)
+
+
 class BatchScheduler:
-    def __init__(self, backend, window_ms: float = 3.0, stop_ids=(65504, 65505, 65508)):
+    def __init__(self, backend, window_ms: float = 3.0, stop_ids=RAVEN_STOP_IDS):
         self.backend, self.window = backend, window_ms / 1e3
         self.stop_ids = set(stop_ids)
         self.q: "queue.Queue[Request]" = queue.Queue()
@@ -134,7 +196,8 @@ class BatchScheduler:
                 r = self.q.get(timeout=max(0.0, deadline - time.time()))
             except queue.Empty:
                 break
-            same = len(r.prompt_ids) == len(first.prompt_ids) and r.options.key() == first.options.key()
+            same = (self.backend.ragged or len(r.prompt_ids) == len(first.prompt_ids)) and \
+                r.options.key() == first.options.key()
             (batch if same else rest).append(r)
         for r in rest:  # incompatible requests go back, in order, for the next round
             self.q.put(r)
@@ -196,7 +259,8 @@ def handle_completion(scheduler: BatchScheduler, body: dict, tokenizer=None, mod
     opt = DecodeOptions(max_tokens=int(body.get("max_tokens", 64)), num_steps=body.get("num_steps"),
                         criterion=body.get("criterion"), exit_threshold=float(body.get("exit_threshold", 5e-4)),
                         max_steps=body.get("max_steps"), continuous_compute=bool(body.get("continuous_compute", False)),
-                        init_scale=float(body.get("init_scale", 1.0)))
+                        init_scale=float(body.get("init_scale", 1.0)),
+                        **{k: body[k] for k in DecodeOptions.SAMPLING if body.get(k) is not None})
     req = scheduler.submit(ids, opt)
     if not req.done.wait(timeout_s):
         raise TimeoutError("generation timed out")

@@ -297,8 +297,8 @@ def ring_attention(L: LatentLayout, inp: torch.Tensor, w_kv: torch.Tensor, norm_
     latents to values and gate -> [B, heads * vdim]."""
     B, hd, cap = inp.shape[0], L.dim + L.rot, cache.shape[1]
     assert cap >= window or not bool(inp.is_cuda), "ring shorter than the window"
-    w_uk, w_uv = w_kv[:L.heads * L.dim], w_kv[L.off_v:L.off_v + L.heads * L.vdim]
     if not inp.is_cuda:
+        w_uk, w_uv = w_kv[:L.heads * L.dim, :L.rank], w_kv[L.off_v:L.off_v + L.heads * L.vdim, :L.rank]
         p, r = pos.long(), row.long()
         cos, sin = rope[0][p], rope[1][p]
         if L.own:
@@ -314,21 +314,44 @@ def ring_attention(L: LatentLayout, inp: torch.Tensor, w_kv: torch.Tensor, norm_
         o = ref.window_attention(ql.to(dtype), lat, lat[..., :L.rank], back <= p[:, None], scale)
         o = torch.einsum("bhr,hvr->bhv", o, w_uv.float().unflatten(0, (L.heads, L.vdim))).flatten(1)
         return (o * torch.sigmoid(inp[:, L.off_g:L.off_g + o.shape[1]].float())).to(dtype)
+    absorb, attend, expand = ring_attention_pieces(L, inp, w_kv, norm_w, eps, rope, pos, row, cache, window, scale, splits, dtype)
+    absorb()
+    attend()
+    return expand()
+
+
+def ring_attention_pieces(L: LatentLayout, inp, w_kv, norm_w, eps: float, rope, pos, row, cache, window: int, scale: float, splits: int,
+                          dtype):
+    """The three launches of ``ring_attention`` on a GPU as callables (the last returns the result)."""
     k = _k()
-    dev = inp.device
+    B, dev, cap, f32 = inp.shape[0], inp.device, cache.shape[1], int(dtype == F32)
+    w_uk, w_uv = w_kv[:L.heads * L.dim], w_kv[L.off_v:L.off_v + L.heads * L.vdim]
     qlat = torch.empty(B, L.heads, L.ld_lat, dtype=dtype, device=dev)
-    s = _row_struct(L, inp, norm_w, eps, rope, pos, row, cap)
-    f32 = int(dtype == F32)
-    k.K._check(k.absorb(inp.data_ptr(), C.byref(s), w_uk.data_ptr(), w_kv.stride(0), cache.data_ptr(), qlat.data_ptr(), B, _f32(inp),
-                        f32, k.K._stream()), "latent_absorb")
     part_o = torch.empty(B, L.heads, splits, L.rank, dtype=F32, device=dev)
     part_ml = torch.empty(B, L.heads, splits, 2, dtype=F32, device=dev)
-    a = _WindowAttn(L.heads, L.ld_lat, 0, L.rank, window, splits, scale, L.heads * L.ld_lat, L.ld_lat, L.ld_lat, 0, 0, L.ld_lat, 0,
-                    0, 0, pos.data_ptr(), row.data_ptr(), cap, 0, 0, part_o.data_ptr(), part_ml.data_ptr())
-    k.K._check(k.attn(qlat.data_ptr(), cache.data_ptr(), 0, cache.data_ptr(), 0, 0, C.byref(a), B, f32, k.K._stream()),
-               "window_attention")
     out = torch.empty(B, L.ld_o, dtype=dtype, device=dev)[:, :L.heads * L.vdim]
     gate = inp[:, L.off_g:]
-    k.K._check(k.expand(part_o.data_ptr(), part_ml.data_ptr(), splits, w_uv.data_ptr(), w_kv.stride(0), gate.data_ptr(), inp.stride(0),
-                        out.data_ptr(), out.stride(0), B, L.heads, L.rank, L.vdim, _f32(inp), f32, k.K._stream()), "latent_expand")
-    return out
+
+    def absorb():
+        s = _row_struct(L, inp, norm_w, eps, rope, pos, row, cap)
+        k.K._check(k.absorb(inp.data_ptr(), C.byref(s), w_uk.data_ptr(), w_kv.stride(0), cache.data_ptr(), qlat.data_ptr(), B, _f32(inp),
+                            f32, k.K._stream()), "latent_absorb")
+
+    def attend():
+        if dtype == BF16:
+            from . import latent_attention as A
+
+            if A.decode_supported(L, cap):
+                A.ring_attention(L, qlat, cache, pos, row, part_o, part_ml, window, splits, scale)
+                return
+        a = _WindowAttn(L.heads, L.ld_lat, 0, L.rank, window, splits, scale, L.heads * L.ld_lat, L.ld_lat, L.ld_lat, 0, 0, L.ld_lat, 0,
+                        0, 0, pos.data_ptr(), row.data_ptr(), cap, 0, 0, part_o.data_ptr(), part_ml.data_ptr())
+        k.K._check(k.attn(qlat.data_ptr(), cache.data_ptr(), 0, cache.data_ptr(), 0, 0, C.byref(a), B, f32, k.K._stream()),
+                   "window_attention")
+
+    def expand():
+        k.K._check(k.expand(part_o.data_ptr(), part_ml.data_ptr(), splits, w_uv.data_ptr(), w_kv.stride(0), gate.data_ptr(), inp.stride(0),
+                            out.data_ptr(), out.stride(0), B, L.heads, L.rank, L.vdim, _f32(inp), f32, k.K._stream()), "latent_expand")
+        return out
+
+    return absorb, attend, expand

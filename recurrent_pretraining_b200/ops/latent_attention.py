@@ -1,5 +1,5 @@
-"""Binding of the tensor-core kernel for windowed latent attention over a packed step's key stream
-(``csrc/latent_attention.cu``)."""
+"""Bindings of the tensor-core kernels of windowed latent attention: over a packed step's key stream
+(``csrc/latent_attention.cu``) and, for decode steps, over the ring cache (``csrc/latent_decode.cu``)."""
 from __future__ import annotations
 
 import ctypes as C
@@ -12,6 +12,8 @@ from . import cuda as K
 _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
 _supported = K._sig("b200_latent_attention_supported", [_i, _i, _i])
 _attn = K._sig("b200_latent_attention", [_vp] * 7 + [_i] * 13 + [_f, _vp, _vp])
+_decode_group = K._sig("b200_latent_decode_group", [_i, _i, _i])
+_decode = K._sig("b200_latent_decode", [_vp] * 6 + [_i] * 8 + [_f, _vp, _vp])
 
 TILE = 256   # queries per CTA
 
@@ -39,3 +41,21 @@ def stream_attention(L, inp, kv, stream, layout, window: int, scale: float, out)
                    out.data_ptr(), tiles.data_ptr(), tiles.shape[0], inp.shape[0], kv.shape[0], L.heads, L.dim, L.rot, L.vdim,
                    inp.stride(0), kv.stride(0), stream.stride(0), inp.stride(0), out.stride(0), min(window, 2**30), scale, K._stream(),
                    K.err_word(inp.device).data_ptr()), "latent_attention")
+
+
+@lru_cache(None)
+def decode_group(heads: int, rank: int, ld_lat: int) -> int:
+    """Heads per CTA of the decode kernel; 0: sizes it does not take (the generic kernel runs)."""
+    return int(_decode_group(heads, rank, ld_lat))
+
+
+def decode_supported(L, cap: int) -> bool:
+    return cap % 128 == 0 and decode_group(L.heads, L.rank, L.ld_lat) > 0
+
+
+def ring_attention(L, qlat, cache, pos, row, part_o, part_ml, window: int, splits: int, scale: float) -> None:
+    """Unnormalised partials [B, H, splits, rank] and (max, sum) of the newest token of every row against its ring."""
+    assert qlat.is_contiguous() and cache.is_contiguous() and cache.shape[2] == L.ld_lat
+    K._check(_decode(qlat.data_ptr(), cache.data_ptr(), pos.data_ptr(), row.data_ptr(), part_o.data_ptr(), part_ml.data_ptr(),
+                     qlat.shape[0], L.heads, L.rank, L.ld_lat, cache.shape[0], cache.shape[1], window, splits, scale, K._stream(),
+                     K.err_word(qlat.device).data_ptr()), "latent_decode")

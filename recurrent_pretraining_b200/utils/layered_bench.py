@@ -1,0 +1,353 @@
+"""Prefill and decode throughput of the layered decoder models beside the recurrent model at equal size, and the time of
+every kernel of a layer against its roofline.
+
+``python -m recurrent_pretraining_b200.utils.layered_bench [--shapes gasovik-1b,gasovik-core-5280] [--ops-only]``.
+Random weights.  Model runs: CUDA events around whole prefill / decode calls of the two engines (graph-replayed decode).
+Kernels: CUDA events around single calls on the shapes of one layer, L2 flushed in between, median.  The comparison
+model is the depth-recurrent model run for one recurrence: as many layers of the same width, head count and value
+size, with a feed-forward that gives the same number of parameters per layer."""
+from __future__ import annotations
+
+import argparse
+import json
+import os
+
+import torch
+
+ROOT = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+
+
+def peaks() -> tuple:
+    """(bytes/s, FLOP/s) measured on this machine type: copy bandwidth and bf16 GEMM rate."""
+    try:
+        p = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12
+    except Exception:
+        return 6.65e12, 1.59e15
+
+
+class Timer:
+    def __init__(self):
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+        self.rows: list = []
+
+    def op(self, name: str, fn, nbytes: float, flops: float, iters: int = 12) -> None:
+        bw, fl = peaks()
+        for _ in range(3):
+            fn()
+        times = []
+        for _ in range(iters):
+            self.flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            times.append(a.elapsed_time(b) * 1e3)
+        us = sorted(times)[len(times) // 2]
+        floor = max(nbytes / bw, flops / fl) * 1e6
+        self.rows.append({"op": name, "us": round(us, 2), "roofline_us": round(floor, 2), "fraction": round(floor / us, 3),
+                          "bound": "memory" if nbytes / bw > flops / fl else "tensor"})
+
+    def take(self) -> list:
+        rows, self.rows = self.rows, []
+        return rows
+
+
+def time_calls(fn, iters: int = 5) -> float:
+    """Milliseconds per call."""
+    fn()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(iters):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / iters
+
+
+def closest_model(cfg):
+    """The recurrent model, one recurrence deep, with the layer count, width, heads and per-layer parameters of ``cfg``."""
+    from ..models.hf import RavenForCausalLM
+    from ..models.hf_config import RavenConfig
+
+    n, E = len(cfg.layers), cfg.width
+    a = cfg.layers[0].mixer
+    per_layer = (cfg.param_count() - 2 * cfg.vocab * E) / n
+    ff = max(256, int((per_layer - 4 * E * E) / (3 * E)) // 64 * 64)
+    core = max(1, n // 2)
+    pre = (n - core) // 2
+    rc = RavenConfig(n_embd=E, n_heads=a.heads, n_layers=n, block_size=16384, vocab_size=cfg.vocab, intermediate_size=ff,
+                     n_layers_in_prelude=max(1, pre), n_layers_in_recurrent_block=core, n_layers_in_coda=n - core - pre,
+                     mean_recurrence=1)
+    torch.manual_seed(0)
+    with torch.device("cuda"):
+        return RavenForCausalLM(rc).to(torch.bfloat16).eval()
+
+
+# ------------------------------------------------------------------------------------------
+# single kernels
+# ------------------------------------------------------------------------------------------
+def visible_pairs(seqs, window: int) -> float:
+    return float(sum(sum(min(i + 1, window) for i in range(n)) for n in seqs))
+
+
+def layer_ops_prefill(model, seqs: list, t: Timer) -> list:
+    """Kernels of one layer (with its own latents) of a packed step of fresh prompts ``seqs``."""
+    from ..models.layered import PackedStep
+    from ..ops import latent as ops
+
+    cfg = model.config
+    layer = model.layers[0]
+    mix, a, L, E = layer.mix, layer.mix.spec, layer.mix.layout, cfg.width
+    T = sum(seqs)
+    cache = model.new_cache(len(seqs), max(seqs))
+    step = PackedStep([(r, 0, [1] * n) for r, n in enumerate(seqs)], "cuda")
+    lay = step.layout(cfg.latent_windows()[0] - 1)
+    x = torch.randn(T, E, device="cuda")
+    xb = x.bfloat16()
+    stream = torch.empty(T, L.ld_lat, dtype=torch.bfloat16, device="cuda")
+    inp = ops.linear(xb, mix.w_in[:, :E])
+    rope = cache.rope[a.rot]
+    ops.latent_prep_(L, inp, mix.latent_norm, mix.eps, rope, step, lay.sidx, cache.data[0], stream)
+    kv = ops.linear(stream[:, :a.kv_rank], mix.w_kv[:, :a.kv_rank])
+    o = ops.stream_attention(L, inp, kv, stream, step, lay, a.window, a.scale)
+    out = ops.linear(o, mix.w_o[:, :a.heads * a.vdim])
+
+    def gemm(name, fn, M, N, K):
+        t.op(name, fn, 2.0 * (M * N + M * K + N * K), 2.0 * M * N * K)
+
+    gemm("q|gate|latent projection", lambda: ops.linear(xb, mix.w_in[:, :E]), T, L.width_in, E)
+    t.op("latent_prep", lambda: ops.latent_prep_(L, inp, mix.latent_norm, mix.eps, rope, step, lay.sidx, cache.data[0], stream),
+         2.0 * T * (2 * a.heads * a.rot_dim + 3 * L.ld_lat), 0)
+    gemm("key|value up-projection", lambda: ops.linear(stream[:, :a.kv_rank], mix.w_kv[:, :a.kv_rank]), T, L.width_kv, a.kv_rank)
+    t.op("latent_attention", lambda: ops.stream_attention(L, inp, kv, stream, step, lay, a.window, a.scale),
+         2.0 * T * (a.heads * (a.dim + a.rot_dim + 2 * a.vdim) + L.width_kv + a.rot_dim),
+         2.0 * visible_pairs(seqs, a.window) * a.heads * (a.dim + a.rot_dim + a.vdim))
+    gemm("output projection", lambda: ops.linear(o, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)
+    t.op("rms_residual", lambda: ops.rms_residual_(x, out, None, layer.norm1, 1e-6, 1e-6, torch.bfloat16), T * E * 12.0, 0)
+    if layer.mlp is not None:
+        ff = layer.mlp.spec.ff
+        h = ops.linear(xb, layer.mlp.w_up[:, :E], layer.mlp.b_up, "relu2")
+        gemm("up projection + bias + relu^2", lambda: ops.linear(xb, layer.mlp.w_up[:, :E], layer.mlp.b_up, "relu2"), T, ff, E)
+        gemm("down projection", lambda: ops.linear(h, layer.mlp.w_down[:, :ff]), T, E, ff)
+    return t.take()
+
+
+def layer_ops_decode(model, B: int, context: int, t: Timer) -> list:
+    from ..engine.layered import LayeredEngine
+    from ..ops import latent as ops
+
+    cfg = model.config
+    layer = model.layers[0]
+    mix, a, L, E = layer.mix, layer.mix.spec, layer.mix.layout, cfg.width
+    eng = LayeredEngine(model, B, context + 1, use_graphs=False)
+    cache = eng.cache
+    for d in cache.data.values():
+        d.normal_()
+    pos = torch.full((B,), context, dtype=torch.int32, device="cuda")
+    row = torch.arange(B, dtype=torch.int32, device="cuda")
+    x = torch.randn(B, E, device="cuda")
+    xb = x.bfloat16()
+    inp, _ = eng._dense(xb, mix.w_in[:, :E], 0)
+    inp = inp.clone()
+    work = torch.zeros(B, max(E, layer.mlp.spec.ff), dtype=torch.float32, device="cuda")
+    pieces = ops.ring_attention_pieces(L, inp, mix.w_kv, mix.latent_norm, mix.eps, cache.rope[a.rot], pos, row, cache.data[0],
+                                       min(a.window, cache.data[0].shape[1]), a.scale, eng._splits(mix, B), torch.bfloat16)
+
+    def skinny(name, xin, w):
+        N, K = w.shape
+        t.op(name, lambda: eng._dense(xin, w, 1), 2.0 * (N * K + B * K + B * N), 2.0 * B * N * K)
+
+    skinny("q|gate|latent projection", xb, mix.w_in[:, :E])
+    keys = min(a.window, context + 1)
+    absorb, attend, expand = pieces
+    t.op("latent_absorb", absorb, 2.0 * (a.heads * a.dim * a.kv_rank + B * (a.heads * (a.dim + a.rot_dim) * 2 + a.heads * L.ld_lat)),
+         2.0 * B * a.heads * a.dim * a.kv_rank)
+    t.op("latent decode attention", attend, 2.0 * B * (keys * L.ld_lat + a.heads * (L.ld_lat + a.kv_rank)),
+         2.0 * B * a.heads * keys * (L.ld_lat + a.kv_rank))
+    t.op("latent_expand", expand, 2.0 * (a.heads * a.vdim * a.kv_rank + B * a.heads * (a.kv_rank * 2 + 2 * a.vdim)),
+         2.0 * B * a.heads * a.vdim * a.kv_rank)
+    o = torch.randn(B, a.heads * a.vdim, device="cuda").bfloat16()
+    skinny("output projection", o, mix.w_o[:, :a.heads * a.vdim])
+    acc = work[:, :E]
+    t.op("rms_residual", lambda: ops.rms_residual_(x, acc, None, layer.norm1, 1e-6, 1e-6, torch.bfloat16), B * E * 14.0, 0)
+    if layer.mlp is not None:
+        ff = layer.mlp.spec.ff
+        skinny("up projection", xb, layer.mlp.w_up[:, :E])
+        t.op("bias + relu^2", lambda: ops.bias_act(work[:, :ff], layer.mlp.b_up, "relu2", torch.bfloat16), B * ff * 6.0, 0)
+        skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), layer.mlp.w_down[:, :ff])
+    return t.take()
+
+
+def closest_ops_prefill(model, B: int, S: int, t: Timer) -> list:
+    from ..ops import attention as A
+    from ..ops import cuda as K
+
+    c = model.config
+    block = model.transformer.core_block[0]
+    H, D, E, T = c.n_heads, c.head_dim, c.n_embd, B * S
+    x = torch.randn(T, E, device="cuda").bfloat16()
+    cos, sin = model._rope(S)
+
+    def gemm(name, fn, M, N, Kd):
+        t.op(name, fn, 2.0 * (M * N + M * Kd + N * Kd), 2.0 * M * N * Kd)
+
+    qkv = K.gemm_nt(x, block.attn.Wqkv.weight)
+    gemm("qkv projection", lambda: K.gemm_nt(x, block.attn.Wqkv.weight), T, 3 * H * D, E)
+    q3 = qkv.view(B, S, -1)
+    bias = block.attn.qk_bias
+    r = K.rope_fwd(q3, bias, cos, sin, H, H, D)
+    t.op("rope", lambda: K.rope_fwd(q3, bias, cos, sin, H, H, D), 2.0 * 2 * T * 3 * H * D, 0)
+    t.op("attention", lambda: A.fwd(r, H, H, D, D ** -0.5), 2.0 * T * 4 * H * D, 2.0 * visible_pairs([S] * B, S) * H * 2 * D)
+    o = torch.randn(T, H * D, device="cuda").bfloat16()
+    gemm("output projection", lambda: K.gemm_nt(o, block.attn.proj.weight), T, E, H * D)
+    t.op("add + rmsnorm", lambda: K.add_rmsnorm_fwd(o, x, block.norm_2.weight, 1e-6), 2.0 * 4 * T * E, 0)
+    I = block.mlp.proj.weight.shape[1]
+    g = torch.randn(T, I, device="cuda").bfloat16()
+    gemm("gate-up projection + swiglu", lambda: K.gemm(x, block.mlp.fc.weight, out_mode=K.OUT_SWIGLU), T, 2 * I, E)
+    gemm("down projection", lambda: K.gemm_nt(g, block.mlp.proj.weight), T, E, I)
+    return t.take()
+
+
+def closest_ops_decode(model, B: int, context: int, t: Timer) -> list:
+    from ..engine import decode as D_
+    from ..engine.decode import DecodeEngine
+    from ..ops import cuda as K
+
+    c = model.config
+    block = model.transformer.core_block[0]
+    H, D, E = c.n_heads, c.head_dim, c.n_embd
+    eng = DecodeEngine(model, B, context + 1, num_steps=1, use_graphs=False)
+    eng.pos.fill_(context)
+    eng.lens.fill_(context + 1)
+    kc, vc = eng.cache.k[0].normal_(), eng.cache.v[0].normal_()
+    x = torch.randn(B, E, device="cuda").bfloat16()
+    I = block.mlp.proj.weight.shape[1]
+
+    def skinny(name, xin, w):
+        N, Kd = w.shape
+        t.op(name, lambda: eng._linear(xin, w, keep_f32=True), 2.0 * (N * Kd + B * Kd + B * N), 2.0 * B * N * Kd)
+
+    skinny("qkv projection", x, block.attn.Wqkv.weight)
+    qkv = torch.randn(B, 3 * H * D, device="cuda").bfloat16()
+    q = torch.empty(B, H * D, dtype=torch.bfloat16, device="cuda")
+    o = torch.empty_like(q)
+    t.op("rope_append", lambda: K._check(D_._rope_append(
+        qkv.data_ptr(), 0, eng.cos.data_ptr(), eng.sin.data_ptr(), eng.pos.data_ptr(), q.data_ptr(), kc.data_ptr(), vc.data_ptr(), B, H, H, D,
+        eng.Lmax, K._stream(), 0), "rope_append"), 2.0 * B * 6 * H * D, 0)
+    t.op("decode attention", lambda: K._check(D_._decode_attn(
+        q.data_ptr(), kc.data_ptr(), vc.data_ptr(), eng.lens.data_ptr(), o.data_ptr(), eng.part_o.data_ptr(), eng.part_ml.data_ptr(), B, H, H, D,
+        eng.Lmax, eng.splits, D ** -0.5, K._stream()), "decode_attention"), 2.0 * B * H * D * (2 * (context + 1) + 2), 4.0 * B * H * D * context)
+    skinny("output projection", o, block.attn.proj.weight)
+    t.op("add + rmsnorm pair", lambda: eng._pair(o, x, block.norm_2, block.norm_3), 2.0 * 4 * B * E, 0)
+    skinny("gate-up projection", x, block.mlp.fc.weight)
+    gu = torch.randn(B, 2 * I, device="cuda")
+    g = torch.empty(B, I, dtype=torch.bfloat16, device="cuda")
+    t.op("swiglu", lambda: K._check(D_._swiglu_acc(gu.data_ptr(), g.data_ptr(), B, I, K._stream()), "swiglu_acc"), B * I * 18.0, 0)
+    skinny("down projection", torch.randn(B, I, device="cuda").bfloat16(), block.mlp.proj.weight)
+    return t.take()
+
+
+# ------------------------------------------------------------------------------------------
+# whole models
+# ------------------------------------------------------------------------------------------
+def model_rates(cfg, prompt: int, new: int, batches) -> dict:
+    from ..engine.decode import DecodeEngine
+    from ..engine.layered import LayeredEngine
+    from ..models.layered import LayeredForCausalLM
+
+    out: dict = {"prompt": prompt, "new_tokens": new, "ours": {}, "closest": {}}
+    model = LayeredForCausalLM(cfg, torch.bfloat16, "cuda").init_weights()
+    out["ours"]["parameters"] = cfg.param_count()
+    for B in batches:
+        eng = LayeredEngine(model, B, prompt + new + 1, prefill_tokens=65536)
+        prompts = torch.randint(0, cfg.vocab, (B, prompt)).tolist()
+
+        def pre():
+            rows = [eng.open() for _ in prompts]
+            eng.prefill(rows, prompts)
+            for r in rows:
+                eng.close(r)
+
+        eng.generate(prompts, 4)
+        t_pre, t_all = time_calls(pre, 3), time_calls(lambda: eng.generate(prompts, new), 2)
+        out["ours"][str(B)] = {"prefill_tok_s": round(B * prompt / t_pre * 1e3), "decode_tok_s": round(B * (new - 1) / (t_all - t_pre) * 1e3, 1),
+                               "decode_ms_per_token": round((t_all - t_pre) / (new - 1), 3), "cache_mib": round(eng.cache.get_memory_usage(), 1)}
+        del eng
+    del model
+    torch.cuda.empty_cache()
+    model = closest_model(cfg)
+    out["closest"]["parameters"] = sum(p.numel() for p in model.parameters())
+    for B in batches:
+        eng = DecodeEngine(model, B, prompt + new + 1, num_steps=1)
+        ids = torch.randint(0, cfg.vocab, (B, prompt), device="cuda")
+        if B * prompt > 65536:
+            continue                      # its prefill returns the logits of every position
+        eng.generate(ids, 4, init_scale=0.0)
+        t_pre = time_calls(lambda: eng.prefill(ids, 1, 0.0), 3)
+        t_all = time_calls(lambda: eng.generate(ids, new, init_scale=0.0), 2)
+        out["closest"][str(B)] = {"prefill_tok_s": round(B * prompt / t_pre * 1e3), "decode_tok_s": round(B * (new - 1) / (t_all - t_pre) * 1e3, 1),
+                                  "decode_ms_per_token": round((t_all - t_pre) / (new - 1), 3),
+                                  "cache_mib": round(eng.cache.get_memory_usage(), 1)}
+        del eng
+    return out
+
+
+def run(shapes=("gasovik-1b", "gasovik-core-5280"), batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
+    from ..models.layered import LayeredForCausalLM
+    from ..models.layered_config import LayeredConfig
+    from ..ops import cuda as K
+
+    rec: dict = {}
+    for name in shapes:
+        cfg = LayeredConfig.from_name(name)
+        r: dict = {}
+        if not ops_only:
+            r["models"] = model_rates(cfg, prompt, new, batches)
+            torch.cuda.empty_cache()
+        t = Timer()
+        one = LayeredConfig(cfg.architecture, 1024, cfg.width, cfg.norm_eps, cfg.residual_mult, cfg.layers[:1])
+        model = LayeredForCausalLM(one, torch.bfloat16, "cuda").init_weights()
+        S = 4096
+        r["prefill_ops"] = {"tokens": S, "ours": layer_ops_prefill(model, [S], t)}
+        r["decode_ops"] = {f"batch {B}": {"context": S, "ours": layer_ops_decode(model, B, S, t)} for B in (1, 8, 64)}
+        del model
+        ref = closest_model(LayeredConfig(cfg.architecture, 1024, cfg.width, cfg.norm_eps, cfg.residual_mult, cfg.layers[:3]))
+        r["prefill_ops"]["closest"] = closest_ops_prefill(ref, 1, S, t)
+        for B in (1, 8, 64):
+            r["decode_ops"][f"batch {B}"]["closest"] = closest_ops_decode(ref, B, S, t)
+            torch.cuda.empty_cache()
+        del ref
+        rec[name] = r
+        torch.cuda.empty_cache()
+    rec["device_status"] = K.check_device_status()
+    return rec
+
+
+def main():
+    ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
+    ap.add_argument("--shapes", default="gasovik-1b,gasovik-core-5280")
+    ap.add_argument("--batches", default="1,8,32")
+    ap.add_argument("--prompt", type=int, default=2048)
+    ap.add_argument("--new", type=int, default=128)
+    ap.add_argument("--ops-only", action="store_true")
+    args = ap.parse_args()
+    rec = run(args.shapes.split(","), [int(b) for b in args.batches.split(",")], args.prompt, args.new, args.ops_only)
+    for name, r in rec.items():
+        if not isinstance(r, dict):
+            print(name, r)
+            continue
+        if "models" in r:
+            for who in ("ours", "closest"):
+                print(name, who, json.dumps(r["models"][who]))
+        for title, block in [("prefill", r["prefill_ops"])] + [(f"decode {b}", d) for b, d in r["decode_ops"].items()]:
+            for who in ("ours", "closest"):
+                for row in block[who]:
+                    print(f"{name:18s} {title:16s} {who:8s} {row['op']:32s} {row['us']:9.2f} us  floor {row['roofline_us']:8.2f}  "
+                          f"{row['fraction']:.3f} {row['bound']}")
+
+
+if __name__ == "__main__":
+    main()

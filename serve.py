@@ -1,8 +1,10 @@
 #!/usr/bin/env python
-"""Serve a recurrent-depth model over HTTP with the native decode engine, one replica per GPU.
+"""Serve a model over HTTP with the native decode engines, one replica per GPU.
 
-    python serve.py --model /path/to/hf_folder --port 8000                # one GPU
+    python serve.py --model /path/to/model_folder --port 8000             # one GPU; the model class follows config.json
     python serve.py --model nebel-raven-3.5b --random-init --replicas 8   # 8 replicas on ports 8000..8007 + router on 7999
+    python serve.py --model gasovik-1b --random-init                      # a layered decoder shape
+    python serve.py --model /path/to/model_folder --prompt-ids 5,17,3 --max-tokens 32   # one completion, no server
 
 ``--replicas N`` starts N child processes (replica i pinned to GPU i via CUDA_VISIBLE_DEVICES) and a round-robin router
 in the parent: inference data parallelism, the deployment shape of the reference's vLLM recipe (vllm/README.md:19-24).
@@ -19,42 +21,46 @@ import urllib.request
 
 
 def load_model(name: str, random_init: bool, device, dtype):
-    import torch
-
-    from recurrent_pretraining_b200.models.hf import RavenForCausalLM
-    from recurrent_pretraining_b200.models.hf_config import RavenConfig
+    from recurrent_pretraining_b200.models import auto
 
     if os.path.isdir(name):
-        return RavenForCausalLM.from_pretrained(name, torch_dtype=dtype).to(device)
+        return auto.load_pretrained(name, dtype, device)
     if not random_init:
         raise SystemExit(f"{name!r} is not a local folder; pass --random-init to serve a registry shape with random weights")
-    from recurrent_pretraining_b200.config import ModelConfig
-
-    torch.manual_seed(0)
-    with torch.device(device):
-        model = RavenForCausalLM(RavenConfig.from_model_config(ModelConfig.from_name(name)))
-    return model.to(dtype)
+    return auto.random_model(name, dtype, device)
 
 
 def run_replica(args):
     import torch
-    import uvicorn
 
-    from recurrent_pretraining_b200.engine.server import BatchScheduler, EngineBackend, ModelBackend, create_app
+    from recurrent_pretraining_b200.engine.server import (RAVEN_STOP_IDS, BatchScheduler, create_app, handle_completion,
+                                                          make_backend)
 
     cuda = torch.cuda.is_available() and not args.cpu
     device = torch.device("cuda", 0) if cuda else torch.device("cpu")
-    model = load_model(args.model, args.random_init, device, torch.bfloat16 if cuda else torch.float32)
+    dtype = getattr(torch, args.dtype) if args.dtype else torch.bfloat16 if cuda else torch.float32
+    model = load_model(args.model, args.random_init, device, dtype)
     tokenizer = None
     if args.tokenizer:
         from recurrent_pretraining_b200.data.tokenizer import Tokenizer
 
         tokenizer = Tokenizer(args.tokenizer)
-    backend = (EngineBackend(model, args.max_batch, args.max_len, args.max_steps, args.cache_lookup_strategy)
-               if cuda else ModelBackend(model, args.max_batch))
-    sched = BatchScheduler(backend, window_ms=args.batch_window_ms)
-    uvicorn.run(create_app(sched, tokenizer, os.path.basename(args.model.rstrip("/"))), host=args.host, port=args.port,
-                log_level="warning")
+    stops = [int(x) for x in args.stop_ids.split(",") if x] if args.stop_ids is not None else None
+    backend = make_backend(model, args.max_batch, args.max_len, args.max_steps, args.cache_lookup_strategy, stops)
+    if stops is None:
+        stops = () if backend.ragged else RAVEN_STOP_IDS
+    sched = BatchScheduler(backend, window_ms=args.batch_window_ms, stop_ids=stops)
+    name = os.path.basename(args.model.rstrip("/"))
+    if args.prompt_ids is not None:
+        body = {"prompt": [int(t) for t in args.prompt_ids.split(",")], "max_tokens": args.max_tokens}
+        if args.temperature:
+            body.update(do_sample=True, temperature=args.temperature)
+        print(json.dumps(handle_completion(sched, body, tokenizer, name)), flush=True)
+        sched.close()
+        return
+    import uvicorn
+
+    uvicorn.run(create_app(sched, tokenizer, name), host=args.host, port=args.port, log_level="warning")
 
 
 def run_router(args, ports):
@@ -95,7 +101,7 @@ def run_router(args, ports):
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("--model", required=True, help="local HF folder or a registry shape name (with --random-init)")
+    ap.add_argument("--model", required=True, help="local model folder or a registry shape name (with --random-init)")
     ap.add_argument("--random-init", action="store_true")
     ap.add_argument("--tokenizer", default=None, help="local tokenizer folder (text prompts); token-id prompts need none")
     ap.add_argument("--host", default="127.0.0.1")
@@ -107,6 +113,11 @@ def main(argv=None):
     ap.add_argument("--cache-lookup-strategy", default="full")
     ap.add_argument("--batch-window-ms", type=float, default=3.0)
     ap.add_argument("--cpu", action="store_true", help="serve through model.generate on CPU (debug)")
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default=None, help="default: bfloat16 on a GPU, float32 on CPU")
+    ap.add_argument("--stop-ids", default=None, help="comma-separated stop token ids (default: the model family's)")
+    ap.add_argument("--prompt-ids", default=None, help="complete this comma-separated prompt once and exit")
+    ap.add_argument("--max-tokens", type=int, default=64, help="new tokens of --prompt-ids")
+    ap.add_argument("--temperature", type=float, default=0.0, help="sampling temperature of --prompt-ids (0: greedy)")
     ap.add_argument("--replica-index", type=int, default=None, help=argparse.SUPPRESS)
     args = ap.parse_args(argv)
     if args.replicas <= 1 or args.replica_index is not None:
