@@ -181,7 +181,7 @@ latent_prep_kernel(T* __restrict__ in, LatentRow L, const int* __restrict__ sidx
 // qlat[b, h, r] = sum_d W_uk[h * dim + d, r] q[b, h, d].
 constexpr int ABS_ROWS = 8, ABS_COLS = 128;
 template <typename TI, typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict__ w_uk, int ldw, T* __restrict__ cache,
                      T* __restrict__ qlat, int B) {
   pdl_trigger();
@@ -215,11 +215,11 @@ latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict
   id /= cols;
   const int h = id % L.H, b0 = (id / L.H) * ABS_ROWS;
   const int nb = min(ABS_ROWS, B - b0);
-  float* qs = sm;                                  // [ABS_ROWS][dim]
+  float* qs = sm;                                  // [dim][ABS_ROWS]
   float* part = sm + ABS_ROWS * ((L.dim + 3) & ~3);   // [8][ABS_ROWS][ABS_COLS]
   for (int i = threadIdx.x; i < ABS_ROWS * L.dim; i += 256) {
     const int b = i / L.dim, d = i - b * L.dim;
-    qs[i] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
+    qs[d * ABS_ROWS + b] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
   }
   __syncthreads();
   const int tx = threadIdx.x & 31, grp = threadIdx.x >> 5;   // four columns per thread, eight groups over d
@@ -231,20 +231,21 @@ latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict
     for (int k = 0; k < 4; ++k) acc[b][k] = 0.f;
   if (r < L.rank) {                                // weight rows are padded to eight: columns up to r + 3 exist
     const T* wp = w_uk + static_cast<size_t>(h) * L.dim * ldw + r;
-    for (int d0 = grp; d0 < L.dim; d0 += 128) {
-      float w[16][4];
+#pragma unroll 1
+    for (int d0 = grp; d0 < L.dim; d0 += 64) {
+      float w[8][4];
 #pragma unroll
-      for (int u = 0; u < 16; ++u)
+      for (int u = 0; u < 8; ++u)
         if (d0 + 8 * u < L.dim) ld4(wp + static_cast<size_t>(d0 + 8 * u) * ldw, w[u]);
 #pragma unroll
-      for (int u = 0; u < 16; ++u) {
+      for (int u = 0; u < 8; ++u) {
         if (d0 + 8 * u < L.dim) {
+          float q[8];
+          ld8(qs + (d0 + 8 * u) * ABS_ROWS, q);
 #pragma unroll
-          for (int b = 0; b < ABS_ROWS; ++b) {
-            const float q = qs[b * L.dim + d0 + 8 * u];
+          for (int b = 0; b < ABS_ROWS; ++b)
 #pragma unroll
-            for (int k = 0; k < 4; ++k) acc[b][k] += q * w[u][k];
-          }
+            for (int k = 0; k < 4; ++k) acc[b][k] += q[b] * w[u][k];
         }
       }
     }
@@ -286,7 +287,7 @@ struct WindowAttn {
   int cap;
   // stream form: normalised, gated output; ring form (splits > 0 partials): unnormalised fp32 partials
   int gate_ld, out_ld;
-  float* part_o;                  // [T, H, splits, vdim]
+  float* part_o;                  // [T, H, splits, vdim padded to eight]
   float* part_ml;                 // [T, H, splits, 2] (max in natural-log units, sum)
 };
 
@@ -363,7 +364,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
     for (int w = 0; w < 4; ++w) o += wgt[w] * os[w * A.vdim + d];
     if (A.part_o) {
       const size_t pi = (static_cast<size_t>(t) * A.H + h) * A.splits + split;
-      A.part_o[pi * A.vdim + d] = o;
+      A.part_o[pi * ((A.vdim + 7) & ~7) + d] = o;
       if (d == 0) { A.part_ml[2 * pi] = mm; A.part_ml[2 * pi + 1] = ll; }
     } else {
       const float g = sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + h * A.vdim + d));
@@ -394,7 +395,8 @@ __device__ __forceinline__ float warp_sum_many(float (&v)[N]) {
   return v[0];
 }
 
-// out[b, h * vdim + v] = sigmoid(gate) * sum_r W_uv[h * vdim + v, r] o[b, h, r], o = merged key splits.
+// out[b, h * vdim + v] = sigmoid(gate) * sum_r W_uv[h * vdim + v, r] o[b, h, r], o = merged key splits (partial rows are
+// padded to eight columns).
 // CTA: (head, 32 values, ROWS rows); a warp forms four values of all its rows at once.
 constexpr int EXP_COLS = 32;
 template <typename TI, typename T, int ROWS>
@@ -418,18 +420,27 @@ latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__
     wgt[warp][lane] = a / ll;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < ROWS * rs; i += 256) {
-    const int b = i / rs, r = i - b * rs;
-    float o = 0.f;
-    if (b < nb && r < rank) {
-      const float* p = part_o + (static_cast<size_t>(b0 + b) * H + h) * splits * rank + r;
-#pragma unroll 8
-      for (int s = 0; s < splits; ++s) {
-        const float w = wgt[b][s], x = p[static_cast<size_t>(s) * rank];
-        o += w != 0.f ? w * x : 0.f;               // an empty split's partial is not initialised
+  {
+    constexpr int WPR = 8 / ROWS;                  // warps per row
+    const int b = warp / WPR;
+    const float* p = part_o + (static_cast<size_t>(b0 + (b < nb ? b : 0)) * H + h) * splits * rs;
+    for (int r = 4 * (lane + 32 * (warp % WPR)); r < rs; r += 128 * WPR) {
+      float o[4] = {0.f, 0.f, 0.f, 0.f};
+      if (b < nb) {
+#pragma unroll 4
+        for (int s = 0; s < splits; ++s) {
+          const float w = wgt[b][s];
+          float x[4];
+          ld4(p + static_cast<size_t>(s) * rs + r, x);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) o[k] += w != 0.f ? w * x[k] : 0.f;   // an empty split's partial is not initialised
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (r + k >= rank) o[k] = 0.f;           // neither are the padding columns
       }
+      *reinterpret_cast<float4*>(os + b * rs + r) = make_float4(o[0], o[1], o[2], o[3]);
     }
-    os[i] = o;
   }
   __syncthreads();
   const int vw = v0 + warp * 4;

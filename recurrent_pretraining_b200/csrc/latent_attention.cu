@@ -34,6 +34,15 @@ struct LatentAttnParams {
   int* err;
 };
 
+// Position in a ring of `n` stages: stage index and the parity of the pass over the ring.
+struct RingPos {
+  int s = 0;
+  uint32_t ph = 0;
+  __device__ __forceinline__ void next(int n) {
+    if (++s == n) { s = 0; ph ^= 1; }
+  }
+};
+
 struct LatentAttnBars {
   uint64_t q_full;
   uint64_t k_full[LA_MAX_STAGES], k_empty[LA_MAX_STAGES], v_full[LA_MAX_STAGES], v_empty[LA_MAX_STAGES];
@@ -82,13 +91,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 
   auto load_q = [&](int x) {
     for (int c = 0; c < p.pn; ++c)
-      tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full, c * 64, h, q0 + x * LA_BM);
+      tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full, c * 64, q0 + x * LA_BM, h);
     for (int c = 0; c < p.pr; ++c)
-      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full, c * 64, h, q0 + x * LA_BM);
+      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full, c * 64, q0 + x * LA_BM, h);
   };
   auto load_k = [&](int j, int s) {
     mbar_expect_tx(&bars->k_full[s], k_bytes);
-    for (int c = 0; c < p.pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, h, kstart + j * BN);
+    for (int c = 0; c < p.pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, h);
     for (int c = 0; c < p.pr; ++c)
       tma_load_2d(sK + s * k_bytes + (p.pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
   };
@@ -129,10 +138,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     if (warp == 8) {
       if (lane == 0) {
         int issued = 1;
-        for (int j = 1; j < nmax; ++j) {
-          const int s = j % p.kst;
-          if (!mbar_wait(&bars->k_empty[s], ((j / p.kst) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
-          load_k(j, s);
+        RingPos k;
+        k.next(p.kst);
+        for (int j = 1; j < nmax; ++j, k.next(p.kst)) {
+          if (!mbar_wait(&bars->k_empty[k.s], k.ph ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
+          load_k(j, k.s);
           issued = j + 1;
         }
         // every issued load must land before the CTA exits
@@ -144,12 +154,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         }
       } else if (lane == 1) {
         int issued = 0;
-        for (int j = 0; j < nmax; ++j) {
-          const int s = j % p.vst;
-          if (!mbar_wait(&bars->v_empty[s], ((j / p.vst) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
+        RingPos v;
+        for (int j = 0; j < nmax; ++j, v.next(p.vst)) {
+          const int s = v.s;
+          if (!mbar_wait(&bars->v_empty[s], v.ph ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
           mbar_expect_tx(&bars->v_full[s], v_bytes);
           for (int c = 0; c < p.pv; ++c)
-            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, h, kstart + j * BN);
+            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, kstart + j * BN, h);
           issued = j + 1;
         }
         for (int j = max(0, issued - p.vst); j < issued; ++j) {
@@ -164,8 +175,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         const int steps_n = (p.dim + 15) >> 4, steps_r = (p.rot + 15) >> 4;
         // descriptors advance by their 16-byte-unit offsets: 2 per 16 K-major columns, 128 per 16 MN-major key rows
         const uint64_t dq0 = make_smem_desc(aQ, 16, 1024), dk0 = make_smem_desc(aK, 16, 1024), dv0 = make_smem_desc(aV, KPANEL, 1024);
-        auto issue_s = [&](int x, int j) {   // S_x = Q_x K_j^T
-          uint64_t qd = dq0 + ((x * q_bytes) >> 4), kd = dk0 + (((j % p.kst) * k_bytes) >> 4);
+        auto issue_s = [&](int x, int ks) {   // S_x = Q_x K^T, keys in stage ks
+          uint64_t qd = dq0 + ((x * q_bytes) >> 4), kd = dk0 + ((ks * k_bytes) >> 4);
           const uint32_t d = tmem_base + x * BN;
           uint32_t acc = 0u;
           for (int c = 0; c < kp; ++c) {
@@ -180,8 +191,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           }
           umma_commit(&bars->s_full[x]);
         };
-        auto issue_pv = [&](int x, int j, bool first) {   // O_x += P_x V_j, P_x over the first BN / 2 columns of S_x
-          const uint64_t vd = dv0 + (((j % p.vst) * v_bytes) >> 4);
+        auto issue_pv = [&](int x, int vs, bool first) {   // O_x += P_x V (stage vs), P_x over the first BN / 2 columns of S_x
+          const uint64_t vd = dv0 + ((vs * v_bytes) >> 4);
           const uint32_t d = tmem_base + O_COL + x * O_WIDTH, a = tmem_base + x * BN;
 #pragma unroll
           for (int t = 0; t < BN / 16; ++t) umma_bf16_ts(d, a + t * 8, vd + t * 128, idesc_o, (first && t == 0) ? 0u : 1u);
@@ -194,12 +205,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           if (je1 > 0 && jb1 == 0) issue_s(1, 0);
           umma_commit(&bars->k_empty[0]);
         }
-        for (int j = 0; j < nmax && ok; ++j) {
-          if (!mbar_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
-          if (j + 1 < nmax && !mbar_wait(&bars->k_full[(j + 1) % p.kst], ((j + 1) / p.kst) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) {
-            ok = false;
-            break;
-          }
+        RingPos k, v;                        // stages of key block j + 1 and value block j
+        for (int j = 0; j < nmax && ok; ++j, v.next(p.vst)) {
+          k.next(p.kst);
+          if (!mbar_wait(&bars->v_full[v.s], v.ph, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
+          if (j + 1 < nmax && !mbar_wait(&bars->k_full[k.s], k.ph, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
           tc_fence_after();
 #pragma unroll
           for (int x = 0; x < 2; ++x) {
@@ -207,14 +217,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
             if (j >= jb && j < je) {
               if (!mbar_wait(&bars->p_ready[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
               tc_fence_after();
-              issue_pv(x, j, j == jb);
+              issue_pv(x, v.s, j == jb);
               if (j + 1 == je) umma_commit(&bars->o_final[x]);
             }
-            if (j + 1 >= jb && j + 1 < je) issue_s(x, j + 1);
+            if (j + 1 >= jb && j + 1 < je) issue_s(x, k.s);
           }
           if (!ok) break;
-          umma_commit(&bars->v_empty[j % p.vst]);
-          if (j + 1 < nmax) umma_commit(&bars->k_empty[(j + 1) % p.kst]);
+          umma_commit(&bars->v_empty[v.s]);
+          if (j + 1 < nmax) umma_commit(&bars->k_empty[k.s]);
         }
       }
     }
@@ -345,7 +355,7 @@ typedef CUresult (*EncodeTiledFnL)(CUtensorMap*, CUtensorMapDataType, cuuint32_t
                                    const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// bf16 tensor [rows, (heads,) cols] with row pitch `ld` and head pitch `head` (elements); box: `box_rows` rows x 64 columns of
+// bf16 tensor [(heads,) rows, cols] with row pitch `ld` and head pitch `head` (elements); box: `box_rows` rows x 64 columns of
 // one head, 128-byte swizzle.  heads = 0: two-dimensional.
 static int make_tmap_rows(CUtensorMap* out, const void* base, uint64_t cols, uint64_t heads, uint64_t rows, uint64_t head, uint64_t ld,
                           uint32_t box_rows) {
@@ -360,9 +370,9 @@ static int make_tmap_rows(CUtensorMap* out, const void* base, uint64_t cols, uin
   }
   if ((reinterpret_cast<uintptr_t>(base) & 15) || (ld & 7) || (heads && (head & 7))) return -2;
   const int rank = heads ? 3 : 2;
-  cuuint64_t dims[3] = {cols, heads ? heads : rows, rows};
-  cuuint64_t strides[2] = {(heads ? head : ld) * 2, ld * 2};
-  cuuint32_t box[3] = {64, heads ? 1u : box_rows, box_rows};
+  cuuint64_t dims[3] = {cols, rows, heads};
+  cuuint64_t strides[2] = {ld * 2, head * 2};
+  cuuint32_t box[3] = {64, box_rows, 1};
   cuuint32_t estr[3] = {1, 1, 1};
   return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), dims, strides, box, estr,
              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

@@ -7,8 +7,9 @@
 // One CTA per (key split, group of N heads, sequence).  A 128-key tile streams through a ring of 32 KB units (128 keys x 128
 // columns) twice, once per product; the second pass hits L2.  S of tile i + 1 is issued before O of tile i, so loads and
 // both products overlap the softmax.
-//   warps 0-3  softmax: one key per thread; column maxima over the 128 keys by halving exchanges and shared memory, lazy
-//              rescale of O^T, bf16 weights to shared memory (K-major, swizzled), per-thread running sums
+//   warps 0-3  softmax: one key per thread, heads in groups of 16 that are read from tensor memory once for the maxima and
+//              once for the weights (column reductions over the 128 keys by halving exchanges and shared memory), lazy
+//              rescale of O^T, bf16 weights to shared memory (K-major, swizzled)
 //   warp 4     TMA           warp 5  MMA issuer
 // Every CTA leaves its unnormalised fp32 partial O [rank] per head with (max, sum); latent_expand merges the splits.
 #include <cuda.h>
@@ -27,7 +28,7 @@ struct LatentDecodeParams {
   float scale_log2;
   const int* pos;               // [B]
   const int* row;               // [B]
-  float* part_o;                // [B, H, splits, rank]
+  float* part_o;                // [B, H, splits, rank padded to eight]
   float* part_ml;               // [B, H, splits, 2]
   int* err;
 };
@@ -38,18 +39,13 @@ struct LatentDecodeBars {
   int abort_flag;
 };
 
-// max (or sum) over the lanes of a warp of 16 or 32 values per lane by halving exchanges: lane l ends with value l % N
-template <int N, bool SUM>
-__device__ __forceinline__ float lane_reduce(float (&v)[N]) {
+// max (or sum) over the lanes of a warp of 16 values per lane by halving exchanges: lane l ends with value l % 16
+template <bool SUM>
+__device__ __forceinline__ float lane_reduce16(float (&v)[16]) {
   const int lane = threadIdx.x & 31;
   auto op = [](float a, float b) { return SUM ? a + b : fmaxf(a, b); };
 #pragma unroll
-  for (int off = 16; off >= N; off >>= 1) {
-#pragma unroll
-    for (int k = 0; k < N; ++k) v[k] = op(v[k], __shfl_xor_sync(0xffffffffu, v[k], off));
-  }
-#pragma unroll
-  for (int off = N / 2; off > 0; off >>= 1) {
+  for (int off = 8; off > 0; off >>= 1) {
 #pragma unroll
     for (int k = 0; k < off; ++k) {
       const bool up = lane & off;
@@ -57,7 +53,7 @@ __device__ __forceinline__ float lane_reduce(float (&v)[N]) {
       v[k] = op(keep, __shfl_xor_sync(0xffffffffu, send, off));
     }
   }
-  return v[0];
+  return op(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
 }
 
 template <int N>
@@ -66,7 +62,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   constexpr int QPANEL = N * 128;
   constexpr uint32_t IDESC_S = make_idesc_bf16(128, N, 0, 0);
   constexpr uint32_t IDESC_O = make_idesc_bf16(128, N, 1, 0);
-  constexpr int RG = N >= 32 ? 32 : N;           // columns per reduction group
   constexpr int TMEM_COLS = 512;
 
   pdl_trigger();
@@ -77,7 +72,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   uint8_t* sQ = sR + p.ring * LD_UNIT;
   uint8_t* sP = sQ + panels * QPANEL;            // [2 panels of 64 keys][N rows][128 bytes]
   float* s_wred = reinterpret_cast<float*>(sP + 2 * QPANEL);   // [4][N]
-  float* s_m = s_wred + 4 * N;                   // [N] running reference maxima (log2 units)
+  float* s_sum = s_wred + 4 * N;                 // [4][N] running sums of every warp's keys
+  float* s_m = s_sum + 4 * N;                    // [N] running reference maxima (log2 units)
   float* s_alpha = s_m + N;                      // [N]
   int* s_flag = reinterpret_cast<int*>(s_alpha + N);           // [2]
   LatentDecodeBars* bars = reinterpret_cast<LatentDecodeBars*>(s_flag + 4);
@@ -101,6 +97,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     fence_proxy_async_smem();
   }
   if (threadIdx.x < N) s_m[threadIdx.x] = -INFINITY;
+  for (int i = threadIdx.x; i < 4 * N; i += 192) s_sum[i] = 0.f;
   if (threadIdx.x < 2) s_flag[threadIdx.x] = 0;
   if (warp == 5) {
     tmem_alloc(&bars->tmem_slot, TMEM_COLS);
@@ -127,17 +124,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       const int row0 = p.row[b] * p.cap;
       mbar_expect_tx(&bars->q_full, panels * QPANEL);
       for (int c = 0; c < panels; ++c) tma_load_2d(sQ + c * QPANEL, &tmQ, &bars->q_full, c * 64, b * p.H + g * N);
-      uint32_t it = 0;
+      uint32_t it = 0, ph = 0;
+      int s = 0;                         // ring unit, parity of the pass over the ring
       bool ok = true;
       auto load_tile = [&](int i, int units) {
         const int y = row0 + tile_of(i) * 128;
         for (int u = 0; u < units && ok; ++u, ++it) {
-          const int s = it % p.ring;
-          if (!mbar_wait(&bars->empty[s], ((it / p.ring) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_STAGE_EMPTY)) { ok = false; break; }
+          if (!mbar_wait(&bars->empty[s], ph ^ 1, abort_flag, p.err, ERR_WAIT_STAGE_EMPTY)) { ok = false; break; }
           const bool two = u * 128 + 64 < p.ld;
           mbar_expect_tx(&bars->full[s], two ? LD_UNIT : LD_UNIT / 2);
           tma_load_2d(sR + s * LD_UNIT, &tmC, &bars->full[s], u * 128, y);
           if (two) tma_load_2d(sR + s * LD_UNIT + LD_UNIT / 2, &tmC, &bars->full[s], u * 128 + 64, y);
+          if (++s == p.ring) { s = 0; ph ^= 1; }
         }
       };
       load_tile(0, units_s);
@@ -158,18 +156,22 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       const uint64_t dA = make_smem_desc(smem_u32(sR), 16, 1024), dAt = make_smem_desc(smem_u32(sR), 128 * 128, 1024);
       const uint64_t dQ = make_smem_desc(smem_u32(sQ), 16, 1024), dP = make_smem_desc(smem_u32(sP), 16, 1024);
       const int steps = (p.ld + 15) >> 4;
-      uint32_t it = 0;
+      int s = 0;
+      uint32_t ph = 0;
       bool ok = mbar_wait(&bars->q_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
-      auto wait_unit = [&](uint32_t i) {
-        if (!mbar_wait(&bars->full[i % p.ring], (i / p.ring) & 1, abort_flag, p.err, ERR_WAIT_TMA_FULL)) return false;
+      auto wait_unit = [&]() {
+        if (!mbar_wait(&bars->full[s], ph, abort_flag, p.err, ERR_WAIT_TMA_FULL)) return false;
         tc_fence_after();
         return true;
       };
+      auto free_unit = [&]() {
+        umma_commit(&bars->empty[s]);
+        if (++s == p.ring) { s = 0; ph ^= 1; }
+      };
       auto issue_s = [&](int i) {          // S^T of the i-th tile into score buffer i & 1
         const uint32_t d = tmem_base + (i & 1) * N;
-        for (int u = 0; u < units_s && ok; ++u, ++it) {
-          if (!wait_unit(it)) { ok = false; break; }
-          const int s = it % p.ring;
+        for (int u = 0; u < units_s && ok; ++u) {
+          if (!wait_unit()) { ok = false; break; }
           for (int c = 0; c < 2; ++c) {
             const int left = steps - (u * 8 + c * 4);
             if (left <= 0) break;
@@ -179,7 +181,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
             if (left > 2) umma_bf16(d, a + 4, q + 4, IDESC_S, 1u);
             if (left > 3) umma_bf16(d, a + 6, q + 6, IDESC_S, 1u);
           }
-          umma_commit(&bars->empty[s]);
+          free_unit();
         }
         if (ok) umma_commit(&bars->s_full[i & 1]);
       };
@@ -188,15 +190,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
         if (i + 1 < n) issue_s(i + 1);     // its score buffer was read before P of tile i - 1 was published
         if (!ok || !mbar_wait(&bars->p_ready, i & 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
         tc_fence_after();
-        for (int u = 0; u < units_o && ok; ++u, ++it) {
-          if (!wait_unit(it)) { ok = false; break; }
-          const int s = it % p.ring;
+        for (int u = 0; u < units_o && ok; ++u) {
+          if (!wait_unit()) { ok = false; break; }
           const uint64_t a = dAt + ((s * LD_UNIT) >> 4);
           const uint32_t d = tmem_base + (2 + u) * N;
 #pragma unroll
           for (int t = 0; t < 8; ++t)      // 16 keys per step; keys 64.. lie in the second panel of P
             umma_bf16(d, a + t * 128, dP + (t >> 2) * (QPANEL >> 4) + (t & 3) * 2, IDESC_O, (i | t) ? 1u : 0u);
-          umma_commit(&bars->empty[s]);
+          free_unit();
         }
         if (ok) umma_commit(&bars->o_done);
       }
@@ -205,9 +206,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     // ------------------------------------------------------------------ softmax: thread = key of the tile
     const int key = threadIdx.x;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    float l[N];
-#pragma unroll
-    for (int c = 0; c < N; ++c) l[c] = 0.f;
+    float* wred = s_wred + warp * N;
+    float* wsum = s_sum + warp * N;
     // A wait that gave up (the abort flag then ends all others quickly) must not take threads away from the named barriers:
     // the loop runs on without waiting and nothing is stored.
     bool ok = true;
@@ -215,28 +215,21 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       const int slot = tile_of(i) * 128 + key;
       int back = head_slot - slot;
       if (back < 0) back += p.cap;
-      const bool visible = back < seen;
+      const float scale = back < seen ? p.scale_log2 : 0.f, shift = back < seen ? 0.f : -INFINITY;   // hidden key: -inf
       ok = ok && mbar_wait(&bars->s_full[i & 1], (i >> 1) & 1, abort_flag, p.err, ERR_WAIT_ATTN);
       __syncwarp();
       tc_fence_after();
-      float s[N];
-#pragma unroll
+      const uint32_t ts = tmem_base + (i & 1) * N + lane_addr;
+#pragma unroll 1
       for (int c = 0; c < N; c += 16) {
         uint32_t v[16];
-        tmem_ld_32x16(tmem_base + (i & 1) * N + c + lane_addr, v);
+        float t[16];
+        tmem_ld_32x16(ts + c, v);
+        tmem_ld_wait();
 #pragma unroll
-        for (int k = 0; k < 16; ++k) s[c + k] = __uint_as_float(v[k]);
-      }
-      tmem_ld_wait();
-#pragma unroll
-      for (int c = 0; c < N; ++c) s[c] = visible ? s[c] * p.scale_log2 : -INFINITY;
-#pragma unroll
-      for (int c0 = 0; c0 < N; c0 += RG) {
-        float t[RG];
-#pragma unroll
-        for (int k = 0; k < RG; ++k) t[k] = s[c0 + k];
-        const float m = lane_reduce<RG, false>(t);
-        if (lane < RG) s_wred[warp * N + c0 + lane] = m;
+        for (int k = 0; k < 16; ++k) t[k] = fmaf(__uint_as_float(v[k]), scale, shift);
+        const float m = lane_reduce16<false>(t);
+        if (lane < 16) wred[c + lane] = m;
       }
       named_barrier_sync(1, 128);
       if (key < N) {
@@ -255,78 +248,78 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       if (i > 0) ok = ok && mbar_wait(&bars->o_done, (i - 1) & 1, abort_flag, p.err, ERR_WAIT_ATTN);
       __syncwarp();
       tc_fence_after();
-      if (s_flag[i & 1]) {
+      if (i > 0 && s_flag[i & 1]) {
+        for (int c = lane; c < N; c += 32) wsum[c] *= s_alpha[c];
+        for (int u = 0; u < units_o; ++u) {
+#pragma unroll 1
+          for (int c = 0; c < N; c += 16) {
+            uint32_t v[16];
+            const uint32_t ta = tmem_base + (2 + u) * N + c + lane_addr;
+            tmem_ld_32x16(ta, v);
+            tmem_ld_wait();
 #pragma unroll
-        for (int c = 0; c < N; ++c) l[c] *= s_alpha[c];
-        if (i > 0) {
-          for (int u = 0; u < units_o; ++u) {
-#pragma unroll
-            for (int c = 0; c < N; c += 16) {
-              uint32_t v[16];
-              const uint32_t ta = tmem_base + (2 + u) * N + c + lane_addr;
-              tmem_ld_32x16(ta, v);
-              tmem_ld_wait();
-#pragma unroll
-              for (int k = 0; k < 16; ++k) v[k] = __float_as_uint(__uint_as_float(v[k]) * s_alpha[c + k]);
-              tmem_st_32x16(ta, v);
-            }
+            for (int k = 0; k < 16; ++k) v[k] = __float_as_uint(__uint_as_float(v[k]) * s_alpha[c + k]);
+            tmem_st_32x16(ta, v);
           }
-          tmem_st_wait();
         }
+        tmem_st_wait();
+        __syncwarp();
       }
       uint8_t* prow = sP + (key >> 6) * QPANEL + (key & 7) * 2;
       const int chunk = (key & 63) >> 3;
+#pragma unroll 1
+      for (int c = 0; c < N; c += 16) {
+        uint32_t v[16];
+        float t[16];
+        tmem_ld_32x16(ts + c, v);
+        tmem_ld_wait();
 #pragma unroll
-      for (int c = 0; c < N; ++c) {
-        const float m = s_m[c];
-        const float e = exp2f(s[c] - (m == -INFINITY ? 0.f : m));
-        l[c] += e;
-        *reinterpret_cast<__nv_bfloat16*>(prow + c * 128 + ((chunk ^ (c & 7)) << 4)) = f2bf(e);
+        for (int k = 0; k < 16; k += 4) {
+          const float4 m4 = *reinterpret_cast<const float4*>(s_m + c + k);   // finite: every tile has a visible key
+          const float m[4] = {m4.x, m4.y, m4.z, m4.w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float e = exp2f(fmaf(__uint_as_float(v[k + j]), scale, shift) - m[j]);
+            t[k + j] = e;
+            *reinterpret_cast<__nv_bfloat16*>(prow + (c + k + j) * 128 + ((chunk ^ ((k + j) & 7)) << 4)) = f2bf(e);
+          }
+        }
+        const float sum = lane_reduce16<true>(t);
+        if (lane < 16) wsum[c + lane] += sum;
       }
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->p_ready);
     }
-    const int heads = min(N, p.H - g * N);
+    const int heads = min(N, p.H - g * N), ld_o = (p.rank + 7) & ~7;
     const size_t base = (static_cast<size_t>(b) * p.H + g * N) * p.splits + split;
-    if (n == 0) {
-      if (key < heads) {
-        p.part_ml[2 * (base + static_cast<size_t>(key) * p.splits)] = -INFINITY;
-        p.part_ml[2 * (base + static_cast<size_t>(key) * p.splits) + 1] = 0.f;
-      }
-    } else {
+    if (n > 0) {
       ok = ok && mbar_wait(&bars->o_done, (n - 1) & 1, abort_flag, p.err, ERR_WAIT_ATTN);
       __syncwarp();
       tc_fence_after();
+#pragma unroll 1
       for (int u = 0; u < units_o; ++u) {
         const int r = u * 128 + warp * 32 + lane;
-#pragma unroll
+#pragma unroll 1
         for (int c = 0; c < N; c += 16) {
           uint32_t v[16];
           tmem_ld_32x16(tmem_base + (2 + u) * N + c + lane_addr, v);
           tmem_ld_wait();
           if (ok && r < p.rank) {
+            float* dst = p.part_o + (base + static_cast<size_t>(c) * p.splits) * ld_o + r;
 #pragma unroll
             for (int k = 0; k < 16; ++k)
-              if (c + k < heads) p.part_o[(base + static_cast<size_t>(c + k) * p.splits) * p.rank + r] = __uint_as_float(v[k]);
+              if (c + k < heads) dst[static_cast<size_t>(k) * p.splits * ld_o] = __uint_as_float(v[k]);
           }
         }
       }
-#pragma unroll
-      for (int c0 = 0; c0 < N; c0 += RG) {
-        float t[RG];
-#pragma unroll
-        for (int k = 0; k < RG; ++k) t[k] = l[c0 + k];
-        const float sum = lane_reduce<RG, true>(t);
-        if (lane < RG) s_wred[warp * N + c0 + lane] = sum;   // the maxima in it were read before the last barrier
-      }
-      named_barrier_sync(1, 128);
-      if (ok && key < heads) {
-        const size_t o = 2 * (base + static_cast<size_t>(key) * p.splits);
-        p.part_ml[o] = s_m[key] * 0.6931471805599453f;
-        p.part_ml[o + 1] = (s_wred[key] + s_wred[N + key]) + (s_wred[2 * N + key] + s_wred[3 * N + key]);
-      }
+    }
+    named_barrier_sync(1, 128);
+    if (ok && key < heads) {
+      const size_t o = 2 * (base + static_cast<size_t>(key) * p.splits);
+      p.part_ml[o] = s_m[key] * 0.6931471805599453f;      // -inf for an empty split
+      p.part_ml[o + 1] = (s_sum[key] + s_sum[N + key]) + (s_sum[2 * N + key] + s_sum[3 * N + key]);
     }
   }
   tc_fence_before();
@@ -350,7 +343,7 @@ static LatentDecodePlan latent_decode_plan(int H, int rank, int ld) {
   const int chunks = (rank + 127) / 128, panels = (ld + 63) / 64;
   for (int n = H > 32 ? 64 : (H > 16 ? 32 : 16); n >= 16; n >>= 1) {
     if (chunks > LD_RANK_CHUNKS || (2 + chunks) * n > 512) continue;
-    const int fixed = 1024 + (panels + 2) * n * 128 + 6 * n * 4 + 64 + 512;
+    const int fixed = 1024 + (panels + 2) * n * 128 + 10 * n * 4 + 64 + 512;
     const int ring = (LIMIT - fixed) / LD_UNIT;
     if (ring >= 2) {
       const int r = ring < LD_MAX_UNITS ? ring : LD_MAX_UNITS;

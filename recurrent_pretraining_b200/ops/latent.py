@@ -327,7 +327,7 @@ def ring_attention_pieces(L: LatentLayout, inp, w_kv, norm_w, eps: float, rope, 
     B, dev, cap, f32 = inp.shape[0], inp.device, cache.shape[1], int(dtype == F32)
     w_uk, w_uv = w_kv[:L.heads * L.dim], w_kv[L.off_v:L.off_v + L.heads * L.vdim]
     qlat = torch.empty(B, L.heads, L.ld_lat, dtype=dtype, device=dev)
-    part_o = torch.empty(B, L.heads, splits, L.rank, dtype=F32, device=dev)
+    part_o = torch.empty(B, L.heads, splits, pad8(L.rank), dtype=F32, device=dev)
     part_ml = torch.empty(B, L.heads, splits, 2, dtype=F32, device=dev)
     out = torch.empty(B, L.ld_o, dtype=dtype, device=dev)[:, :L.heads * L.vdim]
     gate = inp[:, L.off_g:]
