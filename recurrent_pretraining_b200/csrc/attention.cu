@@ -18,6 +18,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "softmax_math.cuh"
 
 namespace b200 {
 
@@ -348,11 +349,6 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tm, const AttnParams p) {
 //               registers, single pass; the running max is only raised (and O rescaled in TMEM) when it grew by more
 //               than 2^8, otherwise the stale max is kept -- P then stays below 256 and the final 1/l fixes the scale
 // TMEM columns: S_A [0,128)  S_B [128,256)  O_A [256,256+D)  O_B [384,384+D).
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 // 2^x on the FMA pipe (no MUFU): floor by the 1.5 * 2^23 trick with round-down, cubic for the fractional part, the
 // integer part added into the exponent field.  Relative error about 1e-4, below bf16 resolution.
 __device__ __forceinline__ float ex2_poly(float x) {
@@ -364,40 +360,6 @@ __device__ __forceinline__ float ex2_poly(float x) {
   pl = fmaf(pl, f, 0.695146143436431885f);
   pl = fmaf(pl, f, 1.f);
   return __int_as_float(__float_as_int(pl) + (__float_as_int(t) << 23));
-}
-
-// three-input max and packed two-wide fp32 arithmetic (sm_100): half the issue slots of the scalar forms
-__device__ __forceinline__ float fmax3(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-__device__ __forceinline__ float2 ffma2(float2 a, float2 b, float2 c) {
-  float2 d;
-  asm("{\n"
-      "  .reg .b64 ra, rb, rc, rd;\n"
-      "  mov.b64 ra, {%2, %3};\n"
-      "  mov.b64 rb, {%4, %5};\n"
-      "  mov.b64 rc, {%6, %7};\n"
-      "  fma.rn.f32x2 rd, ra, rb, rc;\n"
-      "  mov.b64 {%0, %1}, rd;\n"
-      "}\n"
-      : "=f"(d.x), "=f"(d.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-  return d;
-}
-__device__ __forceinline__ float2 fadd2(float2 a, float2 b) {
-  float2 d;
-  asm("{\n"
-      "  .reg .b64 ra, rb, rd;\n"
-      "  mov.b64 ra, {%2, %3};\n"
-      "  mov.b64 rb, {%4, %5};\n"
-      "  add.rn.f32x2 rd, ra, rb;\n"
-      "  mov.b64 {%0, %1}, rd;\n"
-      "}\n"
-      : "=f"(d.x), "=f"(d.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-  return d;
 }
 
 constexpr int FWD2_VSTAGES = 3;  // V is needed one step later than K is released: a third stage hides the load latency

@@ -15,6 +15,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "softmax_math.cuh"
 
 namespace b200 {
 
@@ -44,18 +45,12 @@ struct RingPos {
 };
 
 struct LatentAttnBars {
-  uint64_t q_full;
+  uint64_t q_full[2];
   uint64_t k_full[LA_MAX_STAGES], k_empty[LA_MAX_STAGES], v_full[LA_MAX_STAGES], v_empty[LA_MAX_STAGES];
   uint64_t s_full[2], p_ready[2], o_final[2];
   uint32_t tmem_slot;
   int abort_flag;
 };
-
-__device__ __forceinline__ float la_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 
 template <int BN>
 __global__ void __launch_bounds__(384, 1)
@@ -71,10 +66,10 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int kp = p.pn + p.pr;
   const int q_bytes = kp * LA_QPANEL, k_bytes = kp * KPANEL, v_bytes = p.pv * KPANEL;
-  uint8_t* sQ = smem;                       // tile A, tile B
+  LatentAttnBars* bars = reinterpret_cast<LatentAttnBars*>(smem);   // in front: offsets that do not depend on the sizes
+  uint8_t* sQ = smem + 1024;                // tile A, tile B
   uint8_t* sK = sQ + 2 * q_bytes;
   uint8_t* sV = sK + p.kst * k_bytes;
-  LatentAttnBars* bars = reinterpret_cast<LatentAttnBars*>(sV + p.vst * v_bytes);
   volatile int* abort_flag = &bars->abort_flag;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -90,10 +85,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   const int nmax = max(je0, je1);
 
   auto load_q = [&](int x) {
+    mbar_expect_tx(&bars->q_full[x], q_bytes);
     for (int c = 0; c < p.pn; ++c)
-      tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full, c * 64, q0 + x * LA_BM, h);
+      tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full[x], c * 64, q0 + x * LA_BM, h);
     for (int c = 0; c < p.pr; ++c)
-      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full, c * 64, q0 + x * LA_BM, h);
+      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full[x], c * 64, q0 + x * LA_BM, h);
   };
   auto load_k = [&](int j, int s) {
     mbar_expect_tx(&bars->k_full[s], k_bytes);
@@ -104,7 +100,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 
   // the TMA thread sets up the barriers and requests the queries and the first key block before the CTA-wide sync
   if (threadIdx.x == 256) {
-    mbar_init(&bars->q_full, 1);
+    tma_prefetch_desc(&tmQn);
+    tma_prefetch_desc(&tmQr);
+    tma_prefetch_desc(&tmKn);
+    tma_prefetch_desc(&tmKr);
+    tma_prefetch_desc(&tmV);
     for (int i = 0; i < LA_MAX_STAGES; ++i) {
       mbar_init(&bars->k_full[i], 1);
       mbar_init(&bars->k_empty[i], 1);
@@ -112,6 +112,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       mbar_init(&bars->v_empty[i], 1);
     }
     for (int i = 0; i < 2; ++i) {
+      mbar_init(&bars->q_full[i], 1);
       mbar_init(&bars->s_full[i], 1);
       mbar_init(&bars->p_ready[i], 4);
       mbar_init(&bars->o_final[i], 1);
@@ -119,10 +120,9 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     bars->abort_flag = 0;
     fence_barrier_init();
     fence_proxy_async_smem();
-    mbar_expect_tx(&bars->q_full, 2 * q_bytes);
-    load_q(0);
-    load_q(1);            // rows past the sequence are other tokens or zero; they are never stored
+    load_q(0);            // rows past the sequence are other tokens or zero; they are never stored
     load_k(0, 0);
+    load_q(1);
   }
   if (warp == 9) {
     tmem_alloc(&bars->tmem_slot, 512);
@@ -147,7 +147,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         }
         // every issued load must land before the CTA exits
         unsigned long long t0 = globaltimer_ns();
-        while (!mbar_try_wait(&bars->q_full, 0) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
+        while (!(mbar_try_wait(&bars->q_full[0], 0) && mbar_try_wait(&bars->q_full[1], 0)) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
         for (int j = max(0, issued - p.kst); j < issued; ++j) {
           t0 = globaltimer_ns();
           while (!mbar_try_wait(&bars->k_full[j % p.kst], (j / p.kst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
@@ -167,6 +167,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           const unsigned long long t0 = globaltimer_ns();
           while (!mbar_try_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
         }
+      }
+    } else if (warp >= 10) {
+      // bring the CTA's gate rows into L2 while the blocks are processed
+      const int lines = (2 * p.vdim + 127) / 128;
+      for (int i = threadIdx.x - 320; i < nrows * lines; i += 64) {
+        const char* g = reinterpret_cast<const char*>(p.gate + static_cast<size_t>(q0 + i / lines) * p.ld_gate + h * p.vdim) + (i % lines) * 128;
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(g));
       }
     } else if (warp == 9) {
       if (lane == 0) {
@@ -197,12 +204,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 #pragma unroll
           for (int t = 0; t < BN / 16; ++t) umma_bf16_ts(d, a + t * 8, vd + t * 128, idesc_o, (first && t == 0) ? 0u : 1u);
         };
-        bool ok = mbar_wait(&bars->q_full, 0, abort_flag, p.err, ERR_WAIT_ATTN) &&
+        bool ok = mbar_wait(&bars->q_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN) &&
                   mbar_wait(&bars->k_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN);
         if (ok) {
           tc_fence_after();
           issue_s(0, 0);
-          if (je1 > 0 && jb1 == 0) issue_s(1, 0);
+          ok = mbar_wait(&bars->q_full[1], 0, abort_flag, p.err, ERR_WAIT_ATTN);
+          tc_fence_after();
+          if (ok && je1 > 0 && jb1 == 0) issue_s(1, 0);
           umma_commit(&bars->k_empty[0]);
         }
         RingPos k, v;                        // stages of key block j + 1 and value block j
@@ -232,11 +241,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");
     const int x = warp >> 2;
     const int quad = warp & 3;
-    const int r = x * LA_BM + quad * 32 + lane;              // query row of this thread inside the CTA's 256
     const int jb = x ? jb1 : 0, je = x ? je1 : je0;
-    const int hi = s0 + r, lo = max(kbase, hi - p.window + 1);   // visible stream positions of the row
-    const int hi_first = s0 + x * LA_BM;                      // tile-wide: blocks inside [lo_last, hi_first] need no mask
+    // blocks [j_lo, j_hi) are visible to every row of the tile; the others are masked
     const int lo_last = max(kbase, s0 + (x ? last_b : last_a) - p.window + 1);
+    const int j_lo = (lo_last - kstart + BN - 1) / BN, j_hi = (s0 + x * LA_BM + 1 - kstart) / BN;
+    const int hi = s0 - kstart + x * LA_BM + quad * 32 + lane;   // newest visible key of this thread's row, from kstart
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t ts = tmem_base + x * BN + lane_addr;
     const uint32_t to = tmem_base + O_COL + x * O_WIDTH + lane_addr;
@@ -255,25 +264,28 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
       }
       tmem_ld_wait();
-      const int k0 = kstart + j * BN;
-      if (k0 < lo_last || k0 + BN - 1 > hi_first) {
-        const int cmin = lo - k0, cmax = hi - k0;
+      if (j < j_lo || j >= j_hi) {
+        const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
 #pragma unroll
         for (int i = 0; i < BN; ++i)
           if (i < cmin || i > cmax) sv[i] = -INFINITY;
       }
       float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
-      for (int i = 4; i < BN; i += 4) {
-#pragma unroll
-        for (int k = 0; k < 4; ++k) mx4[k] = fmaxf(mx4[k], sv[i + k]);
+      for (int i = 4; i + 7 < BN; i += 8) {
+        mx4[0] = fmax3(mx4[0], sv[i], sv[i + 1]);
+        mx4[1] = fmax3(mx4[1], sv[i + 2], sv[i + 3]);
+        mx4[2] = fmax3(mx4[2], sv[i + 4], sv[i + 5]);
+        mx4[3] = fmax3(mx4[3], sv[i + 6], sv[i + 7]);
       }
+      mx4[0] = fmax3(mx4[0], sv[BN - 4], sv[BN - 3]);
+      mx4[1] = fmax3(mx4[1], sv[BN - 2], sv[BN - 1]);
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       const float m_new = fmaxf(m, mx * scale_log2);
       // raise the reference max only when it moved by more than the threshold (decided per warp)
       const bool grow = (m_new - m > RESCALE_THRESHOLD) || (m == -INFINITY);
       if (__any_sync(0xffffffffu, grow)) {
-        const float alpha = (m == -INFINITY) ? 0.f : la_ex2(m - m_new);
+        const float alpha = (m == -INFINITY) ? 0.f : ex2_approx(m - m_new);
         if (j > jb) {
 #pragma unroll 1
           for (int c = 0; c < p.vdim; c += 32) {
@@ -289,52 +301,70 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         m = m_new;
       }
       const float neg_m = (m == -INFINITY) ? 0.f : -m;        // a row may see nothing of the tile's first blocks
-      float rs[4] = {0.f, 0.f, 0.f, 0.f};
+      const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(scale_log2, scale_log2);
+      float2 rs[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
       for (int c = 0; c < BN; c += 32) {
         uint32_t packed[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const float a = la_ex2(fmaf(sv[c + i], scale_log2, neg_m)), b = la_ex2(fmaf(sv[c + i + 1], scale_log2, neg_m));
-          rs[i & 2] += a;
-          rs[(i & 2) + 1] += b;
-          packed[i >> 1] = pack_bf16x2(a, b);
+          const float2 a = ffma2(make_float2(sv[c + i], sv[c + i + 1]), scale2, neg_m2);
+          const float2 pr = make_float2(ex2_approx(a.x), ex2_approx(a.y));
+          rs[(i >> 1) & 3] = fadd2(rs[(i >> 1) & 3], pr);
+          packed[i >> 1] = pack_bf16x2(pr.x, pr.y);
         }
         tmem_st_32x16(ts + (c >> 1), packed);
       }
-      l += (rs[0] + rs[1]) + (rs[2] + rs[3]);
+      {
+        const float2 t = fadd2(fadd2(rs[0], rs[1]), fadd2(rs[2], rs[3]));
+        l += t.x + t.y;
+      }
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->p_ready[x]);
     }
     if (ok && je > jb) {
+      const int r = x * LA_BM + quad * 32 + lane;              // query of this thread inside the CTA's 256
+      const bool live = r < nrows;
+      const size_t t = live ? static_cast<size_t>(q0) + r : 0;
+      const __nv_bfloat16* grow_ = p.gate + t * p.ld_gate + h * p.vdim;
+      __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
+      uint4 gq[16];                                             // up to 128 gate values, requested before the last product ends
+      auto load_gate = [&](int c0) {
+#pragma unroll
+        for (int q = 0; q < 16; ++q)
+          if (c0 + 8 * q < p.vdim) gq[q] = *reinterpret_cast<const uint4*>(grow_ + c0 + 8 * q);
+      };
+      load_gate(0);
       if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
         tc_fence_after();
         const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
-        const size_t t = static_cast<size_t>(q0) + r;
-        const bool live = r < nrows;
-        const __nv_bfloat16* grow_ = p.gate + (live ? t : 0) * p.ld_gate + h * p.vdim;
-        __nv_bfloat16* orow = p.out + (live ? t : 0) * p.ld_out + h * p.vdim;
 #pragma unroll 1
-        for (int c = 0; c < p.vdim; c += 32) {
-          uint32_t v[32];
-          tmem_ld_32x32(to + c, v);
-          tmem_ld_wait();
-          if (live) {
+        for (int c0 = 0; c0 < p.vdim; c0 += 128) {
+          if (c0) load_gate(c0);
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-              if (c + 8 * q < p.vdim) {
-                const uint4 g4 = *reinterpret_cast<const uint4*>(grow_ + c + 8 * q);
-                const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
-                uint32_t o[4];
+          for (int b = 0; b < 4; ++b) {
+            const int c = c0 + 32 * b;
+            if (c >= p.vdim) break;
+            uint32_t v[32];
+            tmem_ld_32x32(to + c, v);
+            tmem_ld_wait();
+            if (live) {
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                  const float2 g = unpack_bf16x2(gw[i]);
-                  o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * inv_l / (1.f + __expf(-g.x)),
-                                     __uint_as_float(v[8 * q + 2 * i + 1]) * inv_l / (1.f + __expf(-g.y)));
+              for (int q = 0; q < 4; ++q) {
+                if (c + 8 * q < p.vdim) {
+                  const uint4 g4 = gq[4 * b + q];
+                  const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+                  uint32_t o[4];
+#pragma unroll
+                  for (int i = 0; i < 4; ++i) {
+                    const float2 g = unpack_bf16x2(gw[i]);
+                    o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * inv_l / (1.f + __expf(-g.x)),
+                                       __uint_as_float(v[8 * q + 2 * i + 1]) * inv_l / (1.f + __expf(-g.y)));
+                  }
+                  *reinterpret_cast<uint4*>(orow + c + 8 * q) = make_uint4(o[0], o[1], o[2], o[3]);
                 }
-                *reinterpret_cast<uint4*>(orow + c + 8 * q) = make_uint4(o[0], o[1], o[2], o[3]);
               }
             }
           }
@@ -381,21 +411,21 @@ static int make_tmap_rows(CUtensorMap* out, const void* base, uint64_t cols, uin
 
 struct LatentAttnPlan { int bn, kst, vst, smem; };
 
+static int g_max_bn = 128;
+
 // Key-block width and ring depths for the given sizes; bn = 0: not covered.
 static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   LatentAttnPlan none = {0, 0, 0, 0};
   if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot <= 0 || vdim <= 0) return none;
   const int kp = (dim + 63) / 64 + (rot + 63) / 64, pv = (vdim + 63) / 64;
-  constexpr int LIMIT = 227 * 1024, FIXED = 1024 + 512;
-  for (int bn = 128; bn >= 64; bn -= 64) {
+  constexpr int LIMIT = 227 * 1024, FIXED = 1024 + 1024;   // barriers, alignment
+  for (int bn = g_max_bn; bn >= 64; bn -= 64) {
     if (((vdim + 31) & ~31) > (512 - 2 * bn) / 2) continue;
-    for (int st = 5; st >= 4; --st) {        // three value stages before three key stages
-      const int kst = 2, vst = st - 2;
-      const int need = 2 * kp * LA_QPANEL + (kst * kp + vst * pv) * bn * 128 + FIXED;
-      if (need <= LIMIT) {
-        const int need3 = need + kp * bn * 128;
-        return need3 <= LIMIT ? LatentAttnPlan{bn, 3, vst, need3} : LatentAttnPlan{bn, kst, vst, need};
-      }
+    // 128-key blocks are worth a single value stage: the per-block synchronisation is the larger cost
+    constexpr int STAGES[4][2] = {{3, 3}, {2, 3}, {2, 2}, {2, 1}};
+    for (const auto& st : STAGES) {
+      const int need = 2 * kp * LA_QPANEL + (st[0] * kp + st[1] * pv) * bn * 128 + FIXED;
+      if (need <= LIMIT) return {bn, st[0], st[1], need};
     }
   }
   return none;
@@ -417,6 +447,12 @@ static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, 
 
 using namespace b200;
 
+// Widest key block (128 or 64; the sizes may still ask for the narrower one).  Returns the previous setting.
+B200_API int b200_latent_attention_set_block(int bn) {
+  const int old = g_max_bn;
+  if (bn == 64 || bn == 128) g_max_bn = bn;
+  return old;
+}
 B200_API int b200_latent_attention_supported(int dim, int rot, int vdim) { return latent_attn_plan(dim, rot, vdim).bn > 0; }
 
 // q: [T, ld_q] (head h at column h (dim + rot)), kn / v: [K, ld_kv] (head h at column h dim / h vdim), kr: [K, ld_kr],
