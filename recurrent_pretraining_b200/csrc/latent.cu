@@ -176,77 +176,107 @@ latent_prep_kernel(T* __restrict__ in, LatentRow L, const int* __restrict__ sidx
   }
 }
 
-// Decode: in [B, ld_in] (fp32 accumulator or operand precision, not modified).  CTAs [0, B): row b's latent append and the
-// rotated / padding columns of qlat [B, H, ld_lat].  The others: (head, 128 latent columns, 8 rows) tiles of
-// qlat[b, h, r] = sum_d W_uk[h * dim + d, r] q[b, h, d].
+// Four neighbouring weights as they lie in memory.
+template <typename T> struct Raw4;
+template <> struct Raw4<float> {
+  float4 q;
+  __device__ __forceinline__ void load(const float* p) { q = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void get(float (&v)[4]) const { v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+};
+template <> struct Raw4<__nv_bfloat16> {
+  uint2 q;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void get(float (&v)[4]) const {
+    const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  }
+};
+
+// Decode: in [B, ld_in] (fp32 accumulator or operand precision, not modified).  Three kinds of CTAs:
+//   [0, n_lat)               row b's latent append (layers with latents of their own)
+//   [n_lat, n_lat + n_rot)   rotated and padding columns of qlat [B, H, ld_lat], one pair of columns per thread
+//   the others               (head, 128 latent columns, 8 rows) tiles of qlat[b, h, r] = sum_d W_uk[h * dim + d, r] q[b, h, d]
 constexpr int ABS_ROWS = 8, ABS_COLS = 128;
 template <typename TI, typename T>
 __global__ void __launch_bounds__(256, 3)
 latent_absorb_kernel(const TI* __restrict__ in, LatentRow L, const T* __restrict__ w_uk, int ldw, T* __restrict__ cache,
-                     T* __restrict__ qlat, int B) {
+                     T* __restrict__ qlat, int B, int n_lat, int n_rot) {
   pdl_trigger();
-  pdl_wait();
   extern __shared__ float sm[];
-  const int hd = L.dim + L.rot;
-  if (static_cast<int>(blockIdx.x) < B) {
-    const int b = blockIdx.x, p = L.pos[b], half = L.rot >> 1;
-    const TI* r = in + static_cast<size_t>(b) * L.ld_in;
-    const float* ct = L.cosT + static_cast<size_t>(p) * half;
-    const float* st = L.sinT + static_cast<size_t>(p) * half;
-    const int tail = L.ld_lat - L.rank;      // columns after the latent: padding and rotation
-    for (int i = threadIdx.x; i < L.H * tail; i += 256) {
-      const int h = i / tail, c = L.rank + (i - h * tail), j = c - L.rank_pad;
-      float v = 0.f;
-      if (j >= 0 && j < L.rot) {
-        const TI* q = r + h * hd + L.dim;
-        const float u = ldf(q + (j & ~1)), w = ldf(q + (j | 1)), cs = ct[j >> 1], sn = st[j >> 1];
-        v = (j & 1) ? w * cs + u * sn : u * cs - w * sn;
-      }
-      stf(qlat + (static_cast<size_t>(b) * L.H + h) * L.ld_lat + c, v);
-    }
-    if (L.own)
-      latent_append<TI, T, 256>(L, r, p, cache + (static_cast<size_t>(L.row[b]) * L.cap + p % L.cap) * L.ld_lat,
-                                static_cast<T*>(nullptr), sm);
+  const int hd = L.dim + L.rot, half = L.rot >> 1;
+  int id = blockIdx.x;
+  if (id < n_lat) {
+    pdl_wait();
+    const int b = id, p = L.pos[b];
+    latent_append<TI, T, 256>(L, in + static_cast<size_t>(b) * L.ld_in, p,
+                              cache + (static_cast<size_t>(L.row[b]) * L.cap + p % L.cap) * L.ld_lat, static_cast<T*>(nullptr), sm);
     return;
   }
+  id -= n_lat;
+  if (id < n_rot) {
+    pdl_wait();
+    const int pairs = (L.ld_lat - L.rank_pad) >> 1;
+    const int i = id * 256 + threadIdx.x;
+    if (i >= B * L.H * pairs) return;
+    const int j = i % pairs, bh = i / pairs, b = bh / L.H, h = bh - b * L.H;
+    T* dst = qlat + static_cast<size_t>(bh) * L.ld_lat;
+    float v0 = 0.f, v1 = 0.f;
+    if (j < half) {
+      const TI* q = in + static_cast<size_t>(b) * L.ld_in + h * hd + L.dim + 2 * j;
+      const size_t t = static_cast<size_t>(L.pos[b]) * half + j;
+      const float u = ldf(q), w = ldf(q + 1), c = L.cosT[t], s = L.sinT[t];
+      v0 = u * c - w * s;
+      v1 = w * c + u * s;
+    }
+    stf(dst + L.rank_pad + 2 * j, v0);
+    stf(dst + L.rank_pad + 2 * j + 1, v1);
+    for (int c = L.rank + j; c < L.rank_pad; c += pairs) stf(dst + c, 0.f);
+    return;
+  }
+  id -= n_rot;
   const int cols = (L.rank + ABS_COLS - 1) / ABS_COLS;
-  int id = blockIdx.x - B;
   const int rc = id % cols;
   id /= cols;
   const int h = id % L.H, b0 = (id / L.H) * ABS_ROWS;
   const int nb = min(ABS_ROWS, B - b0);
   float* qs = sm;                                  // [dim][ABS_ROWS]
   float* part = sm + ABS_ROWS * ((L.dim + 3) & ~3);   // [8][ABS_ROWS][ABS_COLS]
-  for (int i = threadIdx.x; i < ABS_ROWS * L.dim; i += 256) {
-    const int b = i / L.dim, d = i - b * L.dim;
-    qs[d * ABS_ROWS + b] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
-  }
-  __syncthreads();
   const int tx = threadIdx.x & 31, grp = threadIdx.x >> 5;   // four columns per thread, eight groups over d
   const int r = rc * ABS_COLS + 4 * tx;
+  const bool live = r < L.rank;                    // weight rows are padded to eight: columns up to r + 3 exist
+  const T* wp = w_uk + static_cast<size_t>(h) * L.dim * ldw + (live ? r : 0);
+  constexpr int U = 16;                            // weight rows in flight per thread; the first ones do not wait for q
+  Raw4<T> w[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+    if (grp + 8 * u < L.dim) w[u].load(wp + static_cast<size_t>(grp + 8 * u) * ldw);
+  pdl_wait();
+  for (int b = grp; b < ABS_ROWS; b += 8)          // warp b reads row b
+    for (int d = tx; d < L.dim; d += 32)
+      qs[d * ABS_ROWS + b] = b < nb ? ldf(in + static_cast<size_t>(b0 + b) * L.ld_in + h * hd + d) : 0.f;
+  __syncthreads();
   float acc[ABS_ROWS][4];
 #pragma unroll
   for (int b = 0; b < ABS_ROWS; ++b)
 #pragma unroll
     for (int k = 0; k < 4; ++k) acc[b][k] = 0.f;
-  if (r < L.rank) {                                // weight rows are padded to eight: columns up to r + 3 exist
-    const T* wp = w_uk + static_cast<size_t>(h) * L.dim * ldw + r;
 #pragma unroll 1
-    for (int d0 = grp; d0 < L.dim; d0 += 64) {
-      float w[8][4];
+  for (int d0 = grp; d0 < L.dim; d0 += 8 * U) {
+    if (d0 != grp) {
 #pragma unroll
-      for (int u = 0; u < 8; ++u)
-        if (d0 + 8 * u < L.dim) ld4(wp + static_cast<size_t>(d0 + 8 * u) * ldw, w[u]);
+      for (int u = 0; u < U; ++u)
+        if (d0 + 8 * u < L.dim) w[u].load(wp + static_cast<size_t>(d0 + 8 * u) * ldw);
+    }
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        if (d0 + 8 * u < L.dim) {
-          float q[8];
-          ld8(qs + (d0 + 8 * u) * ABS_ROWS, q);
+    for (int u = 0; u < U; ++u) {
+      if (d0 + 8 * u < L.dim) {
+        float q[8], wf[4];
+        ld8(qs + (d0 + 8 * u) * ABS_ROWS, q);
+        w[u].get(wf);
 #pragma unroll
-          for (int b = 0; b < ABS_ROWS; ++b)
+        for (int b = 0; b < ABS_ROWS; ++b)
 #pragma unroll
-            for (int k = 0; k < 4; ++k) acc[b][k] += q[b] * w[u][k];
-        }
+          for (int k = 0; k < 4; ++k) acc[b][k] += q[b] * wf[k];
       }
     }
   }
@@ -400,80 +430,94 @@ __device__ __forceinline__ float warp_sum_many(float (&v)[N]) {
 // CTA: (head, 32 values, ROWS rows); a warp forms four values of all its rows at once.
 constexpr int EXP_COLS = 32;
 template <typename TI, typename T, int ROWS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2)
 latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
                      const T* __restrict__ w_uv, int ldw, const TI* __restrict__ gate, int gate_ld, T* __restrict__ out,
                      int out_ld, int B, int H, int rank, int vdim) {
   pdl_trigger();
-  pdl_wait();
   extern __shared__ float os[];                    // [ROWS][rank padded to eight]
-  __shared__ float wgt[ROWS][33];
   const int h = blockIdx.x, v0 = blockIdx.y * EXP_COLS, b0 = blockIdx.z * ROWS;
   const int nb = min(ROWS, B - b0), rs = (rank + 7) & ~7;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (warp < nb) {                                 // warp b: weights of the splits of row b (splits <= 32)
-    const size_t base = (static_cast<size_t>(b0 + warp) * H + h) * splits;
+  // four weight rows per warp; the pieces of the first columns do not wait for the attention
+  const int vw = v0 + warp * 4;
+  const T* wr = w_uv + (static_cast<size_t>(h) * vdim + vw) * ldw;
+  constexpr int PRE = 2;                           // 4-column pieces per row held ahead: 32 lanes x 4 x PRE columns
+  Raw4<T> w[4][PRE];
+  auto load_w = [&](int r0) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+#pragma unroll
+      for (int e = 0; e < PRE; ++e) {
+        const int r = r0 + 128 * e + 4 * lane;
+        if (vw + k < vdim && r < rs) w[k][e].load(wr + static_cast<size_t>(k) * ldw + r);
+      }
+  };
+  load_w(0);
+  pdl_wait();
+  float gv = 0.f;                                  // gate of the one result this lane stores in the end
+  {
+    const int b = lane >> 2, v = vw + (lane & 3);
+    if (lane < 4 * ROWS && b < nb && v < vdim) gv = ldf(gate + static_cast<size_t>(b0 + b) * gate_ld + h * vdim + v);
+  }
+  {                                                // merge: warps b * WPR .. of row b; lane s holds the weight of split s
+    constexpr int WPR = 8 / ROWS;
+    const int b = warp / WPR;
+    const size_t base = (static_cast<size_t>(b0 + (b < nb ? b : 0)) * H + h) * splits;
     const float2 e = lane < splits ? *reinterpret_cast<const float2*>(part_ml + (base + lane) * 2) : make_float2(-INFINITY, 0.f);
     const float mm = warp_max(e.x);
     const float a = e.x == -INFINITY ? 0.f : expf(e.x - mm);
-    const float ll = warp_sum(a * e.y);
-    wgt[warp][lane] = a / ll;
-  }
-  __syncthreads();
-  {
-    constexpr int WPR = 8 / ROWS;                  // warps per row
-    const int b = warp / WPR;
-    const float* p = part_o + (static_cast<size_t>(b0 + (b < nb ? b : 0)) * H + h) * splits * rs;
-    for (int r = 4 * (lane + 32 * (warp % WPR)); r < rs; r += 128 * WPR) {
+    const float mine = b < nb ? a / warp_sum(a * e.y) : 0.f;
+    const float* p = part_o + base * rs;
+    for (int r0 = 128 * (warp % WPR); r0 < rs; r0 += 128 * WPR) {   // uniform over the warp
+      const int r = r0 + 4 * lane;
       float o[4] = {0.f, 0.f, 0.f, 0.f};
-      if (b < nb) {
 #pragma unroll 4
-        for (int s = 0; s < splits; ++s) {
-          const float w = wgt[b][s];
-          float x[4];
-          ld4(p + static_cast<size_t>(s) * rs + r, x);
+      for (int s = 0; s < splits; ++s) {
+        const float w = __shfl_sync(0xffffffffu, mine, s);
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (r < rs) ld4(p + static_cast<size_t>(s) * rs + r, x);
 #pragma unroll
-          for (int k = 0; k < 4; ++k) o[k] += w != 0.f ? w * x[k] : 0.f;   // an empty split's partial is not initialised
-        }
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          if (r + k >= rank) o[k] = 0.f;           // neither are the padding columns
+        for (int k = 0; k < 4; ++k) o[k] += w != 0.f ? w * x[k] : 0.f;   // an empty split's partial is not initialised
       }
-      *reinterpret_cast<float4*>(os + b * rs + r) = make_float4(o[0], o[1], o[2], o[3]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (r + k >= rank) o[k] = 0.f;             // neither are the padding columns
+      if (r < rs) *reinterpret_cast<float4*>(os + b * rs + r) = make_float4(o[0], o[1], o[2], o[3]);
     }
   }
   __syncthreads();
-  const int vw = v0 + warp * 4;
   float acc[4 * ROWS];
 #pragma unroll
   for (int i = 0; i < 4 * ROWS; ++i) acc[i] = 0.f;
-  const T* wr = w_uv + (static_cast<size_t>(h) * vdim + vw) * ldw;
-#pragma unroll 2
-  for (int r = 8 * lane; r < rs; r += 256) {       // weight rows are padded to eight with zeros
-    float w[4][8];
+#pragma unroll 1
+  for (int r0 = 0; r0 < rs; r0 += 128 * PRE) {     // weight rows are padded to eight with zeros
+    if (r0) load_w(r0);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      if (vw + k < vdim) ld8(wr + static_cast<size_t>(k) * ldw + r, w[k]);
-      else {
+    for (int e = 0; e < PRE; ++e) {
+      const int r = r0 + 128 * e + 4 * lane;
+      if (r >= rs) continue;
+      float wf[4][4];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) w[k][j] = 0.f;
+      for (int k = 0; k < 4; ++k) {
+        w[k][e].get(wf[k]);
+        if (vw + k >= vdim) wf[k][0] = wf[k][1] = wf[k][2] = wf[k][3] = 0.f;
       }
-    }
 #pragma unroll
-    for (int b = 0; b < ROWS; ++b) {
-      float o[8];
-      ld8(os + b * rs + r, o);
+      for (int b = 0; b < ROWS; ++b) {
+        float o[4];
+        ld4(os + b * rs + r, o);
 #pragma unroll
-      for (int k = 0; k < 4; ++k)
+        for (int k = 0; k < 4; ++k)
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[b * 4 + k] += w[k][j] * o[j];
+          for (int j = 0; j < 4; ++j) acc[b * 4 + k] += wf[k][j] * o[j];
+      }
     }
   }
   const float s = warp_sum_many<4 * ROWS>(acc);
   const int b = lane >> 2, v = vw + (lane & 3);
   if (lane < 4 * ROWS && b < nb && v < vdim) {
-    const float g = sigmoid_f(ldf(gate + static_cast<size_t>(b0 + b) * gate_ld + h * vdim + v));
-    stf(out + static_cast<size_t>(b0 + b) * out_ld + h * vdim + v, s * g);
+    stf(out + static_cast<size_t>(b0 + b) * out_ld + h * vdim + v, s * sigmoid_f(gv));
   }
 }
 
@@ -651,7 +695,7 @@ B200_API int b200_embed_resid(const long long* tok, const void* table, float* x,
 
 static bool latent_row_ok(const LatentRow& L) {
   return L.H > 0 && L.dim > 0 && L.rot > 0 && !(L.rot & 1) && L.rank > 0 && L.rank_pad >= L.rank && !(L.rank_pad & 1) &&
-         L.ld_lat >= L.rank_pad + L.rot && L.cap > 0;
+         L.ld_lat >= L.rank_pad + L.rot && !(L.ld_lat & 1) && L.cap > 0;
 }
 
 B200_API int b200_latent_prep(void* in, const LatentRow* Lp, const int* sidx, const int* end, void* cache, void* stream_buf, int T,
@@ -668,14 +712,15 @@ B200_API int b200_latent_absorb(const void* in, const LatentRow* Lp, const void*
   const LatentRow L = *Lp;
   if (B <= 0 || !latent_row_ok(L) || (ldw & 7) || ldw < L.rank || (reinterpret_cast<uintptr_t>(w_uk) & 15) || (L.own && !cache) || (f32 && !in_f32)) return -1;
   const int cols = (L.rank + ABS_COLS - 1) / ABS_COLS;
-  const dim3 grid(B + cols * L.H * ((B + ABS_ROWS - 1) / ABS_ROWS));
+  const int n_lat = L.own ? B : 0, n_rot = (B * L.H * ((L.ld_lat - L.rank_pad) / 2) + 255) / 256;
+  const dim3 grid(n_lat + n_rot + cols * L.H * ((B + ABS_ROWS - 1) / ABS_ROWS));
   const size_t smem = (ABS_ROWS * ((L.dim + 3) & ~3) + 8 * ABS_ROWS * ABS_COLS) * sizeof(float);
   if (smem > 200 * 1024) return -1;
 #define GO(TI, T)                                                                                                      \
   {                                                                                                                    \
     if (smem > 48 * 1024 && cudaFuncSetAttribute(latent_absorb_kernel<TI, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                                  static_cast<int>(smem)) != cudaSuccess) return -3;                     \
-    launch_k(latent_absorb_kernel<TI, T>, grid, dim3(256), smem, STREAM, (const TI*)in, L, (const T*)w_uk, ldw, (T*)cache, (T*)qlat, B); \
+    launch_k(latent_absorb_kernel<TI, T>, grid, dim3(256), smem, STREAM, (const TI*)in, L, (const T*)w_uk, ldw, (T*)cache, (T*)qlat, B, n_lat, n_rot); \
   }
   if (f32) GO(float, float)
   else if (in_f32) GO(float, bf16_t)
