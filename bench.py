@@ -5,6 +5,8 @@ with mean 32, truncated backprop depth 8, AdamW with global-norm clip 1.0) on N 
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N --master-addr 127.0.0.1 --master-port P \
         bench.py --gpus N --steps K --warmup W
     python bench.py --impl reference ...      # the unmodified reference from baseline/_ref, same metric/config
+    python bench.py --mode layered            # prefill and decode of the layered decoder shapes beside the recurrent
+                                              # model at equal size, and every kernel of a layer against its roofline
 
 Rank 0 prints ONE JSON line.  Timing: CUDA events on the launching stream around exactly K steps, bracketed by a
 barrier + device synchronise on both sides, max over ranks.  The per-step working set (7.1 GB of bf16 weights
@@ -342,6 +344,28 @@ def run_ours(args):
         fabric.shutdown()
 
 
+def run_layered(args):
+    """Serving throughput of the layered decoder shapes (random weights) on one GPU: see ``utils/layered_bench.py``."""
+    import torch
+
+    from recurrent_pretraining_b200.ops import cuda as C
+    from recurrent_pretraining_b200.utils import layered_bench
+
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    launches0 = C.launch_count()
+    sampler.start()
+    rec = layered_bench.run()
+    clocks = sampler.stop()
+    first = rec["gasovik-1b"]["models"]
+    print(json.dumps({
+        "metric": "decode tokens/sec (gasovik-1b, batch 32, prompt 2048, greedy)", "value": first["ours"]["32"]["decode_tok_s"],
+        "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "impl": "ours",
+        "data": "synthetic uniform-random tokens, random-init weights",
+        "config": {"model": "gasovik-1b, gasovik-core-5280", "l2": "flushed between single-kernel timings; whole models stream more than L2"},
+        "clocks": clocks, "gpu_launches": C.launch_count() - launches0, "layered": rec}), flush=True)
+
+
 # ------------------------------------------------------------------------------------------------------
 def run_reference(args):
     """The unmodified reference (baseline/_ref): its RecurrentGPT, SimpleFabric (bf16-mixed autocast wrapper,
@@ -525,15 +549,18 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default=MODEL)
-    ap.add_argument("--mode", default="dp", choices=["dp", "zero3"],
+    ap.add_argument("--mode", default="dp", choices=["dp", "zero3", "layered"],
                     help="dp: the headline data-parallel config; zero3: fixed r=32, k=8, accumulation 8, parameters, "
-                         "gradients and optimizer state sharded over the GPUs (needs >= 2 GPUs)")
+                         "gradients and optimizer state sharded over the GPUs (needs >= 2 GPUs); layered: serving benchmark of the "
+                         "layered decoder shapes (one GPU)")
     ap.add_argument("--optimizer", default="adamw", choices=["adamw", "ellis"],
                     help="adamw: the headline config; ellis: the reference's production optimizer flags on the same path")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3) if args.model == MODEL else args.warmup
     if args.impl == "reference":
         run_reference(args)
+    elif args.mode == "layered":
+        run_layered(args)
     else:
         run_ours(args)
 
