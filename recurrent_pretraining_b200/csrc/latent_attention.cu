@@ -52,7 +52,10 @@ struct LatentAttnBars {
   int abort_flag;
 };
 
-template <int BN>
+// SN, SR: 16-column MMA steps of the unrotated and rotated parts, known at compile time for common sizes (a block's score
+// product is then a straight line of MMAs: the issuing thread's address arithmetic would otherwise pace the whole block);
+// 0: read from the parameters.
+template <int BN, int SN, int SR>
 __global__ void __launch_bounds__(384, 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
                    const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
@@ -64,7 +67,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int kp = p.pn + p.pr;
+  const int pn = SN ? (SN + 3) / 4 : p.pn, pr = SN ? (SR + 3) / 4 : p.pr, kp = pn + pr;
   const int q_bytes = kp * LA_QPANEL, k_bytes = kp * KPANEL, v_bytes = p.pv * KPANEL;
   LatentAttnBars* bars = reinterpret_cast<LatentAttnBars*>(smem);   // in front: offsets that do not depend on the sizes
   uint8_t* sQ = smem + 1024;                // tile A, tile B
@@ -86,16 +89,16 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 
   auto load_q = [&](int x) {
     mbar_expect_tx(&bars->q_full[x], q_bytes);
-    for (int c = 0; c < p.pn; ++c)
+    for (int c = 0; c < pn; ++c)
       tma_load_3d(sQ + x * q_bytes + c * LA_QPANEL, &tmQn, &bars->q_full[x], c * 64, q0 + x * LA_BM, h);
-    for (int c = 0; c < p.pr; ++c)
-      tma_load_3d(sQ + x * q_bytes + (p.pn + c) * LA_QPANEL, &tmQr, &bars->q_full[x], c * 64, q0 + x * LA_BM, h);
+    for (int c = 0; c < pr; ++c)
+      tma_load_3d(sQ + x * q_bytes + (pn + c) * LA_QPANEL, &tmQr, &bars->q_full[x], c * 64, q0 + x * LA_BM, h);
   };
   auto load_k = [&](int j, int s) {
     mbar_expect_tx(&bars->k_full[s], k_bytes);
-    for (int c = 0; c < p.pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, h);
-    for (int c = 0; c < p.pr; ++c)
-      tma_load_2d(sK + s * k_bytes + (p.pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
+    for (int c = 0; c < pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, h);
+    for (int c = 0; c < pr; ++c)
+      tma_load_2d(sK + s * k_bytes + (pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
   };
 
   // the TMA thread sets up the barriers and requests the queries and the first key block before the CTA-wide sync
@@ -185,9 +188,18 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         auto issue_s = [&](int x, int ks) {   // S_x = Q_x K^T, keys in stage ks
           uint64_t qd = dq0 + ((x * q_bytes) >> 4), kd = dk0 + ((ks * k_bytes) >> 4);
           const uint32_t d = tmem_base + x * BN;
+          if constexpr (SN > 0) {
+#pragma unroll
+            for (int t = 0; t < SN + SR; ++t) {
+              const int c = t < SN ? (t >> 2) : (SN + 3) / 4 + ((t - SN) >> 2), w = 2 * ((t < SN ? t : t - SN) & 3);
+              umma_bf16(d, qd + c * (LA_QPANEL >> 4) + w, kd + c * (KPANEL >> 4) + w, IDESC_S, t ? 1u : 0u);
+            }
+            umma_commit(&bars->s_full[x]);
+            return;
+          }
           uint32_t acc = 0u;
           for (int c = 0; c < kp; ++c) {
-            const int left = c < p.pn ? steps_n - 4 * c : steps_r - 4 * (c - p.pn);
+            const int left = c < pn ? steps_n - 4 * c : steps_r - 4 * (c - pn);
             umma_bf16(d, qd, kd, IDESC_S, acc);
             if (left > 1) umma_bf16(d, qd + 2, kd + 2, IDESC_S, 1u);
             if (left > 2) umma_bf16(d, qd + 4, kd + 4, IDESC_S, 1u);
@@ -431,9 +443,9 @@ static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   return none;
 }
 
-template <int BN>
+template <int BN, int SN, int SR>
 static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
-  auto kern = latent_attn_kernel<BN>;
+  auto kern = latent_attn_kernel<BN, SN, SR>;
   static int configured = 0;
   if (configured < plan.smem) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess) return -10;
@@ -441,6 +453,17 @@ static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, 
   }
   kern<<<dim3(p.H, n_tiles), 384, plan.smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
+}
+
+static int dispatch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
+  const int sn = (p.dim + 15) / 16, sr = (p.rot + 15) / 16;
+  if (plan.bn == 64) return launch_latent_attn<64, 0, 0>(tm, p, plan, n_tiles, st);
+  if (sn == 8 && sr == 4) return launch_latent_attn<128, 8, 4>(tm, p, plan, n_tiles, st);   // 128 + 64
+  if (sn == 8 && sr == 2) return launch_latent_attn<128, 8, 2>(tm, p, plan, n_tiles, st);   // 128 + 32
+  if (sn == 6 && sr == 2) return launch_latent_attn<128, 6, 2>(tm, p, plan, n_tiles, st);   //  96 + 32
+  if (sn == 4 && sr == 4) return launch_latent_attn<128, 4, 4>(tm, p, plan, n_tiles, st);   //  64 + 64
+  if (sn == 4 && sr == 2) return launch_latent_attn<128, 4, 2>(tm, p, plan, n_tiles, st);   //  64 + 32
+  return launch_latent_attn<128, 0, 0>(tm, p, plan, n_tiles, st);
 }
 
 }  // namespace b200
@@ -481,5 +504,5 @@ B200_API int b200_latent_attention(const void* q, const void* kn, const void* kr
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
   p.err = err;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return plan.bn == 128 ? launch_latent_attn<128>(tm, p, plan, n_tiles, st) : launch_latent_attn<64>(tm, p, plan, n_tiles, st);
+  return dispatch_latent_attn(tm, p, plan, n_tiles, st);
 }

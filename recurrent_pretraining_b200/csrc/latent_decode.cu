@@ -155,7 +155,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     if (lane == 0 && n > 0) {
       const uint64_t dA = make_smem_desc(smem_u32(sR), 16, 1024), dAt = make_smem_desc(smem_u32(sR), 128 * 128, 1024);
       const uint64_t dQ = make_smem_desc(smem_u32(sQ), 16, 1024), dP = make_smem_desc(smem_u32(sP), 16, 1024);
-      const int steps = (p.ld + 15) >> 4;
       int s = 0;
       uint32_t ph = 0;
       bool ok = mbar_wait(&bars->q_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
@@ -173,13 +172,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
         for (int u = 0; u < units_s && ok; ++u) {
           if (!wait_unit()) { ok = false; break; }
           for (int c = 0; c < 2; ++c) {
-            const int left = steps - (u * 8 + c * 4);
-            if (left <= 0) break;
+            if (u * 2 + c >= panels) break;      // columns past ld are zero in both operands: whole panels are multiplied
             const uint64_t a = dA + ((s * LD_UNIT + c * (LD_UNIT / 2)) >> 4), q = dQ + (((u * 2 + c) * QPANEL) >> 4);
             umma_bf16(d, a, q, IDESC_S, (u | c) ? 1u : 0u);
-            if (left > 1) umma_bf16(d, a + 2, q + 2, IDESC_S, 1u);
-            if (left > 2) umma_bf16(d, a + 4, q + 4, IDESC_S, 1u);
-            if (left > 3) umma_bf16(d, a + 6, q + 6, IDESC_S, 1u);
+            umma_bf16(d, a + 2, q + 2, IDESC_S, 1u);
+            umma_bf16(d, a + 4, q + 4, IDESC_S, 1u);
+            umma_bf16(d, a + 6, q + 6, IDESC_S, 1u);
           }
           free_unit();
         }
