@@ -589,6 +589,45 @@ def test_trace_replay(run, tmp_path):
 
 
 @gpu
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+def test_trace_command(tmp_path, dtype):
+    """bin/trace_run on a model folder: steps in, one answer per step, logits in the output folder."""
+    import subprocess
+
+    import numpy as np
+    from recurrent_pretraining_b200.models.weights import save_safetensors
+
+    w = O.random_weights(ODD, 21)
+    folder, out = tmp_path / "model", tmp_path / "out"
+    LayeredConfig.from_dict(ODD).save(str(folder))
+    save_safetensors(str(folder / "model.safetensors"), w)
+    a, b = tokens(30, 61, seed=3), tokens(12, 61, seed=4)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": a[:29], "want": [0, 28]}, {"id": "y", "tokens": b[:11], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": a[29:], "want": [0]}, {"id": "y", "tokens": b[11:], "want": [0]}], "end": ["x", "y"]}]
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    r = subprocess.run([os.path.join(root, "bin", "trace_run"), "--model", str(folder), "--dtype", dtype, "--out", str(out),
+                        "--max-tokens", "64"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1"]
+    wa, wb = O.forward(ODD, w, a), O.forward(ODD, w, b)
+    tol = TOL[getattr(torch, dtype)]
+    got = [torch.from_numpy(np.fromfile(out / f"{n}.f32", dtype="<f4")).view(2, -1) for n in (0, 1)]
+    assert O.rel_error(got[0], wa[[0, 28]]) < tol and O.rel_error(got[1], torch.stack([wa[29], wb[11]])) < tol
+
+
+def test_serve_command_completes_a_prompt(tmp_path, capsys):
+    import serve
+
+    cfg = O.config([O.mixer(window=6)], ff=(40,))
+    model, w = make(cfg, ("cpu", torch.float32), seed=22)
+    model.save_pretrained(str(tmp_path))
+    prompt = tokens(5)
+    serve.main(["--model", str(tmp_path), "--cpu", "--prompt-ids", ",".join(map(str, prompt)), "--max-tokens", "6", "--max-len", "64"])
+    out = json.loads(capsys.readouterr().out.strip().splitlines()[-1])
+    assert out["choices"][0]["token_ids"] == O.greedy(cfg, w, prompt, 6)
+
+
+@gpu
 def test_graphs_follow_a_cache_that_moves():
     """A captured decode step is not replayed on the storage of a cache that has grown."""
     run = ("cuda", torch.bfloat16)
