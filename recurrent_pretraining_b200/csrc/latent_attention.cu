@@ -423,15 +423,13 @@ static int make_tmap_rows(CUtensorMap* out, const void* base, uint64_t cols, uin
 
 struct LatentAttnPlan { int bn, kst, vst, smem; };
 
-static int g_max_bn = 128;
-
 // Key-block width and ring depths for the given sizes; bn = 0: not covered.
 static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   LatentAttnPlan none = {0, 0, 0, 0};
   if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot <= 0 || vdim <= 0) return none;
   const int kp = (dim + 63) / 64 + (rot + 63) / 64, pv = (vdim + 63) / 64;
   constexpr int LIMIT = 227 * 1024, FIXED = 1024 + 1024;   // barriers, alignment
-  for (int bn = g_max_bn; bn >= 64; bn -= 64) {
+  for (int bn = 128; bn >= 64; bn -= 64) {
     if (((vdim + 31) & ~31) > (512 - 2 * bn) / 2) continue;
     // 128-key blocks are worth a single value stage: the per-block synchronisation is the larger cost
     constexpr int STAGES[4][2] = {{3, 3}, {2, 3}, {2, 2}, {2, 1}};
@@ -470,12 +468,6 @@ static int dispatch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p
 
 using namespace b200;
 
-// Widest key block (128 or 64; the sizes may still ask for the narrower one).  Returns the previous setting.
-B200_API int b200_latent_attention_set_block(int bn) {
-  const int old = g_max_bn;
-  if (bn == 64 || bn == 128) g_max_bn = bn;
-  return old;
-}
 B200_API int b200_latent_attention_supported(int dim, int rot, int vdim) { return latent_attn_plan(dim, rot, vdim).bn > 0; }
 
 // q: [T, ld_q] (head h at column h (dim + rot)), kn / v: [K, ld_kv] (head h at column h dim / h vdim), kr: [K, ld_kr],

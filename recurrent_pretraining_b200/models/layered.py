@@ -153,12 +153,12 @@ class LatentAttention(nn.Module):
         a = self.spec
         inp = self.project_stream(xb, step, cache, stream, lay, rope)
         kv = ops.linear(stream[:, :a.kv_rank], self.w_kv[:, :a.kv_rank])
-        o = ops.stream_attention(self.layout, inp, kv, stream, step, lay, a.window, a.scale)
+        o = ops.stream_attention(self.layout, inp, kv, stream, lay, a.window, a.scale)
         return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
 
     def decode(self, xb, pos, row, cache, rope, dense, splits: int):
-        """One token per row; ``dense(x, w, which)`` is the engine's narrow-batch product.  Returns (sublayer output,
-        accumulator to hand back or None)."""
+        """One token per row; ``dense(x, w, which)`` is the engine's narrow-batch product.  Returns the sublayer
+        output, whether it is an accumulator that the next kernel clears, and the projection's accumulator or None."""
         a = self.spec
         inp, acc = dense(xb, self.w_in[:, :self.width], 0)
         o = ops.ring_attention(self.layout, inp, self.w_kv, self.latent_norm, self.eps, rope, pos, row, cache,
@@ -285,7 +285,7 @@ class LayeredForCausalLM(nn.Module):
         c = self.config
         return ops.rms_residual_(x, out, bias, layer_norm, c.norm_eps, c.residual_mult, self.dtype, clear, zero)
 
-    def _logits(self, x, idx, dense=None):
+    def _logits(self, x, idx):
         h = ops.rmsnorm_rows(x, idx, self.final_norm, self.config.norm_eps, self.dtype)
         return ops.linear(h, self.head[:, :self.config.width], out_f32=True)
 

@@ -109,6 +109,15 @@ _ACT = {None: 0, "relu2": 1}
 # ------------------------------------------------------------------------------------------
 # matrix products
 # ------------------------------------------------------------------------------------------
+def _pitched(y: torch.Tensor, ld: int) -> torch.Tensor:
+    """``y`` with a row pitch of at least ``ld`` elements."""
+    if ld <= y.shape[1]:
+        return y
+    out = torch.zeros(y.shape[0], ld, dtype=y.dtype)
+    out[:, :y.shape[1]] = y
+    return out[:, :y.shape[1]]
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: Optional[str] = None,
            out_f32: bool = False, ld_out: int = 0) -> torch.Tensor:
     """act(x w^T + bias) for x [M, K] and w [N, K] of one storage dtype (rows may be pitched); result [M, N] in that dtype,
@@ -119,7 +128,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     assert x.dtype == w.dtype and w.shape[1] == Kd and not (out_f32 and (bias is not None or act))
     if not x.is_cuda:
         y = ref.linear_act(x, w, bias, act)
-        return F_pitch(y.float() if out_f32 else y, ld_out)
+        return _pitched(y.float() if out_f32 else y, ld_out)
     k = _k()
     out = torch.empty(M, max(ld_out, pad8(N)), dtype=F32 if out_f32 else x.dtype, device=x.device)[:, :N]
     if x.dtype == F32:
@@ -131,15 +140,6 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     if bias is None and act is None:
         return k.K.gemm(x, w, out=out)
     return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_BF16_BIAS_ACT, bias=bias, act=_ACT[act])
-
-
-def F_pitch(y: torch.Tensor, ld: int) -> torch.Tensor:
-    """``y`` with a row pitch of at least ``ld`` elements."""
-    if ld <= y.shape[1]:
-        return y
-    out = torch.zeros(y.shape[0], ld, dtype=y.dtype)
-    out[:, :y.shape[1]] = y
-    return out[:, :y.shape[1]]
 
 
 def bias_act(a: torch.Tensor, bias: Optional[torch.Tensor], act: Optional[str], dtype: torch.dtype, clear: bool = False) -> torch.Tensor:
@@ -258,7 +258,7 @@ def latent_prep_(L: LatentLayout, inp: torch.Tensor, norm_w, eps: float, rope, s
                       k.K._ptr(cache), stream.data_ptr() if own else 0, T, _f32(inp), k.K._stream()), "latent_prep")
 
 
-def stream_attention(L: LatentLayout, inp: torch.Tensor, kv: torch.Tensor, stream: torch.Tensor, step, layout, window: int,
+def stream_attention(L: LatentLayout, inp: torch.Tensor, kv: torch.Tensor, stream: torch.Tensor, layout, window: int,
                      scale: float) -> torch.Tensor:
     """Gated attention of the step's queries over its key stream -> [T, heads * vdim].  ``inp``: projection rows (q rotated),
     ``kv``: [K, width_kv] up-projected keys and values, ``stream``: [K, ld_lat] latent rows (the rotated key part)."""

@@ -112,7 +112,7 @@ def layer_ops_prefill(model, seqs: list, t: Timer) -> list:
     rope = cache.rope[a.rot]
     ops.latent_prep_(L, inp, mix.latent_norm, mix.eps, rope, step, lay.sidx, cache.data[0], stream)
     kv = ops.linear(stream[:, :a.kv_rank], mix.w_kv[:, :a.kv_rank])
-    o = ops.stream_attention(L, inp, kv, stream, step, lay, a.window, a.scale)
+    o = ops.stream_attention(L, inp, kv, stream, lay, a.window, a.scale)
     out = ops.linear(o, mix.w_o[:, :a.heads * a.vdim])
 
     def gemm(name, fn, M, N, K):
@@ -122,7 +122,7 @@ def layer_ops_prefill(model, seqs: list, t: Timer) -> list:
     t.op("latent_prep", lambda: ops.latent_prep_(L, inp, mix.latent_norm, mix.eps, rope, step, lay.sidx, cache.data[0], stream),
          2.0 * T * (2 * a.heads * a.rot_dim + 3 * L.ld_lat), 0)
     gemm("key|value up-projection", lambda: ops.linear(stream[:, :a.kv_rank], mix.w_kv[:, :a.kv_rank]), T, L.width_kv, a.kv_rank)
-    t.op("latent_attention", lambda: ops.stream_attention(L, inp, kv, stream, step, lay, a.window, a.scale),
+    t.op("latent_attention", lambda: ops.stream_attention(L, inp, kv, stream, lay, a.window, a.scale),
          2.0 * T * (a.heads * (a.dim + a.rot_dim + 2 * a.vdim) + L.width_kv + a.rot_dim),
          2.0 * visible_pairs(seqs, a.window) * a.heads * (a.dim + a.rot_dim + a.vdim))
     gemm("output projection", lambda: ops.linear(o, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)

@@ -316,7 +316,7 @@ def test_stream_attention(run, size, window):
     put = lambda t: t.to(dtype).to(dev)  # noqa: E731
     lay.sidx = torch.tensor([k + h + i for _, n, k, h in seqs for i in range(n)], dtype=torch.int32, device=dev)
     lay.kbase = torch.tensor([k for _, n, k, h in seqs for _ in range(n)], dtype=torch.int32, device=dev)
-    got = ops.stream_attention(L, put(inp), put(kv), put(stream), None, lay, window, scale)
+    got = ops.stream_attention(L, put(inp), put(kv), put(stream), lay, window, scale)
     assert torch.isfinite(got).all()
     d = got.double().cpu() - want
     assert float(d.abs().max()) < (2e-4 if dtype == torch.float32 else 0.35), float(d.abs().max())     # values reach 46
