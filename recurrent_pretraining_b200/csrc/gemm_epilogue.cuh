@@ -50,7 +50,9 @@ struct GemmParams {
   float lse_scale;
   // OUT_BF16_BIAS_ACT
   const float* bias;   // [N] or null
-  int act;             // 0: none, 1: relu^2
+  int act;             // 0: none, 1: relu^2, 2: silu on the columns [act_lo, act_hi) (multiples of eight)
+                       // OUT_SWIGLU: 0: silu gate, 3: tanh-gelu gate
+  int act_lo, act_hi;
 };
 
 // Linear tile index -> (m tile, n tile), grouped: GROUP consecutive m tiles are walked across all n tiles before the
@@ -152,7 +154,21 @@ __device__ __forceinline__ void bias_act_chunk(const GemmParams& p, int col, int
       const float r = fmaxf(f[i], 0.f);
       f[i] = r * r;
     }
+  } else if (p.act == 2) {
+#pragma unroll
+    for (int i = 0; i < 32; i += 8) {
+      if (col + i >= p.act_lo && col + i < p.act_hi) {
+#pragma unroll
+        for (int k = 0; k < 8; ++k) f[i + k] = f[i + k] / (1.f + __expf(-f[i + k]));
+      }
+    }
   }
+}
+
+// Gate of the gated feed-forwards: silu(g), or gelu(g) in its tanh form, g sigmoid(2 u) with u = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float glu_gate(float g, bool gelu) {
+  const float z = gelu ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
+  return g / (1.f + __expf(-z));
 }
 
 // taddr: TMEM address of (this warp's lane quadrant, first accumulator column); row: global row of this thread;
@@ -258,8 +274,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tadd
       float f[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        const float g = __uint_as_float(v[i]);
-        f[i] = g / (1.f + __expf(-g)) * __uint_as_float(u[i]);
+        f[i] = glu_gate(__uint_as_float(v[i]), p.act == 3) * __uint_as_float(u[i]);
       }
       if (nvalid == 16 && ((reinterpret_cast<uintptr_t>(crow) & 15) == 0)) {
         *reinterpret_cast<uint4*>(crow) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]),
@@ -630,7 +645,7 @@ __device__ __forceinline__ void epilogue_tile_tma_map(const GemmParams& p, const
   }
 }
 
-// Gate-up projection without stored pre-activation: silu(gate) * up of 64 output columns at a time (gate in accumulator
+// Gate-up projection without stored pre-activation: act(gate) * up of 64 output columns at a time (gate in accumulator
 // columns [0, BN), up in [BN, 2 BN)), staged and stored as one box.
 template <int BN>
 __device__ __forceinline__ void epilogue_tile_tma_swiglu(const GemmParams& p, const CUtensorMap* tmC, uint32_t taddr, int row0,
@@ -648,8 +663,7 @@ __device__ __forceinline__ void epilogue_tile_tma_swiglu(const GemmParams& p, co
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const float g0 = __uint_as_float(g[2 * i]), g1 = __uint_as_float(g[2 * i + 1]);
-        packed[hh][i] = pack_bf16x2(g0 / (1.f + __expf(-g0)) * __uint_as_float(u[2 * i]),
-                                    g1 / (1.f + __expf(-g1)) * __uint_as_float(u[2 * i + 1]));
+        packed[hh][i] = pack_bf16x2(glu_gate(g0, p.act == 3) * __uint_as_float(u[2 * i]), glu_gate(g1, p.act == 3) * __uint_as_float(u[2 * i + 1]));
       }
     }
     const int col = n0 + c0;

@@ -382,10 +382,10 @@ B200_API void b200_gemm_set_lse(void* part, float* tgt, const long long* labels,
   g_lse = {part, tgt, labels, scale};
 }
 
-// Arguments of the next OUT_BF16_BIAS_ACT call (same convention).
-struct BiasArgs { const float* bias; int act; };
-static thread_local BiasArgs g_bias = {nullptr, 0};
-B200_API void b200_gemm_set_bias(const float* bias, int act) { g_bias = {bias, act}; }
+// Arguments of the next OUT_BF16_BIAS_ACT or OUT_SWIGLU call (same convention).
+struct BiasArgs { const float* bias; int act, act_lo, act_hi; };
+static thread_local BiasArgs g_bias = {nullptr, 0, 0, 0};
+B200_API void b200_gemm_set_bias(const float* bias, int act, int act_lo, int act_hi) { g_bias = {bias, act, act_lo, act_hi}; }
 
 B200_API int b200_gemm(const void* A, const void* A2, const void* B, void* C, const void* resid, int M, int N,
                        int K1, int K2, int lda, int lda2, int ldb, int ldc, int ld_resid, int a_mn, int b_mn,
@@ -411,7 +411,8 @@ B200_API int b200_gemm(const void* A, const void* A2, const void* B, void* C, co
   p.rope_S = g_rope.S; p.rope_D = g_rope.D; p.rope_width = g_rope.width;
   p.lse_part = reinterpret_cast<float4*>(g_lse.part); p.lse_tgt = g_lse.tgt; p.lse_labels = g_lse.labels;
   p.lse_scale = g_lse.scale;
-  p.bias = g_bias.bias; p.act = g_bias.act;
+  p.bias = g_bias.bias; p.act = (out_mode == OUT_BF16_BIAS_ACT || out_mode == OUT_SWIGLU) ? g_bias.act : 0; p.act_lo = g_bias.act_lo; p.act_hi = g_bias.act_hi;
+  if (p.act == 2 && ((p.act_lo | p.act_hi) & 7)) return -28;
   if (out_mode == OUT_BF16_LSE && (!p.lse_part || !p.lse_tgt || !p.lse_labels || a_mn || b_mn || bn != 256)) return -27;
   if (out_mode == OUT_BF16_ROPE && (!p.rope_cos || p.rope_D <= 0 || (p.rope_D & 1) || (p.rope_width & 1))) return -25;
   if (g_use_2cta && M >= 256 && (bn == 256 || bn == 240 || (is_swiglu(out_mode) && !a_mn && !b_mn))) {

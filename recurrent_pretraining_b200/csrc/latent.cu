@@ -11,91 +11,24 @@
 //   * rms_residual     : x += mult * rmsnorm(a + bias) * w on the fp32 residual stream
 //   * bias_act, rmsnorm_rows, gather_rows, sgemm_nt (true fp32 matrix product)
 // Storage types: bf16 (serving) or fp32; arithmetic is fp32.  This file is built without fast-math approximations.
-#include "common.cuh"
+#include "rowops.cuh"
 
 namespace b200 {
-
-template <typename T> __device__ __forceinline__ float ldf(const T* p);
-template <> __device__ __forceinline__ float ldf<float>(const float* p) { return *p; }
-template <> __device__ __forceinline__ float ldf<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat162float(*p); }
-template <typename T> __device__ __forceinline__ void stf(T* p, float v);
-template <> __device__ __forceinline__ void stf<float>(float* p, float v) { *p = v; }
-template <> __device__ __forceinline__ void stf<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-
-// two neighbouring elements (address aligned to the pair)
-template <typename T> __device__ __forceinline__ float2 ld2(const T* p);
-template <> __device__ __forceinline__ float2 ld2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
-template <> __device__ __forceinline__ float2 ld2<__nv_bfloat16>(const __nv_bfloat16* p) {
-  return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
-}
-__device__ __forceinline__ void st2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
-__device__ __forceinline__ void st2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); }
-// four neighbouring elements
-__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
-  const float4 a = *reinterpret_cast<const float4*>(p);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-}
-__device__ __forceinline__ void ld4(const __nv_bfloat16* p, float (&v)[4]) {
-  const uint2 q = *reinterpret_cast<const uint2*>(p);
-  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y);
-  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-}
-// eight neighbouring elements (16-byte aligned rows)
-__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 q = *reinterpret_cast<const uint4*>(p);
-  const uint32_t w[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const float2 f = unpack_bf16x2(w[j]);
-    v[2 * j] = f.x;
-    v[2 * j + 1] = f.y;
-  }
-}
-__device__ __forceinline__ void st8(float* p, const float (&v)[8]) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-}
-__device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&v)[8]) {
-  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
-                                            pack_bf16x2(v[6], v[7]));
-}
-__device__ __forceinline__ void clear8(float* p) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(0.f, 0.f, 0.f, 0.f);
-  reinterpret_cast<float4*>(p)[1] = make_float4(0.f, 0.f, 0.f, 0.f);
-}
-__device__ __forceinline__ void clear8(__nv_bfloat16*) {}
-
-template <int THREADS>
-__device__ __forceinline__ float block_total(float v, float* red) {
-  v = warp_sum(v);
-  __syncthreads();   // the previous use of `red` is over
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float t = 0.f;
-#pragma unroll
-  for (int i = 0; i < THREADS / 32; ++i) t += red[i];
-  return t;
-}
-__device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
 // ------------------------------------------------------------------------------------------------ embedding
 template <typename T>
 __global__ void __launch_bounds__(128)
 embed_resid_kernel(const long long* __restrict__ tok, const T* __restrict__ table, float* __restrict__ x,
-                   T* __restrict__ xb, int E, int ld_table, int ld_xb, long long vocab, int* err) {
+                   T* __restrict__ xb, int E, int ld_table, int ld_xb, float scale, long long vocab, int* err) {
   const size_t t = blockIdx.x;
   long long id = tok[t];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0) atomicCAS(err, 0, ERR_BAD_INDEX);
   const T* src = table + static_cast<size_t>(ok ? id : 0) * ld_table;
   for (int i = threadIdx.x; i < E; i += 128) {
-    const float v = ok ? ldf(src + i) : 0.f;
+    const float v = ok ? ldf(src + i) * scale : 0.f;
     x[t * E + i] = v;
-    stf(xb + t * ld_xb + i, v);
+    if (xb) stf(xb + t * ld_xb + i, v);
   }
 }
 
@@ -319,6 +252,15 @@ struct WindowAttn {
   int gate_ld, out_ld;
   float* part_o;                  // [T, H, splits, vdim padded to eight]
   float* part_ml;                 // [T, H, splits, 2] (max in natural-log units, sum)
+  int group;                      // query heads per key / value head
+  // distance bias (null: none): score += bias[h * bias_len + min(distance, bias_len - 1)]
+  const float* bias;
+  int bias_len;
+  // query temperature (0: none): scores are multiplied by 1 + coef * ln(floor((position + 1) / every) + 1)
+  int temp_every;
+  float temp_coef;
+  int head_gate;                  // stream form: one gate per head (gate row [H]) instead of one per output
+  float gate_mult;                // factor on the gated output
 };
 
 // CTA of four warps per (token, head, key split); a warp takes 32 keys at a time: one key per lane for the scores, one
@@ -344,6 +286,10 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   const int first = max(ring ? 0 : A.kbase[t], last - A.window + 1);
   const size_t ring0 = ring ? static_cast<size_t>(A.row[t]) * A.cap : 0;
   const int nchunk = (last - first) / 32 + 1;
+  const int hk = h / A.group;
+  float scale = A.scale;
+  if (A.temp_every > 0) scale *= query_temperature(ring ? last : last - A.kbase[t], A.temp_every, A.temp_coef);
+  const float* bias = A.bias ? A.bias + static_cast<size_t>(h) * A.bias_len : nullptr;
   float m = -INFINITY, l = 0.f;
   float* op = os + warp * A.vdim;
   float* pp = ps + warp * 32;
@@ -352,14 +298,15 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
     float s = -INFINITY;
     if (j <= last) {
       const size_t key = ring ? ring0 + j % A.cap : static_cast<size_t>(j);
-      const T* a = k1 + key * A.k1_stride + static_cast<size_t>(h) * A.k1_head;
+      const T* a = k1 + key * A.k1_stride + static_cast<size_t>(hk) * A.k1_head;
       s = 0.f;
       for (int i = 0; i < A.d1; ++i) s += qs[i] * ldf(a + i);
       if (A.d2) {
         const T* b = k2 + key * A.k2_stride;
         for (int i = 0; i < A.d2; ++i) s += qs[A.d1 + i] * ldf(b + i);
       }
-      s *= A.scale;
+      s *= scale;
+      if (bias) s += bias[min(last - j, A.bias_len - 1)];
     }
     const float mn = fmaxf(m, warp_max(s));
     const float p = expf(s - mn), alpha = expf(m - mn);
@@ -371,7 +318,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
       float o = op[d] * alpha;
       for (int k = 0; k < n; ++k) {
         const size_t key = ring ? ring0 + (j0 + k) % A.cap : static_cast<size_t>(j0 + k);
-        o += pp[k] * ldf(v + key * A.v_stride + static_cast<size_t>(h) * A.v_head + d);
+        o += pp[k] * ldf(v + key * A.v_stride + static_cast<size_t>(hk) * A.v_head + d);
       }
       op[d] = o;
     }
@@ -397,8 +344,8 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
       A.part_o[pi * ((A.vdim + 7) & ~7) + d] = o;
       if (d == 0) { A.part_ml[2 * pi] = mm; A.part_ml[2 * pi + 1] = ll; }
     } else {
-      const float g = sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + h * A.vdim + d));
-      stf(out + static_cast<size_t>(t) * A.out_ld + h * A.vdim + d, o * inv * g);
+      const float g = sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + (A.head_gate ? h : h * A.vdim + d)));
+      stf(out + static_cast<size_t>(t) * A.out_ld + h * A.vdim + d, o * inv * (g * A.gate_mult));
     }
   }
 }
@@ -635,7 +582,7 @@ bias_act_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __restrict
 constexpr int SG = 64, SGK = 16;
 __global__ void __launch_bounds__(256)
 sgemm_nt_kernel(const float* __restrict__ A, const float* __restrict__ B, const float* __restrict__ bias, float* __restrict__ C,
-                int M, int N, int K, int lda, int ldb, int ldc, int act) {
+                int M, int N, int K, int lda, int ldb, int ldc, int act, int act_lo, int act_hi) {
   __shared__ float as[SGK][SG + 4], bs[SGK][SG + 4];
   const int m0 = blockIdx.x * SG, n0 = blockIdx.y * SG;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -670,6 +617,8 @@ sgemm_nt_kernel(const float* __restrict__ A, const float* __restrict__ B, const 
       if (act == 1) {
         v = fmaxf(v, 0.f);
         v *= v;
+      } else if (act == 2 && n >= act_lo && n < act_hi) {
+        v = silu_f(v);
       }
       C[static_cast<size_t>(m) * ldc + n] = v;
     }
@@ -686,10 +635,10 @@ typedef __nv_bfloat16 bf16_t;
 // Every `f32` argument: the operand storage type is fp32 instead of bf16; `in_f32`: the GEMM output is fp32.
 
 B200_API int b200_embed_resid(const long long* tok, const void* table, float* x, void* xb, int T, int E, int ld_table, int ld_xb,
-                              long long vocab, int f32, int* err, void* stream) {
-  if (T <= 0 || E <= 0 || vocab <= 0 || ld_table < E || ld_xb < E) return -1;
-  if (f32) embed_resid_kernel<float><<<T, 128, 0, STREAM>>>(tok, (const float*)table, x, (float*)xb, E, ld_table, ld_xb, vocab, err);
-  else embed_resid_kernel<bf16_t><<<T, 128, 0, STREAM>>>(tok, (const bf16_t*)table, x, (bf16_t*)xb, E, ld_table, ld_xb, vocab, err);
+                              float scale, long long vocab, int f32, int* err, void* stream) {
+  if (T <= 0 || E <= 0 || vocab <= 0 || ld_table < E || (xb && ld_xb < E)) return -1;
+  if (f32) embed_resid_kernel<float><<<T, 128, 0, STREAM>>>(tok, (const float*)table, x, (float*)xb, E, ld_table, ld_xb, scale, vocab, err);
+  else embed_resid_kernel<bf16_t><<<T, 128, 0, STREAM>>>(tok, (const bf16_t*)table, x, (bf16_t*)xb, E, ld_table, ld_xb, scale, vocab, err);
   return DONE;
 }
 
@@ -739,7 +688,7 @@ B200_API int b200_gather_rows(const void* src, const int* src_idx, void* dst, co
 B200_API int b200_window_attention(const void* q, const void* k1, const void* k2, const void* v, const void* gate, void* out,
                                    const WindowAttn* Ap, int T, int f32, void* stream) {
   const WindowAttn A = *Ap;
-  if (T <= 0 || A.H <= 0 || A.H > 65535 || A.d1 <= 0 || A.d2 < 0 || A.vdim <= 0 || A.window <= 0 || A.splits < 1 || A.splits > 32) return -1;
+  if (T <= 0 || A.H <= 0 || A.H > 65535 || A.group <= 0 || A.H % A.group || (A.bias && A.bias_len <= 0) || A.d1 <= 0 || A.d2 < 0 || A.vdim <= 0 || A.window <= 0 || A.splits < 1 || A.splits > 32) return -1;
   if (A.pos ? (!A.row || A.cap <= 0 || A.cap < A.window || !A.part_o || !A.part_ml) : (!A.sidx || !A.kbase || A.splits != 1 || A.part_o || !gate || !out))
     return -1;
   const size_t smem = (A.d1 + A.d2 + 128 + 4 * A.vdim + 8) * sizeof(float);
@@ -832,8 +781,8 @@ B200_API int b200_bias_act(void* a, int ld_a, int in_f32, int clear, const float
 }
 
 B200_API int b200_sgemm_nt(const float* A, const float* B, const float* bias, float* C, int M, int N, int K, int lda, int ldb, int ldc,
-                           int act, void* stream) {
+                           int act, int act_lo, int act_hi, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || (N + SG - 1) / SG > 65535) return -1;
-  sgemm_nt_kernel<<<dim3((M + SG - 1) / SG, (N + SG - 1) / SG), 256, 0, STREAM>>>(A, B, bias, C, M, N, K, lda, ldb, ldc, act);
+  sgemm_nt_kernel<<<dim3((M + SG - 1) / SG, (N + SG - 1) / SG), 256, 0, STREAM>>>(A, B, bias, C, M, N, K, lda, ldb, ldc, act, act_lo, act_hi);
   return DONE;
 }

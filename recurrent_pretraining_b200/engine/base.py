@@ -54,19 +54,22 @@ class GraphRunner:
 
     use_graphs = True
 
-    def _run(self, key, fn):
-        """Replay ``fn`` as a CUDA graph.  ``fn`` must be idempotent (read inputs, write separate outputs): it is
-        executed once eagerly as a warm-up and once more during capture before the first replay."""
+    def _run(self, key, fn, once: bool = False):
+        """Replay ``fn`` as a CUDA graph.  Before the first replay it is executed eagerly as a warm-up and recorded; ``fn`` must
+        be idempotent then (read inputs, write separate outputs).  With ``once`` every call takes effect exactly once (``fn``
+        updates state): the first call returns the eager execution's result and replays nothing."""
         if not self.use_graphs:
             return self._with_pdl(fn)
         g = self._graphs.get(key)
         if g is None:
-            self._with_pdl(fn)
+            first = self._with_pdl(fn)
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(graph):
                 out = self._with_pdl(fn)
             g = self._graphs[key] = (graph, out)
+            if once:
+                return first
         g[0].replay()
         return g[1]
 

@@ -5,7 +5,7 @@ a single token -- and returns the logits that were asked for; ``generate`` is a 
 
 * Prompt portions are packed without padding (``forward_step``).
 * One token per sequence is a decode step: weight-streaming GEMMs with fp32 accumulators that fused consumers read and
-  clear, attention over the ring cache, everything captured as one CUDA graph per batch size.
+  clear, attention over the cache and updates of recurrent state, everything captured as one CUDA graph per batch size.
 """
 from __future__ import annotations
 
@@ -37,7 +37,7 @@ class LayeredEngine(GraphRunner):
         self._work = [None, None]
         if self.on_gpu and model.dtype == torch.bfloat16:
             widths = [max(m.mix.layout.width_in for m in model.layers),
-                      max([self.cfg.width] + [m.mlp.spec.ff for m in model.layers if m.mlp is not None])]
+                      max([self.cfg.width] + [m.mlp.spec.ff * m.mlp.wide for m in model.layers if m.mlp is not None])]
             self._work = [torch.zeros(n * w, dtype=torch.float32, device=self.dev) for w in widths]
 
     # -- sequences ---------------------------------------------------------------------------------------------------
@@ -88,7 +88,8 @@ class LayeredEngine(GraphRunner):
             self._graphs.clear()
             self._generation = self.cache.generation
         tok, pos, row = self._tok[:B], self._meta[0, :B], self._meta[1, :B]
-        return self._run(("decode", B), lambda: self.model.decode_step(tok, pos, row, self.cache, self._dense, self._splits))
+        return self._run(("decode", B), lambda: self.model.decode_step(tok, pos, row, self.cache, self._dense, self._splits),
+                         once=True)
 
     def _dense(self, x, w, which: int):
         """Narrow-batch product -> (result, whether it is a persistent accumulator that its consumer has to clear)."""
@@ -100,16 +101,8 @@ class LayeredEngine(GraphRunner):
         return y, y.dtype == torch.float32
 
     def _splits(self, mix, B: int) -> int:
-        """Key splits of the decode attention: enough CTAs to fill the machine, at least 128 keys each."""
-        groups, fill = mix.spec.heads, 4 * 148          # generic kernel: a small CTA per head
-        if self.on_gpu and self.model.dtype == torch.bfloat16:
-            from ..ops import latent_attention as A
-
-            n = A.decode_group(mix.spec.heads, mix.spec.kv_rank, mix.layout.ld_lat)
-            if n:                                        # tensor-core kernel: one CTA per SM, n heads each
-                groups, fill = -(-mix.spec.heads // n), 148
-        tiles = min(mix.spec.window, self.max_len) // 128 + 1
-        return max(1, min(tiles, 32, fill // max(1, B * groups)))
+        """Key splits of the decode attention."""
+        return mix.decode_splits(B, self.max_len, self.on_gpu and self.model.dtype == torch.bfloat16)
 
     # -- generation --------------------------------------------------------------------------------------------------
     def prefill(self, rows: list, prompts: list) -> torch.Tensor:

@@ -221,33 +221,30 @@ class StaticRecurrentCache:
 HuginnStaticCache = StaticRecurrentCache
 
 
-class LatentRingCache:
-    """Cache of latent-attention layers: one row of ``ld_lat`` numbers per token (normed latent and rotated key part) in a ring
-    per sequence and source layer.  Position p lives in slot ``p % cap``; ``cap`` covers the widest window among the layers
-    that read the source layer's latents, so a sequence holds a bounded amount however long it grows.
+class RowCache:
+    """Sequence rows of a serving cache.  Rows are handed out by ``alloc`` and taken back by ``free``; a row that is used again
+    needs no clearing, because nothing of its former owner is read.  Rows are added on demand (``generation`` counts those
+    reallocations: captured graphs that hold old addresses are then stale).  Subclasses list their tensors, whose first
+    dimension is the row, in ``_shapes``."""
 
-    Sequence rows are handed out by ``alloc`` and taken back by ``free``; a row that is used again needs no clearing, because
-    a reader only looks at positions its new owner has written.  Rows are added on demand (``generation`` counts those
-    reallocations: captured graphs that hold old addresses are then stale)."""
-
-    SLOTS = 128   # capacities are multiples of this many slots, so that a tile of keys stays inside one sequence's ring
-
-    def __init__(self, layouts: dict, windows: dict, max_rows: int, max_len: int, dtype: torch.dtype, device):
-        self.max_len, self.dtype, self.device = max_len, dtype, torch.device(device)
-        self.layouts, self.windows = layouts, windows
-        self.caps = {i: -(-min(w, max_len) // self.SLOTS) * self.SLOTS for i, w in windows.items()}
+    def __init__(self, max_rows: int, max_len: int, device):
+        self.max_len, self.device = max_len, torch.device(device)
         self.rows, self.generation = 0, 0
         self.data: dict = {}
         self.length: dict = {}            # row -> tokens held
         self._free: list = []
         self._grow(max_rows)
 
+    def _shapes(self) -> dict:
+        """Key -> (shape of one row, dtype)."""
+        raise NotImplementedError
+
     def _grow(self, rows: int) -> None:
-        for i, cap in self.caps.items():
-            new = torch.zeros(rows, cap, self.layouts[i].ld_lat, dtype=self.dtype, device=self.device)
+        for key, (shape, dtype) in self._shapes().items():
+            new = torch.zeros(rows, *shape, dtype=dtype, device=self.device)
             if self.rows:
-                new[:self.rows] = self.data[i]
-            self.data[i] = new
+                new[:self.rows] = self.data[key]
+            self.data[key] = new
         self._free.extend(range(rows - 1, self.rows - 1, -1))
         self._free.sort(reverse=True)
         self.rows = rows
@@ -274,3 +271,37 @@ class LatentRingCache:
 
     def get_memory_usage(self) -> float:
         return sum(t.numel() * t.element_size() for t in self.data.values()) / 2**20
+
+
+class LatentRingCache(RowCache):
+    """Cache of latent-attention layers: one row of ``ld_lat`` numbers per token (normed latent and rotated key part) in a ring
+    per sequence and source layer.  Position p lives in slot ``p % cap``; ``cap`` covers the widest window among the layers
+    that read the source layer's latents, so a sequence holds a bounded amount however long it grows.  A reader only looks
+    at positions that the row's present owner has written."""
+
+    SLOTS = 128   # capacities are multiples of this many slots, so that a tile of keys stays inside one sequence's ring
+
+    def __init__(self, layouts: dict, windows: dict, max_rows: int, max_len: int, dtype: torch.dtype, device):
+        self.dtype, self.layouts, self.windows = dtype, layouts, windows
+        self.caps = {i: -(-min(w, max_len) // self.SLOTS) * self.SLOTS for i, w in windows.items()}
+        super().__init__(max_rows, max_len, device)
+
+    def _shapes(self) -> dict:
+        return {i: ((cap, self.layouts[i].ld_lat), self.dtype) for i, cap in self.caps.items()}
+
+
+class HybridCache(RowCache):
+    """Cache of models that mix attention with recurrent memories: whatever each execution of a layer (``LayerRun.index``)
+    keeps for a sequence, under the key (index, name).
+
+    * keys and values: position p of a row lies at index p of its ``max_len`` slots (attention reads the cache directly;
+      slots past a sequence's newest token are never looked at);
+    * recurrent state: fp32, replaced by every step.  A step that starts at position 0 starts from the empty state, so a row
+      that is used again needs no clearing either."""
+
+    def __init__(self, shapes: dict, max_rows: int, max_len: int, device):
+        self._row_shapes = shapes
+        super().__init__(max_rows, max_len, device)
+
+    def _shapes(self) -> dict:
+        return self._row_shapes

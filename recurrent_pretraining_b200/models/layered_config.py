@@ -8,16 +8,34 @@ Architectures:
 
 * ``Gasovik``: latent attention under a sliding window (optionally on the latents of an earlier layer), gated heads,
   biased squared-ReLU feed-forward, norms on the sublayer outputs only.
+* ``Fatudra``: layers that run grouped-query attention with a learned distance bias beside a memory with fixed decay, or a
+  gated matrix memory; tanh-GELU gated feed-forward; layer norms before and after every sublayer; a range of layers may run
+  several times in a row with the same weights.
 """
 from __future__ import annotations
 
 import json
 import math
 import os
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Optional
 
-ARCHITECTURES = ("Gasovik",)
+
+@dataclass(frozen=True)
+class Design:
+    """What an architecture fixes beside its configuration."""
+
+    mixers: tuple                    # mixer types a layer may have
+    norms: str                       # "post_rms": x += mult * rms(f(x)); "sandwich": x += ln(f(ln(x)))
+    mlp: str                         # "relu2": biased two-matrix form; "geglu": gated, tanh-GELU, no biases
+    keys: tuple                      # keys of config.json beside the common ones
+
+
+DESIGNS = {
+    "Gasovik": Design(("latent_attention",), "post_rms", "relu2", ("residual_mult",)),
+    "Fatudra": Design(("parallel", "mlstm"), "sandwich", "geglu", ("embedding", "loop")),
+}
+ARCHITECTURES = tuple(DESIGNS)
 
 
 def is_layered(config: dict) -> bool:
@@ -128,6 +146,170 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """Queries at position p are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
+
+    coef: float
+    every: int
+
+    def at(self, p: int) -> float:
+        return 1.0 + self.coef * math.log((p + 1) // self.every + 1)
+
+
+@dataclass(frozen=True)
+class BiasedAttentionSpec:
+    """Causal grouped-query attention without rotation: ``heads`` query heads over ``kv_heads`` key / value heads, a learned
+    bias per head and distance bucket, one output gate per head.  ``bias_rows`` (buckets of the table) is a tensor's size:
+    None until a checkpoint or a registry shape gives it."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    bias_max: float
+    q_temp: Optional[QueryTemperature] = None
+    bias_rows: Optional[int] = None
+
+    def bucket(self, n: int) -> int:
+        """Table row of distance ``n``: one per distance up to half the rows, then logarithmic up to ``bias_max``."""
+        half = self.bias_rows // 2
+        if n < half or self.bias_rows == 1:
+            return min(n, self.bias_rows - 1)
+        return min(self.bias_rows - 1,
+                   half + math.floor(math.log(n / half) / math.log(self.bias_max / half) * (self.bias_rows - half)))
+
+    def buckets(self) -> list:
+        """Buckets of the distances 0, 1, .. up to the first one of the last row (every farther distance shares it)."""
+        out = [0]
+        while out[-1] != self.bias_rows - 1:
+            out.append(self.bucket(len(out)))
+        return out
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "BiasedAttentionSpec":
+        _take(d, ("heads", "kv_heads", "dim", "vdim", "scale", "bias_max", "q_temp", "bias_rows"), "mixer.left")
+        t = d.get("q_temp")
+        if t is not None:
+            _take(t, ("coef", "every"), "mixer.left.q_temp")
+            t = QueryTemperature(float(t["coef"]), int(t["every"]))
+            if t.every <= 0:
+                raise ValueError("q_temp.every must be positive")
+        spec = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), float(d["scale"]), d["bias_max"], t,
+                   None if d.get("bias_rows") is None else int(d["bias_rows"]))
+        if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim) <= 0 or spec.heads % spec.kv_heads:
+            raise ValueError(f"attention sizes must be positive, kv_heads a divisor of heads: {d}")
+        return spec if spec.bias_rows is None else spec.with_rows(spec.bias_rows)
+
+    def with_rows(self, rows: int) -> "BiasedAttentionSpec":
+        if rows < 1 or (rows > 1 and self.bias_max <= rows // 2):
+            raise ValueError(f"a distance bias of {rows} rows needs a reach above {rows // 2}, not {self.bias_max}")
+        return replace(self, bias_rows=int(rows))
+
+    def to_dict(self) -> dict:
+        out = {k: getattr(self, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale", "bias_max")}
+        if self.q_temp is not None:
+            out["q_temp"] = {"coef": self.q_temp.coef, "every": self.q_temp.every}
+        if self.bias_rows is not None:
+            out["bias_rows"] = self.bias_rows
+        return out
+
+    def param_count(self, E: int) -> int:
+        qkv = self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+        return qkv * (E + 1) + self.heads * (self.bias_rows or 0) + self.heads * E + E * self.heads * self.vdim + E
+
+
+@dataclass(frozen=True)
+class DecayMemorySpec:
+    """Linear attention with one fixed decay per head."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "DecayMemorySpec":
+        _take(d, ("heads", "dim", "vdim", "decay"), "mixer.right")
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d["vdim"]), tuple(float(x) for x in d["decay"]))
+        if min(spec.heads, spec.dim, spec.vdim) <= 0 or len(spec.decay) != spec.heads or not all(0 <= x <= 1 for x in spec.decay):
+            raise ValueError(f"a decaying memory needs positive sizes and one decay in [0, 1] per head: {d}")
+        return spec
+
+    def to_dict(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay)}
+
+    def param_count(self, E: int) -> int:
+        return self.heads * (2 * self.dim + 3 * self.vdim) * E + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention (left) and a decaying memory (right) on the same input, their outputs added with fixed weights."""
+
+    left: BiasedAttentionSpec
+    right: DecayMemorySpec
+    left_scale: float
+    right_scale: float
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "ParallelSpec":
+        _take(d, ("left", "right", "left_scale", "right_scale"), "mixer")
+        return cls(BiasedAttentionSpec.from_dict(d["left"]), DecayMemorySpec.from_dict(d["right"]), float(d["left_scale"]),
+                   float(d["right_scale"]))
+
+    def to_dict(self) -> dict:
+        return {"left": self.left.to_dict(), "right": self.right.to_dict(), "left_scale": self.left_scale,
+                "right_scale": self.right_scale}
+
+    def param_count(self, E: int) -> int:
+        return self.left.param_count(E) + self.right.param_count(E)
+
+
+@dataclass(frozen=True)
+class GatedMemorySpec:
+    """Matrix memory with exponential input gate, sigmoid forget gate, normaliser and running maximum (mLSTM of xLSTM, Beck et
+    al.); ``gate_cap`` bounds the gates' logarithms."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GatedMemorySpec":
+        _take(d, ("heads", "dim", "vdim", "gate_cap"), "mixer")
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d["vdim"]), float(d["gate_cap"]))
+        if min(spec.heads, spec.dim, spec.vdim) <= 0 or spec.gate_cap <= 0:
+            raise ValueError(f"a gated memory needs positive sizes: {d}")
+        return spec
+
+    def to_dict(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "gate_cap": self.gate_cap}
+
+    def param_count(self, E: int) -> int:
+        return self.heads * (2 * self.dim + 3 * self.vdim + 2) * E + self.heads * (self.vdim + 2)
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start`` .. ``stop - 1`` run ``times`` times in a row, each pass with a cache of its own; a learned vector per
+    pass is added to the residual stream in front of it."""
+
+    start: int
+    stop: int
+    times: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "LoopSpec":
+        _take(d, ("start", "stop", "times"), "loop")
+        return cls(int(d["start"]), int(d["stop"]), int(d["times"]))
+
+    def to_dict(self) -> dict:
+        return {"start": self.start, "stop": self.stop, "times": self.times}
+
+
+@dataclass(frozen=True)
 class DenseMLPSpec:
     ff: int
 
@@ -142,13 +324,13 @@ class DenseMLPSpec:
         return {"kind": "dense", "ff": self.ff}
 
 
-MIXERS = {"latent_attention": LatentAttentionSpec}
+MIXERS = {"latent_attention": LatentAttentionSpec, "parallel": ParallelSpec, "mlstm": GatedMemorySpec}
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     type: str
-    mixer: LatentAttentionSpec
+    mixer: object                    # one of the specs of MIXERS
     mlp: Optional[DenseMLPSpec] = None
 
     @classmethod
@@ -163,15 +345,27 @@ class LayerSpec:
         return {"type": self.type, "mixer": self.mixer.to_dict(), "mlp": None if self.mlp is None else self.mlp.to_dict()}
 
 
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer: ``index`` counts executions (caches belong to them), ``loop_pass`` is set on the first layer
+    of a pass of the loop."""
+
+    index: int
+    layer: int
+    loop_pass: Optional[int] = None
+
+
 @dataclass
 class LayeredConfig:
     architecture: str
     vocab: int
     width: int
     norm_eps: float
-    residual_mult: float
+    residual_mult: float = 1.0
     layers: list = field(default_factory=list)
     name: str = ""
+    embed_scale: float = 1.0
+    loop: Optional[LoopSpec] = None
 
     def __post_init__(self):
         if self.architecture not in ARCHITECTURES:
@@ -179,7 +373,9 @@ class LayeredConfig:
         if not self.layers:
             raise ValueError("a model needs at least one layer")
         for i, layer in enumerate(self.layers):
-            j = layer.mixer.kv_from
+            if layer.type not in self.design.mixers:
+                raise ValueError(f"layer {i}: {self.architecture} has no mixer {layer.type!r}")
+            j = getattr(layer.mixer, "kv_from", None)
             if j is None:
                 continue
             if not 0 <= j < i or self.layers[j].mixer.kv_from is not None:
@@ -187,10 +383,28 @@ class LayeredConfig:
             a, b = layer.mixer, self.layers[j].mixer
             if (a.kv_rank, a.rot_dim, a.rot) != (b.kv_rank, b.rot_dim, b.rot):
                 raise ValueError(f"layer {i}: latent size and rotation must equal those of layer {j}")
+        lp = self.loop
+        if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layers) and lp.times >= 1):
+            raise ValueError(f"loop {lp} does not lie inside {len(self.layers)} layers")
 
     @property
     def architecture_class_name(self) -> str:
         return self.architecture
+
+    @property
+    def design(self) -> Design:
+        return DESIGNS[self.architecture]
+
+    def runs(self) -> list:
+        """The executions of layers, in order."""
+        lp, order = self.loop, []
+        for i in range(len(self.layers)):
+            if lp is not None and lp.start <= i < lp.stop:
+                if i == lp.start:
+                    order += [(k, t if k == lp.start else None) for t in range(lp.times) for k in range(lp.start, lp.stop)]
+            else:
+                order.append((i, None))
+        return [LayerRun(n, i, t) for n, (i, t) in enumerate(order)]
 
     def kv_source(self, i: int) -> int:
         """The layer whose latents layer ``i`` attends to."""
@@ -205,17 +419,44 @@ class LayeredConfig:
             out[s] = max(out.get(s, 0), layer.mixer.window)
         return out
 
+    def with_tensor_shapes(self, shape) -> "LayeredConfig":
+        """Fill in the sizes that only the tensors give; ``shape(name)`` returns a checkpoint tensor's shape."""
+        layers = []
+        for i, layer in enumerate(self.layers):
+            a = layer.mixer
+            if isinstance(a, ParallelSpec) and a.left.bias_rows is None:
+                a = replace(a, left=a.left.with_rows(shape(f"l{i}.mix.left.rel")[0]))
+            layers.append(replace(layer, mixer=a))
+        return replace(self, layers=layers)
+
     # -- construction ------------------------------------------------------------------------------------------------
     @classmethod
     def from_dict(cls, d: dict) -> "LayeredConfig":
-        _take(d, ("architecture", "vocab", "width", "norm", "residual_mult", "layers", "name"), "config")
+        if not is_layered(d):
+            raise ValueError(f"Invalid architecture {d.get('architecture')} provided.")
+        keys = DESIGNS[d["architecture"]].keys
+        _take(d, ("architecture", "vocab", "width", "norm", "layers", "name") + keys, "config")
         _take(d["norm"], ("eps",), "norm")
-        return cls(d["architecture"], int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), float(d["residual_mult"]),
-                   [LayerSpec.from_dict(x) for x in d["layers"]], d.get("name", ""))
+        scale, loop = 1.0, None
+        if "embedding" in keys:
+            _take(d["embedding"], ("scale",), "embedding")
+            scale = float(d["embedding"]["scale"])
+        if d.get("loop") is not None:
+            loop = LoopSpec.from_dict(d["loop"])
+        mult = float(d["residual_mult"]) if "residual_mult" in keys else 1.0
+        return cls(d["architecture"], int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), mult,
+                   [LayerSpec.from_dict(x) for x in d["layers"]], d.get("name", ""), scale, loop)
 
     def to_dict(self) -> dict:
-        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
-               "residual_mult": self.residual_mult, "layers": [x.to_dict() for x in self.layers]}
+        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps}}
+        keys = self.design.keys
+        if "residual_mult" in keys:
+            out["residual_mult"] = self.residual_mult
+        if "embedding" in keys:
+            out["embedding"] = {"scale": self.embed_scale}
+        if self.loop is not None:
+            out["loop"] = self.loop.to_dict()
+        out["layers"] = [x.to_dict() for x in self.layers]
         if self.name:
             out["name"] = self.name
         return out
@@ -243,9 +484,15 @@ class LayeredConfig:
 
     # -- counts ------------------------------------------------------------------------------------------------------
     def param_count(self) -> int:
-        n = 2 * self.vocab * self.width + self.width
+        E = self.width
+        if self.design.norms == "sandwich":
+            n = 2 * self.vocab * E + 2 * E + (0 if self.loop is None else self.loop.times * E)
+            for layer in self.layers:
+                n += layer.mixer.param_count(E) + 4 * E + (0 if layer.mlp is None else 3 * layer.mlp.ff * E + 4 * E)
+            return n
+        n = 2 * self.vocab * E + E
         for i, layer in enumerate(self.layers):
-            a, E = layer.mixer, self.width
+            a = layer.mixer
             n += a.heads * ((a.dim + a.rot_dim) * E + 2 * a.vdim * E + (a.dim + a.vdim) * a.kv_rank) + E
             if a.kv_from is None:
                 n += (a.kv_rank + a.rot_dim) * E + a.kv_rank

@@ -1,0 +1,379 @@
+"""Sublayers of the layered decoder models: mixers and feed-forwards, each in a prompt form (``stream`` / ``forward``, on a
+``PackedStep``) and a decode form (one token per row).
+
+Weights are stored as they are executed: projections that read the same input are one matrix, row pitches are padded to
+eight elements.  ``checkpoint_tensors`` names the views that make up a checkpoint."""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Callable, Optional
+
+import torch
+import torch.nn as nn
+
+from ..ops import latent as ops
+from ..ops import memory as mem_ops
+from ..ops.latent import LatentLayout, pad8
+from ..ops.memory import BiasTable, MemoryLayout, ParallelLayout
+from .layered_config import (DenseMLPSpec, GatedMemorySpec, LatentAttentionSpec, LayeredConfig, LayerRun, ParallelSpec,
+                             RotarySpec)
+
+
+def weight(rows: int, cols: int, dtype, device) -> nn.Parameter:
+    """[rows, cols] matrix with a zero-filled row pitch that is a multiple of eight."""
+    return nn.Parameter(torch.zeros(rows, pad8(cols), dtype=dtype, device=device), requires_grad=False)
+
+
+def vector(n: int, device) -> nn.Parameter:
+    return nn.Parameter(torch.zeros(n, dtype=torch.float32, device=device), requires_grad=False)
+
+
+def rope_tables(rot: RotarySpec, length: int, device) -> tuple:
+    """cos / sin [length, dims / 2] of the spec's (interpolated) frequencies, times its magnitude.  The angles are formed in
+    double precision and stored as fp32."""
+    ang = torch.outer(torch.arange(length, dtype=torch.float64), torch.tensor(rot.frequencies(), dtype=torch.float64))
+    return tuple((f(ang) * rot.magnitude).float().contiguous().to(device) for f in (torch.cos, torch.sin))
+
+
+# ------------------------------------------------------------------------------------------
+# one packed step
+# ------------------------------------------------------------------------------------------
+@dataclass
+class StreamLayout:
+    """Where the keys of a packed step lie for a given history length: per sequence first the cached positions its portion can
+    still see, then the portion itself."""
+
+    sidx: torch.Tensor        # [T] stream index of every token
+    kbase: torch.Tensor       # [T] stream index of the first key of its sequence
+    seqs: list                # (first token, tokens, first key, history) per sequence
+    total: int
+    history: list             # (row, first position, count, first key) of the sequences with history
+
+
+class PackedStep:
+    """Token ids and positions of a batch of prompt portions; ``portions`` are (row, first position, token ids)."""
+
+    def __init__(self, portions: list, device):
+        self.device, self.portions = torch.device(device), [(r, s, len(t)) for r, s, t in portions]
+        tok, pos, row, end = [], [], [], []
+        for r, s, t in portions:
+            n = len(t)
+            tok.extend(t)
+            pos.extend(range(s, s + n))
+            row.extend([r] * n)
+            end.extend([s + n] * n)
+        self.tok = torch.tensor(tok, dtype=torch.int64).to(self.device)
+        meta = torch.tensor([pos, row, end], dtype=torch.int32).to(self.device)
+        self.pos, self.row, self.end = meta[0], meta[1], meta[2]
+        self.T = len(tok)
+        self._layouts: dict = {}
+        self._seq_table = None
+
+    def sequences(self) -> list:
+        """(first token, tokens, cache row, first position) per portion."""
+        out, t0 = [], 0
+        for r, s, n in self.portions:
+            out.append((t0, n, r, s))
+            t0 += n
+        return out
+
+    @property
+    def seq_table(self) -> torch.Tensor:
+        """``sequences`` as int32 [portions, 4] on the device."""
+        if self._seq_table is None:
+            self._seq_table = torch.tensor(self.sequences(), dtype=torch.int32).to(self.device)
+        return self._seq_table
+
+    def layout(self, history: int) -> StreamLayout:
+        """Layout with up to ``history`` cached positions in front of every portion."""
+        if all(s == 0 for _, s, _ in self.portions):
+            history = 0
+        if history not in self._layouts:
+            seqs, sidx, kbase, hist = [], [], [], []
+            t0 = k0 = 0
+            for r, s, n in self.portions:
+                h = min(s, history)
+                seqs.append((t0, n, k0, h))
+                sidx.extend(range(k0 + h, k0 + h + n))
+                kbase.extend([k0] * n)
+                if h:
+                    hist.append((r, s - h, h, k0))
+                t0, k0 = t0 + n, k0 + h + n
+            idx = torch.tensor([sidx, kbase], dtype=torch.int32).to(self.device)
+            self._layouts[history] = StreamLayout(idx[0], idx[1], seqs, k0, hist)
+        return self._layouts[history]
+
+
+@dataclass
+class StepContext:
+    """What the sublayers of a packed step share."""
+
+    config: LayeredConfig
+    step: PackedStep
+    cache: Optional[object]
+    rope: dict = field(default_factory=dict)       # rotary spec -> (cos, sin)
+    windows: dict = field(default_factory=dict)    # latent source layer -> widest window
+    streams: dict = field(default_factory=dict)    # latent source layer -> latent rows of the step
+
+
+@dataclass
+class DecodeContext:
+    """What the sublayers of a decode step share; ``dense(x, w, which)`` is the engine's narrow-batch product, ``splits(mixer, B)``
+    its number of key splits."""
+
+    config: LayeredConfig
+    pos: torch.Tensor
+    row: torch.Tensor
+    cache: object
+    dense: Callable
+    splits: Callable
+
+
+def gather_history(layout: StreamLayout, cache: torch.Tensor, stream: torch.Tensor) -> None:
+    """Copy the cached latents in front of every portion from the ring ``cache`` [rows, cap, ld] into the stream."""
+    if not layout.history:
+        return
+    cap = cache.shape[1]
+    src, dst = [], []
+    for row, p0, n, k0 in layout.history:
+        src.extend(row * cap + (p % cap) for p in range(p0, p0 + n))
+        dst.extend(range(k0, k0 + n))
+    idx = torch.tensor([src, dst], dtype=torch.int32).to(cache.device)
+    ops.gather_rows(cache.view(-1, cache.shape[2]), idx[0], stream, idx[1])
+
+
+# ------------------------------------------------------------------------------------------
+# sublayers
+# ------------------------------------------------------------------------------------------
+class LatentAttention(nn.Module):
+    """Windowed attention over per-token latents with gated heads; see ``LatentAttentionSpec``."""
+
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: LatentAttentionSpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        a = spec
+        self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
+        L = self.layout = LatentLayout(a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, a.kv_from is None)
+        self.w_in = weight(L.width_in, width, dtype, device)
+        self.w_kv = weight(L.width_kv, a.kv_rank, dtype, device)
+        self.w_o = weight(width, a.heads * a.vdim, dtype, device)
+        self.latent_norm = vector(a.kv_rank, device) if L.own else None
+
+    def checkpoint_tensors(self) -> dict:
+        a, L, E = self.spec, self.layout, self.width
+        out = {"q": self.w_in[:a.heads * (a.dim + a.rot_dim), :E], "g": self.w_in[L.off_g:L.off_g + a.heads * a.vdim, :E],
+               "uk": self.w_kv[:a.heads * a.dim, :a.kv_rank], "uv": self.w_kv[L.off_v:L.off_v + a.heads * a.vdim, :a.kv_rank],
+               "o": self.w_o[:, :a.heads * a.vdim]}
+        if L.own:
+            out["dkv"] = self.w_in[L.off_d:L.off_d + a.kv_rank + a.rot_dim, :E]
+            out["dkv.norm"] = self.latent_norm
+        return out
+
+    def project_stream(self, xb, step: PackedStep, cache, stream, lay: StreamLayout, rope):
+        """The portion's projection rows (q rotated); appends the latents of an own layer to ``stream`` and the ring."""
+        inp = ops.linear(xb, self.w_in[:, :self.width])
+        if self.layout.own and cache is not None:
+            gather_history(lay, cache, stream)     # before the ring slots of the oldest positions are written again
+        ops.latent_prep_(self.layout, inp, self.latent_norm, self.eps, rope, step, lay.sidx, cache if self.layout.own else None,
+                         stream)
+        return inp
+
+    def stream(self, xb, run: LayerRun, ctx: "StepContext"):
+        a, src, step = self.spec, ctx.config.kv_source(run.layer), ctx.step
+        cache, lay = None if ctx.cache is None else ctx.cache.data[src], step.layout(ctx.windows[src] - 1)
+        if src == run.layer:
+            ctx.streams[src] = torch.empty(lay.total, self.layout.ld_lat, dtype=self.dtype, device=xb.device)
+        stream = ctx.streams[src]
+        inp = self.project_stream(xb, step, cache, stream, lay, ctx.rope[a.rot])
+        kv = ops.linear(stream[:, :a.kv_rank], self.w_kv[:, :a.kv_rank])
+        o = ops.stream_attention(self.layout, inp, kv, stream, lay, a.window, a.scale)
+        return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
+
+    def decode_splits(self, B: int, max_len: int, tensor_cores: bool) -> int:
+        """Key splits of the decode attention: enough CTAs to fill the machine, at least 128 keys each."""
+        groups, fill = self.spec.heads, 4 * 148          # generic kernel: a small CTA per head
+        if tensor_cores:
+            from ..ops import latent_attention as A
+
+            n = A.decode_group(self.spec.heads, self.spec.kv_rank, self.layout.ld_lat)
+            if n:                                         # tensor-core kernel: one CTA per SM, n heads each
+                groups, fill = -(-self.spec.heads // n), 148
+        tiles = min(self.spec.window, max_len) // 128 + 1
+        return max(1, min(tiles, 32, fill // max(1, B * groups)))
+
+    def decode(self, xb, run: LayerRun, ctx: "DecodeContext"):
+        """One token per row.  Returns the sublayer output, whether it is an accumulator that the next kernel clears, and
+        the projection's accumulator or None."""
+        a, dense = self.spec, ctx.dense
+        cache = ctx.cache.data[ctx.config.kv_source(run.layer)]
+        inp, acc = dense(xb, self.w_in[:, :self.width], 0)
+        o = ops.ring_attention(self.layout, inp, self.w_kv, self.latent_norm, self.eps, ctx.cache.rope[a.rot], ctx.pos, ctx.row, cache,
+                               min(a.window, cache.shape[1]), a.scale, ctx.splits(self, xb.shape[0]), self.dtype)
+        out, clear = dense(o, self.w_o[:, :a.heads * a.vdim], 1)
+        return out, clear, inp if acc else None
+
+
+class DenseMLP(nn.Module):
+    """down(relu(up x)^2) with biases; the bias of the down projection is added by the norm that follows."""
+
+    act = "relu2"
+    wide = 1           # multiples of ``ff`` that its widest product has
+    out_bias_mult = 1.0
+
+    def __init__(self, spec: DenseMLPSpec, width: int, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.dtype = spec, width, dtype
+        self.w_up, self.b_up = weight(spec.ff, width, dtype, device), vector(spec.ff, device)
+        self.w_down, self.b_down = weight(width, spec.ff, dtype, device), vector(width, device)
+
+    @property
+    def out_bias(self):
+        return self.b_down
+
+    def checkpoint_tensors(self) -> dict:
+        return {"up": self.w_up[:, :self.width], "up.b": self.b_up, "down": self.w_down[:, :self.spec.ff], "down.b": self.b_down}
+
+    def forward(self, xb):
+        return ops.linear(ops.linear(xb, self.w_up[:, :self.width], self.b_up, self.act), self.w_down[:, :self.spec.ff])
+
+    def decode(self, xb, dense):
+        h, clear = dense(xb, self.w_up[:, :self.width], 1)
+        h = ops.bias_act(h, self.b_up, self.act, self.dtype, clear)
+        return dense(h, self.w_down[:, :self.spec.ff], 1)
+
+
+class ParallelMixer(nn.Module):
+    """Distance-biased attention and a decaying memory side by side on the same input (``ParallelSpec``).  One projection feeds
+    both; the two output projections are one product over the concatenated halves, whose fixed weights are applied where the
+    halves are gated (so the stored weights stay as they are)."""
+
+    def __init__(self, spec: ParallelSpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        a, r = spec.left, spec.right
+        if a.bias_rows is None:
+            raise ValueError("the height of the distance-bias table is not known: load a checkpoint or set bias_rows")
+        self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
+        L = self.layout = ParallelLayout(a.heads, a.kv_heads, a.dim, a.vdim, r.heads, r.dim, r.vdim)
+        self.w_in, self.b_in = weight(L.width_in, width, dtype, device), vector(L.width_in, device)
+        self.w_o, self.out_bias = weight(width, L.width_o, dtype, device), vector(width, device)
+        self.out_bias_mult = spec.left_scale
+        self.rel = nn.Parameter(torch.zeros(a.bias_rows, a.heads, dtype=torch.float32, device=device), requires_grad=False)
+        self.norm = vector(r.heads * r.vdim, device)
+        self.register_buffer("decay", torch.tensor(r.decay, dtype=torch.float32).to(device), persistent=False)
+        self.table = None
+
+    def checkpoint_tensors(self) -> dict:
+        a, r, L, E = self.spec.left, self.spec.right, self.layout, self.width
+        out = {}
+        for name, at, n in (("q", L.off_q, a.heads * a.dim), ("k", L.off_k, a.kv_heads * a.dim), ("v", L.off_v, a.kv_heads * a.vdim)):
+            out["left." + name], out["left." + name + ".b"] = self.w_in[at:at + n, :E], self.b_in[at:at + n]
+        out.update({"left.g": self.w_in[L.off_lg:L.off_lg + a.heads, :E], "left.rel": self.rel, "left.o": self.w_o[:, :a.heads * a.vdim],
+                    "left.o.b": self.out_bias})
+        hd, hv = r.heads * r.dim, r.heads * r.vdim
+        for name, at, n in (("q", L.off_rq, hd), ("k", L.off_rk, hd), ("v", L.off_rv, hv), ("g", L.off_rg, hv)):
+            out["right." + name] = self.w_in[at:at + n, :E]
+        out.update({"right.o": self.w_o[:, L.off_r:L.off_r + hv], "right.norm": self.norm})
+        return out
+
+    def weights_changed(self) -> None:
+        """Derive what the kernels read instead of the stored tensors."""
+        self.table = BiasTable.build(self.rel, self.spec.left.buckets())
+
+    def cache_shapes(self, max_len: int) -> dict:
+        r, L = self.spec.right, self.layout
+        return {"kv": ((max_len, L.ld_kv), self.dtype), "state": ((r.heads, r.dim, L.ldv), torch.float32)}
+
+    def stream(self, h, run: LayerRun, ctx: StepContext):
+        L, spec, step = self.layout, self.spec, ctx.step
+        kv, state = ctx.cache.data[run.index, "kv"], ctx.cache.data[run.index, "state"]
+        inp = ops.linear(h, self.w_in[:, :self.width], self.b_in, "silu", act_cols=L.act_cols)
+        mem_ops.kv_append(L, inp, None, kv, step.pos, step.row)
+        o = mem_ops.parallel_output(L, h.shape[0], self.dtype, h.device)
+        mem_ops.prompt_attention(L, spec.left, inp, kv, self.table, step, spec.left_scale, o)
+        m = mem_ops.decay_memory_prompt(L, inp, self.decay, state, step)
+        mem_ops.memory_norm(L, inp, m, self.norm, self.eps, spec.right_scale, o)
+        return ops.linear(o, self.w_o[:, :L.width_o])
+
+    def decode_splits(self, B: int, max_len: int, tensor_cores: bool) -> int:
+        """Key splits of the decode attention: enough CTAs to fill the machine, at least 64 keys each."""
+        ctas = B * mem_ops.decode_groups(self.layout, tensor_cores)
+        return max(1, min(max_len // 64 + 1, 32, -(-2 * 148 // ctas)))
+
+    def decode(self, h, run: LayerRun, ctx: DecodeContext):
+        L = self.layout
+        inp, acc = ctx.dense(h, self.w_in[:, :self.width], 0)
+        o = mem_ops.parallel_decode(L, self.spec, inp, self.b_in, ctx.cache.data[run.index, "kv"], ctx.cache.data[run.index, "state"],
+                                    self.table, self.decay, self.norm, self.eps, ctx.pos, ctx.row, ctx.splits(self, h.shape[0]), self.dtype)
+        out, clear = ctx.dense(o, self.w_o[:, :L.width_o], 1)
+        return out, clear, inp if acc else None
+
+
+class GatedMemory(nn.Module):
+    """Gated matrix memory (``GatedMemorySpec``).  The gates' projections are a product of their own with fp32 results."""
+
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: GatedMemorySpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
+        L = self.layout = MemoryLayout(spec.heads, spec.dim, spec.vdim)
+        self.w_in = weight(L.width_in, width, dtype, device)
+        self.w_gate, self.b_gate = weight(2 * spec.heads, width, dtype, device), vector(2 * spec.heads, device)
+        self.w_o, self.norm = weight(width, spec.heads * spec.vdim, dtype, device), vector(spec.heads * spec.vdim, device)
+
+    def checkpoint_tensors(self) -> dict:
+        a, L, E = self.spec, self.layout, self.width
+        hd, hv = a.heads * a.dim, a.heads * a.vdim
+        out = {name: self.w_in[at:at + n, :E] for name, at, n in (("q", L.off_q, hd), ("k", L.off_k, hd), ("v", L.off_v, hv), ("g", L.off_g, hv))}
+        for name, at in (("i", 0), ("f", a.heads)):
+            out[name], out[name + ".b"] = self.w_gate[at:at + a.heads, :E], self.b_gate[at:at + a.heads]
+        out.update({"o": self.w_o[:, :hv], "norm": self.norm})
+        return out
+
+    def cache_shapes(self, max_len: int) -> dict:
+        a = self.spec
+        return {"state": ((a.heads, a.dim, self.layout.ldv), torch.float32), "norm": ((a.heads, a.dim + 1), torch.float32)}
+
+    def stream(self, h, run: LayerRun, ctx: StepContext):
+        a, data = self.spec, ctx.cache.data
+        inp = ops.linear(h, self.w_in[:, :self.width])
+        gates = ops.linear(h, self.w_gate[:, :self.width], out_f32=True)
+        o = mem_ops.gated_memory(self.layout, inp, gates, self.b_gate, a.gate_cap, data[run.index, "state"], data[run.index, "norm"], self.norm,
+                                 self.eps, self.dtype, step=ctx.step)
+        return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
+
+    def decode(self, h, run: LayerRun, ctx: DecodeContext):
+        a, data = self.spec, ctx.cache.data
+        inp, acc = ctx.dense(h, self.w_in[:, :self.width], 0)
+        o = mem_ops.gated_memory(self.layout, inp, None, self.b_gate, a.gate_cap, data[run.index, "state"], data[run.index, "norm"], self.norm,
+                                 self.eps, self.dtype, rows=(ctx.pos, ctx.row), h=h, w_gate=self.w_gate[:, :self.width])
+        out, clear = ctx.dense(o, self.w_o[:, :a.heads * a.vdim], 1)
+        return out, clear, inp if acc else None
+
+
+class GatedMLP(nn.Module):
+    """down(gelu(gate x) * (up x)), tanh form, no biases."""
+
+    wide = 2
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: DenseMLPSpec, width: int, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.dtype = spec, width, dtype
+        self.w_gu, self.w_down = weight(2 * spec.ff, width, dtype, device), weight(width, spec.ff, dtype, device)
+
+    def checkpoint_tensors(self) -> dict:
+        f, E = self.spec.ff, self.width
+        return {"gate": self.w_gu[:f, :E], "up": self.w_gu[f:, :E], "down": self.w_down[:, :f]}
+
+    def forward(self, h):
+        return ops.linear(mem_ops.geglu_linear(h, self.w_gu[:, :self.width], self.spec.ff), self.w_down[:, :self.spec.ff])
+
+    def decode(self, h, dense):
+        a, clear = dense(h, self.w_gu[:, :self.width], 1)
+        return dense(mem_ops.geglu(a, self.spec.ff, self.dtype, clear), self.w_down[:, :self.spec.ff], 1)
+
+
+MIXERS = {"latent_attention": LatentAttention, "parallel": ParallelMixer, "mlstm": GatedMemory}
+MLPS = {"relu2": DenseMLP, "geglu": GatedMLP}

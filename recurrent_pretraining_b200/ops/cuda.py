@@ -65,7 +65,7 @@ OUT_SWIGLU_SAVE = 8     # SwiGLU epilogue that also stores the pre-activation [g
 OUT_DSWIGLU = 9         # input-gradient GEMM whose epilogue applies the gate's derivative (``resid`` = pre-activation)
 OUT_BF16_LSE = 10       # head GEMM: bf16 logits + per-tile softmax partials + target logit (fused linear + CE)
 OUT_BF16_BIAS_ACT = 11  # bf16 act(acc + bias) with an fp32 column bias
-_set_bias = _sig("b200_gemm_set_bias", [_vp, _i])
+_set_bias = _sig("b200_gemm_set_bias", [_vp, _i, _i, _i])
 _set_lse = _sig("b200_gemm_set_lse", [_vp, _vp, _vp, _f])
 _ce_finish = _sig("b200_ce_finish", [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _f, _i, _f, _i, _vp])
 _set_rope = _sig("b200_gemm_set_rope", [_vp, _vp, _vp, _i, _i, _i])
@@ -147,10 +147,11 @@ def _mat(t: torch.Tensor):
 
 
 def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_mode=OUT_BF16, a2=None, resid=None, n_out=None, bn=0,
-         max_ctas=0, rope=None, lse=None, bias=None, act=0):
+         max_ctas=0, rope=None, lse=None, bias=None, act=0, act_cols=(0, 0)):
     """C[M,N] (+)= A B^T.  ``a``: [M,K] (or [K,M] if a_mn), ``b``: [N,K] (or [K,N] if b_mn).
     ``rope`` (OUT_BF16_ROPE): (cos [S, D/2] fp32, sin, bias flat fp32 or None, S, D, width of the q+k columns).
-    ``bias`` / ``act`` (OUT_BF16_BIAS_ACT): fp32 [N] or None, 0 = no activation, 1 = relu^2."""
+    ``bias`` / ``act`` (OUT_BF16_BIAS_ACT): fp32 [N] or None, 0 = no activation, 1 = relu^2, 2 = silu on the columns
+    ``act_cols`` (multiples of eight); OUT_SWIGLU: ``act`` 3 gates with tanh-gelu instead of silu."""
     a, ar, ac, lda = _mat(a)
     b, br, bc, ldb = _mat(b)
     M, K1 = (ac, ar) if a_mn else (ar, ac)
@@ -197,7 +198,9 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_mode=OUT_BF16, a2=None, 
         bn = 256
     if out_mode == OUT_BF16_BIAS_ACT:
         assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= N)
-        _set_bias(_ptr(bias), int(act))
+        _set_bias(_ptr(bias), int(act), int(act_cols[0]), int(act_cols[1]))
+    elif out_mode == OUT_SWIGLU:
+        _set_bias(0, int(act), 0, 0)
     rc = _gemm(_ptr(a), _ptr(a2), _ptr(b), _ptr(out), _ptr(resid), M, N, K1, K2, lda, lda2, ldb, out.stride(0),
                ld_resid, int(a_mn), int(b_mn), out_mode, bn, max_ctas, _stream(), _ptr(err_word(a.device)))
     _check(rc, "b200_gemm")

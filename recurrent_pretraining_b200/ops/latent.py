@@ -67,7 +67,9 @@ class _WindowAttn(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("H", "d1", "d2", "vdim", "window", "splits")] + [("scale", C.c_float)] + \
                [(n, C.c_int) for n in ("q_stride", "q_head", "k1_stride", "k1_head", "k2_stride", "v_stride", "v_head")] + \
                [(n, C.c_void_p) for n in ("sidx", "kbase", "pos", "row")] + [("cap", C.c_int)] + \
-               [(n, C.c_int) for n in ("gate_ld", "out_ld")] + [(n, C.c_void_p) for n in ("part_o", "part_ml")]
+               [(n, C.c_int) for n in ("gate_ld", "out_ld")] + [(n, C.c_void_p) for n in ("part_o", "part_ml")] + \
+               [("group", C.c_int), ("bias", C.c_void_p), ("bias_len", C.c_int), ("temp_every", C.c_int), ("temp_coef", C.c_float),
+                ("head_gate", C.c_int), ("gate_mult", C.c_float)]
 
 
 _fns = None
@@ -85,7 +87,7 @@ def _k():
         row, att = C.POINTER(_LatentRow), C.POINTER(_WindowAttn)
         _fns = SimpleNamespace(
             K=K,
-            embed=K._sig("b200_embed_resid", [vp] * 4 + [i] * 4 + [ll, i, vp, vp]),
+            embed=K._sig("b200_embed_resid", [vp] * 4 + [i] * 4 + [f, ll, i, vp, vp]),
             prep=K._sig("b200_latent_prep", [vp, row] + [vp] * 4 + [i, i, vp]),
             absorb=K._sig("b200_latent_absorb", [vp, row, vp, i, vp, vp, i, i, i, vp]),
             gather=K._sig("b200_gather_rows", [vp] * 4 + [i, i, vp]),
@@ -94,7 +96,7 @@ def _k():
             resid=K._sig("b200_rms_residual", [vp] + [i] * 3 + [vp] * 4 + [i] * 3 + [f, f, vp, i, i, vp]),
             norm_rows=K._sig("b200_rmsnorm_rows", [vp] * 4 + [i] * 3 + [f, i, vp]),
             bias_act=K._sig("b200_bias_act", [vp] + [i] * 3 + [vp, vp] + [i] * 5 + [vp]),
-            sgemm=K._sig("b200_sgemm_nt", [vp] * 4 + [i] * 7 + [vp]),
+            sgemm=K._sig("b200_sgemm_nt", [vp] * 4 + [i] * 9 + [vp]),
         )
     return _fns
 
@@ -103,7 +105,7 @@ def _f32(t) -> int:
     return int(t.dtype == F32)
 
 
-_ACT = {None: 0, "relu2": 1}
+_ACT = {None: 0, "relu2": 1, "silu": 2}
 
 
 # ------------------------------------------------------------------------------------------
@@ -119,27 +121,27 @@ def _pitched(y: torch.Tensor, ld: int) -> torch.Tensor:
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: Optional[str] = None,
-           out_f32: bool = False, ld_out: int = 0) -> torch.Tensor:
+           out_f32: bool = False, ld_out: int = 0, act_cols: tuple = (0, 0)) -> torch.Tensor:
     """act(x w^T + bias) for x [M, K] and w [N, K] of one storage dtype (rows may be pitched); result [M, N] in that dtype,
-    or fp32 with ``out_f32`` (no bias then).  bf16: tcgen05 GEMM with the bias and the activation in its epilogue.
+    or fp32 with ``out_f32`` (no bias then).  ``act`` "silu" applies to the columns ``act_cols`` (multiples of eight).  bf16: tcgen05 GEMM with the bias and the activation in its epilogue.
     fp32: true fp32 product."""
     M, Kd = x.shape
     N = w.shape[0]
     assert x.dtype == w.dtype and w.shape[1] == Kd and not (out_f32 and (bias is not None or act))
     if not x.is_cuda:
-        y = ref.linear_act(x, w, bias, act)
+        y = ref.linear_act(x, w, bias, act, act_cols)
         return _pitched(y.float() if out_f32 else y, ld_out)
     k = _k()
     out = torch.empty(M, max(ld_out, pad8(N)), dtype=F32 if out_f32 else x.dtype, device=x.device)[:, :N]
     if x.dtype == F32:
         k.K._check(k.sgemm(x.data_ptr(), w.data_ptr(), k.K._ptr(bias), out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0),
-                           out.stride(0), _ACT[act], k.K._stream()), "sgemm_nt")
+                           out.stride(0), _ACT[act], act_cols[0], act_cols[1], k.K._stream()), "sgemm_nt")
         return out
     if out_f32:
         return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_F32)
     if bias is None and act is None:
         return k.K.gemm(x, w, out=out)
-    return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_BF16_BIAS_ACT, bias=bias, act=_ACT[act])
+    return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_BF16_BIAS_ACT, bias=bias, act=_ACT[act], act_cols=act_cols)
 
 
 def bias_act(a: torch.Tensor, bias: Optional[torch.Tensor], act: Optional[str], dtype: torch.dtype, clear: bool = False) -> torch.Tensor:
@@ -158,18 +160,18 @@ def bias_act(a: torch.Tensor, bias: Optional[torch.Tensor], act: Optional[str], 
 # ------------------------------------------------------------------------------------------
 # residual stream
 # ------------------------------------------------------------------------------------------
-def embed(tok: torch.Tensor, table: torch.Tensor):
-    """(fp32 residual [T, E], operand copy [T, E]) of token ids [T]."""
+def embed(tok: torch.Tensor, table: torch.Tensor, scale: float = 1.0, copy: bool = True):
+    """(fp32 residual [T, E] = scale * table row, operand copy [T, E] or None) of token ids [T]."""
     T, E = tok.numel(), table.shape[1]
     if not tok.is_cuda:
-        x = table[tok].float()
-        return x, x.to(table.dtype)
+        x = table[tok].float() * scale
+        return x, x.to(table.dtype) if copy else None
     k = _k()
     assert tok.dtype == torch.int64 and tok.is_contiguous()
     x = torch.empty(T, E, dtype=F32, device=tok.device)
-    xb = torch.empty(T, pad8(E), dtype=table.dtype, device=tok.device)[:, :E]
-    k.K._check(k.embed(tok.data_ptr(), table.data_ptr(), x.data_ptr(), xb.data_ptr(), T, E, table.stride(0), xb.stride(0),
-                       table.shape[0], _f32(table), k.K.err_word(tok.device).data_ptr(), k.K._stream()), "embed_resid")
+    xb = torch.empty(T, pad8(E), dtype=table.dtype, device=tok.device)[:, :E] if copy else None
+    k.K._check(k.embed(tok.data_ptr(), table.data_ptr(), x.data_ptr(), k.K._ptr(xb), T, E, table.stride(0), xb.stride(0) if copy else 0,
+                       scale, table.shape[0], _f32(table), k.K.err_word(tok.device).data_ptr(), k.K._stream()), "embed_resid")
     return x, xb
 
 
@@ -284,7 +286,8 @@ def stream_attention(L: LatentLayout, inp: torch.Tensor, kv: torch.Tensor, strea
             A.stream_attention(L, inp, kv, stream, layout, window, scale, out)
             return out
     a = _WindowAttn(L.heads, L.dim, L.rot, L.vdim, window, 1, scale, inp.stride(0), hd, kv.stride(0), L.dim, stream.stride(0),
-                    kv.stride(0), L.vdim, layout.sidx.data_ptr(), layout.kbase.data_ptr(), 0, 0, 0, inp.stride(0), out.stride(0), 0, 0)
+                    kv.stride(0), L.vdim, layout.sidx.data_ptr(), layout.kbase.data_ptr(), 0, 0, 0, inp.stride(0), out.stride(0), 0, 0, 1,
+                    gate_mult=1.0)
     k.K._check(k.attn(inp.data_ptr(), kv.data_ptr(), kr.data_ptr(), kv[:, L.off_v:].data_ptr(), gate.data_ptr(), out.data_ptr(),
                       C.byref(a), T, _f32(inp), k.K._stream()), "window_attention")
     return out
@@ -345,7 +348,7 @@ def ring_attention_pieces(L: LatentLayout, inp, w_kv, norm_w, eps: float, rope, 
                 A.ring_attention(L, qlat, cache, pos, row, part_o, part_ml, window, splits, scale)
                 return
         a = _WindowAttn(L.heads, L.ld_lat, 0, L.rank, window, splits, scale, L.heads * L.ld_lat, L.ld_lat, L.ld_lat, 0, 0, L.ld_lat, 0,
-                        0, 0, pos.data_ptr(), row.data_ptr(), cap, 0, 0, part_o.data_ptr(), part_ml.data_ptr())
+                        0, 0, pos.data_ptr(), row.data_ptr(), cap, 0, 0, part_o.data_ptr(), part_ml.data_ptr(), 1)
         k.K._check(k.attn(qlat.data_ptr(), cache.data_ptr(), 0, cache.data_ptr(), 0, 0, C.byref(a), B, f32, k.K._stream()),
                    "window_attention")
 

@@ -164,13 +164,16 @@ def relu2(x: torch.Tensor) -> torch.Tensor:
     return F.relu(x).square()
 
 
-def linear_act(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None) -> torch.Tensor:
-    """act(x w^T + bias) with an fp32 bias; result in x.dtype."""
+def linear_act(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None,
+               act_cols: tuple = (0, 0)) -> torch.Tensor:
+    """act(x w^T + bias) with an fp32 bias; result in x.dtype.  "silu" applies to the columns ``act_cols``."""
     y = F.linear(x, w).float()
     if bias is not None:
         y = y + bias
     if act == "relu2":
         y = relu2(y)
+    elif act == "silu":
+        y[:, act_cols[0]:act_cols[1]] = F.silu(y[:, act_cols[0]:act_cols[1]])
     elif act is not None:
         raise ValueError(f"unknown activation {act!r}")
     return y.to(x.dtype)
@@ -201,3 +204,53 @@ def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, visible:
     s = torch.einsum("thd,tkhd->thk" if per_query else "thd,khd->thk", q, k) * scale
     p = torch.softmax(s.masked_fill(~visible[:, None], float("-inf")), dim=-1)
     return torch.einsum("thk,tkhd->thd" if per_query else "thk,khd->thd", p, v)
+
+
+# ------------------------------------------------------------------------------------------
+# layered decoder models: layer norms around sublayers, distance-biased attention, matrix memories
+# ------------------------------------------------------------------------------------------
+def layer_norm(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> torch.Tensor:
+    x = x.float()
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt(d.square().mean(-1, keepdim=True) + eps) * w + b
+
+
+def biased_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, bias: torch.Tensor, pos: torch.Tensor, scale: torch.Tensor) -> torch.Tensor:
+    """Causal grouped-query attention of one sequence: q [T, H, D] at positions ``pos`` [T], k, v [N, G, .] of the positions
+    0 .. N - 1, ``bias`` [H, distances] (its last entry holds for every farther distance), ``scale`` [T] on the products."""
+    H, G = q.shape[1], k.shape[1]
+    k, v = (t.float().repeat_interleave(H // G, dim=1) for t in (k, v))
+    dist = pos[:, None] - torch.arange(k.shape[0])[None]
+    s = torch.einsum("thd,khd->thk", q.float(), k) * scale[:, None, None]
+    s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)].transpose(0, 1)
+    p = torch.softmax(s.masked_fill((dist < 0)[:, None], float("-inf")), dim=-1)
+    return torch.einsum("thk,khd->thd", p, v)
+
+
+def memory_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, decay: torch.Tensor) -> torch.Tensor:
+    """S = decay S + k v^T, o = S^T q per token and head; q, k [T, H, D], v [T, H, E], ``state`` [H, D, E] is updated."""
+    out = []
+    for t in range(q.shape[0]):
+        state.copy_(decay[:, None, None] * state + k[t, :, :, None] * v[t, :, None, :])
+        out.append(torch.einsum("hde,hd->he", state, q[t]))
+    return torch.stack(out)
+
+
+def gated_memory_scan(q, k, v, log_i, log_f, state, norm, peak) -> torch.Tensor:
+    """Matrix memory with normaliser ``norm`` [H, D] and running maximum ``peak`` [H] of the log gates [T, H]."""
+    out = []
+    for t in range(q.shape[0]):
+        m = torch.maximum(log_f[t] + peak, log_i[t])
+        a, b = torch.exp(log_f[t] + peak - m), torch.exp(log_i[t] - m)
+        state.copy_(a[:, None, None] * state + b[:, None, None] * k[t, :, :, None] * v[t, :, None, :])
+        norm.copy_(a[:, None] * norm + b[:, None] * k[t])
+        peak.copy_(m)
+        den = torch.maximum((norm * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out.append(torch.einsum("hde,hd->he", state, q[t]) / den[:, None])
+    return torch.stack(out)
+
+
+def log_gates(raw: torch.Tensor, bias: torch.Tensor, cap: float):
+    """Log input gate and log forget gate [T, H] of raw projections [T, 2H]."""
+    i, f = (cap * torch.tanh((raw.float() + bias) / cap)).chunk(2, dim=-1)
+    return i, F.logsigmoid(f)

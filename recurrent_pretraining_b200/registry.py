@@ -204,11 +204,32 @@ def _gasovik(name, vocab, width, layers, heads, dim, rot_dim, vdim, kv_rank, win
             "residual_mult": 0.5, "layers": out}
 
 
+def _fatudra(name, vocab, width, layers, left, right, memory, ff, loop=None, bias_rows=32, bias_max=512):
+    """``layers`` layers in a repeating order of four: parallel, gated memory, parallel, parallel.  ``left``: (heads, kv heads,
+    dim, vdim), ``right`` and ``memory``: (heads, dim, vdim)."""
+    h, g, d, v = left
+    par = {"left": {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": d ** -0.5, "bias_max": bias_max, "bias_rows": bias_rows,
+                    "q_temp": {"coef": 0.1, "every": 4096}},
+           "right": {"heads": right[0], "dim": right[1], "vdim": right[2], "decay": [1 - 2.0 ** -(3 + 6 * i / right[0]) for i in range(right[0])]},
+           "left_scale": 0.7, "right_scale": 0.7}
+    mem = {"heads": memory[0], "dim": memory[1], "vdim": memory[2], "gate_cap": 15.0}
+    out = {"name": name, "architecture": "Fatudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+           "embedding": {"scale": width ** 0.5},
+           "layers": [{"type": "mlstm" if i % 4 == 1 else "parallel", "mixer": mem if i % 4 == 1 else par, "mlp": {"kind": "dense", "ff": ff}}
+                      for i in range(layers)]}
+    if loop is not None:
+        out["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return out
+
+
 layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _gasovik("gasovik-tiny", 512, 128, 3, 4, 32, 16, 32, 64, 24, 256, share_from=2, original=64),
     _gasovik("gasovik-1b", 65536, 2048, 16, 16, 128, 64, 128, 512, 1024, 8192, share_from=12),
     # layers of the width and depth of the 3.5B recurrent flagship's core, for side-by-side timing
     _gasovik("gasovik-core-5280", 65536, 5280, 4, 55, 96, 32, 96, 512, 4096, 17920),
+    _fatudra("fatudra-tiny", 512, 128, 4, (4, 2, 32, 32), (2, 32, 32), (2, 16, 32), 256, loop=(1, 3, 2), bias_rows=8, bias_max=64),
+    _fatudra("fatudra-1b", 65536, 2048, 16, (16, 4, 128, 128), (8, 128, 128), (8, 64, 128), 4608),
+    _fatudra("fatudra-core-5280", 65536, 5280, 4, (55, 11, 96, 96), (22, 96, 96), (22, 96, 192), 14080),
 )}
 
 name_to_config: dict[str, dict] = {c["name"]: c for c in configs}

@@ -126,7 +126,7 @@ def layer_ops_prefill(model, seqs: list, t: Timer) -> list:
          2.0 * T * (a.heads * (a.dim + a.rot_dim + 2 * a.vdim) + L.width_kv + a.rot_dim),
          2.0 * visible_pairs(seqs, a.window) * a.heads * (a.dim + a.rot_dim + a.vdim))
     gemm("output projection", lambda: ops.linear(o, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)
-    t.op("rms_residual", lambda: ops.rms_residual_(x, out, None, layer.norm1, 1e-6, 1e-6, torch.bfloat16), T * E * 12.0, 0)
+    t.op("rms_residual", lambda: ops.rms_residual_(x, out, None, layer.norms["norm1"], 1e-6, 1e-6, torch.bfloat16), T * E * 12.0, 0)
     if layer.mlp is not None:
         ff = layer.mlp.spec.ff
         h = ops.linear(xb, layer.mlp.w_up[:, :E], layer.mlp.b_up, "relu2")
@@ -172,7 +172,7 @@ def layer_ops_decode(model, B: int, context: int, t: Timer) -> list:
     o = torch.randn(B, a.heads * a.vdim, device="cuda").bfloat16()
     skinny("output projection", o, mix.w_o[:, :a.heads * a.vdim])
     acc = work[:, :E]
-    t.op("rms_residual", lambda: ops.rms_residual_(x, acc, None, layer.norm1, 1e-6, 1e-6, torch.bfloat16), B * E * 14.0, 0)
+    t.op("rms_residual", lambda: ops.rms_residual_(x, acc, None, layer.norms["norm1"], 1e-6, 1e-6, torch.bfloat16), B * E * 14.0, 0)
     if layer.mlp is not None:
         ff = layer.mlp.spec.ff
         skinny("up projection", xb, layer.mlp.w_up[:, :E])
