@@ -1,4 +1,5 @@
-// Sliding-window attention of a packed prompt step for latent-attention layers, on the 5th-generation tensor cores.
+// Attention of a packed prompt step of the layered decoder models, on the 5th-generation tensor cores.  Two kinds of layers:
+// sliding-window latent attention, and (BIAS) causal grouped-query attention with a learned bias per head and distance.
 //
 // Queries [T, H, dim + rot], unrotated keys [K, H, dim] and values [K, H, vdim] (one packed matrix), one rotated key part
 // [K, rot] shared by all heads.  Every size that is a multiple of eight is taken as it is: operand panels are 64 columns
@@ -12,6 +13,10 @@
 //   warp 9           MMA issuer: S = Q K^T over the unrotated and rotated panels, O += P V with P in tensor memory
 // Only key blocks that some query of a tile can see are visited.  The epilogue divides by the softmax sum and applies the
 // layer's output gate.
+//
+// BIAS: keys and values come straight from the cache (key index = row * capacity + position), there is no rotated part, a
+// query's scores carry its temperature and the gate is one number per head.  Blocks whose distances all lie in one bucket
+// add a constant; the others (those near the diagonal) read the bias per element, lanes at consecutive distances.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -33,7 +38,16 @@ struct LatentAttnParams {
   __nv_bfloat16* out;           // [T, ld_out]
   int ld_gate, ld_out;
   int* err;
+  // BIAS
+  int group;                    // query heads per key / value head
+  const float* bias;            // [H, ld_bias] in log2 units; distance d at column LA_BIAS_LEAD + d
+  const int* bucket;            // [bias_len] bucket of each distance; the last entry holds for all farther ones
+  int bias_len, ld_bias;
+  int temp_every;               // 0: no temperature
+  float temp_coef, gate_mult;
 };
+// Columns in front of distance 0 and behind the last stored one (repeating the values there): a block's accesses need no clamps.
+constexpr int LA_BIAS_LEAD = 256, LA_BIAS_TAIL = 256;
 
 // Position in a ring of `n` stages: stage index and the parity of the pass over the ring.
 struct RingPos {
@@ -55,7 +69,7 @@ struct LatentAttnBars {
 // SN, SR: 16-column MMA steps of the unrotated and rotated parts, known at compile time for common sizes (a block's score
 // product is then a straight line of MMAs: the issuing thread's address arithmetic would otherwise pace the whole block);
 // 0: read from the parameters.
-template <int BN, int SN, int SR>
+template <int BN, int SN, int SR, bool BIAS = false>
 __global__ void __launch_bounds__(384, 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
                    const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
@@ -76,7 +90,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   volatile int* abort_flag = &bars->abort_flag;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x;
+  const int h = blockIdx.x, hk = BIAS ? h / p.group : h;
   const int4 tile = p.tiles[blockIdx.y];
   const int q0 = tile.x, nrows = tile.y, s0 = tile.z, kbase = tile.w;
   const int kstart = max(kbase, s0 - p.window + 1);
@@ -96,7 +110,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   };
   auto load_k = [&](int j, int s) {
     mbar_expect_tx(&bars->k_full[s], k_bytes);
-    for (int c = 0; c < pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, h);
+    for (int c = 0; c < pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, hk);
     for (int c = 0; c < pr; ++c)
       tma_load_2d(sK + s * k_bytes + (pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
   };
@@ -104,9 +118,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   // the TMA thread sets up the barriers and requests the queries and the first key block before the CTA-wide sync
   if (threadIdx.x == 256) {
     tma_prefetch_desc(&tmQn);
-    tma_prefetch_desc(&tmQr);
     tma_prefetch_desc(&tmKn);
-    tma_prefetch_desc(&tmKr);
+    if constexpr (!BIAS) {
+      tma_prefetch_desc(&tmQr);
+      tma_prefetch_desc(&tmKr);
+    }
     tma_prefetch_desc(&tmV);
     for (int i = 0; i < LA_MAX_STAGES; ++i) {
       mbar_init(&bars->k_full[i], 1);
@@ -163,7 +179,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           if (!mbar_wait(&bars->v_empty[s], v.ph ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
           mbar_expect_tx(&bars->v_full[s], v_bytes);
           for (int c = 0; c < p.pv; ++c)
-            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, kstart + j * BN, h);
+            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, kstart + j * BN, hk);
           issued = j + 1;
         }
         for (int j = max(0, issued - p.vst); j < issued; ++j) {
@@ -171,7 +187,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           while (!mbar_try_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
         }
       }
-    } else if (warp >= 10) {
+    } else if (!BIAS && warp >= 10) {
       // bring the CTA's gate rows into L2 while the blocks are processed
       const int lines = (2 * p.vdim + 127) / 128;
       for (int i = threadIdx.x - 320; i < nrows * lines; i += 64) {
@@ -261,7 +277,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t ts = tmem_base + x * BN + lane_addr;
     const uint32_t to = tmem_base + O_COL + x * O_WIDTH + lane_addr;
-    const float scale_log2 = p.scale_log2;
+    float scale_log2 = p.scale_log2;
+    const float* btab = nullptr;
+    if constexpr (BIAS) {
+      if (p.temp_every > 0)
+        scale_log2 *= 1.f + p.temp_coef * logf(static_cast<float>((kstart + hi - kbase + 1) / p.temp_every + 1));
+      btab = p.bias + static_cast<size_t>(h) * p.ld_bias + LA_BIAS_LEAD;
+    }
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = jb; j < je && ok; ++j) {
@@ -282,6 +304,19 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         for (int i = 0; i < BN; ++i)
           if (i < cmin || i > cmax) sv[i] = -INFINITY;
       }
+      float mul = scale_log2, add = 0.f;      // log2 score = mul * sv + add
+      if constexpr (BIAS) {
+        const int d0 = s0 - kstart + x * LA_BM - j * BN, far = p.bias_len - 1;   // distance of the tile's first row to the block's first key
+        const int dmin = d0 - (BN - 1), dmax = d0 + LA_BM - 1;
+        if (dmin >= far || (dmin >= 0 && p.bucket[dmin] == p.bucket[min(dmax, far)])) {
+          add = btab[min(dmin, far)];
+        } else {
+          const float* b = btab + (hi - j * BN);
+#pragma unroll
+          for (int i = 0; i < BN; ++i) sv[i] = fmaf(sv[i], scale_log2, b[-i]);
+          mul = 1.f;
+        }
+      }
       float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
       for (int i = 4; i + 7 < BN; i += 8) {
@@ -293,7 +328,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       mx4[0] = fmax3(mx4[0], sv[BN - 4], sv[BN - 3]);
       mx4[1] = fmax3(mx4[1], sv[BN - 2], sv[BN - 1]);
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      const float m_new = fmaxf(m, mx * scale_log2);
+      const float m_new = fmaxf(m, fmaf(mx, mul, add));
       // raise the reference max only when it moved by more than the threshold (decided per warp)
       const bool grow = (m_new - m > RESCALE_THRESHOLD) || (m == -INFINITY);
       if (__any_sync(0xffffffffu, grow)) {
@@ -312,8 +347,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         l *= alpha;
         m = m_new;
       }
-      const float neg_m = (m == -INFINITY) ? 0.f : -m;        // a row may see nothing of the tile's first blocks
-      const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(scale_log2, scale_log2);
+      const float neg_m = (m == -INFINITY) ? 0.f : add - m;   // a row may see nothing of the tile's first blocks
+      const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(mul, mul);
       float2 rs[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
       for (int c = 0; c < BN; c += 32) {
@@ -340,25 +375,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       const int r = x * LA_BM + quad * 32 + lane;              // query of this thread inside the CTA's 256
       const bool live = r < nrows;
       const size_t t = live ? static_cast<size_t>(q0) + r : 0;
-      const __nv_bfloat16* grow_ = p.gate + t * p.ld_gate + h * p.vdim;
       __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
-      uint4 gq[16];                                             // up to 128 gate values, requested before the last product ends
-      auto load_gate = [&](int c0) {
-#pragma unroll
-        for (int q = 0; q < 16; ++q)
-          if (c0 + 8 * q < p.vdim) gq[q] = *reinterpret_cast<const uint4*>(grow_ + c0 + 8 * q);
-      };
-      load_gate(0);
-      if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
-        tc_fence_after();
-        const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
+      if constexpr (BIAS) {
+        const float g = p.gate_mult / (1.f + __expf(-bf2f(p.gate[t * p.ld_gate + h])));
+        if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
+          tc_fence_after();
+          const float f = (l > 0.f) ? g / l : 0.f;
 #pragma unroll 1
-        for (int c0 = 0; c0 < p.vdim; c0 += 128) {
-          if (c0) load_gate(c0);
-#pragma unroll
-          for (int b = 0; b < 4; ++b) {
-            const int c = c0 + 32 * b;
-            if (c >= p.vdim) break;
+          for (int c = 0; c < p.vdim; c += 32) {
             uint32_t v[32];
             tmem_ld_32x32(to + c, v);
             tmem_ld_wait();
@@ -366,16 +390,53 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
 #pragma unroll
               for (int q = 0; q < 4; ++q) {
                 if (c + 8 * q < p.vdim) {
-                  const uint4 g4 = gq[4 * b + q];
-                  const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
                   uint32_t o[4];
 #pragma unroll
-                  for (int i = 0; i < 4; ++i) {
-                    const float2 g = unpack_bf16x2(gw[i]);
-                    o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * inv_l / (1.f + __expf(-g.x)),
-                                       __uint_as_float(v[8 * q + 2 * i + 1]) * inv_l / (1.f + __expf(-g.y)));
-                  }
+                  for (int i = 0; i < 4; ++i)
+                    o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * f, __uint_as_float(v[8 * q + 2 * i + 1]) * f);
                   *reinterpret_cast<uint4*>(orow + c + 8 * q) = make_uint4(o[0], o[1], o[2], o[3]);
+                }
+              }
+            }
+          }
+        }
+      } else {
+        const __nv_bfloat16* grow_ = p.gate + t * p.ld_gate + h * p.vdim;
+        uint4 gq[16];                                             // up to 128 gate values, requested before the last product ends
+        auto load_gate = [&](int c0) {
+  #pragma unroll
+          for (int q = 0; q < 16; ++q)
+            if (c0 + 8 * q < p.vdim) gq[q] = *reinterpret_cast<const uint4*>(grow_ + c0 + 8 * q);
+        };
+        load_gate(0);
+        if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
+          tc_fence_after();
+          const float inv_l = (l > 0.f) ? 1.f / l : 0.f;
+  #pragma unroll 1
+          for (int c0 = 0; c0 < p.vdim; c0 += 128) {
+            if (c0) load_gate(c0);
+  #pragma unroll
+            for (int b = 0; b < 4; ++b) {
+              const int c = c0 + 32 * b;
+              if (c >= p.vdim) break;
+              uint32_t v[32];
+              tmem_ld_32x32(to + c, v);
+              tmem_ld_wait();
+              if (live) {
+  #pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                  if (c + 8 * q < p.vdim) {
+                    const uint4 g4 = gq[4 * b + q];
+                    const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+                    uint32_t o[4];
+  #pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                      const float2 g = unpack_bf16x2(gw[i]);
+                      o[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * inv_l / (1.f + __expf(-g.x)),
+                                         __uint_as_float(v[8 * q + 2 * i + 1]) * inv_l / (1.f + __expf(-g.y)));
+                    }
+                    *reinterpret_cast<uint4*>(orow + c + 8 * q) = make_uint4(o[0], o[1], o[2], o[3]);
+                  }
                 }
               }
             }
@@ -426,7 +487,7 @@ struct LatentAttnPlan { int bn, kst, vst, smem; };
 // Key-block width and ring depths for the given sizes; bn = 0: not covered.
 static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   LatentAttnPlan none = {0, 0, 0, 0};
-  if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot <= 0 || vdim <= 0) return none;
+  if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot < 0 || vdim <= 0) return none;
   const int kp = (dim + 63) / 64 + (rot + 63) / 64, pv = (vdim + 63) / 64;
   constexpr int LIMIT = 227 * 1024, FIXED = 1024 + 1024;   // barriers, alignment
   for (int bn = 128; bn >= 64; bn -= 64) {
@@ -441,9 +502,9 @@ static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   return none;
 }
 
-template <int BN, int SN, int SR>
+template <int BN, int SN, int SR, bool BIAS = false>
 static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
-  auto kern = latent_attn_kernel<BN, SN, SR>;
+  auto kern = latent_attn_kernel<BN, SN, SR, BIAS>;
   static int configured = 0;
   if (configured < plan.smem) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess) return -10;
@@ -468,7 +529,7 @@ static int dispatch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p
 
 using namespace b200;
 
-B200_API int b200_latent_attention_supported(int dim, int rot, int vdim) { return latent_attn_plan(dim, rot, vdim).bn > 0; }
+B200_API int b200_latent_attention_supported(int dim, int rot, int vdim) { return rot > 0 && latent_attn_plan(dim, rot, vdim).bn > 0; }
 
 // q: [T, ld_q] (head h at column h (dim + rot)), kn / v: [K, ld_kv] (head h at column h dim / h vdim), kr: [K, ld_kr],
 // gate: [T, ld_gate], out: [T, ld_out]; tiles: int4 [n_tiles] as in LatentAttnParams.
@@ -476,7 +537,7 @@ B200_API int b200_latent_attention(const void* q, const void* kn, const void* kr
                                    const int* tiles, int n_tiles, int T, int K, int H, int dim, int rot, int vdim, int ld_q, int ld_kv,
                                    int ld_kr, int ld_gate, int ld_out, int window, float scale, void* stream, int* err) {
   const LatentAttnPlan plan = latent_attn_plan(dim, rot, vdim);
-  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || T <= 0 || K <= 0 || window <= 0) return -1;
+  if (!plan.bn || rot <= 0 || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || T <= 0 || K <= 0 || window <= 0) return -1;
   if ((reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) || (ld_gate & 7) || (ld_out & 7)) return -2;
   CUtensorMap tm[5];
   const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(q);
@@ -497,4 +558,45 @@ B200_API int b200_latent_attention(const void* q, const void* kn, const void* kr
   p.err = err;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return dispatch_latent_attn(tm, p, plan, n_tiles, st);
+}
+
+B200_API int b200_biased_attention_supported(int dim, int vdim) { return latent_attn_plan(dim, 0, vdim).bn > 0; }
+B200_API int b200_biased_attention_pad(int tail) { return tail ? LA_BIAS_TAIL : LA_BIAS_LEAD; }
+
+// q: [T, ld_q] (head h at column h dim), k / v: cache [K, ld_kv] (head g at column g dim / g vdim), gate: [T, ld_gate] (head h at
+// column h), out: [T, ld_out]; tiles as in LatentAttnParams; bias, bucket: see there.  scale > 0, temp_coef >= 0.
+B200_API int b200_biased_attention(const void* q, const void* k, const void* v, const void* gate, void* out, const int* tiles,
+                                   const float* bias, const int* bucket, int n_tiles, int T, int K, int H, int G, int dim, int vdim,
+                                   int ld_q, int ld_kv, int ld_gate, int ld_out, int bias_len, int ld_bias, int temp_every,
+                                   float temp_coef, float scale, float gate_mult, void* stream, int* err) {
+  const LatentAttnPlan plan = latent_attn_plan(dim, 0, vdim);
+  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || G <= 0 || H % G || T <= 0 || K <= 0 || bias_len <= 0 || !(scale > 0.f) ||
+      temp_coef < 0.f || ld_bias < LA_BIAS_LEAD + bias_len + LA_BIAS_TAIL) return -1;
+  if ((reinterpret_cast<uintptr_t>(out) & 15) || (ld_out & 7)) return -2;
+  CUtensorMap tm[5];
+  int rc = make_tmap_rows(&tm[0], q, dim, H, T, dim, ld_q, LA_BM);
+  if (!rc) rc = make_tmap_rows(&tm[2], k, dim, G, K, dim, ld_kv, plan.bn);
+  if (!rc) rc = make_tmap_rows(&tm[4], v, vdim, G, K, vdim, ld_kv, plan.bn);
+  if (rc) return rc;
+  tm[1] = tm[0];
+  tm[3] = tm[2];
+  LatentAttnParams p = {};
+  p.H = H; p.dim = dim; p.rot = 0; p.vdim = vdim; p.window = 1 << 30;
+  p.pn = (dim + 63) / 64; p.pr = 0; p.pv = (vdim + 63) / 64;
+  p.kst = plan.kst; p.vst = plan.vst;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.tiles = reinterpret_cast<const int4*>(tiles);
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
+  p.err = err;
+  p.group = H / G; p.bias = bias; p.bucket = bucket; p.bias_len = bias_len; p.ld_bias = ld_bias;
+  p.temp_every = temp_every; p.temp_coef = temp_coef; p.gate_mult = gate_mult;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (plan.bn == 64) return launch_latent_attn<64, 0, 0, true>(tm, p, plan, n_tiles, st);
+  switch ((dim + 15) / 16) {
+    case 8: return launch_latent_attn<128, 8, 0, true>(tm, p, plan, n_tiles, st);
+    case 6: return launch_latent_attn<128, 6, 0, true>(tm, p, plan, n_tiles, st);
+    case 4: return launch_latent_attn<128, 4, 0, true>(tm, p, plan, n_tiles, st);
+    default: return launch_latent_attn<128, 0, 0, true>(tm, p, plan, n_tiles, st);
+  }
 }

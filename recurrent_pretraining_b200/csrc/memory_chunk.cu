@@ -1,0 +1,571 @@
+// Matrix memories over packed prompts, in chunks of 128 tokens on the 5th-generation tensor cores.
+//
+// A memory S_t = a_t S_(t-1) + b_t k_t v_t^T with one scalar pair per head and token is a product inside a chunk and a short
+// recurrence between chunks.  With F the running sum of log a inside a chunk and i = log b:
+//   chunk_state : U = sum_j exp(F_end - F_j + i_j - m_loc) k_j v_j^T                              per (chunk, head), in parallel
+//   chunk_scan  : S before every chunk, S <- exp(F_end + m - m') S + exp(m_loc - m') U             per (sequence, head)
+//   chunk_out   : o_t = sum_(j <= t) exp(F_t - F_j + i_j - m_t) (q_t . k_j) v_j + exp(F_t + m - m_t) S^T q_t
+// A fixed decay has i = 0 and needs no maxima m.  A gated memory carries the running maximum m (starting at 0) and its
+// normaliser n, which rides along as one more value column of ones.
+// Decays, gates, maxima, sums and the carried state are fp32.  Operands that stem from the state or carry a decay (S and the
+// weighted keys) enter the products as a bf16 head plus a bf16 remainder.
+// Between the kernels a state is stored transposed, [value rows][key columns], as chunk_out reads it.
+#include <cuda.h>
+
+#include "rowops.cuh"
+#include "softmax_math.cuh"
+
+namespace b200 {
+
+constexpr int MC_C = 128;                     // tokens per chunk
+constexpr int MC_PANEL = MC_C * 128;          // 128 rows x 64 bf16
+constexpr float LOG2E = 1.4426950408889634f;
+
+struct ChunkParams {
+  int H, dim, vdim;
+  int dimp, vpad, vrows;          // key columns padded to eight; value rows padded to 16, plus 16 for the normaliser
+  int pk, pv;                     // 64-column panels
+  int ldv, ld_in, ld_out, ld_gates;
+  float qscale, cap, eps;
+  const int4* chunks;             // {first token, tokens, sequence, cache row if it is the first of a continued sequence, -1 of a fresh one, -2}
+  const int4* seqs;               // {first chunk, chunks, cache row, first position}
+  const float* log2_decay;        // fixed decay: [H]
+  const float* gates;             // gated: raw projections [T, ld_gates], log input | log forget
+  const float* gate_bias;         // [2H]
+  float* u;                       // [chunks * H, vrows, dimp]
+  float2* stat;                   // [chunks * H] {m_loc, F_end}
+  __nv_bfloat16 *s_hi, *s_lo;     // [chunks * H, vrows, dimp]
+  float* m_before;                // [chunks * H]
+  float* m_init;                  // [sequences * H]
+  float* state;                   // cache [rows, H, dim, ldv]
+  float* stab;                    // cache [rows, H, dim + 1]
+  const __nv_bfloat16* gate_out;  // gated: output gate, head h at column h * vdim, pitch ld_in
+  const float* norm_w;
+  __nv_bfloat16* out;             // [T, ld_out]
+  int* err;
+};
+
+struct ChunkBars {
+  uint64_t qk_full, v_full, s_done, o_done;
+  uint32_t tmem_slot;
+  int abort_flag;
+  float red[16];
+};
+
+// log input and log forget gate of a token
+__device__ __forceinline__ void token_gates(const ChunkParams& p, int t, int h, float& li, float& lf) {
+  const float zi = p.gates[static_cast<size_t>(t) * p.ld_gates + h] + p.gate_bias[h];
+  const float zf = p.gates[static_cast<size_t>(t) * p.ld_gates + p.H + h] + p.gate_bias[p.H + h];
+  li = p.cap * tanhf(zi / p.cap);
+  const float z = p.cap * tanhf(zf / p.cap);
+  lf = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+}
+
+// inclusive prefix over the 128 threads (threads in token order)
+template <bool MAX>
+__device__ __forceinline__ float chunk_prefix(float v, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float w = __shfl_up_sync(0xffffffffu, v, o);
+    if (lane >= o) v = MAX ? fmaxf(v, w) : v + w;
+  }
+  __syncthreads();
+  if (lane == 31) red[warp] = v;
+  __syncthreads();
+  for (int w = 0; w < warp; ++w) v = MAX ? fmaxf(v, red[w]) : v + red[w];
+  return v;
+}
+
+__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - h.x, b - h.y);
+}
+
+// ------------------------------------------------------------------------------------------------ states of single chunks
+template <bool GATED>
+__global__ void __launch_bounds__(128)
+chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const ChunkParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  ChunkBars* bars = reinterpret_cast<ChunkBars*>(smem);
+  uint8_t* sKh = smem + 1024;                  // two panels: the product's 128 rows are key columns
+  uint8_t* sKl = sKh + 2 * MC_PANEL;
+  uint8_t* sV = sKl + 2 * MC_PANEL;
+  uint8_t* sOne = sV + p.pv * MC_PANEL;        // gated: a column of ones
+  volatile int* abort_flag = &bars->abort_flag;
+  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x, warp = j >> 5, lane = j & 31;
+  const int4 c = p.chunks[ch];
+  const int t0 = c.x, n = c.y;
+  if (j == 0) {
+    mbar_init(&bars->qk_full, 1);
+    mbar_init(&bars->v_full, 1);
+    mbar_init(&bars->o_done, 1);
+    bars->abort_flag = 0;
+    fence_barrier_init();
+    fence_proxy_async_smem();
+    mbar_expect_tx(&bars->qk_full, p.pk * MC_PANEL);
+    for (int i = 0; i < p.pk; ++i) tma_load_3d(sKh + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, h);
+    mbar_expect_tx(&bars->v_full, p.pv * MC_PANEL);
+    for (int i = 0; i < p.pv; ++i) tma_load_3d(sV + i * MC_PANEL, &tmV, &bars->v_full, i * 64, t0, h);
+  }
+  uint32_t cols = 32;
+  while (cols < static_cast<uint32_t>(p.vrows)) cols <<= 1;
+  if (warp == 1) {
+    tmem_alloc(&bars->tmem_slot, cols);
+    tmem_relinquish();
+  }
+  // weights
+  float w;
+  const size_t idx = static_cast<size_t>(ch) * p.H + h;
+  if constexpr (GATED) {
+    float li = -INFINITY, lf = 0.f;
+    if (j < n) token_gates(p, t0 + j, h, li, lf);
+    const float F = chunk_prefix<false>(lf, bars->red);
+    if (j == MC_C - 1) bars->red[8] = F;       // tokens past the end add nothing
+    __syncthreads();
+    const float Fend = bars->red[8], e = Fend - F + li;
+    const float m = chunk_prefix<true>(e, bars->red);
+    if (j == MC_C - 1) bars->red[9] = m;
+    __syncthreads();
+    const float mloc = bars->red[9];
+    w = j < n ? expf(e - mloc) : 0.f;
+    if (j == 0) {
+      p.stat[idx] = make_float2(mloc, Fend);
+      if (c.w > -2) p.m_init[static_cast<size_t>(c.z) * p.H + h] = c.w < 0 ? 0.f : p.stab[(static_cast<size_t>(c.w) * p.H + h) * (p.dim + 1) + p.dim];
+    }
+    for (int i = 0; i < 8; ++i) {              // the row's pieces, ones in the first column
+      const uint32_t one = i == 0 ? 0x3F80u : 0u;
+      *reinterpret_cast<uint4*>(sOne + j * 128 + ((i ^ (j & 7)) << 4)) = make_uint4(one, 0u, 0u, 0u);
+    }
+  } else {
+    w = j < n ? exp2f(p.log2_decay[h] * static_cast<float>(n - 1 - j)) : 0.f;
+    if (j == 0) p.stat[idx] = make_float2(0.f, p.log2_decay[h] * static_cast<float>(n));
+  }
+  __syncthreads();
+  const bool ok = mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
+  for (int i = 0; i < 16; ++i) {
+    const int off = (i >> 3) * MC_PANEL + j * 128 + (((i & 7) ^ (j & 7)) << 4);
+    uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+    if (w != 0.f && i < 8 * p.pk) {
+      const uint4 k = *reinterpret_cast<const uint4*>(sKh + off);
+      const float2 a = unpack_bf16x2(k.x), b = unpack_bf16x2(k.y), d = unpack_bf16x2(k.z), e = unpack_bf16x2(k.w);
+      split_pack(a.x * w, a.y * w, hi.x, lo.x);
+      split_pack(b.x * w, b.y * w, hi.y, lo.y);
+      split_pack(d.x * w, d.y * w, hi.z, lo.z);
+      split_pack(e.x * w, e.y * w, hi.w, lo.w);
+    }
+    *reinterpret_cast<uint4*>(sKh + off) = hi;
+    *reinterpret_cast<uint4*>(sKl + off) = lo;
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = bars->tmem_slot;
+  if (j == 0) {
+    const bool vok = mbar_wait(&bars->v_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
+    if (ok && vok) {
+      tc_fence_after();
+      const uint32_t idesc = make_idesc_bf16(128, p.vpad, 1, 1), idesc1 = make_idesc_bf16(128, 16, 1, 1);
+      const uint64_t dv = make_smem_desc(smem_u32(sV), MC_PANEL, 1024), d1 = make_smem_desc(smem_u32(sOne), MC_PANEL, 1024);
+      const int steps = (n + 15) >> 4;
+      for (int half = 0; half < 2; ++half) {
+        const uint64_t dk = make_smem_desc(smem_u32(half ? sKl : sKh), MC_PANEL, 1024);
+        for (int t = 0; t < steps; ++t) {
+          umma_bf16(tmem, dk + t * 128, dv + t * 128, idesc, (half || t) ? 1u : 0u);
+          if constexpr (GATED) umma_bf16(tmem + p.vpad, dk + t * 128, d1 + t * 128, idesc1, (half || t) ? 1u : 0u);
+        }
+      }
+      umma_commit(&bars->o_done);
+    } else {
+      bars->abort_flag = 1;
+    }
+  }
+  if (mbar_wait(&bars->o_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
+    tc_fence_after();
+    float* u = p.u + idx * p.vrows * p.dimp + j;
+    const uint32_t ta = tmem + (static_cast<uint32_t>(warp * 32) << 16);
+    for (int v0 = 0; v0 < p.vrows; v0 += 16) {
+      uint32_t r[16];
+      tmem_ld_32x16(ta + v0, r);
+      tmem_ld_wait();
+      if (j < p.dimp) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) u[static_cast<size_t>(v0 + i) * p.dimp] = __uint_as_float(r[i]);
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem, cols);
+  }
+  (void)lane;
+}
+
+// ------------------------------------------------------------------------------------------------ recurrence over chunks
+// A thread carries four key columns of one value row through the chunks of a sequence.
+template <bool GATED>
+__global__ void __launch_bounds__(256)
+chunk_scan_kernel(const ChunkParams p) {
+  const int h = blockIdx.y;
+  const int4 sq = p.seqs[blockIdx.z];
+  const int c0 = sq.x, nc = sq.y, row = sq.z;
+  const bool fresh = sq.w == 0;
+  const int per = p.dimp >> 2, e = blockIdx.x * 256 + threadIdx.x;
+  if (e >= per * p.vrows) return;
+  const int v = e / per, d = 4 * (e - v * per);
+  float* st = p.state + (static_cast<size_t>(row) * p.H + h) * p.dim * p.ldv;
+  float* sb = GATED ? p.stab + (static_cast<size_t>(row) * p.H + h) * (p.dim + 1) : nullptr;
+  const bool is_value = v < p.vdim, is_norm = GATED && v == p.vpad;
+  float s[4] = {0.f, 0.f, 0.f, 0.f};
+  if (!fresh) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (d + i < p.dim) {
+        if (is_value) s[i] = st[static_cast<size_t>(d + i) * p.ldv + v];
+        else if (is_norm) s[i] = sb[d + i];
+      }
+  }
+  float m = GATED ? p.m_init[static_cast<size_t>(blockIdx.z) * p.H + h] : 0.f;
+  const size_t pitch = static_cast<size_t>(p.vrows) * p.dimp, at = static_cast<size_t>(v) * p.dimp + d;
+  constexpr int U = 4;
+  for (int b = 0; b < nc; b += U) {
+    float4 u[U];
+    float2 f[U];
+#pragma unroll
+    for (int k = 0; k < U; ++k)
+      if (b + k < nc) {
+        const size_t idx = static_cast<size_t>(c0 + b + k) * p.H + h;
+        u[k] = *reinterpret_cast<const float4*>(p.u + idx * pitch + at);
+        f[k] = p.stat[idx];
+      }
+#pragma unroll
+    for (int k = 0; k < U; ++k)
+      if (b + k < nc) {
+        const size_t idx = static_cast<size_t>(c0 + b + k) * p.H + h;
+        uint2 hi, lo;
+        split_pack(s[0], s[1], hi.x, lo.x);
+        split_pack(s[2], s[3], hi.y, lo.y);
+        *reinterpret_cast<uint2*>(p.s_hi + idx * pitch + at) = hi;
+        *reinterpret_cast<uint2*>(p.s_lo + idx * pitch + at) = lo;
+        float a, w = 1.f;
+        if constexpr (GATED) {
+          if (e == 0) p.m_before[idx] = m;
+          const float mn = fmaxf(f[k].y + m, f[k].x);
+          a = expf(f[k].y + m - mn);
+          w = expf(f[k].x - mn);
+          m = mn;
+        } else {
+          a = exp2f(f[k].y);
+        }
+        s[0] = a * s[0] + w * u[k].x;
+        s[1] = a * s[1] + w * u[k].y;
+        s[2] = a * s[2] + w * u[k].z;
+        s[3] = a * s[3] + w * u[k].w;
+      }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (d + i < p.dim) {
+      if (is_value) st[static_cast<size_t>(d + i) * p.ldv + v] = s[i];
+      else if (is_norm) sb[d + i] = s[i];
+    }
+  if (GATED && e == 0) sb[p.dim] = m;
+}
+
+// ------------------------------------------------------------------------------------------------ outputs
+template <bool GATED>
+__global__ void __launch_bounds__(128)
+chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                 const __grid_constant__ CUtensorMap tmSh, const __grid_constant__ CUtensorMap tmSl, const ChunkParams p, int tmem_cols) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  ChunkBars* bars = reinterpret_cast<ChunkBars*>(smem);
+  float* gj = reinterpret_cast<float*>(smem + 512);      // [128] exponent of key j
+  const int spanel = p.vrows * 128;
+  uint8_t* sQ = smem + 1024;
+  uint8_t* sK = sQ + p.pk * MC_PANEL;
+  uint8_t* sV = sK + p.pk * MC_PANEL;
+  uint8_t* sSh = sV + p.pv * MC_PANEL;
+  uint8_t* sSl = sSh + p.pk * spanel;
+  volatile int* abort_flag = &bars->abort_flag;
+  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x, warp = j >> 5;
+  const int4 c = p.chunks[ch];
+  const int t0 = c.x, n = c.y;
+  const size_t idx = static_cast<size_t>(ch) * p.H + h;
+  if (j == 0) {
+    mbar_init(&bars->qk_full, 1);
+    mbar_init(&bars->v_full, 1);
+    mbar_init(&bars->s_done, 1);
+    mbar_init(&bars->o_done, 1);
+    bars->abort_flag = 0;
+    fence_barrier_init();
+    fence_proxy_async_smem();
+    mbar_expect_tx(&bars->qk_full, p.pk * 2 * MC_PANEL);
+    for (int i = 0; i < p.pk; ++i) {
+      tma_load_3d(sQ + i * MC_PANEL, &tmQ, &bars->qk_full, i * 64, t0, h);
+      tma_load_3d(sK + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, h);
+    }
+    mbar_expect_tx(&bars->v_full, p.pv * MC_PANEL + 2 * p.pk * spanel);
+    for (int i = 0; i < p.pk; ++i) {
+      tma_load_3d(sSh + i * spanel, &tmSh, &bars->v_full, i * 64, 0, static_cast<int>(idx));
+      tma_load_3d(sSl + i * spanel, &tmSl, &bars->v_full, i * 64, 0, static_cast<int>(idx));
+    }
+    for (int i = 0; i < p.pv; ++i) tma_load_3d(sV + i * MC_PANEL, &tmV, &bars->v_full, i * 64, t0, h);
+  }
+  if (warp == 1) {
+    tmem_alloc(&bars->tmem_slot, tmem_cols);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = bars->tmem_slot;
+  if (j == 0) {
+    const int ks = (p.dim + 15) >> 4;
+    const uint64_t dq = make_smem_desc(smem_u32(sQ), 16, 1024), dk = make_smem_desc(smem_u32(sK), 16, 1024);
+    if (mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
+      tc_fence_after();
+      const uint32_t idesc = make_idesc_bf16(128, MC_C, 0, 0);
+      for (int t = 0; t < ks; ++t) {
+        const int o = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3);
+        umma_bf16(tmem, dq + o, dk + o, idesc, t ? 1u : 0u);
+      }
+      umma_commit(&bars->s_done);
+    } else {
+      bars->abort_flag = 1;
+    }
+    if (mbar_wait(&bars->v_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
+      tc_fence_after();
+      const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 0), idesc1 = make_idesc_bf16(128, 16, 0, 0);
+      for (int half = 0; half < 2; ++half) {
+        const uint64_t ds = make_smem_desc(smem_u32(half ? sSl : sSh), 16, 1024);
+        for (int t = 0; t < ks; ++t) {
+          const int oq = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3), os = (t >> 2) * (spanel >> 4) + 2 * (t & 3);
+          umma_bf16(tmem + MC_C, dq + oq, ds + os, idesc, (half || t) ? 1u : 0u);
+          if constexpr (GATED) umma_bf16(tmem + MC_C + p.vpad, dq + oq, ds + os + p.vpad * 8, idesc1, (half || t) ? 1u : 0u);
+        }
+      }
+      umma_commit(&bars->o_done);
+    } else {
+      bars->abort_flag = 1;
+    }
+  }
+  __syncwarp();
+  // exponents of this thread's row (and, as a key, of its column)
+  float arow, einter, mrow = 0.f;
+  if constexpr (GATED) {
+    float li = -INFINITY, lf = 0.f;
+    if (j < n) token_gates(p, t0 + j, h, li, lf);
+    const float F = chunk_prefix<false>(lf, bars->red);
+    const float pm = chunk_prefix<true>(li - F, bars->red);
+    const float mb = p.m_before[idx];
+    mrow = F + fmaxf(mb, pm);
+    arow = (F - mrow) * LOG2E;
+    einter = expf(F + mb - mrow);
+    gj[j] = (li - F) * LOG2E;
+  } else {
+    const float ld = p.log2_decay[h];
+    arow = ld * static_cast<float>(j);
+    gj[j] = -arow;
+    einter = exp2f(ld * static_cast<float>(j + 1));
+  }
+  einter *= p.qscale;
+  __syncthreads();
+  const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+  const uint32_t ts = tmem + lane_addr, to = ts + MC_C;
+  float nq = 0.f;
+  const bool ok = mbar_wait(&bars->s_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+  if (ok) {
+    tc_fence_after();
+#pragma unroll 1
+    for (int c0 = 0; c0 < MC_C; c0 += 32) {
+      uint32_t v[32];
+      tmem_ld_32x32(ts + c0, v);
+      tmem_ld_wait();
+      uint32_t packed[16];
+#pragma unroll
+      for (int i = 0; i < 32; i += 4) {
+        const float4 g = *reinterpret_cast<const float4*>(gj + c0 + i);
+        float w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          // the difference of the exponents first: it is small where the weight matters
+          w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * p.qscale * ex2_approx(arow + w[k]) : 0.f;
+          nq += w[k];
+        }
+        packed[i >> 1] = pack_bf16x2(w[0], w[1]);
+        packed[(i >> 1) + 1] = pack_bf16x2(w[2], w[3]);
+      }
+      tmem_st_32x16(ts + (c0 >> 1), packed);        // over columns that have been read
+    }
+    tmem_st_wait();
+  }
+  const bool ok2 = mbar_wait(&bars->o_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+  if (ok && ok2) {
+    tc_fence_after();
+#pragma unroll 1
+    for (int c0 = 0; c0 < p.vpad; c0 += 16) {
+      uint32_t v[16];
+      tmem_ld_32x16(to + c0, v);
+      tmem_ld_wait();
+#pragma unroll
+      for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * einter);
+      tmem_st_32x16(to + c0, v);
+    }
+    if constexpr (GATED) {
+      uint32_t v[16];
+      tmem_ld_32x16(to + p.vpad, v);
+      tmem_ld_wait();
+      nq += __uint_as_float(v[0]) * einter;
+    }
+    tmem_st_wait();
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (j == 0 && !*abort_flag) {
+    tc_fence_after();
+    const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 1);
+    const uint64_t dv = make_smem_desc(smem_u32(sV), MC_PANEL, 1024);
+    const int steps = (n + 15) >> 4;
+    for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_C, tmem + t * 8, dv + t * 128, idesc, 1u);
+    umma_commit(&bars->qk_full);                    // its second phase
+  }
+  if (mbar_wait(&bars->qk_full, 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
+    tc_fence_after();
+    const bool live = j < n;
+    const size_t t = static_cast<size_t>(t0) + (live ? j : 0);
+    __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
+    float f = 1.f;
+    if constexpr (GATED) {
+      f = 1.f / (fmaxf(fabsf(nq), expf(-mrow)) + 1e-6f);
+      float ss = 0.f;
+#pragma unroll 1
+      for (int c0 = 0; c0 < p.vpad; c0 += 16) {     // padding columns are zero
+        uint32_t v[16];
+        tmem_ld_32x16(to + c0, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float o = __uint_as_float(v[i]) * f;
+          ss += o * o;
+        }
+      }
+      f /= sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
+    }
+    const __nv_bfloat16* grow = GATED ? p.gate_out + t * p.ld_in + h * p.vdim : nullptr;
+    const float* nw = GATED ? p.norm_w + h * p.vdim : nullptr;
+#pragma unroll 1
+    for (int c0 = 0; c0 < p.vpad; c0 += 16) {
+      uint32_t v[16];
+      tmem_ld_32x16(to + c0, v);
+      tmem_ld_wait();
+      if (!live) continue;
+#pragma unroll
+      for (int q = 0; q < 16; q += 8) {
+        if (c0 + q >= p.vdim) continue;
+        float o[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[q + i]) * f;
+        if constexpr (GATED) {
+          float g[8];
+          ld8(grow + c0 + q, g);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) o[i] *= nw[c0 + q + i] * sigmoid_f(g[i]);
+        }
+        st8(orow + c0 + q, o);
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem, tmem_cols);
+  }
+}
+
+typedef CUresult (*EncodeTiledFnM)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// bf16 [planes, rows, cols] with the given pitches (elements); box: `box_rows` rows x 64 columns of one plane, 128-byte swizzle
+static int make_tmap_planes(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint64_t planes, uint64_t ld, uint64_t plane,
+                            uint32_t box_rows) {
+  static EncodeTiledFnM enc = nullptr;
+  if (!enc) {
+    void* ptr = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess)
+      return -1;
+    enc = reinterpret_cast<EncodeTiledFnM>(ptr);
+  }
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (ld & 7) || (plane & 7)) return -2;
+  cuuint64_t dims[3] = {cols, rows, planes};
+  cuuint64_t strides[2] = {ld * 2, plane * 2};
+  cuuint32_t box[3] = {64, box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? 0 : -3;
+}
+
+static int mc_smem_state(int pv, bool gated) { return 1024 + 1024 + (4 + pv + (gated ? 1 : 0)) * MC_PANEL; }
+static int mc_smem_out(int pk, int pv, int vrows) { return 1024 + 1024 + (2 * pk + pv) * MC_PANEL + 2 * pk * vrows * 128; }
+
+}  // namespace b200
+
+using namespace b200;
+
+static int mc_vrows(int vdim, bool gated) { return ((vdim + 15) & ~15) + (gated ? 16 : 0); }
+
+B200_API int b200_memory_chunk_supported(int dim, int vdim, int gated) {
+  if (dim <= 0 || vdim <= 0 || (dim & 7) || (vdim & 7) || dim > 128 || mc_vrows(vdim, gated) > 256) return 0;
+  const int pk = (dim + 63) / 64, pv = (vdim + 63) / 64, limit = 227 * 1024;
+  return mc_smem_state(pv, gated) <= limit && mc_smem_out(pk, pv, mc_vrows(vdim, gated)) <= limit;
+}
+
+// q, k, v: columns of the packed step's projection rows [T, ld_in] (head h at column h dim / h vdim).  parts: 1 chunk states,
+// 2 recurrence, 4 outputs (all of them in this order for a step).
+B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, const ChunkParams* Pp, int T, int n_chunks, int n_seqs, int parts,
+                                void* stream, int* err) {
+  ChunkParams p = *Pp;
+  const bool gated = p.gates != nullptr;
+  if (!b200_memory_chunk_supported(p.dim, p.vdim, gated) || T <= 0 || n_chunks <= 0 || n_chunks > 65535 || n_seqs <= 0 || n_seqs > 65535 ||
+      p.H <= 0 || p.H > 65535 || (p.ld_in & 7) || (p.ld_out & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return -1;
+  if (gated ? (!p.stab || !p.norm_w || !p.gate_bias || (reinterpret_cast<uintptr_t>(p.gate_out) & 15)) : !p.log2_decay) return -1;
+  p.dimp = (p.dim + 7) & ~7;
+  p.vpad = (p.vdim + 15) & ~15;
+  p.vrows = mc_vrows(p.vdim, gated);
+  p.pk = (p.dim + 63) / 64;
+  p.pv = (p.vdim + 63) / 64;
+  p.err = err;
+  CUtensorMap tq, tk, tv, th, tl;
+  int rc = make_tmap_planes(&tq, q, p.dim, T, p.H, p.ld_in, p.dim, MC_C);
+  if (!rc) rc = make_tmap_planes(&tk, k, p.dim, T, p.H, p.ld_in, p.dim, MC_C);
+  if (!rc) rc = make_tmap_planes(&tv, v, p.vdim, T, p.H, p.ld_in, p.vdim, MC_C);
+  const uint64_t planes = static_cast<uint64_t>(n_chunks) * p.H;
+  if (!rc) rc = make_tmap_planes(&th, p.s_hi, p.dim, p.vrows, planes, p.dimp, static_cast<uint64_t>(p.vrows) * p.dimp, p.vrows);
+  if (!rc) rc = make_tmap_planes(&tl, p.s_lo, p.dim, p.vrows, planes, p.dimp, static_cast<uint64_t>(p.vrows) * p.dimp, p.vrows);
+  if (rc) return rc;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const int sm1 = mc_smem_state(p.pv, gated), sm3 = mc_smem_out(p.pk, p.pv, p.vrows);
+  int cols = 256;
+  while (cols < MC_C + p.vrows) cols <<= 1;
+#define GO(G)                                                                                                          \
+  {                                                                                                                    \
+    if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
+        cudaFuncSetAttribute(chunk_out_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
+    if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 128, sm1, st>>>(tk, tv, p);                              \
+    if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 255) / 256, p.H, n_seqs), 256, 0, st>>>(p);      \
+    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 128, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
+  }
+  if (gated) GO(true) else GO(false)
+#undef GO
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}

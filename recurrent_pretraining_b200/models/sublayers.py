@@ -5,6 +5,7 @@ Weights are stored as they are executed: projections that read the same input ar
 eight elements.  ``checkpoint_tensors`` names the views that make up a checkpoint."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Callable, Optional
 
@@ -68,6 +69,7 @@ class PackedStep:
         self.T = len(tok)
         self._layouts: dict = {}
         self._seq_table = None
+        self.derived: dict = {}           # tables that kernels derive from the portions
 
     def sequences(self) -> list:
         """(first token, tokens, cache row, first position) per portion."""
@@ -261,6 +263,8 @@ class ParallelMixer(nn.Module):
         self.rel = nn.Parameter(torch.zeros(a.bias_rows, a.heads, dtype=torch.float32, device=device), requires_grad=False)
         self.norm = vector(r.heads * r.vdim, device)
         self.register_buffer("decay", torch.tensor(r.decay, dtype=torch.float32).to(device), persistent=False)
+        logs = [math.log2(x) if x > 0 else -1000.0 for x in r.decay]        # finite: 2^-1000 is zero in fp32
+        self.register_buffer("log2_decay", torch.tensor(logs, dtype=torch.float32).to(device), persistent=False)
         self.table = None
 
     def checkpoint_tensors(self) -> dict:
@@ -291,7 +295,7 @@ class ParallelMixer(nn.Module):
         mem_ops.kv_append(L, inp, None, kv, step.pos, step.row)
         o = mem_ops.parallel_output(L, h.shape[0], self.dtype, h.device)
         mem_ops.prompt_attention(L, spec.left, inp, kv, self.table, step, spec.left_scale, o)
-        m = mem_ops.decay_memory_prompt(L, inp, self.decay, state, step)
+        m = mem_ops.decay_memory_prompt(L, inp, self.decay, self.log2_decay, state, step)
         mem_ops.memory_norm(L, inp, m, self.norm, self.eps, spec.right_scale, o)
         return ops.linear(o, self.w_o[:, :L.width_o])
 

@@ -187,6 +187,15 @@ class BiasTable:
 
     values: torch.Tensor
     ids: torch.Tensor
+    _padded: Optional[torch.Tensor] = None
+
+    def padded(self) -> torch.Tensor:
+        """The form of the tensor-core kernels (log2 units, repeated at both ends)."""
+        if self._padded is None:
+            from .memory_kernels import padded_bias
+
+            self._padded = padded_bias(self.values)
+        return self._padded
 
     @classmethod
     def build(cls, rel: torch.Tensor, buckets: list) -> "BiasTable":
@@ -258,7 +267,8 @@ def _rms_gate(o: torch.Tensor, eps: float, w, gate) -> torch.Tensor:
     return ref.rms(o, eps) * w * torch.sigmoid(gate.float())
 
 
-def decay_memory_prompt(L: ParallelLayout, inp: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, step) -> torch.Tensor:
+def decay_memory_prompt(L: ParallelLayout, inp: torch.Tensor, decay: torch.Tensor, log2_decay: torch.Tensor, state: torch.Tensor,
+                        step) -> torch.Tensor:
     """Memory outputs [T, r_heads * r_vdim] of a packed step (activated projections); the sequences' states are carried on."""
     T, H = inp.shape[0], L.r_heads
     if not inp.is_cuda:
@@ -273,8 +283,8 @@ def decay_memory_prompt(L: ParallelLayout, inp: torch.Tensor, decay: torch.Tenso
     if inp.dtype == BF16:
         from . import memory_kernels as MK
 
-        if MK.chunk_supported(L.r_dim, L.r_vdim):
-            return MK.decay_memory(L, inp, decay, state, step)
+        if MK.chunk_supported(L.r_dim, L.r_vdim, False):
+            return MK.decay_memory(L, inp, log2_decay, state, step)()
     return _decay_scan(L, inp, decay, state, step.seq_table, None, None, len(step.portions), 0)
 
 
@@ -335,7 +345,7 @@ def parallel_decode(L: ParallelLayout, spec, inp: torch.Tensor, bias: torch.Tens
             o = _plain_attention(L, a, x[b:b + 1, :L.heads * L.dim], cache[r], table, p)
             g = torch.sigmoid(x[b:b + 1, L.off_lg:L.off_lg + L.heads]) * spec.left_scale
             out[b, :L.heads * L.vdim] = (o * g[:, :, None]).flatten().to(dtype)
-        mem = decay_memory_prompt(L, x, decay, state, _Rows(pos, row))
+        mem = decay_memory_prompt(L, x, decay, None, state, _Rows(pos, row))
         memory_norm(L, x, mem, norm_w, eps, spec.right_scale, out)
         return out
     po = torch.empty(B, L.heads, splits, pad8(L.vdim), dtype=F32, device=inp.device)
@@ -409,8 +419,8 @@ def gated_memory(L: MemoryLayout, inp: torch.Tensor, gates, gate_bias: torch.Ten
     if step is not None and inp.dtype == BF16:
         from . import memory_kernels as MK
 
-        if MK.chunk_supported(L.dim, L.vdim):
-            return MK.gated_memory(L, inp, gates, gate_bias, cap, state, stab, norm_w, eps, step)
+        if MK.chunk_supported(L.dim, L.vdim, True):
+            return MK.gated_memory(L, inp, gates, gate_bias, cap, state, stab, norm_w, eps, step)()
     k = _k()
     p = k.K._ptr
     out = torch.empty(T, pad8(hv), dtype=dtype, device=inp.device)[:, :hv]
