@@ -91,15 +91,22 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   }
   __syncthreads();
   __nv_bfloat16* base = P.cache + static_cast<size_t>(P.row[b]) * P.cap * P.ld_kv;
-  const int kch = P.dim >> 3, vch = P.vdim >> 3, ch = kch + vch;       // 16-byte pieces of a key and of a value
+  // 16-byte pieces of a key row and a value row: a power of two of lanes per key, or several passes of 32
+  const int kch = P.dim >> 3, ch = kch + (P.vdim >> 3);
+  int lpk = 1;
+  while (lpk < ch && lpk < 32) lpk <<= 1;
+  const int kpp = 32 / lpk, lj = lane / lpk, lc = lane % lpk;          // keys per pass, this lane's key and first piece
   auto request = [&](int tile, int st) {
     const uint32_t s = smem_u32(ring + st * stage_bytes);
-    for (int i = lane; i < GD_KEYS * ch; i += 32) {
-      const int j = i / ch, c = i - j * ch;
-      const int key = min(tile * GD_KEYS + j, max(pos - 1, 0));        // keys past the newest repeat one that exists; they are masked
+    const int last = max(pos - 1, 0);                                  // keys past the newest repeat one that exists; they are masked
+    for (int c = lc; c < ch; c += lpk) {
       const bool isk = c < kch;
-      const __nv_bfloat16* src = base + static_cast<size_t>(key) * P.ld_kv + (isk ? g * P.dim + 8 * c : P.kv_v + g * P.vdim + 8 * (c - kch));
-      cp_async16(s + (isk ? j * kp + 16 * c : GD_KEYS * kp + j * vp + 16 * (c - kch)), src);
+      const __nv_bfloat16* src = base + (isk ? g * P.dim + 8 * c : P.kv_v + g * P.vdim + 8 * (c - kch));
+      const uint32_t dst = s + (isk ? 16 * c : GD_KEYS * kp + 16 * (c - kch));
+      const int pitch = isk ? kp : vp;
+#pragma unroll 8
+      for (int j = lj; j < GD_KEYS; j += kpp)
+        cp_async16(dst + j * pitch, src + static_cast<size_t>(min(tile * GD_KEYS + j, last)) * P.ld_kv);
     }
   };
   const int first = tile0 + warp;
@@ -116,6 +123,8 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const float* bias_row[2];
 #pragma unroll
   for (int k = 0; k < 2; ++k) bias_row[k] = P.bias + static_cast<size_t>(min(h0 + ra + 8 * k, P.H - 1)) * P.ld_bias + P.bias_lead;
+  const int far = P.bias_len - 1;
+  const float bias_far[2] = {bias_row[0][far], bias_row[1][far]};
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[NV][2][4];
 #pragma unroll
@@ -164,23 +173,34 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     // c[n][0..1]: head ra, keys key0 + 8 n + 2 (lane & 3) + {0, 1}; c[n][2..3]: head ra + 8
     float p[2][4];
     float mx[2] = {-INFINITY, -INFINITY};
-    const int d0 = pos - key0 - 2 * (lane & 3), far = P.bias_len - 1;
+    if (pos - key0 - (GD_KEYS - 1) >= far) {                           // every distance shares the last bucket
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = d0 - 8 * n - (e & 1);
-        const float v = d >= 0 ? fmaf(c[n][e], rowmul, bias_row[e >> 1][min(max(d, 0), far)]) : -INFINITY;
-        p[n][e] = v;
-        mx[e >> 1] = fmaxf(mx[e >> 1], v);
-      }
+        for (int e = 0; e < 4; ++e) {
+          p[n][e] = fmaf(c[n][e], rowmul, bias_far[e >> 1]);
+          mx[e >> 1] = fmaxf(mx[e >> 1], p[n][e]);
+        }
+    } else {
+      const int d0 = pos - key0 - 2 * (lane & 3);
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = d0 - 8 * n - (e & 1);
+          p[n][e] = d >= 0 ? fmaf(c[n][e], rowmul, bias_row[e >> 1][min(max(d, 0), far)]) : -INFINITY;
+          mx[e >> 1] = fmaxf(mx[e >> 1], p[n][e]);
+        }
+    }
     float alpha[2];
+    bool moved = false;
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 1));
       mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 2));
       const float mn = fmaxf(m[k], mx[k]);                             // finite: the tile's first key is visible
       alpha[k] = exp2f(m[k] - mn);
+      moved |= mn != m[k];
       m[k] = mn;
       l[k] *= alpha[k];
     }
@@ -191,6 +211,15 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
         p[n][e] = exp2f(p[n][e] - m[e >> 1]);
         l[e >> 1] += p[n][e];
       }
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+      for (int n = 0; n < NV; ++n)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          o[n][k][0] *= alpha[0]; o[n][k][1] *= alpha[0];
+          o[n][k][2] *= alpha[1]; o[n][k][3] *= alpha[1];
+        }
+    }
     const uint32_t pa[4] = {pack_bf16x2(p[0][0], p[0][1]), pack_bf16x2(p[0][2], p[0][3]), pack_bf16x2(p[1][0], p[1][1]), pack_bf16x2(p[1][2], p[1][3])};
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
@@ -198,11 +227,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
         uint32_t v4[4];
         ldsm4t(v4, s + bv + 32 * n);
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-          o[n][k][0] *= alpha[0]; o[n][k][1] *= alpha[0];
-          o[n][k][2] *= alpha[1]; o[n][k][3] *= alpha[1];
-          mma_bf16(o[n][k], pa, v4[2 * k], v4[2 * k + 1]);
-        }
+        for (int k = 0; k < 2; ++k) mma_bf16(o[n][k], pa, v4[2 * k], v4[2 * k + 1]);
       }
     }
     __syncwarp();                                                      // the stage may be requested again
@@ -271,6 +296,12 @@ using namespace b200;
 
 B200_API int b200_gqa_decode_supported(int dim, int vdim) {
   return dim > 0 && vdim > 0 && !(dim & 7) && !(vdim & 7) && dim <= 256 && vdim <= 256;
+}
+
+// CTAs of the kernel that fit an SM
+B200_API int b200_gqa_decode_per_sm(int dim, int vdim) {
+  const int n = 227 * 1024 / (gd_smem<3>(dim, vdim) + 1024);
+  return n < 1 ? 1 : n > 4 ? 4 : n;
 }
 
 B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {

@@ -31,6 +31,12 @@ template <typename TI, typename T, int NV>
 __global__ void __launch_bounds__(256)
 sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   pdl_trigger();
+  if (gridDim.x <= 256) {                          // few rows: the weights' way from memory would add to the reductions'
+    for (int i = 32 * threadIdx.x; i < A.E; i += 8192) {
+      if (a) { prefetch_l2(A.w1 + i); prefetch_l2(A.b1 + i); }
+      if (A.w2) { prefetch_l2(A.w2 + i); prefetch_l2(A.b2 + i); }
+    }
+  }
   pdl_wait();
   __shared__ float red[8];
   const size_t row = blockIdx.x;
@@ -209,32 +215,30 @@ geglu_kernel(TI* __restrict__ a, int ld_a, int clear, T* __restrict__ y, int ld_
 // ------------------------------------------------------------------------------------------------ keys and values
 // cache[row[t], pos[t], 0 .. width) = in[t, 0 .. width) (+ bias): the projections of k and v lie side by side in both.
 template <typename TI, typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 kv_append_kernel(const TI* __restrict__ in, int ld_in, const float* __restrict__ bias, T* __restrict__ cache, int width, int ld_kv,
-                 int cap, const int* __restrict__ pos, const int* __restrict__ row) {
+                 int cap, const int* __restrict__ pos, const int* __restrict__ row, int total) {
   pdl_trigger();
   pdl_wait();
-  const size_t t = blockIdx.x;
-  T* dst = cache + (static_cast<size_t>(row[t]) * cap + pos[t]) * ld_kv;
-  const TI* src = in + t * ld_in;
-  for (int i = 8 * threadIdx.x; i < width; i += 1024) {      // rows and widths are multiples of eight
-    float v[8];
-    ld8(src + i, v);
-    if (bias) {
-      float b[8];
-      ld8(bias + i, b);
+  const int i = blockIdx.x * 256 + threadIdx.x;              // eight elements each; rows and widths are multiples of eight
+  if (i >= total) return;
+  const int per = width >> 3, t = i / per, c = 8 * (i - t * per);
+  float v[8];
+  ld8(in + static_cast<size_t>(t) * ld_in + c, v);
+  if (bias) {
+    float b[8];
+    ld8(bias + c, b);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] += b[j];
-    }
-    st8(dst + i, v);
+    for (int j = 0; j < 8; ++j) v[j] += b[j];
   }
+  st8(cache + (static_cast<size_t>(row[t]) * cap + pos[t]) * ld_kv + c, v);
 }
 
 // ------------------------------------------------------------------------------------------------ matrix memories
 struct MemoryArgs {
   int H, dim, vdim, ldv;          // ldv: row pitch of the state [rows, H, dim, ldv]
   int ld_in, off_q, off_k, off_v, off_g;
-  int ld_out, E, ld_h, ld_w, ld_gates;
+  int ld_out, E, ld_h, ld_w, gate_t, gate_h;   // gate_t, gate_h: strides of `gates` per token and per gate
   int silu;                       // q, k and v are raw projections: apply silu
   int stage;                      // keep the state in shared memory between tokens
   float qscale, cap, eps;
@@ -242,7 +246,7 @@ struct MemoryArgs {
   const int* pos;
   const int* row;
   const float* decay;             // fixed decay per head; null: gated
-  const float* gates;             // [T, 2H] raw log input | log forget gate projections; null: formed here from h and w_gate
+  const float* gates;             // [T, 2H] (strided) raw log input | log forget gate projections; null: formed here from h and w_gate
   const float* gate_bias;         // [2H]
   float* state;
   float* stab;                    // [rows, H, dim + 1]: normaliser, running maximum
@@ -276,6 +280,8 @@ memory_scan_kernel(const TI* __restrict__ in, const T* __restrict__ hin, const T
   float* ns = red + 16;                            // [dim]
   float* ss = ns + ((dim + 3) & ~3);               // [dim][ldv] with `stage`
   float* gstate = M.state + (static_cast<size_t>(row) * M.H + h) * dim * ldv;
+  if (!M.seqs && start > 0)                        // the state is on its way while the token's vectors and gates are formed
+    for (int i = 32 * tid; i < dim * ldv; i += 8192) prefetch_l2(gstate + i);
   float* gstab = GATED ? M.stab + (static_cast<size_t>(row) * M.H + h) * (dim + 1) : nullptr;
   // lanes over columns: cl lanes of four columns, 32 / cl rows per warp
   int cl = 1;
@@ -312,8 +318,8 @@ memory_scan_kernel(const TI* __restrict__ in, const T* __restrict__ hin, const T
     if constexpr (GATED) {
       float zi, zf;
       if (M.gates) {
-        zi = M.gates[t * M.ld_gates + h];
-        zf = M.gates[t * M.ld_gates + M.H + h];
+        zi = M.gates[t * M.gate_t + static_cast<size_t>(h) * M.gate_h];
+        zf = M.gates[t * M.gate_t + static_cast<size_t>(M.H + h) * M.gate_h];
       } else {
         const T* x = hin + t * M.ld_h;
         const T* wi = w_gate + static_cast<size_t>(h) * M.ld_w;
@@ -497,14 +503,64 @@ memory_merge_kernel(const TI* __restrict__ in, const TM* __restrict__ mem, T* __
   const float mine = a / warp_sum(a * e.y) * sigmoid_f(ldf(r + A.off_lg + h)) * A.left_scale;
   const int vs = (A.vdim + 7) & ~7;
   const float* p = A.part_o + base * vs;
-  for (int c = lane; c - lane < A.vdim; c += 32) {   // uniform over the warp
-    float o = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < A.splits; ++s) {
-      const float w = __shfl_sync(0xffffffffu, mine, s);
-      if (c < A.vdim && w != 0.f) o += w * p[static_cast<size_t>(s) * vs + c];   // an empty split's partial is not initialised
+  for (int c = 4 * lane; c - 4 * lane < A.vdim; c += 128) {   // uniform over the warp
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+    constexpr int U = 8;                             // split rows in flight
+    for (int s0 = 0; s0 < A.splits; s0 += U) {
+      float x[U][4];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (s0 + u < A.splits && c < vs) ld4(p + static_cast<size_t>(s0 + u) * vs + c, x[u]);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const float w = __shfl_sync(0xffffffffu, mine, (s0 + u) & 31);
+        if (s0 + u < A.splits && c < vs && w != 0.f) {   // an empty split's partial is not initialised
+#pragma unroll
+          for (int k = 0; k < 4; ++k) o[k] += w * x[u][k];
+        }
+      }
     }
-    if (c < A.vdim) stf(out + t * A.ld_out + h * A.vdim + c, o);
+    T* dst = out + t * A.ld_out + h * A.vdim + c;
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (c + k < A.vdim) stf(dst + k, o[k]);
+  }
+}
+
+// The memory half alone, for prompts: a warp per token.  W = HR * rvdim, a multiple of four up to 128 * G.
+template <typename TI, typename TM, typename T, int G>
+__global__ void __launch_bounds__(256)
+memory_norm_rows_kernel(const TI* __restrict__ in, const TM* __restrict__ mem, T* __restrict__ out, const MergeArgs A, int rows) {
+  const size_t t = static_cast<size_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (t >= rows) return;
+  const int lane = threadIdx.x & 31, W = A.HR * A.rvdim;
+  const TM* m = mem + t * A.ld_mem;
+  const TI* g = in + t * A.ld_in + A.off_rg;
+  T* o = out + t * A.ld_out + A.off_r;
+  float v[G][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < G; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    if (i < W) {
+      ld4(m + i, v[k]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss += v[k][j] * v[k][j];
+    }
+  }
+  const float rms = A.right_scale / sqrtf(warp_sum(ss) / static_cast<float>(W) + A.eps);
+#pragma unroll
+  for (int k = 0; k < G; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    if (i < W) {
+      float gv[4], wv[4];
+      ld4(g + i, gv);
+      ld4(A.norm_w + i, wv);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[k][j] *= rms * wv[j] * __fdividef(1.f, 1.f + __expf(-gv[j]));
+      st2(o + i, make_float2(v[k][0], v[k][1]));
+      st2(o + i + 2, make_float2(v[k][2], v[k][3]));
+    }
   }
 }
 
@@ -567,7 +623,9 @@ B200_API int b200_kv_append(const void* in, int ld_in, const float* bias, void* 
                             const int* row, int T, int in_f32, int f32, void* stream) {
   if (T <= 0 || width <= 0 || (width & 7) || (ld_in & 7) || (ld_kv & 7) || width > ld_kv || cap <= 0 || (f32 && !in_f32)) return -1;
   if ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(bias)) & 15) return -1;
-#define GO(TI, T_) launch_k(kv_append_kernel<TI, T_>, dim3(T), dim3(128), 0, STREAM, (const TI*)in, ld_in, bias, (T_*)cache, width, ld_kv, cap, pos, row)
+  const long long total = static_cast<long long>(T) * (width / 8);
+  if (total > 0x7fffffffll - 256) return -1;
+#define GO(TI, T_) launch_k(kv_append_kernel<TI, T_>, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, STREAM, (const TI*)in, ld_in, bias, (T_*)cache, width, ld_kv, cap, pos, row, static_cast<int>(total))
   if (f32) GO(float, float);
   else if (in_f32) GO(float, bf16_t);
   else GO(bf16_t, bf16_t);
@@ -613,6 +671,16 @@ B200_API int b200_memory_merge(const void* in, const void* mem, void* out, const
   const MergeArgs A = *Ap;
   if (T <= 0 || A.HR <= 0 || A.rvdim <= 0 || (A.H && (!A.part_o || !A.part_ml || A.splits < 1 || A.splits > 32)) || (f32 && (!in_f32 || !mem_f32))) return -1;
   if (((A.ld_mem | A.ld_in | A.ld_out | A.off_r | A.off_rg) & 7) || ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(mem) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
+  const int W = A.HR * A.rvdim;
+  if (!f32 && !in_f32 && !mem_f32 && A.H == 0 && T >= 256 && (W & 3) == 0 && W <= 32 * 128) {
+#define GO(G) memory_norm_rows_kernel<bf16_t, bf16_t, bf16_t, G><<<(T + 7) / 8, 256, 0, STREAM>>>((const bf16_t*)in, (const bf16_t*)mem, (bf16_t*)out, A, T)
+    if (W <= 8 * 128) GO(8);
+    else if (W <= 16 * 128) GO(16);
+    else if (W <= 24 * 128) GO(24);
+    else GO(32);
+#undef GO
+    return DONE;
+  }
   const dim3 grid(T, 1 + (A.H + 7) / 8);
 #define GO(TI, TM, T_) launch_k(memory_merge_kernel<TI, TM, T_>, grid, dim3(256), 0, STREAM, (const TI*)in, (const TM*)mem, (T_*)out, A)
   if (f32) GO(float, float, float);

@@ -19,18 +19,19 @@ namespace b200 {
 
 constexpr int MC_C = 128;                     // tokens per chunk
 constexpr int MC_PANEL = MC_C * 128;          // 128 rows x 64 bf16
+constexpr int MC_O = MC_C + MC_C / 2;         // tensor-memory columns: scores, bf16 weights, outputs
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct ChunkParams {
   int H, dim, vdim;
   int dimp, vpad, vrows;          // key columns padded to eight; value rows padded to 16, plus 16 for the normaliser
   int pk, pv;                     // 64-column panels
-  int ldv, ld_in, ld_out, ld_gates;
+  int ldv, ld_in, ld_out, gate_t, gate_h;   // gate_t, gate_h: strides of `gates` per token and per gate
   float qscale, cap, eps;
   const int4* chunks;             // {first token, tokens, sequence, cache row if it is the first of a continued sequence, -1 of a fresh one, -2}
   const int4* seqs;               // {first chunk, chunks, cache row, first position}
   const float* log2_decay;        // fixed decay: [H]
-  const float* gates;             // gated: raw projections [T, ld_gates], log input | log forget
+  const float* gates;             // gated: raw projections [T, 2H] (strided), log input | log forget
   const float* gate_bias;         // [2H]
   float* u;                       // [chunks * H, vrows, dimp]
   float2* stat;                   // [chunks * H] {m_loc, F_end}
@@ -54,17 +55,18 @@ struct ChunkBars {
 
 // log input and log forget gate of a token
 __device__ __forceinline__ void token_gates(const ChunkParams& p, int t, int h, float& li, float& lf) {
-  const float zi = p.gates[static_cast<size_t>(t) * p.ld_gates + h] + p.gate_bias[h];
-  const float zf = p.gates[static_cast<size_t>(t) * p.ld_gates + p.H + h] + p.gate_bias[p.H + h];
+  const float zi = p.gates[static_cast<size_t>(t) * p.gate_t + static_cast<size_t>(h) * p.gate_h] + p.gate_bias[h];
+  const float zf = p.gates[static_cast<size_t>(t) * p.gate_t + static_cast<size_t>(p.H + h) * p.gate_h] + p.gate_bias[p.H + h];
   li = p.cap * tanhf(zi / p.cap);
   const float z = p.cap * tanhf(zf / p.cap);
   lf = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
 }
 
-// inclusive prefix over the 128 threads (threads in token order)
+// inclusive prefix over 128 threads in token order, in both halves of the CTA alike
 template <bool MAX>
-__device__ __forceinline__ float chunk_prefix(float v, float* red) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+__device__ __forceinline__ float chunk_prefix(float v, float* red_all) {
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3;
+  float* red = red_all + 4 * (threadIdx.x >> 7);
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
     const float w = __shfl_up_sync(0xffffffffu, v, o);
@@ -85,7 +87,7 @@ __device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint3
 
 // ------------------------------------------------------------------------------------------------ states of single chunks
 template <bool GATED>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const ChunkParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -95,10 +97,11 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   uint8_t* sV = sKl + 2 * MC_PANEL;
   uint8_t* sOne = sV + p.pv * MC_PANEL;        // gated: a column of ones
   volatile int* abort_flag = &bars->abort_flag;
-  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x, warp = j >> 5, lane = j & 31;
+  // thread: token j of the chunk (later: key column j), half of the row's columns
+  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x & 127, half = threadIdx.x >> 7, warp = threadIdx.x >> 5;
   const int4 c = p.chunks[ch];
   const int t0 = c.x, n = c.y;
-  if (j == 0) {
+  if (threadIdx.x == 0) {
     mbar_init(&bars->qk_full, 1);
     mbar_init(&bars->v_full, 1);
     mbar_init(&bars->o_done, 1);
@@ -131,21 +134,22 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     __syncthreads();
     const float mloc = bars->red[9];
     w = j < n ? expf(e - mloc) : 0.f;
-    if (j == 0) {
+    if (threadIdx.x == 0) {
       p.stat[idx] = make_float2(mloc, Fend);
       if (c.w > -2) p.m_init[static_cast<size_t>(c.z) * p.H + h] = c.w < 0 ? 0.f : p.stab[(static_cast<size_t>(c.w) * p.H + h) * (p.dim + 1) + p.dim];
     }
-    for (int i = 0; i < 8; ++i) {              // the row's pieces, ones in the first column
+    for (int i = 4 * half; i < 4 * half + 4; ++i) {   // the row's pieces, ones in the first column
       const uint32_t one = i == 0 ? 0x3F80u : 0u;
       *reinterpret_cast<uint4*>(sOne + j * 128 + ((i ^ (j & 7)) << 4)) = make_uint4(one, 0u, 0u, 0u);
     }
   } else {
     w = j < n ? exp2f(p.log2_decay[h] * static_cast<float>(n - 1 - j)) : 0.f;
-    if (j == 0) p.stat[idx] = make_float2(0.f, p.log2_decay[h] * static_cast<float>(n));
+    if (threadIdx.x == 0) p.stat[idx] = make_float2(0.f, p.log2_decay[h] * static_cast<float>(n));
   }
   __syncthreads();
   const bool ok = mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
-  for (int i = 0; i < 16; ++i) {
+#pragma unroll 4
+  for (int i = 8 * half; i < 8 * half + 8; ++i) {
     const int off = (i >> 3) * MC_PANEL + j * 128 + (((i & 7) ^ (j & 7)) << 4);
     uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
     if (w != 0.f && i < 8 * p.pk) {
@@ -164,18 +168,18 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = bars->tmem_slot;
-  if (j == 0) {
+  if (threadIdx.x == 0) {
     const bool vok = mbar_wait(&bars->v_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL);
     if (ok && vok) {
       tc_fence_after();
       const uint32_t idesc = make_idesc_bf16(128, p.vpad, 1, 1), idesc1 = make_idesc_bf16(128, 16, 1, 1);
       const uint64_t dv = make_smem_desc(smem_u32(sV), MC_PANEL, 1024), d1 = make_smem_desc(smem_u32(sOne), MC_PANEL, 1024);
       const int steps = (n + 15) >> 4;
-      for (int half = 0; half < 2; ++half) {
-        const uint64_t dk = make_smem_desc(smem_u32(half ? sKl : sKh), MC_PANEL, 1024);
+      for (int part = 0; part < 2; ++part) {
+        const uint64_t dk = make_smem_desc(smem_u32(part ? sKl : sKh), MC_PANEL, 1024);
         for (int t = 0; t < steps; ++t) {
-          umma_bf16(tmem, dk + t * 128, dv + t * 128, idesc, (half || t) ? 1u : 0u);
-          if constexpr (GATED) umma_bf16(tmem + p.vpad, dk + t * 128, d1 + t * 128, idesc1, (half || t) ? 1u : 0u);
+          umma_bf16(tmem, dk + t * 128, dv + t * 128, idesc, (part || t) ? 1u : 0u);
+          if constexpr (GATED) umma_bf16(tmem + p.vpad, dk + t * 128, d1 + t * 128, idesc1, (part || t) ? 1u : 0u);
         }
       }
       umma_commit(&bars->o_done);
@@ -186,8 +190,8 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   if (mbar_wait(&bars->o_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
     tc_fence_after();
     float* u = p.u + idx * p.vrows * p.dimp + j;
-    const uint32_t ta = tmem + (static_cast<uint32_t>(warp * 32) << 16);
-    for (int v0 = 0; v0 < p.vrows; v0 += 16) {
+    const uint32_t ta = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
+    for (int v0 = 16 * half; v0 < p.vrows; v0 += 32) {
       uint32_t r[16];
       tmem_ld_32x16(ta + v0, r);
       tmem_ld_wait();
@@ -204,7 +208,6 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     tc_fence_after();
     tmem_dealloc(tmem, cols);
   }
-  (void)lane;
 }
 
 // ------------------------------------------------------------------------------------------------ recurrence over chunks
@@ -280,25 +283,27 @@ chunk_scan_kernel(const ChunkParams p) {
 
 // ------------------------------------------------------------------------------------------------ outputs
 template <bool GATED>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                  const __grid_constant__ CUtensorMap tmSh, const __grid_constant__ CUtensorMap tmSl, const ChunkParams p, int tmem_cols) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   ChunkBars* bars = reinterpret_cast<ChunkBars*>(smem);
   float* gj = reinterpret_cast<float*>(smem + 512);      // [128] exponent of key j
+  float* nsum = reinterpret_cast<float*>(smem + 1024);   // [2][128] partial n . q
   const int spanel = p.vrows * 128;
-  uint8_t* sQ = smem + 1024;
+  uint8_t* sQ = smem + 2048;
   uint8_t* sK = sQ + p.pk * MC_PANEL;
   uint8_t* sV = sK + p.pk * MC_PANEL;
   uint8_t* sSh = sV + p.pv * MC_PANEL;
   uint8_t* sSl = sSh + p.pk * spanel;
   volatile int* abort_flag = &bars->abort_flag;
-  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x, warp = j >> 5;
+  // thread: token j of the chunk; the two halves of the CTA share a token's columns
+  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x & 127, half = threadIdx.x >> 7, warp = threadIdx.x >> 5;
   const int4 c = p.chunks[ch];
   const int t0 = c.x, n = c.y;
   const size_t idx = static_cast<size_t>(ch) * p.H + h;
-  if (j == 0) {
+  if (threadIdx.x == 0) {
     mbar_init(&bars->qk_full, 1);
     mbar_init(&bars->v_full, 1);
     mbar_init(&bars->s_done, 1);
@@ -326,7 +331,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = bars->tmem_slot;
-  if (j == 0) {
+  if (threadIdx.x == 0) {
     const int ks = (p.dim + 15) >> 4;
     const uint64_t dq = make_smem_desc(smem_u32(sQ), 16, 1024), dk = make_smem_desc(smem_u32(sK), 16, 1024);
     if (mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
@@ -343,12 +348,12 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     if (mbar_wait(&bars->v_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
       tc_fence_after();
       const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 0), idesc1 = make_idesc_bf16(128, 16, 0, 0);
-      for (int half = 0; half < 2; ++half) {
-        const uint64_t ds = make_smem_desc(smem_u32(half ? sSl : sSh), 16, 1024);
+      for (int part = 0; part < 2; ++part) {
+        const uint64_t ds = make_smem_desc(smem_u32(part ? sSl : sSh), 16, 1024);
         for (int t = 0; t < ks; ++t) {
           const int oq = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3), os = (t >> 2) * (spanel >> 4) + 2 * (t & 3);
-          umma_bf16(tmem + MC_C, dq + oq, ds + os, idesc, (half || t) ? 1u : 0u);
-          if constexpr (GATED) umma_bf16(tmem + MC_C + p.vpad, dq + oq, ds + os + p.vpad * 8, idesc1, (half || t) ? 1u : 0u);
+          umma_bf16(tmem + MC_O, dq + oq, ds + os, idesc, (part || t) ? 1u : 0u);
+          if constexpr (GATED) umma_bf16(tmem + MC_O + p.vpad, dq + oq, ds + os + p.vpad * 8, idesc1, (part || t) ? 1u : 0u);
         }
       }
       umma_commit(&bars->o_done);
@@ -377,32 +382,37 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   }
   einter *= p.qscale;
   __syncthreads();
-  const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-  const uint32_t ts = tmem + lane_addr, to = ts + MC_C;
+  const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+  const uint32_t ts = tmem + lane_addr, tp = ts + MC_C, to = ts + MC_O;
   float nq = 0.f;
   const bool ok = mbar_wait(&bars->s_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
   if (ok) {
     tc_fence_after();
 #pragma unroll 1
-    for (int c0 = 0; c0 < MC_C; c0 += 32) {
-      uint32_t v[32];
-      tmem_ld_32x32(ts + c0, v);
-      tmem_ld_wait();
+    for (int c0 = 32 * half; c0 < MC_C; c0 += 64) {
       uint32_t packed[16];
+      if (c0 > (warp & 3) * 32) {                   // keys after every token of this warp
 #pragma unroll
-      for (int i = 0; i < 32; i += 4) {
-        const float4 g = *reinterpret_cast<const float4*>(gj + c0 + i);
-        float w[4] = {g.x, g.y, g.z, g.w};
+        for (int i = 0; i < 16; ++i) packed[i] = 0u;
+      } else {
+        uint32_t v[32];
+        tmem_ld_32x32(ts + c0, v);
+        tmem_ld_wait();
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          // the difference of the exponents first: it is small where the weight matters
-          w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * p.qscale * ex2_approx(arow + w[k]) : 0.f;
-          nq += w[k];
+        for (int i = 0; i < 32; i += 4) {
+          const float4 g = *reinterpret_cast<const float4*>(gj + c0 + i);
+          float w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            // the difference of the exponents first: it is small where the weight matters
+            w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * p.qscale * ex2_approx(arow + w[k]) : 0.f;
+            nq += w[k];
+          }
+          packed[i >> 1] = pack_bf16x2(w[0], w[1]);
+          packed[(i >> 1) + 1] = pack_bf16x2(w[2], w[3]);
         }
-        packed[i >> 1] = pack_bf16x2(w[0], w[1]);
-        packed[(i >> 1) + 1] = pack_bf16x2(w[2], w[3]);
       }
-      tmem_st_32x16(ts + (c0 >> 1), packed);        // over columns that have been read
+      tmem_st_32x16(tp + (c0 >> 1), packed);
     }
     tmem_st_wait();
   }
@@ -410,30 +420,25 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   if (ok && ok2) {
     tc_fence_after();
 #pragma unroll 1
-    for (int c0 = 0; c0 < p.vpad; c0 += 16) {
-      uint32_t v[16];
-      tmem_ld_32x16(to + c0, v);
+    for (int c0 = 32 * half; c0 < p.vrows; c0 += 64) {      // up to 16 unused columns behind the last
+      uint32_t v[32];
+      tmem_ld_32x32(to + c0, v);
       tmem_ld_wait();
 #pragma unroll
-      for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * einter);
-      tmem_st_32x16(to + c0, v);
-    }
-    if constexpr (GATED) {
-      uint32_t v[16];
-      tmem_ld_32x16(to + p.vpad, v);
-      tmem_ld_wait();
-      nq += __uint_as_float(v[0]) * einter;
+      for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * einter);
+      tmem_st_32x32(to + c0, v);
     }
     tmem_st_wait();
   }
+  if constexpr (GATED) nsum[half * MC_C + j] = nq;
   tc_fence_before();
   __syncthreads();
-  if (j == 0 && !*abort_flag) {
+  if (threadIdx.x == 0 && !*abort_flag) {
     tc_fence_after();
     const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 1);
     const uint64_t dv = make_smem_desc(smem_u32(sV), MC_PANEL, 1024);
     const int steps = (n + 15) >> 4;
-    for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_C, tmem + t * 8, dv + t * 128, idesc, 1u);
+    for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_O, tmem + MC_C + t * 8, dv + t * 128, idesc, 1u);
     umma_commit(&bars->qk_full);                    // its second phase
   }
   if (mbar_wait(&bars->qk_full, 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
@@ -443,6 +448,10 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
     float f = 1.f;
     if constexpr (GATED) {
+      uint32_t r[16];
+      tmem_ld_32x16(to + p.vpad, r);                // the state's part of n . q
+      tmem_ld_wait();
+      nq = nsum[j] + nsum[MC_C + j] + __uint_as_float(r[0]);
       f = 1.f / (fmaxf(fabsf(nq), expf(-mrow)) + 1e-6f);
       float ss = 0.f;
 #pragma unroll 1
@@ -461,24 +470,30 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const __nv_bfloat16* grow = GATED ? p.gate_out + t * p.ld_in + h * p.vdim : nullptr;
     const float* nw = GATED ? p.norm_w + h * p.vdim : nullptr;
 #pragma unroll 1
-    for (int c0 = 0; c0 < p.vpad; c0 += 16) {
+    for (int c0 = 16 * half; c0 < p.vpad; c0 += 32) {
+      float g[2][8];
+      if constexpr (GATED) {                        // requested before the accumulator is read
+#pragma unroll
+        for (int q = 0; q < 2; ++q)
+          if (c0 + 8 * q < p.vdim) ld8(grow + c0 + 8 * q, g[q]);
+      }
       uint32_t v[16];
       tmem_ld_32x16(to + c0, v);
       tmem_ld_wait();
       if (!live) continue;
 #pragma unroll
-      for (int q = 0; q < 16; q += 8) {
-        if (c0 + q >= p.vdim) continue;
+      for (int q = 0; q < 2; ++q) {
+        if (c0 + 8 * q >= p.vdim) continue;
         float o[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[q + i]) * f;
+        for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[8 * q + i]) * f;
         if constexpr (GATED) {
-          float g[8];
-          ld8(grow + c0 + q, g);
+          float w[8];
+          ld8(nw + c0 + 8 * q, w);
 #pragma unroll
-          for (int i = 0; i < 8; ++i) o[i] *= nw[c0 + q + i] * sigmoid_f(g[i]);
+          for (int i = 0; i < 8; ++i) o[i] *= w[i] * __fdividef(1.f, 1.f + __expf(-g[q][i]));
         }
-        st8(orow + c0 + q, o);
+        st8(orow + c0 + 8 * q, o);
       }
     }
   }
@@ -516,7 +531,7 @@ static int make_tmap_planes(CUtensorMap* out, const void* base, uint64_t cols, u
 }
 
 static int mc_smem_state(int pv, bool gated) { return 1024 + 1024 + (4 + pv + (gated ? 1 : 0)) * MC_PANEL; }
-static int mc_smem_out(int pk, int pv, int vrows) { return 1024 + 1024 + (2 * pk + pv) * MC_PANEL + 2 * pk * vrows * 128; }
+static int mc_smem_out(int pk, int pv, int vrows) { return 2048 + 1024 + (2 * pk + pv) * MC_PANEL + 2 * pk * vrows * 128; }
 
 }  // namespace b200
 
@@ -538,7 +553,7 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   const bool gated = p.gates != nullptr;
   if (!b200_memory_chunk_supported(p.dim, p.vdim, gated) || T <= 0 || n_chunks <= 0 || n_chunks > 65535 || n_seqs <= 0 || n_seqs > 65535 ||
       p.H <= 0 || p.H > 65535 || (p.ld_in & 7) || (p.ld_out & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return -1;
-  if (gated ? (!p.stab || !p.norm_w || !p.gate_bias || (reinterpret_cast<uintptr_t>(p.gate_out) & 15)) : !p.log2_decay) return -1;
+  if (gated ? (!p.stab || !p.norm_w || !p.gate_bias || ((reinterpret_cast<uintptr_t>(p.gate_out) | reinterpret_cast<uintptr_t>(p.norm_w)) & 15)) : !p.log2_decay) return -1;
   p.dimp = (p.dim + 7) & ~7;
   p.vpad = (p.vdim + 15) & ~15;
   p.vrows = mc_vrows(p.vdim, gated);
@@ -556,14 +571,14 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const int sm1 = mc_smem_state(p.pv, gated), sm3 = mc_smem_out(p.pk, p.pv, p.vrows);
   int cols = 256;
-  while (cols < MC_C + p.vrows) cols <<= 1;
+  while (cols < MC_O + ((p.vrows + 31) & ~31)) cols <<= 1;
 #define GO(G)                                                                                                          \
   {                                                                                                                    \
     if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
         cudaFuncSetAttribute(chunk_out_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
-    if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 128, sm1, st>>>(tk, tv, p);                              \
+    if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 256, sm1, st>>>(tk, tv, p);                              \
     if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 255) / 256, p.H, n_seqs), 256, 0, st>>>(p);      \
-    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 128, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
+    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 256, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
   }
   if (gated) GO(true) else GO(false)
 #undef GO

@@ -70,6 +70,7 @@ __device__ __forceinline__ float block_total(float v, float* red) {
   return t;
 }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 // factor on the queries of position p
 __device__ __forceinline__ float query_temperature(int p, int every, float coef) {
   return 1.f + coef * logf(static_cast<float>((p + 1) / every + 1));

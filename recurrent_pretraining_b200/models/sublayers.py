@@ -300,9 +300,7 @@ class ParallelMixer(nn.Module):
         return ops.linear(o, self.w_o[:, :L.width_o])
 
     def decode_splits(self, B: int, max_len: int, tensor_cores: bool) -> int:
-        """Key splits of the decode attention: enough CTAs to fill the machine, at least 64 keys each."""
-        ctas = B * mem_ops.decode_groups(self.layout, tensor_cores)
-        return max(1, min(max_len // 64 + 1, 32, -(-2 * 148 // ctas)))
+        return mem_ops.decode_splits(self.layout, B, max_len, tensor_cores)
 
     def decode(self, h, run: LayerRun, ctx: DecodeContext):
         L = self.layout
@@ -342,7 +340,7 @@ class GatedMemory(nn.Module):
     def stream(self, h, run: LayerRun, ctx: StepContext):
         a, data = self.spec, ctx.cache.data
         inp = ops.linear(h, self.w_in[:, :self.width])
-        gates = ops.linear(h, self.w_gate[:, :self.width], out_f32=True)
+        gates = mem_ops.gate_projections(h, self.w_gate[:, :self.width])
         o = mem_ops.gated_memory(self.layout, inp, gates, self.b_gate, a.gate_cap, data[run.index, "state"], data[run.index, "norm"], self.norm,
                                  self.eps, self.dtype, step=ctx.step)
         return ops.linear(o, self.w_o[:, :a.heads * a.vdim])

@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass, field
+from functools import lru_cache
 from typing import Optional
 
 import torch
@@ -83,7 +84,7 @@ class _Sandwich(C.Structure):
 
 
 class _Memory(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("H", "dim", "vdim", "ldv", "ld_in", "off_q", "off_k", "off_v", "off_g", "ld_out", "E", "ld_h", "ld_w", "ld_gates",
+    _fields_ = [(n, C.c_int) for n in ("H", "dim", "vdim", "ldv", "ld_in", "off_q", "off_k", "off_v", "off_g", "ld_out", "E", "ld_h", "ld_w", "gate_t", "gate_h",
                                        "silu", "stage")] + [(n, C.c_float) for n in ("qscale", "cap", "eps")] + \
                [(n, C.c_void_p) for n in ("seqs", "pos", "row", "decay", "gates", "gate_bias", "state", "stab", "norm_w", "out32")]
 
@@ -259,6 +260,21 @@ def prompt_attention(L: ParallelLayout, spec, inp: torch.Tensor, cache: torch.Te
 # ------------------------------------------------------------------------------------------
 # memories
 # ------------------------------------------------------------------------------------------
+def gate_projections(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """h w^T in fp32 for a few rows of w; the result may be strided.  bf16: the product streams h through the narrow-batch GEMM
+    (w takes the batch's place), whose split of the contraction fills the machine where a tiled product would run on T / 128
+    CTAs."""
+    T, n = h.shape[0], w.shape[0]
+    if h.is_cuda and h.dtype == BF16 and n <= 64 and 256 <= T <= 128 * 147 and h.shape[1] >= 512:
+        from ..engine.base import skinny_linear
+
+        work = torch.zeros(n * T, dtype=F32, device=h.device)
+        out = skinny_linear(w, h, work, keep_f32=True)
+        if out.dtype == F32:
+            return out.T
+    return linear(h, w, out_f32=True)
+
+
 def _heads(inp, at: int, H: int, n: int) -> torch.Tensor:
     return inp[:, at:at + H * n].float().unflatten(1, (H, n))
 
@@ -288,11 +304,12 @@ def decay_memory_prompt(L: ParallelLayout, inp: torch.Tensor, decay: torch.Tenso
     return _decay_scan(L, inp, decay, state, step.seq_table, None, None, len(step.portions), 0)
 
 
-def _decay_scan(L, inp, decay, state, seqs, pos, row, n: int, raw: int) -> torch.Tensor:
+def _decay_scan(L, inp, decay, state, seqs, pos, row, n: int, raw: int, out=None) -> torch.Tensor:
     k = _k()
     p = k.K._ptr
-    out = torch.empty(inp.shape[0], pad8(L.r_heads * L.r_vdim), dtype=F32, device=inp.device)[:, :L.r_heads * L.r_vdim]
-    m = _Memory(L.r_heads, L.r_dim, L.r_vdim, L.ldv, inp.stride(0), L.off_rq, L.off_rk, L.off_rv, 0, out.stride(0), 0, 0, 0, 0, raw, 0, 1.0, 1.0, 0.0,
+    if out is None:
+        out = torch.empty(inp.shape[0], pad8(L.r_heads * L.r_vdim), dtype=F32, device=inp.device)[:, :L.r_heads * L.r_vdim]
+    m = _Memory(L.r_heads, L.r_dim, L.r_vdim, L.ldv, inp.stride(0), L.off_rq, L.off_rk, L.off_rv, 0, out.stride(0), 0, 0, 0, 0, 0, raw, 0, 1.0, 1.0, 0.0,
                 p(seqs), p(pos), p(row), decay.data_ptr(), 0, 0, state.data_ptr(), 0, 0, out.data_ptr())
     k.K._check(k.scan(inp.data_ptr(), 0, 0, 0, C.byref(m), n, _f32(inp), 0, k.K._stream()), "memory_scan")
     return out
@@ -314,14 +331,17 @@ def memory_norm(L: ParallelLayout, inp: torch.Tensor, mem: torch.Tensor, norm_w:
                "memory_merge")
 
 
-def decode_groups(L: ParallelLayout, tensor_cores: bool) -> int:
-    """CTAs per row and key split of the decode attention."""
+@lru_cache(None)
+def decode_splits(L: ParallelLayout, B: int, max_len: int, tensor_cores: bool) -> int:
+    """Key splits of the decode attention for ``B`` rows: the fewest waves of CTAs, each costing its keys and a fixed part worth
+    about 256 more."""
+    ctas, slots = B * L.heads, 8 * 148                     # generic kernel: a small CTA per head
     if tensor_cores:
         from . import memory_kernels as MK
 
         if MK.decode_supported(L):
-            return L.kv_heads
-    return L.heads
+            ctas, slots = B * L.kv_heads * -(-(L.heads // L.kv_heads) // 16), MK.decode_slots(L)
+    return min(range(1, min(32, max_len // 64 + 1) + 1), key=lambda s: -(-ctas * s // slots) * (max_len / s + 256))
 
 
 def parallel_output(L: ParallelLayout, T: int, dtype, device) -> torch.Tensor:
@@ -351,9 +371,23 @@ def parallel_decode(L: ParallelLayout, spec, inp: torch.Tensor, bias: torch.Tens
     po = torch.empty(B, L.heads, splits, pad8(L.vdim), dtype=F32, device=inp.device)
     ml = torch.empty(B, L.heads, splits, 2, dtype=F32, device=inp.device)
     attend, scan, merge = parallel_decode_pieces(L, spec, inp, bias, cache, state, table, decay, norm_w, eps, pos, row, po, ml, out)
-    attend()
-    merge(scan())
+    if torch.cuda.is_current_stream_capturing():           # the two halves are independent branches of the graph
+        main, side = torch.cuda.current_stream(), _side_stream(inp.device)
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            mem = scan()
+        attend()
+        main.wait_stream(side)
+        merge(mem)
+    else:
+        attend()
+        merge(scan())
     return out
+
+
+@lru_cache(None)
+def _side_stream(device) -> "torch.cuda.Stream":
+    return torch.cuda.Stream(device)
 
 
 def parallel_decode_pieces(L, spec, inp, bias, cache, state, table, decay, norm_w, eps, pos, row, po, ml, out):
@@ -376,8 +410,10 @@ def parallel_decode_pieces(L, spec, inp, bias, cache, state, table, decay, norm_
         k.K._check(k.attn(q.data_ptr(), cache.data_ptr(), 0, cache[:, :, L.kv_v:].data_ptr(), 0, 0, C.byref(s), B, int(dtype == F32), k.K._stream()),
                    "window_attention")
 
+    mem = torch.empty(B, pad8(L.r_heads * L.r_vdim), dtype=F32, device=inp.device)[:, :L.r_heads * L.r_vdim]
+
     def scan():
-        return _decay_scan(L, inp, decay, state, None, pos, row, B, 1)
+        return _decay_scan(L, inp, decay, state, None, pos, row, B, 1, mem)
 
     def merge(mem):
         memory_norm(L, inp, mem, norm_w, eps, spec.right_scale, out, (po, ml), spec.left_scale)
@@ -426,7 +462,8 @@ def gated_memory(L: MemoryLayout, inp: torch.Tensor, gates, gate_bias: torch.Ten
     out = torch.empty(T, pad8(hv), dtype=dtype, device=inp.device)[:, :hv]
     pos, row = rows if rows is not None else (None, None)
     m = _Memory(H, L.dim, L.vdim, L.ldv, inp.stride(0), L.off_q, L.off_k, L.off_v, L.off_g, out.stride(0), 0 if h is None else h.shape[1],
-                0 if h is None else h.stride(0), 0 if w_gate is None else w_gate.stride(0), 0 if gates is None else gates.stride(0), 0, 0, qscale, cap, eps,
+                0 if h is None else h.stride(0), 0 if w_gate is None else w_gate.stride(0), 0 if gates is None else gates.stride(0),
+                0 if gates is None else gates.stride(1), 0, 0, qscale, cap, eps,
                 step.seq_table.data_ptr() if step is not None else 0, p(pos), p(row), 0, p(gates), gate_bias.data_ptr(), state.data_ptr(),
                 stab.data_ptr(), norm_w.data_ptr(), 0)
     k.K._check(k.scan(inp.data_ptr(), p(h), p(w_gate), out.data_ptr(), C.byref(m), len(step.portions) if step is not None else T, _f32(inp),

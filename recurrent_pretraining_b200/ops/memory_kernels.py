@@ -20,7 +20,7 @@ class _GqaDecode(C.Structure):
 
 
 class _Chunks(C.Structure):
-    _fields_ = [(n, _i) for n in ("H", "dim", "vdim", "dimp", "vpad", "vrows", "pk", "pv", "ldv", "ld_in", "ld_out", "ld_gates")] + \
+    _fields_ = [(n, _i) for n in ("H", "dim", "vdim", "dimp", "vpad", "vrows", "pk", "pv", "ldv", "ld_in", "ld_out", "gate_t", "gate_h")] + \
                [(n, _f) for n in ("qscale", "cap", "eps")] + \
                [(n, _vp) for n in ("chunks", "seqs", "log2_decay", "gates", "gate_bias", "u", "stat", "s_hi", "s_lo", "m_before", "m_init", "state",
                                    "stab", "gate_out", "norm_w", "out", "err")]
@@ -30,6 +30,7 @@ _attn_ok = K._sig("b200_biased_attention_supported", [_i, _i])
 _attn_pad = K._sig("b200_biased_attention_pad", [_i])
 _attn = K._sig("b200_biased_attention", [_vp] * 8 + [_i] * 14 + [_f, _f, _f, _vp, _vp])
 _dec_ok = K._sig("b200_gqa_decode_supported", [_i, _i])
+_dec_per_sm = K._sig("b200_gqa_decode_per_sm", [_i, _i])
 _dec = K._sig("b200_gqa_decode", [_vp, C.POINTER(_GqaDecode), _i, _i, _vp])
 _chunk_ok = K._sig("b200_memory_chunk_supported", [_i, _i, _i])
 _chunk = K._sig("b200_memory_chunks", [_vp] * 3 + [C.POINTER(_Chunks)] + [_i] * 4 + [_vp, _vp])
@@ -51,6 +52,12 @@ def prompt_supported(L, spec) -> bool:
 @lru_cache(None)
 def decode_supported(L) -> bool:
     return bool(_dec_ok(L.dim, L.vdim))
+
+
+@lru_cache(None)
+def decode_slots(L) -> int:
+    """CTAs of the decode kernel that the machine holds at a time."""
+    return 148 * int(_dec_per_sm(L.dim, L.vdim))
 
 
 def padded_bias(values: torch.Tensor) -> torch.Tensor:
@@ -120,7 +127,8 @@ def _chunked(step, q, k, v, H: int, dim: int, vdim: int, ldv: int, out, state, q
     scal = torch.empty(3 * n * H + S * H, dtype=F32, device=dev)
     stat, m_before, m_init = scal[:2 * n * H], scal[2 * n * H:3 * n * H], scal[3 * n * H:]
     p = K._ptr
-    c = _Chunks(H, dim, vdim, 0, 0, 0, 0, 0, ldv, q.stride(0), out.stride(0), 0 if gates is None else gates.stride(0), qscale, cap, eps,
+    c = _Chunks(H, dim, vdim, 0, 0, 0, 0, 0, ldv, q.stride(0), out.stride(0), 0 if gates is None else gates.stride(0), 0 if gates is None else gates.stride(1),
+                qscale, cap, eps,
                 chunks.data_ptr(), seqs.data_ptr(), p(decay), p(gates), p(gate_bias), u.data_ptr(), stat.data_ptr(), hi.data_ptr(), lo.data_ptr(),
                 m_before.data_ptr(), m_init.data_ptr(), state.data_ptr(), p(stab), p(gate_out), p(norm_w), out.data_ptr(), 0)
     keep = (u, hi, lo, scal, q, decay, gates, gate_bias, state, stab, gate_out, norm_w)      # alive as long as the callable

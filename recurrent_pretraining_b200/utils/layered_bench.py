@@ -1,7 +1,7 @@
 """Prefill and decode throughput of the layered decoder models beside the recurrent model at equal size, and the time of
 every kernel of a layer against its roofline.
 
-``python -m recurrent_pretraining_b200.utils.layered_bench [--shapes gasovik-1b,gasovik-core-5280] [--ops-only]``.
+``python -m recurrent_pretraining_b200.utils.layered_bench [--shapes gasovik-1b,fatudra-1b,...] [--ops-only]``.
 Random weights.  Model runs: CUDA events around whole prefill / decode calls of the two engines (graph-replayed decode).
 Kernels: CUDA events around single calls on the shapes of one layer, L2 flushed in between, median.  The comparison
 model is the depth-recurrent model run for one recurrence: as many layers of the same width, head count and value
@@ -11,6 +11,7 @@ from __future__ import annotations
 import argparse
 import json
 import os
+from dataclasses import replace
 
 import torch
 
@@ -74,6 +75,7 @@ def closest_model(cfg):
 
     n, E = len(cfg.layers), cfg.width
     a = cfg.layers[0].mixer
+    a = getattr(a, "left", a)
     per_layer = (cfg.param_count() - 2 * cfg.vocab * E) / n
     ff = max(256, int((per_layer - 4 * E * E) / (3 * E)) // 64 * 64)
     core = max(1, n // 2)
@@ -178,6 +180,121 @@ def layer_ops_decode(model, B: int, context: int, t: Timer) -> list:
         skinny("up projection", xb, layer.mlp.w_up[:, :E])
         t.op("bias + relu^2", lambda: ops.bias_act(work[:, :ff], layer.mlp.b_up, "relu2", torch.bfloat16), B * ff * 6.0, 0)
         skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), layer.mlp.w_down[:, :ff])
+    return t.take()
+
+
+def hybrid_ops_prefill(model, seqs: list, t: Timer) -> list:
+    """Kernels of a parallel layer, of a gated memory layer and of a feed-forward of a packed step of fresh prompts ``seqs``."""
+    from ..models.layered import PackedStep
+    from ..ops import latent as ops
+    from ..ops import memory as M
+    from ..ops import memory_kernels as MK
+
+    cfg, E, T = model.config, model.config.width, sum(seqs)
+    kinds = {layer.type: i for i, layer in reversed(list(enumerate(cfg.layers)))}
+    cache = model.new_cache(len(seqs), max(seqs))
+    step = PackedStep([(r, 0, [1] * n) for r, n in enumerate(seqs)], "cuda")
+    x = torch.randn(T, E, device="cuda")
+    h = torch.randn(T, E, device="cuda").bfloat16()
+
+    def gemm(name, fn, M_, N, K):
+        t.op(name, fn, 2.0 * (M_ * N + M_ * K + N * K), 2.0 * M_ * N * K)
+
+    i = kinds["parallel"]
+    mix = model.layers[i].mix
+    L, a, r = mix.layout, mix.spec.left, mix.spec.right
+    kv, state = cache.data[i, "kv"], cache.data[i, "state"]
+    project = lambda: ops.linear(h, mix.w_in[:, :E], mix.b_in, "silu", act_cols=L.act_cols)  # noqa: E731
+    inp = project()
+    o = M.parallel_output(L, T, torch.bfloat16, h.device)
+    gemm("parallel: input projection + bias + silu", project, T, L.width_in, E)
+    t.op("parallel: kv_append", lambda: M.kv_append(L, inp, None, kv, step.pos, step.row), 4.0 * T * L.ld_kv, 0)
+    t.op("parallel: attention (bias, head gate)", lambda: M.prompt_attention(L, a, inp, kv, mix.table, step, 0.7, o),
+         2.0 * T * (a.heads * (a.dim + a.vdim) + L.ld_kv), 2.0 * visible_pairs(seqs, max(seqs)) * a.heads * (a.dim + a.vdim))
+    mem = M.decay_memory_prompt(L, inp, mix.decay, mix.log2_decay, state, step)
+    run = MK.decay_memory(L, inp, mix.log2_decay, state, step)
+    nbytes = 2.0 * T * r.heads * (2 * r.dim + 2 * r.vdim)
+    t.op("parallel: memory (3 kernels)", run, nbytes, 4.0 * T * r.heads * r.dim * r.vdim)
+    for part, name in ((1, "chunk states"), (2, "recurrence"), (4, "outputs")):
+        t.op("  memory: " + name, lambda part=part: run(part), nbytes, 0)
+    t.op("parallel: memory norm + gate", lambda: M.memory_norm(L, inp, mem, mix.norm, 1e-6, 0.7, o), 6.0 * T * r.heads * r.vdim, 0)
+    gemm("parallel: output projection", lambda: ops.linear(o, mix.w_o[:, :L.width_o]), T, E, L.width_o)
+    norms = model.layers[i].norms
+    out = ops.linear(o, mix.w_o[:, :L.width_o])
+    t.op("sandwich_norm", lambda: M.sandwich_norm_(x, out, norms["norm1b"].pair, None, norms["norm2"].pair, 1e-6, torch.bfloat16), T * E * 12.0, 0)
+    i = kinds["mlstm"]
+    mix = model.layers[i].mix
+    L, a = mix.layout, mix.spec
+    state, stab = cache.data[i, "state"], cache.data[i, "norm"]
+    inp, gates = ops.linear(h, mix.w_in[:, :E]), M.gate_projections(h, mix.w_gate[:, :E])
+    gemm("gated memory: input projection", lambda: ops.linear(h, mix.w_in[:, :E]), T, L.width_in, E)
+    gemm("gated memory: gate projection (fp32)", lambda: M.gate_projections(h, mix.w_gate[:, :E]), T, 2 * a.heads, E)
+    run = MK.gated_memory(L, inp, gates, mix.b_gate, a.gate_cap, state, stab, mix.norm, 1e-6, step)
+    nbytes = 2.0 * T * a.heads * (2 * a.dim + 3 * a.vdim)
+    t.op("gated memory: memory (3 kernels)", run, nbytes, 4.0 * T * a.heads * a.dim * a.vdim)
+    for part, name in ((1, "chunk states"), (2, "recurrence"), (4, "outputs + norm + gate")):
+        t.op("  memory: " + name, lambda part=part: run(part), nbytes, 0)
+    mlp = model.layers[i].mlp
+    ff = mlp.spec.ff
+    g = M.geglu_linear(h, mlp.w_gu[:, :E], ff)
+    gemm("gate-up projection + geglu", lambda: M.geglu_linear(h, mlp.w_gu[:, :E], ff), T, 2 * ff, E)
+    gemm("down projection", lambda: ops.linear(g, mlp.w_down[:, :ff]), T, E, ff)
+    return t.take()
+
+
+def hybrid_ops_decode(model, B: int, context: int, t: Timer) -> list:
+    from ..engine.layered import LayeredEngine
+    from ..ops import memory as M
+
+    cfg, E = model.config, model.config.width
+    kinds = {layer.type: i for i, layer in reversed(list(enumerate(cfg.layers)))}
+    eng = LayeredEngine(model, B, context + 1, use_graphs=False)
+    cache = eng.cache
+    for key, d in cache.data.items():
+        d.normal_(std=0.1)
+    pos = torch.full((B,), context, dtype=torch.int32, device="cuda")
+    row = torch.arange(B, dtype=torch.int32, device="cuda")
+    x = torch.randn(B, E, device="cuda")
+    h = x.bfloat16()
+    work = torch.zeros(B, max(E, 2 * cfg.layers[0].mlp.ff), dtype=torch.float32, device="cuda")
+
+    def skinny(name, xin, w):
+        N, K = w.shape
+        t.op(name, lambda: eng._dense(xin, w, 1 if N * B <= eng._work[1].numel() else 0), 2.0 * (N * K + B * K + B * N), 2.0 * B * N * K)
+
+    i = kinds["parallel"]
+    mix = model.layers[i].mix
+    L, a, r = mix.layout, mix.spec.left, mix.spec.right
+    skinny("parallel: input projection", h, mix.w_in[:, :E])
+    inp = torch.randn(B, L.width_in, device="cuda")
+    splits = mix.decode_splits(B, context + 1, True)
+    po = torch.empty(B, L.heads, splits, M.pad8(L.vdim), dtype=torch.float32, device="cuda")
+    ml = torch.empty(B, L.heads, splits, 2, dtype=torch.float32, device="cuda")
+    o = M.parallel_output(L, B, torch.bfloat16, h.device)
+    attend, scan, merge = M.parallel_decode_pieces(L, mix.spec, inp, mix.b_in, cache.data[i, "kv"], cache.data[i, "state"], mix.table, mix.decay,
+                                                   mix.norm, 1e-6, pos, row, po, ml, o)
+    t.op("parallel: decode attention", attend, 2.0 * B * ((context + 1) * L.ld_kv + a.heads * (a.dim + a.vdim)),
+         2.0 * B * a.heads * context * (a.dim + a.vdim))
+    t.op("parallel: memory update", scan, 8.0 * B * r.heads * r.dim * r.vdim, 0)
+    mem = scan()
+    t.op("parallel: merge, norm, gates", lambda: merge(mem), B * (4.0 * splits * a.heads * a.vdim + 2.0 * L.width_o + 8.0 * r.heads * r.vdim), 0)
+    skinny("parallel: output projection", o, mix.w_o[:, :L.width_o])
+    norms = model.layers[i].norms
+    acc = work[:, :E]
+    t.op("sandwich_norm", lambda: M.sandwich_norm_(x, acc, norms["norm1b"].pair, None, norms["norm2"].pair, 1e-6, torch.bfloat16), B * E * 14.0, 0)
+    i = kinds["mlstm"]
+    mix = model.layers[i].mix
+    L, a = mix.layout, mix.spec
+    skinny("gated memory: input projection", h, mix.w_in[:, :E])
+    inp = torch.randn(B, L.width_in, device="cuda")
+    t.op("gated memory: update, norm, gates", lambda: M.gated_memory(L, inp, None, mix.b_gate, a.gate_cap, cache.data[i, "state"], cache.data[i, "norm"],
+                                                                     mix.norm, 1e-6, torch.bfloat16, rows=(pos, row), h=h, w_gate=mix.w_gate[:, :E]),
+         8.0 * B * a.heads * a.dim * (a.vdim + 1) + 4.0 * a.heads * E, 0)
+    mlp = model.layers[i].mlp
+    ff = mlp.spec.ff
+    skinny("gate-up projection", h, mlp.w_gu[:, :E])
+    t.op("geglu", lambda: M.geglu(work[:, :2 * ff], ff, torch.bfloat16), B * ff * 10.0, 0)
+    skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), mlp.w_down[:, :ff])
     return t.take()
 
 
@@ -295,7 +412,7 @@ def model_rates(cfg, prompt: int, new: int, batches) -> dict:
     return out
 
 
-def run(shapes=("gasovik-1b", "gasovik-core-5280"), batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
+def run(shapes=("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5280"), batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
     from ..models.layered import LayeredForCausalLM
     from ..models.layered_config import LayeredConfig
     from ..ops import cuda as K
@@ -308,13 +425,15 @@ def run(shapes=("gasovik-1b", "gasovik-core-5280"), batches=(1, 8, 32), prompt: 
             r["models"] = model_rates(cfg, prompt, new, batches)
             torch.cuda.empty_cache()
         t = Timer()
-        one = LayeredConfig(cfg.architecture, 1024, cfg.width, cfg.norm_eps, cfg.residual_mult, cfg.layers[:1])
-        model = LayeredForCausalLM(one, torch.bfloat16, "cuda").init_weights()
+        hybrid = cfg.design.norms == "sandwich"
+        ops_prefill, ops_decode = (hybrid_ops_prefill, hybrid_ops_decode) if hybrid else (layer_ops_prefill, layer_ops_decode)
+        few = replace(cfg, vocab=1024, layers=cfg.layers[:2 if hybrid else 1], loop=None)
+        model = LayeredForCausalLM(few, torch.bfloat16, "cuda").init_weights()
         S = 4096
-        r["prefill_ops"] = {"tokens": S, "ours": layer_ops_prefill(model, [S], t)}
-        r["decode_ops"] = {f"batch {B}": {"context": S, "ours": layer_ops_decode(model, B, S, t)} for B in (1, 8, 64)}
+        r["prefill_ops"] = {"tokens": S, "ours": ops_prefill(model, [S], t)}
+        r["decode_ops"] = {f"batch {B}": {"context": S, "ours": ops_decode(model, B, S, t)} for B in (1, 8, 64)}
         del model
-        ref = closest_model(LayeredConfig(cfg.architecture, 1024, cfg.width, cfg.norm_eps, cfg.residual_mult, cfg.layers[:3]))
+        ref = closest_model(replace(cfg, vocab=1024, layers=cfg.layers[:3], loop=None))
         r["prefill_ops"]["closest"] = closest_ops_prefill(ref, 1, S, t)
         for B in (1, 8, 64):
             r["decode_ops"][f"batch {B}"]["closest"] = closest_ops_decode(ref, B, S, t)
@@ -328,7 +447,7 @@ def run(shapes=("gasovik-1b", "gasovik-core-5280"), batches=(1, 8, 32), prompt: 
 
 def main():
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("--shapes", default="gasovik-1b,gasovik-core-5280")
+    ap.add_argument("--shapes", default="gasovik-1b,gasovik-core-5280,fatudra-1b,fatudra-core-5280")
     ap.add_argument("--batches", default="1,8,32")
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--new", type=int, default=128)
@@ -345,7 +464,7 @@ def main():
         for title, block in [("prefill", r["prefill_ops"])] + [(f"decode {b}", d) for b, d in r["decode_ops"].items()]:
             for who in ("ours", "closest"):
                 for row in block[who]:
-                    print(f"{name:18s} {title:16s} {who:8s} {row['op']:32s} {row['us']:9.2f} us  floor {row['roofline_us']:8.2f}  "
+                    print(f"{name:18s} {title:16s} {who:8s} {row['op']:42s} {row['us']:9.2f} us  floor {row['roofline_us']:8.2f}  "
                           f"{row['fraction']:.3f} {row['bound']}")
 
 

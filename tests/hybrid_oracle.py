@@ -33,8 +33,8 @@ def layer_norm(x, eps, w, b):
 def bucket(n, rows, reach):
     """Row of the bias table for distance ``n``: exact up to half the rows, then logarithmic up to ``reach``."""
     half = rows // 2
-    if n < half:
-        return n
+    if n < half or rows == 1:
+        return min(n, rows - 1)
     return min(rows - 1, half + math.floor(math.log(n / half) / math.log(reach / half) * (rows - half)))
 
 
