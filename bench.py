@@ -362,7 +362,7 @@ def run_layered(args):
         "metric": "decode tokens/sec (gasovik-1b, batch 32, prompt 2048, greedy)", "value": first["ours"]["32"]["decode_tok_s"],
         "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "impl": "ours",
         "data": "synthetic uniform-random tokens, random-init weights",
-        "config": {"model": "gasovik-1b, gasovik-core-5280", "l2": "flushed between single-kernel timings; whole models stream more than L2"},
+        "config": {"model": ", ".join(k for k, v in rec.items() if isinstance(v, dict)), "l2": "flushed between single-kernel timings; whole models stream more than L2"},
         "clocks": clocks, "gpu_launches": C.launch_count() - launches0, "layered": rec}), flush=True)
 
 

@@ -19,7 +19,6 @@ namespace b200 {
 
 constexpr int MC_C = 128;                     // tokens per chunk
 constexpr int MC_PANEL = MC_C * 128;          // 128 rows x 64 bf16
-constexpr int MC_O = MC_C + MC_C / 2;         // tensor-memory columns: scores, bf16 weights, outputs
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct ChunkParams {
@@ -35,7 +34,8 @@ struct ChunkParams {
   const float* gate_bias;         // [2H]
   float* u;                       // [chunks * H, vrows, dimp]
   float2* stat;                   // [chunks * H] {m_loc, F_end}
-  __nv_bfloat16 *s_hi, *s_lo;     // [chunks * H, vrows, dimp]
+  __nv_bfloat16 *s_hi, *s_lo;     // [chunks * H, vpad, dimp]
+  float* n_before;                // gated: [chunks * H, dimp] normaliser before each chunk
   float* m_before;                // [chunks * H]
   float* m_init;                  // [sequences * H]
   float* state;                   // cache [rows, H, dim, ldv]
@@ -47,7 +47,7 @@ struct ChunkParams {
 };
 
 struct ChunkBars {
-  uint64_t qk_full, v_full, s_done, o_done;
+  uint64_t qk_full, v_full, o_done;
   uint32_t tmem_slot;
   int abort_flag;
   float red[16];
@@ -72,9 +72,9 @@ __device__ __forceinline__ float chunk_prefix(float v, float* red_all) {
     const float w = __shfl_up_sync(0xffffffffu, v, o);
     if (lane >= o) v = MAX ? fmaxf(v, w) : v + w;
   }
-  __syncthreads();
+  named_barrier_sync(1, 256);                  // the eight warps that hold tokens
   if (lane == 31) red[warp] = v;
-  __syncthreads();
+  named_barrier_sync(1, 256);
   for (int w = 0; w < warp; ++w) v = MAX ? fmaxf(v, red[w]) : v + red[w];
   return v;
 }
@@ -235,8 +235,8 @@ chunk_scan_kernel(const ChunkParams p) {
       }
   }
   float m = GATED ? p.m_init[static_cast<size_t>(blockIdx.z) * p.H + h] : 0.f;
-  const size_t pitch = static_cast<size_t>(p.vrows) * p.dimp, at = static_cast<size_t>(v) * p.dimp + d;
-  constexpr int U = 4;
+  const size_t pitch = static_cast<size_t>(p.vrows) * p.dimp, spitch = static_cast<size_t>(p.vpad) * p.dimp, at = static_cast<size_t>(v) * p.dimp + d;
+  constexpr int U = 8;                         // chunks in flight
   for (int b = 0; b < nc; b += U) {
     float4 u[U];
     float2 f[U];
@@ -251,11 +251,15 @@ chunk_scan_kernel(const ChunkParams p) {
     for (int k = 0; k < U; ++k)
       if (b + k < nc) {
         const size_t idx = static_cast<size_t>(c0 + b + k) * p.H + h;
-        uint2 hi, lo;
-        split_pack(s[0], s[1], hi.x, lo.x);
-        split_pack(s[2], s[3], hi.y, lo.y);
-        *reinterpret_cast<uint2*>(p.s_hi + idx * pitch + at) = hi;
-        *reinterpret_cast<uint2*>(p.s_lo + idx * pitch + at) = lo;
+        if (!GATED || v < p.vpad) {
+          uint2 hi, lo;
+          split_pack(s[0], s[1], hi.x, lo.x);
+          split_pack(s[2], s[3], hi.y, lo.y);
+          *reinterpret_cast<uint2*>(p.s_hi + idx * spitch + at) = hi;
+          *reinterpret_cast<uint2*>(p.s_lo + idx * spitch + at) = lo;
+        } else if (is_norm) {
+          *reinterpret_cast<float4*>(p.n_before + idx * p.dimp + d) = make_float4(s[0], s[1], s[2], s[3]);
+        }
         float a, w = 1.f;
         if constexpr (GATED) {
           if (e == 0) p.m_before[idx] = m;
@@ -282,48 +286,57 @@ chunk_scan_kernel(const ChunkParams p) {
 }
 
 // ------------------------------------------------------------------------------------------------ outputs
+struct ChunkOutBars {
+  uint64_t qk_full, v_full, s_full, s_done, o_part, o_done, p_ready, final;
+  uint32_t tmem_slot;
+  int abort_flag;
+  float red[8];
+};
+
+// Warps 0-7: token j = thread & 127 of the chunk, its columns shared by the two halves; warp 8: copies and MMAs.
+// Shared memory is used twice so that two CTAs fit an SM: the values follow the keys once the scores are formed, the state's
+// remainder follows its head once that product is done.  Tensor memory: scores, then bf16 weights over them; outputs at MC_C.
 template <bool GATED>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(288, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                  const __grid_constant__ CUtensorMap tmSh, const __grid_constant__ CUtensorMap tmSl, const ChunkParams p, int tmem_cols) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  ChunkBars* bars = reinterpret_cast<ChunkBars*>(smem);
+  ChunkOutBars* bars = reinterpret_cast<ChunkOutBars*>(smem);
   float* gj = reinterpret_cast<float*>(smem + 512);      // [128] exponent of key j
   float* nsum = reinterpret_cast<float*>(smem + 1024);   // [2][128] partial n . q
-  const int spanel = p.vrows * 128;
-  uint8_t* sQ = smem + 2048;
-  uint8_t* sK = sQ + p.pk * MC_PANEL;
-  uint8_t* sV = sK + p.pk * MC_PANEL;
-  uint8_t* sSh = sV + p.pv * MC_PANEL;
-  uint8_t* sSl = sSh + p.pk * spanel;
+  float* nb = reinterpret_cast<float*>(smem + 2048);     // [128] normaliser before the chunk
+  const int spanel = p.vpad * 128;
+  uint8_t* sQ = smem + 3072;
+  uint8_t* sKV = sQ + p.pk * MC_PANEL;
+  uint8_t* sS = sKV + max(p.pk, p.pv) * MC_PANEL;
   volatile int* abort_flag = &bars->abort_flag;
-  // thread: token j of the chunk; the two halves of the CTA share a token's columns
-  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x & 127, half = threadIdx.x >> 7, warp = threadIdx.x >> 5;
+  const int h = blockIdx.x, ch = blockIdx.y, j = threadIdx.x & 127, half = threadIdx.x >> 7, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int4 c = p.chunks[ch];
   const int t0 = c.x, n = c.y;
   const size_t idx = static_cast<size_t>(ch) * p.H + h;
-  if (threadIdx.x == 0) {
+  if (threadIdx.x == 256) {
     mbar_init(&bars->qk_full, 1);
     mbar_init(&bars->v_full, 1);
+    mbar_init(&bars->s_full, 1);
     mbar_init(&bars->s_done, 1);
+    mbar_init(&bars->o_part, 1);
     mbar_init(&bars->o_done, 1);
+    mbar_init(&bars->p_ready, 8);
+    mbar_init(&bars->final, 1);
     bars->abort_flag = 0;
     fence_barrier_init();
     fence_proxy_async_smem();
     mbar_expect_tx(&bars->qk_full, p.pk * 2 * MC_PANEL);
     for (int i = 0; i < p.pk; ++i) {
       tma_load_3d(sQ + i * MC_PANEL, &tmQ, &bars->qk_full, i * 64, t0, h);
-      tma_load_3d(sK + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, h);
+      tma_load_3d(sKV + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, h);
     }
-    mbar_expect_tx(&bars->v_full, p.pv * MC_PANEL + 2 * p.pk * spanel);
-    for (int i = 0; i < p.pk; ++i) {
-      tma_load_3d(sSh + i * spanel, &tmSh, &bars->v_full, i * 64, 0, static_cast<int>(idx));
-      tma_load_3d(sSl + i * spanel, &tmSl, &bars->v_full, i * 64, 0, static_cast<int>(idx));
-    }
-    for (int i = 0; i < p.pv; ++i) tma_load_3d(sV + i * MC_PANEL, &tmV, &bars->v_full, i * 64, t0, h);
+    mbar_expect_tx(&bars->s_full, p.pk * spanel);
+    for (int i = 0; i < p.pk; ++i) tma_load_3d(sS + i * spanel, &tmSh, &bars->s_full, i * 64, 0, static_cast<int>(idx));
   }
-  if (warp == 1) {
+  if (warp == 8) {
+    __syncwarp();
     tmem_alloc(&bars->tmem_slot, tmem_cols);
     tmem_relinquish();
   }
@@ -331,69 +344,95 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = bars->tmem_slot;
-  if (threadIdx.x == 0) {
-    const int ks = (p.dim + 15) >> 4;
-    const uint64_t dq = make_smem_desc(smem_u32(sQ), 16, 1024), dk = make_smem_desc(smem_u32(sK), 16, 1024);
-    if (mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
-      tc_fence_after();
-      const uint32_t idesc = make_idesc_bf16(128, MC_C, 0, 0);
-      for (int t = 0; t < ks; ++t) {
-        const int o = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3);
-        umma_bf16(tmem, dq + o, dk + o, idesc, t ? 1u : 0u);
-      }
-      umma_commit(&bars->s_done);
-    } else {
-      bars->abort_flag = 1;
-    }
-    if (mbar_wait(&bars->v_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL)) {
-      tc_fence_after();
-      const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 0), idesc1 = make_idesc_bf16(128, 16, 0, 0);
-      for (int part = 0; part < 2; ++part) {
-        const uint64_t ds = make_smem_desc(smem_u32(part ? sSl : sSh), 16, 1024);
+  if (warp == 8) {
+    if (lane == 0) {
+      const int ks = (p.dim + 15) >> 4;
+      const uint64_t dq = make_smem_desc(smem_u32(sQ), 16, 1024), dk = make_smem_desc(smem_u32(sKV), 16, 1024), ds = make_smem_desc(smem_u32(sS), 16, 1024),
+                     dv = make_smem_desc(smem_u32(sKV), MC_PANEL, 1024);
+      const uint32_t idesc_s = make_idesc_bf16(128, MC_C, 0, 0), idesc_o = make_idesc_bf16(128, p.vpad, 0, 0), idesc_v = make_idesc_bf16(128, p.vpad, 0, 1);
+      auto wait = [&](uint64_t* bar, uint32_t ph, int code) { return mbar_wait(bar, ph, abort_flag, p.err, code); };
+      auto state_product = [&](uint32_t acc) {
+        tc_fence_after();
+        for (int t = 0; t < ks; ++t)
+          umma_bf16(tmem + MC_C, dq + (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3), ds + (t >> 2) * (spanel >> 4) + 2 * (t & 3), idesc_o, (acc || t) ? 1u : 0u);
+      };
+      bool ok = wait(&bars->qk_full, 0, ERR_WAIT_TMA_FULL);
+      if (ok) {
+        tc_fence_after();
         for (int t = 0; t < ks; ++t) {
-          const int oq = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3), os = (t >> 2) * (spanel >> 4) + 2 * (t & 3);
-          umma_bf16(tmem + MC_O, dq + oq, ds + os, idesc, (part || t) ? 1u : 0u);
-          if constexpr (GATED) umma_bf16(tmem + MC_O + p.vpad, dq + oq, ds + os + p.vpad * 8, idesc1, (part || t) ? 1u : 0u);
+          const int o = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3);
+          umma_bf16(tmem, dq + o, dk + o, idesc_s, t ? 1u : 0u);
         }
+        umma_commit(&bars->s_done);
+        ok = wait(&bars->s_full, 0, ERR_WAIT_TMA_FULL);
       }
-      umma_commit(&bars->o_done);
-    } else {
-      bars->abort_flag = 1;
+      if (ok) {
+        state_product(0u);
+        umma_commit(&bars->o_part);
+        ok = wait(&bars->s_done, 0, ERR_WAIT_TMEM_FULL);          // the keys have been read
+      }
+      if (ok) {
+        mbar_expect_tx(&bars->v_full, p.pv * MC_PANEL);
+        for (int i = 0; i < p.pv; ++i) tma_load_3d(sKV + i * MC_PANEL, &tmV, &bars->v_full, i * 64, t0, h);
+        ok = wait(&bars->o_part, 0, ERR_WAIT_TMEM_FULL);          // the state's head has been read
+        if (ok) {
+          mbar_expect_tx(&bars->s_full, p.pk * spanel);
+          for (int i = 0; i < p.pk; ++i) tma_load_3d(sS + i * spanel, &tmSl, &bars->s_full, i * 64, 0, static_cast<int>(idx));
+          ok = wait(&bars->s_full, 1, ERR_WAIT_TMA_FULL);
+        }
+        if (ok) {
+          state_product(1u);
+          umma_commit(&bars->o_done);
+        }
+        const bool vok = wait(&bars->v_full, 0, ERR_WAIT_TMA_FULL);   // in any case: the copy has to land before the CTA ends
+        ok = ok && vok && wait(&bars->p_ready, 0, ERR_WAIT_TMEM_FULL);
+      }
+      if (ok) {
+        tc_fence_after();
+        const int steps = (n + 15) >> 4;
+        for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_C, tmem + t * 8, dv + t * 128, idesc_v, 1u);
+        umma_commit(&bars->final);
+      } else {
+        bars->abort_flag = 1;
+        // a copy in flight has to land before the CTA ends
+        const unsigned long long begin = globaltimer_ns();
+        while (!(mbar_try_wait(&bars->qk_full, 0) && mbar_try_wait(&bars->s_full, 0)) && globaltimer_ns() - begin < WAIT_LIMIT_NS) {}
+      }
     }
-  }
-  __syncwarp();
-  // exponents of this thread's row (and, as a key, of its column)
-  float arow, einter, mrow = 0.f;
-  if constexpr (GATED) {
-    float li = -INFINITY, lf = 0.f;
-    if (j < n) token_gates(p, t0 + j, h, li, lf);
-    const float F = chunk_prefix<false>(lf, bars->red);
-    const float pm = chunk_prefix<true>(li - F, bars->red);
-    const float mb = p.m_before[idx];
-    mrow = F + fmaxf(mb, pm);
-    arow = (F - mrow) * LOG2E;
-    einter = expf(F + mb - mrow);
-    gj[j] = (li - F) * LOG2E;
   } else {
-    const float ld = p.log2_decay[h];
-    arow = ld * static_cast<float>(j);
-    gj[j] = -arow;
-    einter = exp2f(ld * static_cast<float>(j + 1));
-  }
-  einter *= p.qscale;
-  __syncthreads();
-  const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
-  const uint32_t ts = tmem + lane_addr, tp = ts + MC_C, to = ts + MC_O;
-  float nq = 0.f;
-  const bool ok = mbar_wait(&bars->s_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
-  if (ok) {
-    tc_fence_after();
-#pragma unroll 1
-    for (int c0 = 32 * half; c0 < MC_C; c0 += 64) {
-      uint32_t packed[16];
-      if (c0 > (warp & 3) * 32) {                   // keys after every token of this warp
+    // exponents of this thread's row (and, as a key, of its column)
+    float arow, einter, mrow = 0.f;
+    if constexpr (GATED) {
+      float li = -INFINITY, lf = 0.f;
+      if (j < n) token_gates(p, t0 + j, h, li, lf);
+      if (threadIdx.x < p.dim) nb[threadIdx.x] = p.n_before[idx * p.dimp + threadIdx.x];
+      const float F = chunk_prefix<false>(lf, bars->red);
+      const float pm = chunk_prefix<true>(li - F, bars->red);
+      const float mb = p.m_before[idx];
+      mrow = F + fmaxf(mb, pm);
+      arow = (F - mrow) * LOG2E;
+      einter = expf(F + mb - mrow);
+      gj[j] = (li - F) * LOG2E;
+    } else {
+      const float ld = p.log2_decay[h];
+      arow = ld * static_cast<float>(j);
+      gj[j] = -arow;
+      einter = exp2f(ld * static_cast<float>(j + 1));
+    }
+    einter *= p.qscale;
+    named_barrier_sync(1, 256);
+    const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const uint32_t ts = tmem + lane_addr, to = ts + MC_C;
+    float nq = 0.f;
+    uint32_t packed[2][16];
+    bool ok = mbar_wait(&bars->s_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    if (ok) tc_fence_after();
 #pragma unroll
-        for (int i = 0; i < 16; ++i) packed[i] = 0u;
+    for (int b = 0; b < 2; ++b) {
+      const int c0 = 32 * half + 64 * b;
+      if (!ok || c0 > (warp & 3) * 32) {              // keys after every token of this warp
+#pragma unroll
+        for (int i = 0; i < 16; ++i) packed[b][i] = 0u;
       } else {
         uint32_t v[32];
         tmem_ld_32x32(ts + c0, v);
@@ -404,102 +443,111 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float w[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
-            // the difference of the exponents first: it is small where the weight matters
             w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * p.qscale * ex2_approx(arow + w[k]) : 0.f;
             nq += w[k];
           }
-          packed[i >> 1] = pack_bf16x2(w[0], w[1]);
-          packed[(i >> 1) + 1] = pack_bf16x2(w[2], w[3]);
+          packed[b][i >> 1] = pack_bf16x2(w[0], w[1]);
+          packed[b][(i >> 1) + 1] = pack_bf16x2(w[2], w[3]);
         }
       }
-      tmem_st_32x16(tp + (c0 >> 1), packed);
     }
-    tmem_st_wait();
-  }
-  const bool ok2 = mbar_wait(&bars->o_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
-  if (ok && ok2) {
-    tc_fence_after();
-#pragma unroll 1
-    for (int c0 = 32 * half; c0 < p.vrows; c0 += 64) {      // up to 16 unused columns behind the last
-      uint32_t v[32];
-      tmem_ld_32x32(to + c0, v);
-      tmem_ld_wait();
-#pragma unroll
-      for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * einter);
-      tmem_st_32x32(to + c0, v);
-    }
-    tmem_st_wait();
-  }
-  if constexpr (GATED) nsum[half * MC_C + j] = nq;
-  tc_fence_before();
-  __syncthreads();
-  if (threadIdx.x == 0 && !*abort_flag) {
-    tc_fence_after();
-    const uint32_t idesc = make_idesc_bf16(128, p.vpad, 0, 1);
-    const uint64_t dv = make_smem_desc(smem_u32(sV), MC_PANEL, 1024);
-    const int steps = (n + 15) >> 4;
-    for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_O, tmem + MC_C + t * 8, dv + t * 128, idesc, 1u);
-    umma_commit(&bars->qk_full);                    // its second phase
-  }
-  if (mbar_wait(&bars->qk_full, 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
-    tc_fence_after();
-    const bool live = j < n;
-    const size_t t = static_cast<size_t>(t0) + (live ? j : 0);
-    __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
-    float f = 1.f;
     if constexpr (GATED) {
-      uint32_t r[16];
-      tmem_ld_32x16(to + p.vpad, r);                // the state's part of n . q
-      tmem_ld_wait();
-      nq = nsum[j] + nsum[MC_C + j] + __uint_as_float(r[0]);
-      f = 1.f / (fmaxf(fabsf(nq), expf(-mrow)) + 1e-6f);
-      float ss = 0.f;
+      // the state's part of n . q: this half's 64 key columns
+      if (ok && mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL) && half < p.pk) {
+        float d = 0.f;
+        const int cols = min(64, p.dim - 64 * half);
+#pragma unroll 4
+        for (int i = 0; i < 8; ++i) {
+          if (8 * i >= cols) break;
+          float q[8];
+          ld8(reinterpret_cast<const __nv_bfloat16*>(sQ + half * MC_PANEL + j * 128 + ((i ^ (j & 7)) << 4)), q);
+          const float4 a = *reinterpret_cast<const float4*>(nb + 64 * half + 8 * i), e = *reinterpret_cast<const float4*>(nb + 64 * half + 8 * i + 4);
+          d += q[0] * a.x + q[1] * a.y + q[2] * a.z + q[3] * a.w + q[4] * e.x + q[5] * e.y + q[6] * e.z + q[7] * e.w;
+        }
+        nq += d * einter;
+      }
+      nsum[half * MC_C + j] = nq;
+    }
+    tc_fence_before();
+    named_barrier_sync(1, 256);                       // all scores have been read: the weights may lie over them
+    tc_fence_after();
+    if (ok) {
+#pragma unroll
+      for (int b = 0; b < 2; ++b) tmem_st_32x16(ts + 16 * half + 32 * b, packed[b]);
+      ok = mbar_wait(&bars->o_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    }
+    if (ok) {
+      tc_fence_after();
 #pragma unroll 1
-      for (int c0 = 0; c0 < p.vpad; c0 += 16) {     // padding columns are zero
+      for (int c0 = 32 * half; c0 < p.vpad; c0 += 64) {       // up to 16 unused columns behind the last
+        uint32_t v[32];
+        tmem_ld_32x32(to + c0, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * einter);
+        tmem_st_32x32(to + c0, v);
+      }
+      tmem_st_wait();
+    }
+    tc_fence_before();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&bars->p_ready);
+    if (ok && mbar_wait(&bars->final, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL)) {
+      tc_fence_after();
+      const bool live = j < n;
+      const size_t t = static_cast<size_t>(t0) + (live ? j : 0);
+      __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
+      float f = 1.f;
+      if constexpr (GATED) {
+        f = 1.f / (fmaxf(fabsf(nsum[j] + nsum[MC_C + j]), expf(-mrow)) + 1e-6f);
+        float ss = 0.f;
+#pragma unroll 1
+        for (int c0 = 0; c0 < p.vpad; c0 += 16) {     // padding columns are zero
+          uint32_t v[16];
+          tmem_ld_32x16(to + c0, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const float o = __uint_as_float(v[i]) * f;
+            ss += o * o;
+          }
+        }
+        f /= sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
+      }
+      const __nv_bfloat16* grow = GATED ? p.gate_out + t * p.ld_in + h * p.vdim : nullptr;
+      const float* nw = GATED ? p.norm_w + h * p.vdim : nullptr;
+#pragma unroll 1
+      for (int c0 = 16 * half; c0 < p.vpad; c0 += 32) {
+        float g[2][8];
+        if constexpr (GATED) {                        // requested before the accumulator is read
+#pragma unroll
+          for (int q = 0; q < 2; ++q)
+            if (c0 + 8 * q < p.vdim) ld8(grow + c0 + 8 * q, g[q]);
+        }
         uint32_t v[16];
         tmem_ld_32x16(to + c0, v);
         tmem_ld_wait();
+        if (!live) continue;
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float o = __uint_as_float(v[i]) * f;
-          ss += o * o;
+        for (int q = 0; q < 2; ++q) {
+          if (c0 + 8 * q >= p.vdim) continue;
+          float o[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[8 * q + i]) * f;
+          if constexpr (GATED) {
+            float w[8];
+            ld8(nw + c0 + 8 * q, w);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[i] *= w[i] * __fdividef(1.f, 1.f + __expf(-g[q][i]));
+          }
+          st8(orow + c0 + 8 * q, o);
         }
-      }
-      f /= sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
-    }
-    const __nv_bfloat16* grow = GATED ? p.gate_out + t * p.ld_in + h * p.vdim : nullptr;
-    const float* nw = GATED ? p.norm_w + h * p.vdim : nullptr;
-#pragma unroll 1
-    for (int c0 = 16 * half; c0 < p.vpad; c0 += 32) {
-      float g[2][8];
-      if constexpr (GATED) {                        // requested before the accumulator is read
-#pragma unroll
-        for (int q = 0; q < 2; ++q)
-          if (c0 + 8 * q < p.vdim) ld8(grow + c0 + 8 * q, g[q]);
-      }
-      uint32_t v[16];
-      tmem_ld_32x16(to + c0, v);
-      tmem_ld_wait();
-      if (!live) continue;
-#pragma unroll
-      for (int q = 0; q < 2; ++q) {
-        if (c0 + 8 * q >= p.vdim) continue;
-        float o[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[8 * q + i]) * f;
-        if constexpr (GATED) {
-          float w[8];
-          ld8(nw + c0 + 8 * q, w);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) o[i] *= w[i] * __fdividef(1.f, 1.f + __expf(-g[q][i]));
-        }
-        st8(orow + c0 + 8 * q, o);
       }
     }
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) {
+  if (warp == 8) {
     __syncwarp();
     tc_fence_after();
     tmem_dealloc(tmem, tmem_cols);
@@ -531,7 +579,7 @@ static int make_tmap_planes(CUtensorMap* out, const void* base, uint64_t cols, u
 }
 
 static int mc_smem_state(int pv, bool gated) { return 1024 + 1024 + (4 + pv + (gated ? 1 : 0)) * MC_PANEL; }
-static int mc_smem_out(int pk, int pv, int vrows) { return 2048 + 1024 + (2 * pk + pv) * MC_PANEL + 2 * pk * vrows * 128; }
+static int mc_smem_out(int pk, int pv, int vpad) { return 3072 + 1024 + (pk + (pk > pv ? pk : pv)) * MC_PANEL + pk * vpad * 128; }
 
 }  // namespace b200
 
@@ -542,7 +590,7 @@ static int mc_vrows(int vdim, bool gated) { return ((vdim + 15) & ~15) + (gated 
 B200_API int b200_memory_chunk_supported(int dim, int vdim, int gated) {
   if (dim <= 0 || vdim <= 0 || (dim & 7) || (vdim & 7) || dim > 128 || mc_vrows(vdim, gated) > 256) return 0;
   const int pk = (dim + 63) / 64, pv = (vdim + 63) / 64, limit = 227 * 1024;
-  return mc_smem_state(pv, gated) <= limit && mc_smem_out(pk, pv, mc_vrows(vdim, gated)) <= limit;
+  return mc_smem_state(pv, gated) <= limit && mc_smem_out(pk, pv, (vdim + 15) & ~15) <= limit;
 }
 
 // q, k, v: columns of the packed step's projection rows [T, ld_in] (head h at column h dim / h vdim).  parts: 1 chunk states,
@@ -553,7 +601,7 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   const bool gated = p.gates != nullptr;
   if (!b200_memory_chunk_supported(p.dim, p.vdim, gated) || T <= 0 || n_chunks <= 0 || n_chunks > 65535 || n_seqs <= 0 || n_seqs > 65535 ||
       p.H <= 0 || p.H > 65535 || (p.ld_in & 7) || (p.ld_out & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return -1;
-  if (gated ? (!p.stab || !p.norm_w || !p.gate_bias || ((reinterpret_cast<uintptr_t>(p.gate_out) | reinterpret_cast<uintptr_t>(p.norm_w)) & 15)) : !p.log2_decay) return -1;
+  if (gated ? (!p.stab || !p.n_before || !p.norm_w || !p.gate_bias || ((reinterpret_cast<uintptr_t>(p.gate_out) | reinterpret_cast<uintptr_t>(p.norm_w)) & 15)) : !p.log2_decay) return -1;
   p.dimp = (p.dim + 7) & ~7;
   p.vpad = (p.vdim + 15) & ~15;
   p.vrows = mc_vrows(p.vdim, gated);
@@ -565,20 +613,20 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   if (!rc) rc = make_tmap_planes(&tk, k, p.dim, T, p.H, p.ld_in, p.dim, MC_C);
   if (!rc) rc = make_tmap_planes(&tv, v, p.vdim, T, p.H, p.ld_in, p.vdim, MC_C);
   const uint64_t planes = static_cast<uint64_t>(n_chunks) * p.H;
-  if (!rc) rc = make_tmap_planes(&th, p.s_hi, p.dim, p.vrows, planes, p.dimp, static_cast<uint64_t>(p.vrows) * p.dimp, p.vrows);
-  if (!rc) rc = make_tmap_planes(&tl, p.s_lo, p.dim, p.vrows, planes, p.dimp, static_cast<uint64_t>(p.vrows) * p.dimp, p.vrows);
+  if (!rc) rc = make_tmap_planes(&th, p.s_hi, p.dim, p.vpad, planes, p.dimp, static_cast<uint64_t>(p.vpad) * p.dimp, p.vpad);
+  if (!rc) rc = make_tmap_planes(&tl, p.s_lo, p.dim, p.vpad, planes, p.dimp, static_cast<uint64_t>(p.vpad) * p.dimp, p.vpad);
   if (rc) return rc;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const int sm1 = mc_smem_state(p.pv, gated), sm3 = mc_smem_out(p.pk, p.pv, p.vrows);
+  const int sm1 = mc_smem_state(p.pv, gated), sm3 = mc_smem_out(p.pk, p.pv, p.vpad);
   int cols = 256;
-  while (cols < MC_O + ((p.vrows + 31) & ~31)) cols <<= 1;
+  while (cols < MC_C + ((p.vpad + 31) & ~31)) cols <<= 1;
 #define GO(G)                                                                                                          \
   {                                                                                                                    \
     if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
         cudaFuncSetAttribute(chunk_out_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
     if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 256, sm1, st>>>(tk, tv, p);                              \
     if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 255) / 256, p.H, n_seqs), 256, 0, st>>>(p);      \
-    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 256, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
+    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 288, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
   }
   if (gated) GO(true) else GO(false)
 #undef GO

@@ -22,7 +22,7 @@ class _GqaDecode(C.Structure):
 class _Chunks(C.Structure):
     _fields_ = [(n, _i) for n in ("H", "dim", "vdim", "dimp", "vpad", "vrows", "pk", "pv", "ldv", "ld_in", "ld_out", "gate_t", "gate_h")] + \
                [(n, _f) for n in ("qscale", "cap", "eps")] + \
-               [(n, _vp) for n in ("chunks", "seqs", "log2_decay", "gates", "gate_bias", "u", "stat", "s_hi", "s_lo", "m_before", "m_init", "state",
+               [(n, _vp) for n in ("chunks", "seqs", "log2_decay", "gates", "gate_bias", "u", "stat", "s_hi", "s_lo", "n_before", "m_before", "m_init", "state",
                                    "stab", "gate_out", "norm_w", "out", "err")]
 
 
@@ -121,17 +121,18 @@ def _chunked(step, q, k, v, H: int, dim: int, vdim: int, ldv: int, out, state, q
     """The three launches of a chunked memory, as a callable taking a mask of the parts to run."""
     chunks, seqs = chunk_tables(step)
     n, S, dev, gated = chunks.shape[0], seqs.shape[0], q.device, gates is not None
-    rows = (vdim + 15) // 16 * 16 + (16 if gated else 0)
-    u = torch.empty(n * H, rows, dim, dtype=F32, device=dev)
-    hi, lo = (torch.empty(n * H, rows, dim, dtype=BF16, device=dev) for _ in range(2))
+    vpad = (vdim + 15) // 16 * 16
+    u = torch.empty(n * H, vpad + (16 if gated else 0), dim, dtype=F32, device=dev)
+    hi, lo = (torch.empty(n * H, vpad, dim, dtype=BF16, device=dev) for _ in range(2))
+    nb = torch.empty(n * H, dim, dtype=F32, device=dev) if gated else None
     scal = torch.empty(3 * n * H + S * H, dtype=F32, device=dev)
     stat, m_before, m_init = scal[:2 * n * H], scal[2 * n * H:3 * n * H], scal[3 * n * H:]
     p = K._ptr
     c = _Chunks(H, dim, vdim, 0, 0, 0, 0, 0, ldv, q.stride(0), out.stride(0), 0 if gates is None else gates.stride(0), 0 if gates is None else gates.stride(1),
                 qscale, cap, eps,
                 chunks.data_ptr(), seqs.data_ptr(), p(decay), p(gates), p(gate_bias), u.data_ptr(), stat.data_ptr(), hi.data_ptr(), lo.data_ptr(),
-                m_before.data_ptr(), m_init.data_ptr(), state.data_ptr(), p(stab), p(gate_out), p(norm_w), out.data_ptr(), 0)
-    keep = (u, hi, lo, scal, q, decay, gates, gate_bias, state, stab, gate_out, norm_w)      # alive as long as the callable
+                p(nb), m_before.data_ptr(), m_init.data_ptr(), state.data_ptr(), p(stab), p(gate_out), p(norm_w), out.data_ptr(), 0)
+    keep = (u, hi, lo, nb, scal, q, decay, gates, gate_bias, state, stab, gate_out, norm_w)      # alive as long as the callable
 
     def run(parts: int = 7):
         assert keep
