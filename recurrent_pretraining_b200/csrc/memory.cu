@@ -527,39 +527,53 @@ memory_merge_kernel(const TI* __restrict__ in, const TM* __restrict__ mem, T* __
   }
 }
 
-// The memory half alone, for prompts: a warp per token.  W = HR * rvdim, a multiple of four up to 128 * G.
-template <typename TI, typename TM, typename T, int G>
-__global__ void __launch_bounds__(256)
-memory_norm_rows_kernel(const TI* __restrict__ in, const TM* __restrict__ mem, T* __restrict__ out, const MergeArgs A, int rows) {
-  const size_t t = static_cast<size_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+// The memory half alone, for prompts (bf16): a warp per token, all of a row's pieces requested at once.  W = HR * rvdim, a
+// multiple of eight up to 256 * G.
+template <int G>
+__global__ void __launch_bounds__(128)
+memory_norm_rows_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ mem, __nv_bfloat16* __restrict__ out,
+                        const MergeArgs A, int rows) {
+  const size_t t = static_cast<size_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
   if (t >= rows) return;
   const int lane = threadIdx.x & 31, W = A.HR * A.rvdim;
-  const TM* m = mem + t * A.ld_mem;
-  const TI* g = in + t * A.ld_in + A.off_rg;
-  T* o = out + t * A.ld_out + A.off_r;
-  float v[G][4];
+  const __nv_bfloat16* m = mem + t * A.ld_mem;
+  const __nv_bfloat16* g = in + t * A.ld_in + A.off_rg;
+  __nv_bfloat16* o = out + t * A.ld_out + A.off_r;
+  uint4 v[G], q[G];
+#pragma unroll
+  for (int k = 0; k < G; ++k) {
+    const int i = 8 * (lane + 32 * k);
+    v[k] = make_uint4(0u, 0u, 0u, 0u);
+    if (i < W) {
+      v[k] = *reinterpret_cast<const uint4*>(m + i);
+      q[k] = *reinterpret_cast<const uint4*>(g + i);
+    }
+  }
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < G; ++k) {
-    const int i = 4 * (lane + 32 * k);
-    if (i < W) {
-      ld4(m + i, v[k]);
+    const uint32_t w[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
 #pragma unroll
-      for (int j = 0; j < 4; ++j) ss += v[k][j] * v[k][j];
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(w[j]);
+      ss += f.x * f.x + f.y * f.y;
     }
   }
   const float rms = A.right_scale / sqrtf(warp_sum(ss) / static_cast<float>(W) + A.eps);
 #pragma unroll
   for (int k = 0; k < G; ++k) {
-    const int i = 4 * (lane + 32 * k);
+    const int i = 8 * (lane + 32 * k);
     if (i < W) {
-      float gv[4], wv[4];
-      ld4(g + i, gv);
-      ld4(A.norm_w + i, wv);
+      const uint32_t vw[4] = {v[k].x, v[k].y, v[k].z, v[k].w}, gw[4] = {q[k].x, q[k].y, q[k].z, q[k].w};
+      float wv[8], r[8];
+      ld8(A.norm_w + i, wv);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[k][j] *= rms * wv[j] * __fdividef(1.f, 1.f + __expf(-gv[j]));
-      st2(o + i, make_float2(v[k][0], v[k][1]));
-      st2(o + i + 2, make_float2(v[k][2], v[k][3]));
+      for (int j = 0; j < 4; ++j) {
+        const float2 x = unpack_bf16x2(vw[j]), z = unpack_bf16x2(gw[j]);
+        r[2 * j] = x.x * rms * wv[2 * j] * __fdividef(1.f, 1.f + __expf(-z.x));
+        r[2 * j + 1] = x.y * rms * wv[2 * j + 1] * __fdividef(1.f, 1.f + __expf(-z.y));
+      }
+      st8(o + i, r);
     }
   }
 }
@@ -672,12 +686,11 @@ B200_API int b200_memory_merge(const void* in, const void* mem, void* out, const
   if (T <= 0 || A.HR <= 0 || A.rvdim <= 0 || (A.H && (!A.part_o || !A.part_ml || A.splits < 1 || A.splits > 32)) || (f32 && (!in_f32 || !mem_f32))) return -1;
   if (((A.ld_mem | A.ld_in | A.ld_out | A.off_r | A.off_rg) & 7) || ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(mem) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
   const int W = A.HR * A.rvdim;
-  if (!f32 && !in_f32 && !mem_f32 && A.H == 0 && T >= 256 && (W & 3) == 0 && W <= 32 * 128) {
-#define GO(G) memory_norm_rows_kernel<bf16_t, bf16_t, bf16_t, G><<<(T + 7) / 8, 256, 0, STREAM>>>((const bf16_t*)in, (const bf16_t*)mem, (bf16_t*)out, A, T)
-    if (W <= 8 * 128) GO(8);
-    else if (W <= 16 * 128) GO(16);
-    else if (W <= 24 * 128) GO(24);
-    else GO(32);
+  if (!f32 && !in_f32 && !mem_f32 && A.H == 0 && T >= 256 && (W & 7) == 0 && W <= 16 * 256 && !(reinterpret_cast<uintptr_t>(A.norm_w) & 15)) {
+#define GO(G) memory_norm_rows_kernel<G><<<(T + 3) / 4, 128, 0, STREAM>>>((const bf16_t*)in, (const bf16_t*)mem, (bf16_t*)out, A, T)
+    if (W <= 4 * 256) GO(4);
+    else if (W <= 9 * 256) GO(9);
+    else GO(16);
 #undef GO
     return DONE;
   }

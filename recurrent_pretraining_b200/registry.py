@@ -227,7 +227,7 @@ layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _gasovik("gasovik-1b", 65536, 2048, 16, 16, 128, 64, 128, 512, 1024, 8192, share_from=12),
     # layers of the width and depth of the 3.5B recurrent flagship's core, for side-by-side timing
     _gasovik("gasovik-core-5280", 65536, 5280, 4, 55, 96, 32, 96, 512, 4096, 17920),
-    _fatudra("fatudra-tiny", 512, 128, 4, (4, 2, 32, 32), (2, 32, 32), (2, 16, 32), 256, loop=(1, 3, 2), bias_rows=8, bias_max=64),
+    _fatudra("fatudra-tiny", 512, 128, 4, (4, 2, 32, 32), (2, 32, 32), (2, 16, 32), 192, loop=(1, 3, 2), bias_rows=8, bias_max=64),
     _fatudra("fatudra-1b", 65536, 2048, 16, (16, 4, 128, 128), (8, 128, 128), (8, 64, 128), 4608),
     _fatudra("fatudra-core-5280", 65536, 5280, 4, (55, 11, 96, 96), (22, 96, 96), (22, 96, 192), 14080),
 )}
