@@ -257,7 +257,7 @@ struct MemoryArgs {
 // CTA per (head, sequence): warps over the key rows, float4 groups of value columns over the lanes.  Fixed decay: out32 gets
 // S^T q.  Gated: the head's output is normalised, RMS-normed, gated and stored in `out`.
 template <typename TI, typename T, bool GATED>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 memory_scan_kernel(const TI* __restrict__ in, const T* __restrict__ hin, const T* __restrict__ w_gate, T* __restrict__ out, const MemoryArgs M) {
   pdl_trigger();
   pdl_wait();

@@ -213,13 +213,13 @@ chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 // ------------------------------------------------------------------------------------------------ recurrence over chunks
 // A thread carries four key columns of one value row through the chunks of a sequence.
 template <bool GATED>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128)
 chunk_scan_kernel(const ChunkParams p) {
   const int h = blockIdx.y;
   const int4 sq = p.seqs[blockIdx.z];
   const int c0 = sq.x, nc = sq.y, row = sq.z;
   const bool fresh = sq.w == 0;
-  const int per = p.dimp >> 2, e = blockIdx.x * 256 + threadIdx.x;
+  const int per = p.dimp >> 2, e = blockIdx.x * 128 + threadIdx.x;
   if (e >= per * p.vrows) return;
   const int v = e / per, d = 4 * (e - v * per);
   float* st = p.state + (static_cast<size_t>(row) * p.H + h) * p.dim * p.ldv;
@@ -625,7 +625,7 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
     if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
         cudaFuncSetAttribute(chunk_out_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
     if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 256, sm1, st>>>(tk, tv, p);                              \
-    if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 255) / 256, p.H, n_seqs), 256, 0, st>>>(p);      \
+    if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 127) / 128, p.H, n_seqs), 128, 0, st>>>(p);      \
     if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 288, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
   }
   if (gated) GO(true) else GO(false)
