@@ -75,21 +75,6 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   uint8_t* sq = smem;                                                  // [16][kp]
   uint8_t* ring = sq + 16 * kp + warp * STAGES * stage_bytes;
   const TI* r = in + static_cast<size_t>(b) * P.ld_in;
-  // queries, zero in the padding rows and columns; the ring's padding columns are zeroed once
-  for (int i = threadIdx.x; i < 16 * (kp / 2); i += 128) {
-    const int hh = i / (kp / 2), c = i - hh * (kp / 2);
-    float v = 0.f;
-    if (hh < nh && c < P.dim) v = ldf(r + (h0 + hh) * P.dim + c) + P.in_bias[(h0 + hh) * P.dim + c];
-    reinterpret_cast<__nv_bfloat16*>(sq)[i] = f2bf(v);
-  }
-  for (int i = lane; i < STAGES * GD_KEYS; i += 32) {
-    uint8_t* s = ring + (i / GD_KEYS) * stage_bytes;
-    __nv_bfloat16* kr = reinterpret_cast<__nv_bfloat16*>(s + (i % GD_KEYS) * kp);
-    __nv_bfloat16* vr = reinterpret_cast<__nv_bfloat16*>(s + GD_KEYS * kp + (i % GD_KEYS) * vp);
-    for (int c = P.dim; c < kp / 2; ++c) kr[c] = f2bf(0.f);
-    for (int c = P.vdim; c < vp / 2; ++c) vr[c] = f2bf(0.f);
-  }
-  __syncthreads();
   __nv_bfloat16* base = P.cache + static_cast<size_t>(P.row[b]) * P.cap * P.ld_kv;
   // 16-byte pieces of a key row and a value row: a power of two of lanes per key, or several passes of 32
   const int kch = P.dim >> 3, ch = kch + (P.vdim >> 3);
@@ -116,6 +101,21 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     if (s < mine) request(first + s * GD_WARPS, s);
     cp_commit();
   }
+  // queries, zero in the padding rows and columns; the ring's padding columns are zeroed once
+  for (int i = threadIdx.x; i < 16 * (kp / 2); i += 128) {
+    const int hh = i / (kp / 2), c = i - hh * (kp / 2);
+    float v = 0.f;
+    if (hh < nh && c < P.dim) v = ldf(r + (h0 + hh) * P.dim + c) + P.in_bias[(h0 + hh) * P.dim + c];
+    reinterpret_cast<__nv_bfloat16*>(sq)[i] = f2bf(v);
+  }
+  for (int i = lane; i < STAGES * GD_KEYS; i += 32) {
+    uint8_t* s = ring + (i / GD_KEYS) * stage_bytes;
+    __nv_bfloat16* kr = reinterpret_cast<__nv_bfloat16*>(s + (i % GD_KEYS) * kp);
+    __nv_bfloat16* vr = reinterpret_cast<__nv_bfloat16*>(s + GD_KEYS * kp + (i % GD_KEYS) * vp);
+    for (int c = P.dim; c < kp / 2; ++c) kr[c] = f2bf(0.f);
+    for (int c = P.vdim; c < vp / 2; ++c) vr[c] = f2bf(0.f);
+  }
+  __syncthreads();
   // rows of this thread's accumulators: heads lane / 4 and lane / 4 + 8
   const int ra = lane >> 2;
   float rowmul = P.scale * 1.4426950408889634f;
