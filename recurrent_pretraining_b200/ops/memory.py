@@ -371,7 +371,10 @@ def parallel_decode(L: ParallelLayout, spec, inp: torch.Tensor, bias: torch.Tens
     po = torch.empty(B, L.heads, splits, pad8(L.vdim), dtype=F32, device=inp.device)
     ml = torch.empty(B, L.heads, splits, 2, dtype=F32, device=inp.device)
     attend, scan, merge = parallel_decode_pieces(L, spec, inp, bias, cache, state, table, decay, norm_w, eps, pos, row, po, ml, out)
-    if torch.cuda.is_current_stream_capturing():           # the two halves are independent branches of the graph
+    from ..engine.base import PDL
+
+    # the two halves are independent branches of a graph, unless programmatic launch ties every kernel to its one predecessor
+    if torch.cuda.is_current_stream_capturing() and not PDL:
         main, side = torch.cuda.current_stream(), _side_stream(inp.device)
         side.wait_stream(main)
         with torch.cuda.stream(side):
