@@ -53,6 +53,9 @@ struct GemmParams {
   int act;             // 0: none, 1: relu^2, 2: silu on the columns [act_lo, act_hi) (multiples of eight)
                        // OUT_SWIGLU: 0: silu gate, 3: tanh-gelu gate
   int act_lo, act_hi;
+  // grouped product: row tile i of the first *n_row_tiles is multiplied with rows [tile_group[i] N, (tile_group[i] + 1) N) of B
+  const int* tile_group;
+  const int* n_row_tiles;
 };
 
 // Linear tile index -> (m tile, n tile), grouped: GROUP consecutive m tiles are walked across all n tiles before the

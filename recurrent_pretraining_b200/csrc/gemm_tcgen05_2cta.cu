@@ -124,7 +124,7 @@ struct Smem2 {
   static constexpr int TOTAL_F32 = TOTAL + C_STAGE_BYTES;
 };
 
-template <int BN, bool A_MN, bool B_MN, int MODE, bool AG = false>
+template <int BN, bool A_MN, bool B_MN, int MODE, bool AG = false, bool GROUPED = false>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(AG ? 320 : 192, 1)
 gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA2,
              const __grid_constant__ CUtensorMap tmB, const GemmParams p, const __grid_constant__ AgParams ag,
@@ -158,7 +158,7 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
   const int cluster_id = blockIdx.x >> 1;
   const int num_clusters = gridDim.x >> 1;
 
-  const int tiles_m = (p.M + 2 * BM2 - 1) / (2 * BM2);
+  const int tiles_m = GROUPED ? min(*p.n_row_tiles, (p.M + 2 * BM2 - 1) / (2 * BM2)) : (p.M + 2 * BM2 - 1) / (2 * BM2);
   const int tiles_n = (p.N + BN_OUT - 1) / BN_OUT;
   const int num_tiles = tiles_m * tiles_n;
   const int nk1 = (p.K1 + BK2 - 1) / BK2;
@@ -216,7 +216,7 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
         tile_mn(tile, mt, nt);
         const int m0 = mt * (2 * BM2) + static_cast<int>(rank) * BM2;
         const int n0 = is_swiglu(MODE) ? nt * BN_OUT + static_cast<int>(rank) * p.swiglu_n
-                                            : nt * BN + static_cast<int>(rank) * BNH;
+                                            : nt * BN + static_cast<int>(rank) * BNH + (GROUPED ? p.tile_group[mt] * p.N : 0);
         if constexpr (AG) {
           // the weight rows of this N-tile must have landed in the local buffer (every CTA's copiers add one)
           const unsigned long long t0 = globaltimer_ns();
@@ -399,12 +399,12 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
   }
 }
 
-template <int BN, bool A_MN, bool B_MN, int MODE, bool AG = false>
+template <int BN, bool A_MN, bool B_MN, int MODE, bool AG = false, bool GROUPED = false>
 static int launch2(const CUtensorMap& ta, const CUtensorMap& ta2, const CUtensorMap& tb, const GemmParams& p,
                    cudaStream_t stream, int max_ctas, const AgParams* agp = nullptr, const CUtensorMap* tcp = nullptr,
                    const CUtensorMap* tcp2 = nullptr, const CUtensorMap* tcp3 = nullptr) {
   using L = Smem2<BN>;
-  auto kern = gemm2_kernel<BN, A_MN, B_MN, MODE, AG>;
+  auto kern = gemm2_kernel<BN, A_MN, B_MN, MODE, AG, GROUPED>;
   constexpr int SMEM = ((MODE == OUT_F32 || MODE == OUT_F32_ACC || MODE == OUT_BF16 || MODE == OUT_BF16_ROPE ||
                          MODE == OUT_BF16_BIAS_ACT || MODE == OUT_SWIGLU || MODE == OUT_SWIGLU_SAVE || MODE == OUT_DSWIGLU) && !AG)
                             ? L::TOTAL_F32 : L::TOTAL;
@@ -536,6 +536,17 @@ int gemm_2cta_dispatch(const void* A, const void* A2, const void* B, const GemmP
   }
 #undef DISPATCH2
   return -100;
+}
+
+// Entry used by b200_gemm_grouped: 256-row tiles.
+int gemm_2cta_grouped(const void* A, const void* B, const GemmParams& p, int lda, int ldb, int groups, cudaStream_t st) {
+  CUtensorMap ta, tb, tc;
+  int rc = make_tmap_2d_bf16(&ta, A, p.M, p.K1, lda, BM2, BK2);
+  if (!rc) rc = make_tmap_2d_bf16(&tb, B, static_cast<uint64_t>(groups) * p.N, p.K1, ldb, 128, BK2);
+  if (rc) return rc;
+  GemmParams pc = p;
+  pc.tma_c = make_tmap_2d_bf16(&tc, p.C, p.M, p.N, p.ldc, 32, 64) == 0;
+  return launch2<256, false, false, OUT_BF16_BIAS_ACT, false, true>(ta, ta, tb, pc, st, 0, nullptr, pc.tma_c ? &tc : nullptr);
 }
 
 }  // namespace b200

@@ -259,8 +259,11 @@ struct WindowAttn {
   // query temperature (0: none): scores are multiplied by 1 + coef * ln(floor((position + 1) / every) + 1)
   int temp_every;
   float temp_coef;
-  int head_gate;                  // stream form: one gate per head (gate row [H]) instead of one per output
+  int head_gate;                  // stream form: one gate per head (gate row [H]) instead of one per output; no gate array: none
   float gate_mult;                // factor on the gated output
+  float softcap;                  // 0: none; otherwise score = softcap * tanh(score / softcap)
+  int chunk;                      // ring form, not 0: the query sees its chunk of that many positions instead of a window
+  const float* sink;              // [H] stream form, null: none; exp(sink) is one more term of the softmax's denominator
 };
 
 // CTA of four warps per (token, head, key split); a warp takes 32 keys at a time: one key per lane for the scores, one
@@ -283,7 +286,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   __syncthreads();
   const bool ring = A.pos != nullptr;
   const int last = ring ? A.pos[t] : A.sidx[t];
-  const int first = max(ring ? 0 : A.kbase[t], last - A.window + 1);
+  const int first = ring && A.chunk ? last - last % A.chunk : max(ring ? 0 : A.kbase[t], last - A.window + 1);
   const size_t ring0 = ring ? static_cast<size_t>(A.row[t]) * A.cap : 0;
   const int nchunk = (last - first) / 32 + 1;
   const int hk = h / A.group;
@@ -307,6 +310,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
       }
       s *= scale;
       if (bias) s += bias[min(last - j, A.bias_len - 1)];
+      if (A.softcap > 0.f) s = A.softcap * tanhf(s / A.softcap);
     }
     const float mn = fmaxf(m, warp_max(s));
     const float p = expf(s - mn), alpha = expf(m - mn);
@@ -329,6 +333,11 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   float mm = -INFINITY, ll = 0.f, wgt[4];
 #pragma unroll
   for (int w = 0; w < 4; ++w) mm = fmaxf(mm, ml[2 * w]);
+  const float sink = A.sink ? A.sink[h] : -INFINITY;
+  if (A.sink) {                                     // stream form: some key is visible
+    mm = fmaxf(mm, sink);
+    ll = expf(sink - mm);
+  }
 #pragma unroll
   for (int w = 0; w < 4; ++w) {
     wgt[w] = ml[2 * w] == -INFINITY ? 0.f : expf(ml[2 * w] - mm);
@@ -344,7 +353,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
       A.part_o[pi * ((A.vdim + 7) & ~7) + d] = o;
       if (d == 0) { A.part_ml[2 * pi] = mm; A.part_ml[2 * pi + 1] = ll; }
     } else {
-      const float g = sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + (A.head_gate ? h : h * A.vdim + d)));
+      const float g = gate ? sigmoid_f(ldf(gate + static_cast<size_t>(t) * A.gate_ld + (A.head_gate ? h : h * A.vdim + d))) : 1.f;
       stf(out + static_cast<size_t>(t) * A.out_ld + h * A.vdim + d, o * inv * (g * A.gate_mult));
     }
   }
@@ -544,11 +553,11 @@ rms_residual_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __rest
   }
 }
 
-// y[i] = rmsnorm(x[idx[i]]) * w in operand precision
+// y[i] = mult * rmsnorm(x[idx[i]]) * (w + w_add) in operand precision
 template <typename T>
 __global__ void __launch_bounds__(256)
 rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ idx, const float* __restrict__ w, T* __restrict__ y,
-                    int ld_y, int E, float eps) {
+                    int ld_y, int E, float eps, float w_add, float mult) {
   pdl_trigger();
   pdl_wait();
   __shared__ float red[8];
@@ -556,7 +565,7 @@ rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ idx, co
   float ss = 0.f;
   for (int i = threadIdx.x; i < E; i += 256) ss += xr[i] * xr[i];
   const float r = 1.f / sqrtf(block_total<256>(ss, red) / static_cast<float>(E) + eps);
-  for (int i = threadIdx.x; i < E; i += 256) stf(y + static_cast<size_t>(blockIdx.x) * ld_y + i, xr[i] * r * w[i]);
+  for (int i = threadIdx.x; i < E; i += 256) stf(y + static_cast<size_t>(blockIdx.x) * ld_y + i, xr[i] * r * (w[i] + w_add) * mult);
 }
 
 // y = act(a + bias); act 0: none, 1: relu^2.  `clear` as above.
@@ -578,11 +587,17 @@ bias_act_kernel(TI* __restrict__ a, int ld_a, int clear, const float* __restrict
 }
 
 // ------------------------------------------------------------------------------------------------ fp32 matrix product
-// C[M, N] = act(A[M, K] B[N, K]^T + bias) in fp32 (FMA pipe): 64 x 64 tile per 256 threads, 4 x 4 per thread.
+// C[M, N] = act(A[M, K] B[N, K]^T + bias) in fp32 (FMA pipe): 64 x 64 tile per 256 threads, 4 x 4 per thread.  Grouped: tile i of the
+// first *n_tiles row tiles is multiplied with rows [group[i] N, (group[i] + 1) N) of B.
 constexpr int SG = 64, SGK = 16;
 __global__ void __launch_bounds__(256)
 sgemm_nt_kernel(const float* __restrict__ A, const float* __restrict__ B, const float* __restrict__ bias, float* __restrict__ C,
-                int M, int N, int K, int lda, int ldb, int ldc, int act, int act_lo, int act_hi) {
+                int M, int N, int K, int lda, int ldb, int ldc, int act, int act_lo, int act_hi, const int* __restrict__ group,
+                const int* __restrict__ n_tiles) {
+  if (group) {
+    if (static_cast<int>(blockIdx.x) >= *n_tiles) return;
+    B += static_cast<size_t>(group[blockIdx.x]) * N * ldb;
+  }
   __shared__ float as[SGK][SG + 4], bs[SGK][SG + 4];
   const int m0 = blockIdx.x * SG, n0 = blockIdx.y * SG;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -689,8 +704,9 @@ B200_API int b200_window_attention(const void* q, const void* k1, const void* k2
                                    const WindowAttn* Ap, int T, int f32, void* stream) {
   const WindowAttn A = *Ap;
   if (T <= 0 || A.H <= 0 || A.H > 65535 || A.group <= 0 || A.H % A.group || (A.bias && A.bias_len <= 0) || A.d1 <= 0 || A.d2 < 0 || A.vdim <= 0 || A.window <= 0 || A.splits < 1 || A.splits > 32) return -1;
-  if (A.pos ? (!A.row || A.cap <= 0 || A.cap < A.window || !A.part_o || !A.part_ml) : (!A.sidx || !A.kbase || A.splits != 1 || A.part_o || !gate || !out))
+  if (A.pos ? (!A.row || A.cap <= 0 || A.cap < A.window || !A.part_o || !A.part_ml || A.sink) : (!A.sidx || !A.kbase || A.splits != 1 || A.part_o || A.chunk || !out))
     return -1;
+  if (A.softcap < 0.f || A.chunk < 0) return -1;
   const size_t smem = (A.d1 + A.d2 + 128 + 4 * A.vdim + 8) * sizeof(float);
   if (smem > 200 * 1024) return -1;
   const dim3 grid(T, A.H, A.splits);
@@ -762,11 +778,11 @@ B200_API int b200_rms_residual(void* a, int ld_a, int in_f32, int clear, const f
   return DONE;
 }
 
-B200_API int b200_rmsnorm_rows(const float* x, const int* idx, const float* w, void* y, int ld_y, int rows, int E, float eps, int f32,
-                               void* stream) {
+B200_API int b200_rmsnorm_rows(const float* x, const int* idx, const float* w, void* y, int ld_y, int rows, int E, float eps, float w_add,
+                               float mult, int f32, void* stream) {
   if (rows <= 0) return 0;
-  if (f32) launch_k(rmsnorm_rows_kernel<float>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (float*)y, ld_y, E, eps);
-  else launch_k(rmsnorm_rows_kernel<bf16_t>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (bf16_t*)y, ld_y, E, eps);
+  if (f32) launch_k(rmsnorm_rows_kernel<float>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (float*)y, ld_y, E, eps, w_add, mult);
+  else launch_k(rmsnorm_rows_kernel<bf16_t>, dim3(rows), dim3(256), 0, STREAM, x, idx, w, (bf16_t*)y, ld_y, E, eps, w_add, mult);
   return DONE;
 }
 
@@ -780,9 +796,12 @@ B200_API int b200_bias_act(void* a, int ld_a, int in_f32, int clear, const float
   return DONE;
 }
 
+B200_API int b200_sgemm_tile_rows() { return SG; }
+
 B200_API int b200_sgemm_nt(const float* A, const float* B, const float* bias, float* C, int M, int N, int K, int lda, int ldb, int ldc,
-                           int act, int act_lo, int act_hi, void* stream) {
-  if (M <= 0 || N <= 0 || K <= 0 || (N + SG - 1) / SG > 65535) return -1;
-  sgemm_nt_kernel<<<dim3((M + SG - 1) / SG, (N + SG - 1) / SG), 256, 0, STREAM>>>(A, B, bias, C, M, N, K, lda, ldb, ldc, act, act_lo, act_hi);
+                           int act, int act_lo, int act_hi, const int* group, const int* n_tiles, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || (N + SG - 1) / SG > 65535 || !group != !n_tiles) return -1;
+  sgemm_nt_kernel<<<dim3((M + SG - 1) / SG, (N + SG - 1) / SG), 256, 0, STREAM>>>(A, B, bias, C, M, N, K, lda, ldb, ldc, act, act_lo, act_hi,
+                                                                                                    group, n_tiles);
   return DONE;
 }

@@ -1,8 +1,8 @@
 // Kernels of the layered decoder models that mix attention with recurrent memories, other than the tensor-core ones:
-//   * sandwich_norm     : x += layernorm(a + bias) [+ step vector] on the fp32 residual stream, then the layernorm that feeds
-//                         the next sublayer
+//   * sandwich_norm     : x += norm(a + bias) [+ step vector] on the fp32 residual stream, then the norm that feeds the next
+//                         sublayer; layer norms, or RMS norms whose weights are stored around zero
 //   * layernorm_rows    : gathered rows of the final norm
-//   * glu               : act(gate) * up of a [gate | up] row
+//   * glu               : act(gate) * up of a [gate | up] row, tanh-GELU or silu
 //   * kv_append         : keys and values of a step into the cache
 //   * memory_scan       : token-by-token recurrence of a matrix memory per (sequence, head): decode steps (one pass over the
 //                         state) and any prompt (state in shared memory); fixed decay, or exponential gates with normaliser
@@ -17,7 +17,7 @@ namespace b200 {
 // ------------------------------------------------------------------------------------------------ layer norms
 struct SandwichArgs {
   int E, ld_a, ld_h, clear, nzero;
-  float eps, bias_mult;
+  float eps, bias_mult, out_mult; // out_mult: factor on the next sublayer's input
   const float* bias;              // on the sublayer output, times bias_mult; null: none
   const float *w1, *b1;           // norm of the sublayer output
   const float* step;              // added to the stream afterwards; null: none
@@ -27,14 +27,17 @@ struct SandwichArgs {
 };
 
 // One CTA per row; NV groups of eight columns per thread held in registers.  A null `a` skips the sublayer output.
-template <typename TI, typename T, int NV>
+// RMS: no means are taken, weights are one plus the stored ones and there are no biases.
+template <typename TI, typename T, int NV, bool RMS>
 __global__ void __launch_bounds__(256)
 sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   pdl_trigger();
   if (gridDim.x <= 256) {                          // few rows: the weights' way from memory would add to the reductions'
     for (int i = 32 * threadIdx.x; i < A.E; i += 8192) {
-      if (a) { prefetch_l2(A.w1 + i); prefetch_l2(A.b1 + i); }
-      if (A.w2) { prefetch_l2(A.w2 + i); prefetch_l2(A.b2 + i); }
+      if (a) prefetch_l2(A.w1 + i);
+      if (A.w2) prefetch_l2(A.w2 + i);
+      if (!RMS && a) prefetch_l2(A.b1 + i);
+      if (!RMS && A.w2) prefetch_l2(A.b2 + i);
     }
   }
   pdl_wait();
@@ -66,7 +69,7 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
   }
   for (int i = threadIdx.x; i < A.nzero; i += 256) A.zero[row * A.nzero + i] = 0.f;
   if (ar) {
-    const float mean = block_total<256>(sum, red) * invE;
+    const float mean = RMS ? 0.f : block_total<256>(sum, red) * invE;
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k)
@@ -83,9 +86,9 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
       if (i < nvec) {
         float wv[8], bv[8];
         ld8(A.w1 + 8 * i, wv);
-        ld8(A.b1 + 8 * i, bv);
+        if (!RMS) ld8(A.b1 + 8 * i, bv);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) xv[k][j] += s[k][j] * r * wv[j] + bv[j];
+        for (int j = 0; j < 8; ++j) xv[k][j] += RMS ? s[k][j] * r * (1.f + wv[j]) : s[k][j] * r * wv[j] + bv[j];
       }
     }
   }
@@ -106,7 +109,7 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
     }
   }
   if (!A.w2) return;
-  const float mean = block_total<256>(sum, red) * invE;
+  const float mean = RMS ? 0.f : block_total<256>(sum, red) * invE;
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < NV; ++k)
@@ -123,16 +126,16 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
     if (i < nvec) {
       float wv[8], bv[8];
       ld8(A.w2 + 8 * i, wv);
-      ld8(A.b2 + 8 * i, bv);
+      if (!RMS) ld8(A.b2 + 8 * i, bv);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) xv[k][j] = xv[k][j] * r * wv[j] + bv[j];
+      for (int j = 0; j < 8; ++j) xv[k][j] = (RMS ? xv[k][j] * r * (1.f + wv[j]) : xv[k][j] * r * wv[j] + bv[j]) * A.out_mult;
       st8(h + row * A.ld_h + 8 * i, xv[k]);
     }
   }
 }
 
 // Any width: several passes over the row.
-template <typename TI, typename T>
+template <typename TI, typename T, bool RMS>
 __global__ void __launch_bounds__(256)
 sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   pdl_trigger();
@@ -148,7 +151,7 @@ sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   if (ar) {
     float sum = 0.f, ss = 0.f;
     for (int i = threadIdx.x; i < A.E; i += 256) sum += in(i);
-    mean = block_total<256>(sum, red) * invE;
+    mean = RMS ? 0.f : block_total<256>(sum, red) * invE;
     for (int i = threadIdx.x; i < A.E; i += 256) {
       const float d = in(i) - mean;
       ss += d * d;
@@ -159,7 +162,7 @@ sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   for (int i = threadIdx.x; i < A.E; i += 256) {
     float v = x[i];
     if (ar) {
-      v += (in(i) - mean) * r * A.w1[i] + A.b1[i];
+      v += RMS ? in(i) * r * (1.f + A.w1[i]) : (in(i) - mean) * r * A.w1[i] + A.b1[i];
       if (A.clear) stf(ar + i, 0.f);
     }
     if (A.step) v += A.step[i];
@@ -167,13 +170,14 @@ sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
     sum += v;
   }
   if (!A.w2) return;
-  mean = block_total<256>(sum, red) * invE;
+  mean = RMS ? 0.f : block_total<256>(sum, red) * invE;
   for (int i = threadIdx.x; i < A.E; i += 256) {
     const float d = x[i] - mean;
     ss += d * d;
   }
   r = 1.f / sqrtf(block_total<256>(ss, red) * invE + A.eps);
-  for (int i = threadIdx.x; i < A.E; i += 256) stf(h + row * A.ld_h + i, (x[i] - mean) * r * A.w2[i] + A.b2[i]);
+  for (int i = threadIdx.x; i < A.E; i += 256)
+    stf(h + row * A.ld_h + i, (RMS ? x[i] * r * (1.f + A.w2[i]) : (x[i] - mean) * r * A.w2[i] + A.b2[i]) * A.out_mult);
 }
 
 template <typename T>
@@ -194,10 +198,10 @@ layernorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ idx, 
 }
 
 // ------------------------------------------------------------------------------------------------ gated feed-forward
-// y = gelu(gate) * up (tanh form) of rows [gate (N) | up (N)]
-template <typename TI, typename T>
+// y = act(gate) * up of rows [gate (N) | up (N)]; act: gelu (tanh form) or silu
+template <typename TI, typename T, bool SILU>
 __global__ void __launch_bounds__(256)
-geglu_kernel(TI* __restrict__ a, int ld_a, int clear, T* __restrict__ y, int ld_y, int N) {
+glu_kernel(TI* __restrict__ a, int ld_a, int clear, T* __restrict__ y, int ld_y, int N) {
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.y;
@@ -209,7 +213,7 @@ geglu_kernel(TI* __restrict__ a, int ld_a, int clear, T* __restrict__ y, int ld_
     stf(p, 0.f);
     stf(p + N, 0.f);
   }
-  stf(y + row * ld_y + i, 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u);
+  stf(y + row * ld_y + i, (SILU ? silu_f(g) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)))) * u);
 }
 
 // ------------------------------------------------------------------------------------------------ keys and values
@@ -587,29 +591,35 @@ typedef __nv_bfloat16 bf16_t;
 
 // Every `f32` argument: the operand storage type is fp32 instead of bf16; `in_f32`: the GEMM output is fp32.
 
-template <typename TI, typename T>
+template <typename TI, typename T, bool RMS>
 static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, cudaStream_t st) {
   const bool vec = A.E % 8 == 0 && A.ld_a % 8 == 0 && A.ld_h % 8 == 0 &&
                    !((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(A.x) |
                       reinterpret_cast<uintptr_t>(A.w1) | reinterpret_cast<uintptr_t>(A.b1) | reinterpret_cast<uintptr_t>(A.w2) |
                       reinterpret_cast<uintptr_t>(A.b2) | reinterpret_cast<uintptr_t>(A.bias) | reinterpret_cast<uintptr_t>(A.step)) & 15);
   const int nv = vec ? (A.E / 8 + 255) / 256 : 0;
-#define GO(NV) launch_k(sandwich_vec_kernel<TI, T, NV>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A)
+#define GO(NV) launch_k(sandwich_vec_kernel<TI, T, NV, RMS>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A)
   if (nv == 1) GO(1);
   else if (nv == 2) GO(2);
   else if (nv == 3) GO(3);
   else if (nv == 4) GO(4);
-  else launch_k(sandwich_kernel<TI, T>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A);
+  else launch_k(sandwich_kernel<TI, T, RMS>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A);
 #undef GO
 }
 
-B200_API int b200_sandwich_norm(void* a, void* h, const SandwichArgs* Ap, int rows, int in_f32, int f32, void* stream) {
+// rms: RMS norms, weights stored around zero, no biases
+B200_API int b200_sandwich_norm(void* a, void* h, const SandwichArgs* Ap, int rows, int in_f32, int f32, int rms, void* stream) {
   const SandwichArgs A = *Ap;
   if (rows <= 0 || A.E <= 0 || !A.x || (A.clear && !in_f32) || (f32 && !in_f32) || (A.nzero && !A.zero)) return -1;
-  if ((a && (!A.w1 || !A.b1)) || (A.w2 && (!A.b2 || !h))) return -1;
-  if (f32) launch_sandwich<float, float>(a, h, A, rows, STREAM);
-  else if (in_f32) launch_sandwich<float, bf16_t>(a, h, A, rows, STREAM);
-  else launch_sandwich<bf16_t, bf16_t>(a, h, A, rows, STREAM);
+  if ((a && (!A.w1 || (!rms && !A.b1))) || (A.w2 && ((!rms && !A.b2) || !h))) return -1;
+#define GO(RMS)                                                                \
+  {                                                                            \
+    if (f32) launch_sandwich<float, float, RMS>(a, h, A, rows, STREAM);        \
+    else if (in_f32) launch_sandwich<float, bf16_t, RMS>(a, h, A, rows, STREAM); \
+    else launch_sandwich<bf16_t, bf16_t, RMS>(a, h, A, rows, STREAM);          \
+  }
+  if (rms) GO(true) else GO(false)
+#undef GO
   return DONE;
 }
 
@@ -621,14 +631,16 @@ B200_API int b200_layernorm_rows(const float* x, const int* idx, const float* w,
   return DONE;
 }
 
-B200_API int b200_geglu(void* a, int ld_a, int in_f32, int clear, void* y, int ld_y, int rows, int N, int f32, void* stream) {
+B200_API int b200_glu(void* a, int ld_a, int in_f32, int clear, void* y, int ld_y, int rows, int N, int silu, int f32, void* stream) {
   if (rows <= 0 || N <= 0 || (clear && !in_f32) || (f32 && !in_f32)) return -1;
   for (int r = 0; r < rows; r += 65535) {
     const dim3 grid((N + 255) / 256, rows - r < 65535 ? rows - r : 65535);
     const size_t ao = static_cast<size_t>(r) * ld_a, yo = static_cast<size_t>(r) * ld_y;
-    if (f32) launch_k(geglu_kernel<float, float>, grid, dim3(256), 0, STREAM, (float*)a + ao, ld_a, clear, (float*)y + yo, ld_y, N);
-    else if (in_f32) launch_k(geglu_kernel<float, bf16_t>, grid, dim3(256), 0, STREAM, (float*)a + ao, ld_a, clear, (bf16_t*)y + yo, ld_y, N);
-    else launch_k(geglu_kernel<bf16_t, bf16_t>, grid, dim3(256), 0, STREAM, (bf16_t*)a + ao, ld_a, clear, (bf16_t*)y + yo, ld_y, N);
+#define GO(TI, T, S) launch_k(glu_kernel<TI, T, S>, grid, dim3(256), 0, STREAM, (TI*)a + ao, ld_a, clear, (T*)y + yo, ld_y, N)
+    if (f32) { if (silu) GO(float, float, true); else GO(float, float, false); }
+    else if (in_f32) { if (silu) GO(float, bf16_t, true); else GO(float, bf16_t, false); }
+    else { if (silu) GO(bf16_t, bf16_t, true); else GO(bf16_t, bf16_t, false); }
+#undef GO
   }
   return DONE;
 }

@@ -4,7 +4,8 @@ A layer is a mixer and an optional feed-forward (``models/sublayers.py``).  How 
 is the design's norm style:
 
 * "post_rms": a sublayer reads the stream itself; ``x += mult * rmsnorm(sublayer(x))``;
-* "sandwich": ``x += layernorm(sublayer(layernorm(x)))``; one kernel adds a sublayer's output and norms the next one's input.
+* "sandwich": ``x += layernorm(sublayer(layernorm(x)))``; one kernel adds a sublayer's output and norms the next one's input;
+* "sandwich_rms": the same with RMS norms whose weights are stored around zero.
 
 The residual stream, norms, rotations, scores, softmax, gates of recurrences and recurrent state are fp32; matrix operands are
 bf16 (serving) or fp32.  A range of layers may be executed several times (``LayeredConfig.runs``); every execution has its own
@@ -40,23 +41,45 @@ class LayerNorm(nn.Module):
     def pair(self) -> tuple:
         return self.w, self.b
 
+    def checkpoint_tensors(self, name: str) -> dict:
+        return {name: self.w, name + ".b": self.b}
+
+
+class CentredRMSNorm(nn.Module):
+    """RMS norm times 1 + w."""
+
+    def __init__(self, width: int, device):
+        super().__init__()
+        self.w = vector(width, device)
+
+    @property
+    def pair(self) -> tuple:
+        return self.w, None
+
+    def checkpoint_tensors(self, name: str) -> dict:
+        return {name: self.w}
+
+
+NORMS = {"sandwich": LayerNorm, "sandwich_rms": CentredRMSNorm}
+
 
 class Layer(nn.Module):
     def __init__(self, cfg: LayeredConfig, i: int, dtype, device):
         super().__init__()
         spec = cfg.layers[i]
         self.mix = MIXERS[spec.type](spec.mixer, cfg.width, cfg.norm_eps, dtype, device)
-        self.mlp = None if spec.mlp is None else MLPS[cfg.design.mlp](spec.mlp, cfg.width, dtype, device)
+        self.mlp = None if spec.mlp is None else MLPS[cfg.design.mlps[spec.mlp_kind]](spec.mlp, cfg.width, dtype, device)
         names = ("norm1",) if self.mlp is None else ("norm1", "norm2")
-        if cfg.design.norms == "sandwich":
-            names = [n + side for n in names for side in ("", "b")]        # before and after the sublayer
-        self.norms = nn.ModuleDict({n: LayerNorm(cfg.width, device) for n in names}) if cfg.design.norms == "sandwich" else \
-            nn.ParameterDict({n: vector(cfg.width, device) for n in names})
+        if cfg.design.sandwich:
+            norm = NORMS[cfg.design.norms]
+            self.norms = nn.ModuleDict({n + side: norm(cfg.width, device) for n in names for side in ("", "b")})   # before and after
+        else:
+            self.norms = nn.ParameterDict({n: vector(cfg.width, device) for n in names})
 
     def checkpoint_tensors(self) -> dict:
         out: dict = {}
         for name, n in self.norms.items():
-            out.update({name: n.w, name + ".b": n.b} if isinstance(n, LayerNorm) else {name: n})
+            out.update(n.checkpoint_tensors(name) if isinstance(n, nn.Module) else {name: n})
         out.update({f"mix.{k}": v for k, v in self.mix.checkpoint_tensors().items()})
         if self.mlp is not None:
             out.update({f"mlp.{k}": v for k, v in self.mlp.checkpoint_tensors().items()})
@@ -73,8 +96,8 @@ class LayeredForCausalLM(nn.Module):
         self.config, self.dtype = config, dtype
         self.embed = weight(config.vocab, config.width, dtype, device)
         self.layers = nn.ModuleList(Layer(config, i, dtype, device) for i in range(len(config.layers)))
-        self.sandwich = config.design.norms == "sandwich"
-        self.final_norm = LayerNorm(config.width, device) if self.sandwich else vector(config.width, device)
+        self.sandwich = config.design.sandwich
+        self.final_norm = NORMS[config.design.norms](config.width, device) if self.sandwich else vector(config.width, device)
         self.head = weight(config.vocab, config.width, dtype, device)
         self.loop_step = None if config.loop is None else nn.Parameter(
             torch.zeros(config.loop.times, config.width, dtype=torch.float32, device=device), requires_grad=False)
@@ -89,7 +112,7 @@ class LayeredForCausalLM(nn.Module):
         """Checkpoint name -> the view of this model's storage that holds it."""
         E = self.config.width
         out = {"embed": self.embed[:, :E], "head": self.head[:, :E]}
-        out.update({"final.norm": self.final_norm.w, "final.norm.b": self.final_norm.b} if self.sandwich else {"final.norm": self.final_norm})
+        out.update(self.final_norm.checkpoint_tensors("final.norm") if self.sandwich else {"final.norm": self.final_norm})
         if self.loop_step is not None:
             out["loop.step"] = self.loop_step
         for i, layer in enumerate(self.layers):
@@ -100,7 +123,8 @@ class LayeredForCausalLM(nn.Module):
     def load_checkpoint(self, source) -> None:
         """``source``: a ``SafetensorsFile`` (or anything with ``keys``, ``shape`` and ``tensor``)."""
         want = self.checkpoint_tensors()
-        missing, extra = sorted(set(want) - set(source.keys())), sorted(set(source.keys()) - set(want))
+        unused = {f"l{i}.mix.{k}" for i, layer in enumerate(self.layers) for k in getattr(layer.mix, "unused_tensors", ())}
+        missing, extra = sorted(set(want) - set(source.keys())), sorted(set(source.keys()) - set(want) - unused)
         if missing or extra:
             raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:8]}, unexpected {extra[:8]}")
         for name, dst in want.items():
@@ -130,14 +154,17 @@ class LayeredForCausalLM(nn.Module):
 
     @torch.no_grad()
     def init_weights(self, seed: int = 0) -> "LayeredForCausalLM":
-        """Random weights: matrices normal with deviation 1 / sqrt(fan in), norm weights one, biases zero (forget gates: spread
-        over 3 .. 6, so that memories of different length exist)."""
+        """Random weights: matrices normal with deviation 1 / sqrt(fan in), norm factors one, biases zero (forget gates: spread
+        over 3 .. 6, so that memories of different length exist), mixed values half and half."""
         g = torch.Generator(device=self.device).manual_seed(seed)
+        zero = (".b", ".sink", ".correction") + ((".norm1", ".norm2", "b", "final.norm") if self.config.design.norms == "sandwich_rms" else ())
         for name, t in self.checkpoint_tensors().items():
             if name.endswith(".mix.f.b"):
                 t.copy_(torch.linspace(3.0, 6.0, t.numel(), device=t.device))
+            elif t.dim() == 0:
+                t.fill_(0.5)
             elif t.dim() == 1:
-                t.fill_(0.0 if name.endswith(".b") else 1.0)
+                t.fill_(0.0 if name.endswith(zero) else 1.0)
             else:
                 std = 1.0 if name == "embed" else t.shape[1] ** -0.5
                 t.copy_(torch.randn(t.shape, generator=g, device=self.device, dtype=torch.float32) * std)
@@ -149,7 +176,9 @@ class LayeredForCausalLM(nn.Module):
         if self.sandwich:
             shapes = {(run.index, name): shape for run in self.runs
                       for name, shape in self.layers[run.layer].mix.cache_shapes(max_len).items()}
-            return HybridCache(shapes, max_rows, max_len, self.device)
+            cache = HybridCache(shapes, max_rows, max_len, self.device)
+            cache.rope = self._rope(max_len)
+            return cache
         windows = self.config.latent_windows()
         cache = LatentRingCache({i: self.layers[i].mix.layout for i in windows}, windows, max_rows, max_len, self.dtype, self.device)
         # kept with the cache: captured graphs hold the addresses of both
@@ -157,7 +186,7 @@ class LayeredForCausalLM(nn.Module):
         return cache
 
     def _rope(self, length: int) -> dict:
-        specs = {layer.mix.spec.rot: None for layer in self.layers}
+        specs = {rot: None for rot in (getattr(layer.mix.spec, "rot", None) for layer in self.layers) if rot is not None}
         return {rot: rope_tables(rot, length, self.device) for rot in specs}
 
     # -- execution ---------------------------------------------------------------------------------------------------
@@ -188,14 +217,15 @@ class LayeredForCausalLM(nn.Module):
             step, pre = self._step_vector(n + 1), self.layers[self.runs[n + 1].layer].norms["norm1"].pair
         elif final:
             pre = self.final_norm.pair
+        last = name == ("norm1" if layer.mlp is None else "norm2") and n + 1 == len(self.runs)
         return mem_ops.sandwich_norm_(x, out, layer.norms[name + "b"].pair, step, pre, c.norm_eps, self.dtype, part.out_bias,
-                                      part.out_bias_mult, clear, zero)
+                                      part.out_bias_mult, clear, zero, c.logit_scale if last else 1.0)
 
     def _logits(self, x, idx, h=None):
-        """``h``: the final norm of all rows, where it is formed already."""
+        """``h``: the final norm of all rows, where it is formed already.  The logits' factor is part of that norm."""
         c = self.config
         if h is None:
-            h = mem_ops.layernorm_rows(x, idx, *self.final_norm.pair, c.norm_eps, self.dtype) if self.sandwich else \
+            h = mem_ops.norm_rows(x, idx, *self.final_norm.pair, c.norm_eps, self.dtype, c.logit_scale) if self.sandwich else \
                 ops.rmsnorm_rows(x, idx, self.final_norm, c.norm_eps, self.dtype)
         return ops.linear(h, self.head[:, :c.width], out_f32=True)
 
@@ -210,7 +240,7 @@ class LayeredForCausalLM(nn.Module):
             ctx.cache = self.new_cache(1 + max(r for r, _, _ in step.portions), max(n for _, _, n in step.portions))
         elif not self.sandwich:
             ctx.windows = self.config.latent_windows()
-            ctx.rope = cache.rope if cache is not None else self._rope(max(s + n for _, s, n in step.portions))
+        ctx.rope = ctx.cache.rope if ctx.cache is not None else self._rope(max(s + n for _, s, n in step.portions))
         x, h = self._start(step.tok)
         for n, run in enumerate(self.runs):
             layer = self.layers[run.layer]

@@ -11,6 +11,9 @@ Architectures:
 * ``Fatudra``: layers that run grouped-query attention with a learned distance bias beside a memory with fixed decay, or a
   gated matrix memory; tanh-GELU gated feed-forward; layer norms before and after every sublayer; a range of layers may run
   several times in a row with the same weights.
+* ``Dusilorn``: grouped-query attention, either inside chunks (normed queries and keys, no rotation, an attention sink) or under
+  a sliding window (rotated), scores capped, values mixed with those of the first such layer; a gated feed-forward or a mixture
+  of experts with identity experts and a gated shared expert; RMS norms before and after every sublayer.
 """
 from __future__ import annotations
 
@@ -26,14 +29,21 @@ class Design:
     """What an architecture fixes beside its configuration."""
 
     mixers: tuple                    # mixer types a layer may have
-    norms: str                       # "post_rms": x += mult * rms(f(x)); "sandwich": x += ln(f(ln(x)))
-    mlp: str                         # "relu2": biased two-matrix form; "geglu": gated, tanh-GELU, no biases
+    norms: str                       # "post_rms": x += mult * rms(f(x)); "sandwich": x += ln(f(ln(x))); "sandwich_rms": the
+                                     # same with RMS norms whose weights are stored around zero
+    mlps: dict                       # feed-forward kinds a layer may have -> form: "relu2": biased, two matrices; "geglu" /
+                                     # "swiglu": gated by tanh-GELU / silu, no biases; "relu2_moe": mixture of squared-ReLU experts
     keys: tuple                      # keys of config.json beside the common ones
+
+    @property
+    def sandwich(self) -> bool:
+        return self.norms.startswith("sandwich")
 
 
 DESIGNS = {
-    "Gasovik": Design(("latent_attention",), "post_rms", "relu2", ("residual_mult",)),
-    "Fatudra": Design(("parallel", "mlstm"), "sandwich", "geglu", ("embedding", "loop")),
+    "Gasovik": Design(("latent_attention",), "post_rms", {"dense": "relu2"}, ("residual_mult",)),
+    "Fatudra": Design(("parallel", "mlstm"), "sandwich", {"dense": "geglu"}, ("embedding", "loop")),
+    "Dusilorn": Design(("attention", "attention_2"), "sandwich_rms", {"dense": "swiglu", "moe": "relu2_moe"}, ("embedding", "logit_scale")),
 }
 ARCHITECTURES = tuple(DESIGNS)
 
@@ -79,7 +89,7 @@ class RotarySpec:
     scaling: Optional[YarnScaling] = None
 
     def frequencies(self) -> list:
-        """Radians per position of every interleaved pair."""
+        """Radians per position of every pair."""
         f = [self.base ** (-2 * i / self.dims) for i in range(self.dims // 2)]
         if self.scaling is None:
             return f
@@ -220,6 +230,67 @@ class BiasedAttentionSpec:
 
 
 @dataclass(frozen=True)
+class GroupedAttentionSpec:
+    """Grouped-query attention with capped scores: ``softcap * tanh(q . k * scale / softcap)`` (None: not capped); ``size`` tokens of a window or a
+    chunk are visible.  Subclasses fix the kind of mask, whether q and k are normed (over the whole projection) or rotated, and
+    whether a learned sink takes part in the softmax.  ``v_mix``: values are mixed with those of the first layer that mixes."""
+
+    chunked = False                  # visible: the own chunk (counted from position 0); else the last ``size`` positions
+    qk_norm = False
+    sink = False
+    rotated = False
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    size: int
+    scale: float
+    softcap: Optional[float]
+    v_mix: bool = False
+    rot: Optional[RotarySpec] = None
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GroupedAttentionSpec":
+        _take(d, ("heads", "kv_heads", "dim", "vdim", "mask", "scale", "softcap", "v_mix") + (("rot",) if cls.rotated else ()), "mixer")
+        _take(d["mask"], ("size",), "mixer.mask")
+        spec = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), int(d["mask"]["size"]), float(d["scale"]),
+                   None if d.get("softcap") is None else float(d["softcap"]), bool(d.get("v_mix", False)), RotarySpec.from_dict(d["rot"]) if cls.rotated else None)
+        if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.size) <= 0 or spec.heads % spec.kv_heads:
+            raise ValueError(f"attention sizes must be positive, kv_heads a divisor of heads: {d}")
+        if spec.softcap is not None and not spec.softcap > 0:
+            raise ValueError(f"softcap must be positive: {d}")
+        if spec.rot is not None and (spec.rot.dims > spec.dim or spec.rot.scaling is not None):
+            raise ValueError(f"rot must turn at most {spec.dim} dimensions, without scaling: {d['rot']}")
+        return spec
+
+    def to_dict(self) -> dict:
+        out = {k: getattr(self, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale", "v_mix")}
+        if self.softcap is not None:
+            out["softcap"] = self.softcap
+        out["mask"] = {"size": self.size}
+        if self.rot is not None:
+            out["rot"] = self.rot.to_dict()
+        return out
+
+    @property
+    def v_width(self) -> int:
+        return self.kv_heads * self.vdim
+
+    def param_count(self, E: int) -> int:
+        n = self.heads * (self.dim + self.vdim) * E + self.kv_heads * (self.dim + self.vdim) * E + int(self.v_mix)
+        return n + (self.heads + self.kv_heads) * self.dim * self.qk_norm + self.heads * self.sink
+
+
+class ChunkAttentionSpec(GroupedAttentionSpec):
+    chunked = qk_norm = sink = True
+
+
+class WindowAttentionSpec(GroupedAttentionSpec):
+    rotated = True
+
+
+@dataclass(frozen=True)
 class DecayMemorySpec:
     """Linear attention with one fixed decay per head."""
 
@@ -316,22 +387,72 @@ class DenseMLPSpec:
     @classmethod
     def from_dict(cls, d: dict) -> "DenseMLPSpec":
         _take(d, ("kind", "ff"), "mlp")
-        if d.get("kind") != "dense":
-            raise ValueError(f"unknown feed-forward kind {d.get('kind')!r}")
+        if d["ff"] <= 0:
+            raise ValueError(f"mlp.ff must be positive: {d}")
         return cls(int(d["ff"]))
 
     def to_dict(self) -> dict:
         return {"kind": "dense", "ff": self.ff}
 
+    def param_count(self, E: int) -> int:
+        """Matrices of the gated form."""
+        return 3 * self.ff * E
 
-MIXERS = {"latent_attention": LatentAttentionSpec, "parallel": ParallelSpec, "mlstm": GatedMemorySpec}
+
+@dataclass(frozen=True)
+class MixtureSpec:
+    """``experts`` feed-forwards of ``ff`` hidden units and ``identity`` experts that return their input, of which each token uses
+    ``top``; ``shared``: hidden units of an expert that runs for every token behind a gate (None: there is none)."""
+
+    ff: int
+    experts: int
+    identity: int
+    top: int
+    shared: Optional[int] = None
+
+    @property
+    def outputs(self) -> int:
+        """Router outputs."""
+        return self.experts + self.identity
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "MixtureSpec":
+        _take(d, ("kind", "expert", "router", "shared"), "mlp")
+        _take(d["expert"], ("ff",), "mlp.expert")
+        _take(d["router"], ("experts", "identity", "top"), "mlp.router")
+        shared = d.get("shared")
+        if shared is not None:
+            _take(shared, ("ff",), "mlp.shared")
+        r = d["router"]
+        spec = cls(int(d["expert"]["ff"]), int(r["experts"]), int(r.get("identity", 0)), int(r["top"]), None if shared is None else int(shared["ff"]))
+        if min(spec.ff, spec.experts, spec.top, 1 if spec.shared is None else spec.shared) <= 0 or spec.identity < 0 or spec.top > spec.outputs:
+            raise ValueError(f"a mixture needs positive sizes and at most as many chosen experts as there are: {d}")
+        return spec
+
+    def to_dict(self) -> dict:
+        out = {"kind": "moe", "expert": {"ff": self.ff}, "router": {"experts": self.experts, "identity": self.identity, "top": self.top}}
+        if self.shared is not None:
+            out["shared"] = {"ff": self.shared}
+        return out
+
+    def param_count(self, E: int) -> int:
+        return 2 * self.experts * self.ff * E + self.outputs * (E + 1) + (0 if self.shared is None else (2 * self.shared + 1) * E)
+
+    def active_params(self, E: int) -> int:
+        """Parameters that a token meets when all its experts have tensors."""
+        return 2 * self.top * self.ff * E + self.outputs * (E + 1) + (0 if self.shared is None else (2 * self.shared + 1) * E)
+
+
+MIXERS = {"latent_attention": LatentAttentionSpec, "parallel": ParallelSpec, "mlstm": GatedMemorySpec, "attention": ChunkAttentionSpec,
+          "attention_2": WindowAttentionSpec}
+MLPS = {"dense": DenseMLPSpec, "moe": MixtureSpec}
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     type: str
     mixer: object                    # one of the specs of MIXERS
-    mlp: Optional[DenseMLPSpec] = None
+    mlp: Optional[object] = None     # one of the specs of MLPS
 
     @classmethod
     def from_dict(cls, d: dict) -> "LayerSpec":
@@ -339,7 +460,13 @@ class LayerSpec:
         if d["type"] not in MIXERS:
             raise ValueError(f"unknown mixer type {d['type']!r}")
         mlp = d.get("mlp")
-        return cls(d["type"], MIXERS[d["type"]].from_dict(d["mixer"]), None if mlp is None else DenseMLPSpec.from_dict(mlp))
+        if mlp is not None and mlp.get("kind") not in MLPS:
+            raise ValueError(f"unknown feed-forward kind {mlp.get('kind')!r}")
+        return cls(d["type"], MIXERS[d["type"]].from_dict(d["mixer"]), None if mlp is None else MLPS[mlp["kind"]].from_dict(mlp))
+
+    @property
+    def mlp_kind(self) -> str:
+        return "moe" if isinstance(self.mlp, MixtureSpec) else "dense"
 
     def to_dict(self) -> dict:
         return {"type": self.type, "mixer": self.mixer.to_dict(), "mlp": None if self.mlp is None else self.mlp.to_dict()}
@@ -366,6 +493,7 @@ class LayeredConfig:
     name: str = ""
     embed_scale: float = 1.0
     loop: Optional[LoopSpec] = None
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         if self.architecture not in ARCHITECTURES:
@@ -375,6 +503,8 @@ class LayeredConfig:
         for i, layer in enumerate(self.layers):
             if layer.type not in self.design.mixers:
                 raise ValueError(f"layer {i}: {self.architecture} has no mixer {layer.type!r}")
+            if layer.mlp is not None and layer.mlp_kind not in self.design.mlps:
+                raise ValueError(f"layer {i}: {self.architecture} has no feed-forward {layer.mlp_kind!r}")
             j = getattr(layer.mixer, "kv_from", None)
             if j is None:
                 continue
@@ -383,6 +513,8 @@ class LayeredConfig:
             a, b = layer.mixer, self.layers[j].mixer
             if (a.kv_rank, a.rot_dim, a.rot) != (b.kv_rank, b.rot_dim, b.rot):
                 raise ValueError(f"layer {i}: latent size and rotation must equal those of layer {j}")
+        if len({layer.mixer.v_width for layer in self.layers if getattr(layer.mixer, "v_mix", False)}) > 1:
+            raise ValueError("layers that mix their values need equally many value rows")
         lp = self.loop
         if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layers) and lp.times >= 1):
             raise ValueError(f"loop {lp} does not lie inside {len(self.layers)} layers")
@@ -405,6 +537,11 @@ class LayeredConfig:
             else:
                 order.append((i, None))
         return [LayerRun(n, i, t) for n, (i, t) in enumerate(order)]
+
+    def mixes_values(self, i: int) -> Optional[str]:
+        """"first": layer ``i`` provides the values that later layers mix in, "mix": it mixes them into its own, None: neither."""
+        mixing = [k for k, layer in enumerate(self.layers) if getattr(layer.mixer, "v_mix", False)]
+        return None if i not in mixing else "first" if i == mixing[0] else "mix"
 
     def kv_source(self, i: int) -> int:
         """The layer whose latents layer ``i`` attends to."""
@@ -444,8 +581,9 @@ class LayeredConfig:
         if d.get("loop") is not None:
             loop = LoopSpec.from_dict(d["loop"])
         mult = float(d["residual_mult"]) if "residual_mult" in keys else 1.0
+        logit = float(d["logit_scale"]) if "logit_scale" in keys else 1.0
         return cls(d["architecture"], int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), mult,
-                   [LayerSpec.from_dict(x) for x in d["layers"]], d.get("name", ""), scale, loop)
+                   [LayerSpec.from_dict(x) for x in d["layers"]], d.get("name", ""), scale, loop, logit)
 
     def to_dict(self) -> dict:
         out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps}}
@@ -454,6 +592,8 @@ class LayeredConfig:
             out["residual_mult"] = self.residual_mult
         if "embedding" in keys:
             out["embedding"] = {"scale": self.embed_scale}
+        if "logit_scale" in keys:
+            out["logit_scale"] = self.logit_scale
         if self.loop is not None:
             out["loop"] = self.loop.to_dict()
         out["layers"] = [x.to_dict() for x in self.layers]
@@ -485,10 +625,11 @@ class LayeredConfig:
     # -- counts ------------------------------------------------------------------------------------------------------
     def param_count(self) -> int:
         E = self.width
-        if self.design.norms == "sandwich":
-            n = 2 * self.vocab * E + 2 * E + (0 if self.loop is None else self.loop.times * E)
+        if self.design.sandwich:
+            norm = 2 * E if self.design.norms == "sandwich" else E
+            n = 2 * self.vocab * E + norm + (0 if self.loop is None else self.loop.times * E)
             for layer in self.layers:
-                n += layer.mixer.param_count(E) + 4 * E + (0 if layer.mlp is None else 3 * layer.mlp.ff * E + 4 * E)
+                n += layer.mixer.param_count(E) + 2 * norm + (0 if layer.mlp is None else layer.mlp.param_count(E) + 2 * norm)
             return n
         n = 2 * self.vocab * E + E
         for i, layer in enumerate(self.layers):

@@ -12,12 +12,15 @@ from typing import Callable, Optional
 import torch
 import torch.nn as nn
 
+from ..ops import grouped as grp_ops
 from ..ops import latent as ops
 from ..ops import memory as mem_ops
+from ..ops import moe as moe_ops
+from ..ops.grouped import GroupedLayout, QkvTransform
 from ..ops.latent import LatentLayout, pad8
 from ..ops.memory import BiasTable, MemoryLayout, ParallelLayout
-from .layered_config import (DenseMLPSpec, GatedMemorySpec, LatentAttentionSpec, LayeredConfig, LayerRun, ParallelSpec,
-                             RotarySpec)
+from .layered_config import (DenseMLPSpec, GatedMemorySpec, GroupedAttentionSpec, LatentAttentionSpec, LayeredConfig, LayerRun,
+                             MixtureSpec, ParallelSpec, RotarySpec)
 
 
 def weight(rows: int, cols: int, dtype, device) -> nn.Parameter:
@@ -41,12 +44,12 @@ def rope_tables(rot: RotarySpec, length: int, device) -> tuple:
 # ------------------------------------------------------------------------------------------
 @dataclass
 class StreamLayout:
-    """Where the keys of a packed step lie for a given history length: per sequence first the cached positions its portion can
-    still see, then the portion itself."""
+    """Where the keys of a packed step lie: per sequence first the cached positions its portion can still see, then the portion
+    itself."""
 
     sidx: torch.Tensor        # [T] stream index of every token
-    kbase: torch.Tensor       # [T] stream index of the first key of its sequence
-    seqs: list                # (first token, tokens, first key, history) per sequence
+    kbase: torch.Tensor       # [T] stream index of the first key of its sequence (of its chunk)
+    seqs: list                # (first token, tokens, first key, keys in front of the first token) per sequence (per chunk of one)
     total: int
     history: list             # (row, first position, count, first key) of the sequences with history
 
@@ -105,6 +108,29 @@ class PackedStep:
             self._layouts[history] = StreamLayout(idx[0], idx[1], seqs, k0, hist)
         return self._layouts[history]
 
+    def chunk_layout(self, size: int) -> StreamLayout:
+        """Layout for attention inside chunks of ``size`` positions: the history of a portion is what its first chunk already
+        holds; every chunk counts as a sequence of its own."""
+        key = ("chunk", size)
+        if key not in self._layouts:
+            seqs, sidx, kbase, hist = [], [], [], []
+            t0 = k0 = 0
+            for r, s, n in self.portions:
+                h = s % size
+                sidx.extend(range(k0 + h, k0 + h + n))
+                if h:
+                    hist.append((r, s - h, h, k0))
+                at, key0, front = 0, k0, h
+                while at < n:                                  # the part of one chunk at a time
+                    m = min(size - front, n - at)
+                    seqs.append((t0 + at, m, key0, front))
+                    kbase.extend([key0] * m)
+                    at, key0, front = at + m, key0 + front + m, 0
+                t0, k0 = t0 + n, k0 + h + n
+            idx = torch.tensor([sidx, kbase], dtype=torch.int32).to(self.device)
+            self._layouts[key] = StreamLayout(idx[0], idx[1], seqs, k0, hist)
+        return self._layouts[key]
+
 
 @dataclass
 class StepContext:
@@ -116,6 +142,7 @@ class StepContext:
     rope: dict = field(default_factory=dict)       # rotary spec -> (cos, sin)
     windows: dict = field(default_factory=dict)    # latent source layer -> widest window
     streams: dict = field(default_factory=dict)    # latent source layer -> latent rows of the step
+    first_values: Optional[torch.Tensor] = None    # values that later layers mix into theirs
 
 
 @dataclass
@@ -129,10 +156,11 @@ class DecodeContext:
     cache: object
     dense: Callable
     splits: Callable
+    first_values: Optional[torch.Tensor] = None    # values that later layers mix into theirs
 
 
 def gather_history(layout: StreamLayout, cache: torch.Tensor, stream: torch.Tensor) -> None:
-    """Copy the cached latents in front of every portion from the ring ``cache`` [rows, cap, ld] into the stream."""
+    """Copy the cached rows in front of every portion from the ring ``cache`` [rows, cap, ld] into the stream."""
     if not layout.history:
         return
     cap = cache.shape[1]
@@ -354,9 +382,77 @@ class GatedMemory(nn.Module):
         return out, clear, inp if acc else None
 
 
-class GatedMLP(nn.Module):
-    """down(gelu(gate x) * (up x)), tanh form, no biases."""
+class GroupedAttention(nn.Module):
+    """Grouped-query attention over a ring of keys and values (``GroupedAttentionSpec``): inside chunks or under a window."""
 
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: GroupedAttentionSpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        a = spec
+        self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
+        L = self.layout = GroupedLayout(a.heads, a.kv_heads, a.dim, a.vdim)
+        self.w_in = weight(L.width_in, width, dtype, device)
+        self.w_o = weight(width, a.heads * a.vdim, dtype, device)
+        self.q_norm, self.k_norm = (vector(n * a.dim, device) if a.qk_norm else None for n in (a.heads, a.kv_heads))
+        self.sink = vector(a.heads, device) if a.sink else None
+        self.vmix = nn.Parameter(torch.zeros((), dtype=torch.float32, device=device), requires_grad=False) if a.v_mix else None
+
+    def checkpoint_tensors(self) -> dict:
+        a, L, E = self.spec, self.layout, self.width
+        out = {name: self.w_in[at:at + n, :E] for name, at, n in (("q", L.off_q, a.heads * a.dim), ("k", L.off_k, a.kv_heads * a.dim),
+                                                                  ("v", L.off_v, L.v_width))}
+        out["o"] = self.w_o[:, :a.heads * a.vdim]
+        out.update({k: v for k, v in (("q.norm", self.q_norm), ("k.norm", self.k_norm), ("sink", self.sink), ("vmix", self.vmix)) if v is not None})
+        return out
+
+    @property
+    def unused_tensors(self) -> tuple:
+        """Checkpoint tensors that may stand beside the others without a use."""
+        return () if self.spec.v_mix else ("vmix",)
+
+    def cache_shapes(self, max_len: int) -> dict:
+        return {"kv": ((min(self.spec.size, max_len), self.layout.ld_kv), self.dtype)}
+
+    def _transform(self, role: Optional[str], rope: dict, first) -> QkvTransform:
+        rot = self.spec.rot
+        mix = role == "mix"
+        return QkvTransform(self.q_norm, self.k_norm, self.eps, 0 if rot is None else rot.dims, None if rot is None else rope[rot],
+                            self.vmix if mix else None, first if mix else None)
+
+    def stream(self, h, run: LayerRun, ctx: StepContext):
+        a, L, step, role = self.spec, self.layout, ctx.step, ctx.config.mixes_values(run.layer)
+        cache = ctx.cache.data[run.index, "kv"]
+        lay = step.chunk_layout(a.size) if a.chunked else step.layout(a.size - 1)
+        inp = ops.linear(h, self.w_in[:, :self.width])
+        kv = torch.empty(lay.total, L.ld_kv, dtype=self.dtype, device=h.device)
+        gather_history(lay, cache, kv)             # before the ring slots of the oldest positions are written again
+        grp_ops.qkv_prep_(L, inp, self._transform(role, ctx.rope, ctx.first_values), step, lay.sidx, cache, kv)
+        if role == "first":
+            ctx.first_values = inp[:, L.off_v:L.off_v + L.v_width]
+        o = grp_ops.stream_attention(L, a, inp, kv, lay, self.sink)
+        return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
+
+    def decode_splits(self, B: int, max_len: int, tensor_cores: bool) -> int:
+        return grp_ops.decode_splits(self.layout, B, min(self.spec.size, max_len), tensor_cores)
+
+    def decode(self, h, run: LayerRun, ctx: DecodeContext):
+        a, L, role = self.spec, self.layout, ctx.config.mixes_values(run.layer)
+        inp, acc = ctx.dense(h, self.w_in[:, :self.width], 0)
+        tr = self._transform(role, ctx.cache.rope, ctx.first_values)
+        first = torch.empty(h.shape[0], pad8(L.v_width), dtype=torch.float32, device=h.device)[:, :L.v_width] if role == "first" else None
+        o = grp_ops.ring_attention(L, a, inp, tr, ctx.cache.data[run.index, "kv"], self.sink, first, ctx.pos, ctx.row, ctx.splits(self, h.shape[0]),
+                                   self.dtype)
+        if first is not None:
+            ctx.first_values = first
+        out, clear = ctx.dense(o, self.w_o[:, :a.heads * a.vdim], 1)
+        return out, clear, inp if acc else None
+
+
+class GatedMLP(nn.Module):
+    """down(act(gate x) * (up x)), no biases; ``act``: "gelu" (tanh form) or "silu"."""
+
+    act = "gelu"
     wide = 2
     out_bias, out_bias_mult = None, 1.0
 
@@ -370,12 +466,55 @@ class GatedMLP(nn.Module):
         return {"gate": self.w_gu[:f, :E], "up": self.w_gu[f:, :E], "down": self.w_down[:, :f]}
 
     def forward(self, h):
-        return ops.linear(mem_ops.geglu_linear(h, self.w_gu[:, :self.width], self.spec.ff), self.w_down[:, :self.spec.ff])
+        return ops.linear(mem_ops.glu_linear(h, self.w_gu[:, :self.width], self.spec.ff, self.act), self.w_down[:, :self.spec.ff])
 
     def decode(self, h, dense):
         a, clear = dense(h, self.w_gu[:, :self.width], 1)
-        return dense(mem_ops.geglu(a, self.spec.ff, self.dtype, clear), self.w_down[:, :self.spec.ff], 1)
+        return dense(mem_ops.glu(a, self.spec.ff, self.act, self.dtype, clear), self.w_down[:, :self.spec.ff], 1)
 
 
-MIXERS = {"latent_attention": LatentAttention, "parallel": ParallelMixer, "mlstm": GatedMemory}
-MLPS = {"relu2": DenseMLP, "geglu": GatedMLP}
+class SiluMLP(GatedMLP):
+    act = "silu"
+
+
+class MixtureMLP(nn.Module):
+    """Mixture of squared-ReLU experts with identity experts and a gated shared expert (``MixtureSpec``).  The experts' matrices lie
+    one below the other; the shared expert's gate is one more row of the router."""
+
+    wide = 0
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: MixtureSpec, width: int, dtype, device):
+        super().__init__()
+        s = spec
+        self.spec, self.width, self.dtype = spec, width, dtype
+        self.w_router, self.correction = weight(s.outputs + (s.shared is not None), width, dtype, device), vector(s.outputs, device)
+        self.w_up, self.w_down = weight(s.experts * s.ff, width, dtype, device), weight(s.experts * width, s.ff, dtype, device)
+        if s.shared is not None:
+            self.s_up, self.s_down = weight(s.shared, width, dtype, device), weight(width, s.shared, dtype, device)
+
+    def checkpoint_tensors(self) -> dict:
+        s, E = self.spec, self.width
+        out = {"router": self.w_router[:s.outputs, :E], "correction": self.correction}
+        for e in range(s.experts):
+            out[f"e{e}.up"], out[f"e{e}.down"] = self.w_up[e * s.ff:(e + 1) * s.ff, :E], self.w_down[e * E:(e + 1) * E, :s.ff]
+        if s.shared is not None:
+            out.update({"shared.sg": self.w_router[s.outputs:, :E], "shared.up": self.s_up[:, :E], "shared.down": self.s_down[:, :s.shared]})
+        return out
+
+    @property
+    def weights(self) -> moe_ops.MoeWeights:
+        s, E = self.spec, self.width
+        up, down = (None, None) if s.shared is None else (self.s_up[:, :E], self.s_down[:, :s.shared])
+        return moe_ops.MoeWeights(s, self.w_router[:, :E], self.correction, self.w_up[:, :E], self.w_down[:, :s.ff], up, down)
+
+    def forward(self, h):
+        return moe_ops.mixture(self.weights, h)
+
+    def decode(self, h, dense):
+        return moe_ops.mixture_rows(self.weights, h), False
+
+
+MIXERS = {"latent_attention": LatentAttention, "parallel": ParallelMixer, "mlstm": GatedMemory, "attention": GroupedAttention,
+          "attention_2": GroupedAttention}
+MLPS = {"relu2": DenseMLP, "geglu": GatedMLP, "swiglu": SiluMLP, "relu2_moe": MixtureMLP}

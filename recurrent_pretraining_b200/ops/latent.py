@@ -69,7 +69,7 @@ class _WindowAttn(C.Structure):
                [(n, C.c_void_p) for n in ("sidx", "kbase", "pos", "row")] + [("cap", C.c_int)] + \
                [(n, C.c_int) for n in ("gate_ld", "out_ld")] + [(n, C.c_void_p) for n in ("part_o", "part_ml")] + \
                [("group", C.c_int), ("bias", C.c_void_p), ("bias_len", C.c_int), ("temp_every", C.c_int), ("temp_coef", C.c_float),
-                ("head_gate", C.c_int), ("gate_mult", C.c_float)]
+                ("head_gate", C.c_int), ("gate_mult", C.c_float), ("softcap", C.c_float), ("chunk", C.c_int), ("sink", C.c_void_p)]
 
 
 _fns = None
@@ -94,9 +94,9 @@ def _k():
             attn=K._sig("b200_window_attention", [vp] * 6 + [att, i, i, vp]),
             expand=K._sig("b200_latent_expand", [vp, vp, i, vp, i, vp, i, vp] + [i] * 7 + [vp]),
             resid=K._sig("b200_rms_residual", [vp] + [i] * 3 + [vp] * 4 + [i] * 3 + [f, f, vp, i, i, vp]),
-            norm_rows=K._sig("b200_rmsnorm_rows", [vp] * 4 + [i] * 3 + [f, i, vp]),
+            norm_rows=K._sig("b200_rmsnorm_rows", [vp] * 4 + [i] * 3 + [f, f, f, i, vp]),
             bias_act=K._sig("b200_bias_act", [vp] + [i] * 3 + [vp, vp] + [i] * 5 + [vp]),
-            sgemm=K._sig("b200_sgemm_nt", [vp] * 4 + [i] * 9 + [vp]),
+            sgemm=K._sig("b200_sgemm_nt", [vp] * 4 + [i] * 9 + [vp] * 3),
         )
     return _fns
 
@@ -135,7 +135,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     out = torch.empty(M, max(ld_out, pad8(N)), dtype=F32 if out_f32 else x.dtype, device=x.device)[:, :N]
     if x.dtype == F32:
         k.K._check(k.sgemm(x.data_ptr(), w.data_ptr(), k.K._ptr(bias), out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0),
-                           out.stride(0), _ACT[act], act_cols[0], act_cols[1], k.K._stream()), "sgemm_nt")
+                           out.stride(0), _ACT[act], act_cols[0], act_cols[1], 0, 0, k.K._stream()), "sgemm_nt")
         return out
     if out_f32:
         return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_F32)
@@ -192,17 +192,18 @@ def rms_residual_(x: torch.Tensor, a: torch.Tensor, bias, w: torch.Tensor, eps: 
     return xb
 
 
-def rmsnorm_rows(x: torch.Tensor, idx: Optional[torch.Tensor], w: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
-    """rmsnorm(x[idx]) * w in ``dtype`` (all rows when ``idx`` is None)."""
+def rmsnorm_rows(x: torch.Tensor, idx: Optional[torch.Tensor], w: torch.Tensor, eps: float, dtype: torch.dtype, w_add: float = 0.0,
+                 mult: float = 1.0) -> torch.Tensor:
+    """mult * rmsnorm(x[idx]) * (w + w_add) in ``dtype`` (all rows when ``idx`` is None)."""
     if not x.is_cuda:
         rows = x if idx is None else x[idx.long()]
-        return (ref.rms(rows, eps) * w).to(dtype)
+        return (ref.rms(rows, eps) * (w + w_add) * mult).to(dtype)
     k = _k()
     n, E = (x.shape[0] if idx is None else idx.numel()), x.shape[1]
     assert idx is None or (idx.dtype == torch.int32 and idx.is_cuda)
     y = torch.empty(n, pad8(E), dtype=dtype, device=x.device)[:, :E]
-    k.K._check(k.norm_rows(x.data_ptr(), k.K._ptr(idx), w.data_ptr(), y.data_ptr(), y.stride(0), n, E, eps, int(dtype == F32),
-                           k.K._stream()), "rmsnorm_rows")
+    k.K._check(k.norm_rows(x.data_ptr(), k.K._ptr(idx), w.data_ptr(), y.data_ptr(), y.stride(0), n, E, eps, w_add, mult,
+                           int(dtype == F32), k.K._stream()), "rmsnorm_rows")
     return y
 
 

@@ -79,7 +79,7 @@ class MemoryLayout:
 
 
 class _Sandwich(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("E", "ld_a", "ld_h", "clear", "nzero")] + [(n, C.c_float) for n in ("eps", "bias_mult")] + \
+    _fields_ = [(n, C.c_int) for n in ("E", "ld_a", "ld_h", "clear", "nzero")] + [(n, C.c_float) for n in ("eps", "bias_mult", "out_mult")] + \
                [(n, C.c_void_p) for n in ("bias", "w1", "b1", "step", "w2", "b2", "x", "zero")]
 
 
@@ -107,9 +107,9 @@ def _k():
         vp, i, f = C.c_void_p, C.c_int, C.c_float
         _fns = SimpleNamespace(
             K=K,
-            sandwich=K._sig("b200_sandwich_norm", [vp, vp, C.POINTER(_Sandwich), i, i, i, vp]),
+            sandwich=K._sig("b200_sandwich_norm", [vp, vp, C.POINTER(_Sandwich), i, i, i, i, vp]),
             rows=K._sig("b200_layernorm_rows", [vp] * 5 + [i] * 3 + [f, i, vp]),
-            geglu=K._sig("b200_geglu", [vp] + [i] * 3 + [vp] + [i] * 4 + [vp]),
+            glu=K._sig("b200_glu", [vp] + [i] * 3 + [vp] + [i] * 5 + [vp]),
             append=K._sig("b200_kv_append", [vp, i, vp, vp] + [i] * 3 + [vp, vp] + [i] * 3 + [vp]),
             scan=K._sig("b200_memory_scan", [vp] * 4 + [C.POINTER(_Memory)] + [i] * 3 + [vp]),
             merge=K._sig("b200_memory_merge", [vp] * 3 + [C.POINTER(_Merge)] + [i] * 4 + [vp]),
@@ -120,19 +120,26 @@ def _k():
 # ------------------------------------------------------------------------------------------
 # layer norms, feed-forward
 # ------------------------------------------------------------------------------------------
+def _norm(x, w, b, eps: float) -> torch.Tensor:
+    """Plain form: layer norm, or without ``b`` the RMS norm with weights 1 + w."""
+    return ref.rms(x, eps) * (1 + w) if b is None else ref.layer_norm(x, w, b, eps)
+
+
 def sandwich_norm_(x: torch.Tensor, a: Optional[torch.Tensor], post, step, pre, eps: float, dtype: torch.dtype, bias=None,
-                   bias_mult: float = 1.0, clear: bool = False, zero: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """x += layernorm(a + bias_mult * bias) [+ step] in place, then layernorm(x) in ``dtype`` (None without ``pre``).  ``post``
-    and ``pre`` are (weight, bias); ``a`` may be None (only ``step`` is added then).  ``clear`` / ``zero``: accumulators that are
-    handed back zeroed (a itself / a second one with the same number of rows)."""
+                   bias_mult: float = 1.0, clear: bool = False, zero: Optional[torch.Tensor] = None,
+                   out_mult: float = 1.0) -> Optional[torch.Tensor]:
+    """x += norm(a + bias_mult * bias) [+ step] in place, then out_mult * norm(x) in ``dtype`` (None without ``pre``).  ``post``
+    and ``pre`` are (weight, bias) of layer norms, or (weight, None) of RMS norms whose weights are stored around zero; ``a``
+    may be None (only ``step`` is added then).  ``clear`` / ``zero``: accumulators that are handed back zeroed (a itself / a
+    second one with the same number of rows)."""
     T, E = x.shape
     if not x.is_cuda:
         if a is not None:
             s = a.float() if bias is None else a.float() + bias_mult * bias
-            x += ref.layer_norm(s, *post, eps)
+            x += _norm(s, *post, eps)
         if step is not None:
             x += step
-        return None if pre is None else ref.layer_norm(x, *pre, eps).to(dtype)
+        return None if pre is None else (_norm(x, *pre, eps) * out_mult).to(dtype)
     k = _k()
     assert x.is_contiguous() and (a is None or a.shape == (T, E)) and (zero is None or zero.is_contiguous())
     h = None if pre is None else torch.empty(T, pad8(E), dtype=dtype, device=x.device)[:, :E]
@@ -140,14 +147,17 @@ def sandwich_norm_(x: torch.Tensor, a: Optional[torch.Tensor], post, step, pre, 
     w1, b1 = post if a is not None else (None, None)
     w2, b2 = pre if pre is not None else (None, None)
     s = _Sandwich(E, 0 if a is None else a.stride(0), 0 if h is None else h.stride(0), int(clear), 0 if zero is None else zero.numel() // T,
-                  eps, bias_mult, p(bias), p(w1), p(b1), p(step), p(w2), p(b2), x.data_ptr(), p(zero))
-    f32 = int(dtype == F32)
-    k.K._check(k.sandwich(p(a), p(h), C.byref(s), T, f32 if a is None else _f32(a), f32, k.K._stream()), "sandwich_norm")
+                  eps, bias_mult, out_mult, p(bias), p(w1), p(b1), p(step), p(w2), p(b2), x.data_ptr(), p(zero))
+    f32, rms = int(dtype == F32), int(b1 is None and b2 is None)
+    k.K._check(k.sandwich(p(a), p(h), C.byref(s), T, f32 if a is None else _f32(a), f32, rms, k.K._stream()), "sandwich_norm")
     return h
 
 
-def layernorm_rows(x: torch.Tensor, idx: Optional[torch.Tensor], w, b, eps: float, dtype: torch.dtype) -> torch.Tensor:
-    """layernorm(x[idx]) in ``dtype`` (all rows when ``idx`` is None)."""
+def norm_rows(x: torch.Tensor, idx: Optional[torch.Tensor], w, b, eps: float, dtype: torch.dtype, mult: float = 1.0) -> torch.Tensor:
+    """mult * norm(x[idx]) in ``dtype`` (all rows when ``idx`` is None); the norm as in ``sandwich_norm_``."""
+    if b is None:
+        return base.rmsnorm_rows(x, idx, w, eps, dtype, 1.0, mult)
+    assert mult == 1.0
     if not x.is_cuda:
         return ref.layer_norm(x if idx is None else x[idx.long()], w, b, eps).to(dtype)
     k = _k()
@@ -158,24 +168,28 @@ def layernorm_rows(x: torch.Tensor, idx: Optional[torch.Tensor], w, b, eps: floa
     return y
 
 
-def geglu(a: torch.Tensor, n: int, dtype: torch.dtype, clear: bool = False) -> torch.Tensor:
-    """gelu(a[:, :n]) * a[:, n:2n] (tanh form) in ``dtype``; ``clear`` hands a stream-K accumulator back zeroed."""
+def glu(a: torch.Tensor, n: int, act: str, dtype: torch.dtype, clear: bool = False) -> torch.Tensor:
+    """act(a[:, :n]) * a[:, n:2n] in ``dtype``, act "gelu" (tanh form) or "silu"; ``clear`` hands a stream-K accumulator back
+    zeroed."""
     M = a.shape[0]
     if not a.is_cuda:
-        return (torch.nn.functional.gelu(a[:, :n].float(), approximate="tanh") * a[:, n:2 * n].float()).to(dtype)
+        g = a[:, :n].float()
+        g = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+        return (g * a[:, n:2 * n].float()).to(dtype)
     k = _k()
     y = torch.empty(M, pad8(n), dtype=dtype, device=a.device)[:, :n]
-    k.K._check(k.geglu(a.data_ptr(), a.stride(0), _f32(a), int(clear), y.data_ptr(), y.stride(0), M, n, int(dtype == F32), k.K._stream()), "geglu")
+    k.K._check(k.glu(a.data_ptr(), a.stride(0), _f32(a), int(clear), y.data_ptr(), y.stride(0), M, n, int(act == "silu"), int(dtype == F32),
+                     k.K._stream()), "glu")
     return y
 
 
-def geglu_linear(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
-    """gelu(x Wg^T) * (x Wu^T) for ``w`` [2n, K] = [Wg; Wu]; bf16: gated in the epilogue of the product."""
+def glu_linear(x: torch.Tensor, w: torch.Tensor, n: int, act: str) -> torch.Tensor:
+    """act(x Wg^T) * (x Wu^T) for ``w`` [2n, K] = [Wg; Wu]; bf16: gated in the epilogue of the product."""
     if not x.is_cuda or x.dtype == F32:
-        return geglu(linear(x, w), n, x.dtype)
+        return glu(linear(x, w), n, act, x.dtype)
     k = _k()
     out = torch.empty(x.shape[0], pad8(n), dtype=x.dtype, device=x.device)[:, :n]
-    return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_SWIGLU, act=3)
+    return k.K.gemm(x, w, out=out, out_mode=k.K.OUT_SWIGLU, act=0 if act == "silu" else 3)
 
 
 # ------------------------------------------------------------------------------------------

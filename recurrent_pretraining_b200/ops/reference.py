@@ -254,3 +254,40 @@ def log_gates(raw: torch.Tensor, bias: torch.Tensor, cap: float):
     """Log input gate and log forget gate [T, H] of raw projections [T, 2H]."""
     i, f = (cap * torch.tanh((raw.float() + bias) / cap)).chunk(2, dim=-1)
     return i, F.logsigmoid(f)
+
+
+# ------------------------------------------------------------------------------------------
+# layered decoder models: capped attention with a sink, mixture of experts
+# ------------------------------------------------------------------------------------------
+def rotate_halves(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """Rotation of entry i of the first half of the last dim with entry i of the second; fp32 result."""
+    u, v = x.float().chunk(2, dim=-1)
+    return torch.cat([u * cos - v * sin, v * cos + u * sin], dim=-1)
+
+
+def capped_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, visible: torch.Tensor, scale: float, softcap: float | None,
+                     sink: torch.Tensor | None) -> torch.Tensor:
+    """Grouped-query attention: q [T, H, D]; k, v [K, G, .] shared by all queries or [T, K, G, .] per query; visible [T, K]; ``sink``
+    [H]: one more term of the softmax's denominator.  fp32."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[-2]
+    q = q.float().unflatten(1, (G, H // G))
+    per_query = k.dim() == 4
+    s = torch.einsum("tgrd,tkgd->tgrk" if per_query else "tgrd,kgd->tgrk", q, k.float()).flatten(1, 2) * scale
+    if softcap:
+        s = softcap * torch.tanh(s / softcap)
+    s = s.masked_fill(~visible[:, None], float("-inf"))
+    if sink is not None:
+        s = torch.cat([s, sink[None, :, None].expand(T, -1, 1)], dim=-1)
+    p = torch.softmax(s, dim=-1)
+    if sink is not None:
+        p = p[..., :-1]
+    v = v.float().masked_fill(~visible[:, :, None, None], 0.0) if per_query else v.float()      # slots that were never written
+    return torch.einsum("tgrk,tkge->tgre" if per_query else "tgrk,kge->tgre", p.unflatten(1, (G, H // G)), v).flatten(1, 2)
+
+
+def route(z: torch.Tensor, correction: torch.Tensor, top: int):
+    """Router logits [T, outputs] -> chosen outputs [T, top], best first, and their normalised scores."""
+    s = torch.softmax(z.float(), dim=-1)
+    idx = torch.sort(s + correction, dim=-1, descending=True, stable=True).indices[:, :top]
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20)

@@ -236,8 +236,8 @@ def hybrid_ops_prefill(model, seqs: list, t: Timer) -> list:
         t.op("  memory: " + name, lambda part=part: run(part), nbytes, 0)
     mlp = model.layers[i].mlp
     ff = mlp.spec.ff
-    g = M.geglu_linear(h, mlp.w_gu[:, :E], ff)
-    gemm("gate-up projection + geglu", lambda: M.geglu_linear(h, mlp.w_gu[:, :E], ff), T, 2 * ff, E)
+    g = M.glu_linear(h, mlp.w_gu[:, :E], ff, "gelu")
+    gemm("gate-up projection + geglu", lambda: M.glu_linear(h, mlp.w_gu[:, :E], ff, "gelu"), T, 2 * ff, E)
     gemm("down projection", lambda: ops.linear(g, mlp.w_down[:, :ff]), T, E, ff)
     return t.take()
 
@@ -293,7 +293,7 @@ def hybrid_ops_decode(model, B: int, context: int, t: Timer) -> list:
     mlp = model.layers[i].mlp
     ff = mlp.spec.ff
     skinny("gate-up projection", h, mlp.w_gu[:, :E])
-    t.op("geglu", lambda: M.geglu(work[:, :2 * ff], ff, torch.bfloat16), B * ff * 10.0, 0)
+    t.op("geglu", lambda: M.glu(work[:, :2 * ff], ff, "gelu", torch.bfloat16), B * ff * 10.0, 0)
     skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), mlp.w_down[:, :ff])
     return t.take()
 

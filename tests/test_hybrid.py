@@ -211,7 +211,7 @@ def test_layer_norms_around_sublayers(run, E):
     close(h, O.layer_norm(x.double() + step.double(), 1e-4, w2.double(), b2.double()), dtype)
     close(y, x.double() + step.double(), torch.float32)
     idx = torch.tensor([3, 1, 3], dtype=torch.int32)
-    close(M.layernorm_rows(x.to(dev), idx.to(dev), *pre, 1e-5, dtype), O.layer_norm(x.double()[[3, 1, 3]], 1e-5, w2.double(), b2.double()), dtype)
+    close(M.norm_rows(x.to(dev), idx.to(dev), *pre, 1e-5, dtype), O.layer_norm(x.double()[[3, 1, 3]], 1e-5, w2.double(), b2.double()), dtype)
 
 
 @pytest.mark.parametrize("T,n,Kd", [(1, 40, 48), (7, 37, 45), (130, 264, 100), (300, 600, 520), (513, 250, 72)])
@@ -221,9 +221,9 @@ def test_gated_feed_forward(run, T, n, Kd):
     pitch = lambda t: torch.nn.functional.pad(t, (0, ops.pad8(Kd) - Kd)).to(dtype).to(dev)[:, :Kd]  # noqa: E731
     z = x.double() @ w.double().T
     want = O.gelu_tanh(z[:, :n]) * z[:, n:]
-    close(M.geglu_linear(pitch(x), pitch(w), n), want, dtype)
+    close(M.glu_linear(pitch(x), pitch(w), n, "gelu"), want, dtype)
     acc = z.float().to(dev)
-    close(M.geglu(acc, n, dtype, dev == "cuda"), want, dtype)
+    close(M.glu(acc, n, "gelu", dtype, dev == "cuda"), want, dtype)
     assert dev == "cpu" or not acc.any()
     # the projection of a parallel layer: a bias on all columns, silu on some
     y = ops.linear(pitch(x), pitch(w), torch.arange(2 * n, device=dev, dtype=torch.float32) / n, "silu", act_cols=(8, ops.pad8(n)))
