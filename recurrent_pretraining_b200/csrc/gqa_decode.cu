@@ -1,12 +1,18 @@
-// Decode attention of grouped-query layers with a learned distance bias: one new token per sequence against its cached keys
-// and values, bf16 matrix units, fp32 softmax.  A decode step is bound by the stream of keys and values, so one warp owns 16
+// Decode attention of grouped-query layers: one new token per sequence against its cached keys and values, bf16 matrix units,
+// fp32 softmax.  Either with a learned distance bias over all cached positions, or (RING) capped scores over the window or the
+// chunk that the sequence's ring holds.  A decode step is bound by the stream of keys and values, so one warp owns 16
 // keys at a time for all heads of a group (padded to the 16 rows of an MMA) and every byte is read once.
 //
 // CTA per (key split, key / value head, sequence), four warps: a warp takes every fourth 16-key tile of the split, staged by
 // cp.async in a ring of its own (no barriers in the loop), and keeps its own running softmax; the warps are joined in shared
 // memory at the end.  The new token's key and value are not in the cache yet: the warp that meets its position forms them
 // from the projection row and appends them.
+//
+// RING: position p lies in slot p % cap.  Queries and the new key are normed over the whole projection and / or rotated, the new
+// value is mixed with another layer's where they are formed.  Bounded scores need no running maximum.  With a single split the
+// sink and the division are applied here.
 #include "rowops.cuh"
+#include "softmax_math.cuh"
 
 namespace b200 {
 
@@ -22,6 +28,15 @@ struct GqaDecode {
   __nv_bfloat16* cache;
   float* part_o;                                   // [B, H, splits, vdim padded to eight], unnormalised
   float* part_ml;                                  // [B, H, splits, 2] (max in natural-log units, sum)
+  // RING
+  int size, chunked;                               // visible: the last `size` positions, or the chunk of `size` positions
+  int rot, ld_first, ld_fout, ld_out;
+  float eps, softcap;                              // softcap 0: scores are not capped
+  const float *q_norm, *k_norm, *cosT, *sinT;      // null: no norm; tables [positions, rot / 2]
+  const float *lam, *first;                        // value mixing: (1 - lam) v + lam first [B, ld_first]; null: none
+  float* first_out;                                // [B, ld_fout] unmixed values; null: not wanted
+  const float* sink;                               // [H]; null: none
+  __nv_bfloat16* out;                              // [B, ld_out] with a single split, else null
 };
 
 constexpr int GD_KEYS = 16, GD_WARPS = 4;
@@ -47,8 +62,22 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 // ldmatrix fall into different banks.
 __host__ __device__ constexpr int gd_pitch(int cols) { return ((cols + 15) & ~15) * 2 + 16; }
 
+// Entry i of a head that is normed (weights w, factor r; null: not) and rotated (halves paired).
+template <typename TI>
+__device__ __forceinline__ float head_entry(const TI* x, int i, const float* w, float r, int rot, const float* ct, const float* st) {
+  float v = ldf(x + i);
+  if (w) v *= r * w[i];
+  if (i < rot) {
+    const int half = rot >> 1, j = i < half ? i : i - half, o = i < half ? i + half : i - half;
+    float u = ldf(x + o);
+    if (w) u *= r * w[o];
+    v = i < half ? v * ct[j] - u * st[j] : v * ct[j] + u * st[j];
+  }
+  return v;
+}
+
 // NV: 16-column steps of the values that the accumulators hold.
-template <typename TI, int NV, int STAGES>
+template <typename TI, int NV, int STAGES, bool RING>
 __global__ void __launch_bounds__(128)
 gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   pdl_trigger();
@@ -58,11 +87,19 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const int split = blockIdx.x, b = blockIdx.z;
   const int group = P.H / P.G, chunks = (group + 15) / 16;
   const int g = blockIdx.y / chunks, h0 = g * group + (blockIdx.y % chunks) * 16, nh = min(16, (g + 1) * group - h0);
-  const int pos = P.pos[b], nkeys = pos + 1;
+  const int pos = P.pos[b];
+  const int key_first = RING ? (P.chunked ? pos - pos % P.size : max(0, pos - P.size + 1)) : 0;
+  const int newest = pos - key_first, nkeys = newest + 1;              // keys are counted from the first visible one
+  const int slot0 = RING ? key_first % P.cap : 0;
+  auto slot_of = [&](int j) {
+    int s = slot0 + j;
+    if (RING && s >= P.cap) s -= P.cap;
+    return s;
+  };
   const int tiles = (nkeys + GD_KEYS - 1) / GD_KEYS, per = (tiles + P.splits - 1) / P.splits;
   const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
   const int vs = (P.vdim + 7) & ~7;
-  if (tile0 >= tile1) {
+  if (tile0 >= tile1) {                                                // not with a single split
     if (threadIdx.x < nh) {
       float* ml = P.part_ml + ((static_cast<size_t>(b) * P.H + h0 + threadIdx.x) * P.splits + split) * 2;
       ml[0] = -INFINITY;
@@ -83,7 +120,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const int kpp = 32 / lpk, lj = lane / lpk, lc = lane % lpk;          // keys per pass, this lane's key and first piece
   auto request = [&](int tile, int st) {
     const uint32_t s = smem_u32(ring + st * stage_bytes);
-    const int last = max(pos - 1, 0);                                  // keys past the newest repeat one that exists; they are masked
+    const int last = max(newest - 1, 0);                               // keys past the newest repeat one that exists; they are masked
     for (int c = lc; c < ch; c += lpk) {
       const bool isk = c < kch;
       const __nv_bfloat16* src = base + (isk ? g * P.dim + 8 * c : P.kv_v + g * P.vdim + 8 * (c - kch));
@@ -91,7 +128,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
       const int pitch = isk ? kp : vp;
 #pragma unroll 8
       for (int j = lj; j < GD_KEYS; j += kpp)
-        cp_async16(dst + j * pitch, src + static_cast<size_t>(min(tile * GD_KEYS + j, last)) * P.ld_kv);
+        cp_async16(dst + j * pitch, src + static_cast<size_t>(slot_of(min(tile * GD_KEYS + j, last))) * P.ld_kv);
     }
   };
   const int first = tile0 + warp;
@@ -101,11 +138,42 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     if (s < mine) request(first + s * GD_WARPS, s);
     cp_commit();
   }
+  float rq = 1.f, rk = 1.f;
+  const float *cos_t = nullptr, *sin_t = nullptr;
+  if constexpr (RING) {
+    cos_t = P.cosT + static_cast<size_t>(pos) * (P.rot >> 1);
+    sin_t = P.sinT + static_cast<size_t>(pos) * (P.rot >> 1);
+    if (P.q_norm) {
+      __shared__ float red[8];
+      const int nq = P.H * P.dim, nk = P.G * P.dim;                    // multiples of eight
+      float sq = 0.f, sk = 0.f;
+      for (int i = 4 * threadIdx.x; i < nq + nk; i += 512) {
+        float v[4];
+        ld4(i < nq ? r + i : r + P.off_k + (i - nq), v);
+        const float t = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+        if (i < nq) sq += t;
+        else sk += t;
+      }
+      sq = warp_sum(sq);
+      sk = warp_sum(sk);
+      if (lane == 0) {
+        red[warp] = sq;
+        red[4 + warp] = sk;
+      }
+      __syncthreads();
+      rq = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / static_cast<float>(nq) + P.eps);
+      rk = 1.f / sqrtf((red[4] + red[5] + red[6] + red[7]) / static_cast<float>(nk) + P.eps);
+    }
+  }
   // queries, zero in the padding rows and columns; the ring's padding columns are zeroed once
   for (int i = threadIdx.x; i < 16 * (kp / 2); i += 128) {
     const int hh = i / (kp / 2), c = i - hh * (kp / 2);
     float v = 0.f;
-    if (hh < nh && c < P.dim) v = ldf(r + (h0 + hh) * P.dim + c) + P.in_bias[(h0 + hh) * P.dim + c];
+    if (hh < nh && c < P.dim) {
+      const int at = (h0 + hh) * P.dim;
+      if constexpr (RING) v = head_entry(r + at, c, P.q_norm ? P.q_norm + at : nullptr, rq, P.rot, cos_t, sin_t);
+      else v = ldf(r + at + c) + P.in_bias[at + c];
+    }
     reinterpret_cast<__nv_bfloat16*>(sq)[i] = f2bf(v);
   }
   for (int i = lane; i < STAGES * GD_KEYS; i += 32) {
@@ -119,13 +187,22 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   // rows of this thread's accumulators: heads lane / 4 and lane / 4 + 8
   const int ra = lane >> 2;
   float rowmul = P.scale * 1.4426950408889634f;
-  if (P.temp_every > 0) rowmul *= query_temperature(pos, P.temp_every, P.temp_coef);
-  const float* bias_row[2];
-#pragma unroll
-  for (int k = 0; k < 2; ++k) bias_row[k] = P.bias + static_cast<size_t>(min(h0 + ra + 8 * k, P.H - 1)) * P.ld_bias + P.bias_lead;
+  if (!RING && P.temp_every > 0) rowmul *= query_temperature(pos, P.temp_every, P.temp_coef);
+  const float* bias_row[2] = {nullptr, nullptr};
+  float bias_far[2] = {0.f, 0.f};
   const int far = P.bias_len - 1;
-  const float bias_far[2] = {bias_row[0][far], bias_row[1][far]};
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if constexpr (!RING) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      bias_row[k] = P.bias + static_cast<size_t>(min(h0 + ra + 8 * k, P.H - 1)) * P.ld_bias + P.bias_lead;
+      bias_far[k] = bias_row[k][far];
+    }
+  }
+  const bool capped = RING && P.softcap > 0.f;
+  const float cap_log2 = P.softcap * 1.4426950408889634f, cap_exp = capped ? 2.f * rowmul / P.softcap : 0.f;
+  const bool bounded = capped && cap_log2 <= 80.f;                     // weights lie in 2^(-80 .. 80): no running maximum
+  const float m_start = bounded ? 0.f : -INFINITY;
+  float m[2] = {m_start, m_start}, l[2] = {0.f, 0.f};
   float o[NV][2][4];
 #pragma unroll
   for (int n = 0; n < NV; ++n)
@@ -148,13 +225,26 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     }
     uint8_t* sb = ring + st * stage_bytes;
     const int key0 = tile * GD_KEYS;
-    if (key0 + GD_KEYS > pos) {                                        // the newest token lies in this tile
-      const int j = pos - key0;
-      __nv_bfloat16* dst = base + static_cast<size_t>(pos) * P.ld_kv;
+    if (key0 + GD_KEYS > newest) {                                     // the newest token lies in this tile
+      const int j = newest - key0;
+      __nv_bfloat16* dst = base + static_cast<size_t>(slot_of(newest)) * P.ld_kv;
+      const float lam = RING && P.lam ? *P.lam : 0.f;
       for (int c = lane; c < P.dim + P.vdim; c += 32) {
         const bool isk = c < P.dim;
         const int cc = isk ? c : c - P.dim, col = isk ? P.off_k + g * P.dim + cc : P.off_v + g * P.vdim + cc;
-        const __nv_bfloat16 v = f2bf(ldf(r + col) + P.in_bias[col]);
+        float f;
+        if constexpr (RING) {
+          if (isk) {
+            f = head_entry(r + P.off_k + g * P.dim, cc, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk, P.rot, cos_t, sin_t);
+          } else {
+            f = ldf(r + col);
+            if (P.first_out) P.first_out[static_cast<size_t>(b) * P.ld_fout + g * P.vdim + cc] = f;
+            if (P.lam) f = (1.f - lam) * f + lam * P.first[static_cast<size_t>(b) * P.ld_first + g * P.vdim + cc];
+          }
+        } else {
+          f = ldf(r + col) + P.in_bias[col];
+        }
+        const __nv_bfloat16 v = f2bf(f);
         reinterpret_cast<__nv_bfloat16*>(sb + (isk ? j * kp : GD_KEYS * kp + j * vp))[cc] = v;
         dst[(isk ? g * P.dim : P.kv_v + g * P.vdim) + cc] = v;
       }
@@ -173,7 +263,17 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     // c[n][0..1]: head ra, keys key0 + 8 n + 2 (lane & 3) + {0, 1}; c[n][2..3]: head ra + 8
     float p[2][4];
     float mx[2] = {-INFINITY, -INFINITY};
-    if (pos - key0 - (GD_KEYS - 1) >= far) {                           // every distance shares the last bucket
+    if constexpr (RING) {
+      const int d0 = newest - key0 - 2 * (lane & 3);
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = capped ? cap_log2 - 2.f * cap_log2 * rcp_approx(1.f + ex2_approx(c[n][e] * cap_exp)) : c[n][e] * rowmul;
+          p[n][e] = d0 - 8 * n - (e & 1) >= 0 ? x : -INFINITY;
+          mx[e >> 1] = fmaxf(mx[e >> 1], p[n][e]);
+        }
+    } else if (pos - key0 - (GD_KEYS - 1) >= far) {                           // every distance shares the last bucket
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -192,17 +292,19 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
           mx[e >> 1] = fmaxf(mx[e >> 1], p[n][e]);
         }
     }
-    float alpha[2];
+    float alpha[2] = {1.f, 1.f};
     bool moved = false;
+    if (!bounded) {
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 1));
-      mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 2));
-      const float mn = fmaxf(m[k], mx[k]);                             // finite: the tile's first key is visible
-      alpha[k] = exp2f(m[k] - mn);
-      moved |= mn != m[k];
-      m[k] = mn;
-      l[k] *= alpha[k];
+      for (int k = 0; k < 2; ++k) {
+        mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 1));
+        mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], 2));
+        const float mn = fmaxf(m[k], mx[k]);                             // finite: the tile's first key is visible
+        alpha[k] = exp2f(m[k] - mn);
+        moved |= mn != m[k];
+        m[k] = mn;
+        l[k] *= alpha[k];
+      }
     }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
@@ -211,7 +313,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
         p[n][e] = exp2f(p[n][e] - m[e >> 1]);
         l[e >> 1] += p[n][e];
       }
-    if (__any_sync(0xffffffffu, moved)) {
+    if (!bounded && __any_sync(0xffffffffu, moved)) {
 #pragma unroll
       for (int n = 0; n < NV; ++n)
 #pragma unroll
@@ -274,6 +376,14 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
       v.x += f * x.x; v.y += f * x.y; v.z += f * x.z; v.w += f * x.w;
       ll += f * sml[(w * 16 + hh) * 2 + 1];
     }
+    if constexpr (RING) {
+      if (P.out) {                                                     // one split: this is all there is
+        const float f = 1.f / (ll + (P.sink ? exp2f(P.sink[h0 + hh] * 1.4426950408889634f - mm) : 0.f));
+        st2(P.out + static_cast<size_t>(b) * P.ld_out + (h0 + hh) * P.vdim + col, make_float2(v.x * f, v.y * f));
+        st2(P.out + static_cast<size_t>(b) * P.ld_out + (h0 + hh) * P.vdim + col + 2, make_float2(v.z * f, v.w * f));
+        continue;
+      }
+    }
     const size_t pi = (static_cast<size_t>(b) * P.H + h0 + hh) * P.splits + split;
     *reinterpret_cast<float4*>(P.part_o + pi * vs + col) = v;
     if (col == 0) {
@@ -304,18 +414,15 @@ B200_API int b200_gqa_decode_per_sm(int dim, int vdim) {
   return n < 1 ? 1 : n > 4 ? 4 : n;
 }
 
-B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
-  const GqaDecode P = *Pp;
-  if (!b200_gqa_decode_supported(P.dim, P.vdim) || B <= 0 || B > 65535 || P.H <= 0 || P.G <= 0 || P.H % P.G || P.splits < 1 || P.splits > 32 ||
-      (P.ld_kv & 7) || (P.kv_v & 7) || P.cap <= 0 || P.bias_len <= 0 || (reinterpret_cast<uintptr_t>(P.cache) & 15)) return -1;
+template <bool RING>
+static int gqa_decode_launch(const void* in, const GqaDecode& P, int B, int in_f32, cudaStream_t st) {
   const int chunks = (P.H / P.G + 15) / 16;
   const dim3 grid(P.splits, P.G * chunks, B);
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
 #define GO2(TI, NV, ST)                                                                                                \
   {                                                                                                                    \
     const int smem = gd_smem<ST>(P.dim, P.vdim);                                                                        \
-    if (cudaFuncSetAttribute(gqa_decode_kernel<TI, NV, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3; \
-    launch_k(gqa_decode_kernel<TI, NV, ST>, grid, dim3(128), smem, st, (const TI*)in, P);                               \
+    if (cudaFuncSetAttribute(gqa_decode_kernel<TI, NV, ST, RING>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3; \
+    launch_k(gqa_decode_kernel<TI, NV, ST, RING>, grid, dim3(128), smem, st, (const TI*)in, P);                         \
   }
 #define GO(TI)                                          \
   {                                                     \
@@ -328,4 +435,23 @@ B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_
 #undef GO
 #undef GO2
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+static bool gqa_decode_ok(const GqaDecode& P, int B) {
+  return b200_gqa_decode_supported(P.dim, P.vdim) && B > 0 && B <= 65535 && P.H > 0 && P.G > 0 && P.H % P.G == 0 && P.splits >= 1 && P.splits <= 32 &&
+         !(P.ld_kv & 7) && !(P.kv_v & 7) && P.cap > 0 && !(reinterpret_cast<uintptr_t>(P.cache) & 15);
+}
+
+B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
+  if (!gqa_decode_ok(*Pp, B) || Pp->bias_len <= 0) return -1;
+  return gqa_decode_launch<false>(in, *Pp, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// The RING form; `out` is written with a single split, the partials otherwise.
+B200_API int b200_ring_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
+  const GqaDecode& P = *Pp;
+  if (!gqa_decode_ok(P, B) || P.size <= 0 || P.rot < 0 || (P.rot & 1) || P.rot > P.dim || (P.rot && (!P.cosT || !P.sinT)) || !P.q_norm != !P.k_norm ||
+      (P.lam && !P.first) || P.softcap < 0.f || (P.ld_in & 7) || (P.off_k & 7) || (reinterpret_cast<uintptr_t>(in) & 15)) return -1;
+  if (P.splits == 1 ? (!P.out || (P.ld_out & 7) || (reinterpret_cast<uintptr_t>(P.out) & 15)) : (P.out || !P.part_o || !P.part_ml)) return -1;
+  return gqa_decode_launch<true>(in, P, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
 }

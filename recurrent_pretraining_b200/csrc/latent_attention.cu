@@ -1,5 +1,6 @@
-// Attention of a packed prompt step of the layered decoder models, on the 5th-generation tensor cores.  Two kinds of layers:
-// sliding-window latent attention, and (BIAS) causal grouped-query attention with a learned bias per head and distance.
+// Attention of a packed prompt step of the layered decoder models, on the 5th-generation tensor cores.  Three kinds of layers:
+// sliding-window latent attention, (BIAS) causal grouped-query attention with a learned bias per head and distance, and (CAPPED)
+// windowed or chunked grouped-query attention with capped scores and an optional sink.
 //
 // Queries [T, H, dim + rot], unrotated keys [K, H, dim] and values [K, H, vdim] (one packed matrix), one rotated key part
 // [K, rot] shared by all heads.  Every size that is a multiple of eight is taken as it is: operand panels are 64 columns
@@ -17,6 +18,11 @@
 // BIAS: keys and values come straight from the cache (key index = row * capacity + position), there is no rotated part, a
 // query's scores carry its temperature and the gate is one number per head.  Blocks whose distances all lie in one bucket
 // add a constant; the others (those near the diagonal) read the bias per element, lanes at consecutive distances.
+//
+// CAPPED: keys and values come from the step's key stream, there is neither a rotated part nor a gate.  A tile lies inside one chunk,
+// so a chunk is nothing but the first key of its tiles.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
+// every score of a warp's block is below the cap, exponential and reciprocal otherwise.  Capped scores are bounded, so (unless the cap is
+// large) the softmax needs no running maximum.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -45,7 +51,13 @@ struct LatentAttnParams {
   int bias_len, ld_bias;
   int temp_every;               // 0: no temperature
   float temp_coef, gate_mult;
+  // CAPPED (and `group`)
+  const float* sink;            // [H] natural-log units; null: none
+  int capped, bounded;          // scores are capped; no running maximum is needed
+  float cap_log2, cap_exp;      // cap in log2 units; exponent of e^(2 score / cap) per raw score, log2 units
+  float cap_poly[6], poly_max;  // capped log2 score = raw * polynomial(raw^2) for |raw| <= poly_max
 };
+enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2 };
 // Columns in front of distance 0 and behind the last stored one (repeating the values there): a block's accesses need no clamps.
 constexpr int LA_BIAS_LEAD = 256, LA_BIAS_TAIL = 256;
 
@@ -69,7 +81,7 @@ struct LatentAttnBars {
 // SN, SR: 16-column MMA steps of the unrotated and rotated parts, known at compile time for common sizes (a block's score
 // product is then a straight line of MMAs: the issuing thread's address arithmetic would otherwise pace the whole block);
 // 0: read from the parameters.
-template <int BN, int SN, int SR, bool BIAS = false>
+template <int BN, int SN, int SR, int KIND = LATENT>
 __global__ void __launch_bounds__(384, 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
                    const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
@@ -90,7 +102,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   volatile int* abort_flag = &bars->abort_flag;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x, hk = BIAS ? h / p.group : h;
+  const int h = blockIdx.x, hk = KIND != LATENT ? h / p.group : h;
   const int4 tile = p.tiles[blockIdx.y];
   const int q0 = tile.x, nrows = tile.y, s0 = tile.z, kbase = tile.w;
   const int kstart = max(kbase, s0 - p.window + 1);
@@ -119,7 +131,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   if (threadIdx.x == 256) {
     tma_prefetch_desc(&tmQn);
     tma_prefetch_desc(&tmKn);
-    if constexpr (!BIAS) {
+    if constexpr (KIND == LATENT) {
       tma_prefetch_desc(&tmQr);
       tma_prefetch_desc(&tmKr);
     }
@@ -187,7 +199,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           while (!mbar_try_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
         }
       }
-    } else if (!BIAS && warp >= 10) {
+    } else if (KIND == LATENT && warp >= 10) {
       // bring the CTA's gate rows into L2 while the blocks are processed
       const int lines = (2 * p.vdim + 127) / 128;
       for (int i = threadIdx.x - 320; i < nrows * lines; i += 64) {
@@ -279,12 +291,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     const uint32_t to = tmem_base + O_COL + x * O_WIDTH + lane_addr;
     float scale_log2 = p.scale_log2;
     const float* btab = nullptr;
-    if constexpr (BIAS) {
+    if constexpr (KIND == BIAS) {
       if (p.temp_every > 0)
         scale_log2 *= 1.f + p.temp_coef * logf(static_cast<float>((kstart + hi - kbase + 1) / p.temp_every + 1));
       btab = p.bias + static_cast<size_t>(h) * p.ld_bias + LA_BIAS_LEAD;
     }
-    float m = -INFINITY, l = 0.f;
+    const bool bounded = KIND == CAPPED && p.bounded;
+    float m = bounded ? 0.f : -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = jb; j < je && ok; ++j) {
       if (!mbar_wait(&bars->s_full[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
@@ -298,14 +311,44 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
       }
       tmem_ld_wait();
+      if constexpr (KIND == CAPPED) {
+        if (p.capped) {
+          float a4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int i = 0; i < BN; i += 8) {
+            a4[0] = fmax3(a4[0], fabsf(sv[i]), fabsf(sv[i + 1]));
+            a4[1] = fmax3(a4[1], fabsf(sv[i + 2]), fabsf(sv[i + 3]));
+            a4[2] = fmax3(a4[2], fabsf(sv[i + 4]), fabsf(sv[i + 5]));
+            a4[3] = fmax3(a4[3], fabsf(sv[i + 6]), fabsf(sv[i + 7]));
+          }
+          if (__all_sync(0xffffffffu, fmaxf(fmaxf(a4[0], a4[1]), fmaxf(a4[2], a4[3])) <= p.poly_max)) {
+            float2 c[6];
+#pragma unroll
+            for (int i = 0; i < 6; ++i) c[i] = make_float2(p.cap_poly[i], p.cap_poly[i]);
+#pragma unroll
+            for (int i = 0; i < BN; i += 2) {
+              const float2 x = make_float2(sv[i], sv[i + 1]), u = fmul2(x, x);
+              float2 y = ffma2(c[5], u, c[4]);
+#pragma unroll
+              for (int k = 3; k >= 0; --k) y = ffma2(y, u, c[k]);
+              y = fmul2(y, x);
+              sv[i] = y.x;
+              sv[i + 1] = y.y;
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < BN; ++i) sv[i] = p.cap_log2 - 2.f * p.cap_log2 * rcp_approx(1.f + ex2_approx(sv[i] * p.cap_exp));
+          }
+        }
+      }
       if (j < j_lo || j >= j_hi) {
         const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
 #pragma unroll
         for (int i = 0; i < BN; ++i)
           if (i < cmin || i > cmax) sv[i] = -INFINITY;
       }
-      float mul = scale_log2, add = 0.f;      // log2 score = mul * sv + add
-      if constexpr (BIAS) {
+      float mul = KIND == CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
+      if constexpr (KIND == BIAS) {
         const int d0 = s0 - kstart + x * LA_BM - j * BN, far = p.bias_len - 1;   // distance of the tile's first row to the block's first key
         const int dmin = d0 - (BN - 1), dmax = d0 + LA_BM - 1;
         if (dmin >= far || (dmin >= 0 && p.bucket[dmin] == p.bucket[min(dmax, far)])) {
@@ -317,35 +360,37 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           mul = 1.f;
         }
       }
-      float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
+      if (!bounded) {
+        float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
-      for (int i = 4; i + 7 < BN; i += 8) {
-        mx4[0] = fmax3(mx4[0], sv[i], sv[i + 1]);
-        mx4[1] = fmax3(mx4[1], sv[i + 2], sv[i + 3]);
-        mx4[2] = fmax3(mx4[2], sv[i + 4], sv[i + 5]);
-        mx4[3] = fmax3(mx4[3], sv[i + 6], sv[i + 7]);
-      }
-      mx4[0] = fmax3(mx4[0], sv[BN - 4], sv[BN - 3]);
-      mx4[1] = fmax3(mx4[1], sv[BN - 2], sv[BN - 1]);
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      const float m_new = fmaxf(m, fmaf(mx, mul, add));
-      // raise the reference max only when it moved by more than the threshold (decided per warp)
-      const bool grow = (m_new - m > RESCALE_THRESHOLD) || (m == -INFINITY);
-      if (__any_sync(0xffffffffu, grow)) {
-        const float alpha = (m == -INFINITY) ? 0.f : ex2_approx(m - m_new);
-        if (j > jb) {
-#pragma unroll 1
-          for (int c = 0; c < p.vdim; c += 32) {
-            uint32_t v[32];
-            tmem_ld_32x32(to + c, v);
-            tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
-            tmem_st_32x32(to + c, v);
-          }
+        for (int i = 4; i + 7 < BN; i += 8) {
+          mx4[0] = fmax3(mx4[0], sv[i], sv[i + 1]);
+          mx4[1] = fmax3(mx4[1], sv[i + 2], sv[i + 3]);
+          mx4[2] = fmax3(mx4[2], sv[i + 4], sv[i + 5]);
+          mx4[3] = fmax3(mx4[3], sv[i + 6], sv[i + 7]);
         }
-        l *= alpha;
-        m = m_new;
+        mx4[0] = fmax3(mx4[0], sv[BN - 4], sv[BN - 3]);
+        mx4[1] = fmax3(mx4[1], sv[BN - 2], sv[BN - 1]);
+        const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+        const float m_new = fmaxf(m, fmaf(mx, mul, add));
+        // raise the reference max only when it moved by more than the threshold (decided per warp)
+        const bool grow = (m_new - m > RESCALE_THRESHOLD) || (m == -INFINITY);
+        if (__any_sync(0xffffffffu, grow)) {
+          const float alpha = (m == -INFINITY) ? 0.f : ex2_approx(m - m_new);
+          if (j > jb) {
+#pragma unroll 1
+            for (int c = 0; c < p.vdim; c += 32) {
+              uint32_t v[32];
+              tmem_ld_32x32(to + c, v);
+              tmem_ld_wait();
+#pragma unroll
+              for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
+              tmem_st_32x32(to + c, v);
+            }
+          }
+          l *= alpha;
+          m = m_new;
+        }
       }
       const float neg_m = (m == -INFINITY) ? 0.f : add - m;   // a row may see nothing of the tile's first blocks
       const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(mul, mul);
@@ -355,7 +400,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         uint32_t packed[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const float2 a = ffma2(make_float2(sv[c + i], sv[c + i + 1]), scale2, neg_m2);
+          float2 a = make_float2(sv[c + i], sv[c + i + 1]);
+          if (!bounded) a = ffma2(a, scale2, neg_m2);
           const float2 pr = make_float2(ex2_approx(a.x), ex2_approx(a.y));
           rs[(i >> 1) & 3] = fadd2(rs[(i >> 1) & 3], pr);
           packed[i >> 1] = pack_bf16x2(pr.x, pr.y);
@@ -376,11 +422,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       const bool live = r < nrows;
       const size_t t = live ? static_cast<size_t>(q0) + r : 0;
       __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
-      if constexpr (BIAS) {
-        const float g = p.gate_mult / (1.f + __expf(-bf2f(p.gate[t * p.ld_gate + h])));
+      if constexpr (KIND != LATENT) {
+        float g = 1.f, den = l;
+        if constexpr (KIND == BIAS) g = p.gate_mult / (1.f + __expf(-bf2f(p.gate[t * p.ld_gate + h])));
+        if constexpr (KIND == CAPPED)
+          if (p.sink) den += ex2_approx(fmaf(p.sink[h], 1.4426950408889634f, -m));
         if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
           tc_fence_after();
-          const float f = (l > 0.f) ? g / l : 0.f;
+          const float f = (l > 0.f) ? g / den : 0.f;
 #pragma unroll 1
           for (int c = 0; c < p.vdim; c += 32) {
             uint32_t v[32];
@@ -502,9 +551,9 @@ static LatentAttnPlan latent_attn_plan(int dim, int rot, int vdim) {
   return none;
 }
 
-template <int BN, int SN, int SR, bool BIAS = false>
+template <int BN, int SN, int SR, int KIND = LATENT>
 static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
-  auto kern = latent_attn_kernel<BN, SN, SR, BIAS>;
+  auto kern = latent_attn_kernel<BN, SN, SR, KIND>;
   static int configured = 0;
   if (configured < plan.smem) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess) return -10;
@@ -524,6 +573,21 @@ static int dispatch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p
   if (sn == 4 && sr == 2) return launch_latent_attn<128, 4, 2>(tm, p, plan, n_tiles, st);   //  64 + 32
   return launch_latent_attn<128, 0, 0>(tm, p, plan, n_tiles, st);
 }
+
+template <int KIND>
+static int dispatch_grouped(const CUtensorMap* tm, const LatentAttnParams& p, const LatentAttnPlan& plan, int n_tiles, cudaStream_t st) {
+  if (plan.bn == 64) return launch_latent_attn<64, 0, 0, KIND>(tm, p, plan, n_tiles, st);
+  switch ((p.dim + 15) / 16) {
+    case 8: return launch_latent_attn<128, 8, 0, KIND>(tm, p, plan, n_tiles, st);
+    case 6: return launch_latent_attn<128, 6, 0, KIND>(tm, p, plan, n_tiles, st);
+    case 4: return launch_latent_attn<128, 4, 0, KIND>(tm, p, plan, n_tiles, st);
+    default: return launch_latent_attn<128, 0, 0, KIND>(tm, p, plan, n_tiles, st);
+  }
+}
+
+// tanh(t) = t sum_i c_i t^(2 i) on |t| <= 1 to 5e-7: interpolation of tanh(sqrt(u)) / sqrt(u) at the Chebyshev nodes of [0, 1].
+static constexpr double TANH_POLY[6] = {0.9999994039535522, -0.3332895040512085, 0.13280721008777618, -0.05158598721027374, 0.016720855608582497,
+                                        -0.0030582291074097157};
 
 }  // namespace b200
 
@@ -592,11 +656,45 @@ B200_API int b200_biased_attention(const void* q, const void* k, const void* v, 
   p.group = H / G; p.bias = bias; p.bucket = bucket; p.bias_len = bias_len; p.ld_bias = ld_bias;
   p.temp_every = temp_every; p.temp_coef = temp_coef; p.gate_mult = gate_mult;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (plan.bn == 64) return launch_latent_attn<64, 0, 0, true>(tm, p, plan, n_tiles, st);
-  switch ((dim + 15) / 16) {
-    case 8: return launch_latent_attn<128, 8, 0, true>(tm, p, plan, n_tiles, st);
-    case 6: return launch_latent_attn<128, 6, 0, true>(tm, p, plan, n_tiles, st);
-    case 4: return launch_latent_attn<128, 4, 0, true>(tm, p, plan, n_tiles, st);
-    default: return launch_latent_attn<128, 0, 0, true>(tm, p, plan, n_tiles, st);
+  return dispatch_grouped<BIAS>(tm, p, plan, n_tiles, st);
+}
+
+B200_API int b200_capped_attention_supported(int dim, int vdim) { return latent_attn_plan(dim, 0, vdim).bn > 0; }
+
+// q: [T, ld_q] (head h at column h dim), k / v: key stream [K, ld_kv] (head g at column g dim / g vdim), out: [T, ld_out]; tiles as in
+// LatentAttnParams, none of them across the border of a chunk (whose first key is the tile's).  window: visible keys.  scale > 0;
+// softcap 0: scores are not capped; sink: [H] or null.
+B200_API int b200_capped_attention(const void* q, const void* k, const void* v, void* out, const int* tiles, const float* sink, int n_tiles, int T,
+                                   int K, int H, int G, int dim, int vdim, int ld_q, int ld_kv, int ld_out, int window, float scale,
+                                   float softcap, void* stream, int* err) {
+  const LatentAttnPlan plan = latent_attn_plan(dim, 0, vdim);
+  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || G <= 0 || H % G || T <= 0 || K <= 0 || window <= 0 || !(scale > 0.f) || softcap < 0.f) return -1;
+  if ((reinterpret_cast<uintptr_t>(out) & 15) || (ld_out & 7)) return -2;
+  CUtensorMap tm[5];
+  int rc = make_tmap_rows(&tm[0], q, dim, H, T, dim, ld_q, LA_BM);
+  if (!rc) rc = make_tmap_rows(&tm[2], k, dim, G, K, dim, ld_kv, plan.bn);
+  if (!rc) rc = make_tmap_rows(&tm[4], v, vdim, G, K, vdim, ld_kv, plan.bn);
+  if (rc) return rc;
+  tm[1] = tm[0];
+  tm[3] = tm[2];
+  LatentAttnParams p = {};
+  p.H = H; p.dim = dim; p.rot = 0; p.vdim = vdim; p.window = window;
+  p.pn = (dim + 63) / 64; p.pr = 0; p.pv = (vdim + 63) / 64;
+  p.kst = plan.kst; p.vst = plan.vst;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.tiles = reinterpret_cast<const int4*>(tiles);
+  p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
+  p.err = err;
+  p.group = H / G; p.sink = sink;
+  if (softcap > 0.f) {
+    const double x = static_cast<double>(scale) / softcap, cap = softcap * 1.4426950408889634;
+    p.capped = 1;
+    p.bounded = cap <= 80.0;            // weights lie in 2^(-80 .. 80): sums and products stay far inside fp32
+    p.cap_log2 = static_cast<float>(cap);
+    p.cap_exp = static_cast<float>(2.0 * x * 1.4426950408889634);
+    double f = cap * x;                 // cap x^(2 i + 1)
+    for (int i = 0; i < 6; ++i, f *= x * x) p.cap_poly[i] = static_cast<float>(TANH_POLY[i] * f);
+    p.poly_max = x > 5e-4 && x < 1e3 ? static_cast<float>(1.0 / x) : -1.f;      // coefficients inside the range of fp32
   }
+  return dispatch_grouped<CAPPED>(tm, p, plan, n_tiles, reinterpret_cast<cudaStream_t>(stream));
 }

@@ -195,13 +195,16 @@ def ring_attention_pieces(L: GroupedLayout, a, inp, tr: QkvTransform, cache, sin
     part_o = torch.empty(B, L.heads, splits, pad8(L.vdim), dtype=F32, device=inp.device)
     part_ml = torch.empty(B, L.heads, splits, 2, dtype=F32, device=inp.device)
 
-    def attend():
-        if dtype == BF16:
-            from . import grouped_kernels as GK
+    fused = False
+    if dtype == BF16:
+        from . import grouped_kernels as GK
 
-            if GK.decode_supported(L):
-                GK.decode_attention(L, a, inp, tr, cache, first_out, pos, row, part_o, part_ml)
-                return
+        fused = GK.decode_supported(L)
+
+    def attend():
+        if fused:
+            GK.decode_attention(L, a, inp, tr, cache, sink, first_out, pos, row, part_o, part_ml, out)
+            return
         q = torch.empty(B, pad8(L.heads * L.dim), dtype=dtype, device=inp.device)
         s = _row_struct(L, inp, tr, q.stride(0), cap, first_out, pos, row)
         k.K._check(k.prep(inp.data_ptr(), q.data_ptr(), p(tr.first), p(first_out), cache.data_ptr(), 0, C.byref(s), B, _f32(inp), int(dtype == F32), 1,
@@ -213,6 +216,8 @@ def ring_attention_pieces(L: GroupedLayout, a, inp, tr: QkvTransform, cache, sin
                    "window_attention")
 
     def merge():
+        if fused and splits == 1:
+            return                                             # done by the attention itself
         k.K._check(k.merge(part_o.data_ptr(), part_ml.data_ptr(), p(sink), out.data_ptr(), out.stride(0), B, L.heads, L.vdim, splits, _f32(out),
                            k.K._stream()), "attention_merge")
 

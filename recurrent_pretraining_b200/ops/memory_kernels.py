@@ -16,7 +16,9 @@ _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
 class _GqaDecode(C.Structure):
     _fields_ = [(n, _i) for n in ("H", "G", "dim", "vdim", "ld_in", "off_k", "off_v", "ld_kv", "kv_v", "cap", "splits", "bias_len", "ld_bias",
                                   "bias_lead", "temp_every")] + [(n, _f) for n in ("temp_coef", "scale")] + \
-               [(n, _vp) for n in ("in_bias", "bias", "pos", "row", "cache", "part_o", "part_ml")]
+               [(n, _vp) for n in ("in_bias", "bias", "pos", "row", "cache", "part_o", "part_ml")] + \
+               [(n, _i) for n in ("size", "chunked", "rot", "ld_first", "ld_fout", "ld_out")] + [(n, _f) for n in ("eps", "softcap")] + \
+               [(n, _vp) for n in ("q_norm", "k_norm", "cosT", "sinT", "lam", "first", "first_out", "sink", "out")]
 
 
 class _Chunks(C.Structure):
