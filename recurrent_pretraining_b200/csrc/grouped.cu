@@ -148,14 +148,20 @@ attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict
   const float w = e.x == -INFINITY ? 0.f : expf(e.x - m);
   const float mine = w / (warp_sum(w * e.y) + (sink ? expf(sk - m) : 0.f));
   const float* p = part_o + static_cast<size_t>(i) * splits * vs;
-  for (int d0 = 0; d0 < vdim; d0 += 32) {                       // uniform over the warp
-    const int d = d0 + lane;
-    float o = 0.f;
+  for (int d0 = 0; d0 < vdim; d0 += 128) {                      // uniform over the warp
+    const int d = d0 + 4 * lane;
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
     for (int s = 0; s < splits; ++s) {
       const float f = __shfl_sync(0xffffffffu, mine, s);
-      if (f != 0.f && d < vdim) o += f * p[static_cast<size_t>(s) * vs + d];   // an empty split's partial is not initialised
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (d < vs) ld4(p + static_cast<size_t>(s) * vs + d, x);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) o[k] += f != 0.f ? f * x[k] : 0.f;   // an empty split's partial is not initialised
     }
-    if (d < vdim) stf(out + static_cast<size_t>(b) * ld_out + h * vdim + d, o);
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (d + k < vdim) stf(out + static_cast<size_t>(b) * ld_out + h * vdim + d + k, o[k]);
   }
 }
 

@@ -21,9 +21,16 @@
 //
 // CAPPED: keys and values come from the step's key stream, there is neither a rotated part nor a gate.  A tile lies inside one chunk,
 // so a chunk is nothing but the first key of its tiles.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
-// every score of a warp's block is below the cap, exponential and reciprocal otherwise.  Capped scores are bounded, so (unless the cap is
-// large) the softmax needs no running maximum.
+// every score of a warp's columns is well below the cap, exponential and reciprocal otherwise.
+//
+// BOUNDED: CAPPED with a cap that is not large.  The softmax needs no running maximum and takes its columns as they come, and a query
+// row is shared by two threads: sixteen softmax warps, each with half of a block's columns and its weights over its own half of the
+// scores.
 #include <cuda.h>
+
+#include <type_traits>
+
+#include <type_traits>
 
 #include "common.cuh"
 #include "softmax_math.cuh"
@@ -53,13 +60,46 @@ struct LatentAttnParams {
   float temp_coef, gate_mult;
   // CAPPED (and `group`)
   const float* sink;            // [H] natural-log units; null: none
-  int capped, bounded;          // scores are capped; no running maximum is needed
+  int capped;                   // scores are capped
   float cap_log2, cap_exp;      // cap in log2 units; exponent of e^(2 score / cap) per raw score, log2 units
-  float cap_poly[6], poly_max;  // capped log2 score = raw * polynomial(raw^2) for |raw| <= poly_max
+  float cap_poly[3], poly_max;  // capped log2 score = raw * polynomial(raw^2) for |raw| <= poly_max
 };
-enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2 };
+enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2, BOUNDED = 3 };
+__host__ __device__ constexpr int la_softmax_warps(int kind) { return kind == BOUNDED ? 16 : 8; }
+__host__ __device__ constexpr int la_threads(int kind) { return 32 * (la_softmax_warps(kind) + 4); }
 // Columns in front of distance 0 and behind the last stored one (repeating the values there): a block's accesses need no clamps.
 constexpr int LA_BIAS_LEAD = 256, LA_BIAS_TAIL = 256;
+
+// The wait names the registers of the load: nothing that reads them moves in front of it.
+__device__ __forceinline__ void tmem_ld_wait(uint32_t (&v)[32]) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]), "+r"(v[9]), "+r"(v[10]),
+                 "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15]), "+r"(v[16]), "+r"(v[17]), "+r"(v[18]), "+r"(v[19]), "+r"(v[20]),
+                 "+r"(v[21]), "+r"(v[22]), "+r"(v[23]), "+r"(v[24]), "+r"(v[25]), "+r"(v[26]), "+r"(v[27]), "+r"(v[28]), "+r"(v[29]), "+r"(v[30]),
+                 "+r"(v[31])::"memory");
+}
+// Largest magnitude among N values.
+template <int N>
+__device__ __forceinline__ float max_abs(const float (&v)[N]) {
+  float a4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < N; i += 8) {
+    a4[0] = fmax3(a4[0], fabsf(v[i]), fabsf(v[i + 1]));
+    a4[1] = fmax3(a4[1], fabsf(v[i + 2]), fabsf(v[i + 3]));
+    a4[2] = fmax3(a4[2], fabsf(v[i + 4]), fabsf(v[i + 5]));
+    a4[3] = fmax3(a4[3], fabsf(v[i + 6]), fabsf(v[i + 7]));
+  }
+  return fmaxf(fmaxf(a4[0], a4[1]), fmaxf(a4[2], a4[3]));
+}
+// Raw score -> capped score in log2 units: small raw scores (two at a time) / any.
+__device__ __forceinline__ float2 cap_small(float2 x, const LatentAttnParams& p) {
+  const float2 u = fmul2(x, x);
+  return fmul2(ffma2(ffma2(make_float2(p.cap_poly[2], p.cap_poly[2]), u, make_float2(p.cap_poly[1], p.cap_poly[1])), u,
+                     make_float2(p.cap_poly[0], p.cap_poly[0])), x);
+}
+__device__ __forceinline__ float cap_any(float x, const LatentAttnParams& p) {
+  return p.cap_log2 - 2.f * p.cap_log2 * rcp_approx(1.f + ex2_approx(x * p.cap_exp));
+}
 
 // Position in a ring of `n` stages: stage index and the parity of the pass over the ring.
 struct RingPos {
@@ -82,7 +122,7 @@ struct LatentAttnBars {
 // product is then a straight line of MMAs: the issuing thread's address arithmetic would otherwise pace the whole block);
 // 0: read from the parameters.
 template <int BN, int SN, int SR, int KIND = LATENT>
-__global__ void __launch_bounds__(384, 1)
+__global__ void __launch_bounds__(la_threads(KIND), 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
                    const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
                    const __grid_constant__ CUtensorMap tmV, const LatentAttnParams p) {
@@ -90,6 +130,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   constexpr uint32_t IDESC_S = make_idesc_bf16(LA_BM, BN, 0, 0);
   constexpr int O_COL = 2 * BN, O_WIDTH = (512 - 2 * BN) / 2;
   constexpr float RESCALE_THRESHOLD = 8.f;   // log2 units
+  constexpr int WARPS = la_softmax_warps(KIND), SPLIT = WARPS / 8;   // SPLIT: threads per query row
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -128,7 +169,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   };
 
   // the TMA thread sets up the barriers and requests the queries and the first key block before the CTA-wide sync
-  if (threadIdx.x == 256) {
+  if (threadIdx.x == 32 * WARPS) {
     tma_prefetch_desc(&tmQn);
     tma_prefetch_desc(&tmKn);
     if constexpr (KIND == LATENT) {
@@ -145,7 +186,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bars->q_full[i], 1);
       mbar_init(&bars->s_full[i], 1);
-      mbar_init(&bars->p_ready[i], 4);
+      mbar_init(&bars->p_ready[i], 4 * SPLIT);
       mbar_init(&bars->o_final[i], 1);
     }
     bars->abort_flag = 0;
@@ -155,7 +196,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     load_k(0, 0);
     load_q(1);
   }
-  if (warp == 9) {
+  if (warp == WARPS + 1) {
     tmem_alloc(&bars->tmem_slot, 512);
     tmem_relinquish();
   }
@@ -164,9 +205,9 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   tc_fence_after();
   const uint32_t tmem_base = bars->tmem_slot;
 
-  if (warp >= 8) {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 72;");
-    if (warp == 8) {
+  if (warp >= WARPS) {
+    if constexpr (SPLIT == 1) asm volatile("setmaxnreg.dec.sync.aligned.u32 72;");
+    if (warp == WARPS) {
       if (lane == 0) {
         int issued = 1;
         RingPos k;
@@ -199,14 +240,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           while (!mbar_try_wait(&bars->v_full[j % p.vst], (j / p.vst) & 1) && globaltimer_ns() - t0 < WAIT_LIMIT_NS) {}
         }
       }
-    } else if (KIND == LATENT && warp >= 10) {
+    } else if (KIND == LATENT && warp >= WARPS + 2) {
       // bring the CTA's gate rows into L2 while the blocks are processed
       const int lines = (2 * p.vdim + 127) / 128;
       for (int i = threadIdx.x - 320; i < nrows * lines; i += 64) {
         const char* g = reinterpret_cast<const char*>(p.gate + static_cast<size_t>(q0 + i / lines) * p.ld_gate + h * p.vdim) + (i % lines) * 128;
         asm volatile("prefetch.global.L2 [%0];" ::"l"(g));
       }
-    } else if (warp == 9) {
+    } else if (warp == WARPS + 1) {
       if (lane == 0) {
         const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV);
         const uint32_t idesc_o = make_idesc_bf16(LA_BM, (p.vdim + 15) & ~15, 0, 1);
@@ -238,11 +279,12 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           }
           umma_commit(&bars->s_full[x]);
         };
-        auto issue_pv = [&](int x, int vs, bool first) {   // O_x += P_x V (stage vs), P_x over the first BN / 2 columns of S_x
+        auto issue_pv = [&](int x, int vs, bool first) {   // O_x += P_x V (stage vs), P_x over the first half of (every part of) S_x
           const uint64_t vd = dv0 + ((vs * v_bytes) >> 4);
           const uint32_t d = tmem_base + O_COL + x * O_WIDTH, a = tmem_base + x * BN;
 #pragma unroll
-          for (int t = 0; t < BN / 16; ++t) umma_bf16_ts(d, a + t * 8, vd + t * 128, idesc_o, (first && t == 0) ? 0u : 1u);
+          for (int t = 0; t < BN / 16; ++t)
+            umma_bf16_ts(d, a + t * 8 + (t * 16 / (BN / SPLIT)) * (BN / SPLIT / 2), vd + t * 128, idesc_o, (first && t == 0) ? 0u : 1u);
         };
         bool ok = mbar_wait(&bars->q_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN) &&
                   mbar_wait(&bars->k_full[0], 0, abort_flag, p.err, ERR_WAIT_ATTN);
@@ -278,8 +320,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       }
     }
   } else {
-    asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");
-    const int x = warp >> 2;
+    if constexpr (SPLIT == 1) asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");
+    const int x = warp / (4 * SPLIT), part = (warp >> 2) % SPLIT;   // tile, part of its columns
     const int quad = warp & 3;
     const int jb = x ? jb1 : 0, je = x ? je1 : je0;
     // blocks [j_lo, j_hi) are visible to every row of the tile; the others are masked
@@ -296,71 +338,99 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         scale_log2 *= 1.f + p.temp_coef * logf(static_cast<float>((kstart + hi - kbase + 1) / p.temp_every + 1));
       btab = p.bias + static_cast<size_t>(h) * p.ld_bias + LA_BIAS_LEAD;
     }
-    const bool bounded = KIND == CAPPED && p.bounded;
-    float m = bounded ? 0.f : -INFINITY, l = 0.f;
+    float m = KIND == BOUNDED ? 0.f : -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = jb; j < je && ok; ++j) {
       if (!mbar_wait(&bars->s_full[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
       tc_fence_after();
-      float sv[BN];
+      if constexpr (KIND == BOUNDED) {        // 32 columns at a time: no maximum to wait for
+        const bool edge = j < j_lo || j >= j_hi;
+        const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
+        float2 rs = make_float2(0.f, 0.f);
+        constexpr int COLS = BN / SPLIT;
 #pragma unroll
-      for (int c = 0; c < BN; c += 32) {
-        uint32_t v[32];
-        tmem_ld_32x32(ts + c, v);
+        for (int c0 = 0; c0 < COLS; c0 += 32) {
+          const int c = part * COLS + c0;
+          uint32_t raw[32], packed[16];
+          tmem_ld_32x32(ts + c, raw);
+          tmem_ld_wait(raw);
+          float sv[32];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
-      }
-      tmem_ld_wait();
-      if constexpr (KIND == CAPPED) {
-        if (p.capped) {
-          float a4[4] = {0.f, 0.f, 0.f, 0.f};
+          for (int i = 0; i < 32; ++i) sv[i] = __uint_as_float(raw[i]);
+          float2 r2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+          auto weigh = [&](auto cap, auto masked) {
+            r2[0] = r2[1] = make_float2(0.f, 0.f);
 #pragma unroll
-          for (int i = 0; i < BN; i += 8) {
-            a4[0] = fmax3(a4[0], fabsf(sv[i]), fabsf(sv[i + 1]));
-            a4[1] = fmax3(a4[1], fabsf(sv[i + 2]), fabsf(sv[i + 3]));
-            a4[2] = fmax3(a4[2], fabsf(sv[i + 4]), fabsf(sv[i + 5]));
-            a4[3] = fmax3(a4[3], fabsf(sv[i + 6]), fabsf(sv[i + 7]));
+            for (int i = 0; i < 32; i += 2) {
+              float2 y = cap(i);
+              if constexpr (decltype(masked)::value) {
+                if (c + i < cmin || c + i > cmax) y.x = -INFINITY;
+                if (c + i + 1 < cmin || c + i + 1 > cmax) y.y = -INFINITY;
+              }
+              const float2 pr = make_float2(ex2_approx(y.x), ex2_approx(y.y));
+              r2[(i >> 1) & 1] = fadd2(r2[(i >> 1) & 1], pr);
+              packed[i >> 1] = pack_bf16x2(pr.x, pr.y);
+            }
+          };
+          auto small = [&](int i) { return cap_small(make_float2(sv[i], sv[i + 1]), p); };
+          if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
+            if (edge) weigh(small, std::true_type());
+            else weigh(small, std::false_type());
+          } else {
+            weigh([&](int i) { return make_float2(cap_any(sv[i], p), cap_any(sv[i + 1], p)); }, std::true_type());
           }
-          if (__all_sync(0xffffffffu, fmaxf(fmaxf(a4[0], a4[1]), fmaxf(a4[2], a4[3])) <= p.poly_max)) {
-            float2 c[6];
+          rs = fadd2(rs, fadd2(r2[0], r2[1]));
+          tmem_st_32x16(ts + part * (COLS / 2) + (c >> 1), packed);
+        }
+        l += rs.x + rs.y;
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&bars->p_ready[x]);
+      } else {
+        float sv[BN];
 #pragma unroll
-            for (int i = 0; i < 6; ++i) c[i] = make_float2(p.cap_poly[i], p.cap_poly[i]);
+        for (int c = 0; c < BN; c += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32(ts + c, v);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
+        }
+        tmem_ld_wait();
+        if constexpr (KIND == CAPPED) {
+          if (p.capped) {
+          if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
 #pragma unroll
             for (int i = 0; i < BN; i += 2) {
-              const float2 x = make_float2(sv[i], sv[i + 1]), u = fmul2(x, x);
-              float2 y = ffma2(c[5], u, c[4]);
-#pragma unroll
-              for (int k = 3; k >= 0; --k) y = ffma2(y, u, c[k]);
-              y = fmul2(y, x);
+              const float2 y = cap_small(make_float2(sv[i], sv[i + 1]), p);
               sv[i] = y.x;
               sv[i + 1] = y.y;
             }
           } else {
 #pragma unroll
-            for (int i = 0; i < BN; ++i) sv[i] = p.cap_log2 - 2.f * p.cap_log2 * rcp_approx(1.f + ex2_approx(sv[i] * p.cap_exp));
+            for (int i = 0; i < BN; ++i) sv[i] = cap_any(sv[i], p);
           }
         }
-      }
-      if (j < j_lo || j >= j_hi) {
-        const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
-#pragma unroll
-        for (int i = 0; i < BN; ++i)
-          if (i < cmin || i > cmax) sv[i] = -INFINITY;
-      }
-      float mul = KIND == CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
-      if constexpr (KIND == BIAS) {
-        const int d0 = s0 - kstart + x * LA_BM - j * BN, far = p.bias_len - 1;   // distance of the tile's first row to the block's first key
-        const int dmin = d0 - (BN - 1), dmax = d0 + LA_BM - 1;
-        if (dmin >= far || (dmin >= 0 && p.bucket[dmin] == p.bucket[min(dmax, far)])) {
-          add = btab[min(dmin, far)];
-        } else {
-          const float* b = btab + (hi - j * BN);
-#pragma unroll
-          for (int i = 0; i < BN; ++i) sv[i] = fmaf(sv[i], scale_log2, b[-i]);
-          mul = 1.f;
         }
-      }
-      if (!bounded) {
+        if (j < j_lo || j >= j_hi) {
+          const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
+#pragma unroll
+          for (int i = 0; i < BN; ++i)
+            if (i < cmin || i > cmax) sv[i] = -INFINITY;
+        }
+        float mul = KIND == CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
+        if constexpr (KIND == BIAS) {
+          const int d0 = s0 - kstart + x * LA_BM - j * BN, far = p.bias_len - 1;   // distance of the tile's first row to the block's first key
+          const int dmin = d0 - (BN - 1), dmax = d0 + LA_BM - 1;
+          if (dmin >= far || (dmin >= 0 && p.bucket[dmin] == p.bucket[min(dmax, far)])) {
+            add = btab[min(dmin, far)];
+          } else {
+            const float* b = btab + (hi - j * BN);
+#pragma unroll
+            for (int i = 0; i < BN; ++i) sv[i] = fmaf(sv[i], scale_log2, b[-i]);
+            mul = 1.f;
+          }
+        }
         float mx4[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
         for (int i = 4; i + 7 < BN; i += 8) {
@@ -391,31 +461,38 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           l *= alpha;
           m = m_new;
         }
-      }
-      const float neg_m = (m == -INFINITY) ? 0.f : add - m;   // a row may see nothing of the tile's first blocks
-      const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(mul, mul);
-      float2 rs[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+        const float neg_m = (m == -INFINITY) ? 0.f : add - m;   // a row may see nothing of the tile's first blocks
+        const float2 neg_m2 = make_float2(neg_m, neg_m), scale2 = make_float2(mul, mul);
+        float2 rs[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
-      for (int c = 0; c < BN; c += 32) {
-        uint32_t packed[16];
+        for (int c = 0; c < BN; c += 32) {
+          uint32_t packed[16];
 #pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-          float2 a = make_float2(sv[c + i], sv[c + i + 1]);
-          if (!bounded) a = ffma2(a, scale2, neg_m2);
-          const float2 pr = make_float2(ex2_approx(a.x), ex2_approx(a.y));
-          rs[(i >> 1) & 3] = fadd2(rs[(i >> 1) & 3], pr);
-          packed[i >> 1] = pack_bf16x2(pr.x, pr.y);
+          for (int i = 0; i < 32; i += 2) {
+            const float2 a = ffma2(make_float2(sv[c + i], sv[c + i + 1]), scale2, neg_m2);
+            const float2 pr = make_float2(ex2_approx(a.x), ex2_approx(a.y));
+            rs[(i >> 1) & 3] = fadd2(rs[(i >> 1) & 3], pr);
+            packed[i >> 1] = pack_bf16x2(pr.x, pr.y);
+          }
+          tmem_st_32x16(ts + (c >> 1), packed);
         }
-        tmem_st_32x16(ts + (c >> 1), packed);
+        {
+          const float2 t = fadd2(fadd2(rs[0], rs[1]), fadd2(rs[2], rs[3]));
+          l += t.x + t.y;
+        }
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&bars->p_ready[x]);
       }
-      {
-        const float2 t = fadd2(fadd2(rs[0], rs[1]), fadd2(rs[2], rs[3]));
-        l += t.x + t.y;
+    }
+    if constexpr (SPLIT == 2) {
+      if (je > jb) {                          // the row's other half of the sum, through the tile's queries: its last scores are formed
+        float* sums = reinterpret_cast<float*>(sQ + x * q_bytes) + quad * 32 + lane;
+        sums[part * LA_BM] = l;
+        named_barrier_sync(1 + x, 256);
+        l += sums[(part ^ 1) * LA_BM];
       }
-      tmem_st_wait();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&bars->p_ready[x]);
     }
     if (ok && je > jb) {
       const int r = x * LA_BM + quad * 32 + lane;              // query of this thread inside the CTA's 256
@@ -425,13 +502,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       if constexpr (KIND != LATENT) {
         float g = 1.f, den = l;
         if constexpr (KIND == BIAS) g = p.gate_mult / (1.f + __expf(-bf2f(p.gate[t * p.ld_gate + h])));
-        if constexpr (KIND == CAPPED)
+        if constexpr (KIND >= CAPPED)
           if (p.sink) den += ex2_approx(fmaf(p.sink[h], 1.4426950408889634f, -m));
         if (mbar_wait(&bars->o_final[x], 0, abort_flag, p.err, ERR_WAIT_ATTN)) {
           tc_fence_after();
           const float f = (l > 0.f) ? g / den : 0.f;
 #pragma unroll 1
-          for (int c = 0; c < p.vdim; c += 32) {
+          for (int c = 32 * part; c < p.vdim; c += 32 * SPLIT) {
             uint32_t v[32];
             tmem_ld_32x32(to + c, v);
             tmem_ld_wait();
@@ -496,7 +573,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 9) {
+  if (warp == WARPS + 1) {
     __syncwarp();
     tc_fence_after();
     tmem_dealloc(tmem_base, 512);
@@ -559,7 +636,7 @@ static int launch_latent_attn(const CUtensorMap* tm, const LatentAttnParams& p, 
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess) return -10;
     configured = plan.smem;
   }
-  kern<<<dim3(p.H, n_tiles), 384, plan.smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  kern<<<dim3(p.H, n_tiles), la_threads(KIND), plan.smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
@@ -585,9 +662,8 @@ static int dispatch_grouped(const CUtensorMap* tm, const LatentAttnParams& p, co
   }
 }
 
-// tanh(t) = t sum_i c_i t^(2 i) on |t| <= 1 to 5e-7: interpolation of tanh(sqrt(u)) / sqrt(u) at the Chebyshev nodes of [0, 1].
-static constexpr double TANH_POLY[6] = {0.9999994039535522, -0.3332895040512085, 0.13280721008777618, -0.05158598721027374, 0.016720855608582497,
-                                        -0.0030582291074097157};
+// tanh(t) = t (c0 + c1 t^2 + c2 t^4) on |t| <= 0.3 to 4e-7: interpolation of tanh(sqrt(u)) / sqrt(u) at Chebyshev nodes of [0, 0.09].
+static constexpr double TANH_RANGE = 0.3, TANH_POLY[3] = {0.9999988351, -0.3330998880, 0.1263358239};
 
 }  // namespace b200
 
@@ -686,15 +762,17 @@ B200_API int b200_capped_attention(const void* q, const void* k, const void* v, 
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
   p.err = err;
   p.group = H / G; p.sink = sink;
+  bool bounded = false;
   if (softcap > 0.f) {
     const double x = static_cast<double>(scale) / softcap, cap = softcap * 1.4426950408889634;
     p.capped = 1;
-    p.bounded = cap <= 80.0;            // weights lie in 2^(-80 .. 80): sums and products stay far inside fp32
+    bounded = cap <= 80.0;              // weights lie in 2^(-80 .. 80): sums and products stay far inside fp32
     p.cap_log2 = static_cast<float>(cap);
     p.cap_exp = static_cast<float>(2.0 * x * 1.4426950408889634);
     double f = cap * x;                 // cap x^(2 i + 1)
-    for (int i = 0; i < 6; ++i, f *= x * x) p.cap_poly[i] = static_cast<float>(TANH_POLY[i] * f);
-    p.poly_max = x > 5e-4 && x < 1e3 ? static_cast<float>(1.0 / x) : -1.f;      // coefficients inside the range of fp32
+    for (int i = 0; i < 3; ++i, f *= x * x) p.cap_poly[i] = static_cast<float>(TANH_POLY[i] * f);
+    p.poly_max = x > 1e-6 && x < 1e6 ? static_cast<float>(TANH_RANGE / x) : -1.f;   // coefficients inside the range of fp32
   }
-  return dispatch_grouped<CAPPED>(tm, p, plan, n_tiles, reinterpret_cast<cudaStream_t>(stream));
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return bounded ? dispatch_grouped<BOUNDED>(tm, p, plan, n_tiles, st) : dispatch_grouped<CAPPED>(tm, p, plan, n_tiles, st);
 }

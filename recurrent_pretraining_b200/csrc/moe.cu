@@ -1,5 +1,5 @@
 // Mixture-of-experts feed-forward around the grouped matrix products:
-//   * moe_router_logits : narrow fp32 product of a decode step's rows with the router
+//   * moe_router_logits : product of a decode step's rows with the router, fp32 operands
 //   * moe_route         : softmax over the router outputs, choice of the best ones (scores plus correction), normalised weights,
 //                         rank of every choice inside its expert
 //   * moe_plan          : first slot of every expert (rows padded to whole tiles), expert of every tile
@@ -72,7 +72,7 @@ __device__ __forceinline__ void route_token(const RouteArgs& R, const float* z, 
   if (lane == 0) R.weight[t * (R.top + 1) + R.top] = R.gate ? sigmoid_f(z[R.outputs]) : 0.f;
 }
 
-// z[b, r] = x[b] . w[r]: CTA per router output
+// z[b, r] = x[b] . w[r]: CTA per router output (fp32 operands; bf16 ones go through moe_rows)
 template <typename T>
 __global__ void __launch_bounds__(128)
 moe_router_logits_kernel(const T* __restrict__ x, int ld_x, const T* __restrict__ w, int ld_w, float* __restrict__ z, int ld_z, int B, int E) {
@@ -98,14 +98,14 @@ moe_router_logits_kernel(const T* __restrict__ x, int ld_x, const T* __restrict_
   }
 }
 
-// Eight warps, four tokens each: choices are ranked inside their expert first within the CTA, then across CTAs.
+// Eight warps, `per` tokens: choices are ranked inside their expert first within the CTA, then across CTAs.
 __global__ void __launch_bounds__(256)
-moe_route_kernel(const float* __restrict__ z, const RouteArgs R, int* __restrict__ count, int* __restrict__ rank, int T) {
+moe_route_kernel(const float* __restrict__ z, const RouteArgs R, int* __restrict__ count, int* __restrict__ rank, int T, int per) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5;
   int* hist = reinterpret_cast<int*>(sm + 16 * R.outputs);       // [experts]: choices of this CTA, then their first rank
   for (int i = threadIdx.x; i < R.experts; i += 256) hist[i] = 0;
-  const int t0 = blockIdx.x * 32, n = min(32, T - t0);
+  const int t0 = blockIdx.x * per, n = min(per, T - t0);
   for (int j = warp; j < n; j += 8)
     route_token(R, z + static_cast<size_t>(t0 + j) * R.ld_z, t0 + j, sm + 2 * warp * R.outputs, sm + (2 * warp + 1) * R.outputs);
   __syncthreads();
@@ -241,11 +241,6 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ uint4 ld_stream(const void* p) {
-  uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-  return v;
-}
 // keep the first n of eight bf16 values
 __device__ __forceinline__ uint4 keep8(uint4 v, int n) {
   uint32_t* w = reinterpret_cast<uint32_t*>(&v);
@@ -254,34 +249,45 @@ __device__ __forceinline__ uint4 keep8(uint4 v, int n) {
   return v;
 }
 
-// CTA: (32 weight rows, chosen expert): two groups of 16 rows x four ranges of K.  The order of the terms of a dot product is free, so
-// a lane takes eight neighbouring columns of its weight rows and of its token as they lie in memory: they serve two MMAs.
-// NT: groups of eight tokens.
-constexpr int ER_ROWS = 32, ER_KW = 4;
-template <typename TO, int NT>
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ void cp_async16_zfill(uint32_t dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// CTA: (16 RG weight rows, chosen expert): RG groups of 16 rows x KW ranges of K, one warp each.  The order of the terms of a dot
+// product is free, so a lane takes eight neighbouring columns of its weight rows and of its token as they lie in memory: they
+// serve two MMAs.  The weights pass through a queue in shared memory that belongs to the thread alone (ER_DEPTH steps of 32 columns in
+// flight, no barriers).  NT: groups of eight tokens; more tokens take more rows per CTA, which share the tokens' way from L2.
+constexpr int ER_DEPTH = 8;
+template <typename TO, int NT, int RG, int KW>
+__global__ void __launch_bounds__(256, NT >= 8 ? 2 : 3)
 moe_rows_kernel(const ExpertRows P) {
+  static_assert(RG * KW == 8, "eight warps");
   pdl_trigger();
-  __shared__ float part[ER_KW - 1][2][16][8 * NT + 1];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = warp & 1, kw = warp >> 1;
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = warp % RG, kw = warp / RG;
   pdl_wait();
-  const bool shared = P.Ns > 0 && blockIdx.y == gridDim.y - 1;
+  const int shared = P.Ns > 0 ? 1 : 0;
+  const bool mine = shared && blockIdx.y == 0;                // the shared expert, which has the most rows, goes first
   int e = 0, s0 = 0, n = P.B;
-  if (!shared) {
-    if (static_cast<int>(blockIdx.y) >= *P.n_active) return;
-    e = P.active[blockIdx.y];
-    s0 = P.first[blockIdx.y];
-    n = P.first[blockIdx.y + 1] - s0;
+  if (!mine) {
+    const int y = blockIdx.y - shared;
+    if (y >= *P.n_active) return;
+    e = P.active[y];
+    s0 = P.first[y];
+    n = P.first[y + 1] - s0;
   }
-  const int N = shared ? P.Ns : P.N, K = shared ? P.Ks : P.K, r0 = blockIdx.x * ER_ROWS;
+  const int N = mine ? P.Ns : P.N, K = mine ? P.Ks : P.K, r0 = blockIdx.x * 16 * RG;
   if (r0 >= N) return;
-  const int ldw = shared ? P.ld_ws : P.ld_w, ldx = shared ? P.ld_xs : P.ld_x;
-  const __nv_bfloat16* w = shared ? P.ws : P.w + static_cast<size_t>(e) * P.N * P.ld_w;
-  const __nv_bfloat16* x = shared ? P.xs : P.x;
+  const int ldw = mine ? P.ld_ws : P.ld_w, ldx = mine ? P.ld_xs : P.ld_x;
+  const __nv_bfloat16* w = mine ? P.ws : P.w + static_cast<size_t>(e) * P.N * P.ld_w;
+  const __nv_bfloat16* x = mine ? P.xs : P.x;
   const int q = lane & 3, rr = r0 + rg * 16 + (lane >> 2);
   const bool live0 = rr < N, live1 = rr + 8 < N;
-  const __nv_bfloat16* w0 = w + static_cast<size_t>(live0 ? rr : 0) * ldw;
-  const __nv_bfloat16* w1 = w + static_cast<size_t>(live1 ? rr + 8 : 0) * ldw;
+  const __nv_bfloat16* w0 = w + static_cast<size_t>(live0 ? rr : 0) * ldw + 8 * q;
+  const __nv_bfloat16* w1 = w + static_cast<size_t>(live1 ? rr + 8 : 0) * ldw + 8 * q;
   const __nv_bfloat16* xp[NT];
   bool xl[NT];
 #pragma unroll
@@ -289,63 +295,105 @@ moe_rows_kernel(const ExpertRows P) {
     const int tk = 8 * j + (lane >> 2);
     xl[j] = tk < n;
     const int s = s0 + (xl[j] ? tk : 0);
-    xp[j] = x + static_cast<size_t>(shared ? (xl[j] ? tk : 0) : P.gather ? P.row[s] : s) * ldx;
+    xp[j] = x + static_cast<size_t>(mine ? (xl[j] ? tk : 0) : P.gather ? P.row[s] : s) * ldx + 8 * q;
   }
-  // K in steps of 32 columns, dealt to the ranges in whole steps
-  const int steps = (K + 31) >> 5, k0 = steps * kw / ER_KW, k1 = steps * (kw + 1) / ER_KW;
+  const int steps = (K + 31) >> 5, k0 = steps * kw / KW, k1 = steps * (kw + 1) / KW;
   float c[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) c[j][0] = c[j][1] = c[j][2] = c[j][3] = 0.f;
-  constexpr int U = NT >= 8 ? 4 : 8;
-  const uint4 zero = make_uint4(0, 0, 0, 0);
-  for (int kb = k0; kb < k1; kb += U) {
-    uint4 a[U], b[U];
+  const uint32_t queue = smem_u32(smem) + threadIdx.x * 16;   // [ER_DEPTH][2][256] pieces
+  auto request = [&](int k) {
+    const uint32_t d = queue + ((k - k0) % ER_DEPTH) * 8192;
+    const bool in = k < k1 && k * 32 + 8 * q < K;
+    const int col = in ? k * 32 : 0;
+    cp_async16_zfill(d, w0 + col, in && live0);
+    cp_async16_zfill(d + 4096, w1 + col, in && live1);
+  };
+  uint4 nx[NT];
+  auto load_x = [&](int k) {
+    const int col = k * 32 + 8 * q;
+    const bool in = k < k1 && col < K;
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int k = (kb + u) * 32 + 8 * q;
-      const bool in = kb + u < k1 && k < K;
-      a[u] = in && live0 ? ld_stream(w0 + k) : zero;
-      b[u] = in && live1 ? ld_stream(w1 + k) : zero;
+    for (int j = 0; j < NT; ++j) {
+      nx[j] = make_uint4(0, 0, 0, 0);
+      if (8 * j < n && in && xl[j]) nx[j] = *reinterpret_cast<const uint4*>(xp[j] + k * 32);
     }
+    if (in && col + 8 > K) {                                  // padding columns of a row are not initialised
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int k = (kb + u) * 32 + 8 * q;
-      const bool in = kb + u < k1 && k < K;
+      for (int j = 0; j < NT; ++j) nx[j] = keep8(nx[j], K - col);
+    }
+  };
 #pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        if (8 * j >= n) break;                              // uniform over the CTA
-        uint4 v = in && xl[j] ? *reinterpret_cast<const uint4*>(xp[j] + k) : zero;
-        if (k + 8 > K && in) v = keep8(v, K - k);           // padding columns of a row are not initialised
-        mma_16816(c[j], a[u].x, b[u].x, a[u].y, b[u].y, v.x, v.y);
-        mma_16816(c[j], a[u].z, b[u].z, a[u].w, b[u].w, v.z, v.w);
-      }
+  for (int s = 0; s < ER_DEPTH - 1; ++s) {
+    request(k0 + s);
+    cp_commit();
+  }
+  load_x(k0);
+  for (int k = k0; k < k1; ++k) {
+    request(k + ER_DEPTH - 1);
+    cp_commit();
+    cp_wait<ER_DEPTH - 1>();
+    const uint8_t* d = smem + threadIdx.x * 16 + ((k - k0) % ER_DEPTH) * 8192;
+    const uint4 a = *reinterpret_cast<const uint4*>(d), b = *reinterpret_cast<const uint4*>(d + 4096);
+    uint4 v[NT];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) v[j] = nx[j];
+    load_x(k + 1);
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      if (8 * j >= n) break;                                  // uniform over the CTA
+      mma_16816(c[j], a.x, b.x, a.y, b.y, v[j].x, v[j].y);
+      mma_16816(c[j], a.z, b.z, a.w, b.w, v[j].z, v[j].w);
     }
   }
+  cp_wait<0>();
   // c[j][0..1]: row rr, tokens 8 j + 2 q + {0, 1}; c[j][2..3]: row rr + 8
-  if (kw) {
+  float* part = reinterpret_cast<float*>(smem);               // [KW - 1][RG][16][8 NT + 1], over the queue
+  constexpr int LP = 8 * NT + 1;
+  if constexpr (KW > 1) {
+    __syncthreads();
+    if (kw) {
+      float* pp = part + ((kw - 1) * RG + rg) * 16 * LP;
 #pragma unroll
-    for (int j = 0; j < NT; ++j)
+      for (int j = 0; j < NT; ++j)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) part[kw - 1][rg][(lane >> 2) + 8 * (i >> 1)][8 * j + 2 * q + (i & 1)] = c[j][i];
+        for (int i = 0; i < 4; ++i) pp[((lane >> 2) + 8 * (i >> 1)) * LP + 8 * j + 2 * q + (i & 1)] = c[j][i];
+    }
+    __syncthreads();
+    if (kw) return;
   }
-  __syncthreads();
-  if (kw) return;
-  TO* y = reinterpret_cast<TO*>(shared ? P.ys : P.y) + (shared ? 0 : static_cast<size_t>(s0) * P.ld_y);
-  const int ldy = shared ? P.ld_ys : P.ld_y;
+  TO* y = reinterpret_cast<TO*>(mine ? P.ys : P.y) + (mine ? 0 : static_cast<size_t>(s0) * P.ld_y);
+  const int ldy = mine ? P.ld_ys : P.ld_y;
 #pragma unroll
-  for (int j = 0; j < NT; ++j)
+  for (int j = 0; j < NT; ++j) {
+    if (8 * j >= n) break;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = (lane >> 2) + 8 * (i >> 1), tk = 8 * j + 2 * q + (i & 1);
       float v = c[j][i];
 #pragma unroll
-      for (int g = 0; g < ER_KW - 1; ++g) v += part[g][rg][r][tk];
+      for (int g = 0; g < KW - 1; ++g) v += part[(g * RG + rg) * 16 * LP + r * LP + tk];
       if (P.relu2) {
         v = fmaxf(v, 0.f);
         v *= v;
       }
       if (tk < n && r0 + rg * 16 + r < N) stf(y + static_cast<size_t>(tk) * ldy + r0 + rg * 16 + r, v);
     }
+  }
+}
+
+template <typename TO, int NT, int RG, int KW>
+static int launch_rows(const ExpertRows& P, int max_active, cudaStream_t st) {
+  constexpr int QUEUE = ER_DEPTH * 8192, PART = (KW - 1) * RG * 16 * (8 * NT + 1) * 4, SMEM = QUEUE > PART ? QUEUE : PART;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(moe_rows_kernel<TO, NT, RG, KW>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return -3;
+    configured = true;
+  }
+  const int rows = P.N > P.Ns ? P.N : P.Ns;
+  const dim3 grid((rows + 16 * RG - 1) / (16 * RG), max_active + (P.Ns ? 1 : 0));
+  launch_k(moe_rows_kernel<TO, NT, RG, KW>, grid, dim3(256), static_cast<size_t>(SMEM), st, P);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
 // ------------------------------------------------------------------------------------------------ sum of the experts
@@ -398,9 +446,8 @@ B200_API int b200_moe_max_outputs() { return MOE_MAX_OUT; }
 
 B200_API int b200_moe_router_logits(const void* x, int ld_x, const void* w, int ld_w, float* z, int ld_z, int B, int R, int E, int f32,
                                     void* stream) {
-  if (B <= 0 || R <= 0 || E <= 0 || ld_z < R || ((ld_x | ld_w) & 7) || ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15)) return -1;
-  if (f32) launch_k(moe_router_logits_kernel<float>, dim3(R), dim3(128), 0, STREAM, (const float*)x, ld_x, (const float*)w, ld_w, z, ld_z, B, E);
-  else launch_k(moe_router_logits_kernel<bf16_t>, dim3(R), dim3(128), 0, STREAM, (const bf16_t*)x, ld_x, (const bf16_t*)w, ld_w, z, ld_z, B, E);
+  if (B <= 0 || R <= 0 || E <= 0 || ld_z < R || !f32 || ((ld_x | ld_w) & 7) || ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15)) return -1;
+  launch_k(moe_router_logits_kernel<float>, dim3(R), dim3(128), 0, STREAM, (const float*)x, ld_x, (const float*)w, ld_w, z, ld_z, B, E);
   return DONE;
 }
 
@@ -415,7 +462,8 @@ B200_API int b200_moe_route(const float* z, const RouteArgs* Rp, int* count, int
   if (T <= 0 || !route_ok(R)) return -1;
   const int smem = (16 * R.outputs + R.experts) * 4;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
-  moe_route_kernel<<<(T + 31) / 32, 256, smem, STREAM>>>(z, R, count, rank, T);
+  const int per = T <= 16384 ? 8 : 32;      // few tokens per CTA: short; many: fewer additions to the counts
+  moe_route_kernel<<<(T + per - 1) / per, 256, smem, STREAM>>>(z, R, count, rank, T, per);
   return DONE;
 }
 
@@ -444,25 +492,26 @@ B200_API int b200_moe_route_rows(const float* z, const RouteArgs* Rp, const Rout
   return DONE;
 }
 
-// max_active: most experts that can have been chosen
-B200_API int b200_moe_rows(const ExpertRows* Pp, int max_active, int out_f32, void* stream) {
+// max_active: most experts that can have been chosen (0: only the shared expert's matrix).  narrow: matrices of few rows.
+B200_API int b200_moe_rows(const ExpertRows* Pp, int max_active, int out_f32, int narrow, void* stream) {
   const ExpertRows P = *Pp;
-  if (P.B <= 0 || P.B > 64 || P.N <= 0 || P.K <= 0 || max_active <= 0 || max_active > 65534 || P.Ns < 0 || (P.Ns && (P.Ks <= 0 || !P.ws || !P.xs || !P.ys))) return -1;
+  if (P.B <= 0 || P.B > 64 || max_active < 0 || max_active > 65534 || P.N < 0 || P.Ns < 0 || (!P.Ns && !max_active)) return -1;
+  if ((max_active && (P.N <= 0 || P.K <= 0 || !P.w || !P.x || !P.y || !P.active || !P.first || !P.n_active || (P.gather && !P.row))) ||
+      (P.Ns && (P.Ks <= 0 || !P.ws || !P.xs || !P.ys))) return -1;
   if (((P.ld_w | P.ld_x | P.ld_ws | P.ld_xs) & 7) || ((reinterpret_cast<uintptr_t>(P.w) | reinterpret_cast<uintptr_t>(P.ws) | reinterpret_cast<uintptr_t>(P.x) |
                                                       reinterpret_cast<uintptr_t>(P.xs)) & 15)) return -1;
-  const int rows = P.N > P.Ns ? P.N : P.Ns;
-  const dim3 grid((rows + ER_ROWS - 1) / ER_ROWS, max_active + (P.Ns ? 1 : 0));
-  const int nt = P.B <= 8 ? 1 : P.B <= 16 ? 2 : P.B <= 32 ? 4 : 8;
-#define GO(TO)                                                                        \
-  {                                                                                   \
-    if (nt == 1) launch_k(moe_rows_kernel<TO, 1>, grid, dim3(256), 0, STREAM, P);      \
-    else if (nt == 2) launch_k(moe_rows_kernel<TO, 2>, grid, dim3(256), 0, STREAM, P); \
-    else if (nt == 4) launch_k(moe_rows_kernel<TO, 4>, grid, dim3(256), 0, STREAM, P); \
-    else launch_k(moe_rows_kernel<TO, 8>, grid, dim3(256), 0, STREAM, P);              \
+#define GO(NT, RG, KW) return out_f32 ? launch_rows<float, NT, RG, KW>(P, max_active, STREAM) : launch_rows<bf16_t, NT, RG, KW>(P, max_active, STREAM)
+  if (narrow) {
+    if (P.B <= 8) GO(1, 1, 8);
+    if (P.B <= 32) GO(4, 1, 8);
+    GO(8, 1, 8);
   }
-  if (out_f32) GO(float) else GO(bf16_t)
+  if (P.B <= 2) GO(1, 1, 8);
+  if (P.B <= 8) GO(1, 2, 4);
+  if (P.B <= 16) GO(2, 4, 2);
+  if (P.B <= 32) GO(4, 8, 1);
+  GO(8, 8, 1);
 #undef GO
-  return DONE;
 }
 
 // y, ys: fp32 with y_f32, else the storage type; out: fp32 with out_f32, else the storage type

@@ -623,6 +623,11 @@ class LayeredConfig:
         return build_model(self, **kwargs)
 
     # -- counts ------------------------------------------------------------------------------------------------------
+    def active_param_count(self) -> int:
+        """Parameters that a token meets: of a mixture of experts only those it can choose."""
+        idle = (layer.mlp for layer in self.layers if isinstance(layer.mlp, MixtureSpec))
+        return self.param_count() - sum(m.param_count(self.width) - m.active_params(self.width) for m in idle)
+
     def param_count(self) -> int:
         E = self.width
         if self.design.sandwich:

@@ -91,8 +91,12 @@ if os.environ.get("B200_GEMM_RASTER"):
 BF16 = torch.bfloat16
 
 
+_raw_stream, _device = torch._C._cuda_getCurrentRawStream, torch._C._cuda_getDevice
+
+
 def _stream() -> int:
-    return torch.cuda.current_stream().cuda_stream
+    """The current stream's handle (asked for at every launch: no stream object is built)."""
+    return _raw_stream(_device())
 
 
 _launches = 0

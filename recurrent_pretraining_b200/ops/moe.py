@@ -64,7 +64,7 @@ def _k():
             plan=K._sig("b200_moe_plan", [vp, i, i, vp, vp, vp, vp]),
             dispatch=K._sig("b200_moe_dispatch", [vp, i, vp, i, i] + [vp] * 4 + [i] * 3 + [vp]),
             route_rows=K._sig("b200_moe_route_rows", [vp, C.POINTER(_Route), C.POINTER(_RouteRows), i, vp]),
-            rows=K._sig("b200_moe_rows", [C.POINTER(_ExpertRows), i, i, vp]),
+            rows=K._sig("b200_moe_rows", [C.POINTER(_ExpertRows), i, i, i, vp]),
             combine=K._sig("b200_moe_combine", [vp, i] * 3 + [vp, vp, vp] + [i] * 7 + [vp]),
             gemm=K._sig("b200_gemm_grouped", [vp] * 3 + [i] * 7 + [vp, vp] + [i] * 3 + [vp, vp]))
     return _fns
@@ -82,6 +82,11 @@ def router_logits(h: torch.Tensor, router: torch.Tensor) -> torch.Tensor:
         return z if z.stride(1) == 1 else z.contiguous()
     k = _k()
     z = torch.empty(B, R, dtype=F32, device=h.device)
+    if h.dtype == BF16:
+        e = _ExpertRows(Ns=R, Ks=h.shape[1], ld_ws=router.stride(0), ld_xs=h.stride(0), ld_ys=R, B=B, ws=router.data_ptr(), xs=h.data_ptr(),
+                        ys=z.data_ptr())
+        k.K._check(k.rows(C.byref(e), 0, 1, 1, k.K._stream()), "moe_rows")
+        return z
     k.K._check(k.logits(h.data_ptr(), h.stride(0), router.data_ptr(), router.stride(0), z.data_ptr(), R, B, R, h.shape[1], _f32(h), k.K._stream()),
                "moe_router_logits")
     return z
@@ -227,30 +232,28 @@ def mixture_rows_pieces(w: MoeWeights, h: torch.Tensor):
     a_s = torch.empty(B, pad8(fs), dtype=BF16, device=dev) if shared else None
     ys = torch.empty(B, pad8(E), dtype=F32, device=dev)[:, :E] if shared else None
     p = k.K._ptr
-    z = torch.empty(B, w.router.shape[0], dtype=F32, device=dev)
     lists = (active.data_ptr(), first.data_ptr(), row.data_ptr(), n_active.data_ptr())
     most = min(s.experts, n)
     ld = lambda t: 0 if t is None else t.stride(0)  # noqa: E731
-    keep = (i32, h)
+    keep = [i32, h]
 
     def logits():
-        assert keep
-        k.K._check(k.logits(h.data_ptr(), h.stride(0), w.router.data_ptr(), w.router.stride(0), z.data_ptr(), z.shape[1], B, z.shape[1], E, 0,
-                            k.K._stream()), "moe_router_logits")
+        keep.append(router_logits(h, w.router))
 
     def route():
+        z = keep[2]
         r, o = _route_struct(w, z, idx, weight), _RouteRows(slot.data_ptr(), *lists)
         k.K._check(k.route_rows(z.data_ptr(), C.byref(r), C.byref(o), B, k.K._stream()), "moe_route_rows")
 
     def up():
         e = _ExpertRows(s.ff, E, w.up.stride(0), fs, E, ld(w.up_s), h.stride(0), a.stride(0), h.stride(0), ld(a_s), B, 1, w.up.data_ptr(), p(w.up_s),
                         h.data_ptr(), h.data_ptr(), 1, a.data_ptr(), p(a_s), *lists)
-        k.K._check(k.rows(C.byref(e), most, 0, k.K._stream()), "moe_rows")
+        k.K._check(k.rows(C.byref(e), most, 0, 0, k.K._stream()), "moe_rows")
 
     def down():
         e = _ExpertRows(E, s.ff, w.down.stride(0), E if shared else 0, fs, ld(w.down_s), a.stride(0), y.stride(0), ld(a_s), ld(ys), B, 0,
                         w.down.data_ptr(), p(w.down_s), a.data_ptr(), p(a_s), 0, y.data_ptr(), p(ys), *lists)
-        k.K._check(k.rows(C.byref(e), most, 1, k.K._stream()), "moe_rows")
+        k.K._check(k.rows(C.byref(e), most, 1, 0, k.K._stream()), "moe_rows")
 
     def add():
         return combine(w, h, y[:, :E], ys, slot, weight, F32)

@@ -222,6 +222,16 @@ def _fatudra(name, vocab, width, layers, left, right, memory, ff, loop=None, bia
     return out
 
 
+def _dusilorn(name, vocab, width, layers, heads, kv_heads, dim, vdim, chunk, window, rot, ff, expert_ff, experts, identity, top, shared):
+    """``layers`` layers, chunked and windowed attention in turn; the first has a dense feed-forward, the others mixtures."""
+    base = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "softcap": 50.0, "v_mix": True}
+    mixers = ({"type": "attention", "mixer": {**base, "mask": {"size": chunk}}},
+              {"type": "attention_2", "mixer": {**base, "mask": {"size": window}, "rot": {"base": 500000.0, "dims": rot}}})
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "identity": identity, "top": top}, "shared": {"ff": shared}}
+    return {"name": name, "architecture": "Dusilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "logit_scale": 0.25, "layers": [{**mixers[i % 2], "mlp": moe if i else {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
 layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _gasovik("gasovik-tiny", 512, 128, 3, 4, 32, 16, 32, 64, 24, 256, share_from=2, original=64),
     _gasovik("gasovik-1b", 65536, 2048, 16, 16, 128, 64, 128, 512, 1024, 8192, share_from=12),
@@ -230,6 +240,9 @@ layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _fatudra("fatudra-tiny", 512, 128, 4, (4, 2, 32, 32), (2, 32, 32), (2, 16, 32), 192, loop=(1, 3, 2), bias_rows=8, bias_max=64),
     _fatudra("fatudra-1b", 65536, 2048, 16, (16, 4, 128, 128), (8, 128, 128), (8, 64, 128), 4608),
     _fatudra("fatudra-core-5280", 65536, 5280, 4, (55, 11, 96, 96), (22, 96, 96), (22, 96, 192), 14080),
+    _dusilorn("dusilorn-tiny", 512, 128, 4, 4, 2, 32, 40, 48, 20, 16, 256, 64, 6, 2, 3, 96),
+    _dusilorn("dusilorn-2b", 65536, 2048, 16, 16, 4, 128, 128, 8192, 1024, 64, 8192, 1024, 32, 4, 4, 2048),
+    _dusilorn("dusilorn-core-5280", 65536, 5280, 4, 55, 11, 96, 96, 8192, 4096, 96, 17920, 2560, 16, 2, 4, 5120),
 )}
 
 name_to_config: dict[str, dict] = {c["name"]: c for c in configs}

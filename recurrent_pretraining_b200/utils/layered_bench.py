@@ -5,7 +5,8 @@ every kernel of a layer against its roofline.
 Random weights.  Model runs: CUDA events around whole prefill / decode calls of the two engines (graph-replayed decode).
 Kernels: CUDA events around single calls on the shapes of one layer, L2 flushed in between, median.  The comparison
 model is the depth-recurrent model run for one recurrence: as many layers of the same width, head count and value
-size, with a feed-forward that gives the same number of parameters per layer."""
+size, with a feed-forward that gives the same number of parameters per layer (of a mixture of experts: those that a token
+meets)."""
 from __future__ import annotations
 
 import argparse
@@ -76,7 +77,7 @@ def closest_model(cfg):
     n, E = len(cfg.layers), cfg.width
     a = cfg.layers[0].mixer
     a = getattr(a, "left", a)
-    per_layer = (cfg.param_count() - 2 * cfg.vocab * E) / n
+    per_layer = (cfg.active_param_count() - 2 * cfg.vocab * E) / n
     ff = max(256, int((per_layer - 4 * E * E) / (3 * E)) // 64 * 64)
     core = max(1, n // 2)
     pre = (n - core) // 2
@@ -298,6 +299,138 @@ def hybrid_ops_decode(model, B: int, context: int, t: Timer) -> list:
     return t.take()
 
 
+def routed_ops_prefill(model, seqs: list, t: Timer) -> list:
+    """Kernels of a chunked and a windowed layer and of a mixture of experts of a packed step of fresh prompts ``seqs``."""
+    from ..models.layered import PackedStep
+    from ..ops import grouped as G
+    from ..ops import latent as ops
+    from ..ops import memory as M
+    from ..ops import moe as X
+
+    cfg, E, T = model.config, model.config.width, sum(seqs)
+    cache = model.new_cache(len(seqs), max(seqs))
+    step = PackedStep([(r, 0, [1] * n) for r, n in enumerate(seqs)], "cuda")
+    x = torch.randn(T, E, device="cuda")
+    h = torch.randn(T, E, device="cuda").bfloat16()
+    first = None
+
+    def gemm(name, fn, M_, N, K, groups=1):
+        t.op(name, fn, 2.0 * (M_ * N + M_ * K + groups * N * K), 2.0 * M_ * N * K)
+
+    for i, kind in ((0, "chunked"), (1, "windowed")):
+        mix = model.layers[i].mix
+        L, a = mix.layout, mix.spec
+        lay = step.chunk_layout(a.size) if a.chunked else step.layout(a.size - 1)
+        inp = ops.linear(h, mix.w_in[:, :E])
+        tr = mix._transform(cfg.mixes_values(i), cache.rope, first)
+        first = inp[:, L.off_v:L.off_v + L.v_width] if first is None else first
+        kv = torch.empty(lay.total, L.ld_kv, dtype=torch.bfloat16, device="cuda")
+        prep = lambda: G.qkv_prep_(L, inp, tr, step, lay.sidx, cache.data[i, "kv"], kv)  # noqa: E731
+        prep()
+        if i == 0:
+            gemm("qkv projection", lambda: ops.linear(h, mix.w_in[:, :E]), T, L.width_in, E)
+        ring = sum(min(n, cache.data[i, "kv"].shape[1]) for n in seqs) * L.ld_kv
+        t.op(f"{kind}: qkv_prep", prep, 2.0 * (T * (2 * a.heads * a.dim + 2 * L.ld_kv + (L.v_width if tr.lam is not None else 0)) + ring), 0)
+        o = G.stream_attention(L, a, inp, kv, lay, mix.sink)
+        pairs = float(sum(m * (m + 1) / 2 + m * f for _, m, _, f in lay.seqs)) if a.chunked else visible_pairs(seqs, a.size)
+        t.op(f"{kind}: attention", lambda: G.stream_attention(L, a, inp, kv, lay, mix.sink), 2.0 * T * (a.heads * (a.dim + a.vdim) + L.ld_kv),
+             2.0 * pairs * a.heads * (a.dim + a.vdim))
+    gemm("output projection", lambda: ops.linear(o, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)
+    norms = model.layers[1].norms
+    out = ops.linear(o, mix.w_o[:, :a.heads * a.vdim])
+    t.op("sandwich_norm", lambda: M.sandwich_norm_(x, out, norms["norm1b"].pair, None, norms["norm2"].pair, 1e-6, torch.bfloat16), T * E * 12.0, 0)
+    w = model.layers[1].mlp.weights
+    s = w.spec
+    z = X.router_logits(h, w.router)
+    gemm("moe: router product (fp32)", lambda: X.router_logits(h, w.router), T, w.router.shape[0], E)
+    rows = X.tile_rows(s, T, torch.bfloat16)
+    p = X.plan(w, z, rows)
+    n = int((p.idx < s.experts).sum())
+    t.op("moe: route + plan", lambda: X.plan(w, z, rows), 4.0 * T * (s.outputs + 4 * s.top), 0)
+    xs = X.dispatch(w, h, p)
+    t.op("moe: dispatch", lambda: X.dispatch(w, h, p), 2.0 * E * (T + n), 0)
+    g = X.grouped_linear(xs, w.up, s.ff, p, True)
+    gemm(f"moe: up (grouped, {rows}-row tiles)", lambda: X.grouped_linear(xs, w.up, s.ff, p, True), n, s.ff, E, s.experts)
+    y = X.grouped_linear(g, w.down, E, p)
+    gemm("moe: down (grouped)", lambda: X.grouped_linear(g, w.down, E, p), n, E, s.ff, s.experts)
+    a_s = ops.linear(h, w.up_s, None, "relu2")
+    gemm("shared expert: up", lambda: ops.linear(h, w.up_s, None, "relu2"), T, s.shared, E)
+    ys = ops.linear(a_s, w.down_s)
+    gemm("shared expert: down", lambda: ops.linear(a_s, w.down_s), T, E, s.shared)
+    t.op("moe: combine", lambda: X.combine(w, h, y, ys, p.slot, p.weight, torch.bfloat16), 2.0 * E * (n + 3 * T), 0)
+    t.op("moe: whole", lambda: X.mixture(w, h), 4.0 * E * (T + s.experts * s.ff + s.shared), 4.0 * E * (n * s.ff + T * s.shared))
+    mlp = model.layers[0].mlp
+    ff = mlp.spec.ff
+    gemm("gate-up projection + swiglu", lambda: M.glu_linear(h, mlp.w_gu[:, :E], ff, "silu"), T, 2 * ff, E)
+    d = M.glu_linear(h, mlp.w_gu[:, :E], ff, "silu")
+    gemm("down projection", lambda: ops.linear(d, mlp.w_down[:, :ff]), T, E, ff)
+    return t.take()
+
+
+def routed_ops_decode(model, B: int, context: int, t: Timer) -> list:
+    from ..engine.layered import LayeredEngine
+    from ..ops import grouped as G
+    from ..ops import memory as M
+    from ..ops import moe as X
+
+    cfg, E = model.config, model.config.width
+    eng = LayeredEngine(model, B, context + 1, use_graphs=False)
+    cache = eng.cache
+    for d in cache.data.values():
+        d.normal_(std=0.1)
+    pos = torch.full((B,), context, dtype=torch.int32, device="cuda")
+    row = torch.arange(B, dtype=torch.int32, device="cuda")
+    x = torch.randn(B, E, device="cuda")
+    h = x.bfloat16()
+
+    def skinny(name, xin, w):
+        N, K = w.shape
+        t.op(name, lambda: eng._dense(xin, w, 1 if N * B <= eng._work[1].numel() else 0), 2.0 * (N * K + B * K + B * N), 2.0 * B * N * K)
+
+    for i, kind in ((0, "chunked"), (1, "windowed")):
+        mix = model.layers[i].mix
+        L, a = mix.layout, mix.spec
+        if i == 0:
+            skinny("qkv projection", h, mix.w_in[:, :E])
+        inp = torch.randn(B, L.width_in, device="cuda")
+        first = torch.randn(B, M.pad8(L.v_width), device="cuda")[:, :L.v_width]
+        tr = mix._transform(cfg.mixes_values(i), cache.rope, first)
+        o = torch.empty(B, M.pad8(a.heads * a.vdim), dtype=torch.bfloat16, device="cuda")[:, :a.heads * a.vdim]
+        splits = eng._splits(mix, B)
+        attend, merge = G.ring_attention_pieces(L, a, inp, tr, cache.data[i, "kv"], mix.sink, None, pos, row, splits, o)
+        keys = context % a.size + 1 if a.chunked else min(a.size, context + 1)
+        t.op(f"{kind}: decode attention ({splits} splits)", attend, 2.0 * B * (keys * L.ld_kv + a.heads * (a.dim + a.vdim)),
+             2.0 * B * a.heads * keys * (a.dim + a.vdim))
+        if splits > 1:
+            t.op(f"{kind}: merge", merge, B * a.heads * a.vdim * (4.0 * splits + 2), 0)
+    skinny("output projection", o, mix.w_o[:, :a.heads * a.vdim])
+    norms = model.layers[1].norms
+    acc = torch.zeros(B, E, device="cuda")
+    t.op("sandwich_norm", lambda: M.sandwich_norm_(x, acc, norms["norm1b"].pair, None, norms["norm2"].pair, 1e-6, torch.bfloat16), B * E * 14.0, 0)
+    w = model.layers[1].mlp.weights
+    s = w.spec
+    parts = X.mixture_rows_pieces(w, h)
+    for f in parts:
+        f()
+    idx = X.plan(w, X.router_logits(h, w.router), 128).idx
+    real = idx[idx < s.experts]
+    n, used = real.numel(), real.unique().numel()
+    weights = 2.0 * E * (used * s.ff + s.shared)
+    R = w.router.shape[0]
+    for name, f, b in (("moe: router product", parts[0], 2.0 * E * (R + B)), ("moe: route", parts[1], 4.0 * B * R),
+                       (f"moe: up ({used} experts + shared)", parts[2], weights + 2.0 * B * E + 2.0 * (n * s.ff + B * s.shared)),
+                       ("moe: down", parts[3], weights + 2.0 * (n * s.ff + B * s.shared) + 4.0 * E * (n + B)),
+                       ("moe: combine", parts[4], E * (4.0 * n + 10.0 * B))):
+        t.op(name, f, b, 0)
+    mlp = model.layers[0].mlp
+    ff = mlp.spec.ff
+    skinny("gate-up projection", h, mlp.w_gu[:, :E])
+    work = torch.zeros(B, 2 * ff, device="cuda")
+    t.op("swiglu", lambda: M.glu(work, ff, "silu", torch.bfloat16), B * ff * 10.0, 0)
+    skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), mlp.w_down[:, :ff])
+    return t.take()
+
+
 def closest_ops_prefill(model, B: int, S: int, t: Timer) -> list:
     from ..ops import attention as A
     from ..ops import cuda as K
@@ -412,7 +545,10 @@ def model_rates(cfg, prompt: int, new: int, batches) -> dict:
     return out
 
 
-def run(shapes=("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5280"), batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
+SHAPES = ("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5280", "dusilorn-2b", "dusilorn-core-5280")
+
+
+def run(shapes=SHAPES, batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
     from ..models.layered import LayeredForCausalLM
     from ..models.layered_config import LayeredConfig
     from ..ops import cuda as K
@@ -425,9 +561,9 @@ def run(shapes=("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5
             r["models"] = model_rates(cfg, prompt, new, batches)
             torch.cuda.empty_cache()
         t = Timer()
-        hybrid = cfg.design.norms == "sandwich"
-        ops_prefill, ops_decode = (hybrid_ops_prefill, hybrid_ops_decode) if hybrid else (layer_ops_prefill, layer_ops_decode)
-        few = replace(cfg, vocab=1024, layers=cfg.layers[:2 if hybrid else 1], loop=None)
+        ops_prefill, ops_decode = {"post_rms": (layer_ops_prefill, layer_ops_decode), "sandwich": (hybrid_ops_prefill, hybrid_ops_decode),
+                                   "sandwich_rms": (routed_ops_prefill, routed_ops_decode)}[cfg.design.norms]
+        few = replace(cfg, vocab=1024, layers=cfg.layers[:2 if cfg.design.sandwich else 1], loop=None)
         model = LayeredForCausalLM(few, torch.bfloat16, "cuda").init_weights()
         S = 4096
         r["prefill_ops"] = {"tokens": S, "ours": ops_prefill(model, [S], t)}
@@ -447,7 +583,7 @@ def run(shapes=("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5
 
 def main():
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("--shapes", default="gasovik-1b,gasovik-core-5280,fatudra-1b,fatudra-core-5280")
+    ap.add_argument("--shapes", default=",".join(SHAPES))
     ap.add_argument("--batches", default="1,8,32")
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--new", type=int, default=128)
