@@ -131,38 +131,42 @@ qkv_prep_kernel(const TI* in, T* q, const TF* __restrict__ first, float* __restr
   }
 }
 
-// out[b, h * vdim + d] = sum over splits / (sum of the softmax + exp(sink)); one warp per (sequence, head).
+// out[b, h * vdim + d] = sum over splits / (sum of the softmax + exp(sink)).  CTA per (sequence, head): every warp takes each fourth
+// split, all its pieces requested at once.
 template <typename T>
 __global__ void __launch_bounds__(128)
 attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
-                       T* __restrict__ out, int ld_out, int H, int vdim, int splits, int total) {
+                       T* __restrict__ out, int ld_out, int H, int vdim, int splits) {
   pdl_trigger();
   pdl_wait();
-  const int i = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (i >= total) return;
-  const int b = i / H, h = i - b * H, vs = (vdim + 7) & ~7;
+  extern __shared__ float sums[];                               // [4][vdim padded to four]
+  const int i = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = i / H, h = i - b * H, vs = (vdim + 7) & ~7, v4 = (vdim + 3) & ~3;
   const float2 e = lane < splits ? *reinterpret_cast<const float2*>(part_ml + (static_cast<size_t>(i) * splits + lane) * 2)
                                  : make_float2(-INFINITY, 0.f);
   const float sk = sink ? sink[h] : -INFINITY;
   const float m = fmaxf(warp_max(e.x), sk);
   const float w = e.x == -INFINITY ? 0.f : expf(e.x - m);
   const float mine = w / (warp_sum(w * e.y) + (sink ? expf(sk - m) : 0.f));
+  float f[8];
+#pragma unroll
+  for (int u = 0; u < 8; ++u) f[u] = __shfl_sync(0xffffffffu, mine, warp + 4 * u);   // zero past the splits
   const float* p = part_o + static_cast<size_t>(i) * splits * vs;
-  for (int d0 = 0; d0 < vdim; d0 += 128) {                      // uniform over the warp
-    const int d = d0 + 4 * lane;
+  for (int d = 4 * lane; d < v4; d += 128) {
+    float x[8][4];
+#pragma unroll
+    for (int u = 0; u < 8; ++u)
+      if (f[u] != 0.f) ld4(p + static_cast<size_t>(warp + 4 * u) * vs + d, x[u]);    // an empty split's partial is not initialised
     float o[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 8
-    for (int s = 0; s < splits; ++s) {
-      const float f = __shfl_sync(0xffffffffu, mine, s);
-      float x[4] = {0.f, 0.f, 0.f, 0.f};
-      if (d < vs) ld4(p + static_cast<size_t>(s) * vs + d, x);
 #pragma unroll
-      for (int k = 0; k < 4; ++k) o[k] += f != 0.f ? f * x[k] : 0.f;   // an empty split's partial is not initialised
-    }
+    for (int u = 0; u < 8; ++u)
 #pragma unroll
-    for (int k = 0; k < 4; ++k)
-      if (d + k < vdim) stf(out + static_cast<size_t>(b) * ld_out + h * vdim + d + k, o[k]);
+      for (int k = 0; k < 4; ++k) o[k] += f[u] != 0.f ? f[u] * x[u][k] : 0.f;
+    *reinterpret_cast<float4*>(sums + warp * v4 + d) = make_float4(o[0], o[1], o[2], o[3]);
   }
+  __syncthreads();
+  for (int d = threadIdx.x; d < vdim; d += 128)
+    stf(out + static_cast<size_t>(b) * ld_out + h * vdim + d, sums[d] + sums[v4 + d] + sums[2 * v4 + d] + sums[3 * v4 + d]);
 }
 
 }  // namespace b200
@@ -200,8 +204,9 @@ B200_API int b200_qkv_prep(const void* in, void* q, const void* first, float* fi
 B200_API int b200_attention_merge(const float* part_o, const float* part_ml, const float* sink, void* out, int ld_out, int B, int H, int vdim,
                                   int splits, int f32, void* stream) {
   if (B <= 0 || H <= 0 || vdim <= 0 || splits < 1 || splits > 32) return -1;
-  const int total = B * H;
-  if (f32) launch_k(attention_merge_kernel<float>, dim3((total + 3) / 4), dim3(128), 0, STREAM, part_o, part_ml, sink, (float*)out, ld_out, H, vdim, splits, total);
-  else launch_k(attention_merge_kernel<bf16_t>, dim3((total + 3) / 4), dim3(128), 0, STREAM, part_o, part_ml, sink, (bf16_t*)out, ld_out, H, vdim, splits, total);
+  const size_t smem = 4 * ((vdim + 3) & ~3) * sizeof(float);
+  if (smem > 48 * 1024 || static_cast<long long>(B) * H > 0x7fffffffll) return -1;
+  if (f32) launch_k(attention_merge_kernel<float>, dim3(B * H), dim3(128), smem, STREAM, part_o, part_ml, sink, (float*)out, ld_out, H, vdim, splits);
+  else launch_k(attention_merge_kernel<bf16_t>, dim3(B * H), dim3(128), smem, STREAM, part_o, part_ml, sink, (bf16_t*)out, ld_out, H, vdim, splits);
   return DONE;
 }

@@ -24,7 +24,56 @@ struct SandwichArgs {
   const float *w2, *b2;           // norm of the next sublayer's input; null: none
   float* x;
   float* zero;                    // second accumulator, re-armed here
+  // sublayer output that is still a sum (`a` holds the rows it picks from): sum_k weight[row, k] a[slot[row, k]], with mix_h[row] in
+  // place of a row whose slot is negative, + weight[row, top] shared[row]
+  int top, ld_mix, ld_shared;     // top 0: `a` is the output itself
+  const int* slot;
+  const float* weight;            // [rows, top + 1]
+  const void *mix_h, *shared;     // operand precision; the type of `a` (null: none)
 };
+
+// Eight columns (V = 8) or one of the output of a sublayer.
+template <int V, typename TI, typename T>
+__device__ __forceinline__ void sublayer_cols(const SandwichArgs& A, const TI* a, size_t row, int i, float* v) {
+  auto load = [](const auto* p, float* o) {
+    if constexpr (V == 8) ld8(p, *reinterpret_cast<float(*)[8]>(o));
+    else *o = ldf(p);
+  };
+  if (!A.top) {
+    load(a + row * A.ld_a + i, v);
+    return;
+  }
+  const int* sl = A.slot + row * A.top;
+  const float* wt = A.weight + row * (A.top + 1);
+#pragma unroll
+  for (int j = 0; j < V; ++j) v[j] = 0.f;
+  for (int k0 = 0; k0 < A.top; k0 += 4) {                 // four rows on their way at a time
+    float y[4][V], f[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      f[u] = 0.f;
+      if (k0 + u < A.top) {
+        const int s = sl[k0 + u];
+        f[u] = wt[k0 + u];
+        if (s < 0) load(reinterpret_cast<const T*>(A.mix_h) + row * A.ld_mix + i, y[u]);
+        else load(a + static_cast<size_t>(s) * A.ld_a + i, y[u]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[u][j] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += f[u] * y[u][j];
+  }
+  if (A.shared) {
+    float y[V];
+    load(reinterpret_cast<const TI*>(A.shared) + row * A.ld_shared + i, y);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] += wt[A.top] * y[j];
+  }
+}
 
 // One CTA per row; NV groups of eight columns per thread held in registers.  A null `a` skips the sublayer output.
 // RMS: no means are taken, weights are one plus the stored ones and there are no biases.
@@ -54,7 +103,8 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
     if (i < nvec) {
       ld8(A.x + row * A.E + 8 * i, xv[k]);
       if (ar) {
-        ld8(ar + 8 * i, s[k]);
+        if constexpr (RMS) sublayer_cols<8, TI, T>(A, a, row, 8 * i, s[k]);
+        else ld8(ar + 8 * i, s[k]);
         if (A.clear) clear8(ar + 8 * i);
         if (A.bias) {
           float b[8];
@@ -146,7 +196,12 @@ sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   TI* ar = a ? a + row * A.ld_a : nullptr;
   float* x = A.x + row * A.E;
   for (int i = threadIdx.x; i < A.nzero; i += 256) A.zero[row * A.nzero + i] = 0.f;
-  auto in = [&](int i) { return ldf(ar + i) + (A.bias ? A.bias_mult * A.bias[i] : 0.f); };
+  auto in = [&](int i) {
+    float v;
+    if constexpr (RMS) sublayer_cols<1, TI, T>(A, a, row, i, &v);
+    else v = ldf(ar + i);
+    return v + (A.bias ? A.bias_mult * A.bias[i] : 0.f);
+  };
   float mean = 0.f, r = 0.f;
   if (ar) {
     float sum = 0.f, ss = 0.f;
@@ -593,7 +648,8 @@ typedef __nv_bfloat16 bf16_t;
 
 template <typename TI, typename T, bool RMS>
 static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, cudaStream_t st) {
-  const bool vec = A.E % 8 == 0 && A.ld_a % 8 == 0 && A.ld_h % 8 == 0 &&
+  const bool vec = A.E % 8 == 0 && A.ld_a % 8 == 0 && A.ld_h % 8 == 0 && A.ld_mix % 8 == 0 && A.ld_shared % 8 == 0 &&
+                   !((reinterpret_cast<uintptr_t>(A.mix_h) | reinterpret_cast<uintptr_t>(A.shared)) & 15) &&
                    !((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(A.x) |
                       reinterpret_cast<uintptr_t>(A.w1) | reinterpret_cast<uintptr_t>(A.b1) | reinterpret_cast<uintptr_t>(A.w2) |
                       reinterpret_cast<uintptr_t>(A.b2) | reinterpret_cast<uintptr_t>(A.bias) | reinterpret_cast<uintptr_t>(A.step)) & 15);
@@ -611,6 +667,7 @@ static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, c
 B200_API int b200_sandwich_norm(void* a, void* h, const SandwichArgs* Ap, int rows, int in_f32, int f32, int rms, void* stream) {
   const SandwichArgs A = *Ap;
   if (rows <= 0 || A.E <= 0 || !A.x || (A.clear && !in_f32) || (f32 && !in_f32) || (A.nzero && !A.zero)) return -1;
+  if (A.top && (!rms || !a || A.top < 0 || A.clear || !A.slot || !A.weight || !A.mix_h)) return -1;
   if ((a && (!A.w1 || (!rms && !A.b1))) || (A.w2 && ((!rms && !A.b2) || !h))) return -1;
 #define GO(RMS)                                                                \
   {                                                                            \

@@ -7,7 +7,7 @@
 //   * moe_route_rows    : the three in one CTA for the few rows of a decode step, slots without padding
 //   * moe_rows          : product of a decode step's rows with their experts' weights: a stream of weights through mma.sync,
 //                         fragments straight from memory
-//   * moe_combine       : weighted sum of a token's experts, identity experts and the gated shared expert
+// The weighted sum of a token's experts is formed by the norm that reads it (sandwich_norm in memory.cu).
 // Storage types: bf16 (serving) or fp32; arithmetic is fp32.  This file is built without fast-math approximations.
 #include "rowops.cuh"
 
@@ -258,13 +258,21 @@ __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0
 
 // CTA: (16 RG weight rows, chosen expert): RG groups of 16 rows x KW ranges of K, one warp each.  The order of the terms of a dot
 // product is free, so a lane takes eight neighbouring columns of its weight rows and of its token as they lie in memory: they
-// serve two MMAs.  The weights pass through a queue in shared memory that belongs to the thread alone (ER_DEPTH steps of 32 columns in
-// flight, no barriers).  NT: groups of eight tokens; more tokens take more rows per CTA, which share the tokens' way from L2.
-constexpr int ER_DEPTH = 8;
+// serve two MMAs.  Weights and tokens pass through a queue in shared memory, several steps of 32 columns in flight: the weights' part
+// belongs to the thread alone, and so does the tokens' when the warps stand at different columns (KW > 1: no barriers).  With KW = 1 all
+// warps share one copy of the tokens and meet once a step.  NT: groups of eight tokens.
+template <int NT, int KW>
+struct RowsQueue {
+  static constexpr bool SHARED_X = KW == 1;
+  static constexpr int X_BYTES = SHARED_X ? NT * 512 : NT * 4096, STEP = 8192 + X_BYTES;
+  static constexpr int DEPTH = SHARED_X ? 8 : (NT >= 8 ? 5 : 8);
+  static constexpr int BYTES = DEPTH * STEP;
+};
 template <typename TO, int NT, int RG, int KW>
-__global__ void __launch_bounds__(256, NT >= 8 ? 2 : 3)
+__global__ void __launch_bounds__(256, NT * KW >= 32 ? 1 : 2)
 moe_rows_kernel(const ExpertRows P) {
   static_assert(RG * KW == 8, "eight warps");
+  using Q = RowsQueue<NT, KW>;
   pdl_trigger();
   extern __shared__ __align__(16) uint8_t smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = warp % RG, kw = warp / RG;
@@ -288,12 +296,13 @@ moe_rows_kernel(const ExpertRows P) {
   const bool live0 = rr < N, live1 = rr + 8 < N;
   const __nv_bfloat16* w0 = w + static_cast<size_t>(live0 ? rr : 0) * ldw + 8 * q;
   const __nv_bfloat16* w1 = w + static_cast<size_t>(live1 ? rr + 8 : 0) * ldw + 8 * q;
-  const __nv_bfloat16* xp[NT];
-  bool xl[NT];
+  // this thread's source of token pieces: its own token of every group, or with SHARED_X one piece of one token
+  const __nv_bfloat16* xp[Q::SHARED_X ? 1 : NT];
+  bool xl[Q::SHARED_X ? 1 : NT];
 #pragma unroll
-  for (int j = 0; j < NT; ++j) {
-    const int tk = 8 * j + (lane >> 2);
-    xl[j] = tk < n;
+  for (int j = 0; j < (Q::SHARED_X ? 1 : NT); ++j) {
+    const int tk = Q::SHARED_X ? threadIdx.x >> 2 : 8 * j + (lane >> 2);
+    xl[j] = tk < n && tk < 8 * NT;
     const int s = s0 + (xl[j] ? tk : 0);
     xp[j] = x + static_cast<size_t>(mine ? (xl[j] ? tk : 0) : P.gather ? P.row[s] : s) * ldx + 8 * q;
   }
@@ -301,50 +310,46 @@ moe_rows_kernel(const ExpertRows P) {
   float c[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) c[j][0] = c[j][1] = c[j][2] = c[j][3] = 0.f;
-  const uint32_t queue = smem_u32(smem) + threadIdx.x * 16;   // [ER_DEPTH][2][256] pieces
-  auto request = [&](int k) {
-    const uint32_t d = queue + ((k - k0) % ER_DEPTH) * 8192;
+  const uint32_t queue = smem_u32(smem);
+  auto request = [&](int k, int slot) {
+    const uint32_t d = queue + slot * Q::STEP + threadIdx.x * 16;      // [weights of rows r, of rows r + 8, tokens]
     const bool in = k < k1 && k * 32 + 8 * q < K;
     const int col = in ? k * 32 : 0;
     cp_async16_zfill(d, w0 + col, in && live0);
     cp_async16_zfill(d + 4096, w1 + col, in && live1);
-  };
-  uint4 nx[NT];
-  auto load_x = [&](int k) {
-    const int col = k * 32 + 8 * q;
-    const bool in = k < k1 && col < K;
+    if constexpr (Q::SHARED_X) {
+      if (threadIdx.x < 32 * NT) cp_async16_zfill(d + 8192, xp[0] + col, in && xl[0]);
+    } else {
 #pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      nx[j] = make_uint4(0, 0, 0, 0);
-      if (8 * j < n && in && xl[j]) nx[j] = *reinterpret_cast<const uint4*>(xp[j] + k * 32);
-    }
-    if (in && col + 8 > K) {                                  // padding columns of a row are not initialised
-#pragma unroll
-      for (int j = 0; j < NT; ++j) nx[j] = keep8(nx[j], K - col);
+      for (int j = 0; j < NT; ++j)
+        if (8 * j < n) cp_async16_zfill(d + 8192 + j * 4096, xp[j] + col, in && xl[j]);
     }
   };
+  int slot = 0, next = Q::DEPTH - 1;
 #pragma unroll
-  for (int s = 0; s < ER_DEPTH - 1; ++s) {
-    request(k0 + s);
+  for (int s = 0; s < Q::DEPTH - 1; ++s) {
+    request(k0 + s, s);
     cp_commit();
   }
-  load_x(k0);
   for (int k = k0; k < k1; ++k) {
-    request(k + ER_DEPTH - 1);
+    cp_wait<Q::DEPTH - 2>();
+    if constexpr (Q::SHARED_X) __syncthreads();               // the step's tokens are there, and everyone is done with the one before
+    request(k + Q::DEPTH - 1, next);
     cp_commit();
-    cp_wait<ER_DEPTH - 1>();
-    const uint8_t* d = smem + threadIdx.x * 16 + ((k - k0) % ER_DEPTH) * 8192;
-    const uint4 a = *reinterpret_cast<const uint4*>(d), b = *reinterpret_cast<const uint4*>(d + 4096);
-    uint4 v[NT];
-#pragma unroll
-    for (int j = 0; j < NT; ++j) v[j] = nx[j];
-    load_x(k + 1);
+    const uint8_t* d = smem + slot * Q::STEP;
+    const uint4 a = *reinterpret_cast<const uint4*>(d + threadIdx.x * 16), b = *reinterpret_cast<const uint4*>(d + 4096 + threadIdx.x * 16);
+    const uint8_t* dx = d + 8192 + (Q::SHARED_X ? lane : static_cast<int>(threadIdx.x)) * 16;
+    const int left = K - (k * 32 + 8 * q);
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       if (8 * j >= n) break;                                  // uniform over the CTA
-      mma_16816(c[j], a.x, b.x, a.y, b.y, v[j].x, v[j].y);
-      mma_16816(c[j], a.z, b.z, a.w, b.w, v[j].z, v[j].w);
+      uint4 v = *reinterpret_cast<const uint4*>(dx + j * (Q::SHARED_X ? 512 : 4096));
+      if (left > 0 && left < 8) v = keep8(v, left);           // padding columns of a row are not initialised
+      mma_16816(c[j], a.x, b.x, a.y, b.y, v.x, v.y);
+      mma_16816(c[j], a.z, b.z, a.w, b.w, v.z, v.w);
     }
+    slot = slot + 1 == Q::DEPTH ? 0 : slot + 1;
+    next = next + 1 == Q::DEPTH ? 0 : next + 1;
   }
   cp_wait<0>();
   // c[j][0..1]: row rr, tokens 8 j + 2 q + {0, 1}; c[j][2..3]: row rr + 8
@@ -384,7 +389,7 @@ moe_rows_kernel(const ExpertRows P) {
 
 template <typename TO, int NT, int RG, int KW>
 static int launch_rows(const ExpertRows& P, int max_active, cudaStream_t st) {
-  constexpr int QUEUE = ER_DEPTH * 8192, PART = (KW - 1) * RG * 16 * (8 * NT + 1) * 4, SMEM = QUEUE > PART ? QUEUE : PART;
+  constexpr int QUEUE = RowsQueue<NT, KW>::BYTES, PART = (KW - 1) * RG * 16 * (8 * NT + 1) * 4, SMEM = QUEUE > PART ? QUEUE : PART;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(moe_rows_kernel<TO, NT, RG, KW>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return -3;
@@ -394,45 +399,6 @@ static int launch_rows(const ExpertRows& P, int max_active, cudaStream_t st) {
   const dim3 grid((rows + 16 * RG - 1) / (16 * RG), max_active + (P.Ns ? 1 : 0));
   launch_k(moe_rows_kernel<TO, NT, RG, KW>, grid, dim3(256), static_cast<size_t>(SMEM), st, P);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
-}
-
-// ------------------------------------------------------------------------------------------------ sum of the experts
-// out[t] = sum_k weight[t, k] * (slot[t, k] < 0 ? h[t] : y[slot[t, k]]) + weight[t, top] * ys[t]
-template <typename T, typename TY, typename TO, int W>
-__global__ void __launch_bounds__(256)
-moe_combine_kernel(const T* __restrict__ h, int ld_h, const TY* __restrict__ y, int ld_y, const TY* __restrict__ ys, int ld_ys,
-                   const int* __restrict__ slot, const float* __restrict__ weight, TO* __restrict__ out, int ld_out, int E, int top) {
-  pdl_trigger();
-  pdl_wait();
-  const size_t t = blockIdx.x;
-  const int* sl = slot + t * top;
-  const float* wt = weight + t * (top + 1);
-  for (int i = threadIdx.x * W; i < E; i += 256 * W) {
-    float acc[W], v[W];
-#pragma unroll
-    for (int j = 0; j < W; ++j) acc[j] = 0.f;
-    for (int k = 0; k < top; ++k) {
-      const int s = sl[k];
-      const float f = wt[k];
-      if constexpr (W == 8) {
-        if (s < 0) ld8(h + t * ld_h + i, v);
-        else ld8(y + static_cast<size_t>(s) * ld_y + i, v);
-      } else {
-        v[0] = s < 0 ? ldf(h + t * ld_h + i) : ldf(y + static_cast<size_t>(s) * ld_y + i);
-      }
-#pragma unroll
-      for (int j = 0; j < W; ++j) acc[j] += f * v[j];
-    }
-    if (ys) {
-      const float f = wt[top];
-      if constexpr (W == 8) ld8(ys + t * ld_ys + i, v);
-      else v[0] = ldf(ys + t * ld_ys + i);
-#pragma unroll
-      for (int j = 0; j < W; ++j) acc[j] += f * v[j];
-    }
-    if constexpr (W == 8) st8(out + t * ld_out + i, acc);
-    else stf(out + t * ld_out + i, acc[0]);
-  }
 }
 
 }  // namespace b200
@@ -512,22 +478,4 @@ B200_API int b200_moe_rows(const ExpertRows* Pp, int max_active, int out_f32, in
   if (P.B <= 32) GO(4, 8, 1);
   GO(8, 8, 1);
 #undef GO
-}
-
-// y, ys: fp32 with y_f32, else the storage type; out: fp32 with out_f32, else the storage type
-B200_API int b200_moe_combine(const void* h, int ld_h, const void* y, int ld_y, const void* ys, int ld_ys, const int* slot, const float* weight,
-                              void* out, int ld_out, int T, int E, int top, int f32, int y_f32, int out_f32, void* stream) {
-  if (T <= 0 || E <= 0 || top <= 0 || (f32 && (!y_f32 || !out_f32))) return -1;
-  const uintptr_t addr = reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(ys) | reinterpret_cast<uintptr_t>(out);
-  const bool vec = !(addr & 15) && !((E | ld_h | ld_y | ld_ys | ld_out) & 7);
-#define GO2(T_, TY, TO, W) \
-  launch_k(moe_combine_kernel<T_, TY, TO, W>, dim3(T), dim3(256), 0, STREAM, (const T_*)h, ld_h, (const TY*)y, ld_y, (const TY*)ys, ld_ys, slot, weight, (TO*)out, ld_out, E, top)
-#define GO(T_, TY, TO) { if (vec) GO2(T_, TY, TO, 8); else GO2(T_, TY, TO, 1); }
-  if (f32) GO(float, float, float)
-  else if (y_f32 && out_f32) GO(bf16_t, float, float)
-  else if (!y_f32 && !out_f32) GO(bf16_t, bf16_t, bf16_t)
-  else return -1;
-#undef GO
-#undef GO2
-  return DONE;
 }

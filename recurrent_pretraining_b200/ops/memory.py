@@ -80,7 +80,8 @@ class MemoryLayout:
 
 class _Sandwich(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("E", "ld_a", "ld_h", "clear", "nzero")] + [(n, C.c_float) for n in ("eps", "bias_mult", "out_mult")] + \
-               [(n, C.c_void_p) for n in ("bias", "w1", "b1", "step", "w2", "b2", "x", "zero")]
+               [(n, C.c_void_p) for n in ("bias", "w1", "b1", "step", "w2", "b2", "x", "zero")] + \
+               [(n, C.c_int) for n in ("top", "ld_mix", "ld_shared")] + [(n, C.c_void_p) for n in ("slot", "weight", "mix_h", "shared")]
 
 
 class _Memory(C.Structure):
@@ -125,16 +126,40 @@ def _norm(x, w, b, eps: float) -> torch.Tensor:
     return ref.rms(x, eps) * (1 + w) if b is None else ref.layer_norm(x, w, b, eps)
 
 
-def sandwich_norm_(x: torch.Tensor, a: Optional[torch.Tensor], post, step, pre, eps: float, dtype: torch.dtype, bias=None,
+@dataclass
+class RowSum:
+    """A sublayer output that is still a sum: row t is sum_k weight[t, k] rows[slot[t, k]] (h[t] where the slot is negative)
+    + weight[t, top] shared[t].  ``rows`` and ``shared`` (or None) have one dtype, ``h`` is in operand precision."""
+
+    rows: torch.Tensor
+    slot: torch.Tensor
+    weight: torch.Tensor
+    h: torch.Tensor
+    shared: Optional[torch.Tensor] = None
+
+    @property
+    def shape(self):
+        return self.h.shape
+
+    def sum(self) -> torch.Tensor:
+        """Plain form."""
+        pick = self.slot.long()
+        y = torch.where((pick < 0)[..., None], self.h[:, None].float(), self.rows[pick.clamp(min=0)].float())
+        out = (self.weight[:, :-1, None] * y).sum(1)
+        return out if self.shared is None else out + self.weight[:, -1:] * self.shared.float()
+
+
+def sandwich_norm_(x: torch.Tensor, a, post, step, pre, eps: float, dtype: torch.dtype, bias=None,
                    bias_mult: float = 1.0, clear: bool = False, zero: Optional[torch.Tensor] = None,
                    out_mult: float = 1.0) -> Optional[torch.Tensor]:
     """x += norm(a + bias_mult * bias) [+ step] in place, then out_mult * norm(x) in ``dtype`` (None without ``pre``).  ``post``
     and ``pre`` are (weight, bias) of layer norms, or (weight, None) of RMS norms whose weights are stored around zero; ``a``
-    may be None (only ``step`` is added then).  ``clear`` / ``zero``: accumulators that are handed back zeroed (a itself / a
+    may be None (only ``step`` is added then) or, with RMS norms, a ``RowSum``.  ``clear`` / ``zero``: accumulators that are handed back zeroed (a itself / a
     second one with the same number of rows)."""
     T, E = x.shape
     if not x.is_cuda:
         if a is not None:
+            a = a.sum() if isinstance(a, RowSum) else a
             s = a.float() if bias is None else a.float() + bias_mult * bias
             x += _norm(s, *post, eps)
         if step is not None:
@@ -146,8 +171,14 @@ def sandwich_norm_(x: torch.Tensor, a: Optional[torch.Tensor], post, step, pre, 
     p = k.K._ptr
     w1, b1 = post if a is not None else (None, None)
     w2, b2 = pre if pre is not None else (None, None)
+    many = {}
+    if isinstance(a, RowSum):
+        assert a.h.dtype == dtype and (a.shared is None or a.shared.dtype == a.rows.dtype) and a.weight.is_contiguous() and a.slot.is_contiguous()
+        many = dict(top=a.weight.shape[1] - 1, ld_mix=a.h.stride(0), ld_shared=0 if a.shared is None else a.shared.stride(0), slot=p(a.slot),
+                    weight=p(a.weight), mix_h=p(a.h), shared=p(a.shared))
+        a = a.rows
     s = _Sandwich(E, 0 if a is None else a.stride(0), 0 if h is None else h.stride(0), int(clear), 0 if zero is None else zero.numel() // T,
-                  eps, bias_mult, out_mult, p(bias), p(w1), p(b1), p(step), p(w2), p(b2), x.data_ptr(), p(zero))
+                  eps, bias_mult, out_mult, p(bias), p(w1), p(b1), p(step), p(w2), p(b2), x.data_ptr(), p(zero), **many)
     f32, rms = int(dtype == F32), int(b1 is None and b2 is None)
     k.K._check(k.sandwich(p(a), p(h), C.byref(s), T, f32 if a is None else _f32(a), f32, rms, k.K._stream()), "sandwich_norm")
     return h

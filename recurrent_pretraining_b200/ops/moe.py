@@ -14,6 +14,7 @@ import torch
 from . import latent as base
 from . import reference as ref
 from .latent import BF16, F32, _f32, pad8
+from .memory import RowSum
 
 ROWS = 64            # widest batch of the decode form
 
@@ -65,7 +66,6 @@ def _k():
             dispatch=K._sig("b200_moe_dispatch", [vp, i, vp, i, i] + [vp] * 4 + [i] * 3 + [vp]),
             route_rows=K._sig("b200_moe_route_rows", [vp, C.POINTER(_Route), C.POINTER(_RouteRows), i, vp]),
             rows=K._sig("b200_moe_rows", [C.POINTER(_ExpertRows), i, i, i, vp]),
-            combine=K._sig("b200_moe_combine", [vp, i] * 3 + [vp, vp, vp] + [i] * 7 + [vp]),
             gemm=K._sig("b200_gemm_grouped", [vp] * 3 + [i] * 7 + [vp, vp] + [i] * 3 + [vp, vp]))
     return _fns
 
@@ -166,16 +166,6 @@ def tile_rows(spec, T: int, dtype: torch.dtype) -> int:
     return 256 if T * spec.top >= 1024 * spec.outputs else 128
 
 
-def combine(w: MoeWeights, h, y, ys, slot, weight, dtype) -> torch.Tensor:
-    """Weighted sum of the experts' rows ``y`` [slots, E], of h for identity experts, and of the gated shared expert's ``ys``."""
-    k, s = _k(), w.spec
-    T, E = h.shape
-    out = torch.empty(T, pad8(E), dtype=dtype, device=h.device)[:, :E]
-    k.K._check(k.combine(h.data_ptr(), h.stride(0), y.data_ptr(), y.stride(0), k.K._ptr(ys), 0 if ys is None else ys.stride(0), slot.data_ptr(),
-                         weight.data_ptr(), out.data_ptr(), out.stride(0), T, E, s.top, _f32(h), _f32(y), _f32(out), k.K._stream()), "moe_combine")
-    return out
-
-
 def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     s, E = w.spec, h.shape[1]
     z = router_logits(h, w.router)
@@ -194,8 +184,8 @@ def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     return out.to(h.dtype)
 
 
-def mixture(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
-    """Mixture of experts of any number of rows h [T, E]."""
+def mixture(w: MoeWeights, h: torch.Tensor):
+    """Mixture of experts of any number of rows h [T, E]; on a GPU the experts' rows, to be summed where they are read."""
     if not h.is_cuda:
         return _plain(w, h)
     s, E = w.spec, h.shape[1]
@@ -203,21 +193,21 @@ def mixture(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     a = grouped_linear(dispatch(w, h, p), w.up, s.ff, p, relu2=True)
     y = grouped_linear(a, w.down, E, p)
     ys = None if w.up_s is None else base.linear(base.linear(h, w.up_s, None, "relu2"), w.down_s)
-    return combine(w, h, y, ys, p.slot, p.weight, h.dtype)
+    return RowSum(y, p.slot, p.weight, h, ys)
 
 
-def mixture_rows(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
-    """The same for the few bf16 rows of a decode step, as a stream of the chosen experts' weights; fp32 result."""
+def mixture_rows(w: MoeWeights, h: torch.Tensor):
+    """The same for the few bf16 rows of a decode step, as a stream of the chosen experts' weights."""
     if not h.is_cuda or h.dtype == F32 or h.shape[0] > ROWS:
         return mixture(w, h)
     parts = mixture_rows_pieces(w, h)
     for f in parts[:-1]:
         f()
-    return parts[-1]()
+    return parts[-1]
 
 
 def mixture_rows_pieces(w: MoeWeights, h: torch.Tensor):
-    """The launches of ``mixture_rows`` as callables (the last returns the result)."""
+    """The launches of ``mixture_rows`` as callables, and its result."""
     k, s = _k(), w.spec
     B, E = h.shape
     dev, n = h.device, B * s.top
@@ -255,7 +245,4 @@ def mixture_rows_pieces(w: MoeWeights, h: torch.Tensor):
                         w.down.data_ptr(), p(w.down_s), a.data_ptr(), p(a_s), 0, y.data_ptr(), p(ys), *lists)
         k.K._check(k.rows(C.byref(e), most, 1, 0, k.K._stream()), "moe_rows")
 
-    def add():
-        return combine(w, h, y[:, :E], ys, slot, weight, F32)
-
-    return logits, route, up, down, add
+    return logits, route, up, down, RowSum(y[:, :E], slot.view(B, s.top), weight, h, ys)

@@ -357,7 +357,9 @@ def routed_ops_prefill(model, seqs: list, t: Timer) -> list:
     gemm("shared expert: up", lambda: ops.linear(h, w.up_s, None, "relu2"), T, s.shared, E)
     ys = ops.linear(a_s, w.down_s)
     gemm("shared expert: down", lambda: ops.linear(a_s, w.down_s), T, E, s.shared)
-    t.op("moe: combine", lambda: X.combine(w, h, y, ys, p.slot, p.weight, torch.bfloat16), 2.0 * E * (n + 3 * T), 0)
+    mixed = M.RowSum(y, p.slot, p.weight, h, ys)
+    t.op("sandwich_norm with the sum of the experts", lambda: M.sandwich_norm_(x, mixed, norms["norm2b"].pair, None, norms["norm1"].pair, 1e-6, torch.bfloat16),
+         2.0 * E * (n + 2 * T) + T * E * 10.0, 0)
     t.op("moe: whole", lambda: X.mixture(w, h), 4.0 * E * (T + s.experts * s.ff + s.shared), 4.0 * E * (n * s.ff + T * s.shared))
     mlp = model.layers[0].mlp
     ff = mlp.spec.ff
@@ -410,7 +412,7 @@ def routed_ops_decode(model, B: int, context: int, t: Timer) -> list:
     w = model.layers[1].mlp.weights
     s = w.spec
     parts = X.mixture_rows_pieces(w, h)
-    for f in parts:
+    for f in parts[:-1]:
         f()
     idx = X.plan(w, X.router_logits(h, w.router), 128).idx
     real = idx[idx < s.experts]
@@ -420,7 +422,9 @@ def routed_ops_decode(model, B: int, context: int, t: Timer) -> list:
     for name, f, b in (("moe: router product", parts[0], 2.0 * E * (R + B)), ("moe: route", parts[1], 4.0 * B * R),
                        (f"moe: up ({used} experts + shared)", parts[2], weights + 2.0 * B * E + 2.0 * (n * s.ff + B * s.shared)),
                        ("moe: down", parts[3], weights + 2.0 * (n * s.ff + B * s.shared) + 4.0 * E * (n + B)),
-                       ("moe: combine", parts[4], E * (4.0 * n + 10.0 * B))):
+                       ("sandwich_norm with the sum of the experts",
+                        lambda: M.sandwich_norm_(x, parts[4], norms["norm2b"].pair, None, norms["norm1"].pair, 1e-6, torch.bfloat16),
+                        E * (4.0 * n + 16.0 * B))):
         t.op(name, f, b, 0)
     mlp = model.layers[0].mlp
     ff = mlp.spec.ff
