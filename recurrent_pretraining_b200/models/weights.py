@@ -65,4 +65,4 @@ def save_safetensors(path: str, tensors: dict) -> None:
         f.write(struct.pack("<Q", len(head)))
         f.write(head)
         for t in host.values():
-            f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")

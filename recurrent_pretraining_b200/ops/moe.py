@@ -163,7 +163,7 @@ def tile_rows(spec, T: int, dtype: torch.dtype) -> int:
     """Slots per tile: whole tiles of the pair kernel when the experts are busy enough to fill them."""
     if dtype == F32:
         return _k().sgemm_rows
-    return 256 if T * spec.top >= 1024 * spec.outputs else 128
+    return 256 if T * spec.top >= 192 * spec.outputs else 128
 
 
 def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
