@@ -24,7 +24,7 @@ struct SandwichArgs {
   const float *w2, *b2;           // norm of the next sublayer's input; null: none
   float* x;
   float* zero;                    // second accumulator, re-armed here
-  // sublayer output that is still a sum (`a` holds the rows it picks from): sum_k weight[row, k] a[slot[row, k]], with mix_h[row] in
+  // sublayer output that is still a sum (`a` holds the fp32 rows it picks from): sum_k weight[row, k] a[slot[row, k]], with mix_h[row] in
   // place of a row whose slot is negative, + weight[row, top] shared[row]
   int top, ld_mix, ld_shared;     // top 0: `a` is the output itself
   const int* slot;
@@ -32,17 +32,13 @@ struct SandwichArgs {
   const void *mix_h, *shared;     // operand precision; the type of `a` (null: none)
 };
 
-// Eight columns (V = 8) or one of the output of a sublayer.
+// Eight columns (V = 8) or one of the output of a sublayer that is still a sum.
 template <int V, typename TI, typename T>
 __device__ __forceinline__ void sublayer_cols(const SandwichArgs& A, const TI* a, size_t row, int i, float* v) {
   auto load = [](const auto* p, float* o) {
     if constexpr (V == 8) ld8(p, *reinterpret_cast<float(*)[8]>(o));
     else *o = ldf(p);
   };
-  if (!A.top) {
-    load(a + row * A.ld_a + i, v);
-    return;
-  }
   const int* sl = A.slot + row * A.top;
   const float* wt = A.weight + row * (A.top + 1);
 #pragma unroll
@@ -76,8 +72,8 @@ __device__ __forceinline__ void sublayer_cols(const SandwichArgs& A, const TI* a
 }
 
 // One CTA per row; NV groups of eight columns per thread held in registers.  A null `a` skips the sublayer output.
-// RMS: no means are taken, weights are one plus the stored ones and there are no biases.
-template <typename TI, typename T, int NV, bool RMS>
+// RMS: no means are taken, weights are one plus the stored ones and there are no biases.  SUM: the output is still a sum.
+template <typename TI, typename T, int NV, bool RMS, bool SUM>
 __global__ void __launch_bounds__(256)
 sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   pdl_trigger();
@@ -103,7 +99,7 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
     if (i < nvec) {
       ld8(A.x + row * A.E + 8 * i, xv[k]);
       if (ar) {
-        if constexpr (RMS) sublayer_cols<8, TI, T>(A, a, row, 8 * i, s[k]);
+        if constexpr (SUM) sublayer_cols<8, TI, T>(A, a, row, 8 * i, s[k]);
         else ld8(ar + 8 * i, s[k]);
         if (A.clear) clear8(ar + 8 * i);
         if (A.bias) {
@@ -185,7 +181,7 @@ sandwich_vec_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A)
 }
 
 // Any width: several passes over the row.
-template <typename TI, typename T, bool RMS>
+template <typename TI, typename T, bool RMS, bool SUM>
 __global__ void __launch_bounds__(256)
 sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   pdl_trigger();
@@ -198,7 +194,7 @@ sandwich_kernel(TI* __restrict__ a, T* __restrict__ h, const SandwichArgs A) {
   for (int i = threadIdx.x; i < A.nzero; i += 256) A.zero[row * A.nzero + i] = 0.f;
   auto in = [&](int i) {
     float v;
-    if constexpr (RMS) sublayer_cols<1, TI, T>(A, a, row, i, &v);
+    if constexpr (SUM) sublayer_cols<1, TI, T>(A, a, row, i, &v);
     else v = ldf(ar + i);
     return v + (A.bias ? A.bias_mult * A.bias[i] : 0.f);
   };
@@ -646,7 +642,7 @@ typedef __nv_bfloat16 bf16_t;
 
 // Every `f32` argument: the operand storage type is fp32 instead of bf16; `in_f32`: the GEMM output is fp32.
 
-template <typename TI, typename T, bool RMS>
+template <typename TI, typename T, bool RMS, bool SUM = false>
 static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, cudaStream_t st) {
   const bool vec = A.E % 8 == 0 && A.ld_a % 8 == 0 && A.ld_h % 8 == 0 && A.ld_mix % 8 == 0 && A.ld_shared % 8 == 0 &&
                    !((reinterpret_cast<uintptr_t>(A.mix_h) | reinterpret_cast<uintptr_t>(A.shared)) & 15) &&
@@ -654,12 +650,12 @@ static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, c
                       reinterpret_cast<uintptr_t>(A.w1) | reinterpret_cast<uintptr_t>(A.b1) | reinterpret_cast<uintptr_t>(A.w2) |
                       reinterpret_cast<uintptr_t>(A.b2) | reinterpret_cast<uintptr_t>(A.bias) | reinterpret_cast<uintptr_t>(A.step)) & 15);
   const int nv = vec ? (A.E / 8 + 255) / 256 : 0;
-#define GO(NV) launch_k(sandwich_vec_kernel<TI, T, NV, RMS>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A)
+#define GO(NV) launch_k(sandwich_vec_kernel<TI, T, NV, RMS, SUM>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A)
   if (nv == 1) GO(1);
   else if (nv == 2) GO(2);
   else if (nv == 3) GO(3);
   else if (nv == 4) GO(4);
-  else launch_k(sandwich_kernel<TI, T, RMS>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A);
+  else launch_k(sandwich_kernel<TI, T, RMS, SUM>, dim3(rows), dim3(256), 0, st, (TI*)a, (T*)h, A);
 #undef GO
 }
 
@@ -667,7 +663,7 @@ static void launch_sandwich(void* a, void* h, const SandwichArgs& A, int rows, c
 B200_API int b200_sandwich_norm(void* a, void* h, const SandwichArgs* Ap, int rows, int in_f32, int f32, int rms, void* stream) {
   const SandwichArgs A = *Ap;
   if (rows <= 0 || A.E <= 0 || !A.x || (A.clear && !in_f32) || (f32 && !in_f32) || (A.nzero && !A.zero)) return -1;
-  if (A.top && (!rms || !a || A.top < 0 || A.clear || !A.slot || !A.weight || !A.mix_h)) return -1;
+  if (A.top && (!rms || !in_f32 || !a || A.top < 0 || A.clear || !A.slot || !A.weight || !A.mix_h)) return -1;
   if ((a && (!A.w1 || (!rms && !A.b1))) || (A.w2 && ((!rms && !A.b2) || !h))) return -1;
 #define GO(RMS)                                                                \
   {                                                                            \
@@ -675,7 +671,10 @@ B200_API int b200_sandwich_norm(void* a, void* h, const SandwichArgs* Ap, int ro
     else if (in_f32) launch_sandwich<float, bf16_t, RMS>(a, h, A, rows, STREAM); \
     else launch_sandwich<bf16_t, bf16_t, RMS>(a, h, A, rows, STREAM);          \
   }
-  if (rms) GO(true) else GO(false)
+  if (A.top) {                       // few rows: the experts' are fp32
+    if (f32) launch_sandwich<float, float, true, true>(a, h, A, rows, STREAM);
+    else launch_sandwich<float, bf16_t, true, true>(a, h, A, rows, STREAM);
+  } else if (rms) GO(true) else GO(false)
 #undef GO
   return DONE;
 }

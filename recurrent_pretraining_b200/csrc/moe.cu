@@ -7,7 +7,8 @@
 //   * moe_route_rows    : the three in one CTA for the few rows of a decode step, slots without padding
 //   * moe_rows          : product of a decode step's rows with their experts' weights: a stream of weights through mma.sync,
 //                         fragments straight from memory
-// The weighted sum of a token's experts is formed by the norm that reads it (sandwich_norm in memory.cu).
+//   * moe_combine       : weighted sum of a token's experts, identity experts and the gated shared expert (prompts; in a decode step
+//                         the norm that reads the sum forms it: sandwich_norm in memory.cu)
 // Storage types: bf16 (serving) or fp32; arithmetic is fp32.  This file is built without fast-math approximations.
 #include "rowops.cuh"
 
@@ -401,6 +402,45 @@ static int launch_rows(const ExpertRows& P, int max_active, cudaStream_t st) {
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
+// ------------------------------------------------------------------------------------------------ sum of the experts
+// out[t] = sum_k weight[t, k] * (slot[t, k] < 0 ? h[t] : y[slot[t, k]]) + weight[t, top] * ys[t]
+template <typename T, int W>
+__global__ void __launch_bounds__(256)
+moe_combine_kernel(const T* __restrict__ h, int ld_h, const T* __restrict__ y, int ld_y, const T* __restrict__ ys, int ld_ys,
+                   const int* __restrict__ slot, const float* __restrict__ weight, T* __restrict__ out, int ld_out, int E, int top) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int* sl = slot + t * top;
+  const float* wt = weight + t * (top + 1);
+  for (int i = threadIdx.x * W; i < E; i += 256 * W) {
+    float acc[W], v[W];
+#pragma unroll
+    for (int j = 0; j < W; ++j) acc[j] = 0.f;
+    for (int k = 0; k < top; ++k) {
+      const int s = sl[k];
+      const float f = wt[k];
+      if constexpr (W == 8) {
+        if (s < 0) ld8(h + t * ld_h + i, v);
+        else ld8(y + static_cast<size_t>(s) * ld_y + i, v);
+      } else {
+        v[0] = s < 0 ? ldf(h + t * ld_h + i) : ldf(y + static_cast<size_t>(s) * ld_y + i);
+      }
+#pragma unroll
+      for (int j = 0; j < W; ++j) acc[j] += f * v[j];
+    }
+    if (ys) {
+      const float f = wt[top];
+      if constexpr (W == 8) ld8(ys + t * ld_ys + i, v);
+      else v[0] = ldf(ys + t * ld_ys + i);
+#pragma unroll
+      for (int j = 0; j < W; ++j) acc[j] += f * v[j];
+    }
+    if constexpr (W == 8) st8(out + t * ld_out + i, acc);
+    else stf(out + t * ld_out + i, acc[0]);
+  }
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -478,4 +518,18 @@ B200_API int b200_moe_rows(const ExpertRows* Pp, int max_active, int out_f32, in
   if (P.B <= 32) GO(4, 8, 1);
   GO(8, 8, 1);
 #undef GO
+}
+
+// all of one storage type
+B200_API int b200_moe_combine(const void* h, int ld_h, const void* y, int ld_y, const void* ys, int ld_ys, const int* slot, const float* weight,
+                              void* out, int ld_out, int T, int E, int top, int f32, void* stream) {
+  if (T <= 0 || E <= 0 || top <= 0) return -1;
+  const uintptr_t addr = reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(ys) | reinterpret_cast<uintptr_t>(out);
+  const bool vec = !(addr & 15) && !((E | ld_h | ld_y | ld_ys | ld_out) & 7);
+#define GO(T_, W) \
+  launch_k(moe_combine_kernel<T_, W>, dim3(T), dim3(256), 0, STREAM, (const T_*)h, ld_h, (const T_*)y, ld_y, (const T_*)ys, ld_ys, slot, weight, (T_*)out, ld_out, E, top)
+  if (f32) { if (vec) GO(float, 8); else GO(float, 1); }
+  else { if (vec) GO(bf16_t, 8); else GO(bf16_t, 1); }
+#undef GO
+  return DONE;
 }

@@ -129,7 +129,7 @@ def _norm(x, w, b, eps: float) -> torch.Tensor:
 @dataclass
 class RowSum:
     """A sublayer output that is still a sum: row t is sum_k weight[t, k] rows[slot[t, k]] (h[t] where the slot is negative)
-    + weight[t, top] shared[t].  ``rows`` and ``shared`` (or None) have one dtype, ``h`` is in operand precision."""
+    + weight[t, top] shared[t].  ``rows`` and ``shared`` (or None) have one dtype (fp32 where the norm kernel forms the sum), ``h`` is in operand precision."""
 
     rows: torch.Tensor
     slot: torch.Tensor
@@ -173,7 +173,7 @@ def sandwich_norm_(x: torch.Tensor, a, post, step, pre, eps: float, dtype: torch
     w2, b2 = pre if pre is not None else (None, None)
     many = {}
     if isinstance(a, RowSum):
-        assert a.h.dtype == dtype and (a.shared is None or a.shared.dtype == a.rows.dtype) and a.weight.is_contiguous() and a.slot.is_contiguous()
+        assert a.h.dtype == dtype and a.rows.dtype == F32 and (a.shared is None or a.shared.dtype == a.rows.dtype) and a.weight.is_contiguous() and a.slot.is_contiguous()
         many = dict(top=a.weight.shape[1] - 1, ld_mix=a.h.stride(0), ld_shared=0 if a.shared is None else a.shared.stride(0), slot=p(a.slot),
                     weight=p(a.weight), mix_h=p(a.h), shared=p(a.shared))
         a = a.rows

@@ -66,6 +66,7 @@ def _k():
             dispatch=K._sig("b200_moe_dispatch", [vp, i, vp, i, i] + [vp] * 4 + [i] * 3 + [vp]),
             route_rows=K._sig("b200_moe_route_rows", [vp, C.POINTER(_Route), C.POINTER(_RouteRows), i, vp]),
             rows=K._sig("b200_moe_rows", [C.POINTER(_ExpertRows), i, i, i, vp]),
+            combine=K._sig("b200_moe_combine", [vp, i] * 3 + [vp, vp, vp] + [i] * 5 + [vp]),
             gemm=K._sig("b200_gemm_grouped", [vp] * 3 + [i] * 7 + [vp, vp] + [i] * 3 + [vp, vp]))
     return _fns
 
@@ -166,6 +167,18 @@ def tile_rows(spec, T: int, dtype: torch.dtype) -> int:
     return 256 if T * spec.top >= 192 * spec.outputs else 128
 
 
+def combine(s: RowSum) -> torch.Tensor:
+    """The sum, in the common dtype of its parts."""
+    if not s.h.is_cuda:
+        return s.sum().to(s.h.dtype)
+    k, (T, E), y, ys = _k(), s.h.shape, s.rows, s.shared
+    assert y.dtype == s.h.dtype and (ys is None or ys.dtype == y.dtype)
+    out = torch.empty(T, pad8(E), dtype=y.dtype, device=y.device)[:, :E]
+    k.K._check(k.combine(s.h.data_ptr(), s.h.stride(0), y.data_ptr(), y.stride(0), k.K._ptr(ys), 0 if ys is None else ys.stride(0), s.slot.data_ptr(),
+                         s.weight.data_ptr(), out.data_ptr(), out.stride(0), T, E, s.slot.shape[1], _f32(y), k.K._stream()), "moe_combine")
+    return out
+
+
 def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     s, E = w.spec, h.shape[1]
     z = router_logits(h, w.router)
@@ -184,8 +197,8 @@ def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     return out.to(h.dtype)
 
 
-def mixture(w: MoeWeights, h: torch.Tensor):
-    """Mixture of experts of any number of rows h [T, E]; on a GPU the experts' rows, to be summed where they are read."""
+def mixture(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
+    """Mixture of experts of any number of rows h [T, E]."""
     if not h.is_cuda:
         return _plain(w, h)
     s, E = w.spec, h.shape[1]
@@ -193,11 +206,12 @@ def mixture(w: MoeWeights, h: torch.Tensor):
     a = grouped_linear(dispatch(w, h, p), w.up, s.ff, p, relu2=True)
     y = grouped_linear(a, w.down, E, p)
     ys = None if w.up_s is None else base.linear(base.linear(h, w.up_s, None, "relu2"), w.down_s)
-    return RowSum(y, p.slot, p.weight, h, ys)
+    return combine(RowSum(y, p.slot, p.weight, h, ys))
 
 
 def mixture_rows(w: MoeWeights, h: torch.Tensor):
-    """The same for the few bf16 rows of a decode step, as a stream of the chosen experts' weights."""
+    """The same for the few bf16 rows of a decode step, as a stream of the chosen experts' weights; on a GPU the experts' fp32 rows,
+    to be summed where they are read."""
     if not h.is_cuda or h.dtype == F32 or h.shape[0] > ROWS:
         return mixture(w, h)
     parts = mixture_rows_pieces(w, h)

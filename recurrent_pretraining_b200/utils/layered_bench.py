@@ -358,8 +358,7 @@ def routed_ops_prefill(model, seqs: list, t: Timer) -> list:
     ys = ops.linear(a_s, w.down_s)
     gemm("shared expert: down", lambda: ops.linear(a_s, w.down_s), T, E, s.shared)
     mixed = M.RowSum(y, p.slot, p.weight, h, ys)
-    t.op("sandwich_norm with the sum of the experts", lambda: M.sandwich_norm_(x, mixed, norms["norm2b"].pair, None, norms["norm1"].pair, 1e-6, torch.bfloat16),
-         2.0 * E * (n + 2 * T) + T * E * 10.0, 0)
+    t.op("moe: combine", lambda: X.combine(mixed), 2.0 * E * (n + 3 * T), 0)
     t.op("moe: whole", lambda: X.mixture(w, h), 4.0 * E * (T + s.experts * s.ff + s.shared), 4.0 * E * (n * s.ff + T * s.shared))
     mlp = model.layers[0].mlp
     ff = mlp.spec.ff

@@ -238,6 +238,10 @@ def test_norm_of_a_sum_of_experts(run, E, top):
         for kind in {dtype, torch.float32}:
             y = x.to(dev).clone()
             a = M.RowSum(pitched(rows, kind, dev), slot.to(dev), weight.to(dev), pitched(h, dtype, dev), pitched(shared, kind, dev) if with_shared else None)
+            if kind == dtype:
+                near(X.combine(a), s, dtype)
+            if kind != torch.float32:
+                continue
             out = M.sandwich_norm_(y, a, (w1.to(dev), None), None, (w1.to(dev), None), 1e-4, dtype)
             near(y, want, torch.float32)
             near(out, O.rms_norm(want, 1e-4, 1 + w1.double()), dtype)
