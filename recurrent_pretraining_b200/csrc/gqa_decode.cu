@@ -76,6 +76,39 @@ __device__ __forceinline__ float head_entry(const TI* x, int i, const float* w, 
   return v;
 }
 
+// Eight entries from i (a multiple of eight) on.
+template <typename TI>
+__device__ __forceinline__ void head_entries8(const TI* x, int i, const float* w, float r, int rot, const float* ct, const float* st, float (&v)[8]) {
+  const int half = rot >> 1;
+  if (i < rot && (half & 7)) {                                         // pairs do not fall into the same places of two groups
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = head_entry(x, i + j, w, r, rot, ct, st);
+    return;
+  }
+  ld8(x + i, v);
+  float f[8];
+  if (w) {
+    ld8(w + i, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= r * f[j];
+  }
+  if (i < rot) {
+    const bool low = i < half;
+    const int c = low ? i : i - half, o = low ? i + half : i - half;
+    float u[8], cs[8], sn[8];
+    ld8(x + o, u);
+    ld8(ct + c, cs);
+    ld8(st + c, sn);
+    if (w) {
+      ld8(w + o, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) u[j] *= r * f[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = low ? v[j] * cs[j] - u[j] * sn[j] : v[j] * cs[j] + u[j] * sn[j];
+  }
+}
+
 // NV: 16-column steps of the values that the accumulators hold.
 template <typename TI, int NV, int STAGES, bool RING>
 __global__ void __launch_bounds__(128)
@@ -147,10 +180,12 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
       __shared__ float red[8];
       const int nq = P.H * P.dim, nk = P.G * P.dim;                    // multiples of eight
       float sq = 0.f, sk = 0.f;
-      for (int i = 4 * threadIdx.x; i < nq + nk; i += 512) {
-        float v[4];
-        ld4(i < nq ? r + i : r + P.off_k + (i - nq), v);
-        const float t = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+#pragma unroll 4
+      for (int i = 8 * threadIdx.x; i < nq + nk; i += 1024) {
+        float v[8], t = 0.f;
+        ld8(i < nq ? r + i : r + P.off_k + (i - nq), v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) t += v[j] * v[j];
         if (i < nq) sq += t;
         else sk += t;
       }
@@ -166,15 +201,24 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     }
   }
   // queries, zero in the padding rows and columns; the ring's padding columns are zeroed once
-  for (int i = threadIdx.x; i < 16 * (kp / 2); i += 128) {
-    const int hh = i / (kp / 2), c = i - hh * (kp / 2);
-    float v = 0.f;
-    if (hh < nh && c < P.dim) {
-      const int at = (h0 + hh) * P.dim;
-      if constexpr (RING) v = head_entry(r + at, c, P.q_norm ? P.q_norm + at : nullptr, rq, P.rot, cos_t, sin_t);
-      else v = ldf(r + at + c) + P.in_bias[at + c];
+  if constexpr (RING) {
+    const int vecs = kp / 16;                                          // groups of eight columns of a staged row
+    for (int i = threadIdx.x; i < 16 * vecs; i += 128) {
+      const int hh = i / vecs, c = 8 * (i - hh * vecs);
+      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (hh < nh && c < P.dim) {
+        const int at = (h0 + hh) * P.dim;
+        head_entries8(r + at, c, P.q_norm ? P.q_norm + at : nullptr, rq, P.rot, cos_t, sin_t, v);
+      }
+      st8(reinterpret_cast<__nv_bfloat16*>(sq) + hh * (kp / 2) + c, v);
     }
-    reinterpret_cast<__nv_bfloat16*>(sq)[i] = f2bf(v);
+  } else {
+    for (int i = threadIdx.x; i < 16 * (kp / 2); i += 128) {
+      const int hh = i / (kp / 2), c = i - hh * (kp / 2);
+      float v = 0.f;
+      if (hh < nh && c < P.dim) v = ldf(r + (h0 + hh) * P.dim + c) + P.in_bias[(h0 + hh) * P.dim + c];
+      reinterpret_cast<__nv_bfloat16*>(sq)[i] = f2bf(v);
+    }
   }
   for (int i = lane; i < STAGES * GD_KEYS; i += 32) {
     uint8_t* s = ring + (i / GD_KEYS) * stage_bytes;
@@ -228,25 +272,35 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
     if (key0 + GD_KEYS > newest) {                                     // the newest token lies in this tile
       const int j = newest - key0;
       __nv_bfloat16* dst = base + static_cast<size_t>(slot_of(newest)) * P.ld_kv;
-      const float lam = RING && P.lam ? *P.lam : 0.f;
-      for (int c = lane; c < P.dim + P.vdim; c += 32) {
-        const bool isk = c < P.dim;
-        const int cc = isk ? c : c - P.dim, col = isk ? P.off_k + g * P.dim + cc : P.off_v + g * P.vdim + cc;
-        float f;
-        if constexpr (RING) {
+      if constexpr (RING) {
+        for (int c = 8 * lane; c < P.dim + P.vdim; c += 256) {
+          const bool isk = c < P.dim;
+          const int cc = isk ? c : c - P.dim, vc = g * P.vdim + cc;
+          float f[8];
           if (isk) {
-            f = head_entry(r + P.off_k + g * P.dim, cc, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk, P.rot, cos_t, sin_t);
+            head_entries8(r + P.off_k + g * P.dim, cc, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk, P.rot, cos_t, sin_t, f);
           } else {
-            f = ldf(r + col);
-            if (P.first_out) P.first_out[static_cast<size_t>(b) * P.ld_fout + g * P.vdim + cc] = f;
-            if (P.lam) f = (1.f - lam) * f + lam * P.first[static_cast<size_t>(b) * P.ld_first + g * P.vdim + cc];
+            ld8(r + P.off_v + vc, f);
+            if (P.first_out) st8(P.first_out + static_cast<size_t>(b) * P.ld_fout + vc, f);
+            if (P.lam) {
+              const float lam = *P.lam;
+              float e[8];
+              ld8(P.first + static_cast<size_t>(b) * P.ld_first + vc, e);
+#pragma unroll
+              for (int k = 0; k < 8; ++k) f[k] = (1.f - lam) * f[k] + lam * e[k];
+            }
           }
-        } else {
-          f = ldf(r + col) + P.in_bias[col];
+          st8(reinterpret_cast<__nv_bfloat16*>(sb + (isk ? j * kp : GD_KEYS * kp + j * vp)) + cc, f);
+          st8(dst + (isk ? g * P.dim : P.kv_v + g * P.vdim) + cc, f);
         }
-        const __nv_bfloat16 v = f2bf(f);
-        reinterpret_cast<__nv_bfloat16*>(sb + (isk ? j * kp : GD_KEYS * kp + j * vp))[cc] = v;
-        dst[(isk ? g * P.dim : P.kv_v + g * P.vdim) + cc] = v;
+      } else {
+        for (int c = lane; c < P.dim + P.vdim; c += 32) {
+          const bool isk = c < P.dim;
+          const int cc = isk ? c : c - P.dim, col = isk ? P.off_k + g * P.dim + cc : P.off_v + g * P.vdim + cc;
+          const __nv_bfloat16 v = f2bf(ldf(r + col) + P.in_bias[col]);
+          reinterpret_cast<__nv_bfloat16*>(sb + (isk ? j * kp : GD_KEYS * kp + j * vp))[cc] = v;
+          dst[(isk ? g * P.dim : P.kv_v + g * P.vdim) + cc] = v;
+        }
       }
       __syncwarp();
     }
@@ -451,7 +505,10 @@ B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_
 B200_API int b200_ring_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
   const GqaDecode& P = *Pp;
   if (!gqa_decode_ok(P, B) || P.size <= 0 || P.rot < 0 || (P.rot & 1) || P.rot > P.dim || (P.rot && (!P.cosT || !P.sinT)) || !P.q_norm != !P.k_norm ||
-      (P.lam && !P.first) || P.softcap < 0.f || (P.ld_in & 7) || (P.off_k & 7) || (reinterpret_cast<uintptr_t>(in) & 15)) return -1;
+      (P.lam && !P.first) || P.softcap < 0.f) return -1;
+  if (((P.ld_in | P.off_k | P.off_v | P.ld_first | P.ld_fout) & 7) ||
+      ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(P.q_norm) | reinterpret_cast<uintptr_t>(P.k_norm) | reinterpret_cast<uintptr_t>(P.cosT) |
+        reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.first) | reinterpret_cast<uintptr_t>(P.first_out)) & 15)) return -1;
   if (P.splits == 1 ? (!P.out || (P.ld_out & 7) || (reinterpret_cast<uintptr_t>(P.out) & 15)) : (P.out || !P.part_o || !P.part_ml)) return -1;
   return gqa_decode_launch<true>(in, P, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
 }
