@@ -25,7 +25,7 @@ NVCC_FLAGS = [
 ]
 
 # sources that keep the accurate forms of exp, division and square root
-ACCURATE = {"latent.cu", "memory.cu", "memory_chunk.cu", "grouped.cu", "moe.cu"}
+ACCURATE = {"latent.cu", "memory.cu", "memory_chunk.cu", "grouped.cu", "moe.cu", "depth.cu", "delta.cu", "delta_chunk.cu"}
 
 
 def flags_for(src: str) -> list:

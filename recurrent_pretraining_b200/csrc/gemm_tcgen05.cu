@@ -137,7 +137,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         for (int wi = 0; ok && more && work_item(wi, ot, kb0, kb1); ++wi) {
           int mt, nt;
           tile_coords(ot, tiles_m, tiles_n, p.raster, mt, nt);
-          const int m0 = mt * BM, n0 = nt * BN + (GROUPED ? p.tile_group[mt] * p.N : 0);
+          const int m0 = mt * BM, n0 = nt * BN + (GROUPED ? p.tile_group[mt] * (is_swiglu(MODE) ? 2 * p.N : p.N) : 0);
           for (int kb = kb0; kb < kb1; ++kb, ++it) {
             if (phase == 0 && it >= STAGES) { more = false; break; }
             const bool a_done = early_thread && phase == 1 && it < STAGES;   // loaded in phase 0
@@ -349,7 +349,7 @@ extern "C" __attribute__((visibility("default"))) int b200_set_pdl(int on) {
 namespace b200 {
 int gemm_2cta_dispatch(const void* A, const void* A2, const void* B, const GemmParams& p, int lda, int lda2, int ldb,
                        int a_mn, int b_mn, int out_mode, int bn, int max_ctas, cudaStream_t st);
-int gemm_2cta_grouped(const void* A, const void* B, const GemmParams& p, int lda, int ldb, int groups, cudaStream_t st);
+int gemm_2cta_grouped(const void* A, const void* B, const GemmParams& p, int lda, int ldb, int groups, bool gated, cudaStream_t st);
 static int g_use_2cta = 1;
 }  // namespace b200
 
@@ -390,20 +390,23 @@ B200_API void b200_gemm_set_bias(const float* bias, int act, int act_lo, int act
 
 // Grouped product C[slots, N] = act(A[slots, K] B_g^T), bf16: the slots lie in whole tiles of `rows` (128, or 256 for the pair kernel);
 // row tile i of the first *n_tiles belongs to group tile_group[i], whose weights are rows [g N, (g + 1) N) of B [groups N, ldb].
-// M: slots of A and C (all that may be used).  act as in OUT_BF16_BIAS_ACT.
+// M: slots of A and C (all that may be used).  act: 0 none, 1 relu^2, 4 silu gate: a group's weights are then 2 N rows [gate; up] and
+// C = silu(gate) * up (bn 128, or the pair kernel's 256).
 B200_API int b200_gemm_grouped(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int groups,
                                const int* tile_group, const int* n_tiles, int rows, int bn, int act, void* stream, int* err) {
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0 || !tile_group || !n_tiles || (rows != 128 && rows != 256) || M % rows || (bn != 128 && bn != 256) ||
-      (act != 0 && act != 1) || static_cast<long long>(groups) * N > 0x7fffffffll) return -29;
+      (act != 0 && act != 1 && act != 4) || static_cast<long long>(groups) * (act == 4 ? 2 : 1) * N > 0x7fffffffll) return -29;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   GemmParams p = {};
   p.M = M; p.N = N; p.K1 = K; p.ldc = ldc; p.swiglu_n = N; p.ksplit = 1; p.C = C; p.err = err;
-  p.raster = g_raster; p.act = act; p.tile_group = tile_group; p.n_row_tiles = n_tiles;
-  if (rows == 256) return bn == 256 ? gemm_2cta_grouped(A, B, p, lda, ldb, groups, st) : -29;
+  p.raster = g_raster; p.act = act == 4 ? 0 : act; p.tile_group = tile_group; p.n_row_tiles = n_tiles;
+  if (rows == 256) return bn == 256 ? gemm_2cta_grouped(A, B, p, lda, ldb, groups, act == 4, st) : -29;
+  if (act == 4 && bn != 128) return -29;
   CUtensorMap ta, tb;
   int rc = make_tmap_2d_bf16(&ta, A, M, K, lda, BM, BK);
-  if (!rc) rc = make_tmap_2d_bf16(&tb, B, static_cast<uint64_t>(groups) * N, K, ldb, bn, BK);
+  if (!rc) rc = make_tmap_2d_bf16(&tb, B, static_cast<uint64_t>(groups) * (act == 4 ? 2 : 1) * N, K, ldb, bn, BK);
   if (rc) return rc;
+  if (act == 4) return launch<128, false, false, OUT_SWIGLU, true>(ta, ta, tb, p, st, 0);
   if (bn == 128) return launch<128, false, false, OUT_BF16_BIAS_ACT, true>(ta, ta, tb, p, st, 0);
   return launch<256, false, false, OUT_BF16_BIAS_ACT, true>(ta, ta, tb, p, st, 0);
 }

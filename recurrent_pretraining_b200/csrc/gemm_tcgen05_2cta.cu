@@ -215,7 +215,7 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
         int mt, nt;
         tile_mn(tile, mt, nt);
         const int m0 = mt * (2 * BM2) + static_cast<int>(rank) * BM2;
-        const int n0 = is_swiglu(MODE) ? nt * BN_OUT + static_cast<int>(rank) * p.swiglu_n
+        const int n0 = is_swiglu(MODE) ? nt * BN_OUT + static_cast<int>(rank) * p.swiglu_n + (GROUPED ? p.tile_group[mt] * 2 * p.N : 0)
                                             : nt * BN + static_cast<int>(rank) * BNH + (GROUPED ? p.tile_group[mt] * p.N : 0);
         if constexpr (AG) {
           // the weight rows of this N-tile must have landed in the local buffer (every CTA's copiers add one)
@@ -539,13 +539,14 @@ int gemm_2cta_dispatch(const void* A, const void* A2, const void* B, const GemmP
 }
 
 // Entry used by b200_gemm_grouped: 256-row tiles.
-int gemm_2cta_grouped(const void* A, const void* B, const GemmParams& p, int lda, int ldb, int groups, cudaStream_t st) {
+int gemm_2cta_grouped(const void* A, const void* B, const GemmParams& p, int lda, int ldb, int groups, bool gated, cudaStream_t st) {
   CUtensorMap ta, tb, tc;
   int rc = make_tmap_2d_bf16(&ta, A, p.M, p.K1, lda, BM2, BK2);
-  if (!rc) rc = make_tmap_2d_bf16(&tb, B, static_cast<uint64_t>(groups) * p.N, p.K1, ldb, 128, BK2);
+  if (!rc) rc = make_tmap_2d_bf16(&tb, B, static_cast<uint64_t>(groups) * (gated ? 2 : 1) * p.N, p.K1, ldb, 128, BK2);
   if (rc) return rc;
   GemmParams pc = p;
   pc.tma_c = make_tmap_2d_bf16(&tc, p.C, p.M, p.N, p.ldc, 32, 64) == 0;
+  if (gated) return launch2<256, false, false, OUT_SWIGLU, false, true>(ta, ta, tb, pc, st, 0, nullptr, pc.tma_c ? &tc : nullptr);
   return launch2<256, false, false, OUT_BF16_BIAS_ACT, false, true>(ta, ta, tb, pc, st, 0, nullptr, pc.tma_c ? &tc : nullptr);
 }
 

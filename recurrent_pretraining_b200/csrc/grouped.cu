@@ -2,6 +2,7 @@
 //   * qkv_prep         : one projection row [q | k | v]: norm over all of q and of k, rotation of the leading dimensions of every
 //                        head (halves paired), values mixed with those of another layer; keys and values go to the step's key
 //                        stream and to the ring of the sequence
+//   * qkv_heads        : the same for layers that norm every head of q and k (after the rotation) and of v by itself
 //   * attention_merge  : key splits of a decode step, with an optional sink in the softmax's denominator
 // Storage types: bf16 (serving) or fp32; arithmetic is fp32.  This file is built without fast-math approximations.
 #include "rowops.cuh"
@@ -19,7 +20,16 @@ struct QkvRow {
   const float* lam;               // value mixing: v = (1 - lam) v + lam first; null: none
   const int *pos, *row;
   const int *sidx, *end;          // stream index; position after the portion's last token (null: every token goes to the ring)
+  int keep;                       // the ring holds the first `keep` positions of a sequence for good
+  const float* bias;              // of the projection row (null: none, or added already)
 };
+
+// The ring row of position p of token t, or null when it is not kept.
+template <typename T>
+__device__ __forceinline__ T* ring_row(const QkvRow& P, T* cache, size_t t, int p) {
+  if (!cache || (P.end && p >= P.keep && p < P.end[t] - (P.cap - P.keep))) return nullptr;
+  return cache + (static_cast<size_t>(P.row[t]) * P.cap + ring_slot(p, P.cap, P.keep)) * P.ld_kv;
+}
 
 template <int W> struct Pack { float v[W]; };
 template <int W, typename T> __device__ __forceinline__ Pack<W> ldw(const T* p) {
@@ -46,7 +56,7 @@ qkv_prep_kernel(const TI* in, T* q, const TF* __restrict__ first, float* __restr
   const TI* r = in + t * P.ld_in;
   const int p = P.pos[t];
   T* qd = q + t * P.ld_q;
-  T* kc = cache && (!P.end || p >= P.end[t] - P.cap) ? cache + (static_cast<size_t>(P.row[t]) * P.cap + p % P.cap) * P.ld_kv : nullptr;
+  T* kc = ring_row(P, cache, t, p);
   T* ks = stream ? stream + static_cast<size_t>(P.sidx[t]) * P.ld_kv : nullptr;
   float rq = 1.f, rk = 1.f;
   if (P.q_norm) {
@@ -131,6 +141,75 @@ qkv_prep_kernel(const TI* in, T* q, const TF* __restrict__ first, float* __restr
   }
 }
 
+// LANES lanes per (token, head of q, k or v): one pass for the sum of squares, which a rotation leaves alone, and one for the result.
+// q may lie in the projection row itself.
+template <typename TI, typename T, int W, int LANES>
+__global__ void __launch_bounds__(128)
+qkv_heads_kernel(const TI* in, T* q, T* __restrict__ cache, T* __restrict__ stream, const QkvRow P, int total) {
+  pdl_trigger();
+  pdl_wait();
+  const int heads = P.H + 2 * P.G, id = blockIdx.x * (128 / LANES) + threadIdx.x / LANES, lane = threadIdx.x % LANES;
+  const bool on = id < total;                                   // every lane takes part in the sums
+  const size_t t = on ? id / heads : 0;
+  const int h = on ? id % heads : 0, p = P.pos[t];
+  const int kind = h < P.H ? 0 : h < P.H + P.G ? 1 : 2, hh = kind == 0 ? h : kind == 1 ? h - P.H : h - P.H - P.G;
+  const int n = kind == 2 ? P.vdim : P.dim, at = hh * n, col = (kind == 0 ? 0 : kind == 1 ? P.off_k : P.off_v) + at;
+  const TI* src = in + t * P.ld_in + col;
+  const float* bias = P.bias ? P.bias + col : nullptr;
+  auto load = [&](int i) {
+    Pack<W> a = ldw<W>(src + i);
+    if (bias) {
+      const Pack<W> b = ldw<W>(bias + i);
+#pragma unroll
+      for (int j = 0; j < W; ++j) a.v[j] += b.v[j];
+    }
+    return a;
+  };
+  float ss = 0.f;
+  for (int i = lane * W; i < n; i += LANES * W) {
+    const Pack<W> a = load(i);
+#pragma unroll
+    for (int j = 0; j < W; ++j) ss += a.v[j] * a.v[j];
+  }
+#pragma unroll
+  for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!on) return;
+  const float f = 1.f / sqrtf(ss / static_cast<float>(n) + P.eps);
+  T* dst[2] = {nullptr, nullptr};
+  if (kind == 0) {
+    dst[0] = q + t * P.ld_q + at;
+  } else {
+    const int off = (kind == 2 ? P.kv_v : 0) + at;
+    if (T* kc = ring_row(P, cache, t, p)) dst[0] = kc + off;
+    if (stream) dst[1] = stream + static_cast<size_t>(P.sidx[t]) * P.ld_kv + off;
+  }
+  const int half = kind == 2 ? 0 : P.rot >> 1, pairs = half / W, units = pairs + (n - 2 * half) / W;
+  const float* ct = P.cosT + static_cast<size_t>(p) * half;
+  const float* st = P.sinT + static_cast<size_t>(p) * half;
+  for (int c = lane; c < units; c += LANES) {
+    const int i0 = c < pairs ? c * W : 2 * half + (c - pairs) * W, i1 = i0 + half;
+    Pack<W> a = load(i0), b;
+#pragma unroll
+    for (int j = 0; j < W; ++j) a.v[j] *= f;
+    if (c < pairs) {
+      b = load(i1);
+      const Pack<W> cs = ldw<W>(ct + i0), sn = ldw<W>(st + i0);
+#pragma unroll
+      for (int j = 0; j < W; ++j) {
+        const float x = a.v[j], y = b.v[j] * f;
+        a.v[j] = x * cs.v[j] - y * sn.v[j];
+        b.v[j] = y * cs.v[j] + x * sn.v[j];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (dst[k]) {
+        stw<W>(dst[k] + i0, a);
+        if (c < pairs) stw<W>(dst[k] + i1, b);
+      }
+  }
+}
+
 // out[b, h * vdim + d] = sum over splits / (sum of the softmax + exp(sink)).  CTA per (sequence, head): every warp takes each fourth
 // split, all its pieces requested at once.
 template <typename T>
@@ -176,14 +255,17 @@ typedef __nv_bfloat16 bf16_t;
 #define STREAM reinterpret_cast<cudaStream_t>(stream)
 #define DONE (cudaGetLastError() == cudaSuccess ? 0 : -2)
 
+static bool row_ok(const QkvRow& P, int T, const void* cache, const void* stream_buf, int in_f32, int f32) {
+  return T > 0 && P.H > 0 && P.G > 0 && P.H % P.G == 0 && P.dim > 0 && P.vdim > 0 && P.rot >= 0 && !(P.rot & 1) && P.rot <= P.dim && P.cap > 0 && P.keep >= 0 &&
+         P.pos && (!cache || P.row) && (!stream_buf || P.sidx) && (!P.rot || (P.cosT && P.sinT)) && (!f32 || in_f32);
+}
+
 // in: T projection rows (fp32 accumulators with in_f32); q: destination of the queries (may be `in`); first: values of the layer
 // that provides them (fp32 with first_f32), first_out: fp32 copy of this layer's unmixed values; stream_buf / cache may be null.
 B200_API int b200_qkv_prep(const void* in, void* q, const void* first, float* first_out, void* cache, void* stream_buf, const QkvRow* Pp,
                            int T, int in_f32, int f32, int first_f32, void* stream) {
   const QkvRow P = *Pp;
-  if (T <= 0 || P.H <= 0 || P.G <= 0 || P.H % P.G || P.dim <= 0 || P.vdim <= 0 || P.rot < 0 || (P.rot & 1) || P.rot > P.dim || P.cap <= 0 || !P.pos ||
-      (cache && !P.row) || (stream_buf && !P.sidx) || (P.lam && !first) || (P.rot && (!P.cosT || !P.sinT)) || (!P.q_norm != !P.k_norm) || (f32 && !in_f32))
-    return -1;
+  if (!row_ok(P, T, cache, stream_buf, in_f32, f32) || (P.lam && !first) || (!P.q_norm != !P.k_norm) || P.bias) return -1;
   const uintptr_t addr = reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(first) |
                          reinterpret_cast<uintptr_t>(first_out) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(stream_buf) |
                          reinterpret_cast<uintptr_t>(P.q_norm) | reinterpret_cast<uintptr_t>(P.k_norm) | reinterpret_cast<uintptr_t>(P.cosT) |
@@ -196,6 +278,26 @@ B200_API int b200_qkv_prep(const void* in, void* q, const void* first, float* fi
   else if (in_f32) GO(float, bf16_t, float)
   else if (first_f32) GO(bf16_t, bf16_t, float)
   else GO(bf16_t, bf16_t, bf16_t)
+#undef GO
+#undef GO2
+  return DONE;
+}
+
+// Arguments as in b200_qkv_prep; neither weighted norms nor value mixing.
+B200_API int b200_qkv_heads(const void* in, void* q, void* cache, void* stream_buf, const QkvRow* Pp, int T, int in_f32, int f32, void* stream) {
+  const QkvRow P = *Pp;
+  const long long total = static_cast<long long>(T) * (P.H + 2 * P.G);
+  if (!row_ok(P, T, cache, stream_buf, in_f32, f32) || P.q_norm || P.lam || total > 0x7fffffffll - 128) return -1;
+  const uintptr_t addr = reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(stream_buf) |
+                         reinterpret_cast<uintptr_t>(P.cosT) | reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.bias);
+  const bool vec = !(addr & 15) && !((P.dim | (P.rot >> 1) | P.vdim | P.ld_in | P.off_k | P.off_v | P.ld_q | P.ld_kv | P.kv_v) & 7);
+  const int n = P.dim > P.vdim ? P.dim : P.vdim;
+#define GO2(TI, T_, W, LN) \
+  launch_k(qkv_heads_kernel<TI, T_, W, LN>, dim3(static_cast<unsigned>((total + 128 / LN - 1) / (128 / LN))), dim3(128), 0, STREAM, (const TI*)in, (T_*)q, (T_*)cache, (T_*)stream_buf, P, static_cast<int>(total))
+#define GO(TI, T_) { if (!vec) GO2(TI, T_, 1, 32); else if (n <= 64) GO2(TI, T_, 8, 8); else if (n <= 128) GO2(TI, T_, 8, 16); else GO2(TI, T_, 8, 32); }
+  if (f32) GO(float, float)
+  else if (in_f32) GO(float, bf16_t)
+  else GO(bf16_t, bf16_t)
 #undef GO
 #undef GO2
   return DONE;

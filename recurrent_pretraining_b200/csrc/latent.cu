@@ -264,6 +264,7 @@ struct WindowAttn {
   float softcap;                  // 0: none; otherwise score = softcap * tanh(score / softcap)
   int chunk;                      // ring form, not 0: the query sees its chunk of that many positions instead of a window
   const float* sink;              // [H] stream form, null: none; exp(sink) is one more term of the softmax's denominator
+  int keep;                       // the first `keep` keys of a sequence are visible beside the window (not with chunks)
 };
 
 // CTA of four warps per (token, head, key split); a warp takes 32 keys at a time: one key per lane for the scores, one
@@ -287,8 +288,14 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   const bool ring = A.pos != nullptr;
   const int last = ring ? A.pos[t] : A.sidx[t];
   const int first = ring && A.chunk ? last - last % A.chunk : max(ring ? 0 : A.kbase[t], last - A.window + 1);
+  // visible keys are counted: kept ones in front of the window, then the window
+  const int origin = ring ? 0 : A.kbase[t], kept = A.chunk ? 0 : min(A.keep, first - origin), nkeys = kept + last - first + 1;
   const size_t ring0 = ring ? static_cast<size_t>(A.row[t]) * A.cap : 0;
-  const int nchunk = (last - first) / 32 + 1;
+  const int nchunk = (nkeys - 1) / 32 + 1;
+  auto key_of = [&](int e) -> size_t {
+    const int j = e < kept ? origin + e : first + (e - kept);
+    return ring ? ring0 + ring_slot(j, A.cap, A.keep) : static_cast<size_t>(j);
+  };
   const int hk = h / A.group;
   float scale = A.scale;
   if (A.temp_every > 0) scale *= query_temperature(ring ? last : last - A.kbase[t], A.temp_every, A.temp_coef);
@@ -297,10 +304,10 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
   float* op = os + warp * A.vdim;
   float* pp = ps + warp * 32;
   for (int c = split * 4 + warp; c < nchunk; c += 4 * A.splits) {
-    const int j0 = first + c * 32, j = j0 + lane, n = min(32, last - j0 + 1);
+    const int j0 = c * 32, n = min(32, nkeys - j0);
     float s = -INFINITY;
-    if (j <= last) {
-      const size_t key = ring ? ring0 + j % A.cap : static_cast<size_t>(j);
+    if (lane < n) {
+      const size_t key = key_of(j0 + lane);
       const T* a = k1 + key * A.k1_stride + static_cast<size_t>(hk) * A.k1_head;
       s = 0.f;
       for (int i = 0; i < A.d1; ++i) s += qs[i] * ldf(a + i);
@@ -309,7 +316,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
         for (int i = 0; i < A.d2; ++i) s += qs[A.d1 + i] * ldf(b + i);
       }
       s *= scale;
-      if (bias) s += bias[min(last - j, A.bias_len - 1)];
+      if (bias) s += bias[min(last - first - (j0 + lane), A.bias_len - 1)];     // not with kept keys
       if (A.softcap > 0.f) s = A.softcap * tanhf(s / A.softcap);
     }
     const float mn = fmaxf(m, warp_max(s));
@@ -321,7 +328,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k1, const T* _
     for (int d = lane; d < A.vdim; d += 32) {
       float o = op[d] * alpha;
       for (int k = 0; k < n; ++k) {
-        const size_t key = ring ? ring0 + (j0 + k) % A.cap : static_cast<size_t>(j0 + k);
+        const size_t key = key_of(j0 + k);
         o += pp[k] * ldf(v + key * A.v_stride + static_cast<size_t>(hk) * A.v_head + d);
       }
       op[d] = o;
@@ -706,7 +713,7 @@ B200_API int b200_window_attention(const void* q, const void* k1, const void* k2
   if (T <= 0 || A.H <= 0 || A.H > 65535 || A.group <= 0 || A.H % A.group || (A.bias && A.bias_len <= 0) || A.d1 <= 0 || A.d2 < 0 || A.vdim <= 0 || A.window <= 0 || A.splits < 1 || A.splits > 32) return -1;
   if (A.pos ? (!A.row || A.cap <= 0 || A.cap < A.window || !A.part_o || !A.part_ml || A.sink) : (!A.sidx || !A.kbase || A.splits != 1 || A.part_o || A.chunk || !out))
     return -1;
-  if (A.softcap < 0.f || A.chunk < 0) return -1;
+  if (A.softcap < 0.f || A.chunk < 0 || A.keep < 0 || (A.keep && (A.bias || A.chunk || A.temp_every > 0))) return -1;
   const size_t smem = (A.d1 + A.d2 + 128 + 4 * A.vdim + 8) * sizeof(float);
   if (smem > 200 * 1024) return -1;
   const dim3 grid(T, A.H, A.splits);

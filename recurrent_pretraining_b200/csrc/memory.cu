@@ -32,45 +32,6 @@ struct SandwichArgs {
   const void *mix_h, *shared;     // operand precision; the type of `a` (null: none)
 };
 
-// Eight columns (V = 8) or one of the output of a sublayer that is still a sum.
-template <int V, typename TI, typename T>
-__device__ __forceinline__ void sublayer_cols(const SandwichArgs& A, const TI* a, size_t row, int i, float* v) {
-  auto load = [](const auto* p, float* o) {
-    if constexpr (V == 8) ld8(p, *reinterpret_cast<float(*)[8]>(o));
-    else *o = ldf(p);
-  };
-  const int* sl = A.slot + row * A.top;
-  const float* wt = A.weight + row * (A.top + 1);
-#pragma unroll
-  for (int j = 0; j < V; ++j) v[j] = 0.f;
-  for (int k0 = 0; k0 < A.top; k0 += 4) {                 // four rows on their way at a time
-    float y[4][V], f[4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      f[u] = 0.f;
-      if (k0 + u < A.top) {
-        const int s = sl[k0 + u];
-        f[u] = wt[k0 + u];
-        if (s < 0) load(reinterpret_cast<const T*>(A.mix_h) + row * A.ld_mix + i, y[u]);
-        else load(a + static_cast<size_t>(s) * A.ld_a + i, y[u]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < V; ++j) y[u][j] = 0.f;
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < 4; ++u)
-#pragma unroll
-      for (int j = 0; j < V; ++j) v[j] += f[u] * y[u][j];
-  }
-  if (A.shared) {
-    float y[V];
-    load(reinterpret_cast<const TI*>(A.shared) + row * A.ld_shared + i, y);
-#pragma unroll
-    for (int j = 0; j < V; ++j) v[j] += wt[A.top] * y[j];
-  }
-}
-
 // One CTA per row; NV groups of eight columns per thread held in registers.  A null `a` skips the sublayer output.
 // RMS: no means are taken, weights are one plus the stored ones and there are no biases.  SUM: the output is still a sum.
 template <typename TI, typename T, int NV, bool RMS, bool SUM>

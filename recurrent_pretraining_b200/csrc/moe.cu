@@ -1,7 +1,7 @@
 // Mixture-of-experts feed-forward around the grouped matrix products:
 //   * moe_router_logits : product of a decode step's rows with the router, fp32 operands
-//   * moe_route         : softmax over the router outputs, choice of the best ones (scores plus correction), normalised weights,
-//                         rank of every choice inside its expert
+//   * moe_route         : softmax or sigmoid of the router outputs, choice of the best ones (scores plus correction; of the best groups
+//                         only), weights (normalised or not), rank of every choice inside its expert
 //   * moe_plan          : first slot of every expert (rows padded to whole tiles), expert of every tile
 //   * moe_dispatch      : rows into their experts' slots
 //   * moe_route_rows    : the three in one CTA for the few rows of a decode step, slots without padding
@@ -19,41 +19,85 @@ constexpr int MOE_MAX_OUT = 1024;       // router outputs
 struct RouteArgs {
   int experts, outputs, top;            // outputs: experts and identity experts
   int ld_z, gate;                       // gate: column `outputs` of z is the shared expert's gate
-  const float* correction;              // [outputs]
+  int sigmoid, normalize;               // scores are sigmoids (else a softmax); the chosen ones are divided by their sum
+  int groups, keep;                     // equal groups of neighbouring outputs; only those of the best `keep` groups can be chosen
+  const float* correction;              // [outputs]; null: none
   int* idx;                             // [T, top] chosen outputs
   float* weight;                        // [T, top + 1] their weights; then the gate's sigmoid
 };
 
-// Softmax and choice for one token by one warp; s, c: [outputs] scratch of the warp in shared memory.
+// Best of the lanes' (value, index) pairs; the lower index among equals.
+__device__ __forceinline__ void warp_best(float& best, int& at) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+    if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+  }
+}
+
+// Scores and choice for one token by one warp; s, c: [outputs] scratch of the warp in shared memory.
 __device__ __forceinline__ void route_token(const RouteArgs& R, const float* z, size_t t, float* s, float* c) {
   const int lane = threadIdx.x & 31;
-  float m = -INFINITY;
-  for (int i = lane; i < R.outputs; i += 32) m = fmaxf(m, z[i]);
-  m = warp_max(m);
-  float sum = 0.f;
-  for (int i = lane; i < R.outputs; i += 32) {
-    const float e = expf(z[i] - m);
-    s[i] = e;
-    sum += e;
+  float sum = 1.f;
+  if (R.sigmoid) {
+    for (int i = lane; i < R.outputs; i += 32) s[i] = sigmoid_f(z[i]);
+  } else {
+    float m = -INFINITY;
+    for (int i = lane; i < R.outputs; i += 32) m = fmaxf(m, z[i]);
+    m = warp_max(m);
+    sum = 0.f;
+    for (int i = lane; i < R.outputs; i += 32) {
+      const float e = expf(z[i] - m);
+      s[i] = e;
+      sum += e;
+    }
+    sum = warp_sum(sum);
   }
-  sum = warp_sum(sum);
   for (int i = lane; i < R.outputs; i += 32) {
     s[i] = s[i] / sum;
-    c[i] = s[i] + R.correction[i];
+    c[i] = s[i] + (R.correction ? R.correction[i] : 0.f);
   }
   __syncwarp();
+  if (R.keep < R.groups) {                // c keeps the scores of the best groups only; a lane owns every 32nd group
+    const int per = R.outputs / R.groups;
+    auto strength = [&](int g) {
+      float a = -INFINITY, b = -INFINITY;                 // the two largest
+      for (int i = g * per; i < (g + 1) * per; ++i) {
+        const float v = c[i];
+        if (v > a) { b = a; a = v; }
+        else if (v > b) b = v;
+      }
+      return per > 1 ? a + b : a;
+    };
+    float last = INFINITY;                // strength and index of the group chosen before
+    int last_at = -1;
+    for (int k = 0; k < R.keep; ++k) {
+      float best = -INFINITY;
+      int at = R.groups;
+      for (int g = lane; g < R.groups; g += 32) {
+        const float v = strength(g);
+        if ((v < last || (v == last && g > last_at)) && (v > best || (v == best && g < at))) { best = v; at = g; }
+      }
+      warp_best(best, at);
+      last = best;
+      last_at = at;
+    }
+    // the groups behind the last chosen one, in order of strength, are out
+    for (int g = lane; g < R.groups; g += 32) {
+      const float v = strength(g);
+      if (v < last || (v == last && g > last_at))
+        for (int i = g * per; i < (g + 1) * per; ++i) c[i] = -INFINITY;
+    }
+    __syncwarp();
+  }
   float total = 0.f, mine = 0.f;
   for (int k = 0; k < R.top; ++k) {
     float best = -INFINITY;
     int at = R.outputs;
     for (int i = lane; i < R.outputs; i += 32)
       if (c[i] > best) { best = c[i]; at = i; }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-      if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-    }
+    warp_best(best, at);
     at = min(at, R.outputs - 1);        // only if every score left is NaN
     const float w = s[at];
     total += w;
@@ -69,7 +113,8 @@ __device__ __forceinline__ void route_token(const RouteArgs& R, const float* z, 
     }
     __syncwarp();
   }
-  for (int k = lane; k < R.top; k += 32) R.weight[t * (R.top + 1) + k] /= total + 1e-20f;
+  if (R.normalize)
+    for (int k = lane; k < R.top; k += 32) R.weight[t * (R.top + 1) + k] /= total + 1e-20f;
   if (lane == 0) R.weight[t * (R.top + 1) + R.top] = R.gate ? sigmoid_f(z[R.outputs]) : 0.f;
 }
 
@@ -230,7 +275,7 @@ struct ExpertRows {
   int N, K, ld_w;                       // weights [groups * N, ld_w] bf16, rows padded to eight
   int Ns, Ks, ld_ws;                    // the shared expert's (Ns = 0: none)
   int ld_x, ld_y, ld_xs, ld_ys;         // input and output row pitches (shared: the same or other buffers)
-  int B, relu2;
+  int B, act;                           // act: 0 none, 1 relu^2, 2 silu gate: an expert's weights are 2 N rows [gate; up]
   const __nv_bfloat16 *w, *ws;
   const __nv_bfloat16 *x, *xs;          // input rows; x is indexed by row[slot] (gather) or by the slot, xs by the token
   int gather;
@@ -261,7 +306,8 @@ __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0
 // product is free, so a lane takes eight neighbouring columns of its weight rows and of its token as they lie in memory: they
 // serve two MMAs.  Weights and tokens pass through a queue in shared memory, several steps of 32 columns in flight: the weights' part
 // belongs to the thread alone, and so does the tokens' when the warps stand at different columns (KW > 1: no barriers).  With KW = 1 all
-// warps share one copy of the tokens and meet once a step.  NT: groups of eight tokens.
+// warps share one copy of the tokens and meet once a step.  NT: groups of eight tokens.  GATED: the sixteen
+// rows of a warp are eight gate rows and the eight up rows that belong to them, so that a thread holds both.
 template <int NT, int KW>
 struct RowsQueue {
   static constexpr bool SHARED_X = KW == 1;
@@ -269,7 +315,7 @@ struct RowsQueue {
   static constexpr int DEPTH = SHARED_X ? 8 : (NT >= 8 ? 5 : 8);
   static constexpr int BYTES = DEPTH * STEP;
 };
-template <typename TO, int NT, int RG, int KW>
+template <typename TO, int NT, int RG, int KW, bool GATED>
 __global__ void __launch_bounds__(256, NT * KW >= 32 ? 1 : 2)
 moe_rows_kernel(const ExpertRows P) {
   static_assert(RG * KW == 8, "eight warps");
@@ -288,15 +334,15 @@ moe_rows_kernel(const ExpertRows P) {
     s0 = P.first[y];
     n = P.first[y + 1] - s0;
   }
-  const int N = mine ? P.Ns : P.N, K = mine ? P.Ks : P.K, r0 = blockIdx.x * 16 * RG;
+  const int N = mine ? P.Ns : P.N, K = mine ? P.Ks : P.K, r0 = blockIdx.x * (GATED ? 8 : 16) * RG;
   if (r0 >= N) return;
   const int ldw = mine ? P.ld_ws : P.ld_w, ldx = mine ? P.ld_xs : P.ld_x;
-  const __nv_bfloat16* w = mine ? P.ws : P.w + static_cast<size_t>(e) * P.N * P.ld_w;
+  const __nv_bfloat16* w = mine ? P.ws : P.w + static_cast<size_t>(e) * (GATED ? 2 : 1) * P.N * P.ld_w;
   const __nv_bfloat16* x = mine ? P.xs : P.x;
-  const int q = lane & 3, rr = r0 + rg * 16 + (lane >> 2);
-  const bool live0 = rr < N, live1 = rr + 8 < N;
+  const int q = lane & 3, rr = r0 + rg * (GATED ? 8 : 16) + (lane >> 2), r1 = GATED ? N + rr : rr + 8;
+  const bool live0 = rr < N, live1 = GATED ? live0 : r1 < N;
   const __nv_bfloat16* w0 = w + static_cast<size_t>(live0 ? rr : 0) * ldw + 8 * q;
-  const __nv_bfloat16* w1 = w + static_cast<size_t>(live1 ? rr + 8 : 0) * ldw + 8 * q;
+  const __nv_bfloat16* w1 = w + static_cast<size_t>(live1 ? r1 : 0) * ldw + 8 * q;
   // this thread's source of token pieces: its own token of every group, or with SHARED_X one piece of one token
   const __nv_bfloat16* xp[Q::SHARED_X ? 1 : NT];
   bool xl[Q::SHARED_X ? 1 : NT];
@@ -373,32 +419,46 @@ moe_rows_kernel(const ExpertRows P) {
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
     if (8 * j >= n) break;
+    float v[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = (lane >> 2) + 8 * (i >> 1), tk = 8 * j + 2 * q + (i & 1);
-      float v = c[j][i];
+      v[i] = c[j][i];
 #pragma unroll
-      for (int g = 0; g < KW - 1; ++g) v += part[(g * RG + rg) * 16 * LP + r * LP + tk];
-      if (P.relu2) {
-        v = fmaxf(v, 0.f);
-        v *= v;
+      for (int g = 0; g < KW - 1; ++g) v[i] += part[(g * RG + rg) * 16 * LP + r * LP + tk];
+    }
+    if constexpr (GATED) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int tk = 8 * j + 2 * q + i;
+        if (tk < n && live0) stf(y + static_cast<size_t>(tk) * ldy + rr, silu_f(v[i]) * v[i + 2]);
       }
-      if (tk < n && r0 + rg * 16 + r < N) stf(y + static_cast<size_t>(tk) * ldy + r0 + rg * 16 + r, v);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int r = (lane >> 2) + 8 * (i >> 1), tk = 8 * j + 2 * q + (i & 1);
+        if (P.act == 1) {
+          v[i] = fmaxf(v[i], 0.f);
+          v[i] *= v[i];
+        }
+        if (tk < n && r0 + rg * 16 + r < N) stf(y + static_cast<size_t>(tk) * ldy + r0 + rg * 16 + r, v[i]);
+      }
     }
   }
 }
 
-template <typename TO, int NT, int RG, int KW>
+template <typename TO, int NT, int RG, int KW, bool GATED = false>
 static int launch_rows(const ExpertRows& P, int max_active, cudaStream_t st) {
   constexpr int QUEUE = RowsQueue<NT, KW>::BYTES, PART = (KW - 1) * RG * 16 * (8 * NT + 1) * 4, SMEM = QUEUE > PART ? QUEUE : PART;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(moe_rows_kernel<TO, NT, RG, KW>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return -3;
+    if (cudaFuncSetAttribute(moe_rows_kernel<TO, NT, RG, KW, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return -3;
     configured = true;
   }
   const int rows = P.N > P.Ns ? P.N : P.Ns;
-  const dim3 grid((rows + 16 * RG - 1) / (16 * RG), max_active + (P.Ns ? 1 : 0));
-  launch_k(moe_rows_kernel<TO, NT, RG, KW>, grid, dim3(256), static_cast<size_t>(SMEM), st, P);
+  constexpr int OUT = (GATED ? 8 : 16) * RG;         // results per CTA and token
+  const dim3 grid((rows + OUT - 1) / OUT, max_active + (P.Ns ? 1 : 0));
+  launch_k(moe_rows_kernel<TO, NT, RG, KW, GATED>, grid, dim3(256), static_cast<size_t>(SMEM), st, P);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
@@ -459,7 +519,7 @@ B200_API int b200_moe_router_logits(const void* x, int ld_x, const void* w, int 
 
 static bool route_ok(const RouteArgs& R) {
   return R.experts > 0 && R.outputs >= R.experts && R.outputs <= MOE_MAX_OUT && R.top > 0 && R.top <= R.outputs && R.ld_z >= R.outputs + (R.gate ? 1 : 0) &&
-         R.correction && R.idx && R.weight;
+         R.groups > 0 && R.outputs % R.groups == 0 && R.keep > 0 && R.keep <= R.groups && R.top <= R.outputs / R.groups * R.keep && R.idx && R.weight;
 }
 
 // z: [T, ld_z] router logits; count: [experts], zero on entry; rank: [T, top]; tile_expert: [max_tiles], rows slots each.
@@ -506,6 +566,15 @@ B200_API int b200_moe_rows(const ExpertRows* Pp, int max_active, int out_f32, in
       (P.Ns && (P.Ks <= 0 || !P.ws || !P.xs || !P.ys))) return -1;
   if (((P.ld_w | P.ld_x | P.ld_ws | P.ld_xs) & 7) || ((reinterpret_cast<uintptr_t>(P.w) | reinterpret_cast<uintptr_t>(P.ws) | reinterpret_cast<uintptr_t>(P.x) |
                                                       reinterpret_cast<uintptr_t>(P.xs)) & 15)) return -1;
+  if (P.act < 0 || P.act > 2) return -1;
+  if (P.act == 2) {
+    if (P.Ns || out_f32 || narrow) return -1;
+    if (P.B <= 2) return launch_rows<bf16_t, 1, 1, 8, true>(P, max_active, STREAM);
+    if (P.B <= 8) return launch_rows<bf16_t, 1, 2, 4, true>(P, max_active, STREAM);
+    if (P.B <= 16) return launch_rows<bf16_t, 2, 4, 2, true>(P, max_active, STREAM);
+    if (P.B <= 32) return launch_rows<bf16_t, 4, 8, 1, true>(P, max_active, STREAM);
+    return launch_rows<bf16_t, 8, 8, 1, true>(P, max_active, STREAM);
+  }
 #define GO(NT, RG, KW) return out_f32 ? launch_rows<float, NT, RG, KW>(P, max_active, STREAM) : launch_rows<bf16_t, NT, RG, KW>(P, max_active, STREAM)
   if (narrow) {
     if (P.B <= 8) GO(1, 1, 8);

@@ -75,6 +75,50 @@ __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefe
 __device__ __forceinline__ float query_temperature(int p, int every, float coef) {
   return 1.f + coef * logf(static_cast<float>((p + 1) / every + 1));
 }
+// slot of position p in a ring of `cap` slots whose first `keep` hold the sequence's first positions for good
+__device__ __forceinline__ int ring_slot(int p, int cap, int keep) { return p < cap ? p : keep + (p - keep) % (cap - keep); }
+// log(1 + exp(v))
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
+
+// Eight columns (V = 8) or one of the output of a sublayer that is still a sum (`Args`: SandwichArgs or DepthArgs): row `row` is
+// sum_k weight[row, k] a[slot[row, k]], with mix_h[row] in place of a row whose slot is negative, + weight[row, top] shared[row].
+template <int V, typename TI, typename T, typename Args>
+__device__ __forceinline__ void sublayer_cols(const Args& A, const TI* a, size_t row, int i, float* v) {
+  auto load = [](const auto* p, float* o) {
+    if constexpr (V == 8) ld8(p, *reinterpret_cast<float(*)[8]>(o));
+    else *o = ldf(p);
+  };
+  const int* sl = A.slot + row * A.top;
+  const float* wt = A.weight + row * (A.top + 1);
+#pragma unroll
+  for (int j = 0; j < V; ++j) v[j] = 0.f;
+  for (int k0 = 0; k0 < A.top; k0 += 4) {                 // four rows on their way at a time
+    float y[4][V], f[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      f[u] = 0.f;
+      if (k0 + u < A.top) {
+        const int s = sl[k0 + u];
+        f[u] = wt[k0 + u];
+        if (s < 0) load(reinterpret_cast<const T*>(A.mix_h) + row * A.ld_mix + i, y[u]);
+        else load(a + static_cast<size_t>(s) * A.ld_a + i, y[u]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[u][j] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += f[u] * y[u][j];
+  }
+  if (A.shared) {
+    float y[V];
+    load(reinterpret_cast<const TI*>(A.shared) + row * A.ld_shared + i, y);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] += wt[A.top] * y[j];
+  }
+}
 
 }  // namespace b200

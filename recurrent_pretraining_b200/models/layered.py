@@ -5,7 +5,9 @@ is the design's norm style:
 
 * "post_rms": a sublayer reads the stream itself; ``x += mult * rmsnorm(sublayer(x))``;
 * "sandwich": ``x += layernorm(sublayer(layernorm(x)))``; one kernel adds a sublayer's output and norms the next one's input;
-* "sandwich_rms": the same with RMS norms whose weights are stored around zero.
+* "sandwich_rms": the same with RMS norms whose weights are stored around zero;
+* "post_group_rms": as "post_rms", with norms over groups of columns, and at the end of a layer the stream is replaced by a weighted
+  sum of the embedding output and all layer results so far.
 
 The residual stream, norms, rotations, scores, softmax, gates of recurrences and recurrent state are fp32; matrix operands are
 bf16 (serving) or fp32.  A range of layers may be executed several times (``LayeredConfig.runs``); every execution has its own
@@ -18,12 +20,14 @@ Execution forms, both over sequence rows of a ``RowCache``:
 """
 from __future__ import annotations
 
+import math
 import os
 from typing import Optional
 
 import torch
 import torch.nn as nn
 
+from ..ops import depth as depth_ops
 from ..ops import latent as ops
 from ..ops import memory as mem_ops
 from .kv_cache import HybridCache, LatentRingCache, RowCache
@@ -67,19 +71,22 @@ class Layer(nn.Module):
     def __init__(self, cfg: LayeredConfig, i: int, dtype, device):
         super().__init__()
         spec = cfg.layers[i]
-        self.mix = MIXERS[spec.type](spec.mixer, cfg.width, cfg.norm_eps, dtype, device)
-        self.mlp = None if spec.mlp is None else MLPS[cfg.design.mlps[spec.mlp_kind]](spec.mlp, cfg.width, dtype, device)
+        self.mix = MIXERS[type(spec.mixer)](spec.mixer, cfg.width, cfg.norm_eps, dtype, device)
+        self.mlp = None if spec.mlp is None else MLPS[cfg.design.mlps[spec.mlp_kind][0]](spec.mlp, cfg.width, dtype, device)
         names = ("norm1",) if self.mlp is None else ("norm1", "norm2")
         if cfg.design.sandwich:
             norm = NORMS[cfg.design.norms]
             self.norms = nn.ModuleDict({n + side: norm(cfg.width, device) for n in names for side in ("", "b")})   # before and after
         else:
             self.norms = nn.ParameterDict({n: vector(cfg.width, device) for n in names})
+        self.dwa = vector(i + 2, device) if cfg.design.depth_average else None
 
     def checkpoint_tensors(self) -> dict:
         out: dict = {}
         for name, n in self.norms.items():
             out.update(n.checkpoint_tensors(name) if isinstance(n, nn.Module) else {name: n})
+        if self.dwa is not None:
+            out["dwa"] = self.dwa
         out.update({f"mix.{k}": v for k, v in self.mix.checkpoint_tensors().items()})
         if self.mlp is not None:
             out.update({f"mlp.{k}": v for k, v in self.mlp.checkpoint_tensors().items()})
@@ -96,7 +103,7 @@ class LayeredForCausalLM(nn.Module):
         self.config, self.dtype = config, dtype
         self.embed = weight(config.vocab, config.width, dtype, device)
         self.layers = nn.ModuleList(Layer(config, i, dtype, device) for i in range(len(config.layers)))
-        self.sandwich = config.design.sandwich
+        self.sandwich, self.depth_average = config.design.sandwich, config.design.depth_average
         self.final_norm = NORMS[config.design.norms](config.width, device) if self.sandwich else vector(config.width, device)
         self.head = weight(config.vocab, config.width, dtype, device)
         self.loop_step = None if config.loop is None else nn.Parameter(
@@ -155,12 +162,20 @@ class LayeredForCausalLM(nn.Module):
     @torch.no_grad()
     def init_weights(self, seed: int = 0) -> "LayeredForCausalLM":
         """Random weights: matrices normal with deviation 1 / sqrt(fan in), norm factors one, biases zero (forget gates: spread
-        over 3 .. 6, so that memories of different length exist), mixed values half and half."""
+        over 3 .. 6, decays of delta memories: 1/16 .. 1 at a step of softplus(-2), so that memories of different length exist), mixed values half and
+        half, sums over depth mostly the layer's own result."""
         g = torch.Generator(device=self.device).manual_seed(seed)
         zero = (".b", ".sink", ".correction") + ((".norm1", ".norm2", "b", "final.norm") if self.config.design.norms == "sandwich_rms" else ())
         for name, t in self.checkpoint_tensors().items():
             if name.endswith(".mix.f.b"):
                 t.copy_(torch.linspace(3.0, 6.0, t.numel(), device=t.device))
+            elif name.endswith(".mix.A_log"):
+                t.copy_(torch.linspace(math.log(1 / 16), 0.0, t.numel(), device=t.device))
+            elif name.endswith(".mix.dt_bias"):
+                t.fill_(-2.0)
+            elif name.endswith(".dwa"):
+                t.fill_(0.5 / max(1, t.numel() - 1))
+                t[-1] = 0.5
             elif t.dim() == 0:
                 t.fill_(0.5)
             elif t.dim() == 1:
@@ -173,7 +188,7 @@ class LayeredForCausalLM(nn.Module):
 
     # -- plumbing ----------------------------------------------------------------------------------------------------
     def new_cache(self, max_rows: int, max_len: int) -> RowCache:
-        if self.sandwich:
+        if not self.config.latent:
             shapes = {(run.index, name): shape for run in self.runs
                       for name, shape in self.layers[run.layer].mix.cache_shapes(max_len).items()}
             cache = HybridCache(shapes, max_rows, max_len, self.device)
@@ -198,6 +213,10 @@ class LayeredForCausalLM(nn.Module):
     def _start(self, tok):
         """Residual stream and the first sublayer's input."""
         c = self.config
+        if self.depth_average:
+            past = torch.empty(len(self.layers), tok.numel(), c.width, dtype=torch.float32, device=tok.device)
+            _, h = ops.embed(tok, self.embed[:, :c.width], out=past[0])
+            return depth_ops.DepthStream.begin(past), h
         if not self.sandwich:
             return ops.embed(tok, self.embed[:, :c.width])
         x, _ = ops.embed(tok, self.embed[:, :c.width], c.embed_scale, copy=False)
@@ -208,6 +227,10 @@ class LayeredForCausalLM(nn.Module):
         """Add the output of sublayer ``name`` ("norm1": mixer, "norm2": feed-forward) of execution ``n`` to the stream; returns
         the next sublayer's input (after the last one: the normed input of the head with ``final``)."""
         c, layer = self.config, self.layers[self.runs[n].layer]
+        if self.depth_average:
+            end = name == ("norm1" if layer.mlp is None else "norm2")
+            return depth_ops.depth_norm_(x, out, layer.norms[name], c.norm_groups, c.norm_eps, self.dtype, part.out_bias, clear, zero,
+                                         layer.dwa if end else None)
         if not self.sandwich:
             return ops.rms_residual_(x, out, part.out_bias, layer.norms[name], c.norm_eps, c.residual_mult, self.dtype, clear, zero)
         step, pre = None, None
@@ -224,7 +247,9 @@ class LayeredForCausalLM(nn.Module):
     def _logits(self, x, idx, h=None):
         """``h``: the final norm of all rows, where it is formed already.  The logits' factor is part of that norm."""
         c = self.config
-        if h is None:
+        if self.depth_average:
+            h = depth_ops.group_norm_rows(x.x, idx, self.final_norm, c.norm_groups, c.norm_eps, self.dtype)
+        elif h is None:
             h = mem_ops.norm_rows(x, idx, *self.final_norm.pair, c.norm_eps, self.dtype, c.logit_scale) if self.sandwich else \
                 ops.rmsnorm_rows(x, idx, self.final_norm, c.norm_eps, self.dtype)
         return ops.linear(h, self.head[:, :c.width], out_f32=True)
@@ -236,9 +261,9 @@ class LayeredForCausalLM(nn.Module):
         empty: nothing is computed past the last layer).  ``hidden`` collects the residual stream after every execution of a
         layer.  Without a cache the portions are whole sequences and nothing is kept."""
         ctx = StepContext(self.config, step, cache)
-        if self.sandwich and cache is None:
+        if not self.config.latent and cache is None:
             ctx.cache = self.new_cache(1 + max(r for r, _, _ in step.portions), max(n for _, _, n in step.portions))
-        elif not self.sandwich:
+        elif self.config.latent:
             ctx.windows = self.config.latent_windows()
         ctx.rope = ctx.cache.rope if ctx.cache is not None else self._rope(max(s + n for _, s, n in step.portions))
         x, h = self._start(step.tok)
@@ -249,7 +274,8 @@ class LayeredForCausalLM(nn.Module):
             if layer.mlp is not None:
                 h = self._add(x, n, "norm2", layer.mlp(h), layer.mlp)
             if hidden is not None:
-                hidden.append(x.clone() if before is None else x - before)     # the stream already holds the next pass's vector
+                stream = x.x if self.depth_average else x
+                hidden.append(stream.clone() if before is None else stream - before)     # the stream already holds the next pass's vector
         if want is not None and not len(want):
             return None
         idx = None if want is None else torch.tensor(want, dtype=torch.int32).to(self.device)

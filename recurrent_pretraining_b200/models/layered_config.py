@@ -14,43 +14,17 @@ Architectures:
 * ``Dusilorn``: grouped-query attention, either inside chunks (normed queries and keys, no rotation, an attention sink) or under
   a sliding window (rotated), scores capped, values mixed with those of the first such layer; a gated feed-forward or a mixture
   of experts with identity experts and a gated shared expert; RMS norms before and after every sublayer.
+* ``Bolovik``: gated delta-rule memories behind short convolutions, or grouped-query attention under a sliding window that keeps the
+  first tokens (biased, rotated, then normed per head); a gated feed-forward or a mixture of gated experts chosen within the best groups;
+  RMS norms over groups of columns on the sublayer outputs only; a weighted sum of all earlier results after every layer.
 """
 from __future__ import annotations
 
 import json
 import math
 import os
-from dataclasses import dataclass, field, replace
-from typing import Optional
-
-
-@dataclass(frozen=True)
-class Design:
-    """What an architecture fixes beside its configuration."""
-
-    mixers: tuple                    # mixer types a layer may have
-    norms: str                       # "post_rms": x += mult * rms(f(x)); "sandwich": x += ln(f(ln(x))); "sandwich_rms": the
-                                     # same with RMS norms whose weights are stored around zero
-    mlps: dict                       # feed-forward kinds a layer may have -> form: "relu2": biased, two matrices; "geglu" /
-                                     # "swiglu": gated by tanh-GELU / silu, no biases; "relu2_moe": mixture of squared-ReLU experts
-    keys: tuple                      # keys of config.json beside the common ones
-
-    @property
-    def sandwich(self) -> bool:
-        return self.norms.startswith("sandwich")
-
-
-DESIGNS = {
-    "Gasovik": Design(("latent_attention",), "post_rms", {"dense": "relu2"}, ("residual_mult",)),
-    "Fatudra": Design(("parallel", "mlstm"), "sandwich", {"dense": "geglu"}, ("embedding", "loop")),
-    "Dusilorn": Design(("attention", "attention_2"), "sandwich_rms", {"dense": "swiglu", "moe": "relu2_moe"}, ("embedding", "logit_scale")),
-}
-ARCHITECTURES = tuple(DESIGNS)
-
-
-def is_layered(config: dict) -> bool:
-    """Whether a parsed ``config.json`` describes a model of this family."""
-    return config.get("architecture") in ARCHITECTURES
+from dataclasses import asdict, dataclass, field, fields, replace
+from typing import ClassVar, Optional
 
 
 def _take(d: dict, known: tuple, where: str) -> None:
@@ -81,31 +55,61 @@ class YarnScaling:
         """Factor on both cos and sin."""
         return 0.1 * math.log(self.factor) + 1.0
 
+    def stretched(self, f: list, dims: int, base: float) -> list:
+        return [v / self.factor * r + v * (1 - r) for v, r in zip(f, self.ramp(dims, base))]
+
+
+@dataclass(frozen=True)
+class WavelengthScaling:
+    """Frequency scaling by wavelength: those of at most ``original / high`` positions stay, those beyond ``original / low`` are
+    divided by ``factor``, the ones between are interpolated."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+    magnitude = 1.0
+
+    def stretched(self, f: list, dims: int, base: float) -> list:
+        out = []
+        for v in f:
+            length = 2 * math.pi / v
+            if length < self.original / self.high:
+                out.append(v)
+            elif length > self.original / self.low:
+                out.append(v / self.factor)
+            else:
+                s = (self.original / length - self.low) / (self.high - self.low) if self.high != self.low else 1.0
+                out.append((1 - s) * v / self.factor + s * v)
+        return out
+
 
 @dataclass(frozen=True)
 class RotarySpec:
     base: float
     dims: int
-    scaling: Optional[YarnScaling] = None
+    scaling: Optional[object] = None         # YarnScaling or WavelengthScaling
 
     def frequencies(self) -> list:
         """Radians per position of every pair."""
         f = [self.base ** (-2 * i / self.dims) for i in range(self.dims // 2)]
         if self.scaling is None:
             return f
-        return [v / self.scaling.factor * r + v * (1 - r) for v, r in zip(f, self.scaling.ramp(self.dims, self.base))]
+        return self.scaling.stretched(f, self.dims, self.base)
 
     @property
     def magnitude(self) -> float:
         return 1.0 if self.scaling is None else self.scaling.magnitude
 
     @classmethod
-    def from_dict(cls, d: dict) -> "RotarySpec":
+    def from_dict(cls, d: dict, scaling=YarnScaling) -> "RotarySpec":
+        """``scaling``: the kind of scaling that the mixer may have."""
         _take(d, ("base", "dims", "scaling"), "rot")
         sc = d.get("scaling")
         if sc is not None:
-            _take(sc, ("factor", "original", "fast", "slow"), "rot.scaling")
-            sc = YarnScaling(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"]))
+            names = [f.name for f in fields(scaling)]
+            _take(sc, tuple(names), "rot.scaling")
+            sc = scaling(**{k: float(sc[k]) for k in names})
         if d["dims"] <= 0 or d["dims"] % 2:
             raise ValueError(f"rot.dims must be a positive even number, not {d['dims']}")
         return cls(float(d["base"]), int(d["dims"]), sc)
@@ -113,8 +117,7 @@ class RotarySpec:
     def to_dict(self) -> dict:
         out = {"base": self.base, "dims": self.dims}
         if self.scaling is not None:
-            s = self.scaling
-            out["scaling"] = {"factor": s.factor, "original": s.original, "fast": s.fast, "slow": s.slow}
+            out["scaling"] = asdict(self.scaling)
         return out
 
 
@@ -232,13 +235,18 @@ class BiasedAttentionSpec:
 @dataclass(frozen=True)
 class GroupedAttentionSpec:
     """Grouped-query attention with capped scores: ``softcap * tanh(q . k * scale / softcap)`` (None: not capped); ``size`` tokens of a window or a
-    chunk are visible.  Subclasses fix the kind of mask, whether q and k are normed (over the whole projection) or rotated, and
+    chunk are visible, under a window the first ``keep`` of the sequence as well.  Subclasses fix the kind of mask, how q, k and v are formed and
     whether a learned sink takes part in the softmax.  ``v_mix``: values are mixed with those of the first layer that mixes."""
 
     chunked = False                  # visible: the own chunk (counted from position 0); else the last ``size`` positions
-    qk_norm = False
+    keeps = False                    # the first tokens may be kept visible
+    capped = True                    # scores may be capped, values mixed
+    biased = False                   # q, k and v have biases
+    qk_norm = False                  # RMS norms with weights over all of q and of k
+    head_norm = False                # RMS norms without weights over every head of q and k (after their rotation) and of v
     sink = False
     rotated = False
+    scaling: ClassVar = None         # kind of frequency scaling that the rotation may have
 
     heads: int
     kv_heads: int
@@ -249,26 +257,34 @@ class GroupedAttentionSpec:
     softcap: Optional[float]
     v_mix: bool = False
     rot: Optional[RotarySpec] = None
+    keep: int = 0
 
     @classmethod
     def from_dict(cls, d: dict) -> "GroupedAttentionSpec":
-        _take(d, ("heads", "kv_heads", "dim", "vdim", "mask", "scale", "softcap", "v_mix") + (("rot",) if cls.rotated else ()), "mixer")
-        _take(d["mask"], ("size",), "mixer.mask")
+        _take(d, ("heads", "kv_heads", "dim", "vdim", "mask", "scale") + (("softcap", "v_mix") if cls.capped else ()) + (("rot",) if cls.rotated else ()), "mixer")
+        _take(d["mask"], ("size",) + (("keep_first",) if cls.keeps else ()), "mixer.mask")
+        rot = None
+        if cls.rotated:
+            if cls.scaling is None and d["rot"].get("scaling") is not None:
+                raise ValueError(f"rot must not be scaled: {d['rot']}")
+            rot = RotarySpec.from_dict(d["rot"], cls.scaling or YarnScaling)
         spec = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), int(d["mask"]["size"]), float(d["scale"]),
-                   None if d.get("softcap") is None else float(d["softcap"]), bool(d.get("v_mix", False)), RotarySpec.from_dict(d["rot"]) if cls.rotated else None)
+                   None if d.get("softcap") is None else float(d["softcap"]), bool(d.get("v_mix", False)), rot, int(d["mask"].get("keep_first", 0)))
         if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.size) <= 0 or spec.heads % spec.kv_heads:
             raise ValueError(f"attention sizes must be positive, kv_heads a divisor of heads: {d}")
         if spec.softcap is not None and not spec.softcap > 0:
             raise ValueError(f"softcap must be positive: {d}")
-        if spec.rot is not None and (spec.rot.dims > spec.dim or spec.rot.scaling is not None):
-            raise ValueError(f"rot must turn at most {spec.dim} dimensions, without scaling: {d['rot']}")
+        if spec.rot is not None and spec.rot.dims > spec.dim:
+            raise ValueError(f"rot must turn at most {spec.dim} dimensions: {d['rot']}")
+        if spec.keep < 0:
+            raise ValueError(f"mask.keep_first must not be negative: {d}")
         return spec
 
     def to_dict(self) -> dict:
-        out = {k: getattr(self, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale", "v_mix")}
+        out = {k: getattr(self, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale") + (("v_mix",) if self.capped else ())}
         if self.softcap is not None:
             out["softcap"] = self.softcap
-        out["mask"] = {"size": self.size}
+        out["mask"] = {"size": self.size, **({"keep_first": self.keep} if self.keeps else {})}
         if self.rot is not None:
             out["rot"] = self.rot.to_dict()
         return out
@@ -277,8 +293,21 @@ class GroupedAttentionSpec:
     def v_width(self) -> int:
         return self.kv_heads * self.vdim
 
+    @property
+    def slots(self) -> int:
+        """Positions that a sequence holds: the kept ones and a window or chunk."""
+        return self.keep + self.size
+
+    @property
+    def score_bound(self) -> Optional[float]:
+        """Largest magnitude of a score, where the design bounds it."""
+        if self.softcap is not None:
+            return self.softcap
+        return abs(self.scale) * self.dim if self.head_norm else None
+
     def param_count(self, E: int) -> int:
         n = self.heads * (self.dim + self.vdim) * E + self.kv_heads * (self.dim + self.vdim) * E + int(self.v_mix)
+        n += ((self.heads + self.kv_heads) * self.dim + self.v_width) * self.biased
         return n + (self.heads + self.kv_heads) * self.dim * self.qk_norm + self.heads * self.sink
 
 
@@ -288,6 +317,40 @@ class ChunkAttentionSpec(GroupedAttentionSpec):
 
 class WindowAttentionSpec(GroupedAttentionSpec):
     rotated = True
+
+
+class KeptWindowAttentionSpec(GroupedAttentionSpec):
+    keeps = biased = head_norm = rotated = True
+    capped = False
+    scaling = WavelengthScaling
+
+
+@dataclass(frozen=True)
+class DeltaMemorySpec:
+    """Matrix memory with the gated delta rule (Gated DeltaNet, Yang et al.): ``heads`` memories of ``dim`` keys and ``vdim`` values, whose
+    queries and keys come from ``kv_heads`` heads; q, k and v pass a causal convolution over ``conv`` tokens."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "DeltaMemorySpec":
+        names = ("heads", "kv_heads", "dim", "vdim", "conv")
+        _take(d, names, "mixer")
+        spec = cls(*(int(d[k]) for k in names))
+        if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv) <= 0 or spec.heads % spec.kv_heads:
+            raise ValueError(f"memory sizes must be positive, kv_heads a divisor of heads: {d}")
+        return spec
+
+    def to_dict(self) -> dict:
+        return asdict(self)
+
+    def param_count(self, E: int) -> int:
+        qk, v = 2 * self.kv_heads * self.dim, self.heads * self.vdim
+        return (qk + v) * (E + self.conv) + (2 * v + 2 * self.heads) * E + 2 * self.heads + self.vdim
 
 
 @dataclass(frozen=True)
@@ -402,67 +465,136 @@ class DenseMLPSpec:
 @dataclass(frozen=True)
 class MixtureSpec:
     """``experts`` feed-forwards of ``ff`` hidden units and ``identity`` experts that return their input, of which each token uses
-    ``top``; ``shared``: hidden units of an expert that runs for every token behind a gate (None: there is none)."""
+    ``top``; ``shared``: hidden units of an expert that runs for every token behind a gate (None: there is none).  With ``group_count`` the
+    experts form groups of neighbours, and only those of the ``group_keep`` groups whose two best scores add up to most can be chosen.
+    Subclasses fix the experts' form and how scores become weights."""
+
+    act: ClassVar = "relu2"          # "relu2": two matrices; "silu": gated, three
+    scores: ClassVar = "softmax"     # of the router's outputs, or "sigmoid"
+    corrected: ClassVar = True       # a correction is added to the scores for the choice
+    normalized: ClassVar = True      # the chosen scores are divided by their sum
+    grouped: ClassVar = False
 
     ff: int
     experts: int
     identity: int
     top: int
     shared: Optional[int] = None
+    group_count: int = 1
+    group_keep: int = 1
 
     @property
     def outputs(self) -> int:
         """Router outputs."""
         return self.experts + self.identity
 
+    @property
+    def gated(self) -> bool:
+        return self.act == "silu"
+
     @classmethod
     def from_dict(cls, d: dict) -> "MixtureSpec":
-        _take(d, ("kind", "expert", "router", "shared"), "mlp")
+        _take(d, ("kind", "expert", "router") + (() if cls.grouped else ("shared",)), "mlp")
         _take(d["expert"], ("ff",), "mlp.expert")
-        _take(d["router"], ("experts", "identity", "top"), "mlp.router")
-        shared = d.get("shared")
+        r = d["router"]
+        _take(r, ("experts", "top") + (("groups",) if cls.grouped else ("identity",)), "mlp.router")
+        shared, groups = d.get("shared"), r.get("groups") or {"count": 1, "keep": 1}
+        _take(groups, ("count", "keep"), "mlp.router.groups")
         if shared is not None:
             _take(shared, ("ff",), "mlp.shared")
-        r = d["router"]
-        spec = cls(int(d["expert"]["ff"]), int(r["experts"]), int(r.get("identity", 0)), int(r["top"]), None if shared is None else int(shared["ff"]))
+        spec = cls(int(d["expert"]["ff"]), int(r["experts"]), int(r.get("identity", 0)), int(r["top"]), None if shared is None else int(shared["ff"]),
+                   int(groups["count"]), int(groups["keep"]))
         if min(spec.ff, spec.experts, spec.top, 1 if spec.shared is None else spec.shared) <= 0 or spec.identity < 0 or spec.top > spec.outputs:
             raise ValueError(f"a mixture needs positive sizes and at most as many chosen experts as there are: {d}")
+        n, k = spec.group_count, spec.group_keep
+        if n < 1 or spec.outputs % n or not 1 <= k <= n or spec.top > spec.outputs // n * k:
+            raise ValueError(f"groups must be equal and hold the chosen experts: {d}")
         return spec
 
     def to_dict(self) -> dict:
-        out = {"kind": "moe", "expert": {"ff": self.ff}, "router": {"experts": self.experts, "identity": self.identity, "top": self.top}}
+        r = {"experts": self.experts, "top": self.top}
+        r.update({"groups": {"count": self.group_count, "keep": self.group_keep}} if self.grouped else {"identity": self.identity})
+        out = {"kind": "moe", "expert": {"ff": self.ff}, "router": r}
         if self.shared is not None:
             out["shared"] = {"ff": self.shared}
         return out
 
+    def _count(self, E: int, experts: int) -> int:
+        return (3 if self.gated else 2) * experts * self.ff * E + self.outputs * (E + self.corrected) + \
+            (0 if self.shared is None else (2 * self.shared + 1) * E)
+
     def param_count(self, E: int) -> int:
-        return 2 * self.experts * self.ff * E + self.outputs * (E + 1) + (0 if self.shared is None else (2 * self.shared + 1) * E)
+        return self._count(E, self.experts)
 
     def active_params(self, E: int) -> int:
         """Parameters that a token meets when all its experts have tensors."""
-        return 2 * self.top * self.ff * E + self.outputs * (E + 1) + (0 if self.shared is None else (2 * self.shared + 1) * E)
+        return self._count(E, self.top)
 
 
-MIXERS = {"latent_attention": LatentAttentionSpec, "parallel": ParallelSpec, "mlstm": GatedMemorySpec, "attention": ChunkAttentionSpec,
-          "attention_2": WindowAttentionSpec}
-MLPS = {"dense": DenseMLPSpec, "moe": MixtureSpec}
+class GroupedMixtureSpec(MixtureSpec):
+    act = "silu"
+    scores = "sigmoid"
+    corrected = normalized = False
+    grouped = True
+
+
+@dataclass(frozen=True)
+class Design:
+    """What an architecture fixes beside its configuration."""
+
+    mixers: dict                     # mixer types a layer may have -> their specs
+    norms: str                       # "post_rms": x += mult * rms(f(x)); "sandwich": x += ln(f(ln(x))); "sandwich_rms": the
+                                     # same with RMS norms whose weights are stored around zero; "post_group_rms": x += rms(f(x)) with
+                                     # norms over groups of columns, then a weighted sum of all earlier results
+    mlps: dict                       # feed-forward kinds a layer may have -> (form, spec); forms: "relu2": biased, two matrices; "geglu" /
+                                     # "swiglu": gated by tanh-GELU / silu, no biases; "moe": mixture of experts
+    keys: tuple                      # keys of config.json beside the common ones
+
+    @property
+    def sandwich(self) -> bool:
+        return self.norms.startswith("sandwich")
+
+    @property
+    def latent(self) -> bool:
+        """Whether layers share rings of latents."""
+        return LatentAttentionSpec in self.mixers.values()
+
+    @property
+    def depth_average(self) -> bool:
+        return self.norms == "post_group_rms"
+
+
+DESIGNS = {
+    "Gasovik": Design({"latent_attention": LatentAttentionSpec}, "post_rms", {"dense": ("relu2", DenseMLPSpec)}, ("residual_mult",)),
+    "Fatudra": Design({"parallel": ParallelSpec, "mlstm": GatedMemorySpec}, "sandwich", {"dense": ("geglu", DenseMLPSpec)}, ("embedding", "loop")),
+    "Dusilorn": Design({"attention": ChunkAttentionSpec, "attention_2": WindowAttentionSpec}, "sandwich_rms",
+                       {"dense": ("swiglu", DenseMLPSpec), "moe": ("moe", MixtureSpec)}, ("embedding", "logit_scale")),
+    "Bolovik": Design({"delta": DeltaMemorySpec, "attention": KeptWindowAttentionSpec}, "post_group_rms",
+                      {"dense": ("geglu", DenseMLPSpec), "moe": ("moe", GroupedMixtureSpec)}, ()),
+}
+ARCHITECTURES = tuple(DESIGNS)
+
+
+def is_layered(config: dict) -> bool:
+    """Whether a parsed ``config.json`` describes a model of this family."""
+    return config.get("architecture") in ARCHITECTURES
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     type: str
-    mixer: object                    # one of the specs of MIXERS
-    mlp: Optional[object] = None     # one of the specs of MLPS
+    mixer: object                    # one of the specs of the design's ``mixers``
+    mlp: Optional[object] = None     # one of the specs of its ``mlps``
 
     @classmethod
-    def from_dict(cls, d: dict) -> "LayerSpec":
+    def from_dict(cls, d: dict, design: Design) -> "LayerSpec":
         _take(d, ("type", "mixer", "mlp"), "layer")
-        if d["type"] not in MIXERS:
+        if d["type"] not in design.mixers:
             raise ValueError(f"unknown mixer type {d['type']!r}")
         mlp = d.get("mlp")
-        if mlp is not None and mlp.get("kind") not in MLPS:
+        if mlp is not None and mlp.get("kind") not in design.mlps:
             raise ValueError(f"unknown feed-forward kind {mlp.get('kind')!r}")
-        return cls(d["type"], MIXERS[d["type"]].from_dict(d["mixer"]), None if mlp is None else MLPS[mlp["kind"]].from_dict(mlp))
+        return cls(d["type"], design.mixers[d["type"]].from_dict(d["mixer"]), None if mlp is None else design.mlps[mlp["kind"]][1].from_dict(mlp))
 
     @property
     def mlp_kind(self) -> str:
@@ -494,6 +626,7 @@ class LayeredConfig:
     embed_scale: float = 1.0
     loop: Optional[LoopSpec] = None
     logit_scale: float = 1.0
+    norm_groups: int = 1
 
     def __post_init__(self):
         if self.architecture not in ARCHITECTURES:
@@ -501,7 +634,7 @@ class LayeredConfig:
         if not self.layers:
             raise ValueError("a model needs at least one layer")
         for i, layer in enumerate(self.layers):
-            if layer.type not in self.design.mixers:
+            if not isinstance(layer.mixer, self.design.mixers.get(layer.type, ())):
                 raise ValueError(f"layer {i}: {self.architecture} has no mixer {layer.type!r}")
             if layer.mlp is not None and layer.mlp_kind not in self.design.mlps:
                 raise ValueError(f"layer {i}: {self.architecture} has no feed-forward {layer.mlp_kind!r}")
@@ -515,6 +648,8 @@ class LayeredConfig:
                 raise ValueError(f"layer {i}: latent size and rotation must equal those of layer {j}")
         if len({layer.mixer.v_width for layer in self.layers if getattr(layer.mixer, "v_mix", False)}) > 1:
             raise ValueError("layers that mix their values need equally many value rows")
+        if self.norm_groups < 1 or self.width % self.norm_groups:
+            raise ValueError(f"norm.groups must divide the width, {self.norm_groups} does not divide {self.width}")
         lp = self.loop
         if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layers) and lp.times >= 1):
             raise ValueError(f"loop {lp} does not lie inside {len(self.layers)} layers")
@@ -526,6 +661,10 @@ class LayeredConfig:
     @property
     def design(self) -> Design:
         return DESIGNS[self.architecture]
+
+    @property
+    def latent(self) -> bool:
+        return self.design.latent
 
     def runs(self) -> list:
         """The executions of layers, in order."""
@@ -571,9 +710,12 @@ class LayeredConfig:
     def from_dict(cls, d: dict) -> "LayeredConfig":
         if not is_layered(d):
             raise ValueError(f"Invalid architecture {d.get('architecture')} provided.")
-        keys = DESIGNS[d["architecture"]].keys
+        design = DESIGNS[d["architecture"]]
+        keys, groups = design.keys, 1
         _take(d, ("architecture", "vocab", "width", "norm", "layers", "name") + keys, "config")
-        _take(d["norm"], ("eps",), "norm")
+        _take(d["norm"], ("eps",) + (("groups",) if design.depth_average else ()), "norm")
+        if design.depth_average:
+            groups = int(d["norm"].get("groups", 1))
         scale, loop = 1.0, None
         if "embedding" in keys:
             _take(d["embedding"], ("scale",), "embedding")
@@ -583,11 +725,13 @@ class LayeredConfig:
         mult = float(d["residual_mult"]) if "residual_mult" in keys else 1.0
         logit = float(d["logit_scale"]) if "logit_scale" in keys else 1.0
         return cls(d["architecture"], int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), mult,
-                   [LayerSpec.from_dict(x) for x in d["layers"]], d.get("name", ""), scale, loop, logit)
+                   [LayerSpec.from_dict(x, design) for x in d["layers"]], d.get("name", ""), scale, loop, logit, groups)
 
     def to_dict(self) -> dict:
         out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps}}
         keys = self.design.keys
+        if self.design.depth_average:
+            out["norm"]["groups"] = self.norm_groups
         if "residual_mult" in keys:
             out["residual_mult"] = self.residual_mult
         if "embedding" in keys:
@@ -637,6 +781,10 @@ class LayeredConfig:
                 n += layer.mixer.param_count(E) + 2 * norm + (0 if layer.mlp is None else layer.mlp.param_count(E) + 2 * norm)
             return n
         n = 2 * self.vocab * E + E
+        if self.design.depth_average:
+            for i, layer in enumerate(self.layers):
+                n += layer.mixer.param_count(E) + E + i + 2 + (0 if layer.mlp is None else layer.mlp.param_count(E) + E)
+            return n
         for i, layer in enumerate(self.layers):
             a = layer.mixer
             n += a.heads * ((a.dim + a.rot_dim) * E + 2 * a.vdim * E + (a.dim + a.vdim) * a.kv_rank) + E

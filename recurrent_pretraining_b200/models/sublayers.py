@@ -12,15 +12,17 @@ from typing import Callable, Optional
 import torch
 import torch.nn as nn
 
+from ..ops import delta as delta_ops
 from ..ops import grouped as grp_ops
 from ..ops import latent as ops
 from ..ops import memory as mem_ops
 from ..ops import moe as moe_ops
-from ..ops.grouped import GroupedLayout, QkvTransform
+from ..ops.delta import DeltaLayout, DeltaWeights
+from ..ops.grouped import GroupedLayout, QkvTransform, ring_slots
 from ..ops.latent import LatentLayout, pad8
 from ..ops.memory import BiasTable, MemoryLayout, ParallelLayout
-from .layered_config import (DenseMLPSpec, GatedMemorySpec, GroupedAttentionSpec, LatentAttentionSpec, LayeredConfig, LayerRun,
-                             MixtureSpec, ParallelSpec, RotarySpec)
+from .layered_config import (ChunkAttentionSpec, DeltaMemorySpec, DenseMLPSpec, GatedMemorySpec, GroupedAttentionSpec, KeptWindowAttentionSpec,
+                             LatentAttentionSpec, LayeredConfig, LayerRun, MixtureSpec, ParallelSpec, RotarySpec, WindowAttentionSpec)
 
 
 def weight(rows: int, cols: int, dtype, device) -> nn.Parameter:
@@ -51,7 +53,7 @@ class StreamLayout:
     kbase: torch.Tensor       # [T] stream index of the first key of its sequence (of its chunk)
     seqs: list                # (first token, tokens, first key, keys in front of the first token) per sequence (per chunk of one)
     total: int
-    history: list             # (row, first position, count, first key) of the sequences with history
+    history: list             # (row, first position, count, first key) of the stretches of history
 
 
 class PackedStep:
@@ -89,24 +91,28 @@ class PackedStep:
             self._seq_table = torch.tensor(self.sequences(), dtype=torch.int32).to(self.device)
         return self._seq_table
 
-    def layout(self, history: int) -> StreamLayout:
-        """Layout with up to ``history`` cached positions in front of every portion."""
+    def layout(self, history: int, keep: int = 0) -> StreamLayout:
+        """Layout with up to ``keep`` + ``history`` cached positions in front of every portion: the first ``keep`` of the sequence
+        and the newest ones.  A distance in the stream that does not reach into the kept positions is a distance in the sequence."""
         if all(s == 0 for _, s, _ in self.portions):
-            history = 0
-        if history not in self._layouts:
+            history = keep = 0
+        if (history, keep) not in self._layouts:
             seqs, sidx, kbase, hist = [], [], [], []
             t0 = k0 = 0
             for r, s, n in self.portions:
-                h = min(s, history)
+                h = min(s, history + keep)
+                first = min(h, keep)
                 seqs.append((t0, n, k0, h))
                 sidx.extend(range(k0 + h, k0 + h + n))
                 kbase.extend([k0] * n)
-                if h:
-                    hist.append((r, s - h, h, k0))
+                if first:
+                    hist.append((r, 0, first, k0))
+                if h > first:
+                    hist.append((r, s - (h - first), h - first, k0 + first))
                 t0, k0 = t0 + n, k0 + h + n
             idx = torch.tensor([sidx, kbase], dtype=torch.int32).to(self.device)
-            self._layouts[history] = StreamLayout(idx[0], idx[1], seqs, k0, hist)
-        return self._layouts[history]
+            self._layouts[history, keep] = StreamLayout(idx[0], idx[1], seqs, k0, hist)
+        return self._layouts[history, keep]
 
     def chunk_layout(self, size: int) -> StreamLayout:
         """Layout for attention inside chunks of ``size`` positions: the history of a portion is what its first chunk already
@@ -159,16 +165,14 @@ class DecodeContext:
     first_values: Optional[torch.Tensor] = None    # values that later layers mix into theirs
 
 
-def gather_history(layout: StreamLayout, cache: torch.Tensor, stream: torch.Tensor) -> None:
+def gather_history(layout: StreamLayout, cache: torch.Tensor, stream: torch.Tensor, keep: int = 0) -> None:
     """Copy the cached rows in front of every portion from the ring ``cache`` [rows, cap, ld] into the stream."""
     if not layout.history:
         return
     cap = cache.shape[1]
-    src, dst = [], []
-    for row, p0, n, k0 in layout.history:
-        src.extend(row * cap + (p % cap) for p in range(p0, p0 + n))
-        dst.extend(range(k0, k0 + n))
-    idx = torch.tensor([src, dst], dtype=torch.int32).to(cache.device)
+    src = [row * cap + ring_slots(torch.arange(p0, p0 + n), cap, keep) for row, p0, n, _ in layout.history]
+    dst = [torch.arange(k0, k0 + n) for _, _, n, k0 in layout.history]
+    idx = torch.stack([torch.cat(src), torch.cat(dst)]).to(torch.int32).to(cache.device)
     ops.gather_rows(cache.view(-1, cache.shape[2]), idx[0], stream, idx[1])
 
 
@@ -382,8 +386,58 @@ class GatedMemory(nn.Module):
         return out, clear, inp if acc else None
 
 
+class DeltaMemory(nn.Module):
+    """Matrix memories with the gated delta rule (``DeltaMemorySpec``).  Step sizes and decays have a product of their own with fp32 results
+    in prompts."""
+
+    out_bias, out_bias_mult = None, 1.0
+
+    def __init__(self, spec: DeltaMemorySpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
+        L = self.layout = DeltaLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim)
+        self.w_in, self.w_o = weight(L.width_in, width, dtype, device), weight(width, spec.heads * spec.vdim, dtype, device)
+        self.conv = nn.Parameter(torch.zeros(spec.conv, L.channels, dtype=torch.float32, device=device), requires_grad=False)
+        self.a_log, self.dt_bias, self.norm = vector(spec.heads, device), vector(spec.heads, device), vector(spec.vdim, device)
+
+    def checkpoint_tensors(self) -> dict:
+        a, L, E = self.spec, self.layout, self.width
+        qk, hv = a.kv_heads * a.dim, a.heads * a.vdim
+        out = {}
+        for name, at, n in (("q", L.off_q, qk), ("k", L.off_k, qk), ("v", L.off_v, hv)):
+            out[name], out[name + ".conv"] = self.w_in[at:at + n, :E], self.conv[:, at:at + n].T
+        for name, at, n in (("g", L.off_g, hv), ("b", L.off_ba, a.heads), ("a", L.off_ba + a.heads, a.heads)):
+            out[name] = self.w_in[at:at + n, :E]
+        out.update({"A_log": self.a_log, "dt_bias": self.dt_bias, "norm": self.norm, "o": self.w_o[:, :hv]})
+        return out
+
+    @property
+    def weights(self) -> DeltaWeights:
+        return DeltaWeights(self.conv, self.a_log, self.dt_bias, self.norm, self.eps)
+
+    def cache_shapes(self, max_len: int) -> dict:
+        a, L = self.spec, self.layout
+        return {"conv": ((a.conv, L.channels), self.dtype), "state": ((a.heads, a.dim, L.ldv), torch.float32)}
+
+    def stream(self, h, run: LayerRun, ctx: StepContext):
+        a, L, E, data = self.spec, self.layout, self.width, ctx.cache.data
+        inp = ops.linear(h, self.w_in[:L.off_ba, :E])
+        ba = mem_ops.gate_projections(h, self.w_in[L.off_ba:L.off_ba + 2 * a.heads, :E])
+        act = delta_ops.short_conv(L, inp, self.conv, data[run.index, "conv"], ctx.step)
+        o = delta_ops.delta_prompt(L, self.weights, act, inp, ba, data[run.index, "state"], ctx.step)
+        return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
+
+    def decode(self, h, run: LayerRun, ctx: DecodeContext):
+        a, L, data = self.spec, self.layout, ctx.cache.data
+        inp, acc = ctx.dense(h, self.w_in[:, :self.width], 0)
+        o = delta_ops.delta_decode(L, self.weights, inp, data[run.index, "conv"], data[run.index, "state"], ctx.pos, ctx.row, self.dtype)
+        out, clear = ctx.dense(o, self.w_o[:, :a.heads * a.vdim], 1)
+        return out, clear, inp if acc else None
+
+
 class GroupedAttention(nn.Module):
-    """Grouped-query attention over a ring of keys and values (``GroupedAttentionSpec``): inside chunks or under a window."""
+    """Grouped-query attention over a ring of keys and values (``GroupedAttentionSpec``): inside chunks or under a window, which may
+    keep a sequence's first tokens."""
 
     out_bias, out_bias_mult = None, 1.0
 
@@ -393,6 +447,7 @@ class GroupedAttention(nn.Module):
         self.spec, self.width, self.eps, self.dtype = spec, width, eps, dtype
         L = self.layout = GroupedLayout(a.heads, a.kv_heads, a.dim, a.vdim)
         self.w_in = weight(L.width_in, width, dtype, device)
+        self.b_in = vector(L.width_in, device) if a.biased else None
         self.w_o = weight(width, a.heads * a.vdim, dtype, device)
         self.q_norm, self.k_norm = (vector(n * a.dim, device) if a.qk_norm else None for n in (a.heads, a.kv_heads))
         self.sink = vector(a.heads, device) if a.sink else None
@@ -400,8 +455,11 @@ class GroupedAttention(nn.Module):
 
     def checkpoint_tensors(self) -> dict:
         a, L, E = self.spec, self.layout, self.width
-        out = {name: self.w_in[at:at + n, :E] for name, at, n in (("q", L.off_q, a.heads * a.dim), ("k", L.off_k, a.kv_heads * a.dim),
-                                                                  ("v", L.off_v, L.v_width))}
+        out = {}
+        for name, at, n in (("q", L.off_q, a.heads * a.dim), ("k", L.off_k, a.kv_heads * a.dim), ("v", L.off_v, L.v_width)):
+            out[name] = self.w_in[at:at + n, :E]
+            if a.biased:
+                out[name + ".b"] = self.b_in[at:at + n]
         out["o"] = self.w_o[:, :a.heads * a.vdim]
         out.update({k: v for k, v in (("q.norm", self.q_norm), ("k.norm", self.k_norm), ("sink", self.sink), ("vmix", self.vmix)) if v is not None})
         return out
@@ -409,24 +467,25 @@ class GroupedAttention(nn.Module):
     @property
     def unused_tensors(self) -> tuple:
         """Checkpoint tensors that may stand beside the others without a use."""
-        return () if self.spec.v_mix else ("vmix",)
+        return () if self.spec.v_mix or not self.spec.capped else ("vmix",)
 
     def cache_shapes(self, max_len: int) -> dict:
-        return {"kv": ((min(self.spec.size, max_len), self.layout.ld_kv), self.dtype)}
+        return {"kv": ((min(self.spec.slots, max_len), self.layout.ld_kv), self.dtype)}
 
-    def _transform(self, role: Optional[str], rope: dict, first) -> QkvTransform:
+    def _transform(self, role: Optional[str], rope: dict, first, raw: bool = False) -> QkvTransform:
+        """``raw``: of a decode step's accumulators."""
         rot = self.spec.rot
         mix = role == "mix"
         return QkvTransform(self.q_norm, self.k_norm, self.eps, 0 if rot is None else rot.dims, None if rot is None else rope[rot],
-                            self.vmix if mix else None, first if mix else None)
+                            self.vmix if mix else None, first if mix else None, self.spec.head_norm, self.b_in if raw else None, self.spec.keep)
 
     def stream(self, h, run: LayerRun, ctx: StepContext):
         a, L, step, role = self.spec, self.layout, ctx.step, ctx.config.mixes_values(run.layer)
         cache = ctx.cache.data[run.index, "kv"]
-        lay = step.chunk_layout(a.size) if a.chunked else step.layout(a.size - 1)
-        inp = ops.linear(h, self.w_in[:, :self.width])
+        lay = step.chunk_layout(a.size) if a.chunked else step.layout(a.size - 1, a.keep)
+        inp = ops.linear(h, self.w_in[:, :self.width], self.b_in)
         kv = torch.empty(lay.total, L.ld_kv, dtype=self.dtype, device=h.device)
-        gather_history(lay, cache, kv)             # before the ring slots of the oldest positions are written again
+        gather_history(lay, cache, kv, a.keep)     # before the ring slots of the oldest positions are written again
         grp_ops.qkv_prep_(L, inp, self._transform(role, ctx.rope, ctx.first_values), step, lay.sidx, cache, kv)
         if role == "first":
             ctx.first_values = inp[:, L.off_v:L.off_v + L.v_width]
@@ -434,12 +493,12 @@ class GroupedAttention(nn.Module):
         return ops.linear(o, self.w_o[:, :a.heads * a.vdim])
 
     def decode_splits(self, B: int, max_len: int, tensor_cores: bool) -> int:
-        return grp_ops.decode_splits(self.layout, B, min(self.spec.size, max_len), tensor_cores)
+        return grp_ops.decode_splits(self.layout, B, min(self.spec.slots, max_len), tensor_cores)
 
     def decode(self, h, run: LayerRun, ctx: DecodeContext):
         a, L, role = self.spec, self.layout, ctx.config.mixes_values(run.layer)
         inp, acc = ctx.dense(h, self.w_in[:, :self.width], 0)
-        tr = self._transform(role, ctx.cache.rope, ctx.first_values)
+        tr = self._transform(role, ctx.cache.rope, ctx.first_values, raw=True)
         first = torch.empty(h.shape[0], pad8(L.v_width), dtype=torch.float32, device=h.device)[:, :L.v_width] if role == "first" else None
         o = grp_ops.ring_attention(L, a, inp, tr, ctx.cache.data[run.index, "kv"], self.sink, first, ctx.pos, ctx.row, ctx.splits(self, h.shape[0]),
                                    self.dtype)
@@ -478,8 +537,8 @@ class SiluMLP(GatedMLP):
 
 
 class MixtureMLP(nn.Module):
-    """Mixture of squared-ReLU experts with identity experts and a gated shared expert (``MixtureSpec``).  The experts' matrices lie
-    one below the other; the shared expert's gate is one more row of the router."""
+    """Mixture of experts (``MixtureSpec``): squared-ReLU or gated ones, identity experts, a gated shared expert.  The experts' matrices lie
+    one below the other (gated: gate and up rows of an expert in turn); the shared expert's gate is one more row of the router."""
 
     wide = 0
     out_bias, out_bias_mult = None, 1.0
@@ -488,16 +547,23 @@ class MixtureMLP(nn.Module):
         super().__init__()
         s = spec
         self.spec, self.width, self.dtype = spec, width, dtype
-        self.w_router, self.correction = weight(s.outputs + (s.shared is not None), width, dtype, device), vector(s.outputs, device)
-        self.w_up, self.w_down = weight(s.experts * s.ff, width, dtype, device), weight(s.experts * width, s.ff, dtype, device)
+        self.w_router = weight(s.outputs + (s.shared is not None), width, dtype, device)
+        self.correction = vector(s.outputs, device) if s.corrected else None
+        self.w_up, self.w_down = weight(s.experts * s.ff * (2 if s.gated else 1), width, dtype, device), weight(s.experts * width, s.ff, dtype, device)
         if s.shared is not None:
             self.s_up, self.s_down = weight(s.shared, width, dtype, device), weight(width, s.shared, dtype, device)
 
     def checkpoint_tensors(self) -> dict:
         s, E = self.spec, self.width
-        out = {"router": self.w_router[:s.outputs, :E], "correction": self.correction}
+        out = {"router": self.w_router[:s.outputs, :E]}
+        if s.corrected:
+            out["correction"] = self.correction
+        names = ("gate", "up") if s.gated else ("up",)
         for e in range(s.experts):
-            out[f"e{e}.up"], out[f"e{e}.down"] = self.w_up[e * s.ff:(e + 1) * s.ff, :E], self.w_down[e * E:(e + 1) * E, :s.ff]
+            for k, name in enumerate(names):
+                at = (e * len(names) + k) * s.ff
+                out[f"e{e}.{name}"] = self.w_up[at:at + s.ff, :E]
+            out[f"e{e}.down"] = self.w_down[e * E:(e + 1) * E, :s.ff]
         if s.shared is not None:
             out.update({"shared.sg": self.w_router[s.outputs:, :E], "shared.up": self.s_up[:, :E], "shared.down": self.s_down[:, :s.shared]})
         return out
@@ -515,6 +581,6 @@ class MixtureMLP(nn.Module):
         return moe_ops.mixture_rows(self.weights, h), False
 
 
-MIXERS = {"latent_attention": LatentAttention, "parallel": ParallelMixer, "mlstm": GatedMemory, "attention": GroupedAttention,
-          "attention_2": GroupedAttention}
-MLPS = {"relu2": DenseMLP, "geglu": GatedMLP, "swiglu": SiluMLP, "relu2_moe": MixtureMLP}
+MIXERS = {LatentAttentionSpec: LatentAttention, ParallelSpec: ParallelMixer, GatedMemorySpec: GatedMemory, DeltaMemorySpec: DeltaMemory,
+          ChunkAttentionSpec: GroupedAttention, WindowAttentionSpec: GroupedAttention, KeptWindowAttentionSpec: GroupedAttention}
+MLPS = {"relu2": DenseMLP, "geglu": GatedMLP, "swiglu": SiluMLP, "moe": MixtureMLP}

@@ -41,7 +41,7 @@ class GroupedLayout:
 
 class _QkvRow(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("ld_in", "off_k", "off_v", "H", "G", "dim", "vdim", "rot", "ld_q", "ld_kv", "kv_v", "cap", "ld_first", "ld_fout")] + \
-               [("eps", C.c_float)] + [(n, C.c_void_p) for n in ("q_norm", "k_norm", "cosT", "sinT", "lam", "pos", "row", "sidx", "end")]
+               [("eps", C.c_float)] + [(n, C.c_void_p) for n in ("q_norm", "k_norm", "cosT", "sinT", "lam", "pos", "row", "sidx", "end")] + [("keep", C.c_int), ("bias", C.c_void_p)]
 
 
 _fns = None
@@ -56,6 +56,7 @@ def _k():
 
         vp, i = C.c_void_p, C.c_int
         _fns = SimpleNamespace(K=K, prep=K._sig("b200_qkv_prep", [vp] * 6 + [C.POINTER(_QkvRow)] + [i] * 4 + [vp]),
+                               heads=K._sig("b200_qkv_heads", [vp] * 4 + [C.POINTER(_QkvRow)] + [i] * 3 + [vp]),
                                merge=K._sig("b200_attention_merge", [vp] * 4 + [i] * 6 + [vp]))
     return _fns
 
@@ -63,7 +64,9 @@ def _k():
 @dataclass
 class QkvTransform:
     """What happens to a projection row before it is used: norms over all of q and of k (``q_norm``, ``k_norm`` or None), rotation
-    (``rope``: cos and sin tables of ``rot`` dimensions, or None), mixing of values (``lam`` and ``first``, or None)."""
+    (``rope``: cos and sin tables of ``rot`` dimensions, or None), mixing of values (``lam`` and ``first``, or None).  ``head_norm``: every head
+    of q and k, once rotated, and of v is normed without weights.  ``bias``: of the raw rows of a decode step (already added in prompts).
+    ``keep``: first positions that the ring keeps."""
 
     q_norm: Optional[torch.Tensor]
     k_norm: Optional[torch.Tensor]
@@ -72,6 +75,14 @@ class QkvTransform:
     rope: Optional[tuple] = None
     lam: Optional[torch.Tensor] = None
     first: Optional[torch.Tensor] = None
+    head_norm: bool = False
+    bias: Optional[torch.Tensor] = None
+    keep: int = 0
+
+
+def ring_slots(p: torch.Tensor, cap: int, keep: int) -> torch.Tensor:
+    """Ring slots of positions; the first ``keep`` have theirs for good."""
+    return torch.where(p < cap, p, keep + (p - keep) % max(1, cap - keep))
 
 
 def _row_struct(L: GroupedLayout, inp, tr: QkvTransform, ld_q: int, cap: int, first_out, pos, row, sidx=None, end=None) -> _QkvRow:
@@ -79,12 +90,14 @@ def _row_struct(L: GroupedLayout, inp, tr: QkvTransform, ld_q: int, cap: int, fi
     cos, sin = tr.rope if tr.rope is not None else (None, None)
     return _QkvRow(inp.stride(0), L.off_k, L.off_v, L.heads, L.kv_heads, L.dim, L.vdim, tr.rot, ld_q, L.ld_kv, L.kv_v, cap,
                    0 if tr.first is None else tr.first.stride(0), 0 if first_out is None else first_out.stride(0), tr.eps, p(tr.q_norm), p(tr.k_norm),
-                   p(cos), p(sin), p(tr.lam), p(pos), p(row), p(sidx), p(end))
+                   p(cos), p(sin), p(tr.lam), p(pos), p(row), p(sidx), p(end), tr.keep, 0)
 
 
 def _plain_rows(L: GroupedLayout, inp, tr: QkvTransform, pos):
     """q [T, H, dim], kv row [T, ld_kv] and unmixed values [T, v_width] of projection rows, fp32."""
     x, T = inp.float(), inp.shape[0]
+    if tr.bias is not None:
+        x = x + tr.bias
     q, k, v = x[:, :L.heads * L.dim], x[:, L.off_k:L.off_k + L.kv_heads * L.dim], x[:, L.off_v:L.off_v + L.v_width]
     if tr.q_norm is not None:
         q, k = ref.rms(q, tr.eps) * tr.q_norm, ref.rms(k, tr.eps) * tr.k_norm
@@ -92,6 +105,8 @@ def _plain_rows(L: GroupedLayout, inp, tr: QkvTransform, pos):
     if tr.rope is not None:
         cos, sin = (t[pos.long()][:, None] for t in tr.rope)
         q, k = (torch.cat([ref.rotate_halves(t[..., :tr.rot], cos, sin), t[..., tr.rot:]], dim=-1) for t in (q, k))
+    if tr.head_norm:
+        q, k, v = ref.rms(q, tr.eps), ref.rms(k, tr.eps), ref.rms(v.unflatten(1, (L.kv_heads, L.vdim)), tr.eps).flatten(1)
     mixed = v if tr.lam is None else (1 - tr.lam) * v + tr.lam * tr.first.float()
     kv = torch.zeros(T, L.ld_kv)
     kv[:, :L.kv_heads * L.dim] = k.flatten(1)
@@ -108,12 +123,16 @@ def qkv_prep_(L: GroupedLayout, inp: torch.Tensor, tr: QkvTransform, step, sidx,
         stream[sidx.long()] = kv.to(stream.dtype)
         if cache is not None:
             cap = cache.shape[1]
-            keep = step.pos >= step.end - cap
-            cache[step.row[keep].long(), step.pos[keep].long() % cap] = kv[keep].to(cache.dtype)
+            keep = (step.pos < tr.keep) | (step.pos >= step.end - (cap - tr.keep))
+            cache[step.row[keep].long(), ring_slots(step.pos[keep].long(), cap, tr.keep)] = kv[keep].to(cache.dtype)
         return
     k = _k()
     p = k.K._ptr
     s = _row_struct(L, inp, tr, inp.stride(0), 1 if cache is None else cache.shape[1], None, step.pos, step.row, sidx, step.end)
+    if tr.head_norm:
+        k.K._check(k.heads(inp.data_ptr(), inp.data_ptr(), p(cache), stream.data_ptr(), C.byref(s), inp.shape[0], _f32(inp), _f32(inp), k.K._stream()),
+                   "qkv_heads")
+        return
     k.K._check(k.prep(inp.data_ptr(), inp.data_ptr(), p(tr.first), 0, p(cache), stream.data_ptr(), C.byref(s), inp.shape[0], _f32(inp), _f32(inp),
                       _f32(inp), k.K._stream()), "qkv_prep")
 
@@ -130,11 +149,12 @@ def _kv_heads(L: GroupedLayout, kv: torch.Tensor):
 def stream_attention(L: GroupedLayout, a, inp: torch.Tensor, stream: torch.Tensor, layout, sink: Optional[torch.Tensor]) -> torch.Tensor:
     """Attention of a packed step's queries (in ``inp``) over its key stream [K, ld_kv] -> [T, heads * vdim].  ``a``: the layer's
     ``GroupedAttentionSpec``; the layout's ``kbase`` bounds the keys of a chunk."""
-    T, window = inp.shape[0], 2**30 if a.chunked else a.size
+    T, window = inp.shape[0], min(2**30, 2**30 if a.chunked else a.size)
     if not inp.is_cuda:
         k, v = _kv_heads(L, stream)
         j, s = torch.arange(stream.shape[0])[None], layout.sidx.long()[:, None]
-        vis = (j <= s) & (j > s - window) & (j >= layout.kbase.long()[:, None])
+        first = layout.kbase.long()[:, None]
+        vis = (j <= s) & (j >= first) & ((j > s - window) | (j < first + a.keep))
         q = inp[:, :L.heads * L.dim].unflatten(1, (L.heads, L.dim))
         return ref.capped_attention(q, k, v, vis, a.scale, a.softcap, sink).flatten(1).to(inp.dtype)
     W = L.heads * L.vdim
@@ -142,12 +162,12 @@ def stream_attention(L: GroupedLayout, a, inp: torch.Tensor, stream: torch.Tenso
     if inp.dtype == BF16:
         from . import grouped_kernels as GK
 
-        if GK.prompt_supported(L, a):
+        if GK.prompt_supported(L, a) and not a.keep:
             GK.stream_attention(L, a, inp, stream, layout, window, sink, out)
             return out
     k = base._k()
     s = _attn_struct(L, a, inp.stride(0), window=window, sidx=layout.sidx.data_ptr(), kbase=layout.kbase.data_ptr(), out_ld=out.stride(0),
-                     sink=k.K._ptr(sink))
+                     sink=k.K._ptr(sink), keep=a.keep)
     k.K._check(k.attn(inp.data_ptr(), stream.data_ptr(), 0, stream[:, L.kv_v:].data_ptr(), 0, out.data_ptr(), C.byref(s), T, _f32(inp),
                       k.K._stream()), "window_attention")
     return out
@@ -176,10 +196,12 @@ def ring_attention(L: GroupedLayout, a, inp: torch.Tensor, tr: QkvTransform, cac
         if first_out is not None:
             first_out.copy_(v)
         p, r = pos.long(), row.long()
-        cache[r, p % cap] = kv.to(cache.dtype)
-        back = torch.arange(min(a.size, cap))[None]                  # key = position p - back
-        see = back <= (p % a.size if a.chunked else p)[:, None]
-        k, v = _kv_heads(L, cache[r[:, None], (p[:, None] - back) % cap])
+        cache[r, ring_slots(p, cap, a.keep)] = kv.to(cache.dtype)
+        n = min(a.size, cap)
+        back = torch.arange(n + a.keep)[None]                        # key = position p - back, then the kept positions in front of the window
+        key = torch.where(back < n, p[:, None] - back, back - n)
+        see = torch.where(back < n, back <= (p % a.size if a.chunked else p)[:, None], key <= (p - n)[:, None])
+        k, v = _kv_heads(L, cache[r[:, None], ring_slots(key.clamp(min=0), cap, a.keep)])
         return ref.capped_attention(q.to(dtype), k, v, see, a.scale, a.softcap, sink).flatten(1).to(dtype)
     out = torch.empty(B, pad8(W), dtype=dtype, device=inp.device)[:, :W]
     attend, merge = ring_attention_pieces(L, a, inp, tr, cache, sink, first_out, pos, row, splits, out)
@@ -199,7 +221,7 @@ def ring_attention_pieces(L: GroupedLayout, a, inp, tr: QkvTransform, cache, sin
     if dtype == BF16:
         from . import grouped_kernels as GK
 
-        fused = GK.decode_supported(L)
+        fused = GK.decode_supported(L) and not tr.head_norm
 
     def attend():
         if fused:
@@ -207,11 +229,15 @@ def ring_attention_pieces(L: GroupedLayout, a, inp, tr: QkvTransform, cache, sin
             return
         q = torch.empty(B, pad8(L.heads * L.dim), dtype=dtype, device=inp.device)
         s = _row_struct(L, inp, tr, q.stride(0), cap, first_out, pos, row)
-        k.K._check(k.prep(inp.data_ptr(), q.data_ptr(), p(tr.first), p(first_out), cache.data_ptr(), 0, C.byref(s), B, _f32(inp), int(dtype == F32), 1,
-                          k.K._stream()), "qkv_prep")
+        if tr.head_norm:
+            s.bias = p(tr.bias)
+            k.K._check(k.heads(inp.data_ptr(), q.data_ptr(), cache.data_ptr(), 0, C.byref(s), B, _f32(inp), int(dtype == F32), k.K._stream()), "qkv_heads")
+        else:
+            k.K._check(k.prep(inp.data_ptr(), q.data_ptr(), p(tr.first), p(first_out), cache.data_ptr(), 0, C.byref(s), B, _f32(inp), int(dtype == F32), 1,
+                              k.K._stream()), "qkv_prep")
         w = base._k()
         s = _attn_struct(L, a, q.stride(0), window=min(a.size, cap), splits=splits, pos=pos.data_ptr(), row=row.data_ptr(), cap=cap,
-                         part_o=part_o.data_ptr(), part_ml=part_ml.data_ptr(), chunk=a.size if a.chunked else 0)
+                         part_o=part_o.data_ptr(), part_ml=part_ml.data_ptr(), chunk=a.size if a.chunked else 0, keep=a.keep)
         k.K._check(w.attn(q.data_ptr(), cache.data_ptr(), 0, cache[:, :, L.kv_v:].data_ptr(), 0, 0, C.byref(s), B, int(dtype == F32), k.K._stream()),
                    "window_attention")
 

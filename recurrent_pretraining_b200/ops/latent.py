@@ -69,7 +69,8 @@ class _WindowAttn(C.Structure):
                [(n, C.c_void_p) for n in ("sidx", "kbase", "pos", "row")] + [("cap", C.c_int)] + \
                [(n, C.c_int) for n in ("gate_ld", "out_ld")] + [(n, C.c_void_p) for n in ("part_o", "part_ml")] + \
                [("group", C.c_int), ("bias", C.c_void_p), ("bias_len", C.c_int), ("temp_every", C.c_int), ("temp_coef", C.c_float),
-                ("head_gate", C.c_int), ("gate_mult", C.c_float), ("softcap", C.c_float), ("chunk", C.c_int), ("sink", C.c_void_p)]
+                ("head_gate", C.c_int), ("gate_mult", C.c_float), ("softcap", C.c_float), ("chunk", C.c_int), ("sink", C.c_void_p),
+                ("keep", C.c_int)]
 
 
 _fns = None
@@ -160,15 +161,17 @@ def bias_act(a: torch.Tensor, bias: Optional[torch.Tensor], act: Optional[str], 
 # ------------------------------------------------------------------------------------------
 # residual stream
 # ------------------------------------------------------------------------------------------
-def embed(tok: torch.Tensor, table: torch.Tensor, scale: float = 1.0, copy: bool = True):
-    """(fp32 residual [T, E] = scale * table row, operand copy [T, E] or None) of token ids [T]."""
+def embed(tok: torch.Tensor, table: torch.Tensor, scale: float = 1.0, copy: bool = True, out: Optional[torch.Tensor] = None):
+    """(fp32 residual [T, E] = scale * table row, operand copy [T, E] or None) of token ids [T]; ``out``: contiguous storage for the first."""
     T, E = tok.numel(), table.shape[1]
     if not tok.is_cuda:
         x = table[tok].float() * scale
+        if out is not None:
+            x = out.copy_(x)
         return x, x.to(table.dtype) if copy else None
     k = _k()
     assert tok.dtype == torch.int64 and tok.is_contiguous()
-    x = torch.empty(T, E, dtype=F32, device=tok.device)
+    x = torch.empty(T, E, dtype=F32, device=tok.device) if out is None else out
     xb = torch.empty(T, pad8(E), dtype=table.dtype, device=tok.device)[:, :E] if copy else None
     k.K._check(k.embed(tok.data_ptr(), table.data_ptr(), x.data_ptr(), k.K._ptr(xb), T, E, table.stride(0), xb.stride(0) if copy else 0,
                        scale, table.shape[0], _f32(table), k.K.err_word(tok.device).data_ptr(), k.K._stream()), "embed_resid")

@@ -14,19 +14,19 @@ import torch
 from . import latent as base
 from . import reference as ref
 from .latent import BF16, F32, _f32, pad8
-from .memory import RowSum
+from .memory import RowSum, glu
 
 ROWS = 64            # widest batch of the decode form
 
 
 @dataclass
 class MoeWeights:
-    """``router`` [outputs (+ 1 with a shared expert: its gate), E], ``correction`` [outputs], ``up`` [experts * ff, E], ``down``
-    [experts * E, ff], ``up_s`` [shared, E], ``down_s`` [E, shared] or None."""
+    """``router`` [outputs (+ 1 with a shared expert: its gate), E], ``correction`` [outputs] or None, ``up`` [experts * ff, E] (gated experts:
+    [experts * 2 ff, E], gate and up rows of an expert in turn), ``down`` [experts * E, ff], ``up_s`` [shared, E], ``down_s`` [E, shared] or None."""
 
     spec: object
     router: torch.Tensor
-    correction: torch.Tensor
+    correction: Optional[torch.Tensor]
     up: torch.Tensor
     down: torch.Tensor
     up_s: Optional[torch.Tensor]
@@ -34,7 +34,7 @@ class MoeWeights:
 
 
 class _Route(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("experts", "outputs", "top", "ld_z", "gate")] + [(n, C.c_void_p) for n in ("correction", "idx", "weight")]
+    _fields_ = [(n, C.c_int) for n in ("experts", "outputs", "top", "ld_z", "gate", "sigmoid", "normalize", "groups", "keep")] + [(n, C.c_void_p) for n in ("correction", "idx", "weight")]
 
 
 class _RouteRows(C.Structure):
@@ -42,7 +42,7 @@ class _RouteRows(C.Structure):
 
 
 class _ExpertRows(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("N", "K", "ld_w", "Ns", "Ks", "ld_ws", "ld_x", "ld_y", "ld_xs", "ld_ys", "B", "relu2")] + \
+    _fields_ = [(n, C.c_int) for n in ("N", "K", "ld_w", "Ns", "Ks", "ld_ws", "ld_x", "ld_y", "ld_xs", "ld_ys", "B", "act")] + \
                [(n, C.c_void_p) for n in ("w", "ws", "x", "xs")] + [("gather", C.c_int)] + \
                [(n, C.c_void_p) for n in ("y", "ys", "active", "first", "row", "n_active")]
 
@@ -95,7 +95,8 @@ def router_logits(h: torch.Tensor, router: torch.Tensor) -> torch.Tensor:
 
 def _route_struct(w: MoeWeights, z, idx, weight) -> _Route:
     s = w.spec
-    return _Route(s.experts, s.outputs, s.top, z.stride(0), int(w.up_s is not None), w.correction.data_ptr(), idx.data_ptr(), weight.data_ptr())
+    return _Route(s.experts, s.outputs, s.top, z.stride(0), int(w.up_s is not None), int(s.scores == "sigmoid"), int(s.normalized), s.group_count,
+                  s.group_keep, _k().K._ptr(w.correction), idx.data_ptr(), weight.data_ptr())
 
 
 @dataclass
@@ -144,20 +145,26 @@ def dispatch(w: MoeWeights, h: torch.Tensor, p: Slots) -> torch.Tensor:
     return xs
 
 
-def grouped_linear(x: torch.Tensor, w: torch.Tensor, N: int, p: Slots, relu2: bool = False) -> torch.Tensor:
-    """Slots x [size, K] times their experts' rows of w [experts * N, K] -> [size, N]."""
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, N: int, p: Slots, act: Optional[str] = None) -> torch.Tensor:
+    """Slots x [size, K] times their experts' rows of w [experts * N, K] -> act(..) [size, N]; ``act`` "relu2", or "silu": w holds [gate; up]
+    rows [experts * 2 N, K] and the result is silu(gate) * up."""
     k = _k()
     M, Kd = x.shape
     out = torch.empty(M, pad8(N), dtype=x.dtype, device=x.device)[:, :N]
     if x.dtype == F32:
-        k.K._check(base._k().sgemm(x.data_ptr(), w.data_ptr(), 0, out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0), out.stride(0), int(relu2), 0, 0,
+        if act == "silu":
+            return glu(grouped_linear(x, w, 2 * N, p), N, "silu", F32)
+        k.K._check(base._k().sgemm(x.data_ptr(), w.data_ptr(), 0, out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0), out.stride(0), int(act == "relu2"), 0, 0,
                                    p.tile_expert.data_ptr(), p.n_tiles.data_ptr(), k.K._stream()), "sgemm_nt")
         return out
-    bn = 256 if p.rows == 256 or N > 128 else 128
-    k.K._check(k.gemm(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0), out.stride(0), w.shape[0] // N,
-                      p.tile_expert.data_ptr(), p.n_tiles.data_ptr(), p.rows, bn, int(relu2), k.K._stream(), k.K.err_word(x.device).data_ptr()),
+    bn = 256 if p.rows == 256 or (N > 128 and act != "silu") else 128
+    k.K._check(k.gemm(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, Kd, x.stride(0), w.stride(0), out.stride(0),
+                      w.shape[0] // (2 * N if act == "silu" else N), p.tile_expert.data_ptr(), p.n_tiles.data_ptr(), p.rows, bn, _GROUPED_ACT[act], k.K._stream(), k.K.err_word(x.device).data_ptr()),
                "b200_gemm_grouped")
     return out
+
+
+_GROUPED_ACT = {None: 0, "relu2": 1, "silu": 4}
 
 
 def tile_rows(spec, T: int, dtype: torch.dtype) -> int:
@@ -182,14 +189,20 @@ def combine(s: RowSum) -> torch.Tensor:
 def _plain(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
     s, E = w.spec, h.shape[1]
     z = router_logits(h, w.router)
-    idx, weight = ref.route(z[:, :s.outputs], w.correction, s.top)
+    idx, weight = ref.route_grouped(z, s.top, s.group_count, s.group_keep) if s.grouped else ref.route(z[:, :s.outputs], w.correction, s.top)
+
+    def hidden(x, e):
+        if s.gated:
+            return glu(base.linear(x, w.up[2 * e * s.ff:2 * (e + 1) * s.ff]), s.ff, "silu", x.dtype)
+        return ref.linear_act(x, w.up[e * s.ff:(e + 1) * s.ff], None, "relu2")
+
     out = torch.zeros(h.shape)
     for e in range(s.outputs):
         t, k = (idx == e).nonzero(as_tuple=True)
         if not len(t):
             continue
         y = h[t].float() if e >= s.experts else \
-            ref.linear_act(ref.linear_act(h[t], w.up[e * s.ff:(e + 1) * s.ff], None, "relu2"), w.down[e * E:(e + 1) * E]).float()
+            ref.linear_act(hidden(h[t], e), w.down[e * E:(e + 1) * E]).float()
         out.index_add_(0, t, weight[t, k][:, None] * y)
     if w.up_s is not None:
         ys = ref.linear_act(ref.linear_act(h, w.up_s, None, "relu2"), w.down_s).float()
@@ -203,7 +216,7 @@ def mixture(w: MoeWeights, h: torch.Tensor) -> torch.Tensor:
         return _plain(w, h)
     s, E = w.spec, h.shape[1]
     p = plan(w, router_logits(h, w.router), tile_rows(s, h.shape[0], h.dtype))
-    a = grouped_linear(dispatch(w, h, p), w.up, s.ff, p, relu2=True)
+    a = grouped_linear(dispatch(w, h, p), w.up, s.ff, p, s.act)
     y = grouped_linear(a, w.down, E, p)
     ys = None if w.up_s is None else base.linear(base.linear(h, w.up_s, None, "relu2"), w.down_s)
     return combine(RowSum(y, p.slot, p.weight, h, ys))
@@ -250,7 +263,7 @@ def mixture_rows_pieces(w: MoeWeights, h: torch.Tensor):
         k.K._check(k.route_rows(z.data_ptr(), C.byref(r), C.byref(o), B, k.K._stream()), "moe_route_rows")
 
     def up():
-        e = _ExpertRows(s.ff, E, w.up.stride(0), fs, E, ld(w.up_s), h.stride(0), a.stride(0), h.stride(0), ld(a_s), B, 1, w.up.data_ptr(), p(w.up_s),
+        e = _ExpertRows(s.ff, E, w.up.stride(0), fs, E, ld(w.up_s), h.stride(0), a.stride(0), h.stride(0), ld(a_s), B, 2 if s.gated else 1, w.up.data_ptr(), p(w.up_s),
                         h.data_ptr(), h.data_ptr(), 1, a.data_ptr(), p(a_s), *lists)
         k.K._check(k.rows(C.byref(e), most, 0, 0, k.K._stream()), "moe_rows")
 

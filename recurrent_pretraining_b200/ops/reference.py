@@ -291,3 +291,37 @@ def route(z: torch.Tensor, correction: torch.Tensor, top: int):
     idx = torch.sort(s + correction, dim=-1, descending=True, stable=True).indices[:, :top]
     w = s.gather(1, idx)
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20)
+
+
+# ------------------------------------------------------------------------------------------
+# layered decoder models: norms over groups of columns, gated delta rule, choice of experts within groups
+# ------------------------------------------------------------------------------------------
+def group_rms(x: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    return rms(x.unflatten(-1, (groups, -1)), eps).flatten(-2)
+
+
+def unit(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x / torch.sqrt(x.square().sum(-1, keepdim=True) + eps)
+
+
+def delta_scan(q, k, v, beta, log_g, state) -> torch.Tensor:
+    """S = g S, u = beta (v - S^T k), S = S + k u^T, o = S^T q per token and head; q, k [T, H, D], v [T, H, E], beta, log_g [T, H],
+    ``state`` [H, D, E] is updated."""
+    out = []
+    for t in range(q.shape[0]):
+        s = torch.exp(log_g[t])[:, None, None] * state
+        u = beta[t][:, None] * (v[t] - torch.einsum("hde,hd->he", s, k[t]))
+        state.copy_(s + k[t, :, :, None] * u[:, None, :])
+        out.append(torch.einsum("hde,hd->he", state, q[t]))
+    return torch.stack(out)
+
+
+def route_grouped(z: torch.Tensor, top: int, groups: int, keep: int):
+    """Router logits [T, outputs] -> chosen outputs [T, top] of the best groups, best first, and their sigmoid scores."""
+    s = torch.sigmoid(z.float())
+    g = s.unflatten(1, (groups, -1))
+    strength = g.topk(min(2, g.shape[2]), dim=-1).values.sum(-1)
+    best = torch.sort(strength, dim=-1, descending=True, stable=True).indices[:, :keep]
+    allowed = torch.zeros_like(strength, dtype=torch.bool).scatter_(1, best, True)[:, :, None].expand_as(g).flatten(1)
+    idx = torch.sort(s.masked_fill(~allowed, float("-inf")), dim=-1, descending=True, stable=True).indices[:, :top]
+    return idx, s.gather(1, idx)

@@ -349,8 +349,8 @@ def routed_ops_prefill(model, seqs: list, t: Timer) -> list:
     t.op("moe: route + plan", lambda: X.plan(w, z, rows), 4.0 * T * (s.outputs + 4 * s.top), 0)
     xs = X.dispatch(w, h, p)
     t.op("moe: dispatch", lambda: X.dispatch(w, h, p), 2.0 * E * (T + n), 0)
-    g = X.grouped_linear(xs, w.up, s.ff, p, True)
-    gemm(f"moe: up (grouped, {rows}-row tiles)", lambda: X.grouped_linear(xs, w.up, s.ff, p, True), n, s.ff, E, s.experts)
+    g = X.grouped_linear(xs, w.up, s.ff, p, s.act)
+    gemm(f"moe: up (grouped, {rows}-row tiles)", lambda: X.grouped_linear(xs, w.up, s.ff, p, s.act), n, s.ff, E, s.experts)
     y = X.grouped_linear(g, w.down, E, p)
     gemm("moe: down (grouped)", lambda: X.grouped_linear(g, w.down, E, p), n, E, s.ff, s.experts)
     a_s = ops.linear(h, w.up_s, None, "relu2")

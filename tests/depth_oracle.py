@@ -1,0 +1,214 @@
+"""Plain, slow statements of the mechanisms of the design ``Bolovik`` in double precision, one function each, and small random models
+to compare the framework with.  Nothing here comes from the package: a model is a configuration dict and a dict of named
+tensors."""
+import math
+
+import torch
+
+from layered_oracle import TensorDict, rel_error, rms_norm  # noqa: F401
+
+D = torch.float64
+
+
+def sigmoid(z):
+    return 1 / (1 + torch.exp(-z))
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def softplus(z):
+    return torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+# ------------------------------------------------------------------------------------------
+# norms and the sums over depth
+# ------------------------------------------------------------------------------------------
+def group_norm(x, w, groups, eps):
+    """Every one of ``groups`` equal parts of a vector is divided by its own root mean square."""
+    parts = x.unflatten(-1, (groups, x.shape[-1] // groups))
+    return rms_norm(parts, eps).flatten(-2) * w
+
+
+def depth_average(past, weights):
+    """``past``: embedding output and layer results so far."""
+    assert len(past) == len(weights)
+    return sum(w * x for w, x in zip(weights, past))
+
+
+# ------------------------------------------------------------------------------------------
+# gated delta rule
+# ------------------------------------------------------------------------------------------
+def short_conv(x, taps):
+    """x [T, channels], taps [channels, n]: the last column meets the current token."""
+    n = taps.shape[1]
+    out = torch.zeros_like(x)
+    for t in range(len(x)):
+        for j in range(n):
+            if t - j >= 0:
+                out[t] += taps[:, n - 1 - j] * x[t - j]
+    return out
+
+
+def unit(x):
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def log_decay(z, a_log, dt_bias):
+    return -torch.exp(a_log) * softplus(z + dt_bias)
+
+
+def delta_scan(q, k, v, beta, log_g):
+    """q, k [T, d], v [T, e], beta and log_g [T] of one head -> read-outs [T, e]."""
+    S = torch.zeros(q.shape[1], v.shape[1], dtype=D)
+    out = []
+    for t in range(len(q)):
+        S = torch.exp(log_g[t]) * S
+        u = beta[t] * (v[t] - S.T @ k[t])
+        S = S + torch.outer(k[t], u)
+        out.append(S.T @ q[t])
+    return torch.stack(out)
+
+
+def head_norm_gate(o, w, z, eps):
+    """o, z [T, H, e]."""
+    return rms_norm(o, eps) * w * silu(z)
+
+
+def delta(h, w, name, a, eps):
+    T, H, G = len(h), a["heads"], a["kv_heads"]
+    q, k, v = (silu(short_conv(h @ w[name + s].T, w[name + s + ".conv"])) for s in "qkv")
+    q, k, v = unit(q.view(T, G, -1)) * a["dim"] ** -0.5, unit(k.view(T, G, -1)), v.view(T, H, -1)
+    beta = sigmoid(h @ w[name + "b"].T)
+    log_g = log_decay(h @ w[name + "a"].T, w[name + "A_log"], w[name + "dt_bias"])
+    o = torch.stack([delta_scan(q[:, i // (H // G)], k[:, i // (H // G)], v[:, i], beta[:, i], log_g[:, i]) for i in range(H)], dim=1)
+    o = head_norm_gate(o, w[name + "norm"], (h @ w[name + "g"].T).view(T, H, -1), eps)
+    return o.flatten(1) @ w[name + "o"].T
+
+
+# ------------------------------------------------------------------------------------------
+# attention
+# ------------------------------------------------------------------------------------------
+def frequencies(rot):
+    """Radians per position of every pair; long wavelengths are stretched, those between the two bounds in part."""
+    out, sc = [], rot.get("scaling")
+    for i in range(rot["dims"] // 2):
+        f = rot["base"] ** (-2.0 * i / rot["dims"])
+        if sc is not None:
+            length = 2 * math.pi / f
+            if length > sc["original"] / sc["low"]:
+                f = f / sc["factor"]
+            elif length >= sc["original"] / sc["high"]:
+                s = (sc["original"] / length - sc["low"]) / (sc["high"] - sc["low"])
+                f = (1 - s) * f / sc["factor"] + s * f
+        out.append(f)
+    return out
+
+
+def rotate_half(vec, position, rot):
+    """One vector (or a stack of one position): entry i of the first half of the leading entries turns with entry i of the
+    second half."""
+    n = rot["dims"]
+    out = vec.clone()
+    for i, f in enumerate(frequencies(rot)):
+        c, s = math.cos(position * f), math.sin(position * f)
+        out[..., i] = vec[..., i] * c - vec[..., i + n // 2] * s
+        out[..., i + n // 2] = vec[..., i + n // 2] * c + vec[..., i] * s
+    return out
+
+
+def visible_keys(i, size, keep):
+    """Positions that position ``i`` sees: the last ``size`` and the first ``keep``."""
+    return [j for j in range(i + 1) if i - j < size or j < keep]
+
+
+def softmax_weights(s):
+    e = torch.exp(s - s.max())
+    return e / e.sum()
+
+
+def attend(q, k, v, a):
+    """q [T, H, d], k, v [T, G, .] of one sequence -> [T, H, vdim]."""
+    T, H = q.shape[:2]
+    m = a["mask"]
+    out = torch.zeros(T, H, v.shape[2], dtype=D)
+    for i in range(T):
+        see = visible_keys(i, m["size"], m["keep_first"])
+        for h in range(H):
+            g = h // (H // k.shape[1])
+            out[i, h] = softmax_weights((k[see, g] @ q[i, h]) * a["scale"]) @ v[see, g]
+    return out
+
+
+def attention(h, w, name, a, eps):
+    T, H, G = len(h), a["heads"], a["kv_heads"]
+    q, k, v = (h @ w[name + s].T + w[name + s + ".b"] for s in "qkv")
+    q, k, v = q.view(T, H, -1), k.view(T, G, -1), v.view(T, G, -1)
+    q = rms_norm(torch.stack([rotate_half(q[t], t, a["rot"]) for t in range(T)]), eps)
+    k = rms_norm(torch.stack([rotate_half(k[t], t, a["rot"]) for t in range(T)]), eps)
+    return attend(q, k, rms_norm(v, eps), a).flatten(1) @ w[name + "o"].T
+
+
+# ------------------------------------------------------------------------------------------
+# feed-forward
+# ------------------------------------------------------------------------------------------
+def gated(h, w, name, act):
+    return (act(h @ w[name + "gate"].T) * (h @ w[name + "up"].T)) @ w[name + "down"].T
+
+
+def route(z, top, groups):
+    """Router logits of one token -> chosen experts and their weights."""
+    s = sigmoid(z)
+    n = len(s) // groups["count"]
+    strength = [sum(sorted(s[g * n:(g + 1) * n].tolist(), reverse=True)[:2]) for g in range(groups["count"])]
+    best = sorted(range(groups["count"]), key=lambda g: -strength[g])[:groups["keep"]]
+    allowed = [e for e in range(len(s)) if e // n in best]
+    chosen = sorted(allowed, key=lambda e: -float(s[e]))[:top]
+    return chosen, s[chosen]
+
+
+def mixture(h, w, name, m):
+    r = m["router"]
+    out = torch.zeros_like(h)
+    for t in range(len(h)):
+        for c, p in zip(*route(w[name + "router"] @ h[t], r["top"], r["groups"])):
+            out[t] += p * gated(h[t], w, f"{name}e{c}.", silu)
+    return out
+
+
+def feed_forward(h, w, name, m):
+    return gated(h, w, name, gelu_tanh) if m["kind"] == "dense" else mixture(h, w, name, m)
+
+
+# ------------------------------------------------------------------------------------------
+# the model
+# ------------------------------------------------------------------------------------------
+def forward(cfg, w, tokens, hidden=None):
+    """Logits [T, vocab] of one whole sequence."""
+    w = {k: v.to(D) for k, v in w.items()}
+    eps, groups = cfg["norm"]["eps"], cfg["norm"]["groups"]
+    x = w["embed"][torch.tensor(tokens)]
+    past = [x]
+    for i, layer in enumerate(cfg["layers"]):
+        n = f"l{i}."
+        mixer = {"delta": delta, "attention": attention}[layer["type"]]
+        x = x + group_norm(mixer(x, w, n + "mix.", layer["mixer"], eps), w[n + "norm1"], groups, eps)
+        if layer["mlp"] is not None:
+            x = x + group_norm(feed_forward(x, w, n + "mlp.", layer["mlp"]), w[n + "norm2"], groups, eps)
+        past.append(x)
+        x = depth_average(past, w[n + "dwa"])
+        if hidden is not None:
+            hidden.append(x)
+    return group_norm(x, w["final.norm"], groups, eps) @ w["head"].T
+
+
+def greedy(cfg, w, prompt, new):
+    seq = list(prompt)
+    for _ in range(new):
+        seq.append(int(forward(cfg, w, seq)[-1].argmax()))
+    return seq[len(prompt):]

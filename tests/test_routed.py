@@ -522,7 +522,7 @@ def test_grouped_products(dtype, rows, N, Kd):
     p = X.plan(w, z.cuda(), rows)
     h, wt = rnd(T, Kd, seed=2), rnd(9 * N, Kd, seed=3, scale=Kd ** -0.5)
     pad = lambda t: torch.nn.functional.pad(t, (0, ops.pad8(Kd) - Kd)).to(dtype).cuda()[:, :Kd]  # noqa: E731
-    y = X.grouped_linear(X.dispatch(w, pad(h), p), pad(wt), N, p, relu2=True)
+    y = X.grouped_linear(X.dispatch(w, pad(h), p), pad(wt), N, p, "relu2")
     idx, slot = p.idx.cpu(), p.slot.cpu()
     assert bool(((slot < 0) == (idx >= 9)).all()) and len(set(slot[slot >= 0].tolist())) == int((idx < 9).sum())
     for t in range(0, T, 37):
