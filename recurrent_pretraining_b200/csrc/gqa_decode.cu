@@ -9,8 +9,9 @@
 // from the projection row and appends them.
 //
 // RING: position p lies in slot p % cap.  Queries and the new key are normed over the whole projection and / or rotated, the new
-// value is mixed with another layer's where they are formed.  Bounded scores need no running maximum.  With a single split the
-// sink and the division are applied here.
+// value is mixed with another layer's where they are formed; or every head is normed by itself (q and k once rotated, v).  Under a window
+// the sequence's first `keep` positions may stay visible: they have the ring's first slots for good and are counted in front of the
+// window's keys.  Bounded scores need no running maximum.  With a single split the sink and the division are applied here.
 #include "rowops.cuh"
 #include "softmax_math.cuh"
 
@@ -37,6 +38,8 @@ struct GqaDecode {
   float* first_out;                                // [B, ld_fout] unmixed values; null: not wanted
   const float* sink;                               // [H]; null: none
   __nv_bfloat16* out;                              // [B, ld_out] with a single split, else null
+  int keep, head_norm;                             // kept first positions; every head of q, k and v is normed without weights
+  float bound;                                     // no score is larger (0: not known)
 };
 
 constexpr int GD_KEYS = 16, GD_WARPS = 4;
@@ -62,15 +65,14 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 // ldmatrix fall into different banks.
 __host__ __device__ constexpr int gd_pitch(int cols) { return ((cols + 15) & ~15) * 2 + 16; }
 
-// Entry i of a head that is normed (weights w, factor r; null: not) and rotated (halves paired).
+// Entry i of a head with bias (null: none), scaled by r and the weights w (null: none) and rotated (halves paired).
 template <typename TI>
-__device__ __forceinline__ float head_entry(const TI* x, int i, const float* w, float r, int rot, const float* ct, const float* st) {
-  float v = ldf(x + i);
-  if (w) v *= r * w[i];
+__device__ __forceinline__ float head_entry(const TI* x, int i, const float* bias, const float* w, float r, int rot, const float* ct, const float* st) {
+  auto entry = [&](int e) { return (ldf(x + e) + (bias ? bias[e] : 0.f)) * (w ? r * w[e] : r); };
+  float v = entry(i);
   if (i < rot) {
     const int half = rot >> 1, j = i < half ? i : i - half, o = i < half ? i + half : i - half;
-    float u = ldf(x + o);
-    if (w) u *= r * w[o];
+    const float u = entry(o);
     v = i < half ? v * ct[j] - u * st[j] : v * ct[j] + u * st[j];
   }
   return v;
@@ -78,32 +80,33 @@ __device__ __forceinline__ float head_entry(const TI* x, int i, const float* w, 
 
 // Eight entries from i (a multiple of eight) on.
 template <typename TI>
-__device__ __forceinline__ void head_entries8(const TI* x, int i, const float* w, float r, int rot, const float* ct, const float* st, float (&v)[8]) {
+__device__ __forceinline__ void head_entries8(const TI* x, int i, const float* bias, const float* w, float r, int rot, const float* ct, const float* st, float (&v)[8]) {
   const int half = rot >> 1;
   if (i < rot && (half & 7)) {                                         // pairs do not fall into the same places of two groups
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = head_entry(x, i + j, w, r, rot, ct, st);
+    for (int j = 0; j < 8; ++j) v[j] = head_entry(x, i + j, bias, w, r, rot, ct, st);
     return;
   }
-  ld8(x + i, v);
-  float f[8];
-  if (w) {
-    ld8(w + i, f);
+  auto entries = [&](int e, float (&y)[8]) {
+    ld8(x + e, y);
+    float f[8];
+    if (bias) {
+      ld8(bias + e, f);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] *= r * f[j];
-  }
+      for (int j = 0; j < 8; ++j) y[j] += f[j];
+    }
+    if (w) ld8(w + e, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) y[j] *= w ? r * f[j] : r;
+  };
+  entries(i, v);
   if (i < rot) {
     const bool low = i < half;
     const int c = low ? i : i - half, o = low ? i + half : i - half;
     float u[8], cs[8], sn[8];
-    ld8(x + o, u);
+    entries(o, u);
     ld8(ct + c, cs);
     ld8(st + c, sn);
-    if (w) {
-      ld8(w + o, f);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) u[j] *= r * f[j];
-    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[j] = low ? v[j] * cs[j] - u[j] * sn[j] : v[j] * cs[j] + u[j] * sn[j];
   }
@@ -122,11 +125,13 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const int g = blockIdx.y / chunks, h0 = g * group + (blockIdx.y % chunks) * 16, nh = min(16, (g + 1) * group - h0);
   const int pos = P.pos[b];
   const int key_first = RING ? (P.chunked ? pos - pos % P.size : max(0, pos - P.size + 1)) : 0;
-  const int newest = pos - key_first, nkeys = newest + 1;              // keys are counted from the first visible one
-  const int slot0 = RING ? key_first % P.cap : 0;
+  const int kept = RING ? min(P.keep, key_first) : 0;                  // keys are counted: kept ones in front of the window, then the window
+  const int newest = kept + pos - key_first, nkeys = newest + 1;
+  const int slot0 = RING ? ring_slot(key_first, P.cap, P.keep) - kept : 0;
   auto slot_of = [&](int j) {
+    if (RING && j < kept) return j;
     int s = slot0 + j;
-    if (RING && s >= P.cap) s -= P.cap;
+    if (RING && s >= P.cap) s -= P.cap - P.keep;
     return s;
   };
   const int tiles = (nkeys + GD_KEYS - 1) / GD_KEYS, per = (tiles + P.splits - 1) / P.splits;
@@ -173,7 +178,24 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   }
   float rq = 1.f, rk = 1.f;
   const float *cos_t = nullptr, *sin_t = nullptr;
+  __shared__ float rh[18];                                             // factors of the heads' own norms: q heads, then k and v
   if constexpr (RING) {
+    if (P.head_norm) {                                                 // a rotation leaves the sum of squares alone
+      for (int i = warp; i < nh + 2; i += GD_WARPS) {
+        const int n = i <= nh ? P.dim : P.vdim, col = i < nh ? (h0 + i) * P.dim : i == nh ? P.off_k + g * P.dim : P.off_v + g * P.vdim;
+        float t = 0.f;
+        for (int c = 8 * lane; c < n; c += 256) {
+          float v[8];
+          head_entries8(r + col, c, P.in_bias ? P.in_bias + col : nullptr, nullptr, 1.f, 0, nullptr, nullptr, v);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) t += v[j] * v[j];
+        }
+        t = warp_sum(t);
+        if (lane == 0) rh[i] = 1.f / sqrtf(t / static_cast<float>(n) + P.eps);
+      }
+      __syncthreads();
+      rk = rh[nh];
+    }
     cos_t = P.cosT + static_cast<size_t>(pos) * (P.rot >> 1);
     sin_t = P.sinT + static_cast<size_t>(pos) * (P.rot >> 1);
     if (P.q_norm) {
@@ -208,7 +230,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
       float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
       if (hh < nh && c < P.dim) {
         const int at = (h0 + hh) * P.dim;
-        head_entries8(r + at, c, P.q_norm ? P.q_norm + at : nullptr, rq, P.rot, cos_t, sin_t, v);
+        head_entries8(r + at, c, P.in_bias ? P.in_bias + at : nullptr, P.q_norm ? P.q_norm + at : nullptr, P.head_norm ? rh[hh] : rq, P.rot, cos_t, sin_t, v);
       }
       st8(reinterpret_cast<__nv_bfloat16*>(sq) + hh * (kp / 2) + c, v);
     }
@@ -244,7 +266,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   }
   const bool capped = RING && P.softcap > 0.f;
   const float cap_log2 = P.softcap * 1.4426950408889634f, cap_exp = capped ? 2.f * rowmul / P.softcap : 0.f;
-  const bool bounded = capped && cap_log2 <= 80.f;                     // weights lie in 2^(-80 .. 80): no running maximum
+  const bool bounded = RING && (capped ? cap_log2 <= 80.f : P.bound > 0.f && P.bound * 1.4426950408889634f <= 80.f);      // weights lie in 2^(-80 .. 80): no running maximum
   const float m_start = bounded ? 0.f : -INFINITY;
   float m[2] = {m_start, m_start}, l[2] = {0.f, 0.f};
   float o[NV][2][4];
@@ -278,9 +300,11 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
           const int cc = isk ? c : c - P.dim, vc = g * P.vdim + cc;
           float f[8];
           if (isk) {
-            head_entries8(r + P.off_k + g * P.dim, cc, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk, P.rot, cos_t, sin_t, f);
+            head_entries8(r + P.off_k + g * P.dim, cc, P.in_bias ? P.in_bias + P.off_k + g * P.dim : nullptr, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk,
+                          P.rot, cos_t, sin_t, f);
           } else {
-            ld8(r + P.off_v + vc, f);
+            head_entries8(r + P.off_v + g * P.vdim, cc, P.in_bias ? P.in_bias + P.off_v + g * P.vdim : nullptr, nullptr, P.head_norm ? rh[nh + 1] : 1.f, 0,
+                          nullptr, nullptr, f);
             if (P.first_out) st8(P.first_out + static_cast<size_t>(b) * P.ld_fout + vc, f);
             if (P.lam) {
               const float lam = *P.lam;
@@ -505,10 +529,10 @@ B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_
 B200_API int b200_ring_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
   const GqaDecode& P = *Pp;
   if (!gqa_decode_ok(P, B) || P.size <= 0 || P.rot < 0 || (P.rot & 1) || P.rot > P.dim || (P.rot && (!P.cosT || !P.sinT)) || !P.q_norm != !P.k_norm ||
-      (P.lam && !P.first) || P.softcap < 0.f) return -1;
+      (P.lam && !P.first) || P.softcap < 0.f || P.keep < 0 || (P.keep && P.chunked) || (P.head_norm && P.q_norm)) return -1;
   if (((P.ld_in | P.off_k | P.off_v | P.ld_first | P.ld_fout) & 7) ||
       ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(P.q_norm) | reinterpret_cast<uintptr_t>(P.k_norm) | reinterpret_cast<uintptr_t>(P.cosT) |
-        reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.first) | reinterpret_cast<uintptr_t>(P.first_out)) & 15)) return -1;
+        reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.in_bias) | reinterpret_cast<uintptr_t>(P.first) | reinterpret_cast<uintptr_t>(P.first_out)) & 15)) return -1;
   if (P.splits == 1 ? (!P.out || (P.ld_out & 7) || (reinterpret_cast<uintptr_t>(P.out) & 15)) : (P.out || !P.part_o || !P.part_ml)) return -1;
   return gqa_decode_launch<true>(in, P, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
 }

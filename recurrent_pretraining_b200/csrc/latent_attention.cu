@@ -20,10 +20,11 @@
 // add a constant; the others (those near the diagonal) read the bias per element, lanes at consecutive distances.
 //
 // CAPPED: keys and values come from the step's key stream, there is neither a rotated part nor a gate.  A tile lies inside one chunk,
-// so a chunk is nothing but the first key of its tiles.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
+// so a chunk is nothing but the first key of its tiles.  The first keys of a sequence may stay visible beside the window: their blocks
+// come in front of the window's when there is a gap between the two, and are the first of one range otherwise.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
 // every score of a warp's columns is well below the cap, exponential and reciprocal otherwise.
 //
-// BOUNDED: CAPPED with a cap that is not large.  The softmax needs no running maximum and takes its columns as they come, and a query
+// BOUNDED: CAPPED with a cap that is not large, or with scores that are known to be small without one.  The softmax needs no running maximum and takes its columns as they come, and a query
 // row is shared by two threads: sixteen softmax warps, each with half of a block's columns and its weights over its own half of the
 // scores.
 #include <cuda.h>
@@ -62,6 +63,7 @@ struct LatentAttnParams {
   const float* sink;            // [H] natural-log units; null: none
   int capped;                   // scores are capped
   float cap_log2, cap_exp;      // cap in log2 units; exponent of e^(2 score / cap) per raw score, log2 units
+  int keep;                     // keys of a sequence that stay visible beside the window
   float cap_poly[3], poly_max;  // capped log2 score = raw * polynomial(raw^2) for |raw| <= poly_max
 };
 enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2, BOUNDED = 3 };
@@ -146,13 +148,25 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   const int h = blockIdx.x, hk = KIND != LATENT ? h / p.group : h;
   const int4 tile = p.tiles[blockIdx.y];
   const int q0 = tile.x, nrows = tile.y, s0 = tile.z, kbase = tile.w;
-  const int kstart = max(kbase, s0 - p.window + 1);
-  // key blocks [jb, je) of both tiles, counted from kstart
+  int kstart = max(kbase, s0 - p.window + 1);
+  // key blocks [jb, je) of both tiles: nkb blocks of kept keys, the others counted from kstart
+  int nkb = 0;
+  if constexpr (KIND >= CAPPED) {
+    if (p.keep > 0) {
+      nkb = (p.keep + BN - 1) / BN;
+      if (kstart - kbase <= nkb * BN) {
+        nkb = 0;
+        kstart = kbase;
+      }
+    }
+  }
+  const bool keeps = KIND >= CAPPED && p.keep > 0;
   const int last_a = min(LA_BM, nrows) - 1, last_b = nrows - 1;
-  const int je0 = (s0 + last_a - kstart) / BN + 1;
-  const int jb1 = nrows > LA_BM ? (max(kbase, s0 + LA_BM - p.window + 1) - kstart) / BN : 0;
-  const int je1 = nrows > LA_BM ? (s0 + last_b - kstart) / BN + 1 : 0;
+  const int je0 = nkb + (s0 + last_a - kstart) / BN + 1;
+  const int jb1 = nrows > LA_BM && !keeps ? (max(kbase, s0 + LA_BM - p.window + 1) - kstart) / BN : 0;
+  const int je1 = nrows > LA_BM ? nkb + (s0 + last_b - kstart) / BN + 1 : 0;
   const int nmax = max(je0, je1);
+  auto block_key = [&](int j) { return KIND >= CAPPED ? (j < nkb ? kbase + j * BN : kstart + (j - nkb) * BN) : kstart + j * BN; };   // first key of a block
 
   auto load_q = [&](int x) {
     mbar_expect_tx(&bars->q_full[x], q_bytes);
@@ -163,7 +177,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   };
   auto load_k = [&](int j, int s) {
     mbar_expect_tx(&bars->k_full[s], k_bytes);
-    for (int c = 0; c < pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, kstart + j * BN, hk);
+    for (int c = 0; c < pn; ++c) tma_load_3d(sK + s * k_bytes + c * KPANEL, &tmKn, &bars->k_full[s], c * 64, block_key(j), hk);
     for (int c = 0; c < pr; ++c)
       tma_load_2d(sK + s * k_bytes + (pn + c) * KPANEL, &tmKr, &bars->k_full[s], c * 64, kstart + j * BN);
   };
@@ -232,7 +246,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           if (!mbar_wait(&bars->v_empty[s], v.ph ^ 1, abort_flag, p.err, ERR_WAIT_ATTN)) break;
           mbar_expect_tx(&bars->v_full[s], v_bytes);
           for (int c = 0; c < p.pv; ++c)
-            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, kstart + j * BN, hk);
+            tma_load_3d(sV + s * v_bytes + c * KPANEL, &tmV, &bars->v_full[s], c * 64, block_key(j), hk);
           issued = j + 1;
         }
         for (int j = max(0, issued - p.vst); j < issued; ++j) {
@@ -326,7 +340,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
     const int jb = x ? jb1 : 0, je = x ? je1 : je0;
     // blocks [j_lo, j_hi) are visible to every row of the tile; the others are masked
     const int lo_last = max(kbase, s0 + (x ? last_b : last_a) - p.window + 1);
-    const int j_lo = (lo_last - kstart + BN - 1) / BN, j_hi = (s0 + x * LA_BM + 1 - kstart) / BN;
+    const int j_lo = nkb + (lo_last - kstart + BN - 1) / BN, j_hi = nkb + (s0 + x * LA_BM + 1 - kstart) / BN;
     const int hi = s0 - kstart + x * LA_BM + quad * 32 + lane;   // newest visible key of this thread's row, from kstart
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t ts = tmem_base + x * BN + lane_addr;
@@ -345,7 +359,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       tc_fence_after();
       if constexpr (KIND == BOUNDED) {        // 32 columns at a time: no maximum to wait for
         const bool edge = j < j_lo || j >= j_hi;
-        const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
+        const int off = block_key(j) - kstart, cmax = hi - off, cmin = max(kbase - kstart - off, cmax - p.window + 1);
+        const int ckeep = kbase + p.keep - kstart - off;            // columns in front of it are kept keys
         float2 rs = make_float2(0.f, 0.f);
         constexpr int COLS = BN / SPLIT;
 #pragma unroll
@@ -364,8 +379,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
             for (int i = 0; i < 32; i += 2) {
               float2 y = cap(i);
               if constexpr (decltype(masked)::value) {
-                if (c + i < cmin || c + i > cmax) y.x = -INFINITY;
-                if (c + i + 1 < cmin || c + i + 1 > cmax) y.y = -INFINITY;
+                if ((c + i < cmin && c + i >= ckeep) || c + i > cmax) y.x = -INFINITY;
+                if ((c + i + 1 < cmin && c + i + 1 >= ckeep) || c + i + 1 > cmax) y.y = -INFINITY;
               }
               const float2 pr = make_float2(ex2_approx(y.x), ex2_approx(y.y));
               r2[(i >> 1) & 1] = fadd2(r2[(i >> 1) & 1], pr);
@@ -373,7 +388,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
             }
           };
           auto small = [&](int i) { return cap_small(make_float2(sv[i], sv[i + 1]), p); };
-          if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
+          auto plain = [&](int i) { return fmul2(make_float2(sv[i], sv[i + 1]), make_float2(scale_log2, scale_log2)); };
+          if (!p.capped) {
+            if (edge) weigh(plain, std::true_type());
+            else weigh(plain, std::false_type());
+          } else if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
             if (edge) weigh(small, std::true_type());
             else weigh(small, std::false_type());
           } else {
@@ -413,10 +432,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         }
         }
         if (j < j_lo || j >= j_hi) {
-          const int cmax = hi - j * BN, cmin = max(kbase - kstart - j * BN, cmax - p.window + 1);
+          const int off = block_key(j) - kstart, cmax = hi - off, cmin = max(kbase - kstart - off, cmax - p.window + 1);
+          const int ckeep = KIND >= CAPPED ? kbase + p.keep - kstart - off : cmin;       // columns in front of it are kept keys
 #pragma unroll
           for (int i = 0; i < BN; ++i)
-            if (i < cmin || i > cmax) sv[i] = -INFINITY;
+            if ((i < cmin && (KIND < CAPPED || i >= ckeep)) || i > cmax) sv[i] = -INFINITY;
         }
         float mul = KIND == CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
         if constexpr (KIND == BIAS) {
@@ -739,12 +759,13 @@ B200_API int b200_capped_attention_supported(int dim, int vdim) { return latent_
 
 // q: [T, ld_q] (head h at column h dim), k / v: key stream [K, ld_kv] (head g at column g dim / g vdim), out: [T, ld_out]; tiles as in
 // LatentAttnParams, none of them across the border of a chunk (whose first key is the tile's).  window: visible keys.  scale > 0;
-// softcap 0: scores are not capped; sink: [H] or null.
+// softcap 0: scores are not capped; sink: [H] or null.  keep: first keys of a sequence that stay visible; bound: no score is larger (0: not
+// known).
 B200_API int b200_capped_attention(const void* q, const void* k, const void* v, void* out, const int* tiles, const float* sink, int n_tiles, int T,
-                                   int K, int H, int G, int dim, int vdim, int ld_q, int ld_kv, int ld_out, int window, float scale,
-                                   float softcap, void* stream, int* err) {
+                                   int K, int H, int G, int dim, int vdim, int ld_q, int ld_kv, int ld_out, int window, int keep,
+                                   float scale, float softcap, float bound, void* stream, int* err) {
   const LatentAttnPlan plan = latent_attn_plan(dim, 0, vdim);
-  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || G <= 0 || H % G || T <= 0 || K <= 0 || window <= 0 || !(scale > 0.f) || softcap < 0.f) return -1;
+  if (!plan.bn || n_tiles <= 0 || n_tiles > 65535 || H <= 0 || G <= 0 || H % G || T <= 0 || K <= 0 || window <= 0 || !(scale > 0.f) || softcap < 0.f || keep < 0) return -1;
   if ((reinterpret_cast<uintptr_t>(out) & 15) || (ld_out & 7)) return -2;
   CUtensorMap tm[5];
   int rc = make_tmap_rows(&tm[0], q, dim, H, T, dim, ld_q, LA_BM);
@@ -762,7 +783,8 @@ B200_API int b200_capped_attention(const void* q, const void* k, const void* v, 
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
   p.err = err;
   p.group = H / G; p.sink = sink;
-  bool bounded = false;
+  p.keep = keep;
+  bool bounded = softcap <= 0.f && bound > 0.f && bound * 1.4426950408889634f <= 80.f;
   if (softcap > 0.f) {
     const double x = static_cast<double>(scale) / softcap, cap = softcap * 1.4426950408889634;
     p.capped = 1;

@@ -162,7 +162,7 @@ def stream_attention(L: GroupedLayout, a, inp: torch.Tensor, stream: torch.Tenso
     if inp.dtype == BF16:
         from . import grouped_kernels as GK
 
-        if GK.prompt_supported(L, a) and not a.keep:
+        if GK.prompt_supported(L, a):
             GK.stream_attention(L, a, inp, stream, layout, window, sink, out)
             return out
     k = base._k()
@@ -201,7 +201,7 @@ def ring_attention(L: GroupedLayout, a, inp: torch.Tensor, tr: QkvTransform, cac
         back = torch.arange(n + a.keep)[None]                        # key = position p - back, then the kept positions in front of the window
         key = torch.where(back < n, p[:, None] - back, back - n)
         see = torch.where(back < n, back <= (p % a.size if a.chunked else p)[:, None], key <= (p - n)[:, None])
-        k, v = _kv_heads(L, cache[r[:, None], ring_slots(key.clamp(min=0), cap, a.keep)])
+        k, v = _kv_heads(L, cache[r[:, None], ring_slots(torch.minimum(key.clamp(min=0), p[:, None]), cap, a.keep)])
         return ref.capped_attention(q.to(dtype), k, v, see, a.scale, a.softcap, sink).flatten(1).to(dtype)
     out = torch.empty(B, pad8(W), dtype=dtype, device=inp.device)[:, :W]
     attend, merge = ring_attention_pieces(L, a, inp, tr, cache, sink, first_out, pos, row, splits, out)
@@ -221,7 +221,7 @@ def ring_attention_pieces(L: GroupedLayout, a, inp, tr: QkvTransform, cache, sin
     if dtype == BF16:
         from . import grouped_kernels as GK
 
-        fused = GK.decode_supported(L) and not tr.head_norm
+        fused = GK.decode_supported(L)
 
     def attend():
         if fused:

@@ -14,7 +14,7 @@ from .memory_kernels import _dec_ok, _dec_per_sm, _GqaDecode
 
 _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
 _attn_ok = K._sig("b200_capped_attention_supported", [_i, _i])
-_attn = K._sig("b200_capped_attention", [_vp] * 6 + [_i] * 11 + [_f, _f, _vp, _vp])
+_attn = K._sig("b200_capped_attention", [_vp] * 6 + [_i] * 12 + [_f, _f, _f, _vp, _vp])
 _dec = K._sig("b200_ring_decode", [_vp, C.POINTER(_GqaDecode), _i, _i, _vp])
 
 
@@ -31,7 +31,7 @@ def stream_attention(L, a, inp, stream, layout, window: int, sink, out) -> None:
     tiles = cache[window]
     K._check(_attn(inp.data_ptr(), stream.data_ptr(), stream[:, L.kv_v:].data_ptr(), out.data_ptr(), tiles.data_ptr(), K._ptr(sink),
                    tiles.shape[0], inp.shape[0], stream.shape[0], L.heads, L.kv_heads, L.dim, L.vdim, inp.stride(0), L.ld_kv, out.stride(0),
-                   min(window, 2**30), a.scale, a.softcap or 0.0, K._stream(), K.err_word(inp.device).data_ptr()), "capped_attention")
+                   min(window, 2**30), a.keep, a.scale, a.softcap or 0.0, a.score_bound or 0.0, K._stream(), K.err_word(inp.device).data_ptr()), "capped_attention")
 
 
 @lru_cache(None)
@@ -55,5 +55,6 @@ def decode_attention(L, a, inp, tr, cache, sink, first_out, pos, row, part_o, pa
                    chunked=int(a.chunked), rot=tr.rot, ld_first=0 if tr.first is None else tr.first.stride(0),
                    ld_fout=0 if first_out is None else first_out.stride(0), ld_out=out.stride(0), eps=tr.eps, softcap=a.softcap or 0.0,
                    q_norm=p(tr.q_norm), k_norm=p(tr.k_norm), cosT=p(cos), sinT=p(sin), lam=p(tr.lam), first=p(tr.first), first_out=p(first_out),
-                   sink=p(sink), out=out.data_ptr() if splits == 1 else 0)
+                   sink=p(sink), out=out.data_ptr() if splits == 1 else 0, in_bias=p(tr.bias), keep=tr.keep, head_norm=int(tr.head_norm),
+                   bound=a.score_bound or 0.0)
     K._check(_dec(inp.data_ptr(), C.byref(s), inp.shape[0], int(inp.dtype == F32), K._stream()), "ring_decode")

@@ -18,7 +18,8 @@ class _GqaDecode(C.Structure):
                                   "bias_lead", "temp_every")] + [(n, _f) for n in ("temp_coef", "scale")] + \
                [(n, _vp) for n in ("in_bias", "bias", "pos", "row", "cache", "part_o", "part_ml")] + \
                [(n, _i) for n in ("size", "chunked", "rot", "ld_first", "ld_fout", "ld_out")] + [(n, _f) for n in ("eps", "softcap")] + \
-               [(n, _vp) for n in ("q_norm", "k_norm", "cosT", "sinT", "lam", "first", "first_out", "sink", "out")]
+               [(n, _vp) for n in ("q_norm", "k_norm", "cosT", "sinT", "lam", "first", "first_out", "sink", "out")] + \
+               [("keep", _i), ("head_norm", _i), ("bound", _f)]
 
 
 class _Chunks(C.Structure):

@@ -232,6 +232,18 @@ def _dusilorn(name, vocab, width, layers, heads, kv_heads, dim, vdim, chunk, win
             "logit_scale": 0.25, "layers": [{**mixers[i % 2], "mlp": moe if i else {"kind": "dense", "ff": ff}} for i in range(layers)]}
 
 
+def _bolovik(name, vocab, width, layers, memory, attention, window, keep, rot, ff, expert_ff, experts, top, groups):
+    """``layers`` layers, three delta memories and one attention in turn; the first has a dense feed-forward, the others mixtures."""
+    delta = {"type": "delta", "mixer": {**dict(zip(("heads", "kv_heads", "dim", "vdim"), memory)), "conv": 4}}
+    heads, kv_heads, dim, vdim = attention
+    attn = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window, "keep_first": keep},
+                                           "rot": {"base": 500000.0, "dims": rot, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}},
+                                           "scale": dim ** -0.5}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "groups": dict(zip(("count", "keep"), groups))}}
+    return {"name": name, "architecture": "Bolovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6, "groups": 2},
+            "layers": [{**(attn if i % 4 == 3 else delta), "mlp": moe if i else {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
 layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _gasovik("gasovik-tiny", 512, 128, 3, 4, 32, 16, 32, 64, 24, 256, share_from=2, original=64),
     _gasovik("gasovik-1b", 65536, 2048, 16, 16, 128, 64, 128, 512, 1024, 8192, share_from=12),
@@ -243,6 +255,9 @@ layered_configs: dict[str, dict] = {c["name"]: c for c in (
     _dusilorn("dusilorn-tiny", 512, 128, 4, 4, 2, 32, 40, 48, 20, 16, 256, 64, 6, 2, 3, 96),
     _dusilorn("dusilorn-2b", 65536, 2048, 16, 16, 4, 128, 128, 8192, 1024, 64, 8192, 1024, 32, 4, 4, 2048),
     _dusilorn("dusilorn-core-5280", 65536, 5280, 4, 55, 11, 96, 96, 8192, 4096, 96, 17920, 2560, 16, 2, 4, 5120),
+    _bolovik("bolovik-tiny", 512, 128, 4, (4, 2, 32, 40), (4, 2, 32, 40), 20, 4, 16, 256, 64, 8, 3, (4, 2)),
+    _bolovik("bolovik-3b", 65536, 2048, 16, (16, 8, 128, 128), (16, 4, 128, 128), 1024, 64, 64, 6144, 1024, 32, 6, (4, 2)),
+    _bolovik("bolovik-core-5280", 65536, 5280, 4, (44, 22, 96, 128), (55, 11, 96, 96), 4096, 128, 96, 17920, 2560, 16, 6, (4, 2)),
 )}
 
 name_to_config: dict[str, dict] = {c["name"]: c for c in configs}

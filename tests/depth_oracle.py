@@ -212,3 +212,92 @@ def greedy(cfg, w, prompt, new):
     for _ in range(new):
         seq.append(int(forward(cfg, w, seq)[-1].argmax()))
     return seq[len(prompt):]
+
+
+# ------------------------------------------------------------------------------------------
+# small models
+# ------------------------------------------------------------------------------------------
+SCALING = {"factor": 3.0, "low": 1.0, "high": 5.0, "original": 60}
+
+
+def attn(heads=4, kv_heads=2, dim=16, vdim=24, size=11, keep=3, scale=None, rot=8, base=500.0, scaling=SCALING):
+    rot = {"base": base, "dims": rot}
+    if scaling is not None:
+        rot["scaling"] = dict(scaling)
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": size, "keep_first": keep},
+                                           "scale": 1.3 * dim ** -0.5 if scale is None else scale, "rot": rot}}
+
+
+def memory(heads=4, kv_heads=2, dim=16, vdim=24, conv=4):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+
+
+def moe(experts=6, top=2, ff=24, count=3, keep=2):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "groups": {"count": count, "keep": keep}, "top": top}}
+
+
+def mlp(ff=40):
+    return {"kind": "dense", "ff": ff}
+
+
+def config(mixers, mlps, vocab=67, width=48, eps=1e-5, groups=3):
+    """One layer per mixer; ``mlps`` is cycled (None: a layer without feed-forward)."""
+    return {"architecture": "Bolovik", "vocab": vocab, "width": width, "norm": {"eps": eps, "groups": groups},
+            "layers": [{**m, "mlp": mlps[i % len(mlps)]} for i, m in enumerate(mixers)]}
+
+
+def shapes(cfg):
+    E, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, E), "final.norm": (E,), "head": (V, E)}
+    for i, layer in enumerate(cfg["layers"]):
+        a, m, n = layer["mixer"], layer["mlp"], f"l{i}."
+        for s in ("norm1",) + (() if m is None else ("norm2",)):
+            out[n + s] = (E,)
+        out[n + "dwa"] = (i + 2,)
+        x, H, G = n + "mix.", a["heads"], a["kv_heads"]
+        out[x + "o"] = (E, H * a["vdim"])
+        if layer["type"] == "attention":
+            for s, r in (("q", H * a["dim"]), ("k", G * a["dim"]), ("v", G * a["vdim"])):
+                out.update({x + s: (r, E), x + s + ".b": (r,)})
+        else:
+            for s, r in (("q", G * a["dim"]), ("k", G * a["dim"]), ("v", H * a["vdim"])):
+                out.update({x + s: (r, E), x + s + ".conv": (r, a["conv"])})
+            out.update({x + "g": (H * a["vdim"], E), x + "b": (H, E), x + "a": (H, E), x + "A_log": (H,), x + "dt_bias": (H,), x + "norm": (a["vdim"],)})
+        f = n + "mlp."
+        if m is not None:
+            parts = [("", m["ff"])] if m["kind"] == "dense" else [(f"e{e}.", m["expert"]["ff"]) for e in range(m["router"]["experts"])]
+            if m["kind"] == "moe":
+                out[f + "router"] = (m["router"]["experts"], E)
+            for p, ff in parts:
+                out.update({f + p + "gate": (ff, E), f + p + "up": (ff, E), f + p + "down": (E, ff)})
+    return out
+
+
+def random_weights(cfg, seed=0, sharp=1.0, router=3.0):
+    """bf16-representable weights.  ``sharp`` scales step sizes and decays, ``router`` the router, so that choices are seldom close.  Memories
+    reach from a few tokens to hundreds."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in shapes(cfg).items():
+        t = torch.randn(shape, generator=g)
+        if name.endswith(".A_log"):
+            t = t * 0.7 - 2.0
+        elif name.endswith(".dt_bias"):
+            t = t * 0.5 - 1.5
+        elif name.endswith(".dwa"):
+            t = 0.3 * t
+            t[-1] = 0.8
+        elif name.endswith(".conv"):
+            t = t * shape[1] ** -0.5
+        elif name.endswith((".q.b", ".k.b", ".v.b")):
+            t = t * 0.5
+        elif len(shape) == 1:
+            t = 1 + 0.3 * t
+        elif name != "embed":
+            t = t * shape[1] ** -0.5
+        if name.endswith(".router"):
+            t = t * router
+        if name.endswith((".mix.b", ".mix.a")):
+            t = t * sharp
+        out[name] = t.bfloat16()
+    return out
