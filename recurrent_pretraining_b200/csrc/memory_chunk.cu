@@ -5,21 +5,16 @@
 //   chunk_state : U = sum_j exp(F_end - F_j + i_j - m_loc) k_j v_j^T                              per (chunk, head), in parallel
 //   chunk_scan  : S before every chunk, S <- exp(F_end + m - m') S + exp(m_loc - m') U             per (sequence, head)
 //   chunk_out   : o_t = sum_(j <= t) exp(F_t - F_j + i_j - m_t) (q_t . k_j) v_j + exp(F_t + m - m_t) S^T q_t
+// The delta rule's u_j (delta_chunk.cu) take the place of v_j in chunk_out, with i = 0 and F from that file's kernels; keys and queries are
+// made unit vectors by factors on the weights, and the read-outs are normed and gated per head.
 // A fixed decay has i = 0 and needs no maxima m.  A gated memory carries the running maximum m (starting at 0) and its
 // normaliser n, which rides along as one more value column of ones.
 // Decays, gates, maxima, sums and the carried state are fp32.  Operands that stem from the state or carry a decay (S and the
 // weighted keys) enter the products as a bf16 head plus a bf16 remainder.
 // Between the kernels a state is stored transposed, [value rows][key columns], as chunk_out reads it.
-#include <cuda.h>
-
-#include "rowops.cuh"
-#include "softmax_math.cuh"
+#include "memory_chunk.cuh"
 
 namespace b200 {
-
-constexpr int MC_C = 128;                     // tokens per chunk
-constexpr int MC_PANEL = MC_C * 128;          // 128 rows x 64 bf16
-constexpr float LOG2E = 1.4426950408889634f;
 
 struct ChunkParams {
   int H, dim, vdim;
@@ -38,9 +33,12 @@ struct ChunkParams {
   float* n_before;                // gated: [chunks * H, dimp] normaliser before each chunk
   float* m_before;                // [chunks * H]
   float* m_init;                  // [sequences * H]
+  // DELTA
+  int group, ld_g;                // value heads per key head; pitch of the output gate's rows
+  const float *prefix, *fk;       // [chunks * H, 128] running sum of log decays; factor that makes the key a unit vector
   float* state;                   // cache [rows, H, dim, ldv]
   float* stab;                    // cache [rows, H, dim + 1]
-  const __nv_bfloat16* gate_out;  // gated: output gate, head h at column h * vdim, pitch ld_in
+  const __nv_bfloat16* gate_out;  // gated: output gate, head h at column h * vdim, pitch ld_g
   const float* norm_w;
   __nv_bfloat16* out;             // [T, ld_out]
   int* err;
@@ -60,29 +58,6 @@ __device__ __forceinline__ void token_gates(const ChunkParams& p, int t, int h, 
   li = p.cap * tanhf(zi / p.cap);
   const float z = p.cap * tanhf(zf / p.cap);
   lf = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-}
-
-// inclusive prefix over 128 threads in token order, in both halves of the CTA alike
-template <bool MAX>
-__device__ __forceinline__ float chunk_prefix(float v, float* red_all) {
-  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3;
-  float* red = red_all + 4 * (threadIdx.x >> 7);
-#pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const float w = __shfl_up_sync(0xffffffffu, v, o);
-    if (lane >= o) v = MAX ? fmaxf(v, w) : v + w;
-  }
-  named_barrier_sync(1, 256);                  // the eight warps that hold tokens
-  if (lane == 31) red[warp] = v;
-  named_barrier_sync(1, 256);
-  for (int w = 0; w < warp; ++w) v = MAX ? fmaxf(v, red[w]) : v + red[w];
-  return v;
-}
-
-__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(a, b);
-  const float2 h = unpack_bf16x2(hi);
-  lo = pack_bf16x2(a - h.x, b - h.y);
 }
 
 // ------------------------------------------------------------------------------------------------ states of single chunks
@@ -286,6 +261,8 @@ chunk_scan_kernel(const ChunkParams p) {
 }
 
 // ------------------------------------------------------------------------------------------------ outputs
+enum MemoryKind { DECAY = 0, GATED = 1, DELTA = 2 };
+
 struct ChunkOutBars {
   uint64_t qk_full, v_full, s_full, s_done, o_part, o_done, p_ready, final;
   uint32_t tmem_slot;
@@ -296,7 +273,7 @@ struct ChunkOutBars {
 // Warps 0-7: token j = thread & 127 of the chunk, its columns shared by the two halves; warp 8: copies and MMAs.
 // Shared memory is used twice so that two CTAs fit an SM: the values follow the keys once the scores are formed, the state's
 // remainder follows its head once that product is done.  Tensor memory: scores, then bf16 weights over them; outputs at MC_C.
-template <bool GATED>
+template <int KIND>
 __global__ void __launch_bounds__(288, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                  const __grid_constant__ CUtensorMap tmSh, const __grid_constant__ CUtensorMap tmSl, const ChunkParams p, int tmem_cols) {
@@ -315,6 +292,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const int4 c = p.chunks[ch];
   const int t0 = c.x, n = c.y;
   const size_t idx = static_cast<size_t>(ch) * p.H + h;
+  const int hk = KIND == DELTA ? h / p.group : h;
   if (threadIdx.x == 256) {
     mbar_init(&bars->qk_full, 1);
     mbar_init(&bars->v_full, 1);
@@ -329,8 +307,8 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     fence_proxy_async_smem();
     mbar_expect_tx(&bars->qk_full, p.pk * 2 * MC_PANEL);
     for (int i = 0; i < p.pk; ++i) {
-      tma_load_3d(sQ + i * MC_PANEL, &tmQ, &bars->qk_full, i * 64, t0, h);
-      tma_load_3d(sKV + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, h);
+      tma_load_3d(sQ + i * MC_PANEL, &tmQ, &bars->qk_full, i * 64, t0, hk);
+      tma_load_3d(sKV + i * MC_PANEL, &tmK, &bars->qk_full, i * 64, t0, hk);
     }
     mbar_expect_tx(&bars->s_full, p.pk * spanel);
     for (int i = 0; i < p.pk; ++i) tma_load_3d(sS + i * spanel, &tmSh, &bars->s_full, i * 64, 0, static_cast<int>(idx));
@@ -402,7 +380,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   } else {
     // exponents of this thread's row (and, as a key, of its column)
     float arow, einter, mrow = 0.f;
-    if constexpr (GATED) {
+    if constexpr (KIND == GATED) {
       float li = -INFINITY, lf = 0.f;
       if (j < n) token_gates(p, t0 + j, h, li, lf);
       if (threadIdx.x < p.dim) nb[threadIdx.x] = p.n_before[idx * p.dimp + threadIdx.x];
@@ -413,6 +391,12 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       arow = (F - mrow) * LOG2E;
       einter = expf(F + mb - mrow);
       gj[j] = (li - F) * LOG2E;
+    } else if constexpr (KIND == DELTA) {
+      const float F = p.prefix[idx * MC_C + j];
+      arow = F * LOG2E;
+      gj[j] = -arow;
+      nb[j] = p.fk[idx * MC_C + j];
+      einter = exp2f(arow);
     } else {
       const float ld = p.log2_decay[h];
       arow = ld * static_cast<float>(j);
@@ -420,6 +404,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       einter = exp2f(ld * static_cast<float>(j + 1));
     }
     einter *= p.qscale;
+    float qscale = p.qscale;
     named_barrier_sync(1, 256);
     const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t ts = tmem + lane_addr, to = ts + MC_C;
@@ -427,6 +412,23 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     uint32_t packed[2][16];
     bool ok = mbar_wait(&bars->s_done, 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
     if (ok) tc_fence_after();
+    if constexpr (KIND == DELTA) {                    // unit vectors: factor of this row's query, half of its columns each
+      float qq = 0.f;
+      if (ok && mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL) && half < p.pk) {
+#pragma unroll 4
+        for (int i = 0; i < 8; ++i) {
+          float q[8];
+          ld8(reinterpret_cast<const __nv_bfloat16*>(sQ + half * MC_PANEL + j * 128 + ((i ^ (j & 7)) << 4)), q);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) qq += q[e] * q[e];
+        }
+      }
+      nsum[half * MC_C + j] = qq;
+      named_barrier_sync(1, 256);
+      const float fq = 1.f / sqrtf(nsum[j] + nsum[MC_C + j] + 1e-6f);
+      qscale *= fq;
+      einter *= fq;
+    }
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
       const int c0 = 32 * half + 64 * b;
@@ -440,10 +442,11 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
           const float4 g = *reinterpret_cast<const float4*>(gj + c0 + i);
-          float w[4] = {g.x, g.y, g.z, g.w};
+          float w[4] = {g.x, g.y, g.z, g.w}, fk[4] = {1.f, 1.f, 1.f, 1.f};
+          if constexpr (KIND == DELTA) ld4(nb + c0 + i, fk);
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
-            w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * p.qscale * ex2_approx(arow + w[k]) : 0.f;
+            w[k] = c0 + i + k <= j ? __uint_as_float(v[i + k]) * qscale * ex2_approx(arow + w[k]) * fk[k] : 0.f;
             nq += w[k];
           }
           packed[b][i >> 1] = pack_bf16x2(w[0], w[1]);
@@ -451,7 +454,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         }
       }
     }
-    if constexpr (GATED) {
+    if constexpr (KIND == GATED) {
       // the state's part of n . q: this half's 64 key columns
       if (ok && mbar_wait(&bars->qk_full, 0, abort_flag, p.err, ERR_WAIT_TMA_FULL) && half < p.pk) {
         float d = 0.f;
@@ -498,8 +501,8 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const size_t t = static_cast<size_t>(t0) + (live ? j : 0);
       __nv_bfloat16* orow = p.out + t * p.ld_out + h * p.vdim;
       float f = 1.f;
-      if constexpr (GATED) {
-        f = 1.f / (fmaxf(fabsf(nsum[j] + nsum[MC_C + j]), expf(-mrow)) + 1e-6f);
+      if constexpr (KIND == GATED) f = 1.f / (fmaxf(fabsf(nsum[j] + nsum[MC_C + j]), expf(-mrow)) + 1e-6f);
+      if constexpr (KIND != DECAY) {
         float ss = 0.f;
 #pragma unroll 1
         for (int c0 = 0; c0 < p.vpad; c0 += 16) {     // padding columns are zero
@@ -514,12 +517,12 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         }
         f /= sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
       }
-      const __nv_bfloat16* grow = GATED ? p.gate_out + t * p.ld_in + h * p.vdim : nullptr;
-      const float* nw = GATED ? p.norm_w + h * p.vdim : nullptr;
+      const __nv_bfloat16* grow = KIND != DECAY ? p.gate_out + t * p.ld_g + h * p.vdim : nullptr;
+      const float* nw = KIND == GATED ? p.norm_w + h * p.vdim : p.norm_w;
 #pragma unroll 1
       for (int c0 = 16 * half; c0 < p.vpad; c0 += 32) {
         float g[2][8];
-        if constexpr (GATED) {                        // requested before the accumulator is read
+        if constexpr (KIND != DECAY) {                // requested before the accumulator is read
 #pragma unroll
           for (int q = 0; q < 2; ++q)
             if (c0 + 8 * q < p.vdim) ld8(grow + c0 + 8 * q, g[q]);
@@ -534,11 +537,11 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[8 * q + i]) * f;
-          if constexpr (GATED) {
+          if constexpr (KIND != DECAY) {
             float w[8];
             ld8(nw + c0 + 8 * q, w);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) o[i] *= w[i] * __fdividef(1.f, 1.f + __expf(-g[q][i]));
+            for (int i = 0; i < 8; ++i) o[i] *= w[i] * __fdividef(KIND == DELTA ? g[q][i] : 1.f, 1.f + __expf(-g[q][i]));
           }
           st8(orow + c0 + 8 * q, o);
         }
@@ -552,30 +555,6 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     tc_fence_after();
     tmem_dealloc(tmem, tmem_cols);
   }
-}
-
-typedef CUresult (*EncodeTiledFnM)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-// bf16 [planes, rows, cols] with the given pitches (elements); box: `box_rows` rows x 64 columns of one plane, 128-byte swizzle
-static int make_tmap_planes(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint64_t planes, uint64_t ld, uint64_t plane,
-                            uint32_t box_rows) {
-  static EncodeTiledFnM enc = nullptr;
-  if (!enc) {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess)
-      return -1;
-    enc = reinterpret_cast<EncodeTiledFnM>(ptr);
-  }
-  if ((reinterpret_cast<uintptr_t>(base) & 15) || (ld & 7) || (plane & 7)) return -2;
-  cuuint64_t dims[3] = {cols, rows, planes};
-  cuuint64_t strides[2] = {ld * 2, plane * 2};
-  cuuint32_t box[3] = {64, box_rows, 1};
-  cuuint32_t estr[3] = {1, 1, 1};
-  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? 0 : -3;
 }
 
 static int mc_smem_state(int pv, bool gated) { return 1024 + 1024 + (4 + pv + (gated ? 1 : 0)) * MC_PANEL; }
@@ -608,6 +587,7 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   p.pk = (p.dim + 63) / 64;
   p.pv = (p.vdim + 63) / 64;
   p.err = err;
+  p.ld_g = p.ld_in;
   CUtensorMap tq, tk, tv, th, tl;
   int rc = make_tmap_planes(&tq, q, p.dim, T, p.H, p.ld_in, p.dim, MC_C);
   if (!rc) rc = make_tmap_planes(&tk, k, p.dim, T, p.H, p.ld_in, p.dim, MC_C);
@@ -623,12 +603,41 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
 #define GO(G)                                                                                                          \
   {                                                                                                                    \
     if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
-        cudaFuncSetAttribute(chunk_out_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
+        cudaFuncSetAttribute(chunk_out_kernel<G ? GATED : DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
     if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 256, sm1, st>>>(tk, tv, p);                              \
     if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 127) / 128, p.H, n_seqs), 128, 0, st>>>(p);      \
-    if (parts & 4) chunk_out_kernel<G><<<dim3(p.H, n_chunks), 288, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
+    if (parts & 4) chunk_out_kernel<G ? GATED : DECAY><<<dim3(p.H, n_chunks), 288, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
   }
   if (gated) GO(true) else GO(false)
 #undef GO
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+// Read-outs of the delta rule: q, k: activated rows [T, ld_in] (key head g at column g dim), u: [T, ld_u] (head h at column h vdim),
+// p.s_hi / s_lo, prefix, fk: from delta_chunk.cu.
+B200_API int b200_delta_out(const void* q, const void* k, const void* u, const ChunkParams* Pp, int ld_u, int T, int n_chunks, void* stream, int* err) {
+  ChunkParams p = *Pp;
+  if (!b200_memory_chunk_supported(p.dim, p.vdim, 0) || T <= 0 || n_chunks <= 0 || n_chunks > 65535 || p.H <= 0 || p.H > 65535 || p.group <= 0 || p.H % p.group ||
+      ((p.ld_in | p.ld_out | p.ld_g | ld_u) & 7) || !p.prefix || !p.fk || !p.chunks) return -1;
+  if ((reinterpret_cast<uintptr_t>(p.out) | reinterpret_cast<uintptr_t>(p.gate_out) | reinterpret_cast<uintptr_t>(p.norm_w)) & 15) return -1;
+  p.dimp = p.dim;
+  p.vpad = (p.vdim + 15) & ~15;
+  p.vrows = p.vpad;
+  p.pk = (p.dim + 63) / 64;
+  p.pv = (p.vdim + 63) / 64;
+  p.err = err;
+  CUtensorMap tq, tk, tu, th, tl;
+  const uint64_t planes = static_cast<uint64_t>(n_chunks) * p.H;
+  int rc = make_tmap_planes(&tq, q, p.dim, T, p.H / p.group, p.ld_in, p.dim, MC_C);
+  if (!rc) rc = make_tmap_planes(&tk, k, p.dim, T, p.H / p.group, p.ld_in, p.dim, MC_C);
+  if (!rc) rc = make_tmap_planes(&tu, u, p.vdim, T, p.H, ld_u, p.vdim, MC_C);
+  if (!rc) rc = make_tmap_planes(&th, p.s_hi, p.dim, p.vpad, planes, p.dimp, static_cast<uint64_t>(p.vpad) * p.dimp, p.vpad);
+  if (!rc) rc = make_tmap_planes(&tl, p.s_lo, p.dim, p.vpad, planes, p.dimp, static_cast<uint64_t>(p.vpad) * p.dimp, p.vpad);
+  if (rc) return rc;
+  const int smem = mc_smem_out(p.pk, p.pv, p.vpad);
+  int cols = 256;
+  while (cols < MC_C + ((p.vpad + 31) & ~31)) cols <<= 1;
+  if (cudaFuncSetAttribute(chunk_out_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
+  chunk_out_kernel<DELTA><<<dim3(p.H, n_chunks), 288, smem, reinterpret_cast<cudaStream_t>(stream)>>>(tq, tk, tu, th, tl, p, cols);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }

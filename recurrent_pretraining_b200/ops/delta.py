@@ -138,6 +138,11 @@ def delta_prompt(L: DeltaLayout, w: DeltaWeights, act: torch.Tensor, inp: torch.
         return _plain(L, w, act, inp, ba, state, step.sequences(), inp.dtype)
     W = L.heads * L.vdim
     out = torch.empty(inp.shape[0], pad8(W), dtype=inp.dtype, device=inp.device)[:, :W]
+    if inp.dtype == BF16:
+        from . import delta_kernels as DK
+
+        if DK.supported(L):
+            return DK.delta_prompt(L, w, act, inp, ba, state, step, out)()
     k = _k()
     m = _struct(L, w, act, inp, out, state, seqs=step.seq_table, ba=ba)
     k.K._check(k.scan(act.data_ptr(), inp.data_ptr(), 0, out.data_ptr(), C.byref(m), len(step.portions), 0, _f32(inp), _f32(inp), k.K._stream()),

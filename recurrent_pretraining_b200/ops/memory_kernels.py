@@ -25,8 +25,8 @@ class _GqaDecode(C.Structure):
 class _Chunks(C.Structure):
     _fields_ = [(n, _i) for n in ("H", "dim", "vdim", "dimp", "vpad", "vrows", "pk", "pv", "ldv", "ld_in", "ld_out", "gate_t", "gate_h")] + \
                [(n, _f) for n in ("qscale", "cap", "eps")] + \
-               [(n, _vp) for n in ("chunks", "seqs", "log2_decay", "gates", "gate_bias", "u", "stat", "s_hi", "s_lo", "n_before", "m_before", "m_init", "state",
-                                   "stab", "gate_out", "norm_w", "out", "err")]
+               [(n, _vp) for n in ("chunks", "seqs", "log2_decay", "gates", "gate_bias", "u", "stat", "s_hi", "s_lo", "n_before", "m_before", "m_init")] + [("group", _i), ("ld_g", _i)] + \
+               [(n, _vp) for n in ("prefix", "fk", "state", "stab", "gate_out", "norm_w", "out", "err")]
 
 
 _attn_ok = K._sig("b200_biased_attention_supported", [_i, _i])
@@ -134,7 +134,7 @@ def _chunked(step, q, k, v, H: int, dim: int, vdim: int, ldv: int, out, state, q
     c = _Chunks(H, dim, vdim, 0, 0, 0, 0, 0, ldv, q.stride(0), out.stride(0), 0 if gates is None else gates.stride(0), 0 if gates is None else gates.stride(1),
                 qscale, cap, eps,
                 chunks.data_ptr(), seqs.data_ptr(), p(decay), p(gates), p(gate_bias), u.data_ptr(), stat.data_ptr(), hi.data_ptr(), lo.data_ptr(),
-                p(nb), m_before.data_ptr(), m_init.data_ptr(), state.data_ptr(), p(stab), p(gate_out), p(norm_w), out.data_ptr(), 0)
+                p(nb), m_before.data_ptr(), m_init.data_ptr(), state=state.data_ptr(), stab=p(stab), gate_out=p(gate_out), norm_w=p(norm_w), out=out.data_ptr())
     keep = (u, hi, lo, nb, scal, q, decay, gates, gate_bias, state, stab, gate_out, norm_w)      # alive as long as the callable
 
     def run(parts: int = 7):

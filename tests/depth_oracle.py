@@ -275,7 +275,7 @@ def shapes(cfg):
 
 def random_weights(cfg, seed=0, sharp=1.0, router=3.0):
     """bf16-representable weights.  ``sharp`` scales step sizes and decays, ``router`` the router, so that choices are seldom close.  Memories
-    reach from a few tokens to hundreds."""
+    reach from a few tokens to hundreds.  Sublayers add a part of the stream's size: rounding is not blown up from layer to layer."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in shapes(cfg).items():
@@ -285,12 +285,14 @@ def random_weights(cfg, seed=0, sharp=1.0, router=3.0):
         elif name.endswith(".dt_bias"):
             t = t * 0.5 - 1.5
         elif name.endswith(".dwa"):
-            t = 0.3 * t
-            t[-1] = 0.8
+            t = 0.15 * t
+            t[-1] = 0.9
         elif name.endswith(".conv"):
             t = t * shape[1] ** -0.5
         elif name.endswith((".q.b", ".k.b", ".v.b")):
             t = t * 0.5
+        elif name.endswith((".norm1", ".norm2")):
+            t = 0.35 + 0.1 * t
         elif len(shape) == 1:
             t = 1 + 0.3 * t
         elif name != "embed":

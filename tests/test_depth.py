@@ -43,6 +43,18 @@ def make(cfg, run, seed=0, **kw):
     return load(cfg, w, run), w
 
 
+def steady(cfg, run):
+    """In bf16 all experts are chosen: a router's nearly equal scores may fall either way, and memories carry the difference on.  (The
+    choice has its own tests.)"""
+    cfg = json.loads(json.dumps(cfg))
+    if run[1] == torch.bfloat16:
+        for layer in cfg["layers"]:
+            if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe":
+                r = layer["mlp"]["router"]
+                r["top"], r["groups"]["keep"] = r["experts"], r["groups"]["count"]
+    return cfg
+
+
 def engine(model, rows=4, max_len=400, **kw):
     from recurrent_pretraining_b200.engine.layered import LayeredEngine
 
@@ -71,7 +83,7 @@ def status_ok(run):
 
 
 def agree(got, want, run, what="", bf16=6e-2):
-    """Logits of every position.  In bf16 a router's nearly equal scores may fall either way: one position in ten may differ more."""
+    """Logits of every position."""
     d = got.double().cpu() - want
     d = d - d.mean(-1, keepdim=True)
     s = want - want.mean(-1, keepdim=True)
@@ -80,8 +92,7 @@ def agree(got, want, run, what="", bf16=6e-2):
     if run[1] == torch.float32:
         assert float(err.max()) < 4e-5, (what, float(err.max()), int(err.argmax()))
     else:
-        bad = int((err > bf16).sum())
-        assert bad <= max(1, len(err) // 10), (what, bad, float(err.max()), int(err.argmax()))
+        assert float(err.max()) < bf16, (what, float(err.max()), int(err.argmax()))
 
 
 def near(got, want, dtype, f32=2e-5, bf16=8e-3, what=""):
@@ -403,7 +414,7 @@ def test_decode_attention(run, size, reach, keep, sharp, splits):
             kv = torch.cat([old[r, :p].double(), new.to(dtype).double()])
             k, v = kv[:, :Gk * dim].view(-1, Gk, dim), kv[:, L.kv_v:L.kv_v + Gk * vdim].view(-1, Gk, vdim)
             want = attention_want(a, fq(full[b, :H * dim], p), k, v, O.visible_keys(p, reach, keep))
-            near(got[b], want.flatten(), dtype, bf16=2.5e-2, what=p)
+            near(got[b], want.flatten(), dtype, bf16=2.5e-2 * max(1.0, sharp / 10), what=p)     # rounding of q and k grows with the scores
             for at, m in ((0, Gk * dim), (L.kv_v, L.v_width)):
                 near(c[r, slot(p), at:at + m], new[0, at:at + m], dtype)
         idle = [5, 10, 16]
@@ -506,7 +517,8 @@ def test_delta_rule_over_prompts(run, size, kind):
         got = torch.cat(outs).double().view(T, L.heads, L.vdim)
         d = (got - want.view(T, L.heads, L.vdim))[~tiny]
         err = float(d.square().mean().sqrt() / want.square().mean().sqrt())
-        assert err < (2e-5 if dtype == torch.float32 else 1.2e-2), (cuts, err)
+        # alike keys: what is written cancels in the read-out, the rounding of what is written does not
+        assert err < (2e-5 if dtype == torch.float32 else 3e-2 if "keys" in kind else 1.2e-2), (cuts, err)
     status_ok(run)
 
 
@@ -620,7 +632,7 @@ def test_choice_within_the_best_groups(run, experts, top, count, keep):
 # ------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("name", list(CONFIGS))
 def test_prompt_matches_oracle(run, name):
-    cfg = CONFIGS[name]
+    cfg = steady(CONFIGS[name], run)
     model, w = make(cfg, run, seed=1)
     seq = tokens(80 if name != "wide" else 60, cfg["vocab"])
     hidden, got_hidden = [], []
@@ -636,7 +648,7 @@ def test_prompt_matches_oracle(run, name):
 @pytest.mark.parametrize("name", list(CONFIGS))
 @pytest.mark.parametrize("cuts", [[1], [2], [3, 1, 7], [40, 1], [13, 2, 1, 1, 30], [64, 5]], ids=str)
 def test_portions_and_decoding_match_the_whole_prompt(run, name, cuts):
-    cfg = CONFIGS[name]
+    cfg = steady(CONFIGS[name], run)
     if run[0] == "cpu" and name == "wide" and cuts != [13, 2, 1, 1, 30]:
         pytest.skip("one on the CPU")
     model, w = make(cfg, run, seed=2)
@@ -685,6 +697,7 @@ def test_every_part_shows(run):
     """Leaving out or changing any part of the design changes the logits far beyond the tolerance: the agreement of the other tests covers
     them."""
     cfg = O.config([O.memory(), O.attn(size=9), O.memory(heads=2, kv_heads=2)], [O.moe(), O.mlp()])
+    cfg = steady(cfg, run)
     model, w = make(cfg, run, seed=3)
     seq = tokens(60)
     want = O.forward(cfg, w, seq)
@@ -722,6 +735,7 @@ def test_far_tokens_come_through_memories_and_kept_positions(run):
 def test_long_decoding(run):
     """Rings that go round many times; the cache is full at the end."""
     cfg = O.config([O.attn(size=17, keep=5), O.memory(), O.attn(size=25, keep=0)], [O.moe(), O.mlp()])
+    cfg = steady(cfg, run)
     model, w = make(cfg, run, seed=8)
     seq = tokens(260)
     want = O.forward(cfg, w, seq)
@@ -733,12 +747,13 @@ def test_long_decoding(run):
 
 
 def test_first_tokens(run):
-    model, w = make(MIXED, run, seed=9)
+    cfg = steady(MIXED, run)
+    model, w = make(cfg, run, seed=9)
     eng = engine(model)
     for t in (0, 66):
-        agree(eng.step([(eng.open(), [t])]), O.forward(MIXED, w, [t]), run)
+        agree(eng.step([(eng.open(), [t])]), O.forward(cfg, w, [t]), run)
     seq = tokens(6)
-    want = O.forward(MIXED, w, seq)
+    want = O.forward(cfg, w, seq)
     for n in range(1, 6):
         row = eng.open()
         got = torch.cat([eng.step([(row, seq[:n])], [list(range(n))]), eng.step([(row, seq[n:])], [list(range(6 - n))])])
@@ -746,10 +761,11 @@ def test_first_tokens(run):
 
 
 def test_unequal_batches_match_each_alone(run):
-    model, w = make(MIXED, run, seed=10)
+    cfg = steady(MIXED, run)
+    model, w = make(cfg, run, seed=10)
     seqs = [tokens(n, seed=n) for n in (1, 33, 130, 5, 64)]
     more = [tokens(7, seed=100 + n) for n in range(5)]
-    wants = [O.forward(MIXED, w, s + m) for s, m in zip(seqs, more)]
+    wants = [O.forward(cfg, w, s + m) for s, m in zip(seqs, more)]
     eng = engine(model, rows=2)                                    # grows on demand
     rows = [eng.open() for _ in seqs]
     got = [[x] for x in eng.step(list(zip(rows, seqs)), [[len(s) - 1] for s in seqs]).split(1)]
@@ -776,14 +792,15 @@ def test_unequal_batches_match_each_alone(run):
 
 def test_rows_are_freed_and_used_again(run):
     """A row's keys, convolution inputs and states of its former sequence are not seen by the next one, which may be shorter or a single token."""
-    model, w = make(MIXED, run, seed=11)
+    cfg = steady(MIXED, run)
+    model, w = make(cfg, run, seed=11)
     eng = engine(model, rows=2)
     for k in range(4):
         a, b = eng.open(), eng.open()
         assert {a, b} == {0, 1} and eng.cache.rows == 2
         for row, n in ((a, 70 - 22 * k), (b, 1 + 20 * k)):
             seq = tokens(n + 4, seed=k)
-            agree(feed(eng, row, seq, [n, 1]), O.forward(MIXED, w, seq), run)
+            agree(feed(eng, row, seq, [n, 1]), O.forward(cfg, w, seq), run)
         eng.close(b)
         eng.close(a)
 
@@ -792,6 +809,7 @@ def test_greedy_generation_through_the_scheduler(run):
     from recurrent_pretraining_b200.engine import server as S
 
     cfg = O.config([O.memory(), O.attn()], [O.moe(), O.mlp()])
+    cfg = steady(cfg, run)
     model, w = make(cfg, run, seed=12)
     prompts = [tokens(n, seed=n) for n in (3, 12, 1, 7)]
     sched = S.BatchScheduler(S.make_backend(model, max_batch=4, max_len=64), window_ms=200.0, stop_ids=())
@@ -813,7 +831,8 @@ def test_greedy_generation_through_the_scheduler(run):
 
 
 def test_generation_stops_and_prefills_in_portions(run):
-    model, w = make(MIXED, run, seed=13)
+    cfg = steady(MIXED, run)
+    model, w = make(cfg, run, seed=13)
     eng = engine(model)
     prompts = [tokens(9), tokens(4)]
     plain = eng.generate(prompts, 20)
@@ -857,7 +876,8 @@ def test_trace_replay(run, tmp_path):
     import numpy as np
     from recurrent_pretraining_b200.engine.trace import replay
 
-    model, w = make(MIXED, run, seed=14)
+    cfg = steady(MIXED, run)
+    model, w = make(cfg, run, seed=14)
     a, b = tokens(20, seed=1), tokens(9, seed=2)
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:18], "want": [0, 17]}, {"id": "b", "tokens": b[:8], "want": [7]}], "end": []},
              {"step": 1, "entries": [{"id": "a", "tokens": a[18:19], "want": []}, {"id": "b", "tokens": b[8:], "want": []}], "end": ["b"]},
@@ -866,7 +886,7 @@ def test_trace_replay(run, tmp_path):
     eng = engine(model, 1, 64)
     replay(eng, [json.dumps(s) + "\n" for s in steps], str(tmp_path), answer)
     assert answer.getvalue() == "done 0\ndone 1\ndone 2\n" and not eng.cache.length
-    wa, wb = O.forward(MIXED, w, a), O.forward(MIXED, w, b)
+    wa, wb = O.forward(cfg, w, a), O.forward(cfg, w, b)
     agree(torch.from_numpy(np.fromfile(tmp_path / "0.f32", dtype="<f4")).view(3, -1), torch.stack([wa[0], wa[17], wb[7]]), run)
     agree(torch.from_numpy(np.fromfile(tmp_path / "2.f32", dtype="<f4")).view(1, -1), wa[19:], run)
 
@@ -890,6 +910,7 @@ def test_decode_steps_on_a_cache_that_grows(graphs):
     run = ("cuda", torch.bfloat16)
     cfg = O.config([O.memory(heads=8, kv_heads=4, dim=32, vdim=64), O.attn(heads=8, kv_heads=2, dim=32, vdim=64, size=25, keep=4)],
                    [O.mlp(1024), O.moe(8, 3, 128, 2, 1)], width=640, groups=2)
+    cfg = steady(cfg, run)
     model, w = make(cfg, run, seed=15)
     eng = engine(model, rows=1, use_graphs=graphs)
     seq = tokens(60)
@@ -910,7 +931,7 @@ def test_decode_steps_on_a_cache_that_grows(graphs):
 @pytest.mark.parametrize("name", ["mixed", "wide"])
 def test_large_batches_decode_in_groups(name):
     run = ("cuda", torch.bfloat16)
-    cfg = CONFIGS[name]
+    cfg = steady(CONFIGS[name], run)
     model, w = make(cfg, run, seed=16)
     eng = engine(model, rows=70)
     seqs = [tokens(3 + i % 9, seed=i) for i in range(70)]
@@ -928,7 +949,7 @@ def test_many_prompt_tokens_against_fp32(run=("cuda", torch.bfloat16)):
                    [O.moe(6, 3, 96, 2, 1), O.mlp(200)], width=256, groups=2)
     w = O.random_weights(cfg, 18, router=6.0)
     seqs = [tokens(n, seed=n) for n in (1500, 900, 3, 257)]
-    outs = []
+    cfg, outs = steady(cfg, run), []
     for dtype in (torch.bfloat16, torch.float32):
         eng = engine(load(cfg, w, ("cuda", dtype)), max_len=1600)
         rows = [eng.open() for _ in seqs]
