@@ -75,7 +75,7 @@ def closest_model(cfg):
     from ..models.hf_config import RavenConfig
 
     n, E = len(cfg.layers), cfg.width
-    a = cfg.layers[0].mixer
+    a = next(layer.mixer for layer in cfg.layers if layer.type != "delta")         # attention heads
     a = getattr(a, "left", a)
     per_layer = (cfg.active_param_count() - 2 * cfg.vocab * E) / n
     ff = max(256, int((per_layer - 4 * E * E) / (3 * E)) // 64 * 64)
@@ -434,6 +434,179 @@ def routed_ops_decode(model, B: int, context: int, t: Timer) -> list:
     return t.take()
 
 
+def _moe_ops_prefill(w, h, t: Timer) -> None:
+    """Pieces of a mixture without identity and shared experts on the rows h."""
+    from ..ops import memory as M
+    from ..ops import moe as X
+
+    s, (T, E) = w.spec, h.shape
+
+    def gemm(name, fn, M_, N, K, groups=1):
+        t.op(name, fn, 2.0 * (M_ * (N if s.act != "silu" or N == E else N // 2) + M_ * K + groups * N * K), 2.0 * M_ * N * K)
+
+    z = X.router_logits(h, w.router)
+    gemm("moe: router product (fp32)", lambda: X.router_logits(h, w.router), T, w.router.shape[0], E)
+    rows = X.tile_rows(s, T, torch.bfloat16)
+    p = X.plan(w, z, rows)
+    n = T * s.top
+    t.op("moe: route + plan", lambda: X.plan(w, z, rows), 4.0 * T * (s.outputs + 4 * s.top), 0)
+    xs = X.dispatch(w, h, p)
+    t.op("moe: dispatch", lambda: X.dispatch(w, h, p), 2.0 * E * (T + n), 0)
+    g = X.grouped_linear(xs, w.up, s.ff, p, s.act)
+    gemm(f"moe: gate-up (grouped, {rows}-row tiles)", lambda: X.grouped_linear(xs, w.up, s.ff, p, s.act), n, 2 * s.ff, E, s.experts)
+    y = X.grouped_linear(g, w.down, E, p)
+    gemm("moe: down (grouped)", lambda: X.grouped_linear(g, w.down, E, p), n, E, s.ff, s.experts)
+    mixed = M.RowSum(y, p.slot, p.weight, h)
+    t.op("moe: combine", lambda: X.combine(mixed), 2.0 * E * (n + T), 0)
+    t.op("moe: whole", lambda: X.mixture(w, h), 4.0 * E * T + 6.0 * E * s.experts * s.ff, 6.0 * E * n * s.ff)
+
+
+def depth_ops_prefill(model, seqs: list, t: Timer) -> list:
+    """Kernels of a delta memory, a windowed layer and both kinds of feed-forward of a packed step of fresh prompts ``seqs``."""
+    from ..models.layered import PackedStep
+    from ..ops import delta as DL
+    from ..ops import delta_kernels as DK
+    from ..ops import depth as DP
+    from ..ops import grouped as G
+    from ..ops import latent as ops
+    from ..ops import memory as M
+
+    cfg, E, T = model.config, model.config.width, sum(seqs)
+    kinds = {layer.type: i for i, layer in reversed(list(enumerate(cfg.layers)))}
+    cache = model.new_cache(len(seqs), max(seqs))
+    step = PackedStep([(r, 0, [1] * n) for r, n in enumerate(seqs)], "cuda")
+    h = torch.randn(T, E, device="cuda").bfloat16()
+
+    def gemm(name, fn, M_, N, K):
+        t.op(name, fn, 2.0 * (M_ * N + M_ * K + N * K), 2.0 * M_ * N * K)
+
+    i = kinds["delta"]
+    mix = model.layers[i].mix
+    L, a, w = mix.layout, mix.spec, mix.weights
+    ring, state = cache.data[i, "conv"], cache.data[i, "state"]
+    w_ba = mix.w_in[L.off_ba:L.off_ba + 2 * a.heads, :E]
+    inp, ba = ops.linear(h, mix.w_in[:L.off_ba, :E]), M.gate_projections(h, w_ba)
+    gemm("delta: input projection", lambda: ops.linear(h, mix.w_in[:L.off_ba, :E]), T, L.off_ba, E)
+    gemm("delta: step size and decay projection (fp32)", lambda: M.gate_projections(h, w_ba), T, 2 * a.heads, E)
+    act = DL.short_conv(L, inp, mix.conv, ring, step)
+    t.op("delta: short convolution", lambda: DL.short_conv(L, inp, mix.conv, ring, step), 4.0 * T * L.channels, 0)
+    out = torch.empty(T, a.heads * a.vdim, dtype=torch.bfloat16, device="cuda")
+    run = DK.delta_prompt(L, w, act, inp, ba, state, step, out)
+    nbytes = 2.0 * T * (L.channels + 2 * a.heads * a.vdim) + 8.0 * T * a.heads
+    t.op("delta: memory (3 kernels)", run, nbytes, 6.0 * T * a.heads * a.dim * a.vdim)
+    for part, name in ((1, "single chunks"), (2, "recurrence"), (4, "read-outs + norm + gate")):
+        t.op("  delta: " + name, lambda part=part: run(part), nbytes, 0)
+    gemm("delta: output projection", lambda: ops.linear(out, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)
+    i = kinds["attention"]
+    mix = model.layers[i].mix
+    L, a = mix.layout, mix.spec
+    lay = step.layout(a.size - 1, a.keep)
+    gemm("attention: qkv projection + bias", lambda: ops.linear(h, mix.w_in[:, :E], mix.b_in), T, L.width_in, E)
+    inp = ops.linear(h, mix.w_in[:, :E], mix.b_in)
+    tr = mix._transform(None, cache.rope, None)
+    kv = torch.empty(lay.total, L.ld_kv, dtype=torch.bfloat16, device="cuda")
+    ring = cache.data[i, "kv"]
+    prep = lambda: G.qkv_prep_(L, inp, tr, step, lay.sidx, ring, kv)  # noqa: E731
+    prep()
+    t.op("attention: qkv_heads", prep, 2.0 * (T * (2 * a.heads * a.dim + 2 * L.ld_kv) + sum(min(n, ring.shape[1]) for n in seqs) * L.ld_kv), 0)
+    pairs = visible_pairs(seqs, a.size) + float(sum(min(a.keep, max(0, p - a.size + 1)) for n in seqs for p in range(n)))
+    t.op("attention: attention", lambda: G.stream_attention(L, a, inp, kv, lay, None), 2.0 * T * (a.heads * (a.dim + a.vdim) + L.ld_kv),
+         2.0 * pairs * a.heads * (a.dim + a.vdim))
+    o = G.stream_attention(L, a, inp, kv, lay, None)
+    gemm("attention: output projection", lambda: ops.linear(o, mix.w_o[:, :a.heads * a.vdim]), T, E, a.heads * a.vdim)
+    sub = ops.linear(o, mix.w_o[:, :a.heads * a.vdim])
+    norm, g = model.layers[i].norms["norm1"], cfg.norm_groups
+    for past in (0, 1, 8):
+        s = DP.DepthStream.begin(torch.randn(past + 1, T, E, device="cuda"))
+        weights = torch.full((past + 1,), 0.3, device="cuda") if past else None
+        t.op(f"depth_norm (sum over {past})" if past else "depth_norm", lambda s=s, weights=weights: DP.depth_norm_(s, sub, norm, g, 1e-6, torch.bfloat16, weights=weights),
+             T * E * (12.0 + (4.0 * past + 4.0 if past else 0)), 0)
+        del s
+    _moe_ops_prefill(next(layer.mlp for layer in model.layers if layer.mlp is not None and layer.mlp.wide == 0).weights, h, t)
+    mlp = model.layers[0].mlp
+    ff = mlp.spec.ff
+    gemm("gate-up projection + geglu", lambda: M.glu_linear(h, mlp.w_gu[:, :E], ff, "gelu"), T, 2 * ff, E)
+    d = M.glu_linear(h, mlp.w_gu[:, :E], ff, "gelu")
+    gemm("down projection", lambda: ops.linear(d, mlp.w_down[:, :ff]), T, E, ff)
+    return t.take()
+
+
+def depth_ops_decode(model, B: int, context: int, t: Timer) -> list:
+    from ..engine.layered import LayeredEngine
+    from ..ops import delta as DL
+    from ..ops import depth as DP
+    from ..ops import grouped as G
+    from ..ops import memory as M
+    from ..ops import moe as X
+
+    cfg, E = model.config, model.config.width
+    kinds = {layer.type: i for i, layer in reversed(list(enumerate(cfg.layers)))}
+    eng = LayeredEngine(model, B, context + 1, use_graphs=False)
+    cache = eng.cache
+    for d in cache.data.values():
+        d.normal_(std=0.1)
+    pos = torch.full((B,), context, dtype=torch.int32, device="cuda")
+    row = torch.arange(B, dtype=torch.int32, device="cuda")
+    h = torch.randn(B, E, device="cuda").bfloat16()
+
+    def skinny(name, xin, w):
+        N, K = w.shape
+        t.op(name, lambda: eng._dense(xin, w, 1 if N * B <= eng._work[1].numel() else 0), 2.0 * (N * K + B * K + B * N), 2.0 * B * N * K)
+
+    i = kinds["delta"]
+    mix = model.layers[i].mix
+    L, a = mix.layout, mix.spec
+    skinny("delta: input projection", h, mix.w_in[:, :E])
+    inp = torch.randn(B, L.width_in, device="cuda")
+    ring, state = cache.data[i, "conv"], cache.data[i, "state"]
+    t.op("delta: conv, update, norm, gate", lambda: DL.delta_decode(L, mix.weights, inp, ring, state, pos, row, torch.bfloat16),
+         8.0 * B * a.heads * a.dim * a.vdim + B * (4.0 * L.width_in + 2.0 * a.conv * L.channels + 2.0 * a.heads * a.vdim), 0)
+    skinny("delta: output projection", torch.randn(B, a.heads * a.vdim, device="cuda").bfloat16(), mix.w_o[:, :a.heads * a.vdim])
+    i = kinds["attention"]
+    mix = model.layers[i].mix
+    L, a = mix.layout, mix.spec
+    skinny("attention: qkv projection", h, mix.w_in[:, :E])
+    inp = torch.randn(B, L.width_in, device="cuda")
+    tr = mix._transform(None, cache.rope, None, raw=True)
+    o = torch.empty(B, M.pad8(a.heads * a.vdim), dtype=torch.bfloat16, device="cuda")[:, :a.heads * a.vdim]
+    splits = eng._splits(mix, B)
+    attend, merge = G.ring_attention_pieces(L, a, inp, tr, cache.data[i, "kv"], None, None, pos, row, splits, o)
+    keys = min(a.slots, context + 1)
+    t.op(f"attention: decode attention ({splits} splits)", attend, 2.0 * B * (keys * L.ld_kv + a.heads * (a.dim + a.vdim)),
+         2.0 * B * a.heads * keys * (a.dim + a.vdim))
+    if splits > 1:
+        t.op("attention: merge", merge, B * a.heads * a.vdim * (4.0 * splits + 2), 0)
+    norm, g = model.layers[i].norms["norm1"], cfg.norm_groups
+    acc = torch.zeros(B, E, device="cuda")
+    for past in (0, 8):
+        s = DP.DepthStream.begin(torch.randn(past + 1, B, E, device="cuda"))
+        weights = torch.full((past + 1,), 0.3, device="cuda") if past else None
+        t.op(f"depth_norm (sum over {past})" if past else "depth_norm", lambda s=s, weights=weights: DP.depth_norm_(s, acc, norm, g, 1e-6, torch.bfloat16, weights=weights),
+             B * E * (14.0 + (4.0 * past + 4.0 if past else 0)), 0)
+    w = next(layer.mlp for layer in model.layers if layer.mlp is not None and layer.mlp.wide == 0).weights
+    s = w.spec
+    parts = X.mixture_rows_pieces(w, h)
+    for f in parts[:-1]:
+        f()
+    used = X.plan(w, X.router_logits(h, w.router), 128).idx.unique().numel()
+    n, R = B * s.top, w.router.shape[0]
+    for name, f, b in (("moe: router product", parts[0], 2.0 * E * (R + B)), ("moe: route", parts[1], 4.0 * B * R),
+                       (f"moe: gate-up ({used} experts)", parts[2], 4.0 * E * used * s.ff + 2.0 * B * E + 2.0 * n * s.ff),
+                       ("moe: down", parts[3], 2.0 * E * used * s.ff + 2.0 * n * s.ff + 4.0 * E * n)):
+        t.op(name, f, b, 0)
+    st = DP.DepthStream.begin(torch.randn(9, B, E, device="cuda"))
+    weights = torch.full((9,), 0.3, device="cuda")
+    t.op("depth_norm with the sum of the experts (sum over 8)", lambda: DP.depth_norm_(st, parts[4], norm, g, 1e-6, torch.bfloat16, weights=weights),
+         E * (4.0 * n + 46.0 * B), 0)
+    mlp = model.layers[0].mlp
+    ff = mlp.spec.ff
+    skinny("gate-up projection", h, mlp.w_gu[:, :E])
+    work = torch.zeros(B, 2 * ff, device="cuda")
+    t.op("geglu", lambda: M.glu(work, ff, "gelu", torch.bfloat16), B * ff * 10.0, 0)
+    skinny("down projection", torch.randn(B, ff, device="cuda").bfloat16(), mlp.w_down[:, :ff])
+    return t.take()
+
+
 def closest_ops_prefill(model, B: int, S: int, t: Timer) -> list:
     from ..ops import attention as A
     from ..ops import cuda as K
@@ -548,7 +721,8 @@ def model_rates(cfg, prompt: int, new: int, batches) -> dict:
     return out
 
 
-SHAPES = ("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5280", "dusilorn-2b", "dusilorn-core-5280")
+SHAPES = ("gasovik-1b", "gasovik-core-5280", "fatudra-1b", "fatudra-core-5280", "dusilorn-2b", "dusilorn-core-5280", "bolovik-3b",
+          "bolovik-core-5280")
 
 
 def run(shapes=SHAPES, batches=(1, 8, 32), prompt: int = 2048, new: int = 128, ops_only: bool = False) -> dict:
@@ -565,14 +739,15 @@ def run(shapes=SHAPES, batches=(1, 8, 32), prompt: int = 2048, new: int = 128, o
             torch.cuda.empty_cache()
         t = Timer()
         ops_prefill, ops_decode = {"post_rms": (layer_ops_prefill, layer_ops_decode), "sandwich": (hybrid_ops_prefill, hybrid_ops_decode),
-                                   "sandwich_rms": (routed_ops_prefill, routed_ops_decode)}[cfg.design.norms]
-        few = replace(cfg, vocab=1024, layers=cfg.layers[:2 if cfg.design.sandwich else 1], loop=None)
+                                   "sandwich_rms": (routed_ops_prefill, routed_ops_decode), "post_group_rms": (depth_ops_prefill, depth_ops_decode)}[cfg.design.norms]
+        kept = 4 if cfg.design.depth_average else 2 if cfg.design.sandwich else 1
+        few = replace(cfg, vocab=1024, layers=cfg.layers[:kept], loop=None)
         model = LayeredForCausalLM(few, torch.bfloat16, "cuda").init_weights()
         S = 4096
         r["prefill_ops"] = {"tokens": S, "ours": ops_prefill(model, [S], t)}
         r["decode_ops"] = {f"batch {B}": {"context": S, "ours": ops_decode(model, B, S, t)} for B in (1, 8, 64)}
         del model
-        ref = closest_model(replace(cfg, vocab=1024, layers=cfg.layers[:3], loop=None))
+        ref = closest_model(replace(cfg, vocab=1024, layers=cfg.layers[:max(3, kept)], loop=None))
         r["prefill_ops"]["closest"] = closest_ops_prefill(ref, 1, S, t)
         for B in (1, 8, 64):
             r["decode_ops"][f"batch {B}"]["closest"] = closest_ops_decode(ref, B, S, t)
