@@ -273,7 +273,9 @@ struct ChunkOutBars {
 // Warps 0-7: token j = thread & 127 of the chunk, its columns shared by the two halves; warp 8: copies and MMAs.
 // Shared memory is used twice so that two CTAs fit an SM: the values follow the keys once the scores are formed, the state's
 // remainder follows its head once that product is done.  Tensor memory: scores, then bf16 weights over them; outputs at MC_C.
-template <int KIND>
+// KS: 16-column steps of the keys, known at compile time for common sizes (the issuing thread's address arithmetic would pace the
+// products otherwise); 0: read from the parameters.
+template <int KIND, int KS>
 __global__ void __launch_bounds__(288, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                  const __grid_constant__ CUtensorMap tmSh, const __grid_constant__ CUtensorMap tmSl, const ChunkParams p, int tmem_cols) {
@@ -331,15 +333,26 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       auto wait = [&](uint64_t* bar, uint32_t ph, int code) { return mbar_wait(bar, ph, abort_flag, p.err, code); };
       auto state_product = [&](uint32_t acc) {
         tc_fence_after();
+        if constexpr (KS > 0) {
+#pragma unroll
+          for (int t = 0; t < KS; ++t)
+            umma_bf16(tmem + MC_C, dq + ((t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3)), ds + (t >> 2) * (spanel >> 4) + 2 * (t & 3), idesc_o, t ? 1u : acc);
+          return;
+        }
         for (int t = 0; t < ks; ++t)
           umma_bf16(tmem + MC_C, dq + (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3), ds + (t >> 2) * (spanel >> 4) + 2 * (t & 3), idesc_o, (acc || t) ? 1u : 0u);
       };
       bool ok = wait(&bars->qk_full, 0, ERR_WAIT_TMA_FULL);
       if (ok) {
         tc_fence_after();
-        for (int t = 0; t < ks; ++t) {
-          const int o = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3);
-          umma_bf16(tmem, dq + o, dk + o, idesc_s, t ? 1u : 0u);
+        if constexpr (KS > 0) {
+#pragma unroll
+          for (int t = 0; t < KS; ++t) umma_bf16(tmem, dq + ((t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3)), dk + ((t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3)), idesc_s, t ? 1u : 0u);
+        } else {
+          for (int t = 0; t < ks; ++t) {
+            const int o = (t >> 2) * (MC_PANEL >> 4) + 2 * (t & 3);
+            umma_bf16(tmem, dq + o, dk + o, idesc_s, t ? 1u : 0u);
+          }
         }
         umma_commit(&bars->s_done);
         ok = wait(&bars->s_full, 0, ERR_WAIT_TMA_FULL);
@@ -367,8 +380,8 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
       if (ok) {
         tc_fence_after();
-        const int steps = (n + 15) >> 4;
-        for (int t = 0; t < steps; ++t) umma_bf16_ts(tmem + MC_C, tmem + t * 8, dv + t * 128, idesc_v, 1u);
+#pragma unroll
+        for (int t = 0; t < MC_C / 16; ++t) umma_bf16_ts(tmem + MC_C, tmem + t * 8, dv + t * 128, idesc_v, 1u);
         umma_commit(&bars->final);
       } else {
         bars->abort_flag = 1;
@@ -557,6 +570,22 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   }
 }
 
+template <int KIND, int KS>
+static int launch_chunk_out(const CUtensorMap* tm, const ChunkParams& p, int n_chunks, int smem, int cols, cudaStream_t st) {
+  if (cudaFuncSetAttribute(chunk_out_kernel<KIND, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
+  chunk_out_kernel<KIND, KS><<<dim3(p.H, n_chunks), 288, smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p, cols);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+template <int KIND>
+static int dispatch_chunk_out(const CUtensorMap* tm, const ChunkParams& p, int n_chunks, int smem, int cols, cudaStream_t st) {
+  switch ((p.dim + 15) / 16) {
+    case 8: return launch_chunk_out<KIND, 8>(tm, p, n_chunks, smem, cols, st);
+    case 6: return launch_chunk_out<KIND, 6>(tm, p, n_chunks, smem, cols, st);
+    case 4: return launch_chunk_out<KIND, 4>(tm, p, n_chunks, smem, cols, st);
+    default: return launch_chunk_out<KIND, 0>(tm, p, n_chunks, smem, cols, st);
+  }
+}
+
 static int mc_smem_state(int pv, bool gated) { return 1024 + 1024 + (4 + pv + (gated ? 1 : 0)) * MC_PANEL; }
 static int mc_smem_out(int pk, int pv, int vpad) { return 3072 + 1024 + (pk + (pk > pv ? pk : pv)) * MC_PANEL + pk * vpad * 128; }
 
@@ -602,11 +631,13 @@ B200_API int b200_memory_chunks(const void* q, const void* k, const void* v, con
   while (cols < MC_C + ((p.vpad + 31) & ~31)) cols <<= 1;
 #define GO(G)                                                                                                          \
   {                                                                                                                    \
-    if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess ||   \
-        cudaFuncSetAttribute(chunk_out_kernel<G ? GATED : DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm3) != cudaSuccess) return -3; \
+    if (cudaFuncSetAttribute(chunk_state_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1) != cudaSuccess) return -3; \
     if (parts & 1) chunk_state_kernel<G><<<dim3(p.H, n_chunks), 256, sm1, st>>>(tk, tv, p);                              \
     if (parts & 2) chunk_scan_kernel<G><<<dim3((p.vrows * (p.dimp / 4) + 127) / 128, p.H, n_seqs), 128, 0, st>>>(p);      \
-    if (parts & 4) chunk_out_kernel<G ? GATED : DECAY><<<dim3(p.H, n_chunks), 288, sm3, st>>>(tq, tk, tv, th, tl, p, cols);               \
+    if (parts & 4) {                                                                                                    \
+      const CUtensorMap tm[5] = {tq, tk, tv, th, tl};                                                                  \
+      return dispatch_chunk_out<G ? GATED : DECAY>(tm, p, n_chunks, sm3, cols, st);                                     \
+    }                                                                                                                  \
   }
   if (gated) GO(true) else GO(false)
 #undef GO
@@ -637,7 +668,6 @@ B200_API int b200_delta_out(const void* q, const void* k, const void* u, const C
   const int smem = mc_smem_out(p.pk, p.pv, p.vpad);
   int cols = 256;
   while (cols < MC_C + ((p.vpad + 31) & ~31)) cols <<= 1;
-  if (cudaFuncSetAttribute(chunk_out_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
-  chunk_out_kernel<DELTA><<<dim3(p.H, n_chunks), 288, smem, reinterpret_cast<cudaStream_t>(stream)>>>(tq, tk, tu, th, tl, p, cols);
-  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+  const CUtensorMap tm[5] = {tq, tk, tu, th, tl};
+  return dispatch_chunk_out<DELTA>(tm, p, n_chunks, smem, cols, reinterpret_cast<cudaStream_t>(stream));
 }
