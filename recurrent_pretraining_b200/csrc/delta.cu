@@ -20,7 +20,28 @@ struct ConvArgs {
   const int4* seqs;                               // {first chunk, chunks, cache row, first position}
 };
 
-// 32 groups of eight channels x 8 runs of 16 tokens.  The CTA of a portion's first chunk is the only one that reads the ring, so it
+// Eight neighbouring elements as they lie in memory.
+template <typename T> struct Raw8;
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+  __device__ __forceinline__ void get(float (&v)[8]) const { v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w; }
+};
+template <> struct Raw8<__nv_bfloat16> {
+  uint4 q;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(w[j]);
+      v[2 * j] = f.x;
+      v[2 * j + 1] = f.y;
+    }
+  }
+};
+
+// 32 groups of eight channels x 8 runs of 16 tokens, eight tokens on their way at a time.  The CTA of a portion's first chunk is the only one that reads the ring, so it
 // may write it afterwards.  TAPS: taps kept in registers (0: any number, inputs read again).
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
@@ -51,21 +72,29 @@ short_conv_kernel(const T* __restrict__ in, T* __restrict__ out, T* __restrict__
       for (int j = 0; j < TAPS; ++j) ld8(A.w + static_cast<size_t>(TAPS - 1 - j) * A.ch + c, w[j]);
 #pragma unroll
       for (int j = 1; j < TAPS; ++j) input(k0 - j, x[j - 1]);
-      for (int k = k0; k < k1; ++k) {
+      for (int b = k0; b < k1; b += 8) {
+        Raw8<T> raw[8];
 #pragma unroll
-        for (int j = TAPS - 1; j > 0; --j)
+        for (int k = 0; k < 8; ++k)
+          if (b + k < k1) raw[k].load(in + static_cast<size_t>(t0 + b + k) * A.ld_in + c);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
-        ld8(in + static_cast<size_t>(t0 + k) * A.ld_in + c, x[0]);
-        float v[8];
+        for (int k = 0; k < 8; ++k) {
+          if (b + k >= k1) break;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          float s = 0.f;
+          for (int j = TAPS - 1; j > 0; --j)
 #pragma unroll
-          for (int j = 0; j < TAPS; ++j) s += w[j][e] * x[j][e];
-          v[e] = silu_f(s);
+            for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+          raw[k].get(x[0]);
+          float v[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) s += w[j][e] * x[j][e];
+            v[e] = sizeof(T) == 2 ? __fdividef(s, 1.f + __expf(-s)) : silu_f(s);
+          }
+          st8(out + static_cast<size_t>(t0 + b + k) * A.ld_out + c, v);
         }
-        st8(out + static_cast<size_t>(t0 + k) * A.ld_out + c, v);
       }
     } else {
       for (int k = k0; k < k1; ++k) {
@@ -160,27 +189,54 @@ delta_scan_kernel(const TI* __restrict__ in, const TI* __restrict__ gate, T* __r
     const size_t t = static_cast<size_t>(t0) + j;
     const TI* r = in + t * M.ld_in;
     __syncthreads();                               // the previous token's vectors have been read
-    // value of a channel: activated already, or convolved here; the channel's ring gets its input from one CTA
-    auto channel = [&](int col, bool keeps) {
-      if constexpr (!RAW) return ldf(r + col);
-      const float x = ldf(r + col);
-      T* rg = ring + static_cast<size_t>(row) * M.taps * M.ch + col;
-      float s = M.conv_w[static_cast<size_t>(M.taps - 1) * M.ch + col] * x;
-      for (int i = 1; i < M.taps && i <= start; ++i)
-        s += M.conv_w[static_cast<size_t>(M.taps - 1 - i) * M.ch + col] * ldf(rg + static_cast<size_t>((start - i) % M.taps) * M.ch);
-      if (keeps) stf(rg + static_cast<size_t>(start % M.taps) * M.ch, x);
-      return silu_f(s);
-    };
+    // channels [q | k | v]: activated already, or convolved here (a channel's ring gets its input from one CTA), two per thread at a time with
+    // everything requested before anything is used
+    const int total = 2 * dim + ldv;
+    auto column = [&](int i) { return i < dim ? M.off_q + g * dim + i : i < 2 * dim ? M.off_k + g * dim + (i - dim) : M.off_v + h * vdim + (i - 2 * dim); };
+    auto put = [&](int i, float v) { (i < dim ? qs + i : i < 2 * dim ? ks + (i - dim) : vs + (i - 2 * dim))[0] = v; };
+    if constexpr (RAW) {
+      constexpr int N = 4;                         // taps held at a time
+      T* rg = ring + static_cast<size_t>(row) * M.taps * M.ch;
+      const int now = start % M.taps;
+      auto slot = [&](int back) { const int s = now - back; return static_cast<size_t>(s < 0 ? s + M.taps : s) * M.ch; };   // of `back` tokens ago
+      for (int i0 = tid; i0 < total; i0 += 512) {
+        float x[2][N], w[2][N];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int i = i0 + 256 * e, col = column(i);
+          const bool on = i < total && i < 2 * dim + vdim;
+#pragma unroll
+          for (int b = 0; b < N; ++b) {
+            const bool has = on && b < M.taps && b <= start;
+            x[e][b] = !has ? 0.f : b == 0 ? ldf(r + col) : ldf(rg + slot(b) + col);
+            w[e][b] = has ? M.conv_w[static_cast<size_t>(M.taps - 1 - b) * M.ch + col] : 0.f;
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int i = i0 + 256 * e, col = column(i);
+          if (i >= total) continue;
+          float s = 0.f;
+#pragma unroll
+          for (int b = 0; b < N; ++b) s += w[e][b] * x[e][b];
+          if (i < 2 * dim + vdim) {
+            for (int b = N; b < M.taps && b <= start; ++b) s += M.conv_w[static_cast<size_t>(M.taps - 1 - b) * M.ch + col] * ldf(rg + slot(b) + col);
+            if (i >= 2 * dim || h == g * group) stf(rg + slot(0) + col, x[e][0]);
+          }
+          put(i, silu_f(s));
+        }
+      }
+    } else {
+      for (int i = tid; i < total; i += 256) put(i, i < 2 * dim + vdim ? ldf(r + column(i)) : 0.f);
+    }
+    __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;
     for (int i = tid; i < dim; i += 256) {
-      const float q = channel(M.off_q + g * dim + i, h == g * group), k = channel(M.off_k + g * dim + i, h == g * group);
-      qs[i] = q;
-      ks[i] = k;
+      const float q = qs[i], k = ks[i];
       qq += q * q;
       kk += k * k;
       qk += q * k;
     }
-    for (int i = tid; i < ldv; i += 256) vs[i] = i < vdim ? channel(M.off_v + h * vdim + i, true) : 0.f;
     qq = warp_sum(qq);
     kk = warp_sum(kk);
     qk = warp_sum(qk);

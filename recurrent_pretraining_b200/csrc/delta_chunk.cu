@@ -357,17 +357,18 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 
 // ------------------------------------------------------------------------------------------------ recurrence over chunks
 struct DeltaStateBars {
-  uint64_t w_full, k_full, u0_full;            // W (head, remainder), keys and U0 of a chunk have landed
+  uint64_t w_full, k_full[2], u0_full;         // W (head, remainder), keys (every other chunk) and U0 of a chunk have landed
   uint64_t s_ready, x_done, u_ready, d_done;   // state in shared memory; W S formed; weighted U in shared memory; K^T U formed
   uint64_t s_free;                             // the state's tile has been copied out
   uint32_t tmem_slot;
   int abort_flag;
 };
 
-__host__ __device__ constexpr int ds_groups(int vb) { return vb > 32 ? vb / 32 : 1; }   // groups of 128 threads, up to 32 value columns each
-__host__ __device__ constexpr int ds_threads(int vb) { return 128 * ds_groups(vb) + 64; }
+constexpr int DS_VC = 16;                      // value columns of a compute thread
+__host__ __device__ constexpr int ds_threads(int vb) { return 128 * (vb / DS_VC) + 64; }
+__host__ __device__ constexpr int ds_u0_tiles(int vb) { return (vb + 31) / 32; }
 
-// CTA: VB value columns of one head of one sequence.  Compute warps: thread = token row of W S and key row of the state; then a warp for the MMAs
+// CTA: VB value columns of one head of one sequence.  Compute warps: thread = token row of W S and key row of the state, sixteen columns; then a warp for the MMAs
 // and one for the copies.  Heads and remainders of S (as rows) and of the weighted U (as columns) lie side by side: one product takes both.
 template <int VB, int KS>
 __global__ void __launch_bounds__(ds_threads(VB), 1)
@@ -376,14 +377,14 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
                    const DeltaChunkParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  constexpr int SPANEL = 2 * VB * 128, NG = ds_groups(VB), VC = VB / NG, UPANELS = (2 * VB + 63) / 64, MMA_WARP = 4 * NG;
+  constexpr int SPANEL = 2 * VB * 128, NG = VB / DS_VC, VC = DS_VC, U0T = ds_u0_tiles(VB), UPANELS = (2 * VB + 63) / 64, MMA_WARP = 4 * NG;
   DeltaStateBars* bars = reinterpret_cast<DeltaStateBars*>(smem);
   uint8_t* sWh = smem + 1024;
   uint8_t* sWl = sWh + p.pk * MC_PANEL;
-  uint8_t* sK = sWl + p.pk * MC_PANEL;         // two panels: the product's 128 rows are key columns
-  uint8_t* sU = sK + 2 * MC_PANEL;             // token rows: head columns, remainder columns
-  uint8_t* sU0 = sU + UPANELS * MC_PANEL;      // fp32 [128][32] per group
-  uint8_t* sS = sU0 + NG * MC_PANEL;           // value rows of the head, then of the remainder; key columns
+  uint8_t* sK = sWl + p.pk * MC_PANEL;         // twice two panels: the product's 128 rows are key columns
+  uint8_t* sU = sK + 4 * MC_PANEL;             // token rows: head columns, remainder columns
+  uint8_t* sU0 = sU + UPANELS * MC_PANEL;      // fp32 tiles [128][32]
+  uint8_t* sS = sU0 + U0T * MC_PANEL;           // value rows of the head, then of the remainder; key columns
   volatile int* abort_flag = &bars->abort_flag;
   const int v0 = blockIdx.x * VB, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int4 sq = p.seqs[blockIdx.z];
@@ -398,16 +399,17 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   };
   auto load_u0 = [&](int c) {
     const int row = ((c0 + c) * p.H + h) * MC_C;
-    mbar_expect_tx(&bars->u0_full, NG * MC_PANEL);
-    for (int i = 0; i < NG; ++i) tma_load_2d(sU0 + i * MC_PANEL, &tmU0, &bars->u0_full, v0 + 32 * i, row);
+    mbar_expect_tx(&bars->u0_full, U0T * MC_PANEL);
+    for (int i = 0; i < U0T; ++i) tma_load_2d(sU0 + i * MC_PANEL, &tmU0, &bars->u0_full, v0 + 32 * i, row);
   };
-  auto load_k = [&](int t0) {
-    mbar_expect_tx(&bars->k_full, p.pk * MC_PANEL);
-    for (int i = 0; i < p.pk; ++i) tma_load_3d(sK + i * MC_PANEL, &tmK, &bars->k_full, i * 64, t0, hk);
+  auto load_k = [&](int t0, int b) {
+    mbar_expect_tx(&bars->k_full[b], p.pk * MC_PANEL);
+    for (int i = 0; i < p.pk; ++i) tma_load_3d(sK + (2 * b + i) * MC_PANEL, &tmK, &bars->k_full[b], i * 64, t0, hk);
   };
   if (tid == 32 * MMA_WARP + 32) {
     mbar_init(&bars->w_full, 1);
-    mbar_init(&bars->k_full, 1);
+    mbar_init(&bars->k_full[0], 1);
+    mbar_init(&bars->k_full[1], 1);
     mbar_init(&bars->u0_full, 1);
     mbar_init(&bars->s_ready, 4 * NG);
     mbar_init(&bars->x_done, 1);
@@ -419,7 +421,8 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     fence_proxy_async_smem();
     load_w(0);
     load_u0(0);
-    load_k(p.chunks[c0].x);
+    load_k(p.chunks[c0].x, 0);
+    if (nc > 1) load_k(p.chunks[c0 + 1].x, 1);
   }
   if (warp == MMA_WARP) {
     tmem_alloc(&bars->tmem_slot, 4 * VB);
@@ -435,10 +438,11 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   if (warp == MMA_WARP) {
     if (lane == 0) {
       constexpr uint32_t idesc_x2 = make_idesc_bf16(128, 2 * VB, 0, 0), idesc_x = make_idesc_bf16(128, VB, 0, 0), idesc_d = make_idesc_bf16(128, 2 * VB, 1, 1);
-      const uint64_t dwh = make_smem_desc(smem_u32(sWh), 16, 1024), dwl = make_smem_desc(smem_u32(sWl), 16, 1024), ds = make_smem_desc(smem_u32(sS), 16, 1024),
+      uint64_t dwh = make_smem_desc(smem_u32(sWh), 16, 1024), dwl = make_smem_desc(smem_u32(sWl), 16, 1024), ds = make_smem_desc(smem_u32(sS), 16, 1024),
                      dk = make_smem_desc(smem_u32(sK), MC_PANEL, 1024), du = make_smem_desc(smem_u32(sU), MC_PANEL, 1024);
       for (int c = 0; c < nc; ++c) {
         const uint32_t ph = c & 1;
+        asm volatile("" : "+l"(dwh), "+l"(dwl), "+l"(ds), "+l"(dk), "+l"(du));      // descriptors are added up here, not kept for the whole loop
         if (!wait(&bars->w_full, ph, ERR_WAIT_TMA_FULL) || !wait(&bars->s_ready, ph, ERR_WAIT_TMEM_FULL)) break;
         tc_fence_after();
         if constexpr (KS > 0) {
@@ -460,21 +464,22 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
           }
         }
         umma_commit(&bars->x_done);
-        if (!wait(&bars->k_full, ph, ERR_WAIT_TMA_FULL) || !wait(&bars->u_ready, ph, ERR_WAIT_TMEM_FULL)) break;
+        if (!wait(&bars->k_full[ph], (c >> 1) & 1, ERR_WAIT_TMA_FULL) || !wait(&bars->u_ready, ph, ERR_WAIT_TMEM_FULL)) break;
         tc_fence_after();
+        const uint64_t dkc = dk + ph * (2 * MC_PANEL >> 4);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) umma_bf16(td, dk + k * 128, du + k * 128, idesc_d, k ? 1u : 0u);
+        for (int k = 0; k < 8; ++k) umma_bf16(td, dkc + k * 128, du + k * 128, idesc_d, k ? 1u : 0u);
         umma_commit(&bars->d_done);
       }
     }
   } else if (warp == MMA_WARP + 1) {
     if (lane == 0) {
-      int w = 1, u = 1, k = 1;                           // loads issued
+      int w = 1, u = 1, k = nc > 1 ? 2 : 1;              // loads issued
       bool ok = true;
       for (int c = 0; c < nc && ok; ++c) {
         const uint32_t ph = c & 1;
         const bool more = c + 1 < nc;
-        const int next = more ? p.chunks[c0 + c + 1].x : 0;
+        const int next = c + 2 < nc ? p.chunks[c0 + c + 2].x : 0;
         ok = wait(&bars->s_ready, ph, ERR_WAIT_TMEM_FULL);
         if (!ok) break;
         const int row = ((c0 + c) * p.H + h) * p.vpad + v0;
@@ -496,14 +501,15 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
           ++u;
         }
         ok = ok && wait(&bars->d_done, ph, ERR_WAIT_TMEM_FULL);
-        if (ok && more) {
-          load_k(next);
+        if (ok && c + 2 < nc) {
+          load_k(next, ph);
           ++k;
         }
       }
       bulk_wait_all();
       const unsigned long long begin = globaltimer_ns();   // a copy in flight has to land before the CTA ends
-      while (!(mbar_try_wait(&bars->w_full, (w - 1) & 1) && mbar_try_wait(&bars->u0_full, (u - 1) & 1) && mbar_try_wait(&bars->k_full, (k - 1) & 1)) &&
+      while (!(mbar_try_wait(&bars->w_full, (w - 1) & 1) && mbar_try_wait(&bars->u0_full, (u - 1) & 1) && mbar_try_wait(&bars->k_full[(k - 1) & 1], ((k - 1) >> 1) & 1) &&
+               (k < 2 || mbar_try_wait(&bars->k_full[k & 1], ((k - 2) >> 1) & 1))) &&
              globaltimer_ns() - begin < WAIT_LIMIT_NS) {}
     }
   } else {
@@ -516,7 +522,8 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     auto put_state = [&]() {
       if (r < p.dim) {
         uint8_t* d = sS + (r >> 6) * SPANEL + vc * 128 + (r & 7) * 2;
-        const int piece = (r & 63) >> 3;
+        int piece = (r & 63) >> 3;
+        asm volatile("" : "+r"(piece));                  // addresses are formed here, not kept for the whole loop
 #pragma unroll
         for (int v = 0; v < VC; ++v) {
           const __nv_bfloat16 hi = f2bf(S[v]);
@@ -529,6 +536,26 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->s_ready);
+    };
+    // v += f (head's columns + remainder's columns) of this thread's row
+    auto add_columns = [&](uint32_t at, float f, float (&v)[16]) {
+      uint32_t x[16];
+      tmem_ld_32x16(at + lane_addr + vc, x);
+      if constexpr (VB < 64) {
+        uint32_t y[16];
+        tmem_ld_32x16(at + lane_addr + VB + vc, y);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] += f * (__uint_as_float(x[i]) + __uint_as_float(y[i]));
+      } else {                                           // one after the other: registers
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] += f * __uint_as_float(x[i]);
+        tmem_ld_32x16(at + lane_addr + VB + vc, x);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] += f * __uint_as_float(x[i]);
+      }
     };
     put_state();
     int4 ck;
@@ -548,52 +575,42 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
       bool ok = wait(&bars->u0_full, ph, ERR_WAIT_TMA_FULL) && wait(&bars->x_done, ph, ERR_WAIT_TMEM_FULL);
       if (!__all_sync(0xffffffffu, ok)) break;
       tc_fence_after();
-#pragma unroll 1
-      for (int b = vc; b < vc + VC; b += 16) {
-        uint32_t x[16], y[16];
-        float u[16];
-        tmem_ld_32x16(tx + lane_addr + b, x);
-        tmem_ld_32x16(tx + lane_addr + VB + b, y);
+      float u[16];
+      int r7 = r & 7;
+      asm volatile("" : "+r"(r7));
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          float z[4];
-          ld4(reinterpret_cast<const float*>(sU0 + (b >> 5) * MC_PANEL + r * 128 + (((((b & 31) >> 2) + q) ^ (r & 7)) << 4)), z);
+      for (int q = 0; q < 4; ++q) {
+        float z[4];
+        ld4(reinterpret_cast<const float*>(sU0 + (vc >> 5) * MC_PANEL + r * 128 + (((((vc & 31) >> 2) + q) ^ r7) << 4)), z);
 #pragma unroll
-          for (int i = 0; i < 4; ++i) u[4 * q + i] = z[i];
-        }
-        tmem_ld_wait();
+        for (int i = 0; i < 4; ++i) u[4 * q + i] = z[i];
+      }
+      add_columns(tx, -1.f, u);
 #pragma unroll
-        for (int i = 0; i < 16; ++i) u[i] -= __uint_as_float(x[i]) + __uint_as_float(y[i]);
+      for (int q = 0; q < 2; ++q) {                      // pieces of eight values of the token's row
+        uint32_t hi[4], lo[4];
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {                    // pieces of eight values of the token's row
-          uint32_t hi[4], lo[4];
-#pragma unroll
-          for (int i = 0; i < 4; ++i) split_pack(u[8 * q + 2 * i] * f, u[8 * q + 2 * i + 1] * f, hi[i], lo[i]);
-          const int ch = b + 8 * q, cl = VB + ch;
-          *reinterpret_cast<uint4*>(sU + (ch >> 6) * MC_PANEL + r * 128 + ((((ch & 63) >> 3) ^ (r & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(sU + (cl >> 6) * MC_PANEL + r * 128 + ((((cl & 63) >> 3) ^ (r & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-          if (dst && v0 + ch < p.vdim)
-            *reinterpret_cast<uint4*>(dst + ch) = make_uint4(pack_bf16x2(u[8 * q], u[8 * q + 1]), pack_bf16x2(u[8 * q + 2], u[8 * q + 3]),
-                                                             pack_bf16x2(u[8 * q + 4], u[8 * q + 5]), pack_bf16x2(u[8 * q + 6], u[8 * q + 7]));
-        }
+        for (int i = 0; i < 4; ++i) split_pack(u[8 * q + 2 * i] * f, u[8 * q + 2 * i + 1] * f, hi[i], lo[i]);
+        const int ch = vc + 8 * q, cl = VB + ch;
+        *reinterpret_cast<uint4*>(sU + (ch >> 6) * MC_PANEL + r * 128 + ((((ch & 63) >> 3) ^ r7) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(sU + (cl >> 6) * MC_PANEL + r * 128 + ((((cl & 63) >> 3) ^ r7) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->u_ready);
+#pragma unroll
+      for (int q = 0; q < 2; ++q)
+        if (dst && v0 + vc + 8 * q < p.vdim)
+          *reinterpret_cast<uint4*>(dst + vc + 8 * q) = make_uint4(pack_bf16x2(u[8 * q], u[8 * q + 1]), pack_bf16x2(u[8 * q + 2], u[8 * q + 3]),
+                                                                   pack_bf16x2(u[8 * q + 4], u[8 * q + 5]), pack_bf16x2(u[8 * q + 6], u[8 * q + 7]));
       if (c + 1 < nc) chunk_info(c + 1);
       ok = wait(&bars->d_done, ph, ERR_WAIT_TMEM_FULL);
       if (!__all_sync(0xffffffffu, ok)) break;
       tc_fence_after();
 #pragma unroll
-      for (int b = 0; b < VC; b += 16) {
-        uint32_t x[16], y[16];
-        tmem_ld_32x16(td + lane_addr + vc + b, x);
-        tmem_ld_32x16(td + lane_addr + VB + vc + b, y);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) S[b + i] = a * S[b + i] + (__uint_as_float(x[i]) + __uint_as_float(y[i]));
-      }
+      for (int i = 0; i < 16; ++i) S[i] *= a;
+      add_columns(td, 1.f, S);
       if (c + 1 < nc) {
         ok = wait(&bars->s_free, ph, ERR_WAIT_TMEM_FULL);
         if (!__all_sync(0xffffffffu, ok)) break;
@@ -615,7 +632,7 @@ delta_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 }
 
 static int dc_smem_chunk(int pk, int pv) { return 1024 + 1024 + (pk > pv ? pk : pv) * MC_PANEL + (MC_C * DC_PITCH + 6 * MC_C) * 4; }
-static int dc_smem_state(int pk, int vb) { return 1024 + 1024 + (2 * pk + 2 + (2 * vb + 63) / 64 + ds_groups(vb)) * MC_PANEL + pk * 2 * vb * 128; }
+static int dc_smem_state(int pk, int vb) { return 1024 + 1024 + (2 * pk + 4 + (2 * vb + 63) / 64 + ds_u0_tiles(vb)) * MC_PANEL + pk * 2 * vb * 128; }
 
 struct DeltaMaps { CUtensorMap k, v, wh, wl, u0, sh, sl; };
 

@@ -141,9 +141,9 @@ qkv_prep_kernel(const TI* in, T* q, const TF* __restrict__ first, float* __restr
   }
 }
 
-// LANES lanes per (token, head of q, k or v): one pass for the sum of squares, which a rotation leaves alone, and one for the result.
-// q may lie in the projection row itself.
-template <typename TI, typename T, int W, int LANES>
+// LANES lanes per (token, head of q, k or v): one pass for the sum of squares, which a rotation leaves alone, and one for the result (ONE:
+// a head is at most one unit per lane and is read once).  q may lie in the projection row itself.
+template <typename TI, typename T, int W, int LANES, bool ONE>
 __global__ void __launch_bounds__(128)
 qkv_heads_kernel(const TI* in, T* q, T* __restrict__ cache, T* __restrict__ stream, const QkvRow P, int total) {
   pdl_trigger();
@@ -165,11 +165,29 @@ qkv_heads_kernel(const TI* in, T* q, T* __restrict__ cache, T* __restrict__ stre
     }
     return a;
   };
+  const int half = kind == 2 ? 0 : P.rot >> 1, pairs = half / W, units = pairs + (n - 2 * half) / W;
+  const float* ct = P.cosT + static_cast<size_t>(p) * half;
+  const float* st = P.sinT + static_cast<size_t>(p) * half;
+  auto first = [&](int c) { return c < pairs ? c * W : 2 * half + (c - pairs) * W; };
   float ss = 0.f;
-  for (int i = lane * W; i < n; i += LANES * W) {
-    const Pack<W> a = load(i);
+  Pack<W> one_a, one_b;
+  if constexpr (ONE) {
+    if (lane < units) {
+      one_a = load(first(lane));
 #pragma unroll
-    for (int j = 0; j < W; ++j) ss += a.v[j] * a.v[j];
+      for (int j = 0; j < W; ++j) ss += one_a.v[j] * one_a.v[j];
+      if (lane < pairs) {
+        one_b = load(first(lane) + half);
+#pragma unroll
+        for (int j = 0; j < W; ++j) ss += one_b.v[j] * one_b.v[j];
+      }
+    }
+  } else {
+    for (int i = lane * W; i < n; i += LANES * W) {
+      const Pack<W> a = load(i);
+#pragma unroll
+      for (int j = 0; j < W; ++j) ss += a.v[j] * a.v[j];
+    }
   }
 #pragma unroll
   for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -183,16 +201,13 @@ qkv_heads_kernel(const TI* in, T* q, T* __restrict__ cache, T* __restrict__ stre
     if (T* kc = ring_row(P, cache, t, p)) dst[0] = kc + off;
     if (stream) dst[1] = stream + static_cast<size_t>(P.sidx[t]) * P.ld_kv + off;
   }
-  const int half = kind == 2 ? 0 : P.rot >> 1, pairs = half / W, units = pairs + (n - 2 * half) / W;
-  const float* ct = P.cosT + static_cast<size_t>(p) * half;
-  const float* st = P.sinT + static_cast<size_t>(p) * half;
   for (int c = lane; c < units; c += LANES) {
-    const int i0 = c < pairs ? c * W : 2 * half + (c - pairs) * W, i1 = i0 + half;
-    Pack<W> a = load(i0), b;
+    const int i0 = first(c), i1 = i0 + half;
+    Pack<W> a = ONE ? one_a : load(i0), b;
 #pragma unroll
     for (int j = 0; j < W; ++j) a.v[j] *= f;
     if (c < pairs) {
-      b = load(i1);
+      b = ONE ? one_b : load(i1);
       const Pack<W> cs = ldw<W>(ct + i0), sn = ldw<W>(st + i0);
 #pragma unroll
       for (int j = 0; j < W; ++j) {
@@ -292,9 +307,9 @@ B200_API int b200_qkv_heads(const void* in, void* q, void* cache, void* stream_b
                          reinterpret_cast<uintptr_t>(P.cosT) | reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.bias);
   const bool vec = !(addr & 15) && !((P.dim | (P.rot >> 1) | P.vdim | P.ld_in | P.off_k | P.off_v | P.ld_q | P.ld_kv | P.kv_v) & 7);
   const int n = P.dim > P.vdim ? P.dim : P.vdim;
-#define GO2(TI, T_, W, LN) \
-  launch_k(qkv_heads_kernel<TI, T_, W, LN>, dim3(static_cast<unsigned>((total + 128 / LN - 1) / (128 / LN))), dim3(128), 0, STREAM, (const TI*)in, (T_*)q, (T_*)cache, (T_*)stream_buf, P, static_cast<int>(total))
-#define GO(TI, T_) { if (!vec) GO2(TI, T_, 1, 32); else if (n <= 64) GO2(TI, T_, 8, 8); else if (n <= 128) GO2(TI, T_, 8, 16); else GO2(TI, T_, 8, 32); }
+#define GO2(TI, T_, W, LN, ONE) \
+  launch_k(qkv_heads_kernel<TI, T_, W, LN, ONE>, dim3(static_cast<unsigned>((total + 128 / LN - 1) / (128 / LN))), dim3(128), 0, STREAM, (const TI*)in, (T_*)q, (T_*)cache, (T_*)stream_buf, P, static_cast<int>(total))
+#define GO(TI, T_) { if (!vec) GO2(TI, T_, 1, 32, false); else if (n <= 64) GO2(TI, T_, 8, 8, true); else if (n <= 128) GO2(TI, T_, 8, 16, true); else if (n <= 256) GO2(TI, T_, 8, 32, true); else GO2(TI, T_, 8, 32, false); }
   if (f32) GO(float, float)
   else if (in_f32) GO(float, bf16_t)
   else GO(bf16_t, bf16_t)
