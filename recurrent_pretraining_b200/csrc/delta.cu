@@ -11,7 +11,7 @@
 namespace b200 {
 
 // ------------------------------------------------------------------------------------------------ short convolution
-constexpr int SC_CHUNK = 128;                     // tokens per CTA
+constexpr int SC_CHUNK = 128, SC_PART = 64;         // tokens per chunk of the table, per CTA
 
 struct ConvArgs {
   int ch, taps, ld_in, ld_out;                    // channels: a multiple of eight
@@ -41,15 +41,17 @@ template <> struct Raw8<__nv_bfloat16> {
   }
 };
 
-// 32 groups of eight channels x 8 runs of 16 tokens, eight tokens on their way at a time.  The CTA of a portion's first chunk is the only one that reads the ring, so it
+// 32 groups of eight channels x 8 runs of eight tokens, which are on their way at a time.  The CTA of a portion's first chunk is the only one that reads the ring, so it
 // may write it afterwards.  TAPS: taps kept in registers (0: any number, inputs read again).
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
 short_conv_kernel(const T* __restrict__ in, T* __restrict__ out, T* __restrict__ ring, const ConvArgs A) {
   const int c = (blockIdx.x * 32 + (threadIdx.x & 31)) * 8, ty = threadIdx.x >> 5;
-  const int4 ck = A.chunks[blockIdx.y];
+  const int chunk = blockIdx.y / (SC_CHUNK / SC_PART), skip = blockIdx.y % (SC_CHUNK / SC_PART) * SC_PART;
+  const int4 ck = A.chunks[chunk];
   const int4 sq = A.seqs[ck.z];
-  const int t0 = ck.x, n = ck.y, i0 = (static_cast<int>(blockIdx.y) - sq.x) * SC_CHUNK;      // i0: index inside the portion
+  const int t0 = ck.x + skip, n = min(SC_PART, ck.y - skip), i0 = (chunk - sq.x) * SC_CHUNK + skip;      // i0: index inside the portion
+  if (n <= 0) return;
   const int taps = TAPS ? TAPS : A.taps;
   const bool live = c < A.ch;
   T* rg = ring + static_cast<size_t>(sq.z) * taps * A.ch + c;
@@ -64,37 +66,35 @@ short_conv_kernel(const T* __restrict__ in, T* __restrict__ out, T* __restrict__
       for (int j = 0; j < 8; ++j) v[j] = 0.f;
     }
   };
-  const int k0 = ty * 16, k1 = min(n, k0 + 16);
+  const int k0 = ty * 8, k1 = min(n, k0 + 8);
   if (live && k0 < k1) {
     if constexpr (TAPS > 0) {
       float w[TAPS][8], x[TAPS][8];                             // x[j]: input of j tokens ago
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) ld8(A.w + static_cast<size_t>(TAPS - 1 - j) * A.ch + c, w[j]);
+      Raw8<T> raw[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+        if (k0 + k < k1) raw[k].load(in + static_cast<size_t>(t0 + k0 + k) * A.ld_in + c);
 #pragma unroll
       for (int j = 1; j < TAPS; ++j) input(k0 - j, x[j - 1]);
-      for (int b = k0; b < k1; b += 8) {
-        Raw8<T> raw[8];
 #pragma unroll
-        for (int k = 0; k < 8; ++k)
-          if (b + k < k1) raw[k].load(in + static_cast<size_t>(t0 + b + k) * A.ld_in + c);
+      for (int k = 0; k < 8; ++k) {
+        if (k0 + k >= k1) break;
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          if (b + k >= k1) break;
+        for (int j = TAPS - 1; j > 0; --j)
 #pragma unroll
-          for (int j = TAPS - 1; j > 0; --j)
+          for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+        raw[k].get(x[0]);
+        float v[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
-          raw[k].get(x[0]);
-          float v[8];
+        for (int e = 0; e < 8; ++e) {
+          float s = 0.f;
 #pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            float s = 0.f;
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) s += w[j][e] * x[j][e];
-            v[e] = sizeof(T) == 2 ? __fdividef(s, 1.f + __expf(-s)) : silu_f(s);
-          }
-          st8(out + static_cast<size_t>(t0 + b + k) * A.ld_out + c, v);
+          for (int j = 0; j < TAPS; ++j) s += w[j][e] * x[j][e];
+          v[e] = sizeof(T) == 2 ? __fdividef(s, 1.f + __expf(-s)) : silu_f(s);
         }
+        st8(out + static_cast<size_t>(t0 + k0 + k) * A.ld_out + c, v);
       }
     } else {
       for (int k = k0; k < k1; ++k) {
@@ -112,7 +112,7 @@ short_conv_kernel(const T* __restrict__ in, T* __restrict__ out, T* __restrict__
       }
     }
   }
-  if (static_cast<int>(blockIdx.y) != sq.x) return;
+  if (i0 != 0) return;
   __syncthreads();                                              // the ring has been read
   if (!live) return;
   const int4 last = A.chunks[sq.x + sq.y - 1];
@@ -143,10 +143,14 @@ struct DeltaArgs {
   float* state;
 };
 
+__device__ __forceinline__ void cp_async16_zfill(uint32_t dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
 // CTA per (head, sequence): warps over the key rows, float4 groups of value columns over the lanes.  R: float4 of the state per thread,
-// held in registers; 0: the state stays in memory.
+// held in registers or (RAW) in shared memory of its own, which leaves room for a third CTA; 0: the state stays in memory.
 template <typename TI, typename T, bool RAW, int R>
-__global__ void __launch_bounds__(256, R ? 2 : 3)
+__global__ void __launch_bounds__(256, R && !RAW ? 2 : 3)
 delta_scan_kernel(const TI* __restrict__ in, const TI* __restrict__ gate, T* __restrict__ ring, T* __restrict__ out, const DeltaArgs M) {
   pdl_trigger();
   pdl_wait();
@@ -173,8 +177,20 @@ delta_scan_kernel(const TI* __restrict__ in, const TI* __restrict__ gate, T* __r
   const int rpw = 32 / cl, sub = lane / cl, col0 = 4 * (lane % cl), rstep = 8 * rpw, r0 = warp * rpw + sub;
   const int nu = (dim + rstep - 1) / rstep, nc = (ldv + 4 * cl - 1) / (4 * cl);      // row steps, column blocks
   const bool fresh = start == 0;
-  float4 S[R ? R : 1];
-  if constexpr (R > 0) {
+  constexpr bool STAGED = RAW && R > 0;
+  float4 S[R && !STAGED ? R : 1];
+  float4* own = reinterpret_cast<float4*>(red + 32) + tid;      // STAGED: piece e of this thread at 256 e
+  if constexpr (STAGED) {
+    int u = 0, cb = 0;
+#pragma unroll
+    for (int e = 0; e < R; ++e) {
+      const int d = r0 + u * rstep, c = cb * 4 * cl + col0;
+      const bool on = !fresh && cb < nc && d < dim && c < ldv;
+      cp_async16_zfill(smem_u32(own + 256 * e), on ? gstate + static_cast<size_t>(d) * ldv + c : gstate, on);
+      if (++u == nu) { u = 0; ++cb; }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  } else if constexpr (R > 0) {
     int u = 0, cb = 0;
 #pragma unroll
     for (int e = 0; e < R; ++e) {
@@ -276,13 +292,18 @@ delta_scan_kernel(const TI* __restrict__ in, const TI* __restrict__ gate, T* __r
       a.x += k * s.x; a.y += k * s.y; a.z += k * s.z; a.w += k * s.w;
       b.x += q * s.x; b.y += q * s.y; b.z += q * s.z; b.w += q * s.w;
     };
+    auto piece = [&](int e) -> float4 {
+      if constexpr (STAGED) return own[256 * e];
+      else return S[e];
+    };
     if constexpr (R > 0) {
+      if constexpr (STAGED) asm volatile("cp.async.wait_group 0;" ::: "memory");   // a thread reads what it has asked for itself
       int u = 0, cb = 0;
 #pragma unroll
       for (int e = 0; e < R; ++e) {
         if (cb < nc) {
           const int d = r0 + u * rstep;
-          if (d < dim) gather(S[e], d);
+          if (d < dim) gather(piece(e), d);
           if (++u == nu) {
             flush(cb, a, b);
             a = b = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -329,8 +350,9 @@ delta_scan_kernel(const TI* __restrict__ in, const TI* __restrict__ gate, T* __r
       for (int e = 0; e < R; ++e) {
         const int d = r0 + u * rstep, c = cb * 4 * cl + col0;
         if (cb < nc && d < dim && c < ldv) {
-          S[e] = update(S[e], d, c);
-          if (j + 1 == n) *reinterpret_cast<float4*>(gstate + static_cast<size_t>(d) * ldv + c) = S[e];
+          const float4 next = update(piece(e), d, c);
+          if constexpr (!STAGED) S[e] = next;
+          if (j + 1 == n) *reinterpret_cast<float4*>(gstate + static_cast<size_t>(d) * ldv + c) = next;
         }
         if (++u == nu) { u = 0; ++cb; }
       }
@@ -357,9 +379,9 @@ typedef __nv_bfloat16 bf16_t;
 // in: projection rows, out: activated rows, ring: [rows, taps, ch]; all of one storage type.
 B200_API int b200_short_conv(const void* in, void* out, void* ring, const ConvArgs* Ap, int n_chunks, int f32, void* stream) {
   const ConvArgs A = *Ap;
-  if (n_chunks <= 0 || n_chunks > 65535 || A.ch <= 0 || ((A.ch | A.ld_in | A.ld_out) & 7) || A.taps < 1 || A.taps > SC_CHUNK || !A.w || !A.chunks || !A.seqs ||
+  if (n_chunks <= 0 || n_chunks > 32767 || A.ch <= 0 || ((A.ch | A.ld_in | A.ld_out) & 7) || A.taps < 1 || A.taps > SC_PART || !A.w || !A.chunks || !A.seqs ||
       ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(A.w)) & 15)) return -1;
-  const dim3 grid((A.ch / 8 + 31) / 32, n_chunks);
+  const dim3 grid((A.ch / 8 + 31) / 32, n_chunks * (SC_CHUNK / SC_PART));
 #define GO2(T_, N) short_conv_kernel<T_, N><<<grid, 256, 0, STREAM>>>((const T_*)in, (T_*)out, (T_*)ring, A)
 #define GO(T_)                        \
   switch (A.taps) {                   \
@@ -388,9 +410,11 @@ B200_API int b200_delta_scan(const void* in, const void* gate, void* ring, void*
   const int rstep = 8 * (32 / cl), held = ((M.dim + rstep - 1) / rstep) * ((M.ldv + 4 * cl - 1) / (4 * cl));
 #define GO2(TI, T_, RAW, R)                                                                                            \
   {                                                                                                                    \
-    if (smem > 48 * 1024 && cudaFuncSetAttribute(delta_scan_kernel<TI, T_, RAW, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                                 static_cast<int>(smem)) != cudaSuccess) return -3;                     \
-    launch_k(delta_scan_kernel<TI, T_, RAW, R>, dim3(M.H, n), dim3(256), smem, STREAM, (const TI*)in, (const TI*)gate, (T_*)ring, (T_*)out, M); \
+    const size_t bytes = smem + (RAW ? R * 4096 : 0);                                                                   \
+    if (bytes > 220 * 1024) return -1;                                                                                  \
+    if (bytes > 48 * 1024 && cudaFuncSetAttribute(delta_scan_kernel<TI, T_, RAW, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                  static_cast<int>(bytes)) != cudaSuccess) return -3;                   \
+    launch_k(delta_scan_kernel<TI, T_, RAW, R>, dim3(M.H, n), dim3(256), bytes, STREAM, (const TI*)in, (const TI*)gate, (T_*)ring, (T_*)out, M); \
   }
 #define GO(TI, T_, RAW) { if (held <= 4) GO2(TI, T_, RAW, 4) else if (held <= 16) GO2(TI, T_, RAW, 16) else GO2(TI, T_, RAW, 0) }
   if (raw) {

@@ -113,7 +113,8 @@ __device__ __forceinline__ void head_entries8(const TI* x, int i, const float* b
 }
 
 // NV: 16-column steps of the values that the accumulators hold.
-template <typename TI, int NV, int STAGES, bool RING>
+// HEADS (with RING): kept positions, biases, heads normed by themselves.
+template <typename TI, int NV, int STAGES, bool RING, bool HEADS>
 __global__ void __launch_bounds__(128)
 gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   pdl_trigger();
@@ -125,13 +126,13 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const int g = blockIdx.y / chunks, h0 = g * group + (blockIdx.y % chunks) * 16, nh = min(16, (g + 1) * group - h0);
   const int pos = P.pos[b];
   const int key_first = RING ? (P.chunked ? pos - pos % P.size : max(0, pos - P.size + 1)) : 0;
-  const int kept = RING ? min(P.keep, key_first) : 0;                  // keys are counted: kept ones in front of the window, then the window
+  const int keep = HEADS ? P.keep : 0, kept = HEADS ? min(keep, key_first) : 0;                  // keys are counted: kept ones in front of the window, then the window
   const int newest = kept + pos - key_first, nkeys = newest + 1;
-  const int slot0 = RING ? ring_slot(key_first, P.cap, P.keep) - kept : 0;
+  const int slot0 = RING ? ring_slot(key_first, P.cap, keep) - kept : 0;
   auto slot_of = [&](int j) {
-    if (RING && j < kept) return j;
+    if (HEADS && j < kept) return j;
     int s = slot0 + j;
-    if (RING && s >= P.cap) s -= P.cap - P.keep;
+    if (RING && s >= P.cap) s -= P.cap - keep;
     return s;
   };
   const int tiles = (nkeys + GD_KEYS - 1) / GD_KEYS, per = (tiles + P.splits - 1) / P.splits;
@@ -158,15 +159,23 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const int kpp = 32 / lpk, lj = lane / lpk, lc = lane % lpk;          // keys per pass, this lane's key and first piece
   auto request = [&](int tile, int st) {
     const uint32_t s = smem_u32(ring + st * stage_bytes);
-    const int last = max(newest - 1, 0);                               // keys past the newest repeat one that exists; they are masked
+    const int last = max(newest - 1, 0), j0 = tile * GD_KEYS;          // keys past the newest repeat one that exists; they are masked
+    const bool plain = j0 + GD_KEYS - 1 <= last && slot_of(j0 + GD_KEYS - 1) - slot_of(j0) == GD_KEYS - 1 && (!HEADS || j0 >= kept || j0 + GD_KEYS <= kept);
+    const __nv_bfloat16* row0 = base + static_cast<size_t>(slot_of(min(j0, last)) + lj) * P.ld_kv;
     for (int c = lc; c < ch; c += lpk) {
       const bool isk = c < kch;
-      const __nv_bfloat16* src = base + (isk ? g * P.dim + 8 * c : P.kv_v + g * P.vdim + 8 * (c - kch));
+      const int at = isk ? g * P.dim + 8 * c : P.kv_v + g * P.vdim + 8 * (c - kch);
       const uint32_t dst = s + (isk ? 16 * c : GD_KEYS * kp + 16 * (c - kch));
       const int pitch = isk ? kp : vp;
+      if (plain) {                                                     // neighbouring slots
+        const __nv_bfloat16* src = row0 + at;
+        const size_t step = static_cast<size_t>(kpp) * P.ld_kv;
 #pragma unroll 8
-      for (int j = lj; j < GD_KEYS; j += kpp)
-        cp_async16(dst + j * pitch, src + static_cast<size_t>(slot_of(min(tile * GD_KEYS + j, last))) * P.ld_kv);
+        for (int j = lj; j < GD_KEYS; j += kpp, src += step) cp_async16(dst + j * pitch, src);
+      } else {
+#pragma unroll 4
+        for (int j = lj; j < GD_KEYS; j += kpp) cp_async16(dst + j * pitch, base + at + static_cast<size_t>(slot_of(min(j0 + j, last))) * P.ld_kv);
+      }
     }
   };
   const int first = tile0 + warp;
@@ -180,7 +189,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   const float *cos_t = nullptr, *sin_t = nullptr;
   __shared__ float rh[18];                                             // factors of the heads' own norms: q heads, then k and v
   if constexpr (RING) {
-    if (P.head_norm) {                                                 // a rotation leaves the sum of squares alone
+    if (HEADS && P.head_norm) {                                                 // a rotation leaves the sum of squares alone
       for (int i = warp; i < nh + 2; i += GD_WARPS) {
         const int n = i <= nh ? P.dim : P.vdim, col = i < nh ? (h0 + i) * P.dim : i == nh ? P.off_k + g * P.dim : P.off_v + g * P.vdim;
         float t = 0.f;
@@ -230,7 +239,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
       float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
       if (hh < nh && c < P.dim) {
         const int at = (h0 + hh) * P.dim;
-        head_entries8(r + at, c, P.in_bias ? P.in_bias + at : nullptr, P.q_norm ? P.q_norm + at : nullptr, P.head_norm ? rh[hh] : rq, P.rot, cos_t, sin_t, v);
+        head_entries8(r + at, c, HEADS && P.in_bias ? P.in_bias + at : nullptr, P.q_norm ? P.q_norm + at : nullptr, HEADS && P.head_norm ? rh[hh] : rq, P.rot, cos_t, sin_t, v);
       }
       st8(reinterpret_cast<__nv_bfloat16*>(sq) + hh * (kp / 2) + c, v);
     }
@@ -266,7 +275,7 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
   }
   const bool capped = RING && P.softcap > 0.f;
   const float cap_log2 = P.softcap * 1.4426950408889634f, cap_exp = capped ? 2.f * rowmul / P.softcap : 0.f;
-  const bool bounded = RING && (capped ? cap_log2 <= 80.f : P.bound > 0.f && P.bound * 1.4426950408889634f <= 80.f);      // weights lie in 2^(-80 .. 80): no running maximum
+  const bool bounded = RING && (capped ? cap_log2 <= 80.f : HEADS && P.bound > 0.f && P.bound * 1.4426950408889634f <= 80.f);      // weights lie in 2^(-80 .. 80): no running maximum
   const float m_start = bounded ? 0.f : -INFINITY;
   float m[2] = {m_start, m_start}, l[2] = {0.f, 0.f};
   float o[NV][2][4];
@@ -300,10 +309,10 @@ gqa_decode_kernel(const TI* __restrict__ in, const GqaDecode P) {
           const int cc = isk ? c : c - P.dim, vc = g * P.vdim + cc;
           float f[8];
           if (isk) {
-            head_entries8(r + P.off_k + g * P.dim, cc, P.in_bias ? P.in_bias + P.off_k + g * P.dim : nullptr, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk,
+            head_entries8(r + P.off_k + g * P.dim, cc, HEADS && P.in_bias ? P.in_bias + P.off_k + g * P.dim : nullptr, P.k_norm ? P.k_norm + g * P.dim : nullptr, rk,
                           P.rot, cos_t, sin_t, f);
           } else {
-            head_entries8(r + P.off_v + g * P.vdim, cc, P.in_bias ? P.in_bias + P.off_v + g * P.vdim : nullptr, nullptr, P.head_norm ? rh[nh + 1] : 1.f, 0,
+            head_entries8(r + P.off_v + g * P.vdim, cc, HEADS && P.in_bias ? P.in_bias + P.off_v + g * P.vdim : nullptr, nullptr, HEADS && P.head_norm ? rh[nh + 1] : 1.f, 0,
                           nullptr, nullptr, f);
             if (P.first_out) st8(P.first_out + static_cast<size_t>(b) * P.ld_fout + vc, f);
             if (P.lam) {
@@ -492,15 +501,15 @@ B200_API int b200_gqa_decode_per_sm(int dim, int vdim) {
   return n < 1 ? 1 : n > 4 ? 4 : n;
 }
 
-template <bool RING>
+template <bool RING, bool HEADS>
 static int gqa_decode_launch(const void* in, const GqaDecode& P, int B, int in_f32, cudaStream_t st) {
   const int chunks = (P.H / P.G + 15) / 16;
   const dim3 grid(P.splits, P.G * chunks, B);
 #define GO2(TI, NV, ST)                                                                                                \
   {                                                                                                                    \
     const int smem = gd_smem<ST>(P.dim, P.vdim);                                                                        \
-    if (cudaFuncSetAttribute(gqa_decode_kernel<TI, NV, ST, RING>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3; \
-    launch_k(gqa_decode_kernel<TI, NV, ST, RING>, grid, dim3(128), smem, st, (const TI*)in, P);                         \
+    if (cudaFuncSetAttribute(gqa_decode_kernel<TI, NV, ST, RING, HEADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3; \
+    launch_k(gqa_decode_kernel<TI, NV, ST, RING, HEADS>, grid, dim3(128), smem, st, (const TI*)in, P);                         \
   }
 #define GO(TI)                                          \
   {                                                     \
@@ -522,7 +531,7 @@ static bool gqa_decode_ok(const GqaDecode& P, int B) {
 
 B200_API int b200_gqa_decode(const void* in, const GqaDecode* Pp, int B, int in_f32, void* stream) {
   if (!gqa_decode_ok(*Pp, B) || Pp->bias_len <= 0) return -1;
-  return gqa_decode_launch<false>(in, *Pp, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
+  return gqa_decode_launch<false, false>(in, *Pp, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
 }
 
 // The RING form; `out` is written with a single split, the partials otherwise.
@@ -534,5 +543,6 @@ B200_API int b200_ring_decode(const void* in, const GqaDecode* Pp, int B, int in
       ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(P.q_norm) | reinterpret_cast<uintptr_t>(P.k_norm) | reinterpret_cast<uintptr_t>(P.cosT) |
         reinterpret_cast<uintptr_t>(P.sinT) | reinterpret_cast<uintptr_t>(P.in_bias) | reinterpret_cast<uintptr_t>(P.first) | reinterpret_cast<uintptr_t>(P.first_out)) & 15)) return -1;
   if (P.splits == 1 ? (!P.out || (P.ld_out & 7) || (reinterpret_cast<uintptr_t>(P.out) & 15)) : (P.out || !P.part_o || !P.part_ml)) return -1;
-  return gqa_decode_launch<true>(in, P, B, in_f32, reinterpret_cast<cudaStream_t>(stream));
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return P.keep || P.head_norm || P.in_bias ? gqa_decode_launch<true, true>(in, P, B, in_f32, st) : gqa_decode_launch<true, false>(in, P, B, in_f32, st);
 }

@@ -20,11 +20,13 @@
 // add a constant; the others (those near the diagonal) read the bias per element, lanes at consecutive distances.
 //
 // CAPPED: keys and values come from the step's key stream, there is neither a rotated part nor a gate.  A tile lies inside one chunk,
-// so a chunk is nothing but the first key of its tiles.  The first keys of a sequence may stay visible beside the window: their blocks
-// come in front of the window's when there is a gap between the two, and are the first of one range otherwise.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
+// so a chunk is nothing but the first key of its tiles.  Scores are cap tanh(score / cap): a polynomial on the FMA pipe as long as
 // every score of a warp's columns is well below the cap, exponential and reciprocal otherwise.
 //
-// BOUNDED: CAPPED with a cap that is not large, or with scores that are known to be small without one.  The softmax needs no running maximum and takes its columns as they come, and a query
+// KEPT: CAPPED with the first keys of a sequence visible beside the window: their blocks come in front of the window's when there is a gap
+// between the two, and are the first of one range otherwise.
+//
+// BOUNDED: CAPPED with a cap that is not large; SMALL: KEPT with scores that are small without a cap.  The softmax needs no running maximum and takes its columns as they come, and a query
 // row is shared by two threads: sixteen softmax warps, each with half of a block's columns and its weights over its own half of the
 // scores.
 #include <cuda.h>
@@ -66,8 +68,10 @@ struct LatentAttnParams {
   int keep;                     // keys of a sequence that stay visible beside the window
   float cap_poly[3], poly_max;  // capped log2 score = raw * polynomial(raw^2) for |raw| <= poly_max
 };
-enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2, BOUNDED = 3 };
-__host__ __device__ constexpr int la_softmax_warps(int kind) { return kind == BOUNDED ? 16 : 8; }
+enum AttnKind { LATENT = 0, BIAS = 1, CAPPED = 2, BOUNDED = 3, KEPT = 4, SMALL = 5 };
+__host__ __device__ constexpr bool la_bounded(int kind) { return kind == BOUNDED || kind == SMALL; }     // no running maximum
+__host__ __device__ constexpr bool la_keeps(int kind) { return kind == KEPT || kind == SMALL; }
+__host__ __device__ constexpr int la_softmax_warps(int kind) { return la_bounded(kind) ? 16 : 8; }
 __host__ __device__ constexpr int la_threads(int kind) { return 32 * (la_softmax_warps(kind) + 4); }
 // Columns in front of distance 0 and behind the last stored one (repeating the values there): a block's accesses need no clamps.
 constexpr int LA_BIAS_LEAD = 256, LA_BIAS_TAIL = 256;
@@ -151,7 +155,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
   int kstart = max(kbase, s0 - p.window + 1);
   // key blocks [jb, je) of both tiles: nkb blocks of kept keys, the others counted from kstart
   int nkb = 0;
-  if constexpr (KIND >= CAPPED) {
+  if constexpr (la_keeps(KIND)) {
     if (p.keep > 0) {
       nkb = (p.keep + BN - 1) / BN;
       if (kstart - kbase <= nkb * BN) {
@@ -160,13 +164,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
       }
     }
   }
-  const bool keeps = KIND >= CAPPED && p.keep > 0;
+  const bool keeps = la_keeps(KIND) && p.keep > 0;
   const int last_a = min(LA_BM, nrows) - 1, last_b = nrows - 1;
   const int je0 = nkb + (s0 + last_a - kstart) / BN + 1;
   const int jb1 = nrows > LA_BM && !keeps ? (max(kbase, s0 + LA_BM - p.window + 1) - kstart) / BN : 0;
   const int je1 = nrows > LA_BM ? nkb + (s0 + last_b - kstart) / BN + 1 : 0;
   const int nmax = max(je0, je1);
-  auto block_key = [&](int j) { return KIND >= CAPPED ? (j < nkb ? kbase + j * BN : kstart + (j - nkb) * BN) : kstart + j * BN; };   // first key of a block
+  auto block_key = [&](int j) { return la_keeps(KIND) ? (j < nkb ? kbase + j * BN : kstart + (j - nkb) * BN) : kstart + j * BN; };   // first key of a block
 
   auto load_q = [&](int x) {
     mbar_expect_tx(&bars->q_full[x], q_bytes);
@@ -352,15 +356,15 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         scale_log2 *= 1.f + p.temp_coef * logf(static_cast<float>((kstart + hi - kbase + 1) / p.temp_every + 1));
       btab = p.bias + static_cast<size_t>(h) * p.ld_bias + LA_BIAS_LEAD;
     }
-    float m = KIND == BOUNDED ? 0.f : -INFINITY, l = 0.f;
+    float m = la_bounded(KIND) ? 0.f : -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = jb; j < je && ok; ++j) {
       if (!mbar_wait(&bars->s_full[x], (j - jb) & 1, abort_flag, p.err, ERR_WAIT_ATTN)) { ok = false; break; }
       tc_fence_after();
-      if constexpr (KIND == BOUNDED) {        // 32 columns at a time: no maximum to wait for
+      if constexpr (la_bounded(KIND)) {       // 32 columns at a time: no maximum to wait for
         const bool edge = j < j_lo || j >= j_hi;
         const int off = block_key(j) - kstart, cmax = hi - off, cmin = max(kbase - kstart - off, cmax - p.window + 1);
-        const int ckeep = kbase + p.keep - kstart - off;            // columns in front of it are kept keys
+        const int ckeep = la_keeps(KIND) ? kbase + p.keep - kstart - off : 0;            // columns in front of it are kept keys
         float2 rs = make_float2(0.f, 0.f);
         constexpr int COLS = BN / SPLIT;
 #pragma unroll
@@ -379,8 +383,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
             for (int i = 0; i < 32; i += 2) {
               float2 y = cap(i);
               if constexpr (decltype(masked)::value) {
-                if ((c + i < cmin && c + i >= ckeep) || c + i > cmax) y.x = -INFINITY;
-                if ((c + i + 1 < cmin && c + i + 1 >= ckeep) || c + i + 1 > cmax) y.y = -INFINITY;
+                if ((c + i < cmin && (!la_keeps(KIND) || c + i >= ckeep)) || c + i > cmax) y.x = -INFINITY;
+                if ((c + i + 1 < cmin && (!la_keeps(KIND) || c + i + 1 >= ckeep)) || c + i + 1 > cmax) y.y = -INFINITY;
               }
               const float2 pr = make_float2(ex2_approx(y.x), ex2_approx(y.y));
               r2[(i >> 1) & 1] = fadd2(r2[(i >> 1) & 1], pr);
@@ -388,8 +392,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
             }
           };
           auto small = [&](int i) { return cap_small(make_float2(sv[i], sv[i + 1]), p); };
-          auto plain = [&](int i) { return fmul2(make_float2(sv[i], sv[i + 1]), make_float2(scale_log2, scale_log2)); };
-          if (!p.capped) {
+          if constexpr (KIND == SMALL) {
+            auto plain = [&](int i) { return fmul2(make_float2(sv[i], sv[i + 1]), make_float2(scale_log2, scale_log2)); };
             if (edge) weigh(plain, std::true_type());
             else weigh(plain, std::false_type());
           } else if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
@@ -416,7 +420,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
           for (int i = 0; i < 32; ++i) sv[c + i] = __uint_as_float(v[i]);
         }
         tmem_ld_wait();
-        if constexpr (KIND == CAPPED) {
+        if constexpr (KIND == CAPPED || KIND == KEPT) {
           if (p.capped) {
           if (__all_sync(0xffffffffu, max_abs(sv) <= p.poly_max)) {
 #pragma unroll
@@ -433,12 +437,12 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_consta
         }
         if (j < j_lo || j >= j_hi) {
           const int off = block_key(j) - kstart, cmax = hi - off, cmin = max(kbase - kstart - off, cmax - p.window + 1);
-          const int ckeep = KIND >= CAPPED ? kbase + p.keep - kstart - off : cmin;       // columns in front of it are kept keys
+          const int ckeep = la_keeps(KIND) ? kbase + p.keep - kstart - off : cmin;       // columns in front of it are kept keys
 #pragma unroll
           for (int i = 0; i < BN; ++i)
-            if ((i < cmin && (KIND < CAPPED || i >= ckeep)) || i > cmax) sv[i] = -INFINITY;
+            if ((i < cmin && (!la_keeps(KIND) || i >= ckeep)) || i > cmax) sv[i] = -INFINITY;
         }
-        float mul = KIND == CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
+        float mul = KIND >= CAPPED && p.capped ? 1.f : scale_log2, add = 0.f;      // log2 score = mul * sv + add
         if constexpr (KIND == BIAS) {
           const int d0 = s0 - kstart + x * LA_BM - j * BN, far = p.bias_len - 1;   // distance of the tile's first row to the block's first key
           const int dmin = d0 - (BN - 1), dmax = d0 + LA_BM - 1;
@@ -784,7 +788,8 @@ B200_API int b200_capped_attention(const void* q, const void* k, const void* v, 
   p.err = err;
   p.group = H / G; p.sink = sink;
   p.keep = keep;
-  bool bounded = softcap <= 0.f && bound > 0.f && bound * 1.4426950408889634f <= 80.f;
+  const bool small = softcap <= 0.f && bound > 0.f && bound * 1.4426950408889634f <= 80.f;
+  bool bounded = false;
   if (softcap > 0.f) {
     const double x = static_cast<double>(scale) / softcap, cap = softcap * 1.4426950408889634;
     p.capped = 1;
@@ -796,5 +801,7 @@ B200_API int b200_capped_attention(const void* q, const void* k, const void* v, 
     p.poly_max = x > 1e-6 && x < 1e6 ? static_cast<float>(TANH_RANGE / x) : -1.f;   // coefficients inside the range of fp32
   }
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (small) return dispatch_grouped<SMALL>(tm, p, plan, n_tiles, st);
+  if (keep > 0) return dispatch_grouped<KEPT>(tm, p, plan, n_tiles, st);
   return bounded ? dispatch_grouped<BOUNDED>(tm, p, plan, n_tiles, st) : dispatch_grouped<CAPPED>(tm, p, plan, n_tiles, st);
 }
